@@ -272,6 +272,24 @@ int32_t b2_model_config_from_json(const char* json, b2_model_config* out);
  * optional quantize-on-load (:97).  `prefix` is prepended to every key ("" for plain checkpoints). */
 int32_t b2_model_from_weights(b2_ctx* ctx, const b2_weights* w, const char* prefix, const b2_model_config* cfg,
                               const b2_quant_spec* quant /* nullable */, b2_model** out);
+/* ---- models by configuration -------------------------------------------------------------------------
+ * The registry of model families: the Llama / Qwen3 families are flat configurations (b2_model_config above); a layered
+ * family names itself in config.json's `architecture` and lists its layers (a token mixer and a feed-forward each). */
+int32_t b2_model_family_from_json(const char* json, char* out, int32_t cap);
+/* Builds the model config.json describes.  compute_f32 != 0: weights, activations, caches and logits in f32. */
+int32_t b2_model_from_json(b2_ctx* ctx, const b2_weights* w, const char* prefix, const char* json,
+                           const b2_quant_spec* quant /* nullable */, int32_t compute_f32, b2_model** out);
+/* ... from a folder with config.json and *.safetensors. */
+int32_t b2_model_open(b2_ctx* ctx, const char* dir, const b2_quant_spec* quant /* nullable */, int32_t compute_f32, b2_model** out);
+/* ... with random weights drawn on the device (benchmarks). */
+int32_t b2_model_synthetic_json(b2_ctx* ctx, const char* json, uint64_t seed, b2_model** out);
+/* 1 when the logits rows a step returns are f32 (f32 models and layered models), 0 for bf16. */
+int32_t b2_model_logits_f32(const b2_model* m);
+/* Bytes of recurrent state one sequence holds besides its pages (0: none). */
+int64_t b2_model_state_bytes(const b2_model* m);
+/* Diagnostics of a layered model: after every following step, out_host (caller-owned, room for layers x tokens x width
+ * floats) holds the residual stream behind every layer, [layers, tokens of the step, width].  NULL switches it off. */
+int32_t b2_model_capture_residual(b2_model* m, float* out_host, int64_t capacity_floats);
 /* Random-init model generated on the device from a counter-based recipe (benchmark / parity helper;
  * no counterpart in the reference). cfg->quant_bits selects dense / Q4 / Q8 projections. */
 int32_t b2_model_synthetic(b2_ctx* ctx, const b2_model_config* cfg, uint64_t seed, b2_model** out);
@@ -389,6 +407,11 @@ int32_t b2_cache_gather_f32(b2_cache* c, int32_t layer, float* k_host, float* v_
 int32_t b2_model_step(b2_model* m, const int32_t* ids_host, const int32_t* n_tokens, int32_t num_seqs, b2_cache** caches,
                       void* logits_host /* nullable; uint16_t (bf16) rows, float rows for an f32 model */,
                       int32_t* argmax_host /* nullable */);
+
+/* The same forward with the logits of listed positions: sequence i asks for n_want[i] of its new tokens, by their place
+ * (0 .. n_tokens[i]-1) in `want`, sequence after sequence; rows come back in that order.  n_want[i] may be 0. */
+int32_t b2_model_step_at(b2_model* m, const int32_t* ids_host, const int32_t* n_tokens, int32_t num_seqs, b2_cache** caches,
+                         const int32_t* n_want, const int32_t* want, void* logits_host, int32_t* argmax_host);
 
 /* FinishReason (src/decode/stream.rs:31-46). */
 enum { B2_FINISH_STOP_TOKEN = 0, B2_FINISH_MAX_TOKENS = 1, B2_FINISH_CANCELLED = 2, B2_FINISH_STOPPED = 3 };

@@ -3,6 +3,7 @@
     python -m mlx_llm_b200.build [--force] [--verbose]
 """
 import concurrent.futures as cf
+import fcntl
 import os
 import shutil
 import subprocess
@@ -51,8 +52,20 @@ def _compile(src, force, verbose):
     return obj, log if verbose else ""
 
 
+def up_to_date():
+    return os.path.exists(LIB) and os.path.getmtime(LIB) >= max(os.path.getmtime(p) for p in sources() + _headers())
+
+
 def build(force=False, verbose=False):
+    if not force and up_to_date():
+        return LIB
     os.makedirs(OBJ, exist_ok=True)
+    with open(os.path.join(OBJ, ".lock"), "w") as lock:  # one build at a time in a checkout
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return _build(force, verbose)
+
+
+def _build(force, verbose):
     srcs = sources()
     with cf.ThreadPoolExecutor(max_workers=min(8, len(srcs))) as ex:
         results = list(ex.map(lambda s: _compile(s, force, verbose), srcs))
@@ -61,10 +74,12 @@ def build(force=False, verbose=False):
         if log:
             print(log)
     if force or not os.path.exists(LIB) or any(os.path.getmtime(o) > os.path.getmtime(LIB) for o in objs):
-        cmd = [_nvcc(), "-shared", "-o", LIB] + objs + ["-lcudart", "-Xlinker", "-rpath,/usr/local/cuda/lib64"]
+        part = LIB + ".part"
+        cmd = [_nvcc(), "-shared", "-o", part] + objs + ["-lcudart", "-Xlinker", "-rpath,/usr/local/cuda/lib64"]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode != 0:
             raise RuntimeError(f"link failed:\n{r.stdout}\n{r.stderr}")
+        os.replace(part, LIB)
     return LIB
 
 

@@ -227,7 +227,7 @@ int32_t b2_profile_read(b2_ctx* ctx, b2_profile_t* out) {
 
 }  // extern "C"
 
-static const char* const kClassNames[8] = {"gemm", "attn_decode", "attn_prefill", "rope_kv", "elementwise", "meta_copies", "collective", "other"};
+static const char* const kClassNames[8] = {"gemm", "attn_decode", "attn_prefill", "rope_kv", "elementwise", "meta_copies", "collective", "recurrent"};
 
 void b2_prof_mark(b2_ctx* ctx, int cls) {
     if (ctx->nvtx) {  // one range per run of launches of a class; cls < 0 closes the step's last range

@@ -9,6 +9,7 @@
 
 #include "common.cuh"
 #include "kernels.h"
+#include "model_spec.h"
 
 // ---- Weights (src/primitives/weights.rs:17-96) -------------------------------------------------
 struct HostTensor {
@@ -111,6 +112,9 @@ struct b2_model {
     bool f32 = false;  // cfg.compute_f32: every weight pointer above then holds float, not bf16
     float *cos_f32 = nullptr, *sin_f32 = nullptr;  // f32 RoPE tables of the f32 path
     struct F32Work* w32 = nullptr;                 // its activations (engine_step_f32.cu)
+    // a model whose layers are described one by one (engine_layers.cu); cfg then holds the common dimensions only
+    struct LayeredModel* layered = nullptr;
+    bool logits_f32() const { return f32 || layered; }  // element type of the logits rows a step returns
     Workspace ws;
     cudaEvent_t ev0 = nullptr, ev1 = nullptr;
     // accumulated by every forward
@@ -130,6 +134,11 @@ struct RefBlockAllocator {
     int64_t shared() const;
 };
 
+// One paged array of a pool: page i lies at base + i * page_bytes.
+struct KvPlane {
+    uint8_t* base = nullptr;
+    size_t page_bytes = 0;
+};
 struct b2_pool {  // BlockPool (paged_kv_cache.rs:72-160) + bounded physical pages
     b2_ctx* ctx = nullptr;
     const b2_model* model = nullptr;
@@ -137,9 +146,15 @@ struct b2_pool {  // BlockPool (paged_kv_cache.rs:72-160) + bounded physical pag
     int64_t max_pages = 0;
     int max_seqs = 0, max_blocks = 0;
     int layers = 0, hkv = 0, hd = 0;
-    uint16_t* kv = nullptr;        // [layers][2][pages][hkv][block][hd], bf16 (f32 for an f32 model)
+    uint8_t* kv = nullptr;         // one allocation that holds every plane, bf16 (f32 for an f32 model)
     int esz = 2;                   // bytes per element
-    size_t page_elems = 0;         // hkv*block*hd
+    // K and V of every attention layer ([pages][hkv][block][hd] each), or the latent rows ([pages][block][row]) of a
+    // latent-attention layer; layers without a per-token cache have none
+    std::vector<KvPlane> planes;
+    std::vector<int> layer_plane;  // first plane of each layer, -1 for none
+    // recurrent state of layers that keep one: a fixed-size f32 record per block-table row
+    float* state = nullptr;
+    int64_t state_floats = 0;      // per row; 0 for a model without recurrent layers
     int32_t* block_tables = nullptr;  // device [max_seqs][max_blocks]
     std::vector<int32_t> free_pages;  // stack, back() is handed out next
     std::vector<int32_t> page_ref;
@@ -149,9 +164,10 @@ struct b2_pool {  // BlockPool (paged_kv_cache.rs:72-160) + bounded physical pag
     std::vector<int32_t> upd_slot, upd_index, upd_page;  // block-table updates not yet on the device
     int64_t live_caches = 0;
     uint64_t step_stamp = 0;  // number of the last forward over this pool (duplicate-cache check)
-    size_t page_bytes() const { return page_elems * (size_t)esz; }
-    uint16_t* k_layer(int l) const { return reinterpret_cast<uint16_t*>(reinterpret_cast<uint8_t*>(kv) + ((size_t)l * 2) * (size_t)max_pages * page_bytes()); }
-    uint16_t* v_layer(int l) const { return reinterpret_cast<uint16_t*>(reinterpret_cast<uint8_t*>(kv) + ((size_t)l * 2 + 1) * (size_t)max_pages * page_bytes()); }
+    uint16_t* k_layer(int l) const { return reinterpret_cast<uint16_t*>(planes[layer_plane[l]].base); }
+    uint16_t* v_layer(int l) const { return reinterpret_cast<uint16_t*>(planes[layer_plane[l] + 1].base); }
+    // copies one page of every plane on the context's stream
+    int32_t copy_page(int32_t from, int32_t to) const;
 };
 
 struct b2_cache {  // PagedKvCache (paged_kv_cache.rs:168-516)
@@ -159,6 +175,7 @@ struct b2_cache {  // PagedKvCache (paged_kv_cache.rs:168-516)
     int slot = -1;
     int len = 0;                     // KvCache::offset
     uint64_t step_stamp = 0;         // pool->step_stamp of the last forward this cache took part in
+    int state_len = 0;               // tokens the recurrent state has seen; differs from len only after an abandoned step
     std::vector<int32_t> pages;      // physical page of every started block (incl. the partial tail)
     std::vector<int64_t> block_ids;  // reference-view ids of the frozen (full) blocks
 };
@@ -171,6 +188,9 @@ struct SeqStep {
     // logits / greedy ids of EVERY new position, not only the last (CausalLm::decode_logits_all, llama.rs:372-392: the
     // verify forward of speculative decoding).  Only for a step of one sequence.
     bool all_positions = false;
+    // explicit list of new positions (0 .. n-1) whose logits are wanted, instead of the last one
+    const int32_t* want = nullptr;
+    int n_want = -1;  // -1: want_logits decides
 };
 // One forward over a ragged batch.  argmax_out[i] (per sequence that wants logits, in batch order)
 // and logits_out (rows in the same order: bf16, or f32 for an f32 model) are host pointers, nullable.
@@ -181,3 +201,26 @@ struct BatchMetaOut;
 int32_t b2_forward_f32(b2_model* m, b2_pool* pool, const BatchMetaOut& mo, const int32_t* seq_slot_dev, const int32_t* ids_dev, int T, int B,
                        int n_logits, const int32_t* logit_rows, int max_ctx, float** logits_dev);
 void b2_forward_f32_release(b2_model* m);
+
+// ---- layered models (engine_layers.cu) ------------------------------------------------------------------
+// Builds a model from its description: weights from `w` (null: random ones drawn from `seed` on the device).
+int32_t b2_model_build_layered(b2_ctx* ctx, const ModelSpec& spec, const b2_weights* w, const std::string& prefix, uint64_t seed, bool f32,
+                               b2_model** out);
+void b2_layered_release(b2_model* m);
+// bytes of one page of every layer's planes, and the floats of the recurrent record
+void b2_layered_cache_layout(const b2_model* m, int block_size, std::vector<std::vector<size_t>>& page_bytes, int64_t& state_floats);
+int32_t b2_layered_ensure_rope(b2_model* m, int positions);
+struct LayeredStep {
+    const BatchMetaOut* mo;
+    const BatchMetaIn* in;
+    const int32_t* ids_dev;
+    int T, B, n_dec, dec_work, pf_work, chunk_tiles, max_ctx;
+    long dec_ctx_sum;
+    double pf_pairs;  // (query, visible key) pairs of the prefilling sequences
+    int pf_tokens, pf_ctx;  // their new tokens and their contexts, summed
+    int n_logits;
+    const int32_t* logit_rows;
+};
+int32_t b2_forward_layered(b2_model* m, b2_pool* pool, const LayeredStep& s, float** logits_dev, int* logits_ld);
+int b2_layered_q_tile(const b2_model* m);
+bool b2_tensor_to_f32(const HostTensor& t, std::vector<float>& out);

@@ -76,6 +76,27 @@ void cache_release_from(b2_cache* c, size_t first_block) {
 
 }  // namespace
 
+int32_t b2_pool::copy_page(int32_t from, int32_t to) const {
+    for (const KvPlane& pl : planes)
+        B2_CUDA(cudaMemcpyAsync(pl.base + (size_t)to * pl.page_bytes, pl.base + (size_t)from * pl.page_bytes, pl.page_bytes, cudaMemcpyDeviceToDevice,
+                                ctx->stream));
+    return B2_OK;
+}
+
+// Make an empty cache start with `n` live full blocks of another sequence.
+void b2_cache_share_blocks(b2_cache* c, const int64_t* ids, int n) {
+    b2_pool* p = c->pool;
+    for (int i = 0; i < n; i++) {
+        const int32_t page = p->id_to_page[ids[i]];
+        p->ids.retain(ids[i]);
+        p->page_ref[page]++;
+        c->block_ids.push_back(ids[i]);
+        c->pages.push_back(page);
+        push_update(p, c->slot, i, page);
+    }
+    c->len = n * p->block_size;  // starts positioned past the shared prefix (:218-220)
+}
+
 // Reserve pages for `n` more tokens of a cache (called by the step before the forward).
 int32_t b2_cache_reserve(b2_cache* c, int n) {
     b2_pool* p = c->pool;
@@ -95,6 +116,7 @@ int32_t b2_cache_reserve(b2_cache* c, int n) {
 void b2_cache_commit(b2_cache* c, int n) {
     b2_pool* p = c->pool;
     c->len += n;
+    c->state_len = c->len;
     const size_t full = (size_t)(c->len / p->block_size);
     while (c->block_ids.size() < full) {
         const int64_t id = p->ids.alloc();
@@ -124,10 +146,26 @@ int32_t b2_pool_new(b2_ctx* ctx, const b2_model* m, int32_t block_size, int64_t 
     p->layers = m->cfg.num_layers;
     p->hkv = m->hkv_l;  // pages hold this rank's KV heads only
     p->hd = m->cfg.head_dim;
-    p->page_elems = (size_t)p->hkv * block_size * p->hd;
     p->esz = m->f32 ? 4 : 2;
-    const size_t bytes = (size_t)p->layers * 2 * (size_t)max_pages * p->page_bytes();
-    cudaError_t e = cudaMalloc((void**)&p->kv, bytes);
+    std::vector<std::vector<size_t>> layout;
+    if (m->layered)
+        b2_layered_cache_layout(m, block_size, layout, p->state_floats);
+    else
+        layout.assign((size_t)p->layers, std::vector<size_t>(2, (size_t)p->hkv * block_size * p->hd * p->esz));  // K, V
+    size_t bytes = 0;
+    for (auto& layer : layout) {
+        p->layer_plane.push_back(layer.empty() ? -1 : (int)p->planes.size());
+        for (size_t pb : layer) {
+            p->planes.push_back(KvPlane{reinterpret_cast<uint8_t*>(bytes), pb});  // offset for now
+            bytes += (size_t)max_pages * pb;
+        }
+    }
+    cudaError_t e = cudaMalloc((void**)&p->kv, std::max<size_t>(bytes, 16));
+    for (KvPlane& pl : p->planes) pl.base = p->kv + reinterpret_cast<size_t>(pl.base);
+    if (e == cudaSuccess && p->state_floats > 0) {
+        e = cudaMalloc((void**)&p->state, (size_t)max_seqs * p->state_floats * 4);
+        if (e != cudaSuccess) cudaFree(p->kv);
+    }
     if (e != cudaSuccess) {
         delete p;
         return b2_fail(B2_ERR_CUDA, std::string("b2_pool_new: cudaMalloc of the KV pool failed: ") + cudaGetErrorString(e));
@@ -135,6 +173,7 @@ int32_t b2_pool_new(b2_ctx* ctx, const b2_model* m, int32_t block_size, int64_t 
     e = cudaMalloc((void**)&p->block_tables, (size_t)max_seqs * max_blocks_per_seq * 4);
     if (e != cudaSuccess) {
         cudaFree(p->kv);
+        if (p->state) cudaFree(p->state);
         delete p;
         return b2_fail(B2_ERR_CUDA, std::string("b2_pool_new: cudaMalloc of the block tables failed: ") + cudaGetErrorString(e));
     }
@@ -142,6 +181,7 @@ int32_t b2_pool_new(b2_ctx* ctx, const b2_model* m, int32_t block_size, int64_t 
     // Masked positions of a partly filled page still enter the P.V product with weight zero, and
     // 0 * NaN is NaN: the pool must never hold non-finite garbage.
     cudaMemsetAsync(p->kv, 0, bytes, ctx->stream);
+    if (p->state) cudaMemsetAsync(p->state, 0, (size_t)max_seqs * p->state_floats * 4, ctx->stream);
     p->free_pages.resize((size_t)max_pages);
     for (int64_t i = 0; i < max_pages; i++) p->free_pages[i] = (int32_t)(max_pages - 1 - i);  // page 0 goes out first
     p->page_ref.assign((size_t)max_pages, 0);
@@ -157,6 +197,7 @@ int32_t b2_pool_free(b2_pool* p) {
     cudaSetDevice(p->ctx->device);
     cudaStreamSynchronize(p->ctx->stream);
     cudaFree(p->kv);
+    if (p->state) cudaFree(p->state);
     cudaFree(p->block_tables);
     delete p;
     return B2_OK;
@@ -188,22 +229,15 @@ int32_t b2_cache_new(b2_pool* p, b2_cache** out) {
 int32_t b2_cache_new_seeded(b2_pool* p, const int64_t* shared_block_ids, int32_t n, b2_cache** out) {
     B2_REQUIRE(p && out && (n == 0 || shared_block_ids), B2_ERR_MSG, "b2_cache_new_seeded: null argument");
     B2_REQUIRE(n <= p->max_blocks, B2_ERR_OOM_PAGES, "b2_cache_new_seeded: prefix longer than max_blocks_per_seq");
+    B2_REQUIRE(n == 0 || p->state_floats == 0, B2_ERR_UNSUPPORTED,
+               "b2_cache_new_seeded: shared blocks do not carry the recurrent state of this model (fork a cache at its end instead)");
     for (int i = 0; i < n; i++) {
         const int64_t id = shared_block_ids[i];
         B2_REQUIRE(id >= 0 && (size_t)id < p->ids.refs.size() && p->ids.refs[id] > 0, B2_ERR_MSG, "b2_cache_new_seeded: block id is not live");
     }
     b2_cache* c = nullptr;
     B2_CHECK(b2_cache_new(p, &c));
-    for (int i = 0; i < n; i++) {
-        const int64_t id = shared_block_ids[i];
-        const int32_t page = p->id_to_page[id];
-        p->ids.retain(id);
-        p->page_ref[page]++;
-        c->block_ids.push_back(id);
-        c->pages.push_back(page);
-        push_update(p, c->slot, i, page);
-    }
-    c->len = n * p->block_size;  // starts positioned past the shared prefix (:218-220)
+    b2_cache_share_blocks(c, shared_block_ids, n);
     *out = c;
     return B2_OK;
 }
@@ -235,7 +269,7 @@ int32_t b2_cache_block_ids(const b2_cache* c, int64_t* out, int32_t cap) {
 int32_t b2_cache_reset(b2_cache* c) {
     B2_REQUIRE(c, B2_ERR_MSG, "b2_cache_reset: null cache");
     cache_release_from(c, 0);
-    c->len = 0;
+    c->len = c->state_len = 0;
     return B2_OK;
 }
 
@@ -251,6 +285,8 @@ int32_t b2_cache_truncate(b2_cache* c, int32_t len) {
     B2_REQUIRE(len >= 0, B2_ERR_MSG, "truncate: negative len");
     if (len >= c->len) return B2_OK;
     b2_pool* p = c->pool;
+    if (len == 0) return b2_cache_reset(c);
+    B2_REQUIRE(p->state_floats == 0, B2_ERR_UNSUPPORTED, "truncate: a recurrent state cannot be rolled back to an earlier position");
     const int bs = p->block_size;
     const size_t keep_full = (size_t)(len / bs);
     const int rem = len % bs;
@@ -265,14 +301,7 @@ int32_t b2_cache_truncate(b2_cache* c, int32_t len) {
         int32_t fresh;
         B2_CHECK(pool_alloc_page(p, &fresh));
         const int32_t old = c->pages[keep_full];
-        for (int l = 0; l < p->layers; l++) {
-            uint8_t* kl = reinterpret_cast<uint8_t*>(p->k_layer(l));
-            uint8_t* vl = reinterpret_cast<uint8_t*>(p->v_layer(l));
-            B2_CUDA(cudaMemcpyAsync(kl + (size_t)fresh * p->page_bytes(), kl + (size_t)old * p->page_bytes(), p->page_bytes(),
-                                    cudaMemcpyDeviceToDevice, p->ctx->stream));
-            B2_CUDA(cudaMemcpyAsync(vl + (size_t)fresh * p->page_bytes(), vl + (size_t)old * p->page_bytes(), p->page_bytes(),
-                                    cudaMemcpyDeviceToDevice, p->ctx->stream));
-        }
+        B2_CHECK(p->copy_page(old, fresh));
         pool_unref_page(p, old);
         c->pages[keep_full] = fresh;
         push_update(p, c->slot, (int)keep_full, fresh);
@@ -294,17 +323,19 @@ static int32_t cache_gather(b2_cache* c, int32_t layer, void* k_host, void* v_ho
     B2_REQUIRE(p->esz == esz, B2_ERR_MSG, esz == 2 ? "b2_cache_gather: the pool holds f32 pages, use b2_cache_gather_f32"
                                                   : "b2_cache_gather_f32: the pool holds bf16 pages, use b2_cache_gather");
     B2_REQUIRE(layer >= 0 && layer < p->layers, B2_ERR_MSG, "b2_cache_gather: layer out of range");
+    B2_REQUIRE(!p->model->layered, B2_ERR_UNSUPPORTED, "b2_cache_gather: this model's layers do not cache keys and values per head");
     B2_REQUIRE(c->len > 0, B2_ERR_MSG, "gather on an empty paged cache");
     const int bs = p->block_size, hd = p->hd, hkv = p->hkv;
-    std::vector<uint8_t> pk(p->page_bytes()), pv(p->page_bytes());
+    const size_t page_bytes = p->planes[p->layer_plane[layer]].page_bytes;
+    std::vector<uint8_t> pk(page_bytes), pv(page_bytes);
     B2_CUDA(cudaStreamSynchronize(p->ctx->stream));
     const uint8_t* kl = reinterpret_cast<const uint8_t*>(p->k_layer(layer));
     const uint8_t* vl = reinterpret_cast<const uint8_t*>(p->v_layer(layer));
     for (size_t b = 0; b < c->pages.size(); b++) {
         const int tokens = std::min(bs, c->len - (int)b * bs);
         if (tokens <= 0) break;
-        B2_CUDA(cudaMemcpy(pk.data(), kl + (size_t)c->pages[b] * p->page_bytes(), p->page_bytes(), cudaMemcpyDeviceToHost));
-        B2_CUDA(cudaMemcpy(pv.data(), vl + (size_t)c->pages[b] * p->page_bytes(), p->page_bytes(), cudaMemcpyDeviceToHost));
+        B2_CUDA(cudaMemcpy(pk.data(), kl + (size_t)c->pages[b] * page_bytes, page_bytes, cudaMemcpyDeviceToHost));
+        B2_CUDA(cudaMemcpy(pv.data(), vl + (size_t)c->pages[b] * page_bytes, page_bytes, cudaMemcpyDeviceToHost));
         for (int h = 0; h < hkv; h++)
             for (int t = 0; t < tokens; t++) {
                 const size_t src = ((size_t)h * bs + t) * hd * esz, dst = ((size_t)h * c->len + b * bs + t) * hd * esz;

@@ -1,0 +1,774 @@
+// Models described layer by layer (model_spec.h): weights, workspace and the forward over one ragged batch.
+//
+// The forward is called by the engine's step (b2_engine_forward) with the packer's metadata, like the flat decoders'
+// layers; pages, block tables, recurrent slots, scheduling and sampling are the engine's.  The residual stream is f32.
+// Every sub-layer leaves what it adds in `y` (f32); the next norm adds it to the stream on its way (b2_add_norm_launch).
+#include <algorithm>
+#include <cmath>
+#include <cstring>
+
+#include "engine.h"
+#include "layer_kernels.h"
+
+namespace {
+
+int up(int n, int to) { return (n + to - 1) / to * to; }
+// Padded dimensions of a projection: features in whole 128-row tiles, inputs in whole 64-wide slabs (256-wide where that
+// costs little), so that every projection kernel is eligible whatever the model's sizes are.  The padding is zero.
+int pad_n(int n) { return up(n, 128); }
+int pad_k(int k) { return k >= 768 ? up(k, 256) : up(k, 64); }
+
+struct GroupW {  // one matrix per group (expert or head), [G][N][K], N and K padded to 64
+    int G = 0, N = 0, K = 0;
+    void* w = nullptr;
+};
+struct LayerP {
+    float *norm1 = nullptr, *norm2 = nullptr;
+    // latent attention
+    Proj qkv, attn_o;  // rows: q | latent | rotated key part
+    float* c_norm = nullptr;
+    GroupW k_up_t, v_up;  // [head][kv_rank][dim] and [head][vdim][kv_rank]
+    int rope = -1;
+    // mamba2
+    Proj ssm_in, ssm_o;
+    float *conv_w = nullptr, *conv_b = nullptr, *dt_bias = nullptr, *A_log = nullptr, *D = nullptr, *ssm_norm = nullptr;
+    int64_t state_off = 0;  // floats into the slot's record
+    // feed-forward
+    Proj gu, down, router;
+    GroupW e_gu, e_down;
+};
+struct RopeTab {
+    PairRotSpec spec;
+    float *cos = nullptr, *sin = nullptr;
+};
+
+}  // namespace
+
+struct LayeredModel {
+    ModelSpec spec;
+    std::vector<LayerP> layers;
+    void* embed = nullptr;  // [pad_n(vocab), pad_k(width)]: embedding table and output projection
+    float* final_norm = nullptr;
+    std::vector<RopeTab> ropes;
+    int rope_positions = 0;
+    int64_t state_floats = 0;
+    int* route_counters = nullptr;
+    uint8_t* arena = nullptr;
+    int t_cap = 0, l_cap = 0;
+    float* capture = nullptr;
+    int64_t capture_cap = 0;
+};
+
+namespace {
+
+size_t esz(const b2_model* m) { return m->f32 ? 4 : 2; }
+
+__device__ inline uint64_t mix64d(uint64_t z) {
+    z = (z ^ (z >> 30)) * 0xBF58476D1CE4E5B9ull;
+    z = (z ^ (z >> 27)) * 0x94D049BB133111EBull;
+    return z ^ (z >> 31);
+}
+// Random block: mean + sd * (sum of four uniforms, unit variance), a function of (seed, element) only
+__global__ void random_fill_kernel(void* dst, bool f32, int64_t ld, int64_t cols, int64_t n, uint64_t seed, float mean, float sd) {
+    const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= n) return;
+    const uint64_t u = mix64d(seed + (uint64_t)(i + 1) * 0x9E3779B97F4A7C15ull);
+    const float s = (float)((u & 0xffff) + ((u >> 16) & 0xffff) + ((u >> 32) & 0xffff) + (u >> 48));
+    const float v = mean + sd * (s - 131070.f) * (1.0f / 37837.2f);
+    const int64_t at = (i / cols) * ld + i % cols;
+    if (f32)
+        reinterpret_cast<float*>(dst)[at] = v;
+    else
+        reinterpret_cast<uint16_t*>(dst)[at] = f2bf(v);
+}
+
+// Fills device tensors from a weights container, or with random values when there is none.
+struct Filler {
+    b2_model* m;
+    const b2_weights* w;
+    std::string prefix;
+    uint64_t seed;
+    int64_t bytes = 0;
+    std::vector<float> host;
+    std::vector<uint16_t> half;
+
+    int32_t alloc(size_t n, void** out) {
+        B2_CUDA(cudaMalloc(out, n ? n : 16));
+        m->allocs.push_back(*out);
+        m->weight_bytes += (int64_t)n;
+        B2_CUDA(cudaMemsetAsync(*out, 0, n ? n : 16, m->ctx->stream));
+        return B2_OK;
+    }
+    int32_t fetch(const std::string& name, std::vector<int64_t> shape) {
+        const std::string key = prefix.empty() ? name : prefix + "." + name;
+        auto it = w->t.find(key);
+        B2_REQUIRE(it != w->t.end(), B2_ERR_MISSING_TENSOR, "missing tensor `" + key + "`");
+        B2_REQUIRE(it->second.shape == shape, B2_ERR_CONFIG, "tensor `" + key + "` does not have the shape config.json implies");
+        B2_REQUIRE(b2_tensor_to_f32(it->second, host), B2_ERR_CONFIG, "tensor `" + key + "` is not a floating-point tensor");
+        return B2_OK;
+    }
+    // rows x cols of `src` (row-major, tight) to dst (row stride ld), in the model's storage format
+    int32_t put(const float* src, int rows, int cols, void* dst, int ld) {
+        const size_t es = esz(m);
+        const void* from = src;
+        if (!m->f32) {
+            half.resize((size_t)rows * cols);
+            for (size_t i = 0; i < half.size(); i++) {
+                uint32_t u;
+                memcpy(&u, &src[i], 4);
+                half[i] = (u & 0x7fffffffu) > 0x7f800000u ? (uint16_t)((u >> 16) | 0x40u) : (uint16_t)((u + 0x7fffu + ((u >> 16) & 1u)) >> 16);
+            }
+            from = half.data();
+        }
+        B2_CUDA(cudaMemcpy2DAsync(dst, (size_t)ld * es, from, (size_t)cols * es, (size_t)cols * es, (size_t)rows, cudaMemcpyHostToDevice, m->ctx->stream));
+        B2_CUDA(cudaStreamSynchronize(m->ctx->stream));
+        return B2_OK;
+    }
+    int32_t random(void* dst, bool f32, int rows, int cols, int ld, float mean, float sd) {
+        const int64_t n = (int64_t)rows * cols;
+        random_fill_kernel<<<(unsigned)((n + 255) / 256), 256, 0, m->ctx->stream>>>(dst, f32, ld, cols, n, ++seed * 0x9E3779B97F4A7C15ull, mean, sd);
+        B2_CUDA(cudaGetLastError());
+        return B2_OK;
+    }
+    void* at(void* base, int64_t elems) const { return (uint8_t*)base + elems * (int64_t)esz(m); }
+
+    int32_t proj(Proj& p, int N, int K) {
+        p.bits = 0;
+        p.N = pad_n(N);
+        p.K = pad_k(K);
+        return alloc((size_t)p.N * p.K * esz(m), &p.w);
+    }
+    // tensor [rows, cols] to rows row0.. of p
+    int32_t rows(Proj& p, int row0, const std::string& key, int rows, int cols) {
+        void* dst = at(p.w, (int64_t)row0 * p.K);
+        if (!w) return random(dst, m->f32, rows, cols, p.K, 0.f, 1.0f / sqrtf((float)cols));
+        B2_CHECK(fetch(key, {rows, cols}));
+        return put(host.data(), rows, cols, dst, p.K);
+    }
+    int32_t vec(float*& dst, const std::string& key, std::vector<int64_t> shape, float mean, float sd) {
+        int64_t n = 1;
+        for (auto d : shape) n *= d;
+        B2_CHECK(alloc((size_t)n * 4, (void**)&dst));
+        if (!w) return random(dst, true, 1, (int)n, (int)n, mean, sd);
+        B2_CHECK(fetch(key, shape));
+        B2_CUDA(cudaMemcpyAsync(dst, host.data(), (size_t)n * 4, cudaMemcpyHostToDevice, m->ctx->stream));
+        B2_CUDA(cudaStreamSynchronize(m->ctx->stream));
+        return B2_OK;
+    }
+    int32_t group(GroupW& g, int G, int N, int K) {
+        g.G = G;
+        g.N = up(N, 64);
+        g.K = up(K, 64);
+        return alloc((size_t)G * g.N * g.K * esz(m), &g.w);
+    }
+    int32_t group_rows(GroupW& g, int i, int row0, const std::string& key, int rows, int cols) {
+        void* dst = at(g.w, ((int64_t)i * g.N + row0) * g.K);
+        if (!w) return random(dst, m->f32, rows, cols, g.K, 0.f, 1.0f / sqrtf((float)cols));
+        B2_CHECK(fetch(key, {rows, cols}));
+        return put(host.data(), rows, cols, dst, g.K);
+    }
+    // tensor [G * rows, cols] split by rows over the groups, each part transposed when asked
+    int32_t group_split(GroupW& g, const std::string& key, int rows, int cols, bool transpose) {
+        if (!w) {
+            for (int i = 0; i < g.G; i++)
+                B2_CHECK(random(at(g.w, (int64_t)i * g.N * g.K), m->f32, transpose ? cols : rows, transpose ? rows : cols, g.K, 0.f, 1.0f / sqrtf((float)cols)));
+            return B2_OK;
+        }
+        B2_CHECK(fetch(key, {(int64_t)g.G * rows, cols}));
+        std::vector<float> part((size_t)rows * cols);
+        for (int i = 0; i < g.G; i++) {
+            const float* s = host.data() + (size_t)i * rows * cols;
+            if (transpose)
+                for (int r = 0; r < rows; r++)
+                    for (int c = 0; c < cols; c++) part[(size_t)c * rows + r] = s[(size_t)r * cols + c];
+            B2_CHECK(put(transpose ? part.data() : s, transpose ? cols : rows, transpose ? rows : cols, at(g.w, (int64_t)i * g.N * g.K), g.K));
+        }
+        return B2_OK;
+    }
+};
+
+int32_t load_layer(Filler& f, LayeredModel& lm, int i) {
+    const LayerSpec& L = lm.spec.layers[i];
+    const TensorNames& tn = lm.spec.names;
+    LayerP& P = lm.layers[i];
+    const int W = lm.spec.width;
+    auto key = [&](const std::string& s) { return tn.layer_key(i, s); };
+    auto mix = [&](const std::string& s) { return tn.layer_key(i, tn.mixer + "." + s); };
+    auto mlp = [&](const std::string& s) { return tn.layer_key(i, tn.mlp + "." + s); };
+    B2_CHECK(f.vec(P.norm1, key(tn.norm1), {W}, 1.f, 0.f));
+    if (L.mixer == MixerKind::LatentAttention) {
+        const LatentAttnSpec& a = L.attn;
+        const int q = a.heads * (a.dim + a.rot_dim);
+        B2_CHECK(f.proj(P.qkv, q + a.row(), W));
+        B2_CHECK(f.rows(P.qkv, 0, mix("q"), q, W));
+        B2_CHECK(f.rows(P.qkv, q, mix("dkv"), a.row(), W));
+        B2_CHECK(f.vec(P.c_norm, mix("dkv.norm"), {a.kv_rank}, 1.f, 0.f));
+        B2_CHECK(f.group(P.k_up_t, a.heads, a.kv_rank, a.dim));
+        B2_CHECK(f.group_split(P.k_up_t, mix("uk"), a.dim, a.kv_rank, true));
+        B2_CHECK(f.group(P.v_up, a.heads, a.vdim, a.kv_rank));
+        B2_CHECK(f.group_split(P.v_up, mix("uv"), a.vdim, a.kv_rank, false));
+        B2_CHECK(f.proj(P.attn_o, W, a.heads * a.vdim));
+        B2_CHECK(f.rows(P.attn_o, 0, mix("o"), W, a.heads * a.vdim));
+        for (size_t r = 0; r < lm.ropes.size(); r++)
+            if (lm.ropes[r].spec.base == a.rot.base && lm.ropes[r].spec.dims == a.rot.dims) P.rope = (int)r;
+        if (P.rope < 0) {
+            P.rope = (int)lm.ropes.size();
+            lm.ropes.push_back(RopeTab{a.rot});
+        }
+    } else {
+        const Mamba2Spec& s = L.ssm;
+        B2_CHECK(f.proj(P.ssm_in, s.in_rows(), W));
+        B2_CHECK(f.rows(P.ssm_in, 0, mix("in"), s.in_rows(), W));
+        B2_CHECK(f.vec(P.conv_w, mix("conv"), {s.channels(), s.conv}, 0.f, 0.5f));
+        B2_CHECK(f.vec(P.conv_b, mix("conv.b"), {s.channels()}, 0.f, 0.1f));
+        B2_CHECK(f.vec(P.dt_bias, mix("dt_bias"), {s.heads}, -3.f, 1.f));
+        B2_CHECK(f.vec(P.A_log, mix("A_log"), {s.heads}, 1.f, 0.7f));
+        B2_CHECK(f.vec(P.D, mix("D"), {s.heads}, 1.f, 0.f));
+        B2_CHECK(f.vec(P.ssm_norm, mix("norm"), {s.inner()}, 1.f, 0.f));
+        B2_CHECK(f.proj(P.ssm_o, W, s.inner()));
+        B2_CHECK(f.rows(P.ssm_o, 0, mix("o"), W, s.inner()));
+        P.state_off = lm.state_floats;
+        lm.state_floats += up(s.inner() * s.state, 4) + up(s.channels() * (s.conv - 1), 4);
+    }
+    if (L.mlp == MlpKind::None) return B2_OK;
+    B2_CHECK(f.vec(P.norm2, key(tn.norm2), {W}, 1.f, 0.f));
+    if (L.mlp == MlpKind::DenseGated) {
+        const int ffp = up(L.ff, 64);
+        B2_CHECK(f.proj(P.gu, 2 * ffp, W));
+        B2_CHECK(f.rows(P.gu, 0, mlp("gate"), L.ff, W));
+        B2_CHECK(f.rows(P.gu, ffp, mlp("up"), L.ff, W));
+        B2_CHECK(f.proj(P.down, W, L.ff));
+        B2_CHECK(f.rows(P.down, 0, mlp("down"), W, L.ff));
+    } else {
+        const RoutedSpec& r = L.moe;
+        const int ffp = up(r.ff, 64);
+        B2_CHECK(f.proj(P.router, r.experts, W));
+        B2_CHECK(f.rows(P.router, 0, mlp("router"), r.experts, W));
+        B2_CHECK(f.group(P.e_gu, r.experts, 2 * ffp, W));
+        B2_CHECK(f.group(P.e_down, r.experts, W, r.ff));
+        for (int e = 0; e < r.experts; e++) {
+            const std::string ek = "e" + std::to_string(e) + ".";
+            B2_CHECK(f.group_rows(P.e_gu, e, 0, mlp(ek + "gate"), r.ff, W));
+            B2_CHECK(f.group_rows(P.e_gu, e, ffp, mlp(ek + "up"), r.ff, W));
+            B2_CHECK(f.group_rows(P.e_down, e, 0, mlp(ek + "down"), W, r.ff));
+        }
+    }
+    return B2_OK;
+}
+
+// ---- workspace ------------------------------------------------------------------------------------------------------
+// One allocation, carved for a capacity of `t` tokens and `l` logits rows; the parts a layer needs only while it runs
+// share one region.  With base == null the carving only measures.
+struct Carver {
+    uint8_t* base;
+    size_t off = 0;
+    template <typename T = void>
+    T* take(size_t bytes) {
+        off = (off + 255) / 256 * 256;
+        T* p = reinterpret_cast<T*>(base ? base + off : nullptr);
+        off += bytes;
+        return p;
+    }
+};
+struct Common {
+    float *x, *y, *logits;
+    void *xn, *last;
+    int ldx, ldn, ldl;
+};
+struct LatentBufs {
+    void *qkv, *q_nope, *q_lat, *o_lat, *att;
+    int dim_pad, o_pad, ld_att;
+};
+struct SsmBufs {
+    void *zx, *xbc, *gn;
+    float* y;
+    int ld_xbc, ld_gn;
+};
+struct DenseBufs {
+    void *gu, *act;
+    int ld_act;
+};
+struct MoeBufs {
+    float *logits, *weight, *row_w;
+    int32_t *expert, *offsets, *pos, *src;
+    void *gu, *act;
+    int ld_act;
+};
+Common carve_common(Carver& c, const LayeredModel& lm, size_t es, size_t t, size_t l) {
+    Common o;
+    int top = 1;
+    for (auto& L : lm.spec.layers)
+        if (L.mlp == MlpKind::Routed) top = std::max(top, L.moe.top);
+    o.ldx = pad_n(lm.spec.width);
+    o.ldn = pad_k(lm.spec.width);
+    o.ldl = pad_n(lm.spec.vocab);
+    o.x = c.take<float>(t * o.ldx * 4);
+    o.y = c.take<float>(t * top * o.ldx * 4);
+    o.xn = c.take(t * o.ldn * es);
+    o.last = c.take(l * o.ldn * es);
+    o.logits = c.take<float>(l * o.ldl * 4);
+    return o;
+}
+LatentBufs carve_latent(Carver c, const LatentAttnSpec& a, const LayerP& P, size_t es, size_t t, size_t* end) {
+    LatentBufs o;
+    o.dim_pad = P.k_up_t.K;
+    o.o_pad = P.v_up.K;
+    o.ld_att = P.attn_o.K;
+    o.qkv = c.take(t * P.qkv.N * es);
+    o.q_nope = c.take(t * a.heads * o.dim_pad * es);
+    o.q_lat = c.take(t * a.heads * a.row_pad() * es);
+    o.o_lat = c.take(t * a.heads * o.o_pad * es);
+    o.att = c.take(t * o.ld_att * es);
+    *end = std::max(*end, c.off);
+    return o;
+}
+SsmBufs carve_ssm(Carver c, const Mamba2Spec& s, const LayerP& P, size_t es, size_t t, size_t* end) {
+    SsmBufs o;
+    o.ld_xbc = up(s.channels(), 8);
+    o.ld_gn = P.ssm_o.K;
+    o.zx = c.take(t * P.ssm_in.N * es);
+    o.xbc = c.take(t * o.ld_xbc * es);
+    o.y = c.take<float>(t * s.inner() * 4);
+    o.gn = c.take(t * o.ld_gn * es);
+    *end = std::max(*end, c.off);
+    return o;
+}
+DenseBufs carve_dense(Carver c, const LayerP& P, size_t es, size_t t, size_t* end) {
+    DenseBufs o;
+    o.ld_act = P.down.K;
+    o.gu = c.take(t * P.gu.N * es);
+    o.act = c.take(t * o.ld_act * es);
+    *end = std::max(*end, c.off);
+    return o;
+}
+MoeBufs carve_moe(Carver c, const RoutedSpec& r, const LayerP& P, size_t es, size_t t, size_t* end) {
+    MoeBufs o;
+    const size_t n = t * r.top;
+    o.ld_act = P.e_down.K;
+    o.logits = c.take<float>(t * P.router.N * 4);
+    o.weight = c.take<float>(n * 4);
+    o.row_w = c.take<float>(n * 4);
+    o.expert = c.take<int32_t>(n * 4);
+    o.pos = c.take<int32_t>(n * 4);
+    o.src = c.take<int32_t>(n * 4);
+    o.offsets = c.take<int32_t>((size_t)(r.experts + 1) * 4);
+    o.gu = c.take(n * P.e_gu.N * es);
+    o.act = c.take(n * o.ld_act * es);
+    *end = std::max(*end, c.off);
+    return o;
+}
+size_t arena_bytes(const LayeredModel& lm, size_t es, size_t t, size_t l) {
+    Carver c{nullptr};
+    carve_common(c, lm, es, t, l);
+    size_t end = c.off;
+    for (size_t i = 0; i < lm.layers.size(); i++) {
+        const LayerSpec& L = lm.spec.layers[i];
+        const LayerP& P = lm.layers[i];
+        if (L.mixer == MixerKind::LatentAttention)
+            carve_latent(c, L.attn, P, es, t, &end);
+        else
+            carve_ssm(c, L.ssm, P, es, t, &end);
+        if (L.mlp == MlpKind::DenseGated) carve_dense(c, P, es, t, &end);
+        if (L.mlp == MlpKind::Routed) carve_moe(c, L.moe, P, es, t, &end);
+    }
+    return end + 256;
+}
+int32_t ensure_arena(b2_model* m, int T, int n_logits) {
+    LayeredModel& lm = *m->layered;
+    if (T <= lm.t_cap && n_logits <= lm.l_cap && lm.arena) return B2_OK;
+    B2_CUDA(cudaStreamSynchronize(m->ctx->stream));
+    if (T > lm.t_cap) lm.t_cap = up(std::max(T, 128) * 9 / 8, 128);  // at least one box of the projections' row loads
+    if (n_logits > lm.l_cap) lm.l_cap = up(std::max(n_logits, 128) * 9 / 8, 128);
+    if (lm.arena) B2_CUDA(cudaFree(lm.arena));
+    lm.arena = nullptr;
+    const size_t bytes = arena_bytes(lm, esz(m), (size_t)lm.t_cap, (size_t)std::max(lm.l_cap, 128));
+    if (lm.l_cap == 0) lm.l_cap = 128;
+    B2_CUDA(cudaMalloc((void**)&lm.arena, bytes));
+    B2_CUDA(cudaMemsetAsync(lm.arena, 0, bytes, m->ctx->stream));
+    return B2_OK;
+}
+
+// ---- forward --------------------------------------------------------------------------------------------------------
+int32_t linear(b2_model* m, const Proj& p, const void* x, int ldx, int M, int rows_cap, void* out, int ldo, bool out_f32) {
+    b2_prof_mark(m->ctx, B2_CLS_GEMM);
+    if (m->f32) return b2_linear_f32_launch(m->ctx, (const float*)x, ldx, (const float*)p.w, M, p.N, p.K, (float*)out, ldo);
+    GemmParams g{};
+    g.x = (const uint16_t*)x;
+    g.w = p.w;
+    g.group = 64;
+    g.M = M;
+    g.N = p.N;
+    g.K = p.K;
+    g.ldx = ldx;
+    g.ldo = ldo;
+    g.ldres = ldo;
+    g.x_rows_cap = rows_cap;
+    g.epilogue = out_f32 ? EPI_F32 : EPI_BF16;
+    if (out_f32)
+        g.out_f32 = (float*)out;
+    else
+        g.out = (uint16_t*)out;
+    return b2_gemm_launch(m->ctx, g);
+}
+
+struct Fwd {  // one step
+    b2_model* m;
+    LayeredModel& lm;
+    b2_pool* pool;
+    const LayeredStep& s;
+    Common c;
+    Carver scratch;
+    size_t es, end = 0;
+
+    int32_t latent(const LayerSpec& L, const LayerP& P, int l);
+    int32_t ssm(const LayerSpec& L, const LayerP& P);
+    int32_t dense(const LayerSpec& L, const LayerP& P);
+    int32_t moe(const LayerSpec& L, const LayerP& P, const int32_t** rows);
+};
+
+int32_t Fwd::latent(const LayerSpec& L, const LayerP& P, int l) {
+    b2_ctx* ctx = m->ctx;
+    const LatentAttnSpec& a = L.attn;
+    const LatentBufs b = carve_latent(scratch, a, P, es, (size_t)lm.t_cap, &end);
+    const int T = s.T, W = a.row_pad();
+    B2_CHECK(linear(m, P.qkv, c.xn, c.ldn, T, lm.t_cap, b.qkv, P.qkv.N, false));
+    LatentPrepParams pp{};
+    pp.qkv = b.qkv;
+    pp.ld = P.qkv.N;
+    pp.T = T;
+    pp.positions = s.mo->positions;
+    pp.slot_mapping = s.mo->slot_mapping;
+    pp.cos_t = lm.ropes[P.rope].cos;
+    pp.sin_t = lm.ropes[P.rope].sin;
+    pp.c_norm = P.c_norm;
+    pp.eps = lm.spec.eps;
+    pp.cache = pool->planes[pool->layer_plane[l]].base;
+    pp.q_nope = b.q_nope;
+    pp.dim_pad = b.dim_pad;
+    pp.q_lat = b.q_lat;
+    b2_prof_mark(ctx, B2_CLS_ROPE_KV);
+    B2_CHECK(b2_latent_prep_launch(ctx, m->f32, a, pp));
+    GroupedGemmParams g{};
+    g.x = b.q_nope;
+    g.x_gstride = b.dim_pad;
+    g.ldx = a.heads * b.dim_pad;
+    g.w = P.k_up_t.w;
+    g.N = P.k_up_t.N;
+    g.K = P.k_up_t.K;
+    g.G = a.heads;
+    g.out = b.q_lat;
+    g.out_gstride = W;
+    g.ldo = a.heads * W;
+    g.n_out = a.kv_rank;
+    g.M = T;
+    b2_prof_mark(ctx, B2_CLS_GEMM);
+    B2_CHECK(b2_grouped_gemm_launch(ctx, m->f32, g));
+    LatentAttnParams ap{};
+    ap.q_lat = b.q_lat;
+    ap.cache = pp.cache;
+    ap.block_tables = pool->block_tables;
+    ap.max_blocks = pool->max_blocks;
+    ap.page_size = pool->block_size;
+    ap.seq_slot = s.in->seq_slot;
+    ap.token_seq = s.mo->token_seq;
+    ap.positions = s.mo->positions;
+    ap.o_lat = b.o_lat;
+    ap.o_pad = b.o_pad;
+    ap.T = T;
+    b2_prof_mark(ctx, B2_CLS_ATTN_PREFILL);
+    B2_CHECK(b2_latent_attn_simple_launch(ctx, m->f32, a, ap));
+    GroupedGemmParams v{};
+    v.x = b.o_lat;
+    v.x_gstride = b.o_pad;
+    v.ldx = a.heads * b.o_pad;
+    v.w = P.v_up.w;
+    v.N = P.v_up.N;
+    v.K = P.v_up.K;
+    v.G = a.heads;
+    v.out = b.att;
+    v.out_gstride = a.vdim;
+    v.ldo = b.ld_att;
+    v.n_out = a.vdim;
+    v.M = T;
+    b2_prof_mark(ctx, B2_CLS_GEMM);
+    B2_CHECK(b2_grouped_gemm_launch(ctx, m->f32, v));
+    B2_CHECK(b2_zero_cols_launch(ctx, m->f32, b.att, b.ld_att, a.heads * a.vdim, b.ld_att, T));
+    return linear(m, P.attn_o, b.att, b.ld_att, T, lm.t_cap, c.y, c.ldx, true);
+}
+
+int32_t Fwd::ssm(const LayerSpec& L, const LayerP& P) {
+    const SsmBufs b = carve_ssm(scratch, L.ssm, P, es, (size_t)lm.t_cap, &end);
+    B2_CHECK(linear(m, P.ssm_in, c.xn, c.ldn, s.T, lm.t_cap, b.zx, P.ssm_in.N, false));
+    SsmParams p{};
+    p.zx = b.zx;
+    p.ld = P.ssm_in.N;
+    p.T = s.T;
+    p.B = s.B;
+    p.cu_seqlens = s.mo->cu_seqlens;
+    p.context_lens = s.mo->context_lens;
+    p.token_seq = s.mo->token_seq;
+    p.seq_slot = s.in->seq_slot;
+    p.state = pool->state + P.state_off;
+    p.slot_stride = pool->state_floats;
+    p.conv_w = P.conv_w;
+    p.conv_b = P.conv_b;
+    p.dt_bias = P.dt_bias;
+    p.A_log = P.A_log;
+    p.D = P.D;
+    p.norm = P.ssm_norm;
+    p.eps = lm.spec.eps;
+    p.xbc = b.xbc;
+    p.ld_xbc = b.ld_xbc;
+    p.y = b.y;
+    p.out = b.gn;
+    p.ldo = b.ld_gn;
+    b2_prof_mark(m->ctx, B2_CLS_RECURRENT);
+    B2_CHECK(b2_ssm_launch(m->ctx, m->f32, L.ssm, p));
+    return linear(m, P.ssm_o, b.gn, b.ld_gn, s.T, lm.t_cap, c.y, c.ldx, true);
+}
+
+int32_t Fwd::dense(const LayerSpec& L, const LayerP& P) {
+    const DenseBufs b = carve_dense(scratch, P, es, (size_t)lm.t_cap, &end);
+    B2_CHECK(linear(m, P.gu, c.xn, c.ldn, s.T, lm.t_cap, b.gu, P.gu.N, false));
+    b2_prof_mark(m->ctx, B2_CLS_ELEMENTWISE);
+    B2_CHECK(b2_gate_launch(m->ctx, m->f32, L.gate, b.gu, P.gu.N, up(L.ff, 64), nullptr, s.T, L.ff, b.act, b.ld_act));
+    return linear(m, P.down, b.act, b.ld_act, s.T, lm.t_cap, c.y, c.ldx, true);
+}
+
+int32_t Fwd::moe(const LayerSpec& L, const LayerP& P, const int32_t** rows) {
+    b2_ctx* ctx = m->ctx;
+    const RoutedSpec& r = L.moe;
+    const MoeBufs b = carve_moe(scratch, r, P, es, (size_t)lm.t_cap, &end);
+    B2_CHECK(linear(m, P.router, c.xn, c.ldn, s.T, lm.t_cap, b.logits, P.router.N, true));
+    RouteParams rp{};
+    rp.logits = b.logits;
+    rp.ld = P.router.N;
+    rp.T = s.T;
+    rp.experts = r.experts;
+    rp.top = r.top;
+    rp.expert = b.expert;
+    rp.weight = b.weight;
+    rp.offsets = b.offsets;
+    rp.pos = b.pos;
+    rp.src = b.src;
+    rp.row_w = b.row_w;
+    rp.counters = lm.route_counters;
+    b2_prof_mark(ctx, B2_CLS_ELEMENTWISE);
+    B2_CHECK(b2_route_launch(ctx, rp));
+    GroupedGemmParams g{};
+    g.x = c.xn;
+    g.ldx = c.ldn;
+    g.row_idx = b.src;
+    g.w = P.e_gu.w;
+    g.N = P.e_gu.N;
+    g.K = P.e_gu.K;
+    g.G = r.experts;
+    g.out = b.gu;
+    g.ldo = g.n_out = P.e_gu.N;
+    g.offsets = b.offsets;
+    g.M = s.T * r.top;
+    b2_prof_mark(ctx, B2_CLS_GEMM);
+    B2_CHECK(b2_grouped_gemm_launch(ctx, m->f32, g));
+    b2_prof_mark(ctx, B2_CLS_ELEMENTWISE);
+    B2_CHECK(b2_gate_launch(ctx, m->f32, r.gate, b.gu, P.e_gu.N, up(r.ff, 64), b.row_w, g.M, r.ff, b.act, b.ld_act));
+    GroupedGemmParams d{};
+    d.x = b.act;
+    d.ldx = b.ld_act;
+    d.w = P.e_down.w;
+    d.N = P.e_down.N;
+    d.K = P.e_down.K;
+    d.G = r.experts;
+    d.out = c.y;
+    d.ldo = c.ldx;
+    d.n_out = lm.spec.width;
+    d.out_f32 = true;
+    d.offsets = b.offsets;
+    d.M = g.M;
+    b2_prof_mark(ctx, B2_CLS_GEMM);
+    B2_CHECK(b2_grouped_gemm_launch(ctx, m->f32, d));
+    *rows = b.pos;
+    return B2_OK;
+}
+
+}  // namespace
+
+int b2_layered_q_tile(const b2_model*) { return 64; }
+
+void b2_layered_cache_layout(const b2_model* m, int block_size, std::vector<std::vector<size_t>>& page_bytes, int64_t& state_floats) {
+    for (auto& L : m->layered->spec.layers) {
+        page_bytes.emplace_back();
+        if (L.mixer == MixerKind::LatentAttention) page_bytes.back().push_back((size_t)block_size * L.attn.row_pad() * esz(m));
+    }
+    state_floats = m->layered->state_floats;
+}
+
+int32_t b2_layered_ensure_rope(b2_model* m, int positions) {
+    LayeredModel& lm = *m->layered;
+    if (positions <= lm.rope_positions || lm.ropes.empty()) return B2_OK;
+    int n = std::max(4096, lm.rope_positions);
+    while (n < positions) n *= 2;
+    B2_CUDA(cudaStreamSynchronize(m->ctx->stream));
+    for (RopeTab& r : lm.ropes) {
+        const int half = r.spec.dims / 2;
+        std::vector<float> c((size_t)n * half), s((size_t)n * half);
+        for (int i = 0; i < half; i++) {
+            const double f = std::pow(r.spec.base, -2.0 * i / r.spec.dims);
+            for (int p = 0; p < n; p++) {  // rounded once, to f32
+                c[(size_t)p * half + i] = (float)std::cos(p * f);
+                s[(size_t)p * half + i] = (float)std::sin(p * f);
+            }
+        }
+        if (r.cos) cudaFree(r.cos);
+        if (r.sin) cudaFree(r.sin);
+        B2_CUDA(cudaMalloc((void**)&r.cos, std::max<size_t>(c.size(), 1) * 4));
+        B2_CUDA(cudaMalloc((void**)&r.sin, std::max<size_t>(s.size(), 1) * 4));
+        B2_CUDA(cudaMemcpyAsync(r.cos, c.data(), c.size() * 4, cudaMemcpyHostToDevice, m->ctx->stream));
+        B2_CUDA(cudaMemcpyAsync(r.sin, s.data(), s.size() * 4, cudaMemcpyHostToDevice, m->ctx->stream));
+        B2_CUDA(cudaStreamSynchronize(m->ctx->stream));
+    }
+    lm.rope_positions = n;
+    return B2_OK;
+}
+
+int32_t b2_model_build_layered(b2_ctx* ctx, const ModelSpec& spec, const b2_weights* w, const std::string& prefix, uint64_t seed, bool f32,
+                               b2_model** out) {
+    B2_CUDA(cudaSetDevice(ctx->device));
+    b2_model* m = new b2_model();
+    m->ctx = ctx;
+    m->f32 = f32;
+    m->layered = new LayeredModel();
+    LayeredModel& lm = *m->layered;
+    lm.spec = spec;
+    lm.layers.resize(spec.layers.size());
+    m->cfg.num_layers = (int32_t)spec.layers.size();
+    m->cfg.hidden_size = spec.width;
+    m->cfg.vocab_size = spec.vocab;
+    m->cfg.rms_norm_eps = spec.eps;
+    m->cfg.tie_word_embeddings = 1;
+    m->cfg.compute_f32 = f32 ? 1 : 0;
+    m->hkv_l = 1;  // the latent is one key/value head
+    Filler f{m, w, prefix, seed};
+    auto build = [&]() -> int32_t {
+        Proj head;
+        B2_CHECK(f.proj(head, spec.vocab, spec.width));
+        B2_CHECK(f.rows(head, 0, spec.names.embed, spec.vocab, spec.width));
+        lm.embed = head.w;
+        for (size_t i = 0; i < spec.layers.size(); i++) B2_CHECK(load_layer(f, lm, (int)i));
+        B2_CHECK(f.vec(lm.final_norm, spec.names.final_norm, {spec.width}, 1.f, 0.f));
+        B2_CUDA(cudaMalloc((void**)&lm.route_counters, 1025 * sizeof(int)));
+        B2_CUDA(cudaMemsetAsync(lm.route_counters, 0, 1025 * sizeof(int), ctx->stream));
+        B2_CUDA(cudaEventCreate(&m->ev0));
+        B2_CUDA(cudaEventCreate(&m->ev1));
+        B2_CUDA(cudaStreamSynchronize(ctx->stream));
+        return B2_OK;
+    };
+    const int32_t rc = build();
+    if (rc != B2_OK) {
+        b2_model_free(m);
+        return rc;
+    }
+    *out = m;
+    return B2_OK;
+}
+
+void b2_layered_release(b2_model* m) {
+    if (!m->layered) return;
+    LayeredModel& lm = *m->layered;
+    for (RopeTab& r : lm.ropes) {
+        if (r.cos) cudaFree(r.cos);
+        if (r.sin) cudaFree(r.sin);
+    }
+    if (lm.route_counters) cudaFree(lm.route_counters);
+    if (lm.arena) cudaFree(lm.arena);
+    delete m->layered;
+    m->layered = nullptr;
+}
+
+int32_t b2_forward_layered(b2_model* m, b2_pool* pool, const LayeredStep& s, float** logits_dev, int* logits_ld) {
+    b2_ctx* ctx = m->ctx;
+    LayeredModel& lm = *m->layered;
+    const ModelSpec& spec = lm.spec;
+    B2_REQUIRE(pool->model == m, B2_ERR_MSG, "forward: the caches belong to another model's pool");
+    B2_REQUIRE(s.T <= 65535, B2_ERR_UNSUPPORTED, "forward: at most 65535 tokens in one step of a layered model");
+    B2_CHECK(ensure_arena(m, s.T, s.n_logits));
+    Carver carver{lm.arena};
+    const Common c = carve_common(carver, lm, esz(m), (size_t)lm.t_cap, (size_t)lm.l_cap);
+    Fwd f{m, lm, pool, s, c, carver, esz(m)};
+    b2_prof_mark(ctx, B2_CLS_ELEMENTWISE);
+    B2_CHECK(b2_embed_residual_launch(ctx, m->f32, lm.embed, c.ldn, s.ids_dev, s.T, spec.width, spec.vocab, c.x, c.ldx));
+    AddNormParams an{};
+    an.x = c.x;
+    an.y = c.y;
+    an.ldx = an.ldy = c.ldx;
+    an.width = spec.width;
+    an.eps = spec.eps;
+    an.n_src = 0;  // nothing is pending behind the embedding
+    auto norm = [&](const float* w, int rows, const int32_t* row_idx, void* out, float scale, bool write) {
+        an.w = w;
+        an.rows = rows;
+        an.row_idx = row_idx;
+        an.out = out;
+        an.ldo = c.ldn;
+        an.out_scale = scale;
+        an.write_x = write && an.n_src > 0;
+        b2_prof_mark(ctx, B2_CLS_ELEMENTWISE);
+        return b2_add_norm_launch(ctx, m->f32, an);
+    };
+    auto pending = [&](const int32_t* rows, int n) {
+        an.y_rows = rows;
+        an.n_src = n;
+    };
+    const int64_t per_layer = (int64_t)s.T * spec.width;
+    const bool capture = lm.capture && lm.capture_cap >= per_layer * (int64_t)spec.layers.size();
+    for (size_t l = 0; l < spec.layers.size(); l++) {
+        const LayerSpec& L = spec.layers[l];
+        const LayerP& P = lm.layers[l];
+        B2_CHECK(norm(P.norm1, s.T, nullptr, c.xn, 1.f, true));
+        B2_CHECK(L.mixer == MixerKind::LatentAttention ? f.latent(L, P, (int)l) : f.ssm(L, P));
+        pending(nullptr, 1);
+        if (L.mlp != MlpKind::None) {
+            B2_CHECK(norm(P.norm2, s.T, nullptr, c.xn, 1.f, true));
+            const int32_t* rows = nullptr;
+            if (L.mlp == MlpKind::DenseGated) {
+                B2_CHECK(f.dense(L, P));
+                pending(nullptr, 1);
+            } else {
+                B2_CHECK(f.moe(L, P, &rows));
+                pending(rows, L.moe.top);
+            }
+        }
+        if (capture) {
+            B2_CHECK(norm(nullptr, s.T, nullptr, nullptr, 1.f, true));  // the addition alone
+            pending(nullptr, 0);
+            B2_CUDA(cudaMemcpy2DAsync(lm.capture + (int64_t)l * per_layer, (size_t)spec.width * 4, c.x, (size_t)c.ldx * 4, (size_t)spec.width * 4, (size_t)s.T,
+                                      cudaMemcpyDeviceToHost, ctx->stream));
+        }
+    }
+    if (s.n_logits > 0) {
+        B2_CHECK(norm(lm.final_norm, s.n_logits, s.logit_rows, c.last, spec.logit_scale, false));
+        Proj head;
+        head.N = pad_n(spec.vocab);
+        head.K = c.ldn;
+        head.w = lm.embed;
+        B2_CHECK(linear(m, head, c.last, c.ldn, s.n_logits, lm.l_cap, c.logits, c.ldl, true));
+        b2_prof_mark(ctx, B2_CLS_ELEMENTWISE);
+        B2_CHECK(b2_argmax_f32_launch(ctx, c.logits, c.ldl, s.n_logits, spec.vocab, m->ws.argmax));
+    }
+    B2_CUDA(cudaGetLastError());
+    *logits_dev = c.logits;
+    *logits_ld = c.ldl;
+    return B2_OK;
+}
+
+extern "C" {
+
+int64_t b2_model_state_bytes(const b2_model* m) { return m && m->layered ? m->layered->state_floats * 4 : 0; }
+
+int32_t b2_model_capture_residual(b2_model* m, float* out_host, int64_t capacity_floats) {
+    B2_REQUIRE(m && m->layered, B2_ERR_UNSUPPORTED, "b2_model_capture_residual: not a layered model");
+    m->layered->capture = out_host;
+    m->layered->capture_cap = out_host ? capacity_floats : 0;
+    return B2_OK;
+}
+
+}  // extern "C"

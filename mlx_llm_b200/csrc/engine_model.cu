@@ -198,6 +198,25 @@ int32_t finish_model(b2_model* m) {
 
 }  // namespace
 
+bool b2_tensor_to_f32(const HostTensor& t, std::vector<float>& out) {
+    out.resize((size_t)t.numel());
+    if (t.dtype == B2_DTYPE_F32) {
+        memcpy(out.data(), t.ptr, out.size() * 4);
+    } else if (t.dtype == B2_DTYPE_BF16 || t.dtype == B2_DTYPE_F16) {
+        const uint16_t* h = (const uint16_t*)t.ptr;
+        for (size_t i = 0; i < out.size(); i++) {
+            const uint32_t u = (uint32_t)h[i] << 16;
+            if (t.dtype == B2_DTYPE_F16)
+                out[i] = h_half2f(h[i]);
+            else
+                memcpy(&out[i], &u, 4);
+        }
+    } else {
+        return false;
+    }
+    return true;
+}
+
 int32_t b2_model_ensure_rope(b2_model* m, int positions) {
     if (positions <= m->rope_positions) return B2_OK;
     int n = std::max(4096, m->rope_positions);
@@ -748,6 +767,7 @@ int32_t b2_model_free(b2_model* m) {
     if (m->cos_f32) cudaFree(m->cos_f32);
     if (m->sin_f32) cudaFree(m->sin_f32);
     b2_forward_f32_release(m);
+    b2_layered_release(m);
     Workspace& w = m->ws;
     void* dev[] = {w.x_in_peer_region ? nullptr : (void*)w.x, w.tp_part, w.xn, w.qkv, w.q, w.attn, w.gu, w.act, w.last, w.logits, w.argmax, w.ids, w.meta, w.stage_dev, w.attn_scratch};
     for (void* p : dev)
@@ -765,6 +785,7 @@ int32_t b2_model_get_config(const b2_model* m, b2_model_config* out) {
     *out = m->cfg;
     return B2_OK;
 }
+int32_t b2_model_logits_f32(const b2_model* m) { return m && m->logits_f32() ? 1 : 0; }
 int32_t b2_model_is_quantized(const b2_model* m) { return m && m->quantized ? 1 : 0; }
 int64_t b2_model_weight_bytes(const b2_model* m) { return m ? m->weight_bytes : 0; }
 

@@ -19,6 +19,7 @@
 #include "engine.h"
 
 int32_t b2_cache_reserve(b2_cache* c, int n);
+void b2_cache_share_blocks(b2_cache* c, const int64_t* ids, int n);
 
 struct PrefixEntry {
     std::vector<int32_t> tokens;
@@ -75,16 +76,15 @@ int32_t b2_cache_fork(const b2_cache* src, int32_t len, b2_cache** out) {
     B2_REQUIRE(src && out, B2_ERR_MSG, "b2_cache_fork: null argument");
     B2_REQUIRE(len >= 0 && len <= src->len, B2_ERR_MSG, "b2_cache_fork: length beyond the source cache");
     b2_pool* p = src->pool;
+    B2_REQUIRE(p->state_floats == 0 || len == 0 || (len == src->len && src->state_len == len), B2_ERR_UNSUPPORTED,
+               "b2_cache_fork: a recurrent state exists only at the end of its sequence");
     const int bs = p->block_size;
     const int full = len / bs, rem = len % bs;
     b2_cache* c = nullptr;
     B2_CHECK(b2_cache_new(p, &c));
     if (full > 0) {
         // the first `full` blocks of the source are frozen (full) blocks with ids: share ids and pages
-        std::vector<int64_t> ids(src->block_ids.begin(), src->block_ids.begin() + full);
-        b2_cache_free(c);
-        c = nullptr;
-        B2_CHECK(b2_cache_new_seeded(p, ids.data(), full, &c));
+        b2_cache_share_blocks(c, src->block_ids.data(), full);
     }
     if (rem > 0) {
         // private copy of the boundary page: reserve a page for one more token, then copy the source's page over it
@@ -94,15 +94,13 @@ int32_t b2_cache_fork(const b2_cache* src, int32_t len, b2_cache** out) {
             return rc;
         }
         const int32_t fresh = c->pages[full], old = src->pages[full];
-        for (int l = 0; l < p->layers; l++) {
-            uint8_t* kl = reinterpret_cast<uint8_t*>(p->k_layer(l));
-            uint8_t* vl = reinterpret_cast<uint8_t*>(p->v_layer(l));
-            B2_CUDA(cudaMemcpyAsync(kl + (size_t)fresh * p->page_bytes(), kl + (size_t)old * p->page_bytes(), p->page_bytes(),
-                                    cudaMemcpyDeviceToDevice, p->ctx->stream));
-            B2_CUDA(cudaMemcpyAsync(vl + (size_t)fresh * p->page_bytes(), vl + (size_t)old * p->page_bytes(), p->page_bytes(),
-                                    cudaMemcpyDeviceToDevice, p->ctx->stream));
-        }
+        B2_CHECK(p->copy_page(old, fresh));
         c->len = len;
+    }
+    if (p->state_floats > 0 && len > 0) {
+        B2_CUDA(cudaMemcpyAsync(p->state + (size_t)c->slot * p->state_floats, p->state + (size_t)src->slot * p->state_floats, (size_t)p->state_floats * 4,
+                                cudaMemcpyDeviceToDevice, p->ctx->stream));
+        c->state_len = len;
     }
     *out = c;
     return B2_OK;
@@ -155,6 +153,7 @@ int32_t b2_generate_cached(b2_model* m, const b2_request* req, const volatile in
         const int lim = std::min({(int)e.tokens.size(), n_prompt, e.cache->len});
         while (common < lim && e.tokens[common] == req->prompt_ids[common]) common++;
         common = std::min(common, n_prompt - 1);
+        if (pc->pool->state_floats > 0 && common != e.cache->len) common = 0;  // a recurrent state is kept at the stored end only
         if (common > best_len || (common == best_len && common > 0 && e.used > pc->entries[best].used)) {
             best = (int)i;
             best_len = common;

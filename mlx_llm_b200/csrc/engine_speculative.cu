@@ -60,6 +60,8 @@ extern "C" int32_t b2_generate_prompt_lookup(b2_model* m, const b2_request* req,
     B2_REQUIRE(req->sampling.temperature <= 0.f && (req->sampling.repetition_penalty == 1.f || req->sampling.repetition_penalty == 0.f),
                B2_ERR_UNSUPPORTED, "only greedy sampling (temperature <= 0, repetition_penalty == 1) runs on the device path");
     if (cancel && *cancel) return b2_fail(B2_ERR_CANCELED, "canceled before inference");
+    B2_REQUIRE(b2_model_state_bytes(m) == 0, B2_ERR_UNSUPPORTED,
+               "speculative decoding: rejected drafts cannot be rolled back out of a recurrent state");
     b2_speculative_stats st{};
     std::vector<int32_t> gen;
     int finish = B2_FINISH_MAX_TOKENS;

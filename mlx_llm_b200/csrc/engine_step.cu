@@ -43,6 +43,10 @@ int32_t ensure_workspace(b2_model* m, int T, int B, int W, int P, size_t stage_i
     }
     if (grow_t) {
         const size_t t = (size_t)std::max(T, 64) * 5 / 4;
+        if (m->layered) {  // its activations live in an arena of its own (engine_layers.cu)
+            B2_CHECK(regrow(w.ids, t));
+            w.t_cap = (int)t;
+        } else {
         const size_t qkv_w = (size_t)(m->hq_l + 2 * m->hkv_l) * c.head_dim;
         if (!w.x_in_peer_region) B2_CHECK(regrow(w.x, t * c.hidden_size));
         B2_CHECK(regrow(w.xn, t * c.hidden_size));
@@ -54,11 +58,14 @@ int32_t ensure_workspace(b2_model* m, int T, int B, int W, int P, size_t stage_i
         if (m->tp && m->tp->world > 1) B2_CHECK(regrow(w.tp_part, t * c.hidden_size));
         B2_CHECK(regrow(w.ids, t));
         w.t_cap = (int)t;
+        }
     }
     if (grow_b) {
         const size_t b = (size_t)std::max(B, 16) * 5 / 4;
-        B2_CHECK(regrow(w.last, b * c.hidden_size));
-        B2_CHECK(regrow(w.logits, b * c.vocab_size));
+        if (!m->layered) {
+            B2_CHECK(regrow(w.last, b * c.hidden_size));
+            B2_CHECK(regrow(w.logits, b * c.vocab_size));
+        }
         B2_CHECK(regrow(w.argmax, b));
         if (w.argmax_host) cudaFreeHost(w.argmax_host);
         B2_CUDA(cudaHostAlloc((void**)&w.argmax_host, b * 4, cudaHostAllocDefault));
@@ -68,10 +75,12 @@ int32_t ensure_workspace(b2_model* m, int T, int B, int W, int P, size_t stage_i
     if (grow_p) w.p_cap = std::max(P, 64) * 5 / 4;
     if (grow_t || grow_b || grow_w || grow_p) {
         B2_CHECK(regrow(w.meta, (size_t)b2_batch_metadata_elems(w.b_cap, w.t_cap, w.w_cap, w.p_cap)));
-        const size_t sb = b2_decode_attn_scratch_bytes(w.w_cap, m->hq_l, c.head_dim);
-        if (w.attn_scratch) cudaFree(w.attn_scratch);
-        B2_CUDA(cudaMalloc((void**)&w.attn_scratch, sb));
-        w.attn_scratch_bytes = sb;
+        if (!m->layered) {
+            const size_t sb = b2_decode_attn_scratch_bytes(w.w_cap, m->hq_l, c.head_dim);
+            if (w.attn_scratch) cudaFree(w.attn_scratch);
+            B2_CUDA(cudaMalloc((void**)&w.attn_scratch, sb));
+            w.attn_scratch_bytes = sb;
+        }
     }
     if (stage_ints > w.stage_cap) {
         B2_CUDA(cudaStreamSynchronize(m->ctx->stream));
@@ -289,13 +298,22 @@ int32_t b2_engine_forward(b2_model* m, std::vector<SeqStep>& seqs, void* logits_
     int T = 0, max_pos = 0, n_logits = 0, n_dec = 0;
     long dec_ctx_sum = 0;
     const bool all_positions = seqs[0].all_positions;
+    bool listed = false;  // rows of the wanted positions come from the host instead of the packer
     B2_REQUIRE(!all_positions || B == 1, B2_ERR_MSG, "forward: logits of every position are available for a step of one sequence");
     for (auto& s : seqs) {
         B2_REQUIRE(s.cache && s.cache->pool == pool, B2_ERR_MSG, "forward: all caches of a step must share one pool");
         B2_REQUIRE(s.n > 0, B2_ERR_MSG, "forward: a sequence contributes no token");
         T += s.n;
         max_pos = std::max(max_pos, s.cache->len + s.n);
-        n_logits += s.want_logits ? 1 : 0;
+        B2_REQUIRE(s.cache->state_len == s.cache->len || s.cache->len == 0 || pool->state_floats == 0, B2_ERR_MSG,
+                   "forward: this cache's recurrent state is ahead of its tokens (an abandoned step); reset it");
+        if (s.n_want >= 0) {
+            listed = true;
+            B2_REQUIRE(s.n_want == 0 || s.want, B2_ERR_MSG, "forward: null list of wanted positions");
+            for (int i = 0; i < s.n_want; i++)
+                B2_REQUIRE(s.want[i] >= 0 && s.want[i] < s.n, B2_ERR_MSG, "forward: a wanted position lies outside the step's tokens");
+        }
+        n_logits += s.n_want >= 0 ? s.n_want : s.want_logits ? 1 : 0;
         if (s.n == 1) {
             n_dec++;
             dec_ctx_sum += s.cache->len + 1;
@@ -309,15 +327,22 @@ int32_t b2_engine_forward(b2_model* m, std::vector<SeqStep>& seqs, void* logits_
         }
     }
     ctx->pdl_consumers = T >= ctx->pdl_min_tokens;  // (see b2_launch_pdl)
-    B2_CHECK(b2_model_ensure_rope(m, max_pos));
+    B2_CHECK(m->layered ? b2_layered_ensure_rope(m, max_pos) : b2_model_ensure_rope(m, max_pos));
     // pages for the new tokens (host allocator), then the step descriptors
     for (auto& s : seqs) B2_CHECK(b2_cache_reserve(s.cache, s.n));
     const int chunk_tiles = pick_chunk_tiles(dec_ctx_sum, m->hkv_l, ctx->sm_count);
-    const int q_tile = b2_prefill_q_tile(ctx, c.head_dim);
+    const int q_tile = m->layered ? b2_layered_q_tile(m) : b2_prefill_q_tile(ctx, c.head_dim);
     int W = 0, P = 0;
     double pf_flops = 0;  // 4*hd*hq flops per (query, visible key) pair
     int pf_max_ctx = 0;   // longest context among the sequences that prefill in this step
+    int pf_tokens = 0, pf_ctx = 0;
+    double pf_pairs = 0;
     for (auto& s : seqs) {
+        if (s.n > 1) {
+            pf_pairs += (double)s.n * s.cache->len + 0.5 * (double)s.n * (s.n + 1);
+            pf_tokens += s.n;
+            pf_ctx += s.cache->len + s.n;
+        }
         if (s.n > 1) pf_max_ctx = std::max(pf_max_ctx, s.cache->len + s.n);
         if (s.n > 1) pf_flops += 4.0 * c.head_dim * m->hq_l * ((double)s.n * s.cache->len + 0.5 * (double)s.n * (s.n + 1));
         if (s.n == 1) {
@@ -329,7 +354,7 @@ int32_t b2_engine_forward(b2_model* m, std::vector<SeqStep>& seqs, void* logits_
     }
     if (all_positions) n_logits = T;  // rows 0..T-1 of the step, in order
     const int U = (int)pool->upd_slot.size();
-    const size_t stage_ints = 4 * (size_t)B + 3 * (size_t)U + (size_t)T;
+    const size_t stage_ints = 4 * (size_t)B + 3 * (size_t)U + (size_t)T + (listed ? (size_t)n_logits : 0);
     B2_CHECK(ensure_workspace(m, T, std::max(B, n_logits), W, P, stage_ints));
     Workspace& w = m->ws;
     int32_t* sh = w.stage_host;
@@ -349,6 +374,16 @@ int32_t b2_engine_forward(b2_model* m, std::vector<SeqStep>& seqs, void* logits_
         for (auto& s : seqs) {
             memcpy(ids, s.ids, (size_t)s.n * 4);
             ids += s.n;
+        }
+        if (listed) {  // behind the ids: the step's row of every wanted position, sequence by sequence
+            int row0 = 0;
+            for (auto& s : seqs) {
+                if (s.n_want >= 0)
+                    for (int i = 0; i < s.n_want; i++) *ids++ = row0 + s.want[i];
+                else if (s.want_logits)
+                    *ids++ = row0 + s.n - 1;
+                row0 += s.n;
+            }
         }
     }
     cudaStream_t st = ctx->stream;
@@ -383,25 +418,49 @@ int32_t b2_engine_forward(b2_model* m, std::vector<SeqStep>& seqs, void* logits_
     B2_CHECK(b2_batch_meta_launch(ctx, in, mo));
 
     float* logits_f32_dev = nullptr;
-    if (m->f32) {
-        B2_CHECK(b2_forward_f32(m, pool, mo, in.seq_slot, ids_dev, T, B, n_logits, all_positions ? nullptr : mo.logit_rows, max_pos, &logits_f32_dev));
+    int logits_ld = c.vocab_size;
+    const int32_t* logit_rows = all_positions ? nullptr : listed ? ids_dev + T : mo.logit_rows;
+    if (m->layered) {
+        LayeredStep ls{};
+        ls.mo = &mo;
+        ls.in = &in;
+        ls.ids_dev = ids_dev;
+        ls.T = T;
+        ls.B = B;
+        ls.n_dec = n_dec;
+        ls.dec_work = W;
+        ls.pf_work = P;
+        ls.chunk_tiles = chunk_tiles;
+        ls.max_ctx = max_pos;
+        ls.dec_ctx_sum = dec_ctx_sum;
+        ls.pf_pairs = pf_pairs;
+        ls.pf_tokens = pf_tokens;
+        ls.pf_ctx = pf_ctx;
+        ls.n_logits = n_logits;
+        ls.logit_rows = logit_rows;
+        if (pool->state_floats > 0)
+            for (auto& s : seqs) s.cache->state_len = -1;  // until the step has completed
+        B2_CHECK(b2_forward_layered(m, pool, ls, &logits_f32_dev, &logits_ld));
+    } else if (m->f32) {
+        B2_CHECK(b2_forward_f32(m, pool, mo, in.seq_slot, ids_dev, T, B, n_logits, logit_rows, max_pos, &logits_f32_dev));
     } else {
-        B2_CHECK(forward_bf16_layers(m, pool, mo, in, ids_dev, T, n_dec, dec_ctx_sum, W, P, pf_flops, pf_max_ctx, chunk_tiles, q_tile, n_logits,
-                                     all_positions ? nullptr : mo.logit_rows));
+        B2_CHECK(forward_bf16_layers(m, pool, mo, in, ids_dev, T, n_dec, dec_ctx_sum, W, P, pf_flops, pf_max_ctx, chunk_tiles, q_tile, n_logits, logit_rows));
     }
+    const int lsz = m->logits_f32() ? 4 : 2;
     if (n_logits > 0) {
         b2_prof_mark(ctx, B2_CLS_META);
         B2_CUDA(cudaMemcpyAsync(w.argmax_host, w.argmax, (size_t)n_logits * 4, cudaMemcpyDeviceToHost, st));
         m->d2h_bytes += (int64_t)n_logits * 4;
         if (logits_out) {
-            const size_t bytes = (size_t)n_logits * c.vocab_size * (m->f32 ? 4 : 2);
+            const size_t bytes = (size_t)n_logits * c.vocab_size * lsz;
             if (bytes > w.logits_host_cap) {
                 B2_CUDA(cudaStreamSynchronize(st));
                 if (w.logits_host) cudaFreeHost(w.logits_host);
                 B2_CUDA(cudaHostAlloc((void**)&w.logits_host, bytes, cudaHostAllocDefault));
                 w.logits_host_cap = bytes;
             }
-            B2_CUDA(cudaMemcpyAsync(w.logits_host, m->f32 ? (const void*)logits_f32_dev : (const void*)w.logits, bytes, cudaMemcpyDeviceToHost, st));
+            B2_CUDA(cudaMemcpy2DAsync(w.logits_host, (size_t)c.vocab_size * lsz, m->logits_f32() ? (const void*)logits_f32_dev : (const void*)w.logits,
+                                      (size_t)logits_ld * lsz, (size_t)c.vocab_size * lsz, (size_t)n_logits, cudaMemcpyDeviceToHost, st));
             m->d2h_bytes += (int64_t)bytes;
         }
     }
@@ -427,7 +486,7 @@ int32_t b2_engine_forward(b2_model* m, std::vector<SeqStep>& seqs, void* logits_
     }
     if (n_logits > 0) {
         if (argmax_out) memcpy(argmax_out, w.argmax_host, (size_t)n_logits * 4);
-        if (logits_out) memcpy(logits_out, w.logits_host, (size_t)n_logits * c.vocab_size * (m->f32 ? 4 : 2));
+        if (logits_out) memcpy(logits_out, w.logits_host, (size_t)n_logits * c.vocab_size * lsz);
     }
     for (auto& s : seqs) b2_cache_commit(s.cache, s.n);
     return B2_OK;
@@ -442,6 +501,24 @@ extern "C" int32_t b2_model_step(b2_model* m, const int32_t* ids_host, const int
         B2_REQUIRE(caches[i], B2_ERR_MSG, "b2_model_step: null cache");
         seqs.push_back(SeqStep{caches[i], cur, n_tokens[i], true});
         cur += n_tokens[i];
+    }
+    return b2_engine_forward(m, seqs, logits_host, argmax_host);
+}
+
+extern "C" int32_t b2_model_step_at(b2_model* m, const int32_t* ids_host, const int32_t* n_tokens, int32_t num_seqs, b2_cache** caches,
+                                    const int32_t* n_want, const int32_t* want, void* logits_host, int32_t* argmax_host) {
+    B2_REQUIRE(m && ids_host && n_tokens && caches && n_want, B2_ERR_MSG, "b2_model_step_at: null argument");
+    std::vector<SeqStep> seqs;
+    const int32_t *cur = ids_host, *w = want;
+    for (int i = 0; i < num_seqs; i++) {
+        B2_REQUIRE(caches[i], B2_ERR_MSG, "b2_model_step_at: null cache");
+        B2_REQUIRE(n_want[i] >= 0 && (n_want[i] == 0 || want), B2_ERR_MSG, "b2_model_step_at: bad list of wanted positions");
+        SeqStep s{caches[i], cur, n_tokens[i], n_want[i] > 0};
+        s.want = w;
+        s.n_want = n_want[i];
+        seqs.push_back(s);
+        cur += n_tokens[i];
+        w += n_want[i];
     }
     return b2_engine_forward(m, seqs, logits_host, argmax_host);
 }

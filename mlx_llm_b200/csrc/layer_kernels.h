@@ -1,0 +1,112 @@
+// Launch interfaces of the layered models' kernels.  `f32` selects the storage format of activations and weights
+// (false: bf16 bits, true: float); pointers to such storage are void*.  Row strides are in elements.
+#pragma once
+#include <stddef.h>
+#include <stdint.h>
+
+#include "model_spec.h"
+
+struct b2_ctx;
+
+// ---- layer_ops.cu ---------------------------------------------------------------------------------------------
+// x[t, :width] (f32 residual stream) = table[ids[t]]
+int32_t b2_embed_residual_launch(b2_ctx* ctx, bool f32, const void* table, int ld_table, const int32_t* ids, int T, int width, int vocab, float* x,
+                                 int ldx);
+struct AddNormParams {
+    float* x;               // [*, ldx] residual stream
+    const float* y;         // what the last sub-layer added (f32), null: nothing
+    const int32_t* y_rows;  // [T, n_src] rows of y summed (in order) into token t; null: row t
+    const float* w;         // norm weight [width]; null: only the addition
+    const int32_t* row_idx; // output row r takes source row row_idx[r]; null: r
+    void* out;              // [rows, ldo], zero beyond width
+    int ldx, ldy, ldo, rows, width, n_src;
+    float eps, out_scale;   // out = norm * w * out_scale
+    bool write_x;
+};
+int32_t b2_add_norm_launch(b2_ctx* ctx, bool f32, const AddNormParams& p);
+// out[r, j] = act(gu[r, j], gu[r, up_off + j]), the pre-activations scaled by row_w[r] when given; zero for j in [ff, ldo)
+int32_t b2_gate_launch(b2_ctx* ctx, bool f32, const GateSpec& g, const void* gu, int ldg, int up_off, const float* row_w, int rows, int ff, void* out,
+                       int ldo);
+int32_t b2_zero_cols_launch(b2_ctx* ctx, bool f32, void* x, int ldx, int c0, int c1, int rows);
+// y[M, N] = x[M, K] . W[N, K]^T in f32 (fused multiply-add, partial sums per 32 inputs)
+int32_t b2_linear_f32_launch(b2_ctx* ctx, const float* x, int ldx, const float* w, int M, int N, int K, float* y, int ldy);
+int32_t b2_argmax_f32_launch(b2_ctx* ctx, const float* logits, int ld, int rows, int vocab, int32_t* out);
+
+// ---- gemm_grouped.cu: one matrix product per group ---------------------------------------------------------------
+struct GroupedGemmParams {
+    const void* x;           // rows of group g: x + g * x_gstride + row * ldx
+    int64_t x_gstride;
+    int ldx;
+    const int32_t* row_idx;  // output row r reads x row row_idx[r] (routed experts); null: r
+    const void* w;           // [G][N][K]
+    int N, K, G;             // N, K padded (multiples of 64)
+    void* out;               // rows of group g: out + g * out_gstride + row * ldo
+    int64_t out_gstride;
+    int ldo, n_out;          // columns stored per row (<= N)
+    bool out_f32;            // f32 results from bf16 operands
+    const int32_t* offsets;  // [G + 1] device: group g owns rows [offsets[g], offsets[g + 1]); null: every group has rows 0..M-1
+    int M;                   // rows per group, or the total number of rows with `offsets`
+};
+int32_t b2_grouped_gemm_launch(b2_ctx* ctx, bool f32, const GroupedGemmParams& p);
+
+// ---- moe.cu -----------------------------------------------------------------------------------------------------
+struct RouteParams {
+    const float* logits;  // [T, ld]
+    int ld, T, experts, top;
+    int32_t* expert;      // [T, top] chosen experts, best first
+    float* weight;        // [T, top]
+    int32_t* offsets;     // [experts + 1]
+    int32_t* pos;         // [T, top] sorted position of each (token, choice)
+    int32_t* src;         // [T * top] token of each sorted position
+    float* row_w;         // [T * top] weight of each sorted position
+    int32_t* counters;    // [experts + 1], zero between launches
+};
+int32_t b2_route_launch(b2_ctx* ctx, const RouteParams& p);
+
+// ---- latent_attn.cu -----------------------------------------------------------------------------------------------
+struct LatentPrepParams {
+    const void* qkv;        // [T, ld]: q heads as [dim | rot_dim], then kv_rank latents, then rot_dim rotated-key inputs
+    int ld, T;
+    const int32_t* positions;
+    const int32_t* slot_mapping;
+    const float *cos_t, *sin_t;  // [positions, rot.dims / 2]
+    const float* c_norm;    // [kv_rank]
+    float eps;
+    void* cache;            // [page * page_size + offset][row_pad]
+    void* q_nope;           // [T, heads, dim_pad], zero beyond dim
+    int dim_pad;
+    void* q_lat;            // [T, heads, row_pad]: the rotated query part goes to columns kv_rank.., zero beyond row()
+};
+int32_t b2_latent_prep_launch(b2_ctx* ctx, bool f32, const LatentAttnSpec& a, const LatentPrepParams& p);
+struct LatentAttnParams {
+    const void* q_lat;      // [T, heads, row_pad] queries in latent coordinates | rotated part
+    const void* cache;
+    const int32_t* block_tables;
+    int max_blocks, page_size;
+    const int32_t* seq_slot;   // [B]
+    const int32_t* token_seq;  // [T]
+    const int32_t* positions;  // [T]
+    void* o_lat;            // [T, heads, o_pad] attention-weighted latents
+    int o_pad, T;
+};
+int32_t b2_latent_attn_simple_launch(b2_ctx* ctx, bool f32, const LatentAttnSpec& a, const LatentAttnParams& p);
+
+// ---- ssm.cu ---------------------------------------------------------------------------------------------------------
+struct SsmParams {
+    const void* zx;       // [T, ld]: z | x | B | C | dt
+    int ld, T, B;
+    const int32_t* cu_seqlens;    // [B + 1]
+    const int32_t* context_lens;  // [B], this step's tokens included
+    const int32_t* token_seq;     // [T]
+    const int32_t* seq_slot;      // [B]
+    float* state;         // slot s: state + s * slot_stride: heads x vdim x state, then channels x (conv - 1)
+    int64_t slot_stride;
+    const float *conv_w, *conv_b, *dt_bias, *A_log, *D, *norm;
+    float eps;
+    void* xbc;            // [T, channels] convolved inputs
+    int ld_xbc;
+    float* y;             // [T, inner]
+    void* out;            // [T, ldo] gated and normed, zero beyond inner
+    int ldo;
+};
+int32_t b2_ssm_launch(b2_ctx* ctx, bool f32, const Mamba2Spec& s, const SsmParams& p);

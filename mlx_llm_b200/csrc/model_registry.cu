@@ -1,0 +1,236 @@
+// Model families: which one a config.json names, and how a model of it is built.
+//
+// The Llama / Qwen3 families (src/config.rs:64-113 decides by `architectures` / `model_type`) are flat configurations
+// (b2_model_config); a layered family names itself in `architecture` and lists its layers, each with a mixer and a
+// feed-forward, which become a ModelSpec.  A new layered design whose mechanisms exist already is one more reader here.
+#include <cstring>
+#include <fstream>
+#include <sstream>
+
+#include "engine.h"
+#include "json_mini.h"
+
+namespace {
+
+using b2json::Value;
+
+struct Reader {  // typed access to one JSON object; remembers the first thing that was missing or malformed
+    std::string err;
+    const Value* obj(const Value* v, const char* key, const std::string& where) {
+        const Value* f = v ? v->get(key) : nullptr;
+        if (!f || f->kind != Value::Object) return fail("object", key, where), nullptr;
+        return f;
+    }
+    int num(const Value* v, const char* key, const std::string& where, int lo = 1) {
+        long long x = 0;
+        const Value* f = v ? v->get(key) : nullptr;
+        if (!f || !f->as_i64(x)) return fail("integer", key, where), 0;
+        if (x < lo || x > (1 << 30)) return fail("in-range integer", key, where), 0;
+        return (int)x;
+    }
+    double real(const Value* v, const char* key, const std::string& where) {
+        double x = 0;
+        const Value* f = v ? v->get(key) : nullptr;
+        if (!f || !f->as_f64(x)) fail("number", key, where);
+        return x;
+    }
+    std::string str(const Value* v, const char* key, const std::string& where) {
+        const Value* f = v ? v->get(key) : nullptr;
+        if (!f || f->kind != Value::String) return fail("string", key, where), std::string();
+        return f->str;
+    }
+    void require(bool ok, const std::string& what) {
+        if (!ok && err.empty()) err = "config.json: " + what;
+    }
+    void fail(const char* type, const char* key, const std::string& where) {
+        if (err.empty()) err = std::string("config.json: missing ") + type + " `" + key + "` in " + where;
+    }
+};
+
+// ---- mixers and feed-forwards by the name a layered config.json gives them ------------------------------------
+void read_latent_attention(Reader& r, const Value* m, const std::string& at, LayerSpec& L) {
+    LatentAttnSpec& a = L.attn;
+    L.mixer = MixerKind::LatentAttention;
+    a.heads = r.num(m, "heads", at);
+    a.dim = r.num(m, "dim", at);
+    a.rot_dim = r.num(m, "rot_dim", at);
+    a.vdim = r.num(m, "vdim", at);
+    a.kv_rank = r.num(m, "kv_rank", at);
+    a.scale = (float)r.real(m, "scale", at);
+    const Value* rot = r.obj(m, "rot", at);
+    a.rot.base = r.real(rot, "base", at + ".rot");
+    a.rot.dims = r.num(rot, "dims", at + ".rot");
+    r.require(a.rot.dims % 2 == 0 && a.rot.dims <= a.rot_dim, at + ": rot.dims must be even and at most rot_dim");
+    r.require(a.rot.base > 0, at + ": rot.base must be positive");
+}
+void read_mamba2(Reader& r, const Value* m, const std::string& at, LayerSpec& L) {
+    Mamba2Spec& s = L.ssm;
+    L.mixer = MixerKind::Mamba2;
+    s.heads = r.num(m, "heads", at);
+    s.vdim = r.num(m, "vdim", at);
+    s.state = r.num(m, "state", at);
+    s.groups = r.num(m, "groups", at);
+    s.norm_groups = r.num(m, "norm_groups", at);
+    s.conv = r.num(m, "conv", at);
+    if (!r.err.empty()) return;
+    r.require(s.heads % s.groups == 0, at + ": groups must divide heads");
+    r.require(s.inner() % s.norm_groups == 0, at + ": norm_groups must divide heads * vdim");
+}
+struct MixerReader {
+    const char* name;
+    void (*read)(Reader&, const Value*, const std::string&, LayerSpec&);
+};
+const MixerReader kMixers[] = {{"latent_attention", read_latent_attention}, {"mamba2", read_mamba2}};
+
+void read_mlp(Reader& r, const Value* mlp, const std::string& at, const GateSpec& dense, float expert_alpha, LayerSpec& L) {
+    if (!mlp || mlp->kind == Value::Null) {
+        L.mlp = MlpKind::None;
+        return;
+    }
+    const std::string kind = r.str(mlp, "kind", at);
+    if (kind == "dense") {
+        L.mlp = MlpKind::DenseGated;
+        L.ff = r.num(mlp, "ff", at);
+        L.gate = dense;
+    } else if (kind == "moe") {
+        L.mlp = MlpKind::Routed;
+        const Value* ro = r.obj(mlp, "router", at);
+        L.moe.experts = r.num(ro, "experts", at + ".router");
+        L.moe.top = r.num(ro, "top", at + ".router");
+        const Value* ex = r.obj(mlp, "expert", at);
+        L.moe.ff = r.num(ex, "ff", at + ".expert");
+        L.moe.gate.act = GateAct::ClippedSwish;
+        L.moe.gate.limit = (float)r.real(ex, "limit", at + ".expert");
+        L.moe.gate.alpha = expert_alpha;
+        r.require(L.moe.top <= L.moe.experts, at + ": more chosen experts than experts");
+    } else {
+        r.require(false, at + ": unknown feed-forward kind `" + kind + "`");
+    }
+}
+
+// ---- Zukitar: latent attention and Mamba-2 layers, dense GELU and clipped-swish routed feed-forwards, tied head -----
+constexpr float kZukitarExpertAlpha = 1.702f;
+bool claims_zukitar(const Value& v) {
+    const Value* a = v.get("architecture");
+    return a && a->kind == Value::String && a->str == "Zukitar";
+}
+int32_t read_zukitar(const Value& v, ModelSpec& spec) {
+    Reader r;
+    spec.family = "Zukitar";
+    spec.vocab = r.num(&v, "vocab", "the model");
+    spec.width = r.num(&v, "width", "the model");
+    spec.eps = (float)r.real(r.obj(&v, "norm", "the model"), "eps", "norm");
+    spec.logit_scale = (float)r.real(&v, "logit_scale", "the model");
+    const Value* ls = v.get("layers");
+    r.require(ls && ls->kind == Value::Array && !ls->arr.empty(), "`layers` must be a non-empty list");
+    if (r.err.empty())
+        for (size_t i = 0; i < ls->arr.size(); i++) {
+            const Value* lv = ls->arr[i].get();
+            const std::string at = "layers[" + std::to_string(i) + "]";
+            const std::string type = r.str(lv, "type", at);
+            LayerSpec L;
+            bool known = false;
+            for (auto& mr : kMixers)
+                if (type == mr.name) {
+                    mr.read(r, r.obj(lv, "mixer", at), at + ".mixer", L);
+                    known = true;
+                }
+            r.require(known, at + ": unknown mixer `" + type + "`");
+            read_mlp(r, lv->get("mlp"), at + ".mlp", GateSpec{GateAct::GeluTanh, 0.f, 0.f}, kZukitarExpertAlpha, L);
+            spec.layers.push_back(L);
+        }
+    B2_REQUIRE(r.err.empty(), B2_ERR_CONFIG, r.err);
+    return B2_OK;
+}
+
+// ---- the table ------------------------------------------------------------------------------------------------
+struct ModelFamily {
+    const char* name;
+    bool (*claims)(const Value& root);
+    int32_t (*read_layers)(const Value& root, ModelSpec& spec);  // null: a flat b2_model_config family
+};
+bool claims_flat(const Value&) { return true; }  // b2_model_config_from_json decides (and refuses what it does not know)
+const ModelFamily kFamilies[] = {{"Zukitar", claims_zukitar, read_zukitar}, {"llama", claims_flat, nullptr}};
+
+int32_t find_family(const char* json, b2json::ValuePtr& root, const ModelFamily** out) {
+    std::string err;
+    root = b2json::parse(json, err);
+    B2_REQUIRE(root && root->kind == Value::Object, B2_ERR_CONFIG, "config.json: " + (err.empty() ? std::string("not an object") : err));
+    const Value* a = root->get("architecture");
+    for (auto& f : kFamilies)
+        if (f.claims(*root)) {
+            B2_REQUIRE(f.read_layers || !(a && a->kind == Value::String), B2_ERR_UNSUPPORTED,
+                       "config.json: unknown architecture `" + (a ? a->str : std::string()) + "`");
+            *out = &f;
+            return B2_OK;
+        }
+    return b2_fail(B2_ERR_UNSUPPORTED, "config.json: no model family claims this configuration");
+}
+
+int32_t read_spec(const char* json, ModelSpec& spec, bool* layered) {
+    b2json::ValuePtr root;
+    const ModelFamily* f = nullptr;
+    B2_CHECK(find_family(json, root, &f));
+    *layered = f->read_layers != nullptr;
+    return *layered ? f->read_layers(*root, spec) : B2_OK;
+}
+
+}  // namespace
+
+extern "C" {
+
+int32_t b2_model_family_from_json(const char* json, char* out, int32_t cap) {
+    B2_REQUIRE(json && out && cap > 0, B2_ERR_MSG, "b2_model_family_from_json: null argument");
+    b2json::ValuePtr root;
+    const ModelFamily* f = nullptr;
+    B2_CHECK(find_family(json, root, &f));
+    ModelSpec spec;
+    b2_model_config c;
+    B2_CHECK(f->read_layers ? f->read_layers(*root, spec) : b2_model_config_from_json(json, &c));  // a malformed one is refused here too
+    strncpy(out, f->name, (size_t)cap - 1);
+    out[cap - 1] = 0;
+    return B2_OK;
+}
+
+int32_t b2_model_from_json(b2_ctx* ctx, const b2_weights* w, const char* prefix, const char* json, const b2_quant_spec* quant,
+                           int32_t compute_f32, b2_model** out) {
+    B2_REQUIRE(ctx && w && json && out, B2_ERR_MSG, "b2_model_from_json: null argument");
+    ModelSpec spec;
+    bool layered = false;
+    B2_CHECK(read_spec(json, spec, &layered));
+    if (layered) {
+        B2_REQUIRE(!quant, B2_ERR_UNSUPPORTED, spec.family + ": quantize-on-load is available for the flat families only");
+        return b2_model_build_layered(ctx, spec, w, prefix ? prefix : "", 0, compute_f32 != 0, out);
+    }
+    b2_model_config c;
+    B2_CHECK(b2_model_config_from_json(json, &c));
+    c.compute_f32 = compute_f32 ? 1 : 0;
+    return b2_model_from_weights(ctx, w, prefix, &c, quant, out);
+}
+
+int32_t b2_model_synthetic_json(b2_ctx* ctx, const char* json, uint64_t seed, b2_model** out) {
+    B2_REQUIRE(ctx && json && out, B2_ERR_MSG, "b2_model_synthetic_json: null argument");
+    ModelSpec spec;
+    bool layered = false;
+    B2_CHECK(read_spec(json, spec, &layered));
+    if (layered) return b2_model_build_layered(ctx, spec, nullptr, "", seed, false, out);
+    b2_model_config c;
+    B2_CHECK(b2_model_config_from_json(json, &c));
+    return b2_model_synthetic(ctx, &c, seed, out);
+}
+
+int32_t b2_model_open(b2_ctx* ctx, const char* dir, const b2_quant_spec* quant, int32_t compute_f32, b2_model** out) {
+    B2_REQUIRE(ctx && dir && out, B2_ERR_MSG, "b2_model_open: null argument");
+    const std::string path = std::string(dir) + "/config.json";
+    std::ifstream f(path);
+    B2_REQUIRE(f.good(), B2_ERR_IO, "cannot open " + path);
+    std::stringstream ss;
+    ss << f.rdbuf();
+    b2_weights* w = nullptr;
+    B2_CHECK(b2_weights_from_dir(dir, &w));
+    const int32_t rc = b2_model_from_json(ctx, w, "", ss.str().c_str(), quant, compute_f32, out);
+    b2_weights_free(w);
+    return rc;
+}
+
+}  // extern "C"

@@ -96,6 +96,15 @@ def model_config_from_json(text):
     return c
 
 
+def model_family(text):
+    """Name of the registered model family a config.json belongs to."""
+    if not isinstance(text, str):
+        text = json.dumps(text)
+    buf = C.create_string_buffer(64)
+    check(load().b2_model_family_from_json(text.encode(), buf, 64))
+    return buf.value.decode()
+
+
 def model_config(**kw):
     c = CModelConfig(rms_norm_eps=1e-5, rope_theta=500000.0, rope_factor=1.0, rope_low_freq_factor=1.0, rope_high_freq_factor=4.0,
                      rope_original_context=8192.0)
@@ -157,6 +166,65 @@ class CausalLm:
         check(load().b2_model_synthetic_tp(ctx.h, C.byref(config), C.c_uint64(seed), tp.h if tp is not None else None, C.byref(h)))
         return cls(ctx, h)
 
+    @classmethod
+    def from_json(cls, ctx, weights, config, prefix="", quant: Optional[QuantSpec] = None, f32=False):
+        """The model config.json describes, by the registry of model families (b2_model_from_json)."""
+        h = C.c_void_p()
+        q = C.byref(CQuantSpec(quant.group_size, quant.bits)) if quant else None
+        text = config if isinstance(config, str) else json.dumps(config)
+        check(load().b2_model_from_json(ctx.h, weights.h, prefix.encode(), text.encode(), q, int(bool(f32)), C.byref(h)))
+        return cls(ctx, h)
+
+    @classmethod
+    def open(cls, ctx, path, quant: Optional[QuantSpec] = None, f32=False):
+        """... from a folder with config.json and *.safetensors."""
+        h = C.c_void_p()
+        q = C.byref(CQuantSpec(quant.group_size, quant.bits)) if quant else None
+        check(load().b2_model_open(ctx.h, str(path).encode(), q, int(bool(f32)), C.byref(h)))
+        return cls(ctx, h)
+
+    @classmethod
+    def synthetic_json(cls, ctx, config, seed=0):
+        h = C.c_void_p()
+        text = config if isinstance(config, str) else json.dumps(config)
+        check(load().b2_model_synthetic_json(ctx.h, text.encode(), C.c_uint64(seed), C.byref(h)))
+        return cls(ctx, h)
+
+    def logits_f32(self):
+        """True when logits rows are float32 (f32 models and layered models), False for bf16 bit patterns."""
+        return bool(load().b2_model_logits_f32(self.h))
+
+    def state_bytes(self):
+        """Bytes of recurrent state per sequence (0 for pure attention models)."""
+        lib = load()
+        lib.b2_model_state_bytes.restype = C.c_int64
+        return int(lib.b2_model_state_bytes(self.h))
+
+    def step_at(self, seqs, wants):
+        """One ragged forward with the logits of listed places: wants[i] holds places (0-based) among sequence i's new
+        tokens.  Returns (logits [sum of wants, vocab] as float32, argmax)."""
+        ids = np.concatenate([np.ascontiguousarray(s[0], np.int32) for s in seqs])
+        n = np.array([len(s[0]) for s in seqs], np.int32)
+        nw = np.array([len(w) for w in wants], np.int32)
+        flat = np.array([p for w in wants for p in w], np.int32)
+        arr = (C.c_void_p * len(seqs))(*[s[1].h for s in seqs])
+        f32 = self.logits_f32()
+        rows = int(nw.sum())
+        logits = np.empty((rows, self.config().vocab_size), np.float32 if f32 else np.uint16)
+        am = np.empty(max(rows, 1), np.int32)
+        vp = lambda a: a.ctypes.data_as(C.c_void_p)
+        check(load().b2_model_step_at(self.h, vp(ids), vp(n), len(seqs), arr, vp(nw), vp(flat), vp(logits) if rows else None, vp(am)))
+        if not f32:
+            logits = (logits.astype(np.uint32) << 16).view(np.float32)
+        return logits, am[:rows]
+
+    def capture_residual(self, buf):
+        """After every following step `buf` (float32, [layers, tokens, width]) holds the residual stream behind each layer;
+        None switches it off."""
+        self._capture = buf
+        check(load().b2_model_capture_residual(self.h, buf.ctypes.data_as(C.c_void_p) if buf is not None else None,
+                                               C.c_int64(buf.size if buf is not None else 0)))
+
     def config(self):
         c = CModelConfig()
         check(load().b2_model_get_config(self.h, C.byref(c)))
@@ -182,7 +250,7 @@ class CausalLm:
         arr = (C.c_void_p * len(seqs))(*[s[1].h for s in seqs])
         cfg = self.config()
         vocab = cfg.vocab_size
-        logits = np.empty((len(seqs), vocab), np.float32 if cfg.compute_f32 else np.uint16) if want_logits else None
+        logits = np.empty((len(seqs), vocab), np.float32 if self.logits_f32() else np.uint16) if want_logits else None
         am = np.empty(len(seqs), np.int32)
         check(load().b2_model_step(self.h, ids.ctypes.data_as(C.c_void_p), n.ctypes.data_as(C.c_void_p), len(seqs), arr,
                                    logits.ctypes.data_as(C.c_void_p) if want_logits else None, am.ctypes.data_as(C.c_void_p)))
@@ -640,7 +708,7 @@ class CProfile(C.Structure):
                 ("attn_decode_bytes", C.c_double), ("attn_prefill_flops", C.c_double)]
 
 
-PROFILE_CLASSES = ["gemm", "attn_decode", "attn_prefill", "rope_kv", "elementwise", "meta_copies", "collective"]
+PROFILE_CLASSES = ["gemm", "attn_decode", "attn_prefill", "rope_kv", "elementwise", "meta_copies", "collective", "recurrent"]
 
 
 def profile_enable(ctx, on=True):
