@@ -217,10 +217,12 @@ struct LayeredStep {
     int T, B, n_dec, dec_work, pf_work, chunk_tiles, max_ctx;
     long dec_ctx_sum;
     double pf_pairs;  // (query, visible key) pairs of the prefilling sequences
-    int pf_tokens, pf_ctx;  // their new tokens and their contexts, summed
+    int pf_ctx;                 // their contexts (this step's tokens included), summed
+    const int32_t* pf_kv_off;   // [B] device: running sum of those contexts, -1 for sequences with a single token
     int n_logits;
     const int32_t* logit_rows;
 };
 int32_t b2_forward_layered(b2_model* m, b2_pool* pool, const LayeredStep& s, float** logits_dev, int* logits_ld);
 int b2_layered_q_tile(const b2_model* m);
+int b2_layered_chunk_tiles(const b2_model* m, long dec_ctx_sum);  // 16-key tiles per work item of the decode attention
 bool b2_tensor_to_f32(const HostTensor& t, std::vector<float>& out);

@@ -28,6 +28,7 @@ struct LayerP {
     Proj qkv, attn_o;  // rows: q | latent | rotated key part
     float* c_norm = nullptr;
     GroupW k_up_t, v_up;  // [head][kv_rank][dim] and [head][vdim][kv_rank]
+    Proj kv_up;           // the same matrices for whole contexts (bf16): plain keys, then values, heads padded to 64-row blocks
     int rope = -1;
     // mamba2
     Proj ssm_in, ssm_o;
@@ -53,6 +54,14 @@ struct LayeredModel {
     int rope_positions = 0;
     int64_t state_floats = 0;
     int* route_counters = nullptr;
+    // prefill attention: gathered latents, rotated key parts and expanded keys / values of the contexts in a step
+    uint16_t *kv_lat = nullptr, *kv_rot = nullptr, *kv_exp = nullptr;
+    int kv_cap = 0, kv_ld_lat = 0, kv_ld_rot = 0, kv_ld_exp = 0;  // rows; widest rows over the layers
+    // decode attention: partial results per work item, arrival counters per row
+    float* dec_part = nullptr;
+    size_t dec_part_floats = 0, dec_part_row = 0;  // capacity; heads * (kv_rank + 2) of the largest layer
+    int* dec_counters = nullptr;
+    int dec_counters_cap = 0;
     uint8_t* arena = nullptr;
     int t_cap = 0, l_cap = 0;
     float* capture = nullptr;
@@ -145,6 +154,18 @@ struct Filler {
         B2_CHECK(fetch(key, {rows, cols}));
         return put(host.data(), rows, cols, dst, p.K);
     }
+    // tensor [parts * part_rows, cols]: part i to rows row0 + i * stride of p
+    int32_t rows_split(Proj& p, int row0, int stride, const std::string& key, int parts, int part_rows, int cols) {
+        if (w) B2_CHECK(fetch(key, {(int64_t)parts * part_rows, cols}));
+        for (int i = 0; i < parts; i++) {
+            void* dst = at(p.w, (int64_t)(row0 + i * stride) * p.K);
+            if (w)
+                B2_CHECK(put(host.data() + (size_t)i * part_rows * cols, part_rows, cols, dst, p.K));
+            else
+                B2_CHECK(random(dst, m->f32, part_rows, cols, p.K, 0.f, 1.0f / sqrtf((float)cols)));
+        }
+        return B2_OK;
+    }
     int32_t vec(float*& dst, const std::string& key, std::vector<int64_t> shape, float mean, float sd) {
         int64_t n = 1;
         for (auto d : shape) n *= d;
@@ -207,6 +228,16 @@ int32_t load_layer(Filler& f, LayeredModel& lm, int i) {
         B2_CHECK(f.group_split(P.k_up_t, mix("uk"), a.dim, a.kv_rank, true));
         B2_CHECK(f.group(P.v_up, a.heads, a.vdim, a.kv_rank));
         B2_CHECK(f.group_split(P.v_up, mix("uv"), a.vdim, a.kv_rank, false));
+        if (!f.m->f32 && b2_latent_prefill_eligible(a)) {
+            const int kb = up(a.dim, 64), vb = up(a.vdim, 64), v0 = a.heads * kb;
+            B2_CHECK(f.proj(P.kv_up, v0 + a.heads * vb, a.kv_rank));
+            B2_CHECK(f.rows_split(P.kv_up, 0, kb, mix("uk"), a.heads, a.dim, a.kv_rank));
+            B2_CHECK(f.rows_split(P.kv_up, v0, vb, mix("uv"), a.heads, a.vdim, a.kv_rank));
+            lm.kv_ld_lat = std::max(lm.kv_ld_lat, P.kv_up.K);
+            lm.kv_ld_rot = std::max(lm.kv_ld_rot, up(a.rot_dim, 64));
+            lm.kv_ld_exp = std::max(lm.kv_ld_exp, P.kv_up.N);
+        }
+        lm.dec_part_row = std::max(lm.dec_part_row, (size_t)a.heads * (a.kv_rank + 2));
         B2_CHECK(f.proj(P.attn_o, W, a.heads * a.vdim));
         B2_CHECK(f.rows(P.attn_o, 0, mix("o"), W, a.heads * a.vdim));
         for (size_t r = 0; r < lm.ropes.size(); r++)
@@ -276,8 +307,8 @@ struct Common {
     int ldx, ldn, ldl;
 };
 struct LatentBufs {
-    void *qkv, *q_nope, *q_lat, *o_lat, *att;
-    int dim_pad, o_pad, ld_att;
+    void *qkv, *q, *q_lat, *o_lat, *att;
+    int plain_pad, rot_pad, o_pad, ld_att;
 };
 struct SsmBufs {
     void *zx, *xbc, *gn;
@@ -311,11 +342,12 @@ Common carve_common(Carver& c, const LayeredModel& lm, size_t es, size_t t, size
 }
 LatentBufs carve_latent(Carver c, const LatentAttnSpec& a, const LayerP& P, size_t es, size_t t, size_t* end) {
     LatentBufs o;
-    o.dim_pad = P.k_up_t.K;
+    o.plain_pad = P.k_up_t.K;
+    o.rot_pad = up(a.rot_dim, 64);
     o.o_pad = P.v_up.K;
     o.ld_att = P.attn_o.K;
     o.qkv = c.take(t * P.qkv.N * es);
-    o.q_nope = c.take(t * a.heads * o.dim_pad * es);
+    o.q = c.take(t * a.heads * (o.plain_pad + o.rot_pad) * es);
     o.q_lat = c.take(t * a.heads * a.row_pad() * es);
     o.o_lat = c.take(t * a.heads * o.o_pad * es);
     o.att = c.take(t * o.ld_att * es);
@@ -388,6 +420,44 @@ int32_t ensure_arena(b2_model* m, int T, int n_logits) {
     return B2_OK;
 }
 
+constexpr size_t kMaxExpandBytes = 8ull << 30;  // expanded keys and values of one layer; longer contexts stay latent
+
+template <typename T>
+int32_t regrow_zero(b2_ctx* ctx, T*& p, size_t elems) {
+    if (p) B2_CUDA(cudaFree(p));
+    p = nullptr;
+    B2_CUDA(cudaMalloc((void**)&p, elems * sizeof(T)));
+    B2_CUDA(cudaMemsetAsync(p, 0, elems * sizeof(T), ctx->stream));
+    return B2_OK;
+}
+// Buffers of their own, not parts of the arena: rows past the contexts in use are read with weight zero, so they must
+// never hold anything but bf16 numbers.
+int32_t ensure_expand(b2_model* m, int rows) {
+    LayeredModel& lm = *m->layered;
+    if (rows <= lm.kv_cap) return B2_OK;
+    B2_CUDA(cudaStreamSynchronize(m->ctx->stream));
+    lm.kv_cap = up(std::max(rows + rows / 8, 1024), 128);
+    B2_CHECK(regrow_zero(m->ctx, lm.kv_lat, (size_t)lm.kv_cap * lm.kv_ld_lat));
+    B2_CHECK(regrow_zero(m->ctx, lm.kv_rot, (size_t)lm.kv_cap * lm.kv_ld_rot));
+    return regrow_zero(m->ctx, lm.kv_exp, (size_t)lm.kv_cap * lm.kv_ld_exp);
+}
+int32_t ensure_decode(b2_model* m, int items, int counters) {
+    LayeredModel& lm = *m->layered;
+    const size_t need = (size_t)items * lm.dec_part_row;
+    if (need > lm.dec_part_floats || counters > lm.dec_counters_cap) {
+        B2_CUDA(cudaStreamSynchronize(m->ctx->stream));
+        if (need > lm.dec_part_floats) {
+            lm.dec_part_floats = need * 5 / 4;
+            B2_CHECK(regrow_zero(m->ctx, lm.dec_part, lm.dec_part_floats));
+        }
+        if (counters > lm.dec_counters_cap) {
+            lm.dec_counters_cap = counters * 5 / 4 + 64;
+            B2_CHECK(regrow_zero(m->ctx, lm.dec_counters, (size_t)lm.dec_counters_cap));
+        }
+    }
+    return B2_OK;
+}
+
 // ---- forward --------------------------------------------------------------------------------------------------------
 int32_t linear(b2_model* m, const Proj& p, const void* x, int ldx, int M, int rows_cap, void* out, int ldo, bool out_f32) {
     b2_prof_mark(m->ctx, B2_CLS_GEMM);
@@ -430,7 +500,9 @@ int32_t Fwd::latent(const LayerSpec& L, const LayerP& P, int l) {
     b2_ctx* ctx = m->ctx;
     const LatentAttnSpec& a = L.attn;
     const LatentBufs b = carve_latent(scratch, a, P, es, (size_t)lm.t_cap, &end);
-    const int T = s.T, W = a.row_pad();
+    const int T = s.T, W = a.row_pad(), q_row = b.plain_pad + b.rot_pad;
+    const float scale_log2 = a.scale * 1.4426950408889634f;
+    void* cache = pool->planes[pool->layer_plane[l]].base;
     B2_CHECK(linear(m, P.qkv, c.xn, c.ldn, T, lm.t_cap, b.qkv, P.qkv.N, false));
     LatentPrepParams pp{};
     pp.qkv = b.qkv;
@@ -442,56 +514,150 @@ int32_t Fwd::latent(const LayerSpec& L, const LayerP& P, int l) {
     pp.sin_t = lm.ropes[P.rope].sin;
     pp.c_norm = P.c_norm;
     pp.eps = lm.spec.eps;
-    pp.cache = pool->planes[pool->layer_plane[l]].base;
-    pp.q_nope = b.q_nope;
-    pp.dim_pad = b.dim_pad;
+    pp.cache = cache;
+    pp.q = b.q;
+    pp.plain_pad = b.plain_pad;
+    pp.rot_pad = b.rot_pad;
     pp.q_lat = b.q_lat;
     b2_prof_mark(ctx, B2_CLS_ROPE_KV);
     B2_CHECK(b2_latent_prep_launch(ctx, m->f32, a, pp));
-    GroupedGemmParams g{};
-    g.x = b.q_nope;
-    g.x_gstride = b.dim_pad;
-    g.ldx = a.heads * b.dim_pad;
-    g.w = P.k_up_t.w;
-    g.N = P.k_up_t.N;
-    g.K = P.k_up_t.K;
-    g.G = a.heads;
-    g.out = b.q_lat;
-    g.out_gstride = W;
-    g.ldo = a.heads * W;
-    g.n_out = a.kv_rank;
-    g.M = T;
-    b2_prof_mark(ctx, B2_CLS_GEMM);
-    B2_CHECK(b2_grouped_gemm_launch(ctx, m->f32, g));
-    LatentAttnParams ap{};
-    ap.q_lat = b.q_lat;
-    ap.cache = pp.cache;
-    ap.block_tables = pool->block_tables;
-    ap.max_blocks = pool->max_blocks;
-    ap.page_size = pool->block_size;
-    ap.seq_slot = s.in->seq_slot;
-    ap.token_seq = s.mo->token_seq;
-    ap.positions = s.mo->positions;
-    ap.o_lat = b.o_lat;
-    ap.o_pad = b.o_pad;
-    ap.T = T;
-    b2_prof_mark(ctx, B2_CLS_ATTN_PREFILL);
-    B2_CHECK(b2_latent_attn_simple_launch(ctx, m->f32, a, ap));
-    GroupedGemmParams v{};
-    v.x = b.o_lat;
-    v.x_gstride = b.o_pad;
-    v.ldx = a.heads * b.o_pad;
-    v.w = P.v_up.w;
-    v.N = P.v_up.N;
-    v.K = P.v_up.K;
-    v.G = a.heads;
-    v.out = b.att;
-    v.out_gstride = a.vdim;
-    v.ldo = b.ld_att;
-    v.n_out = a.vdim;
-    v.M = T;
-    b2_prof_mark(ctx, B2_CLS_GEMM);
-    B2_CHECK(b2_grouped_gemm_launch(ctx, m->f32, v));
+
+    // Portions of more than a token: keys and values of their contexts expanded per head.  Otherwise (single tokens, f32,
+    // head sizes or contexts outside that kernel's reach) attention in latent coordinates.
+    const bool expand = s.pf_work > 0 && P.kv_up.w && (size_t)s.pf_ctx * P.kv_up.N * 2 <= kMaxExpandBytes;
+    if (expand) {
+        B2_CHECK(ensure_expand(m, s.pf_ctx));
+        LatentGatherParams gp{};
+        gp.cache = cache;
+        gp.block_tables = pool->block_tables;
+        gp.max_blocks = pool->max_blocks;
+        gp.page_size = pool->block_size;
+        gp.B = s.B;
+        gp.rows = s.pf_ctx;
+        gp.seq_slot = s.in->seq_slot;
+        gp.context_lens = s.mo->context_lens;
+        gp.kv_off = s.pf_kv_off;
+        gp.lat = lm.kv_lat;
+        gp.ld_lat = P.kv_up.K;
+        gp.rot = lm.kv_rot;
+        gp.rot_pad = b.rot_pad;
+        B2_CHECK(b2_latent_gather_launch(ctx, a, gp));
+        B2_CHECK(linear(m, P.kv_up, lm.kv_lat, P.kv_up.K, s.pf_ctx, lm.kv_cap, lm.kv_exp, P.kv_up.N, false));
+        LatentPrefillParams fp{};
+        fp.q = b.q;
+        fp.q_rows = lm.t_cap;
+        fp.kv = lm.kv_exp;
+        fp.rot = lm.kv_rot;
+        fp.kv_rows = lm.kv_cap;
+        fp.ld_kv = P.kv_up.N;
+        fp.v_col0 = a.heads * b.plain_pad;
+        fp.plain_blocks = b.plain_pad / 64;
+        fp.pf_seq = s.mo->pf_seq;
+        fp.pf_qstart = s.mo->pf_qstart;
+        fp.n_work = s.mo->counts + 3;
+        fp.cu_seqlens = s.mo->cu_seqlens;
+        fp.context_lens = s.mo->context_lens;
+        fp.kv_off = s.pf_kv_off;
+        fp.scale_log2 = scale_log2;
+        fp.out = b.att;
+        fp.ldo = b.ld_att;
+        fp.vdim = a.vdim;
+        b2_prof_mark(ctx, B2_CLS_ATTN_PREFILL);
+        B2_CHECK(b2_latent_prefill_launch(ctx, a, fp, s.pf_work));
+        ctx->attn_prefill_flops += 2.0 * (a.dim + a.rot_dim + a.vdim) * a.heads * s.pf_pairs;
+    }
+    // rows that attend in latent coordinates: the single tokens, or every token
+    const int rows = expand ? s.n_dec : T;
+    const bool listed = rows == s.n_dec;  // the packer's decode list describes them
+    const int32_t* row_idx = rows < T ? s.mo->dec_qrow : nullptr;
+    if (rows > 0) {
+        GroupedGemmParams g{};
+        g.x = b.q;
+        g.x_gstride = q_row;
+        g.ldx = a.heads * q_row;
+        g.row_idx = row_idx;
+        g.map_out = row_idx != nullptr;
+        g.w = P.k_up_t.w;
+        g.N = P.k_up_t.N;
+        g.K = P.k_up_t.K;
+        g.G = a.heads;
+        g.out = b.q_lat;
+        g.out_gstride = W;
+        g.ldo = a.heads * W;
+        g.n_out = a.kv_rank;
+        g.M = rows;
+        b2_prof_mark(ctx, B2_CLS_GEMM);
+        B2_CHECK(b2_grouped_gemm_launch(ctx, m->f32, g));
+        if (!m->f32 && b2_latent_decode_eligible(a)) {
+            LatentDecodeParams dp{};
+            dp.q_lat = b.q_lat;
+            dp.cache = cache;
+            dp.block_tables = pool->block_tables;
+            dp.max_blocks = pool->max_blocks;
+            dp.page_size = pool->block_size;
+            int items = rows;
+            if (listed) {
+                dp.ctx = s.mo->dec_ctx;
+                dp.qrow = s.mo->dec_qrow;
+                dp.slot = s.mo->dec_slot;
+                dp.work_seq = s.mo->dec_work_seq;
+                dp.work_chunk = s.mo->dec_work_chunk;
+                dp.work_off = s.mo->dec_work_off;
+                dp.n_work = s.mo->counts + 2;
+                dp.chunk_tiles = s.chunk_tiles;
+                items = s.dec_work;
+                B2_CHECK(ensure_decode(m, items, rows * b2_latent_decode_head_groups(a)));
+                dp.part_o = lm.dec_part;
+                dp.part_ml = lm.dec_part + (size_t)items * a.heads * a.kv_rank;
+                dp.counters = lm.dec_counters;
+                ctx->attn_decode_bytes += (double)s.dec_ctx_sum * W * 2;
+            } else {  // one work item per token: nothing is split, no partial results
+                dp.positions = s.mo->positions;
+                dp.token_seq = s.mo->token_seq;
+                dp.seq_slot = s.in->seq_slot;
+                dp.max_chunks = 1;
+                dp.chunk_tiles = (s.max_ctx + 15) / 16;
+            }
+            dp.scale_log2 = scale_log2;
+            dp.o_lat = b.o_lat;
+            dp.o_pad = b.o_pad;
+            b2_prof_mark(ctx, B2_CLS_ATTN_DECODE);
+            B2_CHECK(b2_latent_decode_launch(ctx, a, dp, items));
+        } else {
+            LatentAttnParams ap{};
+            ap.q_lat = b.q_lat;
+            ap.cache = cache;
+            ap.block_tables = pool->block_tables;
+            ap.max_blocks = pool->max_blocks;
+            ap.page_size = pool->block_size;
+            ap.seq_slot = s.in->seq_slot;
+            ap.token_seq = s.mo->token_seq;
+            ap.positions = s.mo->positions;
+            ap.row_idx = row_idx;
+            ap.o_lat = b.o_lat;
+            ap.o_pad = b.o_pad;
+            ap.T = rows;
+            b2_prof_mark(ctx, B2_CLS_ATTN_DECODE);
+            B2_CHECK(b2_latent_attn_simple_launch(ctx, m->f32, a, ap));
+        }
+        GroupedGemmParams v{};
+        v.x = b.o_lat;
+        v.x_gstride = b.o_pad;
+        v.ldx = a.heads * b.o_pad;
+        v.row_idx = row_idx;
+        v.map_out = row_idx != nullptr;
+        v.w = P.v_up.w;
+        v.N = P.v_up.N;
+        v.K = P.v_up.K;
+        v.G = a.heads;
+        v.out = b.att;
+        v.out_gstride = a.vdim;
+        v.ldo = b.ld_att;
+        v.n_out = a.vdim;
+        v.M = rows;
+        b2_prof_mark(ctx, B2_CLS_GEMM);
+        B2_CHECK(b2_grouped_gemm_launch(ctx, m->f32, v));
+    }
     B2_CHECK(b2_zero_cols_launch(ctx, m->f32, b.att, b.ld_att, a.heads * a.vdim, b.ld_att, T));
     return linear(m, P.attn_o, b.att, b.ld_att, T, lm.t_cap, c.y, c.ldx, true);
 }
@@ -592,7 +758,12 @@ int32_t Fwd::moe(const LayerSpec& L, const LayerP& P, const int32_t** rows) {
 
 }  // namespace
 
-int b2_layered_q_tile(const b2_model*) { return 64; }
+int b2_layered_q_tile(const b2_model*) { return 128; }
+int b2_layered_chunk_tiles(const b2_model* m, long dec_ctx_sum) {
+    // about three CTAs per SM (one is resident), 128 to 2048 keys each, whole 64-key tiles
+    const long keys = dec_ctx_sum / (3l * m->ctx->sm_count);
+    return up((int)std::min(2048l, std::max(128l, keys)), 64) / 16;
+}
 
 void b2_layered_cache_layout(const b2_model* m, int block_size, std::vector<std::vector<size_t>>& page_bytes, int64_t& state_floats) {
     for (auto& L : m->layered->spec.layers) {
@@ -679,7 +850,8 @@ void b2_layered_release(b2_model* m) {
         if (r.sin) cudaFree(r.sin);
     }
     if (lm.route_counters) cudaFree(lm.route_counters);
-    if (lm.arena) cudaFree(lm.arena);
+    for (void* p : {(void*)lm.arena, (void*)lm.kv_lat, (void*)lm.kv_rot, (void*)lm.kv_exp, (void*)lm.dec_part, (void*)lm.dec_counters})
+        if (p) cudaFree(p);
     delete m->layered;
     m->layered = nullptr;
 }

@@ -330,17 +330,16 @@ int32_t b2_engine_forward(b2_model* m, std::vector<SeqStep>& seqs, void* logits_
     B2_CHECK(m->layered ? b2_layered_ensure_rope(m, max_pos) : b2_model_ensure_rope(m, max_pos));
     // pages for the new tokens (host allocator), then the step descriptors
     for (auto& s : seqs) B2_CHECK(b2_cache_reserve(s.cache, s.n));
-    const int chunk_tiles = pick_chunk_tiles(dec_ctx_sum, m->hkv_l, ctx->sm_count);
+    const int chunk_tiles = m->layered ? b2_layered_chunk_tiles(m, dec_ctx_sum) : pick_chunk_tiles(dec_ctx_sum, m->hkv_l, ctx->sm_count);
     const int q_tile = m->layered ? b2_layered_q_tile(m) : b2_prefill_q_tile(ctx, c.head_dim);
     int W = 0, P = 0;
     double pf_flops = 0;  // 4*hd*hq flops per (query, visible key) pair
     int pf_max_ctx = 0;   // longest context among the sequences that prefill in this step
-    int pf_tokens = 0, pf_ctx = 0;
+    int pf_ctx = 0;
     double pf_pairs = 0;
     for (auto& s : seqs) {
         if (s.n > 1) {
             pf_pairs += (double)s.n * s.cache->len + 0.5 * (double)s.n * (s.n + 1);
-            pf_tokens += s.n;
             pf_ctx += s.cache->len + s.n;
         }
         if (s.n > 1) pf_max_ctx = std::max(pf_max_ctx, s.cache->len + s.n);
@@ -354,7 +353,7 @@ int32_t b2_engine_forward(b2_model* m, std::vector<SeqStep>& seqs, void* logits_
     }
     if (all_positions) n_logits = T;  // rows 0..T-1 of the step, in order
     const int U = (int)pool->upd_slot.size();
-    const size_t stage_ints = 4 * (size_t)B + 3 * (size_t)U + (size_t)T + (listed ? (size_t)n_logits : 0);
+    const size_t stage_ints = 4 * (size_t)B + 3 * (size_t)U + (size_t)T + (listed ? (size_t)n_logits : 0) + (m->layered ? (size_t)B : 0);
     B2_CHECK(ensure_workspace(m, T, std::max(B, n_logits), W, P, stage_ints));
     Workspace& w = m->ws;
     int32_t* sh = w.stage_host;
@@ -383,6 +382,13 @@ int32_t b2_engine_forward(b2_model* m, std::vector<SeqStep>& seqs, void* logits_
                 else if (s.want_logits)
                     *ids++ = row0 + s.n - 1;
                 row0 += s.n;
+            }
+        }
+        if (m->layered) {  // first row of every prefilling sequence among the gathered context rows
+            int row0 = 0;
+            for (auto& s : seqs) {
+                *ids++ = s.n > 1 ? row0 : -1;
+                if (s.n > 1) row0 += s.cache->len + s.n;
             }
         }
     }
@@ -434,8 +440,8 @@ int32_t b2_engine_forward(b2_model* m, std::vector<SeqStep>& seqs, void* logits_
         ls.max_ctx = max_pos;
         ls.dec_ctx_sum = dec_ctx_sum;
         ls.pf_pairs = pf_pairs;
-        ls.pf_tokens = pf_tokens;
         ls.pf_ctx = pf_ctx;
+        ls.pf_kv_off = ids_dev + T + (listed ? n_logits : 0);
         ls.n_logits = n_logits;
         ls.logit_rows = logit_rows;
         if (pool->state_floats > 0)

@@ -102,7 +102,8 @@ __global__ void __launch_bounds__(kThreads) grouped_tile_kernel(const GroupedGem
             for (int e = 0; e < 4; e++) {
                 const int r = mt * 16 + (lane >> 2) + (e >> 1) * 8, n = n0 + warp * 16 + nt * 8 + 2 * (lane & 3) + (e & 1);
                 if (r >= rows || n >= p.n_out) continue;
-                const size_t o = (size_t)g * p.out_gstride + (size_t)(r0 + r) * p.ldo + n;
+                const int orow = p.map_out ? p.row_idx[r0 + r] : r0 + r;
+                const size_t o = (size_t)g * p.out_gstride + (size_t)orow * p.ldo + n;
                 if (F32OUT)
                     reinterpret_cast<float*>(p.out)[o] = acc[mt][nt][e];
                 else
@@ -133,7 +134,7 @@ __global__ void __launch_bounds__(256) grouped_f32_kernel(const GroupedGemmParam
         acc += part;
         __syncthreads();
     }
-    if (ty < rows && n0 + tx < p.n_out) reinterpret_cast<float*>(p.out)[(size_t)g * p.out_gstride + (size_t)(r0 + ty) * p.ldo + n0 + tx] = acc;
+    if (ty < rows && n0 + tx < p.n_out) reinterpret_cast<float*>(p.out)[(size_t)g * p.out_gstride + (size_t)(p.map_out ? src : r0 + ty) * p.ldo + n0 + tx] = acc;
 }
 
 // upper bound of the number of row tiles (what the grid must cover)

@@ -39,13 +39,15 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentAttnSpec a
         for (int i = threadIdx.x; i < W; i += blockDim.x)
             Elt<T>::st(crow + i, i < R ? Elt<T>::ld(lat + i) * inv * p.c_norm[i] : (i < R + rot ? turned(lat + R, i - R) : 0.f));
     }
-    T* qn = reinterpret_cast<T*>(p.q_nope) + (size_t)t * a.heads * p.dim_pad;
-    for (int i = threadIdx.x; i < a.heads * p.dim_pad; i += blockDim.x) {
-        const int h = i / p.dim_pad, d = i - h * p.dim_pad;
+    const int QW = p.plain_pad + p.rot_pad;
+    T* qo = reinterpret_cast<T*>(p.q) + (size_t)t * a.heads * QW;
+    for (int i = threadIdx.x; i < a.heads * QW; i += blockDim.x) {
+        const int h = i / QW, d = i - h * QW;
+        const T* qh = row + h * (a.dim + rot);
         if (d < a.dim)
-            qn[i] = row[h * (a.dim + rot) + d];
+            qo[i] = qh[d];
         else
-            Elt<T>::st(qn + i, 0.f);
+            Elt<T>::st(qo + i, d >= p.plain_pad && d - p.plain_pad < rot ? turned(qh + a.dim, d - p.plain_pad) : 0.f);
     }
     T* ql = reinterpret_cast<T*>(p.q_lat) + (size_t)t * a.heads * W;
     const int tail = W - R;
@@ -61,7 +63,7 @@ __global__ void __launch_bounds__(128) latent_attn_simple_kernel(const LatentAtt
     pdl_wait();
     extern __shared__ float sm[];  // q [W] | acc [R] | p [128]
     __shared__ float red[33];
-    const int t = blockIdx.x, h = blockIdx.y, W = a.row_pad(), R = a.kv_rank;
+    const int t = p.row_idx ? p.row_idx[blockIdx.x] : blockIdx.x, h = blockIdx.y, W = a.row_pad(), R = a.kv_rank;
     float *q = sm, *acc = sm + W, *pr = acc + R;
     const int n = p.positions[t] + 1;
     const int32_t* bt = p.block_tables + (size_t)p.seq_slot[p.token_seq[t]] * p.max_blocks;
@@ -108,7 +110,304 @@ __global__ void __launch_bounds__(128) latent_attn_simple_kernel(const LatentAtt
     for (int i = threadIdx.x; i < p.o_pad; i += 128) Elt<T>::st(o + i, i < R ? acc[i] / l : 0.f);
 }
 
+// ---- decode: tensor cores, keys split over CTAs ---------------------------------------------------------------------
+// One cached row serves every head, so the heads are the rows of the matrix products:
+//   S [heads x keys] = Q [heads x W] . K^T,   O [heads x R] += P [heads x keys] . K[:, :R]
+// CTA = (one chunk of one sequence's keys, up to MT * 16 heads), 8 warps, 64 keys per tile, double-buffered cp.async.
+// Scores and weights are f32; the weights enter the second product as their bf16 head plus bf16 remainder.  For the
+// second product the warps split the R columns (16-column tiles w, w + 8, ...).  With more than one chunk a sequence's
+// partial results (f32) are added in chunk order by the CTA that arrives last; nobody waits.
+constexpr int DK_KEYS = 64, DK_NJ = 4;  // keys per tile; 16-column tiles per warp (R up to 512)
+constexpr int kDecodeMaxRank = DK_NJ * 8 * 16;
+constexpr int PS = DK_KEYS + 8;         // row stride of the weights in shared memory
+
+template <int MT>
+struct DecodeSmem {
+    static constexpr int H = MT * 16;
+    static __host__ __device__ int qk_bytes(int W) { return (H + 2 * DK_KEYS) * (W + 8) * 2; }
+    static __host__ __device__ int bytes(int W) { return qk_bytes(W) + 2 * H * PS * 2 + (8 * H * 2 + 3 * H) * 4 + 16; }
+};
+
+template <int MT>
+__global__ void __launch_bounds__(256, 1) latent_decode_kernel(const LatentAttnSpec a, const LatentDecodeParams p) {
+    asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
+    pdl_wait();
+    constexpr int H = MT * 16, KW = MT == 2 ? 4 : 8, NK = 8 / KW;  // key groups of a tile, 8-key tiles per warp
+    extern __shared__ __align__(16) uint8_t smem[];
+    const int W = a.row_pad(), R = a.kv_rank, LD = W + 8;
+    const uint32_t sQ = smem_u32(smem), sK = sQ + H * LD * 2;
+    uint8_t* tail = smem + DecodeSmem<MT>::qk_bytes(W);
+    uint16_t *ph = reinterpret_cast<uint16_t*>(tail), *pl = ph + H * PS;
+    float *wmax = reinterpret_cast<float*>(pl + H * PS), *wsum = wmax + 8 * H, *rowm = wsum + 8 * H, *rowl = rowm + 2 * H;
+    int* flag = reinterpret_cast<int*>(rowl + H);
+    const uint32_t sPh = smem_u32(ph), sPl = smem_u32(pl);
+
+    const int item = blockIdx.x, h0 = blockIdx.y * H;
+    int sd, chunk, n_chunks, part0;  // row of the list, its chunk, chunks of the row, first partial slot of the row
+    if (p.work_seq) {
+        if (item >= *p.n_work) return;
+        sd = p.work_seq[item];
+        chunk = p.work_chunk[item];
+        part0 = p.work_off[sd];
+    } else {  // every row has the same number of work items
+        sd = item / p.max_chunks;
+        chunk = item - sd * p.max_chunks;
+        part0 = sd * p.max_chunks;
+    }
+    const int ctx = p.ctx ? p.ctx[sd] : p.positions[sd] + 1, qrow = p.qrow ? p.qrow[sd] : sd;
+    const int slot = p.slot ? p.slot[sd] : p.seq_slot[p.token_seq[sd]];
+    const int chunk_keys = p.chunk_tiles * 16;
+    n_chunks = (ctx + chunk_keys - 1) / chunk_keys;
+    if (chunk >= n_chunks) return;
+    const int k_lo = chunk * chunk_keys, k_hi = min(ctx, k_lo + chunk_keys);
+    const int n_tiles = (k_hi - k_lo + DK_KEYS - 1) / DK_KEYS;
+    const int32_t* bt = p.block_tables + (size_t)slot * p.max_blocks;
+    const uint16_t* cache = reinterpret_cast<const uint16_t*>(p.cache);
+    const uint16_t* q = reinterpret_cast<const uint16_t*>(p.q_lat) + (size_t)qrow * a.heads * W;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, mi = lane >> 3, lr = lane & 7;
+
+    for (int r = warp; r < H; r += 8) {
+        const bool ok = h0 + r < a.heads;
+        for (int c = lane; c < W / 8; c += 32) cp_async16_zfill(sQ + (r * LD + c * 8) * 2, q + (size_t)(ok ? h0 + r : 0) * W + c * 8, ok);
+    }
+    auto load = [&](int j) {
+        const int k0 = k_lo + j * DK_KEYS;
+        const uint32_t dst = sK + (j & 1) * DK_KEYS * LD * 2;
+        for (int r = warp; r < DK_KEYS; r += 8) {
+            const int key = k0 + r;
+            const bool ok = key < k_hi;
+            const int kk = ok ? key : k_lo;
+            const uint16_t* src = cache + ((size_t)bt[kk / p.page_size] * p.page_size + kk % p.page_size) * W;
+            for (int c = lane; c < W / 8; c += 32) cp_async16_zfill(dst + (r * LD + c * 8) * 2, src + c * 8, ok);
+        }
+    };
+    load(0);
+    cp_async_commit();
+    if (tid < H) {
+        rowm[tid] = -INFINITY;
+        rowl[tid] = 0.f;
+    }
+    float acc[MT][DK_NJ * 2][4];
+#pragma unroll
+    for (int m = 0; m < MT; m++)
+#pragma unroll
+        for (int n = 0; n < DK_NJ * 2; n++) acc[m][n][0] = acc[m][n][1] = acc[m][n][2] = acc[m][n][3] = 0.f;
+    const int mw = MT == 2 ? (warp & 1) : 0, kw = MT == 2 ? (warp >> 1) : warp;
+    const int KS = W / 16, CT = (R + 15) / 16;
+    const int row_a = mw * 16 + (lane >> 2), row_b = row_a + 8;
+    for (int j = 0; j < n_tiles; j++) {
+        if (j + 1 < n_tiles) load(j + 1);
+        cp_async_commit();
+        cp_async_wait<1>();
+        __syncthreads();
+        const uint32_t kb = sK + (j & 1) * DK_KEYS * LD * 2;
+        // ---- scores of this warp: 16 heads x NK * 8 keys
+        float s[NK][4];
+#pragma unroll
+        for (int n = 0; n < NK; n++) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
+        const uint32_t qa = sQ + ((mw * 16 + lr + (mi & 1) * 8) * LD + (mi >> 1) * 8) * 2;
+        if (NK == 2) {
+            const uint32_t ka = kb + ((kw * 16 + lr + (mi >> 1) * 8) * LD + (mi & 1) * 8) * 2;
+#pragma unroll 4
+            for (int k = 0; k < KS; k++) {
+                uint32_t af[4], b0[2], b1[2];
+                ldmatrix_x4(af[0], af[1], af[2], af[3], qa + k * 32);
+                ldmatrix_x4(b0[0], b0[1], b1[0], b1[1], ka + k * 32);
+                mma_bf16_16816(s[0], af, b0);
+                mma_bf16_16816(s[NK - 1], af, b1);
+            }
+        } else {
+            const uint32_t ka = kb + ((kw * 8 + lr) * LD + (mi & 1) * 8) * 2;
+#pragma unroll 4
+            for (int k = 0; k < KS; k++) {
+                uint32_t af[4], b0[2];
+                ldmatrix_x4(af[0], af[1], af[2], af[3], qa + k * 32);
+                ldmatrix_x2(b0[0], b0[1], ka + k * 32);
+                mma_bf16_16816(s[0], af, b0);
+            }
+        }
+        float m0 = -INFINITY, m1 = -INFINITY;
+#pragma unroll
+        for (int n = 0; n < NK; n++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                const int key = k_lo + j * DK_KEYS + kw * NK * 8 + n * 8 + 2 * (lane & 3) + (e & 1);
+                s[n][e] = key < k_hi ? s[n][e] * p.scale_log2 : -INFINITY;
+                if (e < 2)
+                    m0 = fmaxf(m0, s[n][e]);
+                else
+                    m1 = fmaxf(m1, s[n][e]);
+            }
+#pragma unroll
+        for (int o = 1; o < 4; o <<= 1) {
+            m0 = fmaxf(m0, __shfl_xor_sync(0xffffffffu, m0, o));
+            m1 = fmaxf(m1, __shfl_xor_sync(0xffffffffu, m1, o));
+        }
+        if ((lane & 3) == 0) {
+            wmax[kw * H + row_a] = m0;
+            wmax[kw * H + row_b] = m1;
+        }
+        __syncthreads();
+        // ---- weights: the tile's row maximum over all warps, then exp2; the first tile always has a visible key
+        const float *old_m = rowm + (j & 1) * H, *cur_m;
+        float* new_m = rowm + ((j & 1) ^ 1) * H;
+        m0 = old_m[row_a];
+        m1 = old_m[row_b];
+#pragma unroll
+        for (int w = 0; w < KW; w++) {
+            m0 = fmaxf(m0, wmax[w * H + row_a]);
+            m1 = fmaxf(m1, wmax[w * H + row_b]);
+        }
+        float l0 = 0.f, l1 = 0.f;
+#pragma unroll
+        for (int n = 0; n < NK; n++) {
+            const float e0 = exp2f(s[n][0] - m0), e1 = exp2f(s[n][1] - m0), e2 = exp2f(s[n][2] - m1), e3 = exp2f(s[n][3] - m1);
+            l0 += e0 + e1;
+            l1 += e2 + e3;
+            const int col = kw * NK * 8 + n * 8 + 2 * (lane & 3);
+            const uint32_t ha = pack_bf2(e0, e1), hb = pack_bf2(e2, e3);
+            *reinterpret_cast<uint32_t*>(ph + row_a * PS + col) = ha;
+            *reinterpret_cast<uint32_t*>(ph + row_b * PS + col) = hb;
+            *reinterpret_cast<uint32_t*>(pl + row_a * PS + col) = pack_bf2(e0 - bflo(ha), e1 - bfhi(ha));
+            *reinterpret_cast<uint32_t*>(pl + row_b * PS + col) = pack_bf2(e2 - bflo(hb), e3 - bfhi(hb));
+        }
+#pragma unroll
+        for (int o = 1; o < 4; o <<= 1) {
+            l0 += __shfl_xor_sync(0xffffffffu, l0, o);
+            l1 += __shfl_xor_sync(0xffffffffu, l1, o);
+        }
+        if ((lane & 3) == 0) {
+            wsum[kw * H + row_a] = l0;
+            wsum[kw * H + row_b] = l1;
+            if (kw == 0) {
+                new_m[row_a] = m0;
+                new_m[row_b] = m1;
+            }
+        }
+        __syncthreads();
+        // ---- O = alpha O + P K[:, :R]
+        cur_m = new_m;
+        if (tid < H) {
+            float l = rowl[tid] * exp2f(old_m[tid] - cur_m[tid]);
+#pragma unroll
+            for (int w = 0; w < KW; w++) l += wsum[w * H + tid];
+            rowl[tid] = l;
+        }
+#pragma unroll
+        for (int m = 0; m < MT; m++) {
+            const int ra = m * 16 + (lane >> 2);
+            const float a0 = exp2f(old_m[ra] - cur_m[ra]), a1 = exp2f(old_m[ra + 8] - cur_m[ra + 8]);
+            if (__any_sync(0xffffffffu, a0 != 1.f || a1 != 1.f)) {
+#pragma unroll
+                for (int n = 0; n < DK_NJ * 2; n++) acc[m][n][0] *= a0, acc[m][n][1] *= a0, acc[m][n][2] *= a1, acc[m][n][3] *= a1;
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < DK_KEYS / 16; k++) {
+            uint32_t fh[MT][4], fl[MT][4];
+#pragma unroll
+            for (int m = 0; m < MT; m++) {
+                const uint32_t off = ((m * 16 + lr + (mi & 1) * 8) * PS + k * 16 + (mi >> 1) * 8) * 2;
+                ldmatrix_x4(fh[m][0], fh[m][1], fh[m][2], fh[m][3], sPh + off);
+                ldmatrix_x4(fl[m][0], fl[m][1], fl[m][2], fl[m][3], sPl + off);
+            }
+#pragma unroll
+            for (int c = 0; c < DK_NJ; c++) {
+                const int ct = warp + c * 8;
+                if (ct < CT) {
+                    uint32_t v0[2], v1[2];
+                    ldmatrix_x4_trans(v0[0], v0[1], v1[0], v1[1], kb + ((k * 16 + lr + (mi & 1) * 8) * LD + ct * 16 + (mi >> 1) * 8) * 2);
+#pragma unroll
+                    for (int m = 0; m < MT; m++) {
+                        mma_bf16_16816(acc[m][2 * c], fh[m], v0);
+                        mma_bf16_16816(acc[m][2 * c + 1], fh[m], v1);
+                        mma_bf16_16816(acc[m][2 * c], fl[m], v0);
+                        mma_bf16_16816(acc[m][2 * c + 1], fl[m], v1);
+                    }
+                }
+            }
+        }
+        __syncthreads();  // the tile's buffer, the weights and the row statistics may be overwritten
+    }
+    const float* fin_m = rowm + (n_tiles & 1) * H;
+    uint16_t* out = reinterpret_cast<uint16_t*>(p.o_lat) + (size_t)qrow * a.heads * p.o_pad;
+#pragma unroll
+    for (int m = 0; m < MT; m++)
+#pragma unroll
+        for (int half = 0; half < 2; half++) {
+            const int r = m * 16 + (lane >> 2) + half * 8, h = h0 + r;
+            if (h >= a.heads) continue;
+            const float inv = 1.0f / rowl[r];
+#pragma unroll
+            for (int c = 0; c < DK_NJ * 2; c++) {
+                const int col = (warp + (c >> 1) * 8) * 16 + (c & 1) * 8 + 2 * (lane & 3);
+                if ((warp + (c >> 1) * 8) >= CT) continue;
+#pragma unroll
+                for (int e = 0; e < 2; e++) {
+                    if (col + e >= R) continue;
+                    const float v = acc[m][c][half * 2 + e];
+                    if (n_chunks == 1)
+                        out[(size_t)h * p.o_pad + col + e] = f2bf(v * inv);
+                    else
+                        p.part_o[((size_t)(part0 + chunk) * a.heads + h) * R + col + e] = v;
+                }
+            }
+            if (n_chunks > 1 && warp == 0 && (lane & 3) == 0) {
+                p.part_ml[((size_t)(part0 + chunk) * a.heads + h) * 2] = fin_m[r];
+                p.part_ml[((size_t)(part0 + chunk) * a.heads + h) * 2 + 1] = rowl[r];
+            }
+        }
+    if (n_chunks > 1) {  // the last CTA of this (row, head group) adds the chunks up
+        __threadfence();
+        __syncthreads();
+        if (tid == 0) *flag = atomicAdd(&p.counters[(size_t)sd * gridDim.y + blockIdx.y], 1) == n_chunks - 1;
+        __syncthreads();
+        if (!*flag) return;
+        __threadfence();
+        if (tid == 0) p.counters[(size_t)sd * gridDim.y + blockIdx.y] = 0;
+        for (int r = warp; r < H && h0 + r < a.heads; r += 8) {
+            const int h = h0 + r;
+            float M = -INFINITY, L = 0.f;
+            for (int c = 0; c < n_chunks; c++) M = fmaxf(M, __ldcg(&p.part_ml[((size_t)(part0 + c) * a.heads + h) * 2]));
+            for (int c = 0; c < n_chunks; c++) {
+                const float* ml = &p.part_ml[((size_t)(part0 + c) * a.heads + h) * 2];
+                L += exp2f(__ldcg(ml) - M) * __ldcg(ml + 1);
+            }
+            const float inv = 1.0f / L;
+            for (int col = lane; col < R; col += 32) {
+                float v = 0.f;
+                for (int c = 0; c < n_chunks; c++) {
+                    const size_t at = (size_t)(part0 + c) * a.heads + h;
+                    v = fmaf(exp2f(__ldcg(&p.part_ml[at * 2]) - M), __ldcg(&p.part_o[at * R + col]), v);
+                }
+                out[(size_t)h * p.o_pad + col] = f2bf(v * inv);
+            }
+        }
+    }
+    if (R < p.o_pad && chunk == 0)  // the padding the value projection reads
+        for (int r = warp; r < H && h0 + r < a.heads; r += 8)
+            for (int col = R + lane; col < p.o_pad; col += 32) out[(size_t)(h0 + r) * p.o_pad + col] = 0;
+}
+
 }  // namespace
+
+bool b2_latent_decode_eligible(const LatentAttnSpec& a) {
+    return a.kv_rank <= kDecodeMaxRank && (a.heads > 16 ? DecodeSmem<2>::bytes(a.row_pad()) : DecodeSmem<1>::bytes(a.row_pad())) <= 226 * 1024;
+}
+int b2_latent_decode_head_groups(const LatentAttnSpec& a) { return a.heads > 16 ? (a.heads + 31) / 32 : 1; }
+int32_t b2_latent_decode_launch(b2_ctx* ctx, const LatentAttnSpec& a, const LatentDecodeParams& p, int items) {
+    if (items <= 0) return B2_OK;
+    const dim3 grid(items, b2_latent_decode_head_groups(a));
+    if (a.heads > 16) {
+        B2_SMEM_ONCE(ctx, latent_decode_kernel<2>, 226 * 1024);
+        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, latent_decode_kernel<2>, grid, dim3(256), (size_t)DecodeSmem<2>::bytes(a.row_pad()), ctx->stream, a, p));
+    } else {
+        B2_SMEM_ONCE(ctx, latent_decode_kernel<1>, 226 * 1024);
+        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, latent_decode_kernel<1>, grid, dim3(256), (size_t)DecodeSmem<1>::bytes(a.row_pad()), ctx->stream, a, p));
+    }
+    B2_LAUNCHED(ctx);
+    return B2_OK;
+}
 
 int32_t b2_latent_prep_launch(b2_ctx* ctx, bool f32, const LatentAttnSpec& a, const LatentPrepParams& p) {
     if (p.T <= 0) return B2_OK;

@@ -37,7 +37,8 @@ struct GroupedGemmParams {
     const void* x;           // rows of group g: x + g * x_gstride + row * ldx
     int64_t x_gstride;
     int ldx;
-    const int32_t* row_idx;  // output row r reads x row row_idx[r] (routed experts); null: r
+    const int32_t* row_idx;  // output row r reads x row row_idx[r]; null: r
+    bool map_out;            // ... and is stored at row row_idx[r] of out as well
     const void* w;           // [G][N][K]
     int N, K, G;             // N, K padded (multiples of 64)
     void* out;               // rows of group g: out + g * out_gstride + row * ldo
@@ -73,8 +74,8 @@ struct LatentPrepParams {
     const float* c_norm;    // [kv_rank]
     float eps;
     void* cache;            // [page * page_size + offset][row_pad]
-    void* q_nope;           // [T, heads, dim_pad], zero beyond dim
-    int dim_pad;
+    void* q;                // [T, heads, plain_pad + rot_pad]: plain | rotated part, each zero-padded
+    int plain_pad, rot_pad;
     void* q_lat;            // [T, heads, row_pad]: the rotated query part goes to columns kv_rank.., zero beyond row()
 };
 int32_t b2_latent_prep_launch(b2_ctx* ctx, bool f32, const LatentAttnSpec& a, const LatentPrepParams& p);
@@ -86,10 +87,61 @@ struct LatentAttnParams {
     const int32_t* seq_slot;   // [B]
     const int32_t* token_seq;  // [T]
     const int32_t* positions;  // [T]
-    void* o_lat;            // [T, heads, o_pad] attention-weighted latents
+    const int32_t* row_idx;    // [T] token rows to run (null: 0 .. T-1)
+    void* o_lat;            // [token rows, heads, o_pad] attention-weighted latents
     int o_pad, T;
 };
+// Tensor-core form for single tokens (bf16): rows of a list, each with its own context, keys split over CTAs.
+struct LatentDecodeParams {
+    const void* q_lat;
+    const void* cache;
+    const int32_t* block_tables;
+    int max_blocks, page_size;
+    // rows: the packer's decode list (context, token row, block-table row), or (ctx null) every token of the step
+    const int32_t *ctx, *qrow, *slot;
+    const int32_t *positions, *token_seq, *seq_slot;
+    // work items (row, chunk): the packer's list, or (work_seq null) max_chunks items per row
+    const int32_t *work_seq, *work_chunk, *work_off, *n_work;
+    int max_chunks;
+    int chunk_tiles;   // 16-key tiles per chunk
+    float scale_log2;  // scale * log2(e)
+    float *part_o, *part_ml;  // [work item][head][kv_rank], [work item][head][2]
+    int* counters;     // [row][head group], zero between launches
+    void* o_lat;
+    int o_pad;
+};
+bool b2_latent_decode_eligible(const LatentAttnSpec& a);
+int b2_latent_decode_head_groups(const LatentAttnSpec& a);
+int32_t b2_latent_decode_launch(b2_ctx* ctx, const LatentAttnSpec& a, const LatentDecodeParams& p, int items);
 int32_t b2_latent_attn_simple_launch(b2_ctx* ctx, bool f32, const LatentAttnSpec& a, const LatentAttnParams& p);
+
+// ---- latent_prefill.cu: portions of more than one token (bf16), keys and values expanded per head --------------------
+struct LatentGatherParams {
+    const void* cache;
+    const int32_t* block_tables;
+    int max_blocks, page_size, B, rows;
+    const int32_t* seq_slot;      // [B]
+    const int32_t* context_lens;  // [B]
+    const int32_t* kv_off;        // [B] first gathered row of each prefilling sequence, -1 for the others
+    void* lat;                    // [rows, ld_lat]
+    int ld_lat;
+    void* rot;                    // [rows, rot_pad]
+    int rot_pad;
+};
+int32_t b2_latent_gather_launch(b2_ctx* ctx, const LatentAttnSpec& a, const LatentGatherParams& p);
+struct LatentPrefillParams {
+    const void* q;      // [q_rows, heads, (plain_blocks + rotated blocks) * 64]: plain | rotated part, each zero-padded
+    int q_rows;
+    const void* kv;     // [kv_rows, ld_kv]: plain keys head by head (plain_blocks * 64 each), from column v_col0 the values
+    const void* rot;    // [kv_rows, rotated blocks * 64]
+    int kv_rows, ld_kv, v_col0, plain_blocks;
+    const int32_t *pf_seq, *pf_qstart, *n_work, *cu_seqlens, *context_lens, *kv_off;
+    float scale_log2;
+    void* out;          // [T, ldo]: heads * vdim columns
+    int ldo, vdim;
+};
+bool b2_latent_prefill_eligible(const LatentAttnSpec& a);
+int32_t b2_latent_prefill_launch(b2_ctx* ctx, const LatentAttnSpec& a, const LatentPrefillParams& p, int grid_work);
 
 // ---- ssm.cu ---------------------------------------------------------------------------------------------------------
 struct SsmParams {

@@ -77,14 +77,13 @@ def causal_conv_silu(u, w, b):
 def ssd_recurrence(x, B, C, dt, A_log, D):
     """x [T, heads, P], B / C [T, groups, N], dt [T, heads] -> y [T, heads, P], one token after the other."""
     T, H, P = x.shape
-    per = H // B.shape[1]
+    of = np.arange(H) // (H // B.shape[1])                     # group of every head
     S = np.zeros((H, B.shape[2], P), F)
     y = np.zeros_like(x)
     for t in range(T):
-        for h in range(H):
-            b, c = B[t, h // per], C[t, h // per]
-            S[h] = np.exp(-np.exp(A_log[h]) * dt[t, h]) * S[h] + dt[t, h] * np.outer(b, x[t, h])
-            y[t, h] = S[h].T @ c + D[h] * x[t, h]
+        decay = np.exp(-np.exp(A_log) * dt[t])
+        S = decay[:, None, None] * S + dt[t][:, None, None] * B[t][of][:, :, None] * x[t][:, None, :]
+        y[t] = np.einsum("hnp,hn->hp", S, C[t][of]) + D[:, None] * x[t]
     return y
 
 

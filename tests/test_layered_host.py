@@ -1,0 +1,99 @@
+"""Host-side checks of the layered models: the model registry and the reader of config.json, and the restatement the GPU
+tests compare with (its mechanisms against independent formulations).  No GPU needed."""
+import copy
+
+import numpy as np
+import pytest
+
+from oracle import layered as ref
+from tests import layered_models as lm
+
+
+@pytest.fixture(scope="module")
+def eng():
+    from mlx_llm_b200 import build, engine
+
+    build.build()
+    return engine
+
+
+def test_registry_names_the_family(eng):
+    assert eng.model_family(lm.CASES["mixed"]) == "Zukitar"
+    llama = dict(hidden_size=64, intermediate_size=128, num_hidden_layers=2, num_attention_heads=4, vocab_size=32)
+    assert eng.model_family(llama) == "llama"
+
+
+def test_registry_refuses_what_it_does_not_know(eng):
+    from mlx_llm_b200._lib import B2Error
+
+    def code(change):
+        cfg = copy.deepcopy(lm.CASES["mixed"])
+        change(cfg)
+        with pytest.raises(B2Error) as e:
+            eng.model_family(cfg)
+        return e.value.code, str(e.value)
+
+    assert code(lambda c: c.update(architecture="Other"))[0] == -5
+    for change, word in ((lambda c: c.pop("logit_scale"), "logit_scale"), (lambda c: c["layers"][0].update(type="conv"), "conv"),
+                         (lambda c: c["layers"][0]["mixer"].pop("kv_rank"), "kv_rank"), (lambda c: c["layers"][1]["mixer"].update(groups=3), "groups"),
+                         (lambda c: c["layers"][1]["mlp"]["router"].update(top=9), "experts"), (lambda c: c["layers"][0]["mlp"].update(kind="x"), "kind"),
+                         (lambda c: c["layers"][0]["mixer"]["rot"].update(dims=7), "rot"), (lambda c: c.update(layers=[]), "layers"),
+                         (lambda c: c["norm"].update(eps="small"), "eps")):
+        rc, msg = code(change)
+        assert rc == -4 and word in msg, msg
+
+
+def test_latent_attention_absorbed_form_is_the_same():
+    """Scores and outputs computed in latent coordinates equal the per-head form."""
+    cfg = lm.config([(lm.latent(), None)])
+    w = lm.weights(cfg, 1)
+    m = cfg["layers"][0]["mixer"]
+    h = np.random.default_rng(0).standard_normal((30, cfg["width"]))
+    g = lambda n: w["l0.mix." + n]
+    H, D, R, V, K = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+    pos = np.arange(30.0)
+    q = (h @ g("q").T).reshape(30, H, D + R)
+    ck = h @ g("dkv").T
+    c = ref.rms_norm(ck[:, :K], g("dkv.norm"), 3e-5)
+    kr = ref.rotate_pairs(ck[:, K:], pos, m["rot"]["base"], R)
+    out = np.zeros((30, H, V))
+    for hd in range(H):
+        ql = q[:, hd, :D] @ g("uk")[hd * D:(hd + 1) * D]
+        qr = ref.rotate_pairs(q[:, hd, D:], pos, m["rot"]["base"], R)
+        for t in range(30):
+            s = (c[:t + 1] @ ql[t] + kr[:t + 1] @ qr[t]) * m["scale"]
+            p = np.exp(s - s.max())
+            out[t, hd] = g("uv")[hd * V:(hd + 1) * V] @ (p / p.sum() @ c[:t + 1])
+    assert np.allclose(out.reshape(30, -1) @ g("o").T, ref.latent_attention(h, g, m, 3e-5))
+
+
+def test_recurrence_equals_its_closed_form():
+    """y_t = sum over s <= t of C_t . B_s  d_s  exp(-A sum of d over (s, t])  x_s  + D x_t."""
+    rng = np.random.default_rng(2)
+    T, H, P, G, N = 12, 4, 3, 2, 5
+    x, B, C = rng.standard_normal((T, H, P)), rng.standard_normal((T, G, N)), rng.standard_normal((T, G, N))
+    dt, A_log, D = rng.random((T, H)), rng.standard_normal(H), rng.standard_normal(H)
+    y = ref.ssd_recurrence(x, B, C, dt, A_log, D)
+    for t in range(T):
+        for h in range(H):
+            want = D[h] * x[t, h]
+            for s in range(t + 1):
+                want = want + (C[t, h // 2] @ B[s, h // 2]) * dt[s, h] * np.exp(-np.exp(A_log[h]) * dt[s + 1:t + 1, h].sum()) * x[s, h]
+            assert np.allclose(y[t, h], want)
+
+
+def test_small_pieces():
+    u, w, b = np.random.default_rng(0).standard_normal((6, 2)), np.array([[1.0, 2.0, 3.0], [0.0, 0.0, 1.0]]), np.array([0.5, 0.0])
+    c = ref.causal_conv_silu(u, w, b)
+    assert np.allclose(c[0, 0], ref.silu(3 * u[0, 0] + 0.5)) and np.allclose(c[4, 0], ref.silu(u[2, 0] + 2 * u[3, 0] + 3 * u[4, 0] + 0.5))
+    assert np.allclose(c[:, 1], ref.silu(u[:, 1]))
+    v = np.array([[[1.0, 0.0, 5.0]]])
+    r = ref.rotate_pairs(v, np.array([1.0]), 100.0, 2)
+    assert np.allclose(r, [[[np.cos(1.0), np.sin(1.0), 5.0]]])
+    y = ref.gated_group_norm(np.ones((1, 4)), np.array([[1.0, 1.0, 2.0, 2.0]]), np.ones(4), 2, 0.0)
+    assert np.allclose(y, 1.0)
+    one = dict(router=dict(experts=2, top=1), expert=dict(ff=1, limit=0.5))
+    W = {"router": np.array([[3.0], [-1.0]]), "e0.gate": np.array([[2.0]]), "e0.up": np.array([[-9.0]]), "e0.down": np.array([[1.0]]),
+         "e1.gate": np.zeros((1, 1)), "e1.up": np.zeros((1, 1)), "e1.down": np.zeros((1, 1))}
+    got = ref.routed_ff(np.array([[1.0]]), W.__getitem__, one)
+    assert np.allclose(got, 0.5 / (1 + np.exp(-1.702 * 0.5)) * 0.5)  # gate cut at 0.5, up at -0.5
