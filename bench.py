@@ -15,6 +15,8 @@ Prints ONE JSON line (rank 0).  Workloads:
                            Llama-3-8B projection shapes at 1, 8, 32, 128 and 256 tokens.
   decode_only              decode iterations without prefill (the weight-streaming regime).
   qwen3_32b_q8_tp          BASELINE configuration 4: one Qwen3-32B-architecture Q8 model over N ranks.
+  layered                  the layered design (latent attention, Mamba-2, routed experts) at sizes of real models beside the
+                           flat decoder of equal width, both dense bf16: prefill and decode steps at a few sizes.
 A "step" is one iteration of the serving loop (one ragged forward over one batch).  The engine is
 first rolled to its steady state (`ramp` iterations, untimed, all requests available at t = 0), then W
 warm-up and K timed iterations follow.  `value` = generated tokens / device time of the K forwards
@@ -688,13 +690,124 @@ def run_reference(args, rank, world):
                 e2e=dict(value=v, unit="tok/s", h2d_bytes_per_step=0, d2h_bytes_per_step=0), gpu_launches=0)
 
 
+# ------------------------------------------------------------------------------------------------
+# Layered design (latent attention, Mamba-2, routed experts) beside the flat decoder of equal width
+def layered_point(eng, ctx, model, kind, seqs, tokens, context, steps, warm, seed):
+    """One operating point: `prefill` = one step of `tokens` new tokens behind `context` cached ones; `decode` = one token
+    for each of `seqs` sequences at about `context` cached tokens.  Device time per step by CUDA events around the step (the
+    step's copies included), wall time, and the time per kernel class of an extra profiled pass."""
+    rng = np.random.default_rng(seed)
+    vocab = model.config().vocab_size
+    pages = seqs * ((context + tokens + steps + warm + 64) // 16 + 2)
+    pool = eng.BlockPool(ctx, model, 16, pages, seqs, pages // seqs)
+    ids = [rng.integers(0, vocab, context + tokens, dtype=np.int32) for _ in range(seqs)]
+
+    def fresh():
+        caches = [eng.PagedKvCache(pool) for _ in range(seqs)]
+        for c, t in zip(caches, ids):
+            for i in range(0, context, 2048):
+                model.step([(t[i:min(i + 2048, context)], c)], want_logits=False)
+        return caches
+
+    caches = fresh()
+    feed = [rng.integers(0, vocab, 1, dtype=np.int32) for _ in range(seqs)]
+
+    def once():
+        if kind == "decode":
+            ctx.timer_start()
+            t0 = time.perf_counter()
+            model.step(list(zip(feed, caches)), want_logits=False)
+        else:
+            for c in caches:
+                c.free()
+            caches[:] = fresh()
+            ctx.flush_l2()
+            ctx.timer_start()
+            t0 = time.perf_counter()
+            model.step([(t[context:], c) for t, c in zip(ids, caches)], want_logits=False)
+        return ctx.timer_stop_ms(), (time.perf_counter() - t0) * 1e3
+
+    for _ in range(max(warm, 3)):
+        once()
+    launches = ctx.launch_count()
+    times = [once() for _ in range(steps)]
+    launches = (ctx.launch_count() - launches) // steps
+    dev, wall = float(np.mean([t[0] for t in times])), float(np.mean([t[1] for t in times]))
+    if kind == "prefill":
+        for c in caches:
+            c.free()
+        caches[:] = fresh()
+    eng.profile_enable(ctx, True)
+    if kind == "decode":
+        once()
+    else:
+        model.step([(t[context:], c) for t, c in zip(ids, caches)], want_logits=False)
+    prof = eng.profile_read(ctx)
+    eng.profile_enable(ctx, False)
+    for c in caches:
+        c.free()
+    pool.free()
+    n = seqs if kind == "decode" else seqs * tokens
+    out = dict(kind=kind, sequences=seqs, new_tokens=tokens, context=context, ms=round(dev, 4), wall_ms=round(wall, 4), tok_per_s=round(n / dev * 1e3, 1),
+               launches=int(launches), class_ms={k: round(v, 4) for k, v in prof["ms"].items() if v > 0})
+    gemm = prof["ms"]["gemm"]
+    if gemm > 0:
+        out["gemm_tflops"] = round(prof["gemm_flops"] / gemm / 1e9, 1)
+        out["gemm_weight_gbs"] = round(prof["gemm_weight_bytes"] / gemm / 1e6, 1)
+    if prof["ms"]["attn_decode"] > 0:
+        out["attn_decode_gbs"] = round(prof["attn_decode_bytes"] / prof["ms"]["attn_decode"] / 1e6, 1)
+    if prof["ms"]["attn_prefill"] > 0:
+        out["attn_prefill_tflops"] = round(prof["attn_prefill_flops"] / prof["ms"]["attn_prefill"] / 1e9, 1)
+    return out
+
+
+def run_layered(args, rank, world, local_rank, barrier, reduce_max, reduce_sum):
+    from mlx_llm_b200 import _lib, engine as eng, workloads as wl
+
+    ctx = _lib.Context(local_rank)
+    steps, warm = min(args.steps, 20), max(args.warmup, 3)
+    pairs = max(args.layers // 2, 1) if args.layers > 0 else 4
+    points = [("prefill", 1, 512, 0), ("prefill", 1, 2048, 0), ("prefill", 1, 512, 4096), ("decode", 1, 1, 2048), ("decode", 16, 1, 2048),
+              ("decode", 64, 1, 2048)]
+    if args.layered_only:
+        points = [points[int(i)] for i in args.layered_only.split(",")]
+    sampler = ClockSampler(local_rank)
+    sampler.start()
+    barrier()
+    sizes = {}
+    for size in args.layered_sizes.split(","):
+        rows = {}
+        for arm in ("layered", "flat"):
+            if args.layered_arm not in ("both", arm):
+                continue
+            model = eng.CausalLm.synthetic_json(ctx, wl.layered_config(size, pairs), 1) if arm == "layered" else \
+                eng.CausalLm.synthetic(ctx, eng.model_config(**wl.flat_twin(size, 2 * pairs)), seed=1)
+            rows[arm] = dict(weight_gb=round(model.weight_bytes() / 1e9, 3),
+                             points=[layered_point(eng, ctx, model, k, b, n, c, steps, warm, 7) for k, b, n, c in points])
+            model.free()
+        sizes[size] = rows
+    barrier()
+    clocks = sampler.stop()
+    first = next(iter(sizes.values()))
+    head = next((r for r in first.get("layered", first.get("flat"))["points"] if r["kind"] == "decode"), first.get("layered", first.get("flat"))["points"][-1])
+    peaks = measured_peaks()
+    return dict(metric="decode tok/s, layered design (latent attention, Mamba-2, routed experts)", value=reduce_sum(head["tok_per_s"]), unit="tok/s",
+                n_gpus=world, steps=steps, warmup=warm, ms_per_step=reduce_max(head["ms"]), higher_is_better=True, scaling="weak", vs_baseline=None,
+                dtype="bf16", data="synthetic",
+                config=dict(workload="layered design beside the flat decoder of equal width, dense bf16", layers=2 * pairs, page=16,
+                            parallelism=f"replica x{world}", l2="weights exceed L2; prefill steps behind a flush", sizes=sizes),
+                peaks=peaks, e2e=dict(value=reduce_sum(head["tok_per_s"] * head["ms"] / head["wall_ms"]), unit="tok/s", h2d_bytes_per_step=None,
+                                      d2h_bytes_per_step=None),
+                gpu_launches=head["launches"] * steps, clocks=clocks)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=100)
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="llama3_8b_q4_continuous", choices=["llama3_8b_q4_continuous", "paged_attn_decode", "qwen3_32b_q8_tp", "decode_only", "qmm"])
+    ap.add_argument("--workload", default="llama3_8b_q4_continuous", choices=["llama3_8b_q4_continuous", "paged_attn_decode", "qwen3_32b_q8_tp", "decode_only", "qmm", "layered"])
     ap.add_argument("--chunk-tokens", dest="chunk_tokens", type=int, default=0, help="paged_attn_decode: split-K chunk")
     ap.add_argument("--requests", type=int, default=2048)
     ap.add_argument("--arrivals", default="saturated", choices=["saturated", "poisson"])
@@ -711,6 +824,9 @@ def main():
     ap.add_argument("--profiler-range", dest="profiler_range", action="store_true",
                     help="bracket the timed region with cudaProfilerStart/Stop (for `ncu --profile-from-start off`)")
     ap.add_argument("--qmm-only", dest="qmm_only", default="", help="qmm: comma-separated OUTxINxBITSxTOKENS cases to run (profiling); not a valid bench line")
+    ap.add_argument("--layered-sizes", dest="layered_sizes", default="w4096,w2048", help="layered: comma-separated sizes (workloads.LAYERED_SIZES)")
+    ap.add_argument("--layered-arm", dest="layered_arm", default="both", choices=["both", "layered", "flat"])
+    ap.add_argument("--layered-only", dest="layered_only", default="", help="layered: indices of the operating points to run (profiling)")
     ap.add_argument("--no-cpu-baseline", dest="cpu_baseline", action="store_false")
     args = ap.parse_args()
 
@@ -733,6 +849,8 @@ def main():
         out = run_paged_attn(args, rank, world, local_rank, barrier, reduce_max, reduce_sum)
     elif args.workload == "qmm":
         out = run_qmm(args, rank, world, local_rank, barrier, reduce_max, reduce_sum)
+    elif args.workload == "layered":
+        out = run_layered(args, rank, world, local_rank, barrier, reduce_max, reduce_sum)
     elif args.workload == "decode_only":
         out = run_decode_only(args, rank, world, local_rank, barrier, reduce_max, reduce_sum)
     else:

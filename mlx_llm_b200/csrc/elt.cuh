@@ -15,6 +15,13 @@ struct Elt<uint16_t> {
 #pragma unroll
         for (int i = 0; i < 4; i++) v[2 * i] = bflo(w[i]), v[2 * i + 1] = bfhi(w[i]);
     }
+    static __device__ __forceinline__ void ld4(const uint16_t* p, float (&v)[4]) {  // 8-byte aligned
+        const uint2 u = *reinterpret_cast<const uint2*>(p);
+        v[0] = bflo(u.x), v[1] = bfhi(u.x), v[2] = bflo(u.y), v[3] = bfhi(u.y);
+    }
+    static __device__ __forceinline__ void st4(uint16_t* p, const float (&v)[4]) {
+        *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf2(v[0], v[1]), pack_bf2(v[2], v[3]));
+    }
     static __device__ __forceinline__ void st8(uint16_t* p, const float (&v)[8]) {
         *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf2(v[0], v[1]), pack_bf2(v[2], v[3]), pack_bf2(v[4], v[5]), pack_bf2(v[6], v[7]));
     }
@@ -27,6 +34,11 @@ struct Elt<float> {
         const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
         v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w, v[4] = b.x, v[5] = b.y, v[6] = b.z, v[7] = b.w;
     }
+    static __device__ __forceinline__ void ld4(const float* p, float (&v)[4]) {
+        const float4 a = *reinterpret_cast<const float4*>(p);
+        v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w;
+    }
+    static __device__ __forceinline__ void st4(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
     static __device__ __forceinline__ void st8(float* p, const float (&v)[8]) {
         *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
         *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);

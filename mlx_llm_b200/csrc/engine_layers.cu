@@ -57,11 +57,9 @@ struct LayeredModel {
     // prefill attention: gathered latents, rotated key parts and expanded keys / values of the contexts in a step
     uint16_t *kv_lat = nullptr, *kv_rot = nullptr, *kv_exp = nullptr;
     int kv_cap = 0, kv_ld_lat = 0, kv_ld_rot = 0, kv_ld_exp = 0;  // rows; widest rows over the layers
-    // decode attention: partial results per work item, arrival counters per row
+    // decode attention: partial results per work item
     float* dec_part = nullptr;
     size_t dec_part_floats = 0, dec_part_row = 0;  // capacity; heads * (kv_rank + 2) of the largest layer
-    int* dec_counters = nullptr;
-    int dec_counters_cap = 0;
     uint8_t* arena = nullptr;
     int t_cap = 0, l_cap = 0;
     float* capture = nullptr;
@@ -441,21 +439,13 @@ int32_t ensure_expand(b2_model* m, int rows) {
     B2_CHECK(regrow_zero(m->ctx, lm.kv_rot, (size_t)lm.kv_cap * lm.kv_ld_rot));
     return regrow_zero(m->ctx, lm.kv_exp, (size_t)lm.kv_cap * lm.kv_ld_exp);
 }
-int32_t ensure_decode(b2_model* m, int items, int counters) {
+int32_t ensure_decode(b2_model* m, int items) {
     LayeredModel& lm = *m->layered;
     const size_t need = (size_t)items * lm.dec_part_row;
-    if (need > lm.dec_part_floats || counters > lm.dec_counters_cap) {
-        B2_CUDA(cudaStreamSynchronize(m->ctx->stream));
-        if (need > lm.dec_part_floats) {
-            lm.dec_part_floats = need * 5 / 4;
-            B2_CHECK(regrow_zero(m->ctx, lm.dec_part, lm.dec_part_floats));
-        }
-        if (counters > lm.dec_counters_cap) {
-            lm.dec_counters_cap = counters * 5 / 4 + 64;
-            B2_CHECK(regrow_zero(m->ctx, lm.dec_counters, (size_t)lm.dec_counters_cap));
-        }
-    }
-    return B2_OK;
+    if (need <= lm.dec_part_floats) return B2_OK;
+    B2_CUDA(cudaStreamSynchronize(m->ctx->stream));
+    lm.dec_part_floats = need * 5 / 4;
+    return regrow_zero(m->ctx, lm.dec_part, lm.dec_part_floats);
 }
 
 // ---- forward --------------------------------------------------------------------------------------------------------
@@ -606,10 +596,9 @@ int32_t Fwd::latent(const LayerSpec& L, const LayerP& P, int l) {
                 dp.n_work = s.mo->counts + 2;
                 dp.chunk_tiles = s.chunk_tiles;
                 items = s.dec_work;
-                B2_CHECK(ensure_decode(m, items, rows * b2_latent_decode_head_groups(a)));
+                B2_CHECK(ensure_decode(m, items));
                 dp.part_o = lm.dec_part;
                 dp.part_ml = lm.dec_part + (size_t)items * a.heads * a.kv_rank;
-                dp.counters = lm.dec_counters;
                 ctx->attn_decode_bytes += (double)s.dec_ctx_sum * W * 2;
             } else {  // one work item per token: nothing is split, no partial results
                 dp.positions = s.mo->positions;
@@ -622,7 +611,7 @@ int32_t Fwd::latent(const LayerSpec& L, const LayerP& P, int l) {
             dp.o_lat = b.o_lat;
             dp.o_pad = b.o_pad;
             b2_prof_mark(ctx, B2_CLS_ATTN_DECODE);
-            B2_CHECK(b2_latent_decode_launch(ctx, a, dp, items));
+            B2_CHECK(b2_latent_decode_launch(ctx, a, dp, items, rows));
         } else {
             LatentAttnParams ap{};
             ap.q_lat = b.q_lat;
@@ -850,7 +839,7 @@ void b2_layered_release(b2_model* m) {
         if (r.sin) cudaFree(r.sin);
     }
     if (lm.route_counters) cudaFree(lm.route_counters);
-    for (void* p : {(void*)lm.arena, (void*)lm.kv_lat, (void*)lm.kv_rot, (void*)lm.kv_exp, (void*)lm.dec_part, (void*)lm.dec_counters})
+    for (void* p : {(void*)lm.arena, (void*)lm.kv_lat, (void*)lm.kv_rot, (void*)lm.kv_exp, (void*)lm.dec_part})
         if (p) cudaFree(p);
     delete m->layered;
     m->layered = nullptr;

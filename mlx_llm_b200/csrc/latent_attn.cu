@@ -116,7 +116,8 @@ __global__ void __launch_bounds__(128) latent_attn_simple_kernel(const LatentAtt
 // CTA = (one chunk of one sequence's keys, up to MT * 16 heads), 8 warps, 64 keys per tile, double-buffered cp.async.
 // Scores and weights are f32; the weights enter the second product as their bf16 head plus bf16 remainder.  For the
 // second product the warps split the R columns (16-column tiles w, w + 8, ...).  With more than one chunk a sequence's
-// partial results (f32) are added in chunk order by the CTA that arrives last; nobody waits.
+// partial results (f32) are added in chunk order by a second kernel: one block per (sequence, head), so that the sums of a
+// long context spread over the machine.
 constexpr int DK_KEYS = 64, DK_NJ = 4;  // keys per tile; 16-column tiles per warp (R up to 512)
 constexpr int kDecodeMaxRank = DK_NJ * 8 * 16;
 constexpr int PS = DK_KEYS + 8;         // row stride of the weights in shared memory
@@ -125,7 +126,7 @@ template <int MT>
 struct DecodeSmem {
     static constexpr int H = MT * 16;
     static __host__ __device__ int qk_bytes(int W) { return (H + 2 * DK_KEYS) * (W + 8) * 2; }
-    static __host__ __device__ int bytes(int W) { return qk_bytes(W) + 2 * H * PS * 2 + (8 * H * 2 + 3 * H) * 4 + 16; }
+    static __host__ __device__ int bytes(int W) { return qk_bytes(W) + 2 * H * PS * 2 + (8 * H * 2 + 3 * H) * 4; }
 };
 
 template <int MT>
@@ -139,7 +140,6 @@ __global__ void __launch_bounds__(256, 1) latent_decode_kernel(const LatentAttnS
     uint8_t* tail = smem + DecodeSmem<MT>::qk_bytes(W);
     uint16_t *ph = reinterpret_cast<uint16_t*>(tail), *pl = ph + H * PS;
     float *wmax = reinterpret_cast<float*>(pl + H * PS), *wsum = wmax + 8 * H, *rowm = wsum + 8 * H, *rowl = rowm + 2 * H;
-    int* flag = reinterpret_cast<int*>(rowl + H);
     const uint32_t sPh = smem_u32(ph), sPl = smem_u32(pl);
 
     const int item = blockIdx.x, h0 = blockIdx.y * H;
@@ -357,36 +357,40 @@ __global__ void __launch_bounds__(256, 1) latent_decode_kernel(const LatentAttnS
                 p.part_ml[((size_t)(part0 + chunk) * a.heads + h) * 2 + 1] = rowl[r];
             }
         }
-    if (n_chunks > 1) {  // the last CTA of this (row, head group) adds the chunks up
-        __threadfence();
-        __syncthreads();
-        if (tid == 0) *flag = atomicAdd(&p.counters[(size_t)sd * gridDim.y + blockIdx.y], 1) == n_chunks - 1;
-        __syncthreads();
-        if (!*flag) return;
-        __threadfence();
-        if (tid == 0) p.counters[(size_t)sd * gridDim.y + blockIdx.y] = 0;
-        for (int r = warp; r < H && h0 + r < a.heads; r += 8) {
-            const int h = h0 + r;
-            float M = -INFINITY, L = 0.f;
-            for (int c = 0; c < n_chunks; c++) M = fmaxf(M, __ldcg(&p.part_ml[((size_t)(part0 + c) * a.heads + h) * 2]));
-            for (int c = 0; c < n_chunks; c++) {
-                const float* ml = &p.part_ml[((size_t)(part0 + c) * a.heads + h) * 2];
-                L += exp2f(__ldcg(ml) - M) * __ldcg(ml + 1);
-            }
-            const float inv = 1.0f / L;
-            for (int col = lane; col < R; col += 32) {
-                float v = 0.f;
-                for (int c = 0; c < n_chunks; c++) {
-                    const size_t at = (size_t)(part0 + c) * a.heads + h;
-                    v = fmaf(exp2f(__ldcg(&p.part_ml[at * 2]) - M), __ldcg(&p.part_o[at * R + col]), v);
-                }
-                out[(size_t)h * p.o_pad + col] = f2bf(v * inv);
-            }
-        }
-    }
     if (R < p.o_pad && chunk == 0)  // the padding the value projection reads
         for (int r = warp; r < H && h0 + r < a.heads; r += 8)
             for (int col = R + lane; col < p.o_pad; col += 32) out[(size_t)(h0 + r) * p.o_pad + col] = 0;
+}
+
+// Sum of a row's chunks: out = sum_c 2^(m_c - M) O_c / sum_c 2^(m_c - M) l_c, M the largest m_c, chunks in order.
+__global__ void __launch_bounds__(128) latent_merge_kernel(const LatentAttnSpec a, const LatentDecodeParams p) {
+    asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
+    pdl_wait();
+    const int sd = blockIdx.x, h = blockIdx.y, R = a.kv_rank, chunk_keys = p.chunk_tiles * 16;
+    const int n = (p.ctx[sd] + chunk_keys - 1) / chunk_keys;
+    if (n <= 1) return;
+    const size_t at0 = (size_t)p.work_off[sd] * a.heads + h;
+    float M = -INFINITY;
+    for (int c = 0; c < n; c++) M = fmaxf(M, p.part_ml[(at0 + (size_t)c * a.heads) * 2]);
+    float acc[DK_NJ] = {0.f, 0.f, 0.f, 0.f}, L = 0.f;  // columns threadIdx.x + 128 i (R up to 512)
+#pragma unroll 4
+    for (int c = 0; c < n; c++) {
+        const size_t at = at0 + (size_t)c * a.heads;
+        const float w = exp2f(p.part_ml[at * 2] - M);
+        L = fmaf(w, p.part_ml[at * 2 + 1], L);
+#pragma unroll
+        for (int i = 0; i < DK_NJ; i++) {
+            const int col = threadIdx.x + i * 128;
+            if (col < R) acc[i] = fmaf(w, p.part_o[at * R + col], acc[i]);
+        }
+    }
+    const float inv = 1.0f / L;
+    uint16_t* out = reinterpret_cast<uint16_t*>(p.o_lat) + ((size_t)p.qrow[sd] * a.heads + h) * p.o_pad;
+#pragma unroll
+    for (int i = 0; i < DK_NJ; i++) {
+        const int col = threadIdx.x + i * 128;
+        if (col < R) out[col] = f2bf(acc[i] * inv);
+    }
 }
 
 }  // namespace
@@ -394,10 +398,9 @@ __global__ void __launch_bounds__(256, 1) latent_decode_kernel(const LatentAttnS
 bool b2_latent_decode_eligible(const LatentAttnSpec& a) {
     return a.kv_rank <= kDecodeMaxRank && (a.heads > 16 ? DecodeSmem<2>::bytes(a.row_pad()) : DecodeSmem<1>::bytes(a.row_pad())) <= 226 * 1024;
 }
-int b2_latent_decode_head_groups(const LatentAttnSpec& a) { return a.heads > 16 ? (a.heads + 31) / 32 : 1; }
-int32_t b2_latent_decode_launch(b2_ctx* ctx, const LatentAttnSpec& a, const LatentDecodeParams& p, int items) {
+int32_t b2_latent_decode_launch(b2_ctx* ctx, const LatentAttnSpec& a, const LatentDecodeParams& p, int items, int rows) {
     if (items <= 0) return B2_OK;
-    const dim3 grid(items, b2_latent_decode_head_groups(a));
+    const dim3 grid(items, a.heads > 16 ? (a.heads + 31) / 32 : 1);
     if (a.heads > 16) {
         B2_SMEM_ONCE(ctx, latent_decode_kernel<2>, 226 * 1024);
         B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, latent_decode_kernel<2>, grid, dim3(256), (size_t)DecodeSmem<2>::bytes(a.row_pad()), ctx->stream, a, p));
@@ -406,6 +409,10 @@ int32_t b2_latent_decode_launch(b2_ctx* ctx, const LatentAttnSpec& a, const Late
         B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, latent_decode_kernel<1>, grid, dim3(256), (size_t)DecodeSmem<1>::bytes(a.row_pad()), ctx->stream, a, p));
     }
     B2_LAUNCHED(ctx);
+    if (items > rows) {  // some row has more than one chunk
+        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, latent_merge_kernel, dim3(rows, a.heads), dim3(128), 0, ctx->stream, a, p));
+        B2_LAUNCHED(ctx);
+    }
     return B2_OK;
 }
 

@@ -106,13 +106,11 @@ struct LatentDecodeParams {
     int chunk_tiles;   // 16-key tiles per chunk
     float scale_log2;  // scale * log2(e)
     float *part_o, *part_ml;  // [work item][head][kv_rank], [work item][head][2]
-    int* counters;     // [row][head group], zero between launches
     void* o_lat;
     int o_pad;
 };
 bool b2_latent_decode_eligible(const LatentAttnSpec& a);
-int b2_latent_decode_head_groups(const LatentAttnSpec& a);
-int32_t b2_latent_decode_launch(b2_ctx* ctx, const LatentAttnSpec& a, const LatentDecodeParams& p, int items);
+int32_t b2_latent_decode_launch(b2_ctx* ctx, const LatentAttnSpec& a, const LatentDecodeParams& p, int items, int rows);
 int32_t b2_latent_attn_simple_launch(b2_ctx* ctx, bool f32, const LatentAttnSpec& a, const LatentAttnParams& p);
 
 // ---- latent_prefill.cu: portions of more than one token (bf16), keys and values expanded per head --------------------
@@ -160,5 +158,6 @@ struct SsmParams {
     float* y;             // [T, inner]
     void* out;            // [T, ldo] gated and normed, zero beyond inner
     int ldo;
+    bool chunked;         // set by the launcher: longer portions belong to the chunked form
 };
 int32_t b2_ssm_launch(b2_ctx* ctx, bool f32, const Mamba2Spec& s, const SsmParams& p);

@@ -53,3 +53,29 @@ def step_weight_bytes(cfg, bits):
 
 def kv_bytes_per_token(cfg):
     return cfg["num_layers"] * 2 * cfg["num_kv_heads"] * cfg["head_dim"] * 2
+
+
+# Layered design (latent attention + dense feed-forward, Mamba-2 + routed experts, alternating) at sizes of real models, and
+# the flat decoder of equal width it is measured beside.
+LAYERED_SIZES = {
+    "w4096": dict(width=4096, latent=dict(heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512), ff=14336,
+                  mamba=dict(heads=128, vdim=64, state=128, groups=8, norm_groups=8, conv=4), experts=32, top=4, expert_ff=1792),
+    "w2048": dict(width=2048, latent=dict(heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512), ff=8192,
+                  mamba=dict(heads=64, vdim=64, state=128, groups=4, norm_groups=4, conv=4), experts=32, top=4, expert_ff=1024),
+}
+
+
+def layered_config(size, pairs, vocab=32000):
+    s = LAYERED_SIZES[size]
+    lat = dict(s["latent"], rot=dict(base=500000.0, dims=s["latent"]["rot_dim"]), scale=(s["latent"]["dim"] + s["latent"]["rot_dim"]) ** -0.5)
+    moe = dict(kind="moe", expert=dict(ff=s["expert_ff"], limit=7.0), router=dict(experts=s["experts"], top=s["top"]))
+    layers = [dict(type="latent_attention", mixer=lat, mlp=dict(kind="dense", ff=s["ff"])), dict(type="mamba2", mixer=s["mamba"], mlp=moe)] * pairs
+    return dict(architecture="Zukitar", width=s["width"], vocab=vocab, norm=dict(eps=1e-5), logit_scale=1.0, layers=layers)
+
+
+def flat_twin(size, layers, vocab=32000):
+    """Llama-architecture model of the same width, feed-forward and layer count, dense bf16."""
+    s = LAYERED_SIZES[size]
+    hq = s["width"] // 128
+    return dict(num_layers=layers, hidden_size=s["width"], num_heads=hq, num_kv_heads=max(hq // 4, 1), head_dim=128, intermediate_size=s["ff"],
+                vocab_size=vocab, rms_norm_eps=1e-5, rope_theta=500000.0)
