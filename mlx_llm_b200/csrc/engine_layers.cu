@@ -320,7 +320,7 @@ struct DenseBufs {
 struct MoeBufs {
     float *logits, *weight, *row_w;
     int32_t *expert, *offsets, *pos, *src;
-    void *gu, *act;
+    void *xs, *gu, *act;
     int ld_act;
 };
 Common carve_common(Carver& c, const LayeredModel& lm, size_t es, size_t t, size_t l) {
@@ -371,7 +371,7 @@ DenseBufs carve_dense(Carver c, const LayerP& P, size_t es, size_t t, size_t* en
     *end = std::max(*end, c.off);
     return o;
 }
-MoeBufs carve_moe(Carver c, const RoutedSpec& r, const LayerP& P, size_t es, size_t t, size_t* end) {
+MoeBufs carve_moe(Carver c, const RoutedSpec& r, const LayerP& P, int ldn, size_t es, size_t t, size_t* end) {
     MoeBufs o;
     const size_t n = t * r.top;
     o.ld_act = P.e_down.K;
@@ -382,6 +382,7 @@ MoeBufs carve_moe(Carver c, const RoutedSpec& r, const LayerP& P, size_t es, siz
     o.pos = c.take<int32_t>(n * 4);
     o.src = c.take<int32_t>(n * 4);
     o.offsets = c.take<int32_t>((size_t)(r.experts + 1) * 4);
+    o.xs = c.take(es == 2 ? n * ldn * es : 0);
     o.gu = c.take(n * P.e_gu.N * es);
     o.act = c.take(n * o.ld_act * es);
     *end = std::max(*end, c.off);
@@ -399,7 +400,7 @@ size_t arena_bytes(const LayeredModel& lm, size_t es, size_t t, size_t l) {
         else
             carve_ssm(c, L.ssm, P, es, t, &end);
         if (L.mlp == MlpKind::DenseGated) carve_dense(c, P, es, t, &end);
-        if (L.mlp == MlpKind::Routed) carve_moe(c, L.moe, P, es, t, &end);
+        if (L.mlp == MlpKind::Routed) carve_moe(c, L.moe, P, pad_k(lm.spec.width), es, t, &end);
     }
     return end + 256;
 }
@@ -576,6 +577,7 @@ int32_t Fwd::latent(const LayerSpec& L, const LayerP& P, int l) {
         g.ldo = a.heads * W;
         g.n_out = a.kv_rank;
         g.M = rows;
+        g.x_rows = lm.t_cap;
         b2_prof_mark(ctx, B2_CLS_GEMM);
         B2_CHECK(b2_grouped_gemm_launch(ctx, m->f32, g));
         if (!m->f32 && b2_latent_decode_eligible(a)) {
@@ -644,6 +646,7 @@ int32_t Fwd::latent(const LayerSpec& L, const LayerP& P, int l) {
         v.ldo = b.ld_att;
         v.n_out = a.vdim;
         v.M = rows;
+        v.x_rows = lm.t_cap;
         b2_prof_mark(ctx, B2_CLS_GEMM);
         B2_CHECK(b2_grouped_gemm_launch(ctx, m->f32, v));
     }
@@ -693,7 +696,7 @@ int32_t Fwd::dense(const LayerSpec& L, const LayerP& P) {
 int32_t Fwd::moe(const LayerSpec& L, const LayerP& P, const int32_t** rows) {
     b2_ctx* ctx = m->ctx;
     const RoutedSpec& r = L.moe;
-    const MoeBufs b = carve_moe(scratch, r, P, es, (size_t)lm.t_cap, &end);
+    const MoeBufs b = carve_moe(scratch, r, P, c.ldn, es, (size_t)lm.t_cap, &end);
     B2_CHECK(linear(m, P.router, c.xn, c.ldn, s.T, lm.t_cap, b.logits, P.router.N, true));
     RouteParams rp{};
     rp.logits = b.logits;
@@ -714,6 +717,12 @@ int32_t Fwd::moe(const LayerSpec& L, const LayerP& P, const int32_t** rows) {
     g.x = c.xn;
     g.ldx = c.ldn;
     g.row_idx = b.src;
+    if (!m->f32 && b2_grouped_gemm_wants_rows(ctx, s.T * r.top, true, r.experts, P.e_gu.N)) {
+        B2_CHECK(b2_gather_rows_launch(ctx, (const uint16_t*)c.xn, b.src, s.T * r.top, c.ldn, c.ldn, (uint16_t*)b.xs));
+        g.x = b.xs;
+        g.row_idx = nullptr;
+        g.x_rows = lm.t_cap * r.top;
+    }
     g.w = P.e_gu.w;
     g.N = P.e_gu.N;
     g.K = P.e_gu.K;
@@ -739,6 +748,7 @@ int32_t Fwd::moe(const LayerSpec& L, const LayerP& P, const int32_t** rows) {
     d.out_f32 = true;
     d.offsets = b.offsets;
     d.M = g.M;
+    d.x_rows = lm.t_cap * r.top;
     b2_prof_mark(ctx, B2_CLS_GEMM);
     B2_CHECK(b2_grouped_gemm_launch(ctx, m->f32, d));
     *rows = b.pos;

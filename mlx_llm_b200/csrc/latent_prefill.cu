@@ -343,11 +343,12 @@ __global__ void __launch_bounds__(kThreads, 1)
                 uint32_t v[32];
                 const int c0 = wg * (VDB * 32) + c * 32;
                 tc_ld32(tmem_o + lane_addr + (uint32_t)c0, v);
-                if (!row_ok) continue;
 #pragma unroll
                 for (int g = 0; g < 4; g++) {
                     const int col = c0 + g * 8;
-                    if (vec && col < p.vdim) {
+                    if (!row_ok) {
+                        // nothing to store; the warp stays together for the next load
+                    } else if (vec && col < p.vdim) {
                         uint4 o4;
                         o4.x = pack_bf2(__uint_as_float(v[g * 8 + 0]) * inv, __uint_as_float(v[g * 8 + 1]) * inv);
                         o4.y = pack_bf2(__uint_as_float(v[g * 8 + 2]) * inv, __uint_as_float(v[g * 8 + 3]) * inv);
@@ -360,6 +361,7 @@ __global__ void __launch_bounds__(kThreads, 1)
                             if (col + i < p.vdim) dst[col + i] = f2bf(__uint_as_float(v[g * 8 + i]) * inv);
                     }
                 }
+                __syncwarp();
             }
         } else if (lane == 0) {
             atomicExch(err, 4);

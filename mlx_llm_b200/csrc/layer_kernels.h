@@ -47,7 +47,12 @@ struct GroupedGemmParams {
     bool out_f32;            // f32 results from bf16 operands
     const int32_t* offsets;  // [G + 1] device: group g owns rows [offsets[g], offsets[g + 1]); null: every group has rows 0..M-1
     int M;                   // rows per group, or the total number of rows with `offsets`
+    int x_rows;              // rows of the x allocation (0: unknown; the TMA kernel needs 128)
+    bool vec_out;            // set by the launcher: 16-byte stores are aligned
 };
+// True when a product of this size takes the kernel whose operands must be consecutive rows (row_idx null): a caller that
+// gathers rows does so beforehand then.
+bool b2_grouped_gemm_wants_rows(const b2_ctx* ctx, int M, bool sorted, int G, int N);
 int32_t b2_grouped_gemm_launch(b2_ctx* ctx, bool f32, const GroupedGemmParams& p);
 
 // ---- moe.cu -----------------------------------------------------------------------------------------------------
@@ -63,6 +68,9 @@ struct RouteParams {
     int32_t* counters;    // [experts + 1], zero between launches
 };
 int32_t b2_route_launch(b2_ctx* ctx, const RouteParams& p);
+
+// out[i] = x[src[i]] (rows of `cols` elements, a multiple of 8, both row strides ld)
+int32_t b2_gather_rows_launch(b2_ctx* ctx, const uint16_t* x, const int32_t* src, int n, int cols, int ld, uint16_t* out);
 
 // ---- latent_attn.cu -----------------------------------------------------------------------------------------------
 struct LatentPrepParams {

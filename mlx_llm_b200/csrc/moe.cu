@@ -77,8 +77,23 @@ __global__ void __launch_bounds__(kThreads) route_kernel(const RouteParams p) {
     }
 }
 
+__global__ void __launch_bounds__(128) gather_rows_kernel(const uint16_t* __restrict__ x, const int32_t* __restrict__ src, int cols, int ld,
+                                                          uint16_t* __restrict__ out) {
+    asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
+    pdl_wait();
+    const uint16_t* s = x + (size_t)src[blockIdx.x] * ld;
+    uint16_t* o = out + (size_t)blockIdx.x * ld;
+    for (int i = threadIdx.x * 8; i < cols; i += 128 * 8) *reinterpret_cast<uint4*>(o + i) = *reinterpret_cast<const uint4*>(s + i);
+}
+
 }  // namespace
 
+int32_t b2_gather_rows_launch(b2_ctx* ctx, const uint16_t* x, const int32_t* src, int n, int cols, int ld, uint16_t* out) {
+    if (n <= 0) return B2_OK;
+    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, gather_rows_kernel, dim3(n), dim3(128), 0, ctx->stream, x, src, cols, ld, out));
+    B2_LAUNCHED(ctx);
+    return B2_OK;
+}
 int32_t b2_route_launch(b2_ctx* ctx, const RouteParams& p) {
     if (p.T <= 0) return B2_OK;
     B2_REQUIRE(p.experts <= kMaxExperts, B2_ERR_UNSUPPORTED, "routing: at most 1024 experts");
