@@ -164,12 +164,18 @@ struct Filler {
         }
         return B2_OK;
     }
-    int32_t vec(float*& dst, const std::string& key, std::vector<int64_t> shape, float mean, float sd) {
+    // a small tensor kept in f32, as stored or (two dimensions) transposed
+    int32_t vec(float*& dst, const std::string& key, std::vector<int64_t> shape, float mean, float sd, bool transpose = false) {
         int64_t n = 1;
         for (auto d : shape) n *= d;
         B2_CHECK(alloc((size_t)n * 4, (void**)&dst));
         if (!w) return random(dst, true, 1, (int)n, (int)n, mean, sd);
         B2_CHECK(fetch(key, shape));
+        if (transpose) {
+            const std::vector<float> a = host;
+            for (int64_t r = 0; r < shape[0]; r++)
+                for (int64_t c = 0; c < shape[1]; c++) host[(size_t)(c * shape[0] + r)] = a[(size_t)(r * shape[1] + c)];
+        }
         B2_CUDA(cudaMemcpyAsync(dst, host.data(), (size_t)n * 4, cudaMemcpyHostToDevice, m->ctx->stream));
         B2_CUDA(cudaStreamSynchronize(m->ctx->stream));
         return B2_OK;
@@ -248,7 +254,7 @@ int32_t load_layer(Filler& f, LayeredModel& lm, int i) {
         const Mamba2Spec& s = L.ssm;
         B2_CHECK(f.proj(P.ssm_in, s.in_rows(), W));
         B2_CHECK(f.rows(P.ssm_in, 0, mix("in"), s.in_rows(), W));
-        B2_CHECK(f.vec(P.conv_w, mix("conv"), {s.channels(), s.conv}, 0.f, 0.5f));
+        B2_CHECK(f.vec(P.conv_w, mix("conv"), {s.channels(), s.conv}, 0.f, 0.5f, true));
         B2_CHECK(f.vec(P.conv_b, mix("conv.b"), {s.channels()}, 0.f, 0.1f));
         B2_CHECK(f.vec(P.dt_bias, mix("dt_bias"), {s.heads}, -3.f, 1.f));
         B2_CHECK(f.vec(P.A_log, mix("A_log"), {s.heads}, 1.f, 0.7f));

@@ -8,53 +8,57 @@
 
 namespace {
 
-// One block per token: norm of the latent, rotation of the shared key part and of every head's rotated part, cache row
-// and query buffers.
+// Block = (token, eight heads): a warp per head copies the plain part of the query and rotates the rest; the blocks of the
+// first eight heads also norm the latent, rotate the shared key part and write the cache row.
 template <typename T>
 __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentAttnSpec a, const LatentPrepParams p) {
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     pdl_wait();
     __shared__ float red[33];
     const int t = blockIdx.x, R = a.kv_rank, rot = a.rot_dim, dims = a.rot.dims, half = dims / 2, W = a.row_pad();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, h = blockIdx.y * 8 + warp;
     const T* row = reinterpret_cast<const T*>(p.qkv) + (size_t)t * p.ld;
-    const int pos = p.positions[t], slot = p.slot_mapping[t];
-    const float* ct = p.cos_t + (size_t)pos * half;
-    const float* st = p.sin_t + (size_t)pos * half;
+    const float* ct = p.cos_t + (size_t)p.positions[t] * half;
+    const float* st = p.sin_t + (size_t)p.positions[t] * half;
     auto turned = [&](const T* v, int d) -> float {  // element d of the rotated vector v
         const float x = Elt<T>::ld(v + d);
         if (d >= dims) return x;
         const float c = ct[d >> 1], s = st[d >> 1], o = Elt<T>::ld(v + (d ^ 1));
         return (d & 1) ? x * c + o * s : x * c - o * s;
     };
+    if (h < a.heads) {
+        const T* qh = row + h * (a.dim + rot);
+        T* qo = reinterpret_cast<T*>(p.q) + ((size_t)t * a.heads + h) * (p.plain_pad + p.rot_pad);
+        T* ql = reinterpret_cast<T*>(p.q_lat) + ((size_t)t * a.heads + h) * W + R;
+        if ((a.dim + rot) % 8 == 0 && a.dim % 8 == 0) {
+            for (int i = lane * 8; i < p.plain_pad; i += 256) {
+                float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+                if (i < a.dim) Elt<T>::ld8(qh + i, v);
+                Elt<T>::st8(qo + i, v);
+            }
+        } else {
+            for (int i = lane; i < p.plain_pad; i += 32) Elt<T>::st(qo + i, i < a.dim ? Elt<T>::ld(qh + i) : 0.f);
+        }
+        for (int i = lane; i < max(p.rot_pad, W - R); i += 32) {
+            const float v = i < rot ? turned(qh + a.dim, i) : 0.f;
+            if (i < p.rot_pad) Elt<T>::st(qo + p.plain_pad + i, v);
+            if (i < W - R) Elt<T>::st(ql + i, v);
+        }
+    }
+    if (blockIdx.y > 0) return;
     const T* lat = row + a.heads * (a.dim + rot);
+    const int slot = p.slot_mapping[t];
     float ss = 0.f;
-    for (int i = threadIdx.x; i < R; i += blockDim.x) {
+    for (int i = threadIdx.x; i < R; i += 256) {
         const float v = Elt<T>::ld(lat + i);
         ss += v * v;
     }
     ss = elt_block_sum(ss, red);
     const float inv = 1.0f / sqrtf(ss / (float)R + p.eps);
-    if (slot >= 0) {
-        T* crow = reinterpret_cast<T*>(p.cache) + (size_t)slot * W;
-        for (int i = threadIdx.x; i < W; i += blockDim.x)
-            Elt<T>::st(crow + i, i < R ? Elt<T>::ld(lat + i) * inv * p.c_norm[i] : (i < R + rot ? turned(lat + R, i - R) : 0.f));
-    }
-    const int QW = p.plain_pad + p.rot_pad;
-    T* qo = reinterpret_cast<T*>(p.q) + (size_t)t * a.heads * QW;
-    for (int i = threadIdx.x; i < a.heads * QW; i += blockDim.x) {
-        const int h = i / QW, d = i - h * QW;
-        const T* qh = row + h * (a.dim + rot);
-        if (d < a.dim)
-            qo[i] = qh[d];
-        else
-            Elt<T>::st(qo + i, d >= p.plain_pad && d - p.plain_pad < rot ? turned(qh + a.dim, d - p.plain_pad) : 0.f);
-    }
-    T* ql = reinterpret_cast<T*>(p.q_lat) + (size_t)t * a.heads * W;
-    const int tail = W - R;
-    for (int i = threadIdx.x; i < a.heads * tail; i += blockDim.x) {
-        const int h = i / tail, d = i - h * tail;
-        Elt<T>::st(ql + (size_t)h * W + R + d, d < rot ? turned(row + h * (a.dim + rot) + a.dim, d) : 0.f);
-    }
+    if (slot < 0) return;
+    T* crow = reinterpret_cast<T*>(p.cache) + (size_t)slot * W;
+    for (int i = threadIdx.x; i < W; i += 256)
+        Elt<T>::st(crow + i, i < R ? Elt<T>::ld(lat + i) * inv * p.c_norm[i] : (i < R + rot ? turned(lat + R, i - R) : 0.f));
 }
 
 // Plain form: one block per (token, head), 128 keys at a time with an online softmax, everything f32.
@@ -170,15 +174,22 @@ __global__ void __launch_bounds__(256, 1) latent_decode_kernel(const LatentAttnS
         const bool ok = h0 + r < a.heads;
         for (int c = lane; c < W / 8; c += 32) cp_async16_zfill(sQ + (r * LD + c * 8) * 2, q + (size_t)(ok ? h0 + r : 0) * W + c * 8, ok);
     }
+    // cache row of key (tile j, row warp + 8 * lane) in lanes 0-7, looked up a tile ahead; -1 past the chunk
+    auto rows_of = [&](int j) {
+        const int key = k_lo + j * DK_KEYS + warp + 8 * (lane & 7);
+        return key < k_hi ? bt[key / p.page_size] * p.page_size + key % p.page_size : -1;
+    };
+    int row_next = rows_of(0);
     auto load = [&](int j) {
-        const int k0 = k_lo + j * DK_KEYS;
         const uint32_t dst = sK + (j & 1) * DK_KEYS * LD * 2;
-        for (int r = warp; r < DK_KEYS; r += 8) {
-            const int key = k0 + r;
-            const bool ok = key < k_hi;
-            const int kk = ok ? key : k_lo;
-            const uint16_t* src = cache + ((size_t)bt[kk / p.page_size] * p.page_size + kk % p.page_size) * W;
-            for (int c = lane; c < W / 8; c += 32) cp_async16_zfill(dst + (r * LD + c * 8) * 2, src + c * 8, ok);
+        const int mine = row_next;
+        row_next = rows_of(j + 1);
+#pragma unroll
+        for (int i = 0; i < DK_KEYS / 8; i++) {
+            const int row = __shfl_sync(0xffffffffu, mine, i);
+            const uint16_t* src = cache + (size_t)max(row, 0) * W;
+            const uint32_t d = dst + (warp + 8 * i) * LD * 2;
+            for (int c = lane; c < W / 8; c += 32) cp_async16_zfill(d + c * 16, src + c * 8, row >= 0);
         }
     };
     load(0);
@@ -362,6 +373,7 @@ __global__ void __launch_bounds__(256, 1) latent_decode_kernel(const LatentAttnS
             for (int col = R + lane; col < p.o_pad; col += 32) out[(size_t)(h0 + r) * p.o_pad + col] = 0;
 }
 
+constexpr int kMergeTile = 128;
 // Sum of a row's chunks: out = sum_c 2^(m_c - M) O_c / sum_c 2^(m_c - M) l_c, M the largest m_c, chunks in order.
 __global__ void __launch_bounds__(128) latent_merge_kernel(const LatentAttnSpec a, const LatentDecodeParams p) {
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
@@ -370,18 +382,33 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const LatentAttnSpec 
     const int n = (p.ctx[sd] + chunk_keys - 1) / chunk_keys;
     if (n <= 1) return;
     const size_t at0 = (size_t)p.work_off[sd] * a.heads + h;
+    __shared__ float w[kMergeTile], sum[kMergeTile];  // maxima, then weights, of up to kMergeTile chunks; row sums
     float M = -INFINITY;
-    for (int c = 0; c < n; c++) M = fmaxf(M, p.part_ml[(at0 + (size_t)c * a.heads) * 2]);
+    for (int c = threadIdx.x; c < n; c += 128) M = fmaxf(M, p.part_ml[(at0 + (size_t)c * a.heads) * 2]);
+    M = elt_warp_max(M);
+    __shared__ float red[4];
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = M;
+    __syncthreads();
+    M = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
     float acc[DK_NJ] = {0.f, 0.f, 0.f, 0.f}, L = 0.f;  // columns threadIdx.x + 128 i (R up to 512)
+    for (int c0 = 0; c0 < n; c0 += kMergeTile) {
+        const int cnt = min(kMergeTile, n - c0);
+        __syncthreads();
+        for (int c = threadIdx.x; c < cnt; c += 128) {
+            const float2 ml = *reinterpret_cast<const float2*>(&p.part_ml[(at0 + (size_t)(c0 + c) * a.heads) * 2]);
+            w[c] = exp2f(ml.x - M);
+            sum[c] = ml.y;
+        }
+        __syncthreads();
 #pragma unroll 4
-    for (int c = 0; c < n; c++) {
-        const size_t at = at0 + (size_t)c * a.heads;
-        const float w = exp2f(p.part_ml[at * 2] - M);
-        L = fmaf(w, p.part_ml[at * 2 + 1], L);
+        for (int c = 0; c < cnt; c++) {
+            const float* o = p.part_o + (at0 + (size_t)(c0 + c) * a.heads) * R;
+            L = fmaf(w[c], sum[c], L);
 #pragma unroll
-        for (int i = 0; i < DK_NJ; i++) {
-            const int col = threadIdx.x + i * 128;
-            if (col < R) acc[i] = fmaf(w, p.part_o[at * R + col], acc[i]);
+            for (int i = 0; i < DK_NJ; i++) {
+                const int col = threadIdx.x + i * 128;
+                if (col < R) acc[i] = fmaf(w[c], o[col], acc[i]);
+            }
         }
     }
     const float inv = 1.0f / L;
@@ -418,7 +445,7 @@ int32_t b2_latent_decode_launch(b2_ctx* ctx, const LatentAttnSpec& a, const Late
 
 int32_t b2_latent_prep_launch(b2_ctx* ctx, bool f32, const LatentAttnSpec& a, const LatentPrepParams& p) {
     if (p.T <= 0) return B2_OK;
-    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, f32 ? latent_prep_kernel<float> : latent_prep_kernel<uint16_t>, dim3(p.T), dim3(256), 0, ctx->stream, a, p));
+    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, f32 ? latent_prep_kernel<float> : latent_prep_kernel<uint16_t>, dim3(p.T, (a.heads + 7) / 8), dim3(256), 0, ctx->stream, a, p));
     B2_LAUNCHED(ctx);
     return B2_OK;
 }

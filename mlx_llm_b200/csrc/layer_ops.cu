@@ -136,8 +136,13 @@ __global__ void argmax_rows_f32_kernel(const float* __restrict__ logits, int ld,
     const float* row = logits + (size_t)blockIdx.x * ld;
     float best = -INFINITY;
     int idx = 0x7fffffff;
-    for (int i = threadIdx.x; i < vocab; i += blockDim.x)
-        if (row[i] > best) best = row[i], idx = i;  // a thread's ids ascend: its first maximum is kept
+    for (int i = threadIdx.x * 4; i < vocab; i += blockDim.x * 4) {  // (ld is a multiple of 128) a thread's ids ascend: its first maximum is kept
+        const float4 v = *reinterpret_cast<const float4*>(row + i);
+        if (v.x > best) best = v.x, idx = i;
+        if (i + 1 < vocab && v.y > best) best = v.y, idx = i + 1;
+        if (i + 2 < vocab && v.z > best) best = v.z, idx = i + 2;
+        if (i + 3 < vocab && v.w > best) best = v.w, idx = i + 3;
+    }
     auto take = [&](float ov, int oi) {
         if (ov > best || (ov == best && oi < idx)) best = ov, idx = oi;
     };
@@ -222,7 +227,7 @@ int32_t b2_linear_f32_launch(b2_ctx* ctx, const float* x, int ldx, const float* 
 }
 int32_t b2_argmax_f32_launch(b2_ctx* ctx, const float* logits, int ld, int rows, int vocab, int32_t* out) {
     if (rows <= 0) return B2_OK;
-    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, argmax_rows_f32_kernel, dim3(rows), dim3(512), 0, ctx->stream, logits, ld, vocab, out));
+    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, argmax_rows_f32_kernel, dim3(rows), dim3(1024), 0, ctx->stream, logits, ld, vocab, out));
     B2_LAUNCHED(ctx);
     return B2_OK;
 }

@@ -9,15 +9,15 @@
 
 namespace {
 
-constexpr int kThreads = 256, kMaxExperts = 1024;
+constexpr int kMaxThreads = 1024, kMaxExperts = 1024;
 
-__global__ void __launch_bounds__(kThreads) route_kernel(const RouteParams p) {
+__global__ void __launch_bounds__(kMaxThreads) route_kernel(const RouteParams p) {
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     pdl_wait();
     extern __shared__ float sc[];  // [warps][experts]: logits of the token, -inf once taken
     __shared__ int cursor[kMaxExperts];
     __shared__ bool last;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = kThreads / 32, E = p.experts;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5, E = p.experts;
     float* s = sc + (size_t)warp * E;
     for (int t = blockIdx.x * warps + warp; t < p.T; t += gridDim.x * warps) {
         for (int e = lane; e < E; e += 32) s[e] = p.logits[(size_t)t * p.ld + e];
@@ -68,8 +68,8 @@ __global__ void __launch_bounds__(kThreads) route_kernel(const RouteParams p) {
         if (lane == 0) p.offsets[E] = base;
     }
     __syncthreads();
-    for (int e = threadIdx.x; e <= E; e += kThreads) p.counters[e] = 0;  // ready for the next launch
-    for (int i = threadIdx.x; i < p.T * p.top; i += kThreads) {
+    for (int e = threadIdx.x; e <= E; e += blockDim.x) p.counters[e] = 0;  // ready for the next launch
+    for (int i = threadIdx.x; i < p.T * p.top; i += blockDim.x) {
         const int e = __ldcg(&p.expert[i]), at = atomicAdd(&cursor[e], 1);
         p.pos[i] = at;
         p.src[at] = i / p.top;
@@ -97,10 +97,10 @@ int32_t b2_gather_rows_launch(b2_ctx* ctx, const uint16_t* x, const int32_t* src
 int32_t b2_route_launch(b2_ctx* ctx, const RouteParams& p) {
     if (p.T <= 0) return B2_OK;
     B2_REQUIRE(p.experts <= kMaxExperts, B2_ERR_UNSUPPORTED, "routing: at most 1024 experts");
-    const int warps = kThreads / 32;
+    const int warps = p.T <= 8 || p.experts > 256 ? 8 : 32;
     int grid = (p.T + warps - 1) / warps;
     if (grid > ctx->sm_count) grid = ctx->sm_count;
-    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, route_kernel, dim3(grid), dim3(kThreads), (size_t)warps * p.experts * 4, ctx->stream, p));
+    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, route_kernel, dim3(grid), dim3(warps * 32), (size_t)warps * p.experts * 4, ctx->stream, p));
     B2_LAUNCHED(ctx);
     return B2_OK;
 }

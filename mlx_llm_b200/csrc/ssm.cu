@@ -3,7 +3,7 @@
 //
 // Recurrent state of a sequence (f32, one slot per block-table row of the pool):
 //   S     [heads][vdim][state]
-//   conv  [channels][taps - 1]   the last inputs of the convolution, oldest first
+//   conv  [taps - 1][channels]   the last inputs of the convolution, oldest first
 // A sequence that starts in this step (nothing cached) starts from zero, whatever its slot held before.
 //
 // Per token and head:  d = softplus(dt + bias),  S <- exp(-exp(A_log) d) S + d x B^T,  y = S C + D x   (all f32).
@@ -23,40 +23,36 @@ __global__ void __launch_bounds__(256) conv_silu_kernel(const Mamba2Spec s, cons
     const int b = p.token_seq[t], start = p.cu_seqlens[b], i = t - start;
     const int before = p.context_lens[b] - (p.cu_seqlens[b + 1] - start);  // tokens the state has seen
     const T* u = reinterpret_cast<const T*>(p.zx) + s.inner() + ch;
-    const float* cs = p.state + (size_t)p.seq_slot[b] * p.slot_stride + (size_t)s.heads * s.vdim * s.state + (size_t)ch * (taps - 1);
+    const float* cs = p.state + (size_t)p.seq_slot[b] * p.slot_stride + (size_t)s.heads * s.vdim * s.state + ch;
     float v = p.conv_b[ch];
     for (int j = 0; j < taps; j++) {
         const int k = i - (taps - 1) + j;  // token of this step, or (negative) a kept one
-        const float in = k >= 0 ? Elt<T>::ld(u + (size_t)(start + k) * p.ld) : (before > 0 ? cs[k + taps - 1] : 0.f);
-        v = fmaf(p.conv_w[(size_t)ch * taps + j], in, v);
+        const float in = k >= 0 ? Elt<T>::ld(u + (size_t)(start + k) * p.ld) : (before > 0 ? cs[(size_t)(k + taps - 1) * C] : 0.f);
+        v = fmaf(p.conv_w[(size_t)j * C + ch], in, v);
     }
     Elt<T>::st(reinterpret_cast<T*>(p.xbc) + (size_t)t * p.ld_xbc + ch, silu_f32(v));
 }
 
-// The same for eight channels and CV_T tokens per thread (sizes and offsets that allow 16-byte accesses): weights stay in
+// The same for eight channels and a run of tokens per thread (sizes and offsets that allow 16-byte accesses): weights stay in
 // registers, the window slides while the tokens belong to one sequence.
-constexpr int CV_T = 8;
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(128) conv_silu8_kernel(const Mamba2Spec s, const SsmParams p) {
+__global__ void __launch_bounds__(128) conv_silu8_kernel(const Mamba2Spec s, const SsmParams p, int run) {
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     pdl_wait();
     const int ch = (blockIdx.x * 128 + threadIdx.x) * 8, C = s.channels();
     if (ch >= C) return;
     float w[TAPS][8], bias[8], win[TAPS][8];
+    Elt<float>::ld8(p.conv_b + ch, bias);
 #pragma unroll
-    for (int e = 0; e < 8; e++) {
-        bias[e] = p.conv_b[ch + e];
-#pragma unroll
-        for (int j = 0; j < TAPS; j++) w[j][e] = p.conv_w[(size_t)(ch + e) * TAPS + j];
-    }
+    for (int j = 0; j < TAPS; j++) Elt<float>::ld8(p.conv_w + (size_t)j * C + ch, w[j]);
     const T* u = reinterpret_cast<const T*>(p.zx) + s.inner() + ch;
     int cur = -1;
-    for (int t = blockIdx.y * CV_T; t < min((int)(blockIdx.y + 1) * CV_T, p.T); t++) {
+    for (int t = blockIdx.y * run; t < min((int)(blockIdx.y + 1) * run, p.T); t++) {
         const int b = p.token_seq[t];
         if (b != cur) {  // the inputs before this token: of this step, or the kept ones
             cur = b;
             const int start = p.cu_seqlens[b], before = p.context_lens[b] - (p.cu_seqlens[b + 1] - start);
-            const float* cs = p.state + (size_t)p.seq_slot[b] * p.slot_stride + (size_t)s.heads * s.vdim * s.state + (size_t)ch * (TAPS - 1);
+            const float* cs = p.state + (size_t)p.seq_slot[b] * p.slot_stride + (size_t)s.heads * s.vdim * s.state + ch;
 #pragma unroll
             for (int j = 1; j < TAPS; j++) {
                 const int k = t - start - TAPS + j;
@@ -64,7 +60,7 @@ __global__ void __launch_bounds__(128) conv_silu8_kernel(const Mamba2Spec s, con
                     Elt<T>::ld8(u + (size_t)(start + k) * p.ld, win[j]);
                 } else {
 #pragma unroll
-                    for (int e = 0; e < 8; e++) win[j][e] = before > 0 ? cs[e * (TAPS - 1) + k + TAPS - 1] : 0.f;
+                    for (int e = 0; e < 8; e++) win[j][e] = before > 0 ? cs[(size_t)(k + TAPS - 1) * C + e] : 0.f;
                 }
             }
         }
@@ -90,14 +86,14 @@ __global__ void __launch_bounds__(128) conv_silu8_kernel(const Mamba2Spec s, con
 template <typename T>
 __device__ __forceinline__ void keep_conv_inputs(const Mamba2Spec& s, const SsmParams& p, float* slot, int start, int n, int before, int h, int p0, int rows,
                                                  bool first_block) {
-    const int P = s.vdim, N = s.state, inner = s.inner(), taps = s.conv, per = s.heads / s.groups, grp = h / per;
+    const int P = s.vdim, N = s.state, inner = s.inner(), taps = s.conv, per = s.heads / s.groups, grp = h / per, C = s.channels();
     float* conv = slot + (size_t)s.heads * P * N;
     auto keep = [&](int ch) {
-        float* c = conv + (size_t)ch * (taps - 1);
+        float* c = conv + ch;
         const T* u = reinterpret_cast<const T*>(p.zx) + inner + ch;
         for (int j = 0; j < taps - 1; j++) {  // ascending: a shift reads places it has not overwritten yet
             const int k = n - (taps - 1) + j;
-            c[j] = k >= 0 ? Elt<T>::ld(u + (size_t)(start + k) * p.ld) : (before > 0 ? c[j + n] : 0.f);
+            c[(size_t)j * C] = k >= 0 ? Elt<T>::ld(u + (size_t)(start + k) * p.ld) : (before > 0 ? c[(size_t)(j + n) * C] : 0.f);
         }
     };
     for (int c = threadIdx.x; c < rows && p0 + c < P; c += blockDim.x) keep(h * P + p0 + c);
@@ -210,7 +206,7 @@ constexpr int CH_LN = CH_N + 8, CH_LP = CH_P + 8;            // row strides in s
 struct ChunkSmem {
     static constexpr int kIn = (2 * CH_T * CH_LN + CH_T * CH_LP) * 2;  // C | B | x of one chunk
     static constexpr int kXw = 2 * CH_T * CH_LP * 2, kS = 2 * CH_N * CH_LP * 2;
-    static constexpr int kBytes = 2 * kIn + kXw + kS + 4 * CH_T * 4;
+    static constexpr int kBytes = 2 * kIn + kXw + kS + 2 * 4 * CH_T * 4;
 };
 
 __global__ void __launch_bounds__(256, 1) chunk_scan_kernel(const Mamba2Spec s, const SsmParams p) {
@@ -226,8 +222,7 @@ __global__ void __launch_bounds__(256, 1) chunk_scan_kernel(const Mamba2Spec s, 
     uint8_t* const in0 = smem;
     uint16_t* xw = reinterpret_cast<uint16_t*>(smem + 2 * ChunkSmem::kIn);  // head, remainder [token][value row]
     uint16_t* sh = reinterpret_cast<uint16_t*>(smem + 2 * ChunkSmem::kIn + ChunkSmem::kXw);  // head, remainder [state row][value row]
-    float* dts = reinterpret_cast<float*>(smem + 2 * ChunkSmem::kIn + ChunkSmem::kXw + ChunkSmem::kS);
-    float *cum = dts + CH_T, *ecum = cum + CH_T, *wend = ecum + CH_T;
+    float* steps = reinterpret_cast<float*>(smem + 2 * ChunkSmem::kIn + ChunkSmem::kXw + ChunkSmem::kS);  // two chunks' step sizes and decays
     const uint16_t* zx = reinterpret_cast<const uint16_t*>(p.zx);
     const uint16_t* xbc = reinterpret_cast<const uint16_t*>(p.xbc) + (size_t)start * p.ld_xbc;
     const float A = expf(p.A_log[h]), bias = p.dt_bias[h], D = p.D[h];
@@ -276,36 +271,52 @@ __global__ void __launch_bounds__(256, 1) chunk_scan_kernel(const Mamba2Spec s, 
         }
     const int mt = warp >> 1, pc = (warp & 1) * 32;  // y: tokens mt * 16.., value rows pc..
     const int chunks = (n + CH_T - 1) / CH_T;
+    // Step sizes and decays of a chunk, two tokens per lane of warp 0 (which has the least of the triangular product): the raw
+    // values are fetched when the chunk before it begins and turned into factors when that warp is done with its part.
+    float raw[2] = {0.f, 0.f};
+    auto fetch_steps = [&](int c) {
+#pragma unroll
+        for (int i = 0; i < 2; i++) {
+            const int t = c * CH_T + 2 * lane + i;
+            raw[i] = t < n ? bf2f(zx[(size_t)(start + t) * p.ld + 2 * inner + 2 * s.groups * N + h]) : 0.f;
+        }
+    };
+    auto make_steps = [&](int c) {
+        float* dts = steps + (c & 1) * 4 * CH_T;
+        float d[2], run = 0.f;
+#pragma unroll
+        for (int i = 0; i < 2; i++) {
+            d[i] = c * CH_T + 2 * lane + i < n ? softplus_f32(raw[i] + bias) : 0.f;
+            run += -A * d[i];
+        }
+        float incl = run;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float u = __shfl_up_sync(0xffffffffu, incl, o);
+            if (lane >= o) incl += u;
+        }
+        const float end = __shfl_sync(0xffffffffu, incl, 31);
+        float at = incl - run;
+#pragma unroll
+        for (int i = 0; i < 2; i++) {
+            const int t = 2 * lane + i;
+            at += -A * d[i];
+            dts[t] = d[i];
+            dts[CH_T + t] = at;
+            dts[2 * CH_T + t] = expf(at);
+            dts[3 * CH_T + t] = expf(end - at) * d[i];
+        }
+    };
     load(0);
     cp_async_commit();
+    if (warp == 0) {
+        fetch_steps(0);
+        make_steps(0);
+    }
     for (int c = 0; c < chunks; c++) {
+        if (warp == 0 && c + 1 < chunks) fetch_steps(c + 1);
         const int t0 = c * CH_T, cnt = min(CH_T, n - t0);
-        if (warp == 0) {  // step sizes and decays: two tokens per lane
-            float d[2], run = 0.f;
-#pragma unroll
-            for (int i = 0; i < 2; i++) {
-                const int t = 2 * lane + i;
-                d[i] = t < cnt ? softplus_f32(bf2f(zx[(size_t)(start + t0 + t) * p.ld + 2 * inner + 2 * s.groups * N + h]) + bias) : 0.f;
-                run += -A * d[i];
-            }
-            float incl = run;
-#pragma unroll
-            for (int o = 1; o < 32; o <<= 1) {
-                const float u = __shfl_up_sync(0xffffffffu, incl, o);
-                if (lane >= o) incl += u;
-            }
-            const float end = __shfl_sync(0xffffffffu, incl, 31);
-            float at = incl - run;
-#pragma unroll
-            for (int i = 0; i < 2; i++) {
-                const int t = 2 * lane + i;
-                at += -A * d[i];
-                dts[t] = d[i];
-                cum[t] = at;
-                ecum[t] = expf(at);
-                wend[t] = expf(end - at) * d[i];
-            }
-        }
+        const float *dts = steps + (c & 1) * 4 * CH_T, *cum = dts + CH_T, *ecum = cum + CH_T, *wend = ecum + CH_T;
         // the state before this chunk, as operand of C S0
 #pragma unroll
         for (int j = 0; j < 8; j++)
@@ -396,10 +407,20 @@ __global__ void __launch_bounds__(256, 1) chunk_scan_kernel(const Mamba2Spec s, 
 #pragma unroll
         for (int j = 0; j < 4; j++)
 #pragma unroll
-            for (int e = 0; e < 4; e++) {
-                const int t = e < 2 ? ta : tb, q = pc + j * 8 + 2 * t4 + (e & 1);
-                if (t < cnt && p0 + q < P) p.y[(size_t)(start + t0 + t) * inner + h * P + p0 + q] = fmaf(D, bf2f(sx[t * CH_LP + q]), y[j][e]);
+            for (int half = 0; half < 2; half++) {
+                const int t = half ? tb : ta, q = pc + j * 8 + 2 * t4;
+                if (t >= cnt) continue;
+                const uint32_t x2 = *reinterpret_cast<const uint32_t*>(sx + t * CH_LP + q);
+                const float y0 = fmaf(D, bflo(x2), y[j][2 * half]), y1 = fmaf(D, bfhi(x2), y[j][2 * half + 1]);
+                float* o = p.y + (size_t)(start + t0 + t) * inner + h * P + p0 + q;
+                if (vec && p0 + q < P) {
+                    *reinterpret_cast<float2*>(o) = make_float2(y0, y1);
+                } else {
+                    if (p0 + q < P) o[0] = y0;
+                    if (p0 + q + 1 < P) o[1] = y1;
+                }
             }
+        if (warp == 0 && c + 1 < chunks) make_steps(c + 1);
         __syncthreads();  // xw is complete
         // ---- state of this warp
         if (warp < KN) {
@@ -489,9 +510,11 @@ template <typename T>
 int32_t launch_ssm(b2_ctx* ctx, const Mamba2Spec& s, const SsmParams& p) {
     B2_REQUIRE(p.T <= 65535, B2_ERR_UNSUPPORTED, "mamba2: too many tokens in one step");
     if (s.channels() % 8 == 0 && s.inner() % 8 == 0 && s.conv >= 2 && s.conv <= 4) {
-        const dim3 cgrid((s.channels() / 8 + 127) / 128, (p.T + CV_T - 1) / CV_T);
+        const int bx = (s.channels() / 8 + 127) / 128, want = 12 * ctx->sm_count / bx + 1;  // blocks along the tokens
+        const int run = p.T > want ? (p.T + want - 1) / want : 1;
+        const dim3 cgrid(bx, (p.T + run - 1) / run);
         auto ck = s.conv == 2 ? conv_silu8_kernel<T, 2> : s.conv == 3 ? conv_silu8_kernel<T, 3> : conv_silu8_kernel<T, 4>;
-        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, ck, cgrid, dim3(128), 0, ctx->stream, s, p));
+        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, ck, cgrid, dim3(128), 0, ctx->stream, s, p, run));
     } else {
         B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, conv_silu_kernel<T>, dim3((s.channels() + 255) / 256, p.T), dim3(256), 0, ctx->stream, s, p));
     }
