@@ -593,6 +593,7 @@ int32_t Fwd::latent(const LayerSpec& L, const LayerP& P, int l) {
             dp.block_tables = pool->block_tables;
             dp.max_blocks = pool->max_blocks;
             dp.page_size = pool->block_size;
+            dp.cache_rows = pool->max_pages * pool->block_size;
             int items = rows;
             if (listed) {
                 dp.ctx = s.mo->dec_ctx;
@@ -612,8 +613,7 @@ int32_t Fwd::latent(const LayerSpec& L, const LayerP& P, int l) {
                 dp.positions = s.mo->positions;
                 dp.token_seq = s.mo->token_seq;
                 dp.seq_slot = s.in->seq_slot;
-                dp.max_chunks = 1;
-                dp.chunk_tiles = (s.max_ctx + 15) / 16;
+                dp.chunk_tiles = up(s.max_ctx, 64) / 16;
             }
             dp.scale_log2 = scale_log2;
             dp.o_lat = b.o_lat;

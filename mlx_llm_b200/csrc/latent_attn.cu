@@ -5,6 +5,7 @@
 // so attention runs over the cached rows [c | rotated key] themselves, as one key/value head shared by every query head.
 #include "elt.cuh"
 #include "layer_kernels.h"
+#include "tc5.cuh"
 
 namespace {
 
@@ -117,197 +118,225 @@ __global__ void __launch_bounds__(128) latent_attn_simple_kernel(const LatentAtt
 // ---- decode: tensor cores, keys split over CTAs ---------------------------------------------------------------------
 // One cached row serves every head, so the heads are the rows of the matrix products:
 //   S [heads x keys] = Q [heads x W] . K^T,   O [heads x R] += P [heads x keys] . K[:, :R]
-// CTA = (one chunk of one sequence's keys, up to MT * 16 heads), 8 warps, 64 keys per tile, double-buffered cp.async.
-// Scores and weights are f32; the weights enter the second product as their bf16 head plus bf16 remainder.  For the
-// second product the warps split the R columns (16-column tiles w, w + 8, ...).  With more than one chunk a sequence's
-// partial results (f32) are added in chunk order by a second kernel: one block per (sequence, head), so that the sums of a
-// long context spread over the machine.
-constexpr int DK_KEYS = 64, DK_NJ = 4;  // keys per tile; 16-column tiles per warp (R up to 512)
-constexpr int kDecodeMaxRank = DK_NJ * 8 * 16;
-constexpr int PS = DK_KEYS + 8;         // row stride of the weights in shared memory
+// CTA = (one chunk of one sequence's keys, up to MT * 16 heads), 16 warps, 64 keys per tile.  Tiles arrive by TMA, a box of 16
+// keys x 64 values per copy located through the block table, into two 128-byte-swizzled buffers; the first warp issues
+// them.  Scores: warp = 16 heads x 8 MT keys x every other 64-wide block of W; the two halves of W are added through shared
+// memory, after which a warp owns 16 heads x 8 keys.  Scores and weights are f32; the weights enter the second product as
+// their bf16 head plus bf16 remainder, the warps splitting the R columns (16-column tiles w, w + 16).  Keys past the chunk
+// are other tokens' rows (finite) and get weight zero.  With more than one chunk a sequence's partial results (f32) are
+// added in chunk order by a second kernel: one block per (sequence, head), so that long contexts spread over the machine.
+constexpr int DK_KEYS = 64, DK_WARPS = 16, DK_NJ = 2;  // keys per tile; 16-column tiles per warp (R up to 512)
+constexpr int kDecodeMaxRank = DK_NJ * DK_WARPS * 16;
+constexpr int PS = DK_KEYS + 8;                        // row stride of the weights in shared memory
+constexpr int DK_BLOCK = DK_KEYS * 128;                // 64 keys x 64 values
 
 template <int MT>
 struct DecodeSmem {
-    static constexpr int H = MT * 16;
-    static __host__ __device__ int qk_bytes(int W) { return (H + 2 * DK_KEYS) * (W + 8) * 2; }
-    static __host__ __device__ int bytes(int W) { return qk_bytes(W) + 2 * H * PS * 2 + (8 * H * 2 + 3 * H) * 4; }
+    static constexpr int H = MT * 16, kQBlock = H * 128;
+    static __host__ __device__ int blocks(int W) { return (W + 63) / 64; }
+    static __host__ __device__ int q_off(int W) { return 2 * blocks(W) * DK_BLOCK; }
+    static __host__ __device__ int p_off(int W) { return q_off(W) + blocks(W) * kQBlock; }
+    static __host__ __device__ int bytes(int W) { return p_off(W) + 2 * H * PS * 2 + DK_WARPS * 32 * 4 * 4 + (2 * 8 * H + 3 * H) * 4 + 16; }
 };
 
 template <int MT>
-__global__ void __launch_bounds__(256, 1) latent_decode_kernel(const LatentAttnSpec a, const LatentDecodeParams p) {
+__global__ void __launch_bounds__(DK_WARPS * 32, 1)
+    latent_decode_kernel(const LatentAttnSpec a, const LatentDecodeParams p, int* err, const __grid_constant__ CUtensorMap map) {
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     pdl_wait();
-    constexpr int H = MT * 16, KW = MT == 2 ? 4 : 8, NK = 8 / KW;  // key groups of a tile, 8-key tiles per warp
-    extern __shared__ __align__(16) uint8_t smem[];
-    const int W = a.row_pad(), R = a.kv_rank, LD = W + 8;
-    const uint32_t sQ = smem_u32(smem), sK = sQ + H * LD * 2;
-    uint8_t* tail = smem + DecodeSmem<MT>::qk_bytes(W);
-    uint16_t *ph = reinterpret_cast<uint16_t*>(tail), *pl = ph + H * PS;
-    float *wmax = reinterpret_cast<float*>(pl + H * PS), *wsum = wmax + 8 * H, *rowm = wsum + 8 * H, *rowl = rowm + 2 * H;
+    using L = DecodeSmem<MT>;
+    constexpr int H = L::H;
+    extern __shared__ __align__(1024) uint8_t smem[];
+    const int W = a.row_pad(), R = a.kv_rank, NB = L::blocks(W);
+    const uint32_t base = smem_u32(smem);
+    if (base & 1023u) {  // the swizzled layout needs this alignment; every thread sees the same value
+        if (threadIdx.x == 0) atomicExch(err, 7);
+        return;
+    }
+    const uint32_t sQ = base + L::q_off(W);
+    uint16_t *ph = reinterpret_cast<uint16_t*>(smem + L::p_off(W)), *pl = ph + H * PS;
+    float *xch = reinterpret_cast<float*>(pl + H * PS), *wmax = xch + DK_WARPS * 32 * 4, *wsum = wmax + 8 * H, *rowm = wsum + 8 * H, *rowl = rowm + 2 * H;
+    const uint32_t full0 = smem_u32(rowl + H);
     const uint32_t sPh = smem_u32(ph), sPl = smem_u32(pl);
 
     const int item = blockIdx.x, h0 = blockIdx.y * H;
-    int sd, chunk, n_chunks, part0;  // row of the list, its chunk, chunks of the row, first partial slot of the row
+    int sd, chunk, part0;  // row of the list, its chunk, first partial slot of the row
     if (p.work_seq) {
         if (item >= *p.n_work) return;
         sd = p.work_seq[item];
         chunk = p.work_chunk[item];
         part0 = p.work_off[sd];
-    } else {  // every row has the same number of work items
-        sd = item / p.max_chunks;
-        chunk = item - sd * p.max_chunks;
-        part0 = sd * p.max_chunks;
+    } else {  // one work item per row
+        sd = item;
+        chunk = 0;
+        part0 = item;
     }
     const int ctx = p.ctx ? p.ctx[sd] : p.positions[sd] + 1, qrow = p.qrow ? p.qrow[sd] : sd;
     const int slot = p.slot ? p.slot[sd] : p.seq_slot[p.token_seq[sd]];
     const int chunk_keys = p.chunk_tiles * 16;
-    n_chunks = (ctx + chunk_keys - 1) / chunk_keys;
+    const int n_chunks = (ctx + chunk_keys - 1) / chunk_keys;
     if (chunk >= n_chunks) return;
     const int k_lo = chunk * chunk_keys, k_hi = min(ctx, k_lo + chunk_keys);
     const int n_tiles = (k_hi - k_lo + DK_KEYS - 1) / DK_KEYS;
     const int32_t* bt = p.block_tables + (size_t)slot * p.max_blocks;
-    const uint16_t* cache = reinterpret_cast<const uint16_t*>(p.cache);
     const uint16_t* q = reinterpret_cast<const uint16_t*>(p.q_lat) + (size_t)qrow * a.heads * W;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, mi = lane >> 3, lr = lane & 7;
 
-    for (int r = warp; r < H; r += 8) {
-        const bool ok = h0 + r < a.heads;
-        for (int c = lane; c < W / 8; c += 32) cp_async16_zfill(sQ + (r * LD + c * 8) * 2, q + (size_t)(ok ? h0 + r : 0) * W + c * 8, ok);
+    if (tid == 0) {
+        tc5::mbar_init(full0, 1);
+        tc5::mbar_init(full0 + 8, 1);
+        asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
     }
-    // cache row of key (tile j, row warp + 8 * lane) in lanes 0-7, looked up a tile ahead; -1 past the chunk
-    auto rows_of = [&](int j) {
-        const int key = k_lo + j * DK_KEYS + warp + 8 * (lane & 7);
-        return key < k_hi ? bt[key / p.page_size] * p.page_size + key % p.page_size : -1;
-    };
-    int row_next = rows_of(0);
-    auto load = [&](int j) {
-        const uint32_t dst = sK + (j & 1) * DK_KEYS * LD * 2;
-        const int mine = row_next;
-        row_next = rows_of(j + 1);
-#pragma unroll
-        for (int i = 0; i < DK_KEYS / 8; i++) {
-            const int row = __shfl_sync(0xffffffffu, mine, i);
-            const uint16_t* src = cache + (size_t)max(row, 0) * W;
-            const uint32_t d = dst + (warp + 8 * i) * LD * 2;
-            for (int c = lane; c < W / 8; c += 32) cp_async16_zfill(d + c * 16, src + c * 8, row >= 0);
-        }
-    };
-    load(0);
+    // queries: [64-value block][head][64 values], swizzled like the keys
+    for (int i = tid; i < H * NB * 8; i += DK_WARPS * 32) {
+        const int r = i / (NB * 8), c = i - r * (NB * 8);
+        const bool ok = h0 + r < a.heads && c * 8 < W;
+        cp_async16_zfill(sQ + (c >> 3) * L::kQBlock + r * 128 + (((c & 7) ^ (r & 7)) << 4), q + (ok ? (size_t)(h0 + r) * W + c * 8 : 0), ok);
+    }
     cp_async_commit();
     if (tid < H) {
         rowm[tid] = -INFINITY;
         rowl[tid] = 0.f;
     }
+    cp_async_wait<0>();
+    __syncthreads();
+    // warp 0: the copies of tile j, four boxes of 16 keys per 64-value block
+    auto load = [&](int j) {
+        const uint32_t full = full0 + (j & 1) * 8, dst = base + (j & 1) * NB * DK_BLOCK;
+        if (lane == 0) tc5::mbar_expect_tx(full, (uint32_t)NB * DK_BLOCK);
+        int row[4];  // a box past the chunk repeats the chunk's first page: any finite rows will do
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            const int key = k_lo + j * DK_KEYS + i * 16, kk = key < k_hi ? key : k_lo;
+            row[i] = bt[kk / p.page_size] * p.page_size + kk % p.page_size;
+        }
+        __syncwarp();
+        for (int i = lane; i < NB * 4; i += 32) {
+            const int s = i & 3;
+            tc5::tma_load_2d(dst + (i >> 2) * DK_BLOCK + s * 2048, &map, (i >> 2) * 64, s == 0 ? row[0] : s == 1 ? row[1] : s == 2 ? row[2] : row[3], full);
+        }
+    };
+    if (warp == 0) load(0);
+
     float acc[MT][DK_NJ * 2][4];
 #pragma unroll
     for (int m = 0; m < MT; m++)
 #pragma unroll
         for (int n = 0; n < DK_NJ * 2; n++) acc[m][n][0] = acc[m][n][1] = acc[m][n][2] = acc[m][n][3] = 0.f;
-    const int mw = MT == 2 ? (warp & 1) : 0, kw = MT == 2 ? (warp >> 1) : warp;
-    const int KS = W / 16, CT = (R + 15) / 16;
+    // scores: heads mw * 16.., keys kw * 8 MT.., blocks ks, ks + 2, ...
+    const int ks = warp & 1, mw = MT == 2 ? (warp >> 1) & 1 : 0, kw = MT == 2 ? warp >> 2 : warp >> 1;
+    const int own = MT == 2 ? kw * 2 + ks : kw;  // the 8 keys this warp turns into weights (MT 1: even warps only)
+    const bool owner = MT == 2 || ks == 0;
+    const int CT = (R + 15) / 16;
     const int row_a = mw * 16 + (lane >> 2), row_b = row_a + 8;
+    const uint32_t qa = sQ + (mw * 16 + lr + (mi & 1) * 8) * 128;
+    const uint32_t k_row = MT == 2 ? (uint32_t)(kw * 16 + lr + (mi >> 1) * 8) * 128 : (uint32_t)(kw * 8 + lr) * 128;
+    uint32_t offa[4], offb[4];
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        offa[i] = (uint32_t)(((2 * i + (mi >> 1)) ^ lr) << 4);
+        offb[i] = (uint32_t)(((2 * i + (mi & 1)) ^ lr) << 4);
+    }
+    bool alive = true;
     for (int j = 0; j < n_tiles; j++) {
-        if (j + 1 < n_tiles) load(j + 1);
-        cp_async_commit();
-        cp_async_wait<1>();
+        if (warp == 0 && j + 1 < n_tiles) load(j + 1);
+        alive = alive && tc5::mbar_wait(full0 + (j & 1) * 8, (uint32_t)(j >> 1) & 1u);
+        const uint32_t kb = base + (j & 1) * NB * DK_BLOCK;
+        float s[MT][4];
+#pragma unroll
+        for (int n = 0; n < MT; n++) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
+        for (int blk = ks; blk < NB; blk += 2) {
+            const uint32_t qb = qa + blk * L::kQBlock, kk = kb + k_row + blk * DK_BLOCK;
+#pragma unroll
+            for (int i = 0; i < 4; i++) {
+                uint32_t af[4];
+                ldmatrix_x4(af[0], af[1], af[2], af[3], qb + offa[i]);
+                if (MT == 2) {
+                    uint32_t b0[2], b1[2];
+                    ldmatrix_x4(b0[0], b0[1], b1[0], b1[1], kk + offb[i]);
+                    mma_bf16_16816(s[0], af, b0);
+                    mma_bf16_16816(s[MT - 1], af, b1);
+                } else {
+                    uint32_t b0[2];
+                    ldmatrix_x2(b0[0], b0[1], kk + offb[i]);
+                    mma_bf16_16816(s[0], af, b0);
+                }
+            }
+        }
+        // hand over what the other half's warp owns, take what this one owns
+        if (MT == 2)
+            *reinterpret_cast<float4*>(xch + (warp * 32 + lane) * 4) = ks ? make_float4(s[0][0], s[0][1], s[0][2], s[0][3])
+                                                                          : make_float4(s[MT - 1][0], s[MT - 1][1], s[MT - 1][2], s[MT - 1][3]);
+        else if (ks)
+            *reinterpret_cast<float4*>(xch + (warp * 32 + lane) * 4) = make_float4(s[0][0], s[0][1], s[0][2], s[0][3]);
         __syncthreads();
-        const uint32_t kb = sK + (j & 1) * DK_KEYS * LD * 2;
-        // ---- scores of this warp: 16 heads x NK * 8 keys
-        float s[NK][4];
+        float v[4], m0 = -INFINITY, m1 = -INFINITY;
+        if (owner) {
+            const float4 o = *reinterpret_cast<const float4*>(xch + ((warp ^ 1) * 32 + lane) * 4);
+            const float* mine = MT == 2 && ks ? s[MT - 1] : s[0];
+            v[0] = mine[0] + o.x, v[1] = mine[1] + o.y, v[2] = mine[2] + o.z, v[3] = mine[3] + o.w;
+            const int key = k_lo + j * DK_KEYS + own * 8 + 2 * (lane & 3);
+            const bool ok0 = key < k_hi, ok1 = key + 1 < k_hi;
+            v[0] = ok0 ? v[0] * p.scale_log2 : -INFINITY, v[1] = ok1 ? v[1] * p.scale_log2 : -INFINITY;
+            v[2] = ok0 ? v[2] * p.scale_log2 : -INFINITY, v[3] = ok1 ? v[3] * p.scale_log2 : -INFINITY;
+            m0 = fmaxf(v[0], v[1]);
+            m1 = fmaxf(v[2], v[3]);
 #pragma unroll
-        for (int n = 0; n < NK; n++) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
-        const uint32_t qa = sQ + ((mw * 16 + lr + (mi & 1) * 8) * LD + (mi >> 1) * 8) * 2;
-        if (NK == 2) {
-            const uint32_t ka = kb + ((kw * 16 + lr + (mi >> 1) * 8) * LD + (mi & 1) * 8) * 2;
-#pragma unroll 4
-            for (int k = 0; k < KS; k++) {
-                uint32_t af[4], b0[2], b1[2];
-                ldmatrix_x4(af[0], af[1], af[2], af[3], qa + k * 32);
-                ldmatrix_x4(b0[0], b0[1], b1[0], b1[1], ka + k * 32);
-                mma_bf16_16816(s[0], af, b0);
-                mma_bf16_16816(s[NK - 1], af, b1);
+            for (int o2 = 1; o2 < 4; o2 <<= 1) {
+                m0 = fmaxf(m0, __shfl_xor_sync(0xffffffffu, m0, o2));
+                m1 = fmaxf(m1, __shfl_xor_sync(0xffffffffu, m1, o2));
             }
-        } else {
-            const uint32_t ka = kb + ((kw * 8 + lr) * LD + (mi & 1) * 8) * 2;
-#pragma unroll 4
-            for (int k = 0; k < KS; k++) {
-                uint32_t af[4], b0[2];
-                ldmatrix_x4(af[0], af[1], af[2], af[3], qa + k * 32);
-                ldmatrix_x2(b0[0], b0[1], ka + k * 32);
-                mma_bf16_16816(s[0], af, b0);
+            if ((lane & 3) == 0) {
+                wmax[own * H + row_a] = m0;
+                wmax[own * H + row_b] = m1;
             }
-        }
-        float m0 = -INFINITY, m1 = -INFINITY;
-#pragma unroll
-        for (int n = 0; n < NK; n++)
-#pragma unroll
-            for (int e = 0; e < 4; e++) {
-                const int key = k_lo + j * DK_KEYS + kw * NK * 8 + n * 8 + 2 * (lane & 3) + (e & 1);
-                s[n][e] = key < k_hi ? s[n][e] * p.scale_log2 : -INFINITY;
-                if (e < 2)
-                    m0 = fmaxf(m0, s[n][e]);
-                else
-                    m1 = fmaxf(m1, s[n][e]);
-            }
-#pragma unroll
-        for (int o = 1; o < 4; o <<= 1) {
-            m0 = fmaxf(m0, __shfl_xor_sync(0xffffffffu, m0, o));
-            m1 = fmaxf(m1, __shfl_xor_sync(0xffffffffu, m1, o));
-        }
-        if ((lane & 3) == 0) {
-            wmax[kw * H + row_a] = m0;
-            wmax[kw * H + row_b] = m1;
         }
         __syncthreads();
-        // ---- weights: the tile's row maximum over all warps, then exp2; the first tile always has a visible key
-        const float *old_m = rowm + (j & 1) * H, *cur_m;
+        // weights: the row maximum over the tile and the tiles before, then exp2 (a chunk's first key is visible)
+        const float* old_m = rowm + (j & 1) * H;
         float* new_m = rowm + ((j & 1) ^ 1) * H;
-        m0 = old_m[row_a];
-        m1 = old_m[row_b];
+        if (owner) {
+            m0 = old_m[row_a];
+            m1 = old_m[row_b];
 #pragma unroll
-        for (int w = 0; w < KW; w++) {
-            m0 = fmaxf(m0, wmax[w * H + row_a]);
-            m1 = fmaxf(m1, wmax[w * H + row_b]);
-        }
-        float l0 = 0.f, l1 = 0.f;
-#pragma unroll
-        for (int n = 0; n < NK; n++) {
-            const float e0 = exp2f(s[n][0] - m0), e1 = exp2f(s[n][1] - m0), e2 = exp2f(s[n][2] - m1), e3 = exp2f(s[n][3] - m1);
-            l0 += e0 + e1;
-            l1 += e2 + e3;
-            const int col = kw * NK * 8 + n * 8 + 2 * (lane & 3);
+            for (int w = 0; w < 8; w++) {
+                m0 = fmaxf(m0, wmax[w * H + row_a]);
+                m1 = fmaxf(m1, wmax[w * H + row_b]);
+            }
+            const float e0 = fast_exp2(v[0] - m0), e1 = fast_exp2(v[1] - m0), e2 = fast_exp2(v[2] - m1), e3 = fast_exp2(v[3] - m1);
+            float l0 = e0 + e1, l1 = e2 + e3;
+            const int col = own * 8 + 2 * (lane & 3);
             const uint32_t ha = pack_bf2(e0, e1), hb = pack_bf2(e2, e3);
             *reinterpret_cast<uint32_t*>(ph + row_a * PS + col) = ha;
             *reinterpret_cast<uint32_t*>(ph + row_b * PS + col) = hb;
             *reinterpret_cast<uint32_t*>(pl + row_a * PS + col) = pack_bf2(e0 - bflo(ha), e1 - bfhi(ha));
             *reinterpret_cast<uint32_t*>(pl + row_b * PS + col) = pack_bf2(e2 - bflo(hb), e3 - bfhi(hb));
-        }
 #pragma unroll
-        for (int o = 1; o < 4; o <<= 1) {
-            l0 += __shfl_xor_sync(0xffffffffu, l0, o);
-            l1 += __shfl_xor_sync(0xffffffffu, l1, o);
-        }
-        if ((lane & 3) == 0) {
-            wsum[kw * H + row_a] = l0;
-            wsum[kw * H + row_b] = l1;
-            if (kw == 0) {
-                new_m[row_a] = m0;
-                new_m[row_b] = m1;
+            for (int o2 = 1; o2 < 4; o2 <<= 1) {
+                l0 += __shfl_xor_sync(0xffffffffu, l0, o2);
+                l1 += __shfl_xor_sync(0xffffffffu, l1, o2);
+            }
+            if ((lane & 3) == 0) {
+                wsum[own * H + row_a] = l0;
+                wsum[own * H + row_b] = l1;
+                if (own == 0) {
+                    new_m[row_a] = m0;
+                    new_m[row_b] = m1;
+                }
             }
         }
         __syncthreads();
-        // ---- O = alpha O + P K[:, :R]
-        cur_m = new_m;
+        // O = alpha O + P K[:, :R]
         if (tid < H) {
-            float l = rowl[tid] * exp2f(old_m[tid] - cur_m[tid]);
+            float l = rowl[tid] * fast_exp2(old_m[tid] - new_m[tid]);
 #pragma unroll
-            for (int w = 0; w < KW; w++) l += wsum[w * H + tid];
+            for (int w = 0; w < 8; w++) l += wsum[w * H + tid];
             rowl[tid] = l;
         }
 #pragma unroll
         for (int m = 0; m < MT; m++) {
             const int ra = m * 16 + (lane >> 2);
-            const float a0 = exp2f(old_m[ra] - cur_m[ra]), a1 = exp2f(old_m[ra + 8] - cur_m[ra + 8]);
+            const float a0 = fast_exp2(old_m[ra] - new_m[ra]), a1 = fast_exp2(old_m[ra + 8] - new_m[ra + 8]);
             if (__any_sync(0xffffffffu, a0 != 1.f || a1 != 1.f)) {
 #pragma unroll
                 for (int n = 0; n < DK_NJ * 2; n++) acc[m][n][0] *= a0, acc[m][n][1] *= a0, acc[m][n][2] *= a1, acc[m][n][3] *= a1;
@@ -324,22 +353,21 @@ __global__ void __launch_bounds__(256, 1) latent_decode_kernel(const LatentAttnS
             }
 #pragma unroll
             for (int c = 0; c < DK_NJ; c++) {
-                const int ct = warp + c * 8;
+                const int ct = warp + c * DK_WARPS;  // values ct * 16 ..: block ct / 4, 16-byte chunks (ct % 4) * 2, + 1
                 if (ct < CT) {
                     uint32_t v0[2], v1[2];
-                    ldmatrix_x4_trans(v0[0], v0[1], v1[0], v1[1], kb + ((k * 16 + lr + (mi & 1) * 8) * LD + ct * 16 + (mi >> 1) * 8) * 2);
+                    ldmatrix_x4_trans(v0[0], v0[1], v1[0], v1[1],
+                                      kb + (ct >> 2) * DK_BLOCK + (k * 16 + lr + (mi & 1) * 8) * 128 + ((((ct & 3) * 2 + (mi >> 1)) ^ lr) << 4));
 #pragma unroll
-                    for (int m = 0; m < MT; m++) {
-                        mma_bf16_16816(acc[m][2 * c], fh[m], v0);
-                        mma_bf16_16816(acc[m][2 * c + 1], fh[m], v1);
-                        mma_bf16_16816(acc[m][2 * c], fl[m], v0);
-                        mma_bf16_16816(acc[m][2 * c + 1], fl[m], v1);
-                    }
+                    for (int m = 0; m < MT; m++) mma_bf16_16816(acc[m][2 * c], fh[m], v0), mma_bf16_16816(acc[m][2 * c + 1], fh[m], v1);
+#pragma unroll
+                    for (int m = 0; m < MT; m++) mma_bf16_16816(acc[m][2 * c], fl[m], v0), mma_bf16_16816(acc[m][2 * c + 1], fl[m], v1);
                 }
             }
         }
         __syncthreads();  // the tile's buffer, the weights and the row statistics may be overwritten
     }
+    if (!alive && lane == 0) atomicExch(err, 15);
     const float* fin_m = rowm + (n_tiles & 1) * H;
     uint16_t* out = reinterpret_cast<uint16_t*>(p.o_lat) + (size_t)qrow * a.heads * p.o_pad;
 #pragma unroll
@@ -351,8 +379,8 @@ __global__ void __launch_bounds__(256, 1) latent_decode_kernel(const LatentAttnS
             const float inv = 1.0f / rowl[r];
 #pragma unroll
             for (int c = 0; c < DK_NJ * 2; c++) {
-                const int col = (warp + (c >> 1) * 8) * 16 + (c & 1) * 8 + 2 * (lane & 3);
-                if ((warp + (c >> 1) * 8) >= CT) continue;
+                const int ct = warp + (c >> 1) * DK_WARPS, col = ct * 16 + (c & 1) * 8 + 2 * (lane & 3);
+                if (ct >= CT) continue;
 #pragma unroll
                 for (int e = 0; e < 2; e++) {
                     if (col + e >= R) continue;
@@ -369,7 +397,7 @@ __global__ void __launch_bounds__(256, 1) latent_decode_kernel(const LatentAttnS
             }
         }
     if (R < p.o_pad && chunk == 0)  // the padding the value projection reads
-        for (int r = warp; r < H && h0 + r < a.heads; r += 8)
+        for (int r = warp; r < H && h0 + r < a.heads; r += DK_WARPS)
             for (int col = R + lane; col < p.o_pad; col += 32) out[(size_t)(h0 + r) * p.o_pad + col] = 0;
 }
 
@@ -390,7 +418,7 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const LatentAttnSpec 
     if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = M;
     __syncthreads();
     M = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
-    float acc[DK_NJ] = {0.f, 0.f, 0.f, 0.f}, L = 0.f;  // columns threadIdx.x + 128 i (R up to 512)
+    float acc[4] = {0.f, 0.f, 0.f, 0.f}, L = 0.f;  // columns threadIdx.x + 128 i (R up to 512)
     for (int c0 = 0; c0 < n; c0 += kMergeTile) {
         const int cnt = min(kMergeTile, n - c0);
         __syncthreads();
@@ -405,7 +433,7 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const LatentAttnSpec 
             const float* o = p.part_o + (at0 + (size_t)(c0 + c) * a.heads) * R;
             L = fmaf(w[c], sum[c], L);
 #pragma unroll
-            for (int i = 0; i < DK_NJ; i++) {
+            for (int i = 0; i < 4; i++) {
                 const int col = threadIdx.x + i * 128;
                 if (col < R) acc[i] = fmaf(w[c], o[col], acc[i]);
             }
@@ -414,7 +442,7 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const LatentAttnSpec 
     const float inv = 1.0f / L;
     uint16_t* out = reinterpret_cast<uint16_t*>(p.o_lat) + ((size_t)p.qrow[sd] * a.heads + h) * p.o_pad;
 #pragma unroll
-    for (int i = 0; i < DK_NJ; i++) {
+    for (int i = 0; i < 4; i++) {
         const int col = threadIdx.x + i * 128;
         if (col < R) out[col] = f2bf(acc[i] * inv);
     }
@@ -428,13 +456,13 @@ bool b2_latent_decode_eligible(const LatentAttnSpec& a) {
 int32_t b2_latent_decode_launch(b2_ctx* ctx, const LatentAttnSpec& a, const LatentDecodeParams& p, int items, int rows) {
     if (items <= 0) return B2_OK;
     const dim3 grid(items, a.heads > 16 ? (a.heads + 31) / 32 : 1);
-    if (a.heads > 16) {
-        B2_SMEM_ONCE(ctx, latent_decode_kernel<2>, 226 * 1024);
-        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, latent_decode_kernel<2>, grid, dim3(256), (size_t)DecodeSmem<2>::bytes(a.row_pad()), ctx->stream, a, p));
-    } else {
-        B2_SMEM_ONCE(ctx, latent_decode_kernel<1>, 226 * 1024);
-        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, latent_decode_kernel<1>, grid, dim3(256), (size_t)DecodeSmem<1>::bytes(a.row_pad()), ctx->stream, a, p));
-    }
+    CUtensorMap map;
+    B2_CHECK(tc5::get_map(ctx, p.cache, (uint64_t)p.cache_rows, (uint64_t)a.row_pad(), (uint64_t)a.row_pad(), 16, &map));
+    B2_SMEM_ONCE(ctx, latent_decode_kernel<1>, 226 * 1024);
+    B2_SMEM_ONCE(ctx, latent_decode_kernel<2>, 226 * 1024);
+    const int smem = a.heads > 16 ? DecodeSmem<2>::bytes(a.row_pad()) : DecodeSmem<1>::bytes(a.row_pad());
+    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, a.heads > 16 ? latent_decode_kernel<2> : latent_decode_kernel<1>, grid, dim3(DK_WARPS * 32), (size_t)smem, ctx->stream, a,
+                          p, ctx->dev_err, map));
     B2_LAUNCHED(ctx);
     if (items > rows) {  // some row has more than one chunk
         B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, latent_merge_kernel, dim3(rows, a.heads), dim3(128), 0, ctx->stream, a, p));

@@ -108,10 +108,10 @@ struct LatentDecodeParams {
     // rows: the packer's decode list (context, token row, block-table row), or (ctx null) every token of the step
     const int32_t *ctx, *qrow, *slot;
     const int32_t *positions, *token_seq, *seq_slot;
-    // work items (row, chunk): the packer's list, or (work_seq null) max_chunks items per row
+    // work items (row, chunk): the packer's list, or (work_seq null) one per row, whose chunk must hold its whole context
     const int32_t *work_seq, *work_chunk, *work_off, *n_work;
-    int max_chunks;
-    int chunk_tiles;   // 16-key tiles per chunk
+    int chunk_tiles;   // 16-key tiles per chunk (a multiple of 4)
+    int64_t cache_rows;  // rows of the cache allocation
     float scale_log2;  // scale * log2(e)
     float *part_o, *part_ml;  // [work item][head][kv_rank], [work item][head][2]
     void* o_lat;

@@ -29,7 +29,8 @@ struct LatentAttnSpec {
     float scale = 0.f;
     PairRotSpec rot;
     constexpr int row() const { return kv_rank + rot_dim; }               // values cached per token
-    constexpr int row_pad() const { return (row() + 15) / 16 * 16; }      // ... padded for 16-wide tensor-core steps
+    // ... padded for 16-wide tensor-core steps, and to one 64-wide load box at least
+    constexpr int row_pad() const { return row() < 64 ? 64 : (row() + 15) / 16 * 16; }
 };
 // Selective state space with a scalar decay per head: inputs pass a short causal convolution, the state is
 // [heads][vdim][state] in f32, the output is gated and normed in groups.
