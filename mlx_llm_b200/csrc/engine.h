@@ -224,5 +224,5 @@ struct LayeredStep {
 };
 int32_t b2_forward_layered(b2_model* m, b2_pool* pool, const LayeredStep& s, float** logits_dev, int* logits_ld);
 int b2_layered_q_tile(const b2_model* m);
-int b2_layered_chunk_tiles(const b2_model* m, long dec_ctx_sum);  // 16-key tiles per work item of the decode attention
+int b2_layered_chunk_tiles(const b2_model* m, const std::vector<SeqStep>& seqs);  // 16-key tiles per work item of the decode attention
 bool b2_tensor_to_f32(const HostTensor& t, std::vector<float>& out);

@@ -764,10 +764,34 @@ int32_t Fwd::moe(const LayerSpec& L, const LayerP& P, const int32_t** rows) {
 }  // namespace
 
 int b2_layered_q_tile(const b2_model*) { return 128; }
-int b2_layered_chunk_tiles(const b2_model* m, long dec_ctx_sum) {
-    // about three CTAs per SM (one is resident), 128 to 2048 keys each, whole 64-key tiles
-    const long keys = dec_ctx_sum / (3l * m->ctx->sm_count);
-    return up((int)std::min(2048l, std::max(128l, keys)), 64) / 16;
+// One CTA of the decode attention fills an SM, so the work items (times the head groups) should fill whole rounds of the
+// machine: the smallest chunk, in whole 64-key tiles from 128 keys on, that does not open another round.
+int b2_layered_chunk_tiles(const b2_model* m, const std::vector<SeqStep>& seqs) {
+    int groups = 1;
+    for (auto& L : m->layered->spec.layers)
+        if (L.mixer == MixerKind::LatentAttention && L.attn.heads > 16) groups = std::max(groups, (L.attn.heads + 31) / 32);
+    int rows = 0, longest = 1;
+    for (auto& s : seqs)
+        if (s.n == 1) {
+            rows++;
+            longest = std::max(longest, s.cache->len + 1);
+        }
+    const int sms = m->ctx->sm_count, budget = std::max(1, (rows * groups + sms - 1) / sms) * sms / groups;
+    auto items = [&](int keys) {
+        int n = 0;
+        for (auto& s : seqs)
+            if (s.n == 1) n += (s.cache->len + keys) / keys;
+        return n;
+    };
+    int lo = 2, hi = std::max(2, (longest + 63) / 64);  // in 64-key tiles; a chunk of the longest context is one item per row
+    while (lo < hi) {
+        const int mid = (lo + hi) / 2;
+        if (items(mid * 64) <= budget)
+            hi = mid;
+        else
+            lo = mid + 1;
+    }
+    return lo * 4;
 }
 
 void b2_layered_cache_layout(const b2_model* m, int block_size, std::vector<std::vector<size_t>>& page_bytes, int64_t& state_floats) {

@@ -330,7 +330,7 @@ int32_t b2_engine_forward(b2_model* m, std::vector<SeqStep>& seqs, void* logits_
     B2_CHECK(m->layered ? b2_layered_ensure_rope(m, max_pos) : b2_model_ensure_rope(m, max_pos));
     // pages for the new tokens (host allocator), then the step descriptors
     for (auto& s : seqs) B2_CHECK(b2_cache_reserve(s.cache, s.n));
-    const int chunk_tiles = m->layered ? b2_layered_chunk_tiles(m, dec_ctx_sum) : pick_chunk_tiles(dec_ctx_sum, m->hkv_l, ctx->sm_count);
+    const int chunk_tiles = m->layered ? b2_layered_chunk_tiles(m, seqs) : pick_chunk_tiles(dec_ctx_sum, m->hkv_l, ctx->sm_count);
     const int q_tile = m->layered ? b2_layered_q_tile(m) : b2_prefill_q_tile(ctx, c.head_dim);
     int W = 0, P = 0;
     double pf_flops = 0;  // 4*hd*hq flops per (query, visible key) pair

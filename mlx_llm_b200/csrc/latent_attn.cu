@@ -119,8 +119,8 @@ __global__ void __launch_bounds__(128) latent_attn_simple_kernel(const LatentAtt
 // One cached row serves every head, so the heads are the rows of the matrix products:
 //   S [heads x keys] = Q [heads x W] . K^T,   O [heads x R] += P [heads x keys] . K[:, :R]
 // CTA = (one chunk of one sequence's keys, up to MT * 16 heads), 16 warps, 64 keys per tile.  Tiles arrive by TMA, a box of 16
-// keys x 64 values per copy located through the block table, into two 128-byte-swizzled buffers; the first warp issues
-// them.  Scores: warp = 16 heads x 8 MT keys x every other 64-wide block of W; the two halves of W are added through shared
+// keys x 64 values per copy located through the block table, into two 128-byte-swizzled buffers; a seventeenth warp
+// issues them.  Scores: warp = 16 heads x 8 MT keys x every other 64-wide block of W; the two halves of W are added through shared
 // memory, after which a warp owns 16 heads x 8 keys.  Scores and weights are f32; the weights enter the second product as
 // their bf16 head plus bf16 remainder, the warps splitting the R columns (16-column tiles w, w + 16).  Keys past the chunk
 // are other tokens' rows (finite) and get weight zero.  With more than one chunk a sequence's partial results (f32) are
@@ -136,11 +136,14 @@ struct DecodeSmem {
     static __host__ __device__ int blocks(int W) { return (W + 63) / 64; }
     static __host__ __device__ int q_off(int W) { return 2 * blocks(W) * DK_BLOCK; }
     static __host__ __device__ int p_off(int W) { return q_off(W) + blocks(W) * kQBlock; }
-    static __host__ __device__ int bytes(int W) { return p_off(W) + 2 * H * PS * 2 + DK_WARPS * 32 * 4 * 4 + (2 * 8 * H + 3 * H) * 4 + 16; }
+    static __host__ __device__ int bytes(int W) { return p_off(W) + 2 * H * PS * 2 + DK_WARPS * 32 * 4 * 4 + (2 * 8 * H + 3 * H) * 4 + 32; }
 };
 
+// barrier of the sixteen computing warps
+__device__ __forceinline__ void dk_sync() { asm volatile("bar.sync 1, %0;\n" ::"n"(DK_WARPS * 32) : "memory"); }
+
 template <int MT>
-__global__ void __launch_bounds__(DK_WARPS * 32, 1)
+__global__ void __launch_bounds__(DK_WARPS * 32 + 32, 1)
     latent_decode_kernel(const LatentAttnSpec a, const LatentDecodeParams p, int* err, const __grid_constant__ CUtensorMap map) {
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     pdl_wait();
@@ -182,41 +185,51 @@ __global__ void __launch_bounds__(DK_WARPS * 32, 1)
     const uint16_t* q = reinterpret_cast<const uint16_t*>(p.q_lat) + (size_t)qrow * a.heads * W;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, mi = lane >> 3, lr = lane & 7;
 
+    const uint32_t empty0 = full0 + 16;
     if (tid == 0) {
-        tc5::mbar_init(full0, 1);
-        tc5::mbar_init(full0 + 8, 1);
+        for (int i = 0; i < 2; i++) {
+            tc5::mbar_init(full0 + 8 * i, 1);
+            tc5::mbar_init(empty0 + 8 * i, DK_WARPS);
+        }
         asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
     }
-    // queries: [64-value block][head][64 values], swizzled like the keys
-    for (int i = tid; i < H * NB * 8; i += DK_WARPS * 32) {
-        const int r = i / (NB * 8), c = i - r * (NB * 8);
-        const bool ok = h0 + r < a.heads && c * 8 < W;
-        cp_async16_zfill(sQ + (c >> 3) * L::kQBlock + r * 128 + (((c & 7) ^ (r & 7)) << 4), q + (ok ? (size_t)(h0 + r) * W + c * 8 : 0), ok);
-    }
-    cp_async_commit();
     if (tid < H) {
         rowm[tid] = -INFINITY;
         rowl[tid] = 0.f;
     }
-    cp_async_wait<0>();
     __syncthreads();
-    // warp 0: the copies of tile j, four boxes of 16 keys per 64-value block
-    auto load = [&](int j) {
-        const uint32_t full = full0 + (j & 1) * 8, dst = base + (j & 1) * NB * DK_BLOCK;
-        if (lane == 0) tc5::mbar_expect_tx(full, (uint32_t)NB * DK_BLOCK);
-        int row[4];  // a box past the chunk repeats the chunk's first page: any finite rows will do
-#pragma unroll
-        for (int i = 0; i < 4; i++) {
-            const int key = k_lo + j * DK_KEYS + i * 16, kk = key < k_hi ? key : k_lo;
-            row[i] = bt[kk / p.page_size] * p.page_size + kk % p.page_size;
+    if (warp == DK_WARPS) {
+        // tile j: four boxes of 16 keys per 64-value block, spread over the lanes; page rows looked up a tile ahead
+        const int sub = lane & 3;
+        auto row_of = [&](int j) {  // a box past the chunk repeats the chunk's first page: any finite rows will do
+            const int key = k_lo + j * DK_KEYS + sub * 16, kk = key < k_hi ? key : k_lo;
+            return bt[kk / p.page_size] * p.page_size + kk % p.page_size;
+        };
+        int next = row_of(0);
+        for (int j = 0; j < n_tiles; j++) {
+            const int row = next, st = j & 1;
+            next = row_of(j + 1);
+            if (!__all_sync(0xffffffffu, tc5::mbar_wait(empty0 + 8 * st, ((uint32_t)(j >> 1) & 1u) ^ 1u))) {
+                if (lane == 0) atomicExch(err, 16);
+                return;
+            }
+            if (lane == 0) tc5::mbar_expect_tx(full0 + 8 * st, (uint32_t)NB * DK_BLOCK);
+            __syncwarp();
+            for (int i = lane >> 2; i < NB; i += 8) tc5::tma_load_2d(base + (st * NB + i) * DK_BLOCK + sub * 2048, &map, i * 64, row, full0 + 8 * st);
         }
-        __syncwarp();
-        for (int i = lane; i < NB * 4; i += 32) {
-            const int s = i & 3;
-            tc5::tma_load_2d(dst + (i >> 2) * DK_BLOCK + s * 2048, &map, (i >> 2) * 64, s == 0 ? row[0] : s == 1 ? row[1] : s == 2 ? row[2] : row[3], full);
+        return;
+    }
+    // queries: [64-value block][head][64 values], swizzled like the keys
+    for (int r = warp; r < H; r += DK_WARPS) {
+        const bool ok = h0 + r < a.heads;
+        for (int c = lane; c < NB * 8; c += 32) {
+            const bool in = ok && c * 8 < W;
+            cp_async16_zfill(sQ + (c >> 3) * L::kQBlock + r * 128 + (((c & 7) ^ (r & 7)) << 4), q + (in ? (size_t)(h0 + r) * W + c * 8 : 0), in);
         }
-    };
-    if (warp == 0) load(0);
+    }
+    cp_async_commit();
+    cp_async_wait<0>();
+    dk_sync();
 
     float acc[MT][DK_NJ * 2][4];
 #pragma unroll
@@ -239,7 +252,6 @@ __global__ void __launch_bounds__(DK_WARPS * 32, 1)
     }
     bool alive = true;
     for (int j = 0; j < n_tiles; j++) {
-        if (warp == 0 && j + 1 < n_tiles) load(j + 1);
         alive = alive && tc5::mbar_wait(full0 + (j & 1) * 8, (uint32_t)(j >> 1) & 1u);
         const uint32_t kb = base + (j & 1) * NB * DK_BLOCK;
         float s[MT][4];
@@ -269,7 +281,7 @@ __global__ void __launch_bounds__(DK_WARPS * 32, 1)
                                                                           : make_float4(s[MT - 1][0], s[MT - 1][1], s[MT - 1][2], s[MT - 1][3]);
         else if (ks)
             *reinterpret_cast<float4*>(xch + (warp * 32 + lane) * 4) = make_float4(s[0][0], s[0][1], s[0][2], s[0][3]);
-        __syncthreads();
+        dk_sync();
         float v[4], m0 = -INFINITY, m1 = -INFINITY;
         if (owner) {
             const float4 o = *reinterpret_cast<const float4*>(xch + ((warp ^ 1) * 32 + lane) * 4);
@@ -291,7 +303,7 @@ __global__ void __launch_bounds__(DK_WARPS * 32, 1)
                 wmax[own * H + row_b] = m1;
             }
         }
-        __syncthreads();
+        dk_sync();
         // weights: the row maximum over the tile and the tiles before, then exp2 (a chunk's first key is visible)
         const float* old_m = rowm + (j & 1) * H;
         float* new_m = rowm + ((j & 1) ^ 1) * H;
@@ -325,7 +337,7 @@ __global__ void __launch_bounds__(DK_WARPS * 32, 1)
                 }
             }
         }
-        __syncthreads();
+        dk_sync();
         // O = alpha O + P K[:, :R]
         if (tid < H) {
             float l = rowl[tid] * fast_exp2(old_m[tid] - new_m[tid]);
@@ -365,7 +377,9 @@ __global__ void __launch_bounds__(DK_WARPS * 32, 1)
                 }
             }
         }
-        __syncthreads();  // the tile's buffer, the weights and the row statistics may be overwritten
+        __syncwarp();
+        if (lane == 0) tc5::mbar_arrive(empty0 + 8 * (j & 1));  // (behind the warp's last read of the tile)
+        dk_sync();  // the weights and the row statistics may be overwritten
     }
     if (!alive && lane == 0) atomicExch(err, 15);
     const float* fin_m = rowm + (n_tiles & 1) * H;
@@ -377,18 +391,20 @@ __global__ void __launch_bounds__(DK_WARPS * 32, 1)
             const int r = m * 16 + (lane >> 2) + half * 8, h = h0 + r;
             if (h >= a.heads) continue;
             const float inv = 1.0f / rowl[r];
+            uint16_t* orow = out + (size_t)h * p.o_pad;
+            float* prow = p.part_o + ((size_t)(part0 + chunk) * a.heads + h) * R;
 #pragma unroll
             for (int c = 0; c < DK_NJ * 2; c++) {
                 const int ct = warp + (c >> 1) * DK_WARPS, col = ct * 16 + (c & 1) * 8 + 2 * (lane & 3);
-                if (ct >= CT) continue;
-#pragma unroll
-                for (int e = 0; e < 2; e++) {
-                    if (col + e >= R) continue;
-                    const float v = acc[m][c][half * 2 + e];
-                    if (n_chunks == 1)
-                        out[(size_t)h * p.o_pad + col + e] = f2bf(v * inv);
-                    else
-                        p.part_o[((size_t)(part0 + chunk) * a.heads + h) * R + col + e] = v;
+                if (ct >= CT || col >= R) continue;
+                const float v0 = acc[m][c][half * 2], v1 = acc[m][c][half * 2 + 1];
+                if (n_chunks == 1) {  // columns up to o_pad may be written: those past R are zero weights' inputs, cleared below
+                    *reinterpret_cast<uint32_t*>(orow + col) = pack_bf2(v0 * inv, col + 1 < R ? v1 * inv : 0.f);
+                } else if (R % 2 == 0) {
+                    *reinterpret_cast<float2*>(prow + col) = make_float2(v0, v1);
+                } else {
+                    prow[col] = v0;
+                    if (col + 1 < R) prow[col + 1] = v1;
                 }
             }
             if (n_chunks > 1 && warp == 0 && (lane & 3) == 0) {
@@ -461,7 +477,7 @@ int32_t b2_latent_decode_launch(b2_ctx* ctx, const LatentAttnSpec& a, const Late
     B2_SMEM_ONCE(ctx, latent_decode_kernel<1>, 226 * 1024);
     B2_SMEM_ONCE(ctx, latent_decode_kernel<2>, 226 * 1024);
     const int smem = a.heads > 16 ? DecodeSmem<2>::bytes(a.row_pad()) : DecodeSmem<1>::bytes(a.row_pad());
-    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, a.heads > 16 ? latent_decode_kernel<2> : latent_decode_kernel<1>, grid, dim3(DK_WARPS * 32), (size_t)smem, ctx->stream, a,
+    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, a.heads > 16 ? latent_decode_kernel<2> : latent_decode_kernel<1>, grid, dim3(DK_WARPS * 32 + 32), (size_t)smem, ctx->stream, a,
                           p, ctx->dev_err, map));
     B2_LAUNCHED(ctx);
     if (items > rows) {  // some row has more than one chunk
