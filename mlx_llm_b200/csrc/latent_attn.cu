@@ -115,54 +115,67 @@ __global__ void __launch_bounds__(128) latent_attn_simple_kernel(const LatentAtt
     for (int i = threadIdx.x; i < p.o_pad; i += 128) Elt<T>::st(o + i, i < R ? acc[i] / l : 0.f);
 }
 
-// ---- decode: tensor cores, keys split over CTAs ---------------------------------------------------------------------
-// One cached row serves every head, so the heads are the rows of the matrix products:
-//   S [heads x keys] = Q [heads x W] . K^T,   O [heads x R] += P [heads x keys] . K[:, :R]
-// CTA = (one chunk of one sequence's keys, up to MT * 16 heads), 16 warps, 64 keys per tile.  Tiles arrive by TMA, a box of 16
-// keys x 64 values per copy located through the block table, into two 128-byte-swizzled buffers; a seventeenth warp
-// issues them.  Scores: warp = 16 heads x 8 MT keys x every other 64-wide block of W; the two halves of W are added through shared
-// memory, after which a warp owns 16 heads x 8 keys.  Scores and weights are f32; the weights enter the second product as
-// their bf16 head plus bf16 remainder, the warps splitting the R columns (16-column tiles w, w + 16).  Keys past the chunk
-// are other tokens' rows (finite) and get weight zero.  With more than one chunk a sequence's partial results (f32) are
-// added in chunk order by a second kernel: one block per (sequence, head), so that long contexts spread over the machine.
-constexpr int DK_KEYS = 64, DK_WARPS = 16, DK_NJ = 2;  // keys per tile; 16-column tiles per warp (R up to 512)
-constexpr int kDecodeMaxRank = DK_NJ * DK_WARPS * 16;
-constexpr int PS = DK_KEYS + 8;                        // row stride of the weights in shared memory
-constexpr int DK_BLOCK = DK_KEYS * 128;                // 64 keys x 64 values
+// ---- decode: tcgen05, keys split over CTAs -----------------------------------------------------------------------------
+// One cached row serves every head, so the heads are rows of one product and columns of the other:
+//   S [heads x keys] = Q [heads x W] . K^T,   O^T [R x heads] += K[:, :R]^T [R x keys] . P^T [keys x heads]
+// CTA = (one chunk of one sequence's keys, up to NH heads), 64 keys per tile, two tiles in shared memory:
+//   warp 1           TMA: boxes of 16 keys x 64 values located through the block table, 128-byte swizzle
+//   warp 2           one thread issues tcgen05.mma: S of the next tile into one of two TMEM buffers, then O^T of this one.  The
+//                    tile is the K-major B operand of the first product and, transposed, the MN-major A operand of the second;
+//                    Q has fewer than the 128 rows the first product computes: the rows past NH are whatever follows in shared
+//                    memory and end in TMEM lanes nobody reads
+//   warps 0 4 8 12   softmax (these warps reach TMEM lanes 0-31): thread = (head, 16 keys); P goes to shared memory, K-major,
+//                    as bf16 head and bf16 remainder (2 NH columns of the second product: an MMA costs the same at 32 and at 64)
+//   warps 16-19      follow the row maxima and rescale O^T in TMEM when one rises by more than 2^8 (lazily: the division by
+//                    the row sum makes the result independent of the reference point); epilogue, thread = latent value
+// Scores and weights are f32.  Keys past the chunk are other tokens' rows (finite) and get weight zero.  Every wait is
+// bounded.  With more than one chunk a sequence's partial results (f32) are added in chunk order by a second kernel: one block
+// per (sequence, head), so that long contexts spread over the machine.
+constexpr int DK_KEYS = 64, DK_BLOCK = DK_KEYS * 128;  // keys per tile; 64 keys x 64 values
+constexpr int kDecodeMaxRank = 512, kDecodeThreads = 640;
+constexpr float kDecodeRescale = 8.0f;                 // log2 units
 
-template <int MT>
+template <int NH>
 struct DecodeSmem {
-    static constexpr int H = MT * 16, kQBlock = H * 128;
+    static constexpr int kQBlock = NH * 128, kP = NH * 128;  // one 64-value block of Q; one operand of P
     static __host__ __device__ int blocks(int W) { return (W + 63) / 64; }
     static __host__ __device__ int q_off(int W) { return 2 * blocks(W) * DK_BLOCK; }
     static __host__ __device__ int p_off(int W) { return q_off(W) + blocks(W) * kQBlock; }
-    static __host__ __device__ int bytes(int W) { return p_off(W) + 2 * H * PS * 2 + DK_WARPS * 32 * 4 * 4 + (2 * 8 * H + 3 * H) * 4 + 32; }
+    // behind P (two tiles x head, remainder): barriers, maxima and sums, then room for the rows past NH of the last Q block
+    static __host__ __device__ int x_off(int W) { return p_off(W) + 4 * kP; }
+    static __host__ __device__ int bytes(int W) {
+        const int used = x_off(W) + 256 + 3 * 4 * 32 * 4, reach = p_off(W) - kQBlock + 128 * 128;
+        return used > reach ? used : reach;
+    }
 };
 
-// barrier of the sixteen computing warps
-__device__ __forceinline__ void dk_sync() { asm volatile("bar.sync 1, %0;\n" ::"n"(DK_WARPS * 32) : "memory"); }
-
-template <int MT>
-__global__ void __launch_bounds__(DK_WARPS * 32 + 32, 1)
+template <int NH>
+__global__ void __launch_bounds__(kDecodeThreads, 1)
     latent_decode_kernel(const LatentAttnSpec a, const LatentDecodeParams p, int* err, const __grid_constant__ CUtensorMap map) {
+    using namespace tc5;
+    using L = DecodeSmem<NH>;
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     pdl_wait();
-    using L = DecodeSmem<MT>;
-    constexpr int H = L::H;
     extern __shared__ __align__(1024) uint8_t smem[];
-    const int W = a.row_pad(), R = a.kv_rank, NB = L::blocks(W);
+    const int W = a.row_pad(), R = a.kv_rank, NB = L::blocks(W), MB = (R + 127) / 128;
     const uint32_t base = smem_u32(smem);
-    if (base & 1023u) {  // the swizzled layout needs this alignment; every thread sees the same value
+    if (base & 1023u) {  // the swizzled layouts need this alignment; every thread sees the same value
         if (threadIdx.x == 0) atomicExch(err, 7);
         return;
     }
-    const uint32_t sQ = base + L::q_off(W);
-    uint16_t *ph = reinterpret_cast<uint16_t*>(smem + L::p_off(W)), *pl = ph + H * PS;
-    float *xch = reinterpret_cast<float*>(pl + H * PS), *wmax = xch + DK_WARPS * 32 * 4, *wsum = wmax + 8 * H, *rowm = wsum + 8 * H, *rowl = rowm + 2 * H;
-    const uint32_t full0 = smem_u32(rowl + H);
-    const uint32_t sPh = smem_u32(ph), sPl = smem_u32(pl);
+    const uint32_t sQ = base + L::q_off(W), sP = base + L::p_off(W), bar = base + L::x_off(W);
+    auto full = [&](int s) { return bar + 8u * s; };
+    auto empty = [&](int s) { return bar + 8u * (2 + s); };
+    auto s_ready = [&](int s) { return bar + 8u * (4 + s); };
+    auto p_ready = [&](int s) { return bar + 8u * (6 + s); };
+    auto pv_done = [&](int s) { return bar + 8u * (8 + s); };
+    auto o_ready = [&](int s) { return bar + 8u * (10 + s); };
+    const uint32_t slot_addr = bar + 8u * 12;
+    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(smem + L::x_off(W) + 8 * 12);
+    float* xm = reinterpret_cast<float*>(smem + L::x_off(W) + 256);  // [2 tiles][4 warps][32 heads] maxima
+    float* xl = xm + 2 * 4 * 32;                                     // [4 warps][32 heads] row sums
 
-    const int item = blockIdx.x, h0 = blockIdx.y * H;
+    const int item = blockIdx.x, h0 = blockIdx.y * NH;
     int sd, chunk, part0;  // row of the list, its chunk, first partial slot of the row
     if (p.work_seq) {
         if (item >= *p.n_work) return;
@@ -181,25 +194,44 @@ __global__ void __launch_bounds__(DK_WARPS * 32 + 32, 1)
     if (chunk >= n_chunks) return;
     const int k_lo = chunk * chunk_keys, k_hi = min(ctx, k_lo + chunk_keys);
     const int n_tiles = (k_hi - k_lo + DK_KEYS - 1) / DK_KEYS;
-    const int32_t* bt = p.block_tables + (size_t)slot * p.max_blocks;
-    const uint16_t* q = reinterpret_cast<const uint16_t*>(p.q_lat) + (size_t)qrow * a.heads * W;
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, mi = lane >> 3, lr = lane & 7;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
 
-    const uint32_t empty0 = full0 + 16;
     if (tid == 0) {
         for (int i = 0; i < 2; i++) {
-            tc5::mbar_init(full0 + 8 * i, 1);
-            tc5::mbar_init(empty0 + 8 * i, DK_WARPS);
+            mbar_init(full(i), 1);
+            mbar_init(empty(i), 1);
+            mbar_init(s_ready(i), 1);
+            mbar_init(p_ready(i), 4);
+            mbar_init(pv_done(i), 1);
+            mbar_init(o_ready(i), 4);
         }
         asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
     }
-    if (tid < H) {
-        rowm[tid] = -INFINITY;
-        rowl[tid] = 0.f;
+    if (warp == 2) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;\n" ::"r"(slot_addr), "r"(512) : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;\n" ::: "memory");
     }
+    {  // queries: [64-value block][head][64 values], swizzled like the keys
+        const uint16_t* q = reinterpret_cast<const uint16_t*>(p.q_lat) + (size_t)qrow * a.heads * W;
+        for (int r = warp; r < NH; r += kDecodeThreads / 32) {
+            const bool ok = h0 + r < a.heads;
+            for (int c = lane; c < NB * 8; c += 32) {
+                const bool in = ok && c * 8 < W;
+                cp_async16_zfill(sQ + (c >> 3) * L::kQBlock + r * 128 + (((c & 7) ^ (r & 7)) << 4), q + (in ? (size_t)(h0 + r) * W + c * 8 : 0), in);
+            }
+        }
+        cp_async_commit();
+        cp_async_wait<0>();
+        fence_proxy_async();
+    }
+    tc_fence_before();
     __syncthreads();
-    if (warp == DK_WARPS) {
-        // tile j: four boxes of 16 keys per 64-value block, spread over the lanes; page rows looked up a tile ahead
+    tc_fence_after();
+    const uint32_t tmem = *tmem_slot, tmem_o = tmem + 128u;
+    bool alive = true;
+
+    if (warp == 1) {
+        const int32_t* bt = p.block_tables + (size_t)slot * p.max_blocks;
         const int sub = lane & 3;
         auto row_of = [&](int j) {  // a box past the chunk repeats the chunk's first page: any finite rows will do
             const int key = k_lo + j * DK_KEYS + sub * 16, kk = key < k_hi ? key : k_lo;
@@ -209,212 +241,178 @@ __global__ void __launch_bounds__(DK_WARPS * 32 + 32, 1)
         for (int j = 0; j < n_tiles; j++) {
             const int row = next, st = j & 1;
             next = row_of(j + 1);
-            if (!__all_sync(0xffffffffu, tc5::mbar_wait(empty0 + 8 * st, ((uint32_t)(j >> 1) & 1u) ^ 1u))) {
+            if (!__all_sync(0xffffffffu, mbar_wait(empty(st), ((uint32_t)(j >> 1) & 1u) ^ 1u))) {
                 if (lane == 0) atomicExch(err, 16);
-                return;
+                break;
             }
-            if (lane == 0) tc5::mbar_expect_tx(full0 + 8 * st, (uint32_t)NB * DK_BLOCK);
+            if (lane == 0) mbar_expect_tx(full(st), (uint32_t)NB * DK_BLOCK);
             __syncwarp();
-            for (int i = lane >> 2; i < NB; i += 8) tc5::tma_load_2d(base + (st * NB + i) * DK_BLOCK + sub * 2048, &map, i * 64, row, full0 + 8 * st);
-        }
-        return;
-    }
-    // queries: [64-value block][head][64 values], swizzled like the keys
-    for (int r = warp; r < H; r += DK_WARPS) {
-        const bool ok = h0 + r < a.heads;
-        for (int c = lane; c < NB * 8; c += 32) {
-            const bool in = ok && c * 8 < W;
-            cp_async16_zfill(sQ + (c >> 3) * L::kQBlock + r * 128 + (((c & 7) ^ (r & 7)) << 4), q + (in ? (size_t)(h0 + r) * W + c * 8 : 0), in);
-        }
-    }
-    cp_async_commit();
-    cp_async_wait<0>();
-    dk_sync();
-
-    float acc[MT][DK_NJ * 2][4];
-#pragma unroll
-    for (int m = 0; m < MT; m++)
-#pragma unroll
-        for (int n = 0; n < DK_NJ * 2; n++) acc[m][n][0] = acc[m][n][1] = acc[m][n][2] = acc[m][n][3] = 0.f;
-    // scores: heads mw * 16.., keys kw * 8 MT.., blocks ks, ks + 2, ...
-    const int ks = warp & 1, mw = MT == 2 ? (warp >> 1) & 1 : 0, kw = MT == 2 ? warp >> 2 : warp >> 1;
-    const int own = MT == 2 ? kw * 2 + ks : kw;  // the 8 keys this warp turns into weights (MT 1: even warps only)
-    const bool owner = MT == 2 || ks == 0;
-    const int CT = (R + 15) / 16;
-    const int row_a = mw * 16 + (lane >> 2), row_b = row_a + 8;
-    const uint32_t qa = sQ + (mw * 16 + lr + (mi & 1) * 8) * 128;
-    const uint32_t k_row = MT == 2 ? (uint32_t)(kw * 16 + lr + (mi >> 1) * 8) * 128 : (uint32_t)(kw * 8 + lr) * 128;
-    uint32_t offa[4], offb[4];
-#pragma unroll
-    for (int i = 0; i < 4; i++) {
-        offa[i] = (uint32_t)(((2 * i + (mi >> 1)) ^ lr) << 4);
-        offb[i] = (uint32_t)(((2 * i + (mi & 1)) ^ lr) << 4);
-    }
-    bool alive = true;
-    for (int j = 0; j < n_tiles; j++) {
-        alive = alive && tc5::mbar_wait(full0 + (j & 1) * 8, (uint32_t)(j >> 1) & 1u);
-        const uint32_t kb = base + (j & 1) * NB * DK_BLOCK;
-        float s[MT][4];
-#pragma unroll
-        for (int n = 0; n < MT; n++) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
-        for (int blk = ks; blk < NB; blk += 2) {
-            const uint32_t qb = qa + blk * L::kQBlock, kk = kb + k_row + blk * DK_BLOCK;
-#pragma unroll
-            for (int i = 0; i < 4; i++) {
-                uint32_t af[4];
-                ldmatrix_x4(af[0], af[1], af[2], af[3], qb + offa[i]);
-                if (MT == 2) {
-                    uint32_t b0[2], b1[2];
-                    ldmatrix_x4(b0[0], b0[1], b1[0], b1[1], kk + offb[i]);
-                    mma_bf16_16816(s[0], af, b0);
-                    mma_bf16_16816(s[MT - 1], af, b1);
-                } else {
-                    uint32_t b0[2];
-                    ldmatrix_x2(b0[0], b0[1], kk + offb[i]);
-                    mma_bf16_16816(s[0], af, b0);
-                }
-            }
-        }
-        // hand over what the other half's warp owns, take what this one owns
-        if (MT == 2)
-            *reinterpret_cast<float4*>(xch + (warp * 32 + lane) * 4) = ks ? make_float4(s[0][0], s[0][1], s[0][2], s[0][3])
-                                                                          : make_float4(s[MT - 1][0], s[MT - 1][1], s[MT - 1][2], s[MT - 1][3]);
-        else if (ks)
-            *reinterpret_cast<float4*>(xch + (warp * 32 + lane) * 4) = make_float4(s[0][0], s[0][1], s[0][2], s[0][3]);
-        dk_sync();
-        float v[4], m0 = -INFINITY, m1 = -INFINITY;
-        if (owner) {
-            const float4 o = *reinterpret_cast<const float4*>(xch + ((warp ^ 1) * 32 + lane) * 4);
-            const float* mine = MT == 2 && ks ? s[MT - 1] : s[0];
-            v[0] = mine[0] + o.x, v[1] = mine[1] + o.y, v[2] = mine[2] + o.z, v[3] = mine[3] + o.w;
-            const int key = k_lo + j * DK_KEYS + own * 8 + 2 * (lane & 3);
-            const bool ok0 = key < k_hi, ok1 = key + 1 < k_hi;
-            v[0] = ok0 ? v[0] * p.scale_log2 : -INFINITY, v[1] = ok1 ? v[1] * p.scale_log2 : -INFINITY;
-            v[2] = ok0 ? v[2] * p.scale_log2 : -INFINITY, v[3] = ok1 ? v[3] * p.scale_log2 : -INFINITY;
-            m0 = fmaxf(v[0], v[1]);
-            m1 = fmaxf(v[2], v[3]);
-#pragma unroll
-            for (int o2 = 1; o2 < 4; o2 <<= 1) {
-                m0 = fmaxf(m0, __shfl_xor_sync(0xffffffffu, m0, o2));
-                m1 = fmaxf(m1, __shfl_xor_sync(0xffffffffu, m1, o2));
-            }
-            if ((lane & 3) == 0) {
-                wmax[own * H + row_a] = m0;
-                wmax[own * H + row_b] = m1;
-            }
-        }
-        dk_sync();
-        // weights: the row maximum over the tile and the tiles before, then exp2 (a chunk's first key is visible)
-        const float* old_m = rowm + (j & 1) * H;
-        float* new_m = rowm + ((j & 1) ^ 1) * H;
-        if (owner) {
-            m0 = old_m[row_a];
-            m1 = old_m[row_b];
-#pragma unroll
-            for (int w = 0; w < 8; w++) {
-                m0 = fmaxf(m0, wmax[w * H + row_a]);
-                m1 = fmaxf(m1, wmax[w * H + row_b]);
-            }
-            const float e0 = fast_exp2(v[0] - m0), e1 = fast_exp2(v[1] - m0), e2 = fast_exp2(v[2] - m1), e3 = fast_exp2(v[3] - m1);
-            float l0 = e0 + e1, l1 = e2 + e3;
-            const int col = own * 8 + 2 * (lane & 3);
-            const uint32_t ha = pack_bf2(e0, e1), hb = pack_bf2(e2, e3);
-            *reinterpret_cast<uint32_t*>(ph + row_a * PS + col) = ha;
-            *reinterpret_cast<uint32_t*>(ph + row_b * PS + col) = hb;
-            *reinterpret_cast<uint32_t*>(pl + row_a * PS + col) = pack_bf2(e0 - bflo(ha), e1 - bfhi(ha));
-            *reinterpret_cast<uint32_t*>(pl + row_b * PS + col) = pack_bf2(e2 - bflo(hb), e3 - bfhi(hb));
-#pragma unroll
-            for (int o2 = 1; o2 < 4; o2 <<= 1) {
-                l0 += __shfl_xor_sync(0xffffffffu, l0, o2);
-                l1 += __shfl_xor_sync(0xffffffffu, l1, o2);
-            }
-            if ((lane & 3) == 0) {
-                wsum[own * H + row_a] = l0;
-                wsum[own * H + row_b] = l1;
-                if (own == 0) {
-                    new_m[row_a] = m0;
-                    new_m[row_b] = m1;
-                }
-            }
-        }
-        dk_sync();
-        // O = alpha O + P K[:, :R]
-        if (tid < H) {
-            float l = rowl[tid] * fast_exp2(old_m[tid] - new_m[tid]);
-#pragma unroll
-            for (int w = 0; w < 8; w++) l += wsum[w * H + tid];
-            rowl[tid] = l;
-        }
-#pragma unroll
-        for (int m = 0; m < MT; m++) {
-            const int ra = m * 16 + (lane >> 2);
-            const float a0 = fast_exp2(old_m[ra] - new_m[ra]), a1 = fast_exp2(old_m[ra + 8] - new_m[ra + 8]);
-            if (__any_sync(0xffffffffu, a0 != 1.f || a1 != 1.f)) {
-#pragma unroll
-                for (int n = 0; n < DK_NJ * 2; n++) acc[m][n][0] *= a0, acc[m][n][1] *= a0, acc[m][n][2] *= a1, acc[m][n][3] *= a1;
-            }
-        }
-#pragma unroll
-        for (int k = 0; k < DK_KEYS / 16; k++) {
-            uint32_t fh[MT][4], fl[MT][4];
-#pragma unroll
-            for (int m = 0; m < MT; m++) {
-                const uint32_t off = ((m * 16 + lr + (mi & 1) * 8) * PS + k * 16 + (mi >> 1) * 8) * 2;
-                ldmatrix_x4(fh[m][0], fh[m][1], fh[m][2], fh[m][3], sPh + off);
-                ldmatrix_x4(fl[m][0], fl[m][1], fl[m][2], fl[m][3], sPl + off);
-            }
-#pragma unroll
-            for (int c = 0; c < DK_NJ; c++) {
-                const int ct = warp + c * DK_WARPS;  // values ct * 16 ..: block ct / 4, 16-byte chunks (ct % 4) * 2, + 1
-                if (ct < CT) {
-                    uint32_t v0[2], v1[2];
-                    ldmatrix_x4_trans(v0[0], v0[1], v1[0], v1[1],
-                                      kb + (ct >> 2) * DK_BLOCK + (k * 16 + lr + (mi & 1) * 8) * 128 + ((((ct & 3) * 2 + (mi >> 1)) ^ lr) << 4));
-#pragma unroll
-                    for (int m = 0; m < MT; m++) mma_bf16_16816(acc[m][2 * c], fh[m], v0), mma_bf16_16816(acc[m][2 * c + 1], fh[m], v1);
-#pragma unroll
-                    for (int m = 0; m < MT; m++) mma_bf16_16816(acc[m][2 * c], fl[m], v0), mma_bf16_16816(acc[m][2 * c + 1], fl[m], v1);
-                }
-            }
+            for (int i = lane >> 2; i < NB; i += 8) tma_load_2d(base + (st * NB + i) * DK_BLOCK + sub * 2048, &map, i * 64, row, full(st));
         }
         __syncwarp();
-        if (lane == 0) tc5::mbar_arrive(empty0 + 8 * (j & 1));  // (behind the warp's last read of the tile)
-        dk_sync();  // the weights and the row statistics may be overwritten
-    }
-    if (!alive && lane == 0) atomicExch(err, 15);
-    const float* fin_m = rowm + (n_tiles & 1) * H;
-    uint16_t* out = reinterpret_cast<uint16_t*>(p.o_lat) + (size_t)qrow * a.heads * p.o_pad;
+    } else if (warp == 2) {
+        if (lane == 0) {
+            constexpr uint32_t kQK = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(DK_KEYS >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
+            constexpr uint32_t kPV = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 15) | ((uint32_t)(2 * NH >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
+            auto issue_s = [&](int j) {
+                const uint32_t ts = tmem + (uint32_t)(j & 1) * 64u;
+                for (int b = 0; b < NB; b++) {
+                    const uint64_t dq = desc_kmajor(sQ + b * L::kQBlock), dk = desc_kmajor(base + ((j & 1) * NB + b) * DK_BLOCK);
 #pragma unroll
-    for (int m = 0; m < MT; m++)
-#pragma unroll
-        for (int half = 0; half < 2; half++) {
-            const int r = m * 16 + (lane >> 2) + half * 8, h = h0 + r;
-            if (h >= a.heads) continue;
-            const float inv = 1.0f / rowl[r];
-            uint16_t* orow = out + (size_t)h * p.o_pad;
-            float* prow = p.part_o + ((size_t)(part0 + chunk) * a.heads + h) * R;
-#pragma unroll
-            for (int c = 0; c < DK_NJ * 2; c++) {
-                const int ct = warp + (c >> 1) * DK_WARPS, col = ct * 16 + (c & 1) * 8 + 2 * (lane & 3);
-                if (ct >= CT || col >= R) continue;
-                const float v0 = acc[m][c][half * 2], v1 = acc[m][c][half * 2 + 1];
-                if (n_chunks == 1) {  // columns up to o_pad may be written: those past R are zero weights' inputs, cleared below
-                    *reinterpret_cast<uint32_t*>(orow + col) = pack_bf2(v0 * inv, col + 1 < R ? v1 * inv : 0.f);
-                } else if (R % 2 == 0) {
-                    *reinterpret_cast<float2*>(prow + col) = make_float2(v0, v1);
-                } else {
-                    prow[col] = v0;
-                    if (col + 1 < R) prow[col + 1] = v1;
+                    for (int i = 0; i < 4; i++) tc_mma(ts, dq + 2 * i, dk + 2 * i, kQK, (b > 0 || i > 0) ? 1u : 0u);
                 }
+                tc_commit(s_ready(j & 1));
+            };
+            alive = mbar_wait(full(0), 0);
+            if (alive) {
+                tc_fence_after();
+                issue_s(0);
             }
-            if (n_chunks > 1 && warp == 0 && (lane & 3) == 0) {
-                p.part_ml[((size_t)(part0 + chunk) * a.heads + h) * 2] = fin_m[r];
-                p.part_ml[((size_t)(part0 + chunk) * a.heads + h) * 2 + 1] = rowl[r];
+            for (int j = 0; j < n_tiles && alive; j++) {
+                const int st = j & 1;
+                const uint32_t ph = (uint32_t)(j >> 1) & 1u;
+                if (j + 1 < n_tiles) {
+                    alive = mbar_wait(full(st ^ 1), (uint32_t)((j + 1) >> 1) & 1u);
+                    if (!alive) break;
+                    tc_fence_after();
+                    issue_s(j + 1);
+                }
+                alive = mbar_wait(p_ready(st), ph) && mbar_wait(o_ready(st), ph);
+                if (!alive) break;
+                tc_fence_after();
+                const uint64_t dp = desc_kmajor(sP + st * 2 * L::kP);
+                for (int m = 0; m < MB; m++) {
+                    // 128 latent values = two 64-wide blocks DK_BLOCK apart (LBO); 16 keys per step, 2 KB further each
+                    const uint64_t dv = desc_mnmajor(base + (st * NB + 2 * m) * DK_BLOCK, DK_BLOCK);
+#pragma unroll
+                    for (int k = 0; k < DK_KEYS / 16; k++)
+                        tc_mma(tmem_o + (uint32_t)(m * 2 * NH), dv + (uint64_t)(k * (2048 >> 4)), dp + 2 * k, kPV, (j > 0 || k > 0) ? 1u : 0u);
+                }
+                tc_commit(pv_done(st));
+                tc_commit(empty(st));
+            }
+            if (!alive) atomicExch(err, 17);
+        }
+        __syncwarp();
+    } else if (warp >= 16 || (warp & 3) == 0) {
+        // softmax warps and O^T warps walk the tiles together: one barrier per tile, behind the tile's row maxima
+        const bool soft = warp < 16;
+        const int q = warp >> 2;  // softmax: keys q * 16 .. of the tile
+        const uint32_t lane_addr = (uint32_t)((warp & 3) * 32) << 16;
+        const bool real = lane < NH && h0 + lane < a.heads;
+        float m_run = -INFINITY, l = 0.f;
+        for (int j = 0; j < n_tiles; j++) {
+            const int st = j & 1;
+            float* mx = xm + st * 128;
+            uint32_t v[16];
+            if (soft) {
+                alive = __all_sync(0xffffffffu, alive && mbar_wait(s_ready(st), (uint32_t)(j >> 1) & 1u));
+                tc_fence_after();
+                tc_ld16(tmem + (uint32_t)st * 64u + (uint32_t)q * 16u, v);
+                const int key0 = k_lo + j * DK_KEYS + q * 16;
+                float m = -INFINITY;
+#pragma unroll
+                for (int i = 0; i < 16; i++) {
+                    const float s = !real ? 0.f : key0 + i < k_hi ? __uint_as_float(v[i]) * p.scale_log2 : -INFINITY;
+                    v[i] = __float_as_uint(s);
+                    m = fmaxf(m, s);
+                }
+                mx[q * 32 + lane] = m;
+            }
+            asm volatile("bar.sync 1, 256;\n" ::: "memory");
+            // every warp follows the reference points by itself (lane = head), from the same numbers
+            const float m = fmaxf(fmaxf(mx[lane], mx[32 + lane]), fmaxf(mx[64 + lane], mx[96 + lane]));
+            float alpha = 1.f;
+            if (j == 0) {
+                m_run = m;  // a chunk's first key is visible
+            } else if (m > m_run + kDecodeRescale) {
+                alpha = fast_exp2(m_run - m);
+                m_run = m;
+            }
+            if (soft) {
+                l *= alpha;
+                uint32_t hi[8], lo[8];
+#pragma unroll
+                for (int i = 0; i < 8; i++) {
+                    const float e0 = fast_exp2(__uint_as_float(v[2 * i]) - m_run), e1 = fast_exp2(__uint_as_float(v[2 * i + 1]) - m_run);
+                    l += e0 + e1;
+                    hi[i] = pack_bf2(e0, e1);
+                    lo[i] = pack_bf2(e0 - bflo(hi[i]), e1 - bfhi(hi[i]));
+                }
+                if (lane < NH) {
+                    uint8_t* dst = smem + L::p_off(W) + st * 2 * L::kP + lane * 128;
+#pragma unroll
+                    for (int i = 0; i < 2; i++) {
+                        const int at = ((2 * q + i) ^ (lane & 7)) << 4;
+                        *reinterpret_cast<uint4*>(dst + at) = make_uint4(hi[4 * i], hi[4 * i + 1], hi[4 * i + 2], hi[4 * i + 3]);
+                        *reinterpret_cast<uint4*>(dst + L::kP + at) = make_uint4(lo[4 * i], lo[4 * i + 1], lo[4 * i + 2], lo[4 * i + 3]);
+                    }
+                }
+                fence_proxy_async();
+                tc_fence_before();
+                __syncwarp();
+                if (lane == 0) mbar_arrive(p_ready(st));
+            } else {
+                if (__any_sync(0xffffffffu, alpha != 1.f)) {
+                    // P V of the tile before must be complete (that of the tile before it is: its stage has been loaded again)
+                    alive = __all_sync(0xffffffffu, alive && mbar_wait(pv_done(st ^ 1), (uint32_t)((j - 1) >> 1) & 1u));
+                    tc_fence_after();
+                    for (int c = 0; c < MB * 2 * NH; c += 16) {
+                        uint32_t o[16];
+                        tc_ld16(tmem_o + lane_addr + (uint32_t)c, o);
+#pragma unroll
+                        for (int i = 0; i < 16; i++) o[i] = __float_as_uint(__uint_as_float(o[i]) * __shfl_sync(0xffffffffu, alpha, (c + i) % NH));
+                        tc_st16(tmem_o + lane_addr + (uint32_t)c, o);
+                    }
+                }
+                tc_fence_before();
+                __syncwarp();
+                if (lane == 0) mbar_arrive(o_ready(st));
             }
         }
-    if (R < p.o_pad && chunk == 0)  // the padding the value projection reads
-        for (int r = warp; r < H && h0 + r < a.heads; r += DK_WARPS)
-            for (int col = R + lane; col < p.o_pad; col += 32) out[(size_t)(h0 + r) * p.o_pad + col] = 0;
+        if (soft) xl[q * 32 + lane] = l;
+        asm volatile("bar.sync 1, 256;\n" ::: "memory");
+        if (!soft) {
+            alive = __all_sync(0xffffffffu, alive && mbar_wait(pv_done((n_tiles - 1) & 1), (uint32_t)((n_tiles - 1) >> 1) & 1u));
+            tc_fence_after();
+            l = xl[lane] + xl[32 + lane] + xl[64 + lane] + xl[96 + lane];
+            const float inv = 1.0f / l;
+            uint16_t* out = reinterpret_cast<uint16_t*>(p.o_lat) + ((size_t)qrow * a.heads + h0) * p.o_pad;
+            const size_t slot0 = (size_t)(part0 + chunk) * a.heads + h0;
+            const int heads = min(NH, a.heads - h0);
+            for (int m = 0; m < MB; m++) {
+                const int d = m * 128 + (warp & 3) * 32 + lane;  // this thread's latent value
+#pragma unroll
+                for (int c = 0; c < NH; c += 16) {
+                    uint32_t o[16], o_lo[16];
+                    tc_ld16(tmem_o + lane_addr + (uint32_t)(m * 2 * NH + c), o);
+                    tc_ld16(tmem_o + lane_addr + (uint32_t)(m * 2 * NH + NH + c), o_lo);
+#pragma unroll
+                    for (int i = 0; i < 16; i++) {
+                        const float w = __shfl_sync(0xffffffffu, inv, c + i);
+                        o[i] = __float_as_uint(__uint_as_float(o[i]) + __uint_as_float(o_lo[i]));
+                        if (c + i < heads && d < R) {
+                            if (n_chunks == 1)
+                                out[(size_t)(c + i) * p.o_pad + d] = f2bf(__uint_as_float(o[i]) * w);
+                            else
+                                p.part_o[(slot0 + c + i) * R + d] = __uint_as_float(o[i]);
+                        }
+                    }
+                }
+            }
+            if (n_chunks > 1 && warp == 16 && lane < heads) {
+                p.part_ml[(slot0 + lane) * 2] = m_run;
+                p.part_ml[(slot0 + lane) * 2 + 1] = l;
+            }
+            if (R < p.o_pad && chunk == 0)  // the padding the value projection reads
+                for (int r = warp & 3; r < heads; r += 4)
+                    for (int col = R + lane; col < p.o_pad; col += 32) out[(size_t)r * p.o_pad + col] = 0;
+        }
+        if (!alive && lane == 0) atomicExch(err, 15);
+    }
+    tc_fence_before();
+    __syncthreads();
+    if (warp == 2) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;\n" ::"r"(tmem), "r"(512) : "memory");
 }
 
 constexpr int kMergeTile = 128;
@@ -467,17 +465,17 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const LatentAttnSpec 
 }  // namespace
 
 bool b2_latent_decode_eligible(const LatentAttnSpec& a) {
-    return a.kv_rank <= kDecodeMaxRank && (a.heads > 16 ? DecodeSmem<2>::bytes(a.row_pad()) : DecodeSmem<1>::bytes(a.row_pad())) <= 226 * 1024;
+    return a.kv_rank <= kDecodeMaxRank && (a.heads > 16 ? DecodeSmem<32>::bytes(a.row_pad()) : DecodeSmem<16>::bytes(a.row_pad())) <= 226 * 1024;
 }
 int32_t b2_latent_decode_launch(b2_ctx* ctx, const LatentAttnSpec& a, const LatentDecodeParams& p, int items, int rows) {
     if (items <= 0) return B2_OK;
     const dim3 grid(items, a.heads > 16 ? (a.heads + 31) / 32 : 1);
     CUtensorMap map;
     B2_CHECK(tc5::get_map(ctx, p.cache, (uint64_t)p.cache_rows, (uint64_t)a.row_pad(), (uint64_t)a.row_pad(), 16, &map));
-    B2_SMEM_ONCE(ctx, latent_decode_kernel<1>, 226 * 1024);
-    B2_SMEM_ONCE(ctx, latent_decode_kernel<2>, 226 * 1024);
-    const int smem = a.heads > 16 ? DecodeSmem<2>::bytes(a.row_pad()) : DecodeSmem<1>::bytes(a.row_pad());
-    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, a.heads > 16 ? latent_decode_kernel<2> : latent_decode_kernel<1>, grid, dim3(DK_WARPS * 32 + 32), (size_t)smem, ctx->stream, a,
+    B2_SMEM_ONCE(ctx, latent_decode_kernel<16>, 226 * 1024);
+    B2_SMEM_ONCE(ctx, latent_decode_kernel<32>, 226 * 1024);
+    const int smem = a.heads > 16 ? DecodeSmem<32>::bytes(a.row_pad()) : DecodeSmem<16>::bytes(a.row_pad());
+    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, a.heads > 16 ? latent_decode_kernel<32> : latent_decode_kernel<16>, grid, dim3(kDecodeThreads), (size_t)smem, ctx->stream, a,
                           p, ctx->dev_err, map));
     B2_LAUNCHED(ctx);
     if (items > rows) {  // some row has more than one chunk

@@ -28,11 +28,6 @@ constexpr int kSoftmaxWarps = 8, kKWarp = 8, kVWarp = 9, kMmaWarp = 10, kThreads
 constexpr int BLOCK_BYTES = 128 * 128;  // 128 rows x 64 bf16, 128-byte swizzle
 constexpr float kRescaleThreshold = 8.0f;  // log2 units
 
-// MN-major operand, 128-byte swizzle: a V block holds 128 keys x 64 values; the next 64 values are one block further (LBO),
-// 8-key groups 1024 B apart (SBO), and a 16-key MMA step starts 2 KB after the one before.
-__device__ __forceinline__ uint64_t desc_mnmajor(uint32_t smem_addr) {
-    return (uint64_t)((smem_addr >> 4) & 0x3fff) | ((uint64_t)(BLOCK_BYTES >> 4) << 16) | (64ull << 32) | (1ull << 46) | (2ull << 61);
-}
 // f32 accumulate, bf16 x bf16, M = 128; bit 16 set = B is MN-major
 constexpr uint32_t idesc(int n, bool b_mn) {
     return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(n >> 3) << 17) | ((uint32_t)(128 >> 4) << 24) | (b_mn ? (1u << 16) : 0u);
@@ -151,7 +146,7 @@ __global__ void __launch_bounds__(kThreads, 1)
     } else if (warp == kMmaWarp) {
         if (lane == 0) {
             constexpr uint32_t kQK = idesc(128, false), kPV = idesc(VDB * 64, true);
-            const uint64_t dq0 = desc_kmajor(base + L::Q), dk0 = desc_kmajor(base + L::K), dv0 = desc_mnmajor(base + L::V);
+            const uint64_t dq0 = desc_kmajor(base + L::Q), dk0 = desc_kmajor(base + L::K), dv0 = desc_mnmajor(base + L::V, BLOCK_BYTES);
             auto issue_qk = [&](int j, int kst) {  // S[j & 1] = Q K_j^T
                 const uint64_t dk = dk0 + (uint64_t)((uint32_t)kst * DKB * (BLOCK_BYTES >> 4));
                 const uint32_t ts = tmem_base + (uint32_t)(j & 1) * 128u;
@@ -183,6 +178,7 @@ __global__ void __launch_bounds__(kThreads, 1)
                 for (int k = 0; k < KT / 16; k++) {
                     // keys 0-63 of the tile: head in columns 0-31 of the buffer, remainder in 32-63; keys 64-127: 64-95, 96-127
                     const uint32_t ta = tP + (uint32_t)(k >> 2) * 64u + (uint32_t)(k & 3) * 8u;
+                    // 16 keys of a V block (128 keys x 64 values; the next 64 values are a block further)
                     const uint64_t dv = dvs + (uint64_t)((uint32_t)k * (2048u >> 4));
                     tc_mma_ts(tmem_o, ta, dv, kPV, (j > 0 || k > 0) ? 1u : 0u);
                     tc_mma_ts(tmem_o, ta + 32u, dv, kPV, 1u);
