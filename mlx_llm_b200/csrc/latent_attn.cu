@@ -120,8 +120,8 @@ __global__ void __launch_bounds__(128) latent_attn_simple_kernel(const LatentAtt
 //   S [heads x keys] = Q [heads x W] . K^T,   O^T [R x heads] += K[:, :R]^T [R x keys] . P^T [keys x heads]
 // CTA = (one chunk of one sequence's keys, up to NH heads), 64 keys per tile, two tiles in shared memory:
 //   warp 1           TMA: boxes of 16 keys x 64 values located through the block table, 128-byte swizzle
-//   warp 2           one thread issues tcgen05.mma: S of the next tile into one of two TMEM buffers, then O^T of this one.  The
-//                    tile is the K-major B operand of the first product and, transposed, the MN-major A operand of the second;
+//   warp 2           one thread issues tcgen05.mma, whichever is ready first: the next part of S (a few 64-value blocks of a tile,
+//                    as they arrive; one of two TMEM buffers) or O^T of a tile whose P is complete, which frees its place.  The tile is the K-major B operand of the first product and, transposed, the MN-major A operand of the second;
 //                    Q has fewer than the 128 rows the first product computes: the rows past NH are whatever follows in shared
 //                    memory and end in TMEM lanes nobody reads
 //   warps 0 4 8 12   softmax (these warps reach TMEM lanes 0-31): thread = (head, 16 keys); P goes to shared memory, K-major,
@@ -133,6 +133,7 @@ __global__ void __launch_bounds__(128) latent_attn_simple_kernel(const LatentAtt
 // per (sequence, head), so that long contexts spread over the machine.
 constexpr int DK_KEYS = 64, DK_BLOCK = DK_KEYS * 128;  // keys per tile; 64 keys x 64 values
 constexpr int kDecodeMaxRank = 512, kDecodeThreads = 640;
+constexpr int DK_GB = 3, DK_NG = 4;                    // 64-value blocks per arrival barrier; barriers per tile (W up to 768)
 constexpr float kDecodeRescale = 8.0f;                 // log2 units
 
 template <int NH>
@@ -157,21 +158,21 @@ __global__ void __launch_bounds__(kDecodeThreads, 1)
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     pdl_wait();
     extern __shared__ __align__(1024) uint8_t smem[];
-    const int W = a.row_pad(), R = a.kv_rank, NB = L::blocks(W), MB = (R + 127) / 128;
+    const int W = a.row_pad(), R = a.kv_rank, NB = L::blocks(W), NG = (NB + DK_GB - 1) / DK_GB, MB = (R + 127) / 128;
     const uint32_t base = smem_u32(smem);
     if (base & 1023u) {  // the swizzled layouts need this alignment; every thread sees the same value
         if (threadIdx.x == 0) atomicExch(err, 7);
         return;
     }
     const uint32_t sQ = base + L::q_off(W), sP = base + L::p_off(W), bar = base + L::x_off(W);
-    auto full = [&](int s) { return bar + 8u * s; };
-    auto empty = [&](int s) { return bar + 8u * (2 + s); };
-    auto s_ready = [&](int s) { return bar + 8u * (4 + s); };
-    auto p_ready = [&](int s) { return bar + 8u * (6 + s); };
-    auto pv_done = [&](int s) { return bar + 8u * (8 + s); };
-    auto o_ready = [&](int s) { return bar + 8u * (10 + s); };
-    const uint32_t slot_addr = bar + 8u * 12;
-    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(smem + L::x_off(W) + 8 * 12);
+    auto empty = [&](int s) { return bar + 8u * s; };
+    auto s_ready = [&](int s) { return bar + 8u * (2 + s); };
+    auto p_ready = [&](int s) { return bar + 8u * (4 + s); };
+    auto pv_done = [&](int s) { return bar + 8u * (6 + s); };
+    auto o_ready = [&](int s) { return bar + 8u * (8 + s); };
+    const uint32_t slot_addr = bar + 8u * 10;
+    auto full = [&](int s, int g) { return bar + 8u * (12 + s * DK_NG + g); };
+    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(smem + L::x_off(W) + 8 * 10);
     float* xm = reinterpret_cast<float*>(smem + L::x_off(W) + 256);  // [2 tiles][4 warps][32 heads] maxima
     float* xl = xm + 2 * 4 * 32;                                     // [4 warps][32 heads] row sums
 
@@ -198,7 +199,7 @@ __global__ void __launch_bounds__(kDecodeThreads, 1)
 
     if (tid == 0) {
         for (int i = 0; i < 2; i++) {
-            mbar_init(full(i), 1);
+            for (int g = 0; g < DK_NG; g++) mbar_init(full(i, g), 1);
             mbar_init(empty(i), 1);
             mbar_init(s_ready(i), 1);
             mbar_init(p_ready(i), 4);
@@ -245,51 +246,55 @@ __global__ void __launch_bounds__(kDecodeThreads, 1)
                 if (lane == 0) atomicExch(err, 16);
                 break;
             }
-            if (lane == 0) mbar_expect_tx(full(st), (uint32_t)NB * DK_BLOCK);
+            if (lane < NG) mbar_expect_tx(full(st, lane), (uint32_t)min(DK_GB, NB - lane * DK_GB) * DK_BLOCK);
             __syncwarp();
-            for (int i = lane >> 2; i < NB; i += 8) tma_load_2d(base + (st * NB + i) * DK_BLOCK + sub * 2048, &map, i * 64, row, full(st));
+            for (int i = lane >> 2; i < NB; i += 8) tma_load_2d(base + (st * NB + i) * DK_BLOCK + sub * 2048, &map, i * 64, row, full(st, i / DK_GB));
         }
         __syncwarp();
     } else if (warp == 2) {
         if (lane == 0) {
             constexpr uint32_t kQK = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(DK_KEYS >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
             constexpr uint32_t kPV = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 15) | ((uint32_t)(2 * NH >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
-            auto issue_s = [&](int j) {
-                const uint32_t ts = tmem + (uint32_t)(j & 1) * 64u;
-                for (int b = 0; b < NB; b++) {
-                    const uint64_t dq = desc_kmajor(sQ + b * L::kQBlock), dk = desc_kmajor(base + ((j & 1) * NB + b) * DK_BLOCK);
-#pragma unroll
-                    for (int i = 0; i < 4; i++) tc_mma(ts, dq + 2 * i, dk + 2 * i, kQK, (b > 0 || i > 0) ? 1u : 0u);
-                }
-                tc_commit(s_ready(j & 1));
-            };
-            alive = mbar_wait(full(0), 0);
-            if (alive) {
-                tc_fence_after();
-                issue_s(0);
-            }
-            for (int j = 0; j < n_tiles && alive; j++) {
-                const int st = j & 1;
-                const uint32_t ph = (uint32_t)(j >> 1) & 1u;
-                if (j + 1 < n_tiles) {
-                    alive = mbar_wait(full(st ^ 1), (uint32_t)((j + 1) >> 1) & 1u);
-                    if (!alive) break;
+            int ns = 0, ng = 0, np = 0;  // next part of S: tile and group of blocks; next tile of O^T
+            long long since = 0;         // of the last progress
+            while (np < n_tiles) {
+                if (np < ns && mbar_test(p_ready(np & 1), (uint32_t)(np >> 1) & 1u) && mbar_test(o_ready(np & 1), (uint32_t)(np >> 1) & 1u)) {
+                    const int st = np & 1;
                     tc_fence_after();
-                    issue_s(j + 1);
-                }
-                alive = mbar_wait(p_ready(st), ph) && mbar_wait(o_ready(st), ph);
-                if (!alive) break;
-                tc_fence_after();
-                const uint64_t dp = desc_kmajor(sP + st * 2 * L::kP);
-                for (int m = 0; m < MB; m++) {
-                    // 128 latent values = two 64-wide blocks DK_BLOCK apart (LBO); 16 keys per step, 2 KB further each
-                    const uint64_t dv = desc_mnmajor(base + (st * NB + 2 * m) * DK_BLOCK, DK_BLOCK);
+                    const uint64_t dp = desc_kmajor(sP + st * 2 * L::kP);
+                    for (int m = 0; m < MB; m++) {
+                        // 128 latent values = two 64-wide blocks DK_BLOCK apart (LBO); 16 keys per step, 2 KB further each
+                        const uint64_t dv = desc_mnmajor(base + (st * NB + 2 * m) * DK_BLOCK, DK_BLOCK);
 #pragma unroll
-                    for (int k = 0; k < DK_KEYS / 16; k++)
-                        tc_mma(tmem_o + (uint32_t)(m * 2 * NH), dv + (uint64_t)(k * (2048 >> 4)), dp + 2 * k, kPV, (j > 0 || k > 0) ? 1u : 0u);
+                        for (int k = 0; k < DK_KEYS / 16; k++)
+                            tc_mma(tmem_o + (uint32_t)(m * 2 * NH), dv + (uint64_t)(k * (2048 >> 4)), dp + 2 * k, kPV, (np > 0 || k > 0) ? 1u : 0u);
+                    }
+                    tc_commit(pv_done(st));
+                    tc_commit(empty(st));
+                    np++;
+                    since = 0;
+                } else if (ns < n_tiles && mbar_test(full(ns & 1, ng), (uint32_t)(ns >> 1) & 1u)) {
+                    const uint32_t ts = tmem + (uint32_t)(ns & 1) * 64u;
+                    tc_fence_after();
+                    for (int b = ng * DK_GB; b < min(NB, (ng + 1) * DK_GB); b++) {
+                        const uint64_t dq = desc_kmajor(sQ + b * L::kQBlock), dk = desc_kmajor(base + ((ns & 1) * NB + b) * DK_BLOCK);
+#pragma unroll
+                        for (int i = 0; i < 4; i++) tc_mma(ts, dq + 2 * i, dk + 2 * i, kQK, (b > 0 || i > 0) ? 1u : 0u);
+                    }
+                    if (++ng == NG) {
+                        tc_commit(s_ready(ns & 1));
+                        ng = 0;
+                        ns++;
+                    }
+                    since = 0;
+                } else {
+                    const long long now = clock64();
+                    if (since == 0) since = now;
+                    if (now - since > 4000000000ll) {  // about 2 s without progress
+                        alive = false;
+                        break;
+                    }
                 }
-                tc_commit(pv_done(st));
-                tc_commit(empty(st));
             }
             if (!alive) atomicExch(err, 17);
         }
@@ -465,7 +470,7 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const LatentAttnSpec 
 }  // namespace
 
 bool b2_latent_decode_eligible(const LatentAttnSpec& a) {
-    return a.kv_rank <= kDecodeMaxRank && (a.heads > 16 ? DecodeSmem<32>::bytes(a.row_pad()) : DecodeSmem<16>::bytes(a.row_pad())) <= 226 * 1024;
+    return a.kv_rank <= kDecodeMaxRank && a.row_pad() <= DK_NG * DK_GB * 64 && (a.heads > 16 ? DecodeSmem<32>::bytes(a.row_pad()) : DecodeSmem<16>::bytes(a.row_pad())) <= 226 * 1024;
 }
 int32_t b2_latent_decode_launch(b2_ctx* ctx, const LatentAttnSpec& a, const LatentDecodeParams& p, int items, int rows) {
     if (items <= 0) return B2_OK;
