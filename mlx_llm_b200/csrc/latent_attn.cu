@@ -120,8 +120,9 @@ __global__ void __launch_bounds__(128) latent_attn_simple_kernel(const LatentAtt
 //   S [heads x keys] = Q [heads x W] . K^T,   O^T [R x heads] += K[:, :R]^T [R x keys] . P^T [keys x heads]
 // CTA = (one chunk of one sequence's keys, up to NH heads), 64 keys per tile, two tiles in shared memory:
 //   warp 1           TMA: boxes of 16 keys x 64 values located through the block table, 128-byte swizzle
-//   warp 2           one thread issues tcgen05.mma, whichever is ready first: the next part of S (a few 64-value blocks of a tile,
-//                    as they arrive; one of two TMEM buffers) or O^T of a tile whose P is complete, which frees its place.  The tile is the K-major B operand of the first product and, transposed, the MN-major A operand of the second;
+//   warps 2, 3       one thread each issues tcgen05.mma: S, a few 64-value blocks of a tile at a time as they arrive, into one
+//                    of two TMEM buffers; O^T of a tile when its P is complete, which frees its place.  The tile is the
+//                    K-major B operand of the first product and, transposed, the MN-major A operand of the second;
 //                    Q has fewer than the 128 rows the first product computes: the rows past NH are whatever follows in shared
 //                    memory and end in TMEM lanes nobody reads
 //   warps 0 4 8 12   softmax (these warps reach TMEM lanes 0-31): thread = (head, 16 keys); P goes to shared memory, K-major,
@@ -156,7 +157,6 @@ __global__ void __launch_bounds__(kDecodeThreads, 1)
     using namespace tc5;
     using L = DecodeSmem<NH>;
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
-    pdl_wait();
     extern __shared__ __align__(1024) uint8_t smem[];
     const int W = a.row_pad(), R = a.kv_rank, NB = L::blocks(W), NG = (NB + DK_GB - 1) / DK_GB, MB = (R + 127) / 128;
     const uint32_t base = smem_u32(smem);
@@ -176,6 +176,19 @@ __global__ void __launch_bounds__(kDecodeThreads, 1)
     float* xm = reinterpret_cast<float*>(smem + L::x_off(W) + 256);  // [2 tiles][4 warps][32 heads] maxima
     float* xl = xm + 2 * 4 * 32;                                     // [4 warps][32 heads] row sums
 
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    if (tid == 0) {
+        for (int i = 0; i < 2; i++) {
+            for (int g = 0; g < DK_NG; g++) mbar_init(full(i, g), 1);
+            mbar_init(empty(i), 1);
+            mbar_init(s_ready(i), 1);
+            mbar_init(p_ready(i), 4);
+            mbar_init(pv_done(i), 1);
+            mbar_init(o_ready(i), 4);
+        }
+        asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
+    }
+    pdl_wait();  // (the barriers above may be set up while earlier kernels finish)
     const int item = blockIdx.x, h0 = blockIdx.y * NH;
     int sd, chunk, part0;  // row of the list, its chunk, first partial slot of the row
     if (p.work_seq) {
@@ -195,19 +208,7 @@ __global__ void __launch_bounds__(kDecodeThreads, 1)
     if (chunk >= n_chunks) return;
     const int k_lo = chunk * chunk_keys, k_hi = min(ctx, k_lo + chunk_keys);
     const int n_tiles = (k_hi - k_lo + DK_KEYS - 1) / DK_KEYS;
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
 
-    if (tid == 0) {
-        for (int i = 0; i < 2; i++) {
-            for (int g = 0; g < DK_NG; g++) mbar_init(full(i, g), 1);
-            mbar_init(empty(i), 1);
-            mbar_init(s_ready(i), 1);
-            mbar_init(p_ready(i), 4);
-            mbar_init(pv_done(i), 1);
-            mbar_init(o_ready(i), 4);
-        }
-        asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
-    }
     if (warp == 2) {
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;\n" ::"r"(slot_addr), "r"(512) : "memory");
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;\n" ::: "memory");
@@ -254,49 +255,45 @@ __global__ void __launch_bounds__(kDecodeThreads, 1)
     } else if (warp == 2) {
         if (lane == 0) {
             constexpr uint32_t kQK = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(DK_KEYS >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
-            constexpr uint32_t kPV = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 15) | ((uint32_t)(2 * NH >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
-            int ns = 0, ng = 0, np = 0;  // next part of S: tile and group of blocks; next tile of O^T
-            long long since = 0;         // of the last progress
-            while (np < n_tiles) {
-                if (np < ns && mbar_test(p_ready(np & 1), (uint32_t)(np >> 1) & 1u) && mbar_test(o_ready(np & 1), (uint32_t)(np >> 1) & 1u)) {
-                    const int st = np & 1;
+            for (int j = 0; j < n_tiles && alive; j++) {
+                const int st = j & 1;
+                for (int g = 0; g < NG; g++) {
+                    alive = mbar_wait(full(st, g), (uint32_t)(j >> 1) & 1u);
+                    if (!alive) break;
                     tc_fence_after();
-                    const uint64_t dp = desc_kmajor(sP + st * 2 * L::kP);
-                    for (int m = 0; m < MB; m++) {
-                        // 128 latent values = two 64-wide blocks DK_BLOCK apart (LBO); 16 keys per step, 2 KB further each
-                        const uint64_t dv = desc_mnmajor(base + (st * NB + 2 * m) * DK_BLOCK, DK_BLOCK);
+                    for (int b = g * DK_GB; b < min(NB, (g + 1) * DK_GB); b++) {
+                        const uint64_t dq = desc_kmajor(sQ + b * L::kQBlock), dk = desc_kmajor(base + (st * NB + b) * DK_BLOCK);
 #pragma unroll
-                        for (int k = 0; k < DK_KEYS / 16; k++)
-                            tc_mma(tmem_o + (uint32_t)(m * 2 * NH), dv + (uint64_t)(k * (2048 >> 4)), dp + 2 * k, kPV, (np > 0 || k > 0) ? 1u : 0u);
-                    }
-                    tc_commit(pv_done(st));
-                    tc_commit(empty(st));
-                    np++;
-                    since = 0;
-                } else if (ns < n_tiles && mbar_test(full(ns & 1, ng), (uint32_t)(ns >> 1) & 1u)) {
-                    const uint32_t ts = tmem + (uint32_t)(ns & 1) * 64u;
-                    tc_fence_after();
-                    for (int b = ng * DK_GB; b < min(NB, (ng + 1) * DK_GB); b++) {
-                        const uint64_t dq = desc_kmajor(sQ + b * L::kQBlock), dk = desc_kmajor(base + ((ns & 1) * NB + b) * DK_BLOCK);
-#pragma unroll
-                        for (int i = 0; i < 4; i++) tc_mma(ts, dq + 2 * i, dk + 2 * i, kQK, (b > 0 || i > 0) ? 1u : 0u);
-                    }
-                    if (++ng == NG) {
-                        tc_commit(s_ready(ns & 1));
-                        ng = 0;
-                        ns++;
-                    }
-                    since = 0;
-                } else {
-                    const long long now = clock64();
-                    if (since == 0) since = now;
-                    if (now - since > 4000000000ll) {  // about 2 s without progress
-                        alive = false;
-                        break;
+                        for (int i = 0; i < 4; i++) tc_mma(tmem + (uint32_t)st * 64u, dq + 2 * i, dk + 2 * i, kQK, (b > 0 || i > 0) ? 1u : 0u);
                     }
                 }
+                if (alive) tc_commit(s_ready(st));
             }
             if (!alive) atomicExch(err, 17);
+        }
+        __syncwarp();
+    } else if (warp == 3) {
+        if (lane == 0) {
+            constexpr uint32_t kPV = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 15) | ((uint32_t)(2 * NH >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
+            for (int j = 0; j < n_tiles && alive; j++) {
+                const int st = j & 1;
+                const uint32_t ph = (uint32_t)(j >> 1) & 1u;
+                // (P exists, so S of this tile has been computed: its stage may be freed when these products are done)
+                alive = mbar_wait(p_ready(st), ph) && mbar_wait(o_ready(st), ph);
+                if (!alive) break;
+                tc_fence_after();
+                const uint64_t dp = desc_kmajor(sP + st * 2 * L::kP);
+                for (int m = 0; m < MB; m++) {
+                    // 128 latent values = two 64-wide blocks DK_BLOCK apart (LBO); 16 keys per step, 2 KB further each
+                    const uint64_t dv = desc_mnmajor(base + (st * NB + 2 * m) * DK_BLOCK, DK_BLOCK);
+#pragma unroll
+                    for (int k = 0; k < DK_KEYS / 16; k++)
+                        tc_mma(tmem_o + (uint32_t)(m * 2 * NH), dv + (uint64_t)(k * (2048 >> 4)), dp + 2 * k, kPV, (j > 0 || k > 0) ? 1u : 0u);
+                }
+                tc_commit(pv_done(st));
+                tc_commit(empty(st));
+            }
+            if (!alive) atomicExch(err, 18);
         }
         __syncwarp();
     } else if (warp >= 16 || (warp & 3) == 0) {
