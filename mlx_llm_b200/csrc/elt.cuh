@@ -70,3 +70,8 @@ __device__ __forceinline__ float elt_block_sum(float v, float* red) {
 }
 __device__ __forceinline__ float sigmoid_f32(float x) { return 1.0f / (1.0f + expf(-x)); }
 __device__ __forceinline__ float silu_f32(float x) { return x * sigmoid_f32(x); }
+// ... with the fast exponential and division where the result is rounded to bf16 anyway
+template <typename T>
+__device__ __forceinline__ float silu_for(float x) {
+    return sizeof(T) == 2 ? __fdividef(x, 1.0f + __expf(-x)) : silu_f32(x);
+}

@@ -43,22 +43,19 @@ int32_t ensure_workspace(b2_model* m, int T, int B, int W, int P, size_t stage_i
     }
     if (grow_t) {
         const size_t t = (size_t)std::max(T, 64) * 5 / 4;
-        if (m->layered) {  // its activations live in an arena of its own (engine_layers.cu)
-            B2_CHECK(regrow(w.ids, t));
-            w.t_cap = (int)t;
-        } else {
-        const size_t qkv_w = (size_t)(m->hq_l + 2 * m->hkv_l) * c.head_dim;
-        if (!w.x_in_peer_region) B2_CHECK(regrow(w.x, t * c.hidden_size));
-        B2_CHECK(regrow(w.xn, t * c.hidden_size));
-        B2_CHECK(regrow(w.qkv, t * qkv_w));
-        B2_CHECK(regrow(w.q, t * m->hq_l * c.head_dim));
-        B2_CHECK(regrow(w.attn, t * m->hq_l * c.head_dim));
-        B2_CHECK(regrow(w.gu, t * 2 * m->inter_l));
-        B2_CHECK(regrow(w.act, t * m->inter_l));
-        if (m->tp && m->tp->world > 1) B2_CHECK(regrow(w.tp_part, t * c.hidden_size));
+        if (!m->layered) {  // (a layered model's activations live in an arena of its own, engine_layers.cu)
+            const size_t qkv_w = (size_t)(m->hq_l + 2 * m->hkv_l) * c.head_dim;
+            if (!w.x_in_peer_region) B2_CHECK(regrow(w.x, t * c.hidden_size));
+            B2_CHECK(regrow(w.xn, t * c.hidden_size));
+            B2_CHECK(regrow(w.qkv, t * qkv_w));
+            B2_CHECK(regrow(w.q, t * m->hq_l * c.head_dim));
+            B2_CHECK(regrow(w.attn, t * m->hq_l * c.head_dim));
+            B2_CHECK(regrow(w.gu, t * 2 * m->inter_l));
+            B2_CHECK(regrow(w.act, t * m->inter_l));
+            if (m->tp && m->tp->world > 1) B2_CHECK(regrow(w.tp_part, t * c.hidden_size));
+        }
         B2_CHECK(regrow(w.ids, t));
         w.t_cap = (int)t;
-        }
     }
     if (grow_b) {
         const size_t b = (size_t)std::max(B, 16) * 5 / 4;

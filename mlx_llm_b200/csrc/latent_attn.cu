@@ -444,7 +444,7 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const LatentAttnSpec 
             sum[c] = ml.y;
         }
         __syncthreads();
-#pragma unroll 4
+#pragma unroll 8
         for (int c = 0; c < cnt; c++) {
             const float* o = p.part_o + (at0 + (size_t)(c0 + c) * a.heads) * R;
             L = fmaf(w[c], sum[c], L);

@@ -47,7 +47,11 @@ __global__ void __launch_bounds__(128) conv_silu8_kernel(const Mamba2Spec s, con
     for (int j = 0; j < TAPS; j++) Elt<float>::ld8(p.conv_w + (size_t)j * C + ch, w[j]);
     const T* u = reinterpret_cast<const T*>(p.zx) + s.inner() + ch;
     int cur = -1;
-    for (int t = blockIdx.y * run; t < min((int)(blockIdx.y + 1) * run, p.T); t++) {
+    const int t_end = min((int)(blockIdx.y + 1) * run, p.T);
+    float next[8];  // the input of the token after this one is on its way
+    Elt<T>::ld8(u + (size_t)(blockIdx.y * run) * p.ld, next);
+#pragma unroll 4
+    for (int t = blockIdx.y * run; t < t_end; t++) {
         const int b = p.token_seq[t];
         if (b != cur) {  // the inputs before this token: of this step, or the kept ones
             cur = b;
@@ -68,14 +72,16 @@ __global__ void __launch_bounds__(128) conv_silu8_kernel(const Mamba2Spec s, con
         for (int j = 0; j + 1 < TAPS; j++)
 #pragma unroll
             for (int e = 0; e < 8; e++) win[j][e] = win[j + 1][e];
-        Elt<T>::ld8(u + (size_t)t * p.ld, win[TAPS - 1]);
+#pragma unroll
+        for (int e = 0; e < 8; e++) win[TAPS - 1][e] = next[e];
+        if (t + 1 < t_end) Elt<T>::ld8(u + (size_t)(t + 1) * p.ld, next);
         float v[8];
 #pragma unroll
         for (int e = 0; e < 8; e++) {
             v[e] = bias[e];
 #pragma unroll
             for (int j = 0; j < TAPS; j++) v[e] = fmaf(w[j][e], win[j][e], v[e]);
-            v[e] = silu_f32(v[e]);
+            v[e] = silu_for<T>(v[e]);
         }
         Elt<T>::st8(reinterpret_cast<T*>(p.xbc) + (size_t)t * p.ld_xbc + ch, v);
     }
@@ -199,17 +205,18 @@ __global__ void __launch_bounds__(128) scan_kernel(const Mamba2Spec s, const Ssm
 // nature -- the state, the decays, the step sizes and what they multiply -- enters as a bf16 head plus a bf16 remainder,
 // and all sums are f32.  The state stays in f32 registers from chunk to chunk.
 //
-// Block = (64 value rows of one head, sequence), 8 warps.  y: warp = 16 tokens x 32 value rows; state: warp = 16 state rows
-// x 64 value rows.  The next chunk's x, B and C arrive by cp.async while this one is computed.
-constexpr int CH_T = 64, CH_P = 64, CH_N = 128;  // tokens, value rows, largest state
-constexpr int CH_LN = CH_N + 8, CH_LP = CH_P + 8;            // row strides in shared memory (conflict-free ldmatrix)
+// Block = (64 value rows of one head, sequence), 16 warps.  First the weights (C_t . B_s) exp(c_t - c_s) d_s of the chunk, a
+// 16 x 16 tile per warp up to the diagonal, into shared memory; then y, a warp per 16 tokens x 16 value rows; then the
+// state, a warp per 16 state rows x 32 value rows.  The next chunk's x, B and C arrive by cp.async meanwhile.
+constexpr int CH_T = 64, CH_P = 64, CH_N = 128, CH_THREADS = 512;  // tokens, value rows, largest state
+constexpr int CH_LN = CH_N + 8, CH_LP = CH_P + 8, CH_LM = CH_T + 8;  // row strides in shared memory (conflict-free ldmatrix)
 struct ChunkSmem {
     static constexpr int kIn = (2 * CH_T * CH_LN + CH_T * CH_LP) * 2;  // C | B | x of one chunk
-    static constexpr int kXw = 2 * CH_T * CH_LP * 2, kS = 2 * CH_N * CH_LP * 2;
-    static constexpr int kBytes = 2 * kIn + kXw + kS + 2 * 4 * CH_T * 4;
+    static constexpr int kXw = 2 * CH_T * CH_LP * 2, kM = 2 * CH_T * CH_LM * 2, kS = 2 * CH_N * CH_LP * 2;
+    static constexpr int kBytes = 2 * kIn + kXw + kM + kS + 2 * 4 * CH_T * 4;
 };
 
-__global__ void __launch_bounds__(256, 1) chunk_scan_kernel(const Mamba2Spec s, const SsmParams p) {
+__global__ void __launch_bounds__(CH_THREADS, 1) chunk_scan_kernel(const Mamba2Spec s, const SsmParams p) {
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     pdl_wait();
     const int h = blockIdx.y, b = blockIdx.z, p0 = blockIdx.x * CH_P;
@@ -221,8 +228,9 @@ __global__ void __launch_bounds__(256, 1) chunk_scan_kernel(const Mamba2Spec s, 
     const int KN = (N + 15) / 16;
     uint8_t* const in0 = smem;
     uint16_t* xw = reinterpret_cast<uint16_t*>(smem + 2 * ChunkSmem::kIn);  // head, remainder [token][value row]
-    uint16_t* sh = reinterpret_cast<uint16_t*>(smem + 2 * ChunkSmem::kIn + ChunkSmem::kXw);  // head, remainder [state row][value row]
-    float* steps = reinterpret_cast<float*>(smem + 2 * ChunkSmem::kIn + ChunkSmem::kXw + ChunkSmem::kS);  // two chunks' step sizes and decays
+    uint16_t* sm = reinterpret_cast<uint16_t*>(smem + 2 * ChunkSmem::kIn + ChunkSmem::kXw);  // weights, head, remainder [token][earlier token]
+    uint16_t* sh = reinterpret_cast<uint16_t*>(smem + 2 * ChunkSmem::kIn + ChunkSmem::kXw + ChunkSmem::kM);  // head, remainder [state row][value row]
+    float* steps = reinterpret_cast<float*>(smem + 2 * ChunkSmem::kIn + ChunkSmem::kXw + ChunkSmem::kM + ChunkSmem::kS);  // two chunks' step sizes and decays
     const uint16_t* zx = reinterpret_cast<const uint16_t*>(p.zx);
     const uint16_t* xbc = reinterpret_cast<const uint16_t*>(p.xbc) + (size_t)start * p.ld_xbc;
     const float A = expf(p.A_log[h]), bias = p.dt_bias[h], D = p.D[h];
@@ -233,45 +241,47 @@ __global__ void __launch_bounds__(256, 1) chunk_scan_kernel(const Mamba2Spec s, 
         uint16_t *dB = dC + CH_T * CH_LN, *dx = dB + CH_T * CH_LN;
         const int t0 = c * CH_T, cB = inner + grp * N, cC = cB + s.groups * N, cx = h * P + p0;
         if (vec) {
-            for (int i = tid; i < CH_T * (CH_N / 8); i += 256) {
+            for (int i = tid; i < CH_T * (CH_N / 8); i += CH_THREADS) {
                 const int t = i / (CH_N / 8), k = (i % (CH_N / 8)) * 8;
                 const bool ok = t0 + t < n && k < N;
                 const uint16_t* r = xbc + (size_t)(ok ? t0 + t : 0) * p.ld_xbc;
                 cp_async16_zfill(smem_u32(dC + t * CH_LN + k), r + (ok ? cC + k : 0), ok);
                 cp_async16_zfill(smem_u32(dB + t * CH_LN + k), r + (ok ? cB + k : 0), ok);
             }
-            for (int i = tid; i < CH_T * (CH_P / 8); i += 256) {
+            for (int i = tid; i < CH_T * (CH_P / 8); i += CH_THREADS) {
                 const int t = i / (CH_P / 8), k = (i % (CH_P / 8)) * 8;
                 const bool ok = t0 + t < n && p0 + k < P;
                 cp_async16_zfill(smem_u32(dx + t * CH_LP + k), xbc + (size_t)(ok ? t0 + t : 0) * p.ld_xbc + (ok ? cx + k : 0), ok);
             }
         } else {
-            for (int i = tid; i < CH_T * CH_N; i += 256) {
+            for (int i = tid; i < CH_T * CH_N; i += CH_THREADS) {
                 const int t = i / CH_N, k = i % CH_N;
                 const bool ok = t0 + t < n && k < N;
                 dC[t * CH_LN + k] = ok ? xbc[(size_t)(t0 + t) * p.ld_xbc + cC + k] : 0;
                 dB[t * CH_LN + k] = ok ? xbc[(size_t)(t0 + t) * p.ld_xbc + cB + k] : 0;
             }
-            for (int i = tid; i < CH_T * CH_P; i += 256) {
+            for (int i = tid; i < CH_T * CH_P; i += CH_THREADS) {
                 const int t = i / CH_P, k = i % CH_P;
                 dx[t * CH_LP + k] = t0 + t < n && p0 + k < P ? xbc[(size_t)(t0 + t) * p.ld_xbc + cx + k] : 0;
             }
         }
     };
-    // state of this warp: rows warp * 16 + g4 (+ 8), value rows 8 j + 2 t4 (+ 1)
-    float S[8][4];
+    // state of this warp: rows sr + g4 (+ 8), value rows sp + 8 j + 2 t4 (+ 1)
+    const int sr = (warp >> 1) * 16, sp = (warp & 1) * 32;
+    float S[4][4];
     float* slot = p.state + (size_t)p.seq_slot[b] * p.slot_stride;
     float* Sg = slot + ((size_t)h * P + p0) * N;
 #pragma unroll
-    for (int j = 0; j < 8; j++)
+    for (int j = 0; j < 4; j++)
 #pragma unroll
         for (int e = 0; e < 4; e++) {
-            const int r = warp * 16 + g4 + (e >> 1) * 8, q = j * 8 + 2 * t4 + (e & 1);
+            const int r = sr + g4 + (e >> 1) * 8, q = sp + j * 8 + 2 * t4 + (e & 1);
             S[j][e] = before > 0 && r < N && p0 + q < P ? Sg[(size_t)q * N + r] : 0.f;
         }
-    const int mt = warp >> 1, pc = (warp & 1) * 32;  // y: tokens mt * 16.., value rows pc..
+    const int mt = warp >> 2, jt = warp & 3;  // tokens mt * 16..; earlier tokens jt * 16.. (weights), value rows jt * 16.. (y)
+    const int ta = mt * 16 + g4, tb = ta + 8;
     const int chunks = (n + CH_T - 1) / CH_T;
-    // Step sizes and decays of a chunk, two tokens per lane of warp 0 (which has the least of the triangular product): the raw
+    // Step sizes and decays of a chunk, two tokens per lane of warp 3 (whose tile of the weights is above the diagonal): the raw
     // values are fetched when the chunk before it begins and turned into factors when that warp is done with its part.
     float raw[2] = {0.f, 0.f};
     auto fetch_steps = [&](int c) {
@@ -309,20 +319,20 @@ __global__ void __launch_bounds__(256, 1) chunk_scan_kernel(const Mamba2Spec s, 
     };
     load(0);
     cp_async_commit();
-    if (warp == 0) {
+    if (warp == 3) {
         fetch_steps(0);
         make_steps(0);
     }
     for (int c = 0; c < chunks; c++) {
-        if (warp == 0 && c + 1 < chunks) fetch_steps(c + 1);
+        if (warp == 3 && c + 1 < chunks) fetch_steps(c + 1);
         const int t0 = c * CH_T, cnt = min(CH_T, n - t0);
         const float *dts = steps + (c & 1) * 4 * CH_T, *cum = dts + CH_T, *ecum = cum + CH_T, *wend = ecum + CH_T;
         // the state before this chunk, as operand of C S0
 #pragma unroll
-        for (int j = 0; j < 8; j++)
+        for (int j = 0; j < 4; j++)
 #pragma unroll
             for (int half = 0; half < 2; half++) {
-                const int at = (warp * 16 + g4 + half * 8) * CH_LP + j * 8 + 2 * t4;
+                const int at = (sr + g4 + half * 8) * CH_LP + sp + j * 8 + 2 * t4;
                 const uint32_t hi = pack_bf2(S[j][2 * half], S[j][2 * half + 1]);
                 *reinterpret_cast<uint32_t*>(sh + at) = hi;
                 *reinterpret_cast<uint32_t*>(sh + CH_N * CH_LP + at) = pack_bf2(S[j][2 * half] - bflo(hi), S[j][2 * half + 1] - bfhi(hi));
@@ -333,7 +343,7 @@ __global__ void __launch_bounds__(256, 1) chunk_scan_kernel(const Mamba2Spec s, 
         __syncthreads();
         const uint16_t* sC = reinterpret_cast<const uint16_t*>(in0 + (c & 1) * ChunkSmem::kIn);
         const uint16_t *sB = sC + CH_T * CH_LN, *sx = sB + CH_T * CH_LN;
-        for (int i = tid; i < CH_T * CH_P / 2; i += 256) {  // what the tokens add to the state: exp(c_end - c_s) d_s x_s
+        for (int i = tid; i < CH_T * CH_P / 2; i += CH_THREADS) {  // what the tokens add to the state: exp(c_end - c_s) d_s x_s
             const int t = i / (CH_P / 2), at = t * CH_LP + (i % (CH_P / 2)) * 2;
             const uint32_t x2 = *reinterpret_cast<const uint32_t*>(sx + at);
             const float a0 = bflo(x2) * wend[t], a1 = bfhi(x2) * wend[t];
@@ -341,74 +351,76 @@ __global__ void __launch_bounds__(256, 1) chunk_scan_kernel(const Mamba2Spec s, 
             *reinterpret_cast<uint32_t*>(xw + at) = hi;
             *reinterpret_cast<uint32_t*>(xw + CH_T * CH_LP + at) = pack_bf2(a0 - bflo(hi), a1 - bfhi(hi));
         }
-        // ---- y of this warp
-        float y[4][4], m[8][4];
-#pragma unroll
-        for (int j = 0; j < 4; j++) y[j][0] = y[j][1] = y[j][2] = y[j][3] = 0.f;
-#pragma unroll
-        for (int j = 0; j < 8; j++) m[j][0] = m[j][1] = m[j][2] = m[j][3] = 0.f;
         const uint32_t aC = smem_u32(sC + (mt * 16 + lr + (mi & 1) * 8) * CH_LN + (mi >> 1) * 8);
-        const uint32_t bB = smem_u32(sB + (lr + (mi >> 1) * 8) * CH_LN + (mi & 1) * 8);
-        const uint32_t bS = smem_u32(sh + (lr + (mi & 1) * 8) * CH_LP + pc + (mi >> 1) * 8);
+        if (jt <= mt) {  // weights of 16 tokens on 16 earlier ones
+            float m[2][4];
+#pragma unroll
+            for (int half = 0; half < 2; half++) m[half][0] = m[half][1] = m[half][2] = m[half][3] = 0.f;
+            const uint32_t bB = smem_u32(sB + (jt * 16 + lr + (mi >> 1) * 8) * CH_LN + (mi & 1) * 8);
+            for (int k = 0; k < KN; k++) {
+                uint32_t af[4], v0[2], v1[2];
+                ldmatrix_x4(af[0], af[1], af[2], af[3], aC + k * 32);
+                ldmatrix_x4(v0[0], v0[1], v1[0], v1[1], bB + k * 32);
+                mma_bf16_16816(m[0], af, v0);
+                mma_bf16_16816(m[1], af, v1);
+            }
+            const float ca = cum[ta], cb = cum[tb];
+#pragma unroll
+            for (int half = 0; half < 2; half++) {
+                const int s0 = jt * 16 + half * 8 + 2 * t4;
+#pragma unroll
+                for (int e = 0; e < 4; e++) {
+                    const int si = s0 + (e & 1);
+                    m[half][e] = si <= (e < 2 ? ta : tb) ? m[half][e] * __expf((e < 2 ? ca : cb) - cum[si]) * dts[si] : 0.f;
+                }
+#pragma unroll
+                for (int row = 0; row < 2; row++) {
+                    const int at = (row ? tb : ta) * CH_LM + s0;
+                    const uint32_t hi = pack_bf2(m[half][2 * row], m[half][2 * row + 1]);
+                    *reinterpret_cast<uint32_t*>(sm + at) = hi;
+                    *reinterpret_cast<uint32_t*>(sm + CH_T * CH_LM + at) = pack_bf2(m[half][2 * row] - bflo(hi), m[half][2 * row + 1] - bfhi(hi));
+                }
+            }
+        }
+        // ---- y of this warp: first C S0 (needs nothing of the other warps' weights)
+        float y[2][4];
+        y[0][0] = y[0][1] = y[0][2] = y[0][3] = y[1][0] = y[1][1] = y[1][2] = y[1][3] = 0.f;
+        const uint32_t bS = smem_u32(sh + (lr + (mi & 1) * 8) * CH_LP + jt * 16 + (mi >> 1) * 8);
         for (int k = 0; k < KN; k++) {
             uint32_t af[4];
             ldmatrix_x4(af[0], af[1], af[2], af[3], aC + k * 32);
 #pragma unroll
-            for (int j = 0; j < 2; j++) {  // C S0, head and remainder
-#pragma unroll
-                for (int part = 0; part < 2; part++) {
-                    uint32_t v0[2], v1[2];
-                    ldmatrix_x4_trans(v0[0], v0[1], v1[0], v1[1], bS + (part * CH_N * CH_LP + k * 16 * CH_LP + j * 16) * 2);
-                    mma_bf16_16816(y[2 * j], af, v0);
-                    mma_bf16_16816(y[2 * j + 1], af, v1);
-                }
+            for (int part = 0; part < 2; part++) {
+                uint32_t v0[2], v1[2];
+                ldmatrix_x4_trans(v0[0], v0[1], v1[0], v1[1], bS + (part * CH_N * CH_LP + k * 16 * CH_LP) * 2);
+                mma_bf16_16816(y[0], af, v0);
+                mma_bf16_16816(y[1], af, v1);
             }
-#pragma unroll
-            for (int j = 0; j < 4; j++)
-                if (j <= mt) {  // C B^T up to the diagonal
-                    uint32_t v0[2], v1[2];
-                    ldmatrix_x4(v0[0], v0[1], v1[0], v1[1], bB + (j * 16 * CH_LN + k * 16) * 2);
-                    mma_bf16_16816(m[2 * j], af, v0);
-                    mma_bf16_16816(m[2 * j + 1], af, v1);
-                }
         }
-        const int ta = mt * 16 + g4, tb = ta + 8;
-        const float ca = cum[ta], cb = cum[tb], ea = ecum[ta], eb = ecum[tb];
+        const float ea = ecum[ta], eb = ecum[tb];
 #pragma unroll
-        for (int j = 0; j < 4; j++) y[j][0] *= ea, y[j][1] *= ea, y[j][2] *= eb, y[j][3] *= eb;
-        const uint32_t bX = smem_u32(sx + (lr + (mi & 1) * 8) * CH_LP + pc + (mi >> 1) * 8);
+        for (int q = 0; q < 2; q++) y[q][0] *= ea, y[q][1] *= ea, y[q][2] *= eb, y[q][3] *= eb;
+        if (warp == 3 && c + 1 < chunks) make_steps(c + 1);
+        __syncthreads();  // the weights and the state's increments are complete
+        const uint32_t aM = smem_u32(sm + (mt * 16 + lr + (mi & 1) * 8) * CH_LM + (mi >> 1) * 8);
+        const uint32_t bX = smem_u32(sx + (lr + (mi & 1) * 8) * CH_LP + jt * 16 + (mi >> 1) * 8);
 #pragma unroll
-        for (int j = 0; j < 4; j++)
-            if (j <= mt) {  // 16 earlier tokens: weights from the accumulator layout to the operand layout
-                uint32_t hi[4], lo[4];
-#pragma unroll
-                for (int half = 0; half < 2; half++) {
-                    float* v = m[2 * j + half];
-#pragma unroll
-                    for (int e = 0; e < 4; e++) {
-                        const int sidx = j * 16 + half * 8 + 2 * t4 + (e & 1), t = e < 2 ? ta : tb;
-                        v[e] = sidx <= t ? v[e] * expf((e < 2 ? ca : cb) - cum[sidx]) * dts[sidx] : 0.f;
-                    }
-                    hi[2 * half] = pack_bf2(v[0], v[1]);
-                    hi[2 * half + 1] = pack_bf2(v[2], v[3]);
-                    lo[2 * half] = pack_bf2(v[0] - bflo(hi[2 * half]), v[1] - bfhi(hi[2 * half]));
-                    lo[2 * half + 1] = pack_bf2(v[2] - bflo(hi[2 * half + 1]), v[3] - bfhi(hi[2 * half + 1]));
-                }
-#pragma unroll
-                for (int q = 0; q < 2; q++) {
-                    uint32_t v0[2], v1[2];
-                    ldmatrix_x4_trans(v0[0], v0[1], v1[0], v1[1], bX + (j * 16 * CH_LP + q * 16) * 2);
-                    mma_bf16_16816(y[2 * q], hi, v0);
-                    mma_bf16_16816(y[2 * q + 1], hi, v1);
-                    mma_bf16_16816(y[2 * q], lo, v0);
-                    mma_bf16_16816(y[2 * q + 1], lo, v1);
-                }
+        for (int k = 0; k < CH_T / 16; k++)
+            if (k <= mt) {
+                uint32_t hi[4], lo[4], v0[2], v1[2];
+                ldmatrix_x4(hi[0], hi[1], hi[2], hi[3], aM + k * 32);
+                ldmatrix_x4(lo[0], lo[1], lo[2], lo[3], aM + CH_T * CH_LM * 2 + k * 32);
+                ldmatrix_x4_trans(v0[0], v0[1], v1[0], v1[1], bX + k * 16 * CH_LP * 2);
+                mma_bf16_16816(y[0], hi, v0);
+                mma_bf16_16816(y[1], hi, v1);
+                mma_bf16_16816(y[0], lo, v0);
+                mma_bf16_16816(y[1], lo, v1);
             }
 #pragma unroll
-        for (int j = 0; j < 4; j++)
+        for (int j = 0; j < 2; j++)
 #pragma unroll
             for (int half = 0; half < 2; half++) {
-                const int t = half ? tb : ta, q = pc + j * 8 + 2 * t4;
+                const int t = half ? tb : ta, q = jt * 16 + j * 8 + 2 * t4;
                 if (t >= cnt) continue;
                 const uint32_t x2 = *reinterpret_cast<const uint32_t*>(sx + t * CH_LP + q);
                 const float y0 = fmaf(D, bflo(x2), y[j][2 * half]), y1 = fmaf(D, bfhi(x2), y[j][2 * half + 1]);
@@ -420,21 +432,19 @@ __global__ void __launch_bounds__(256, 1) chunk_scan_kernel(const Mamba2Spec s, 
                     if (p0 + q + 1 < P) o[1] = y1;
                 }
             }
-        if (warp == 0 && c + 1 < chunks) make_steps(c + 1);
-        __syncthreads();  // xw is complete
         // ---- state of this warp
-        if (warp < KN) {
+        if (sr < N) {
             const float dec = ecum[CH_T - 1];
 #pragma unroll
-            for (int j = 0; j < 8; j++) S[j][0] *= dec, S[j][1] *= dec, S[j][2] *= dec, S[j][3] *= dec;
-            const uint32_t aB = smem_u32(sB + (lr + (mi >> 1) * 8) * CH_LN + warp * 16 + (mi & 1) * 8);
-            const uint32_t bW = smem_u32(xw + (lr + (mi & 1) * 8) * CH_LP + (mi >> 1) * 8);
+            for (int j = 0; j < 4; j++) S[j][0] *= dec, S[j][1] *= dec, S[j][2] *= dec, S[j][3] *= dec;
+            const uint32_t aB = smem_u32(sB + (lr + (mi >> 1) * 8) * CH_LN + sr + (mi & 1) * 8);
+            const uint32_t bW = smem_u32(xw + (lr + (mi & 1) * 8) * CH_LP + sp + (mi >> 1) * 8);
 #pragma unroll
             for (int k = 0; k < CH_T / 16; k++) {
                 uint32_t af[4];
                 ldmatrix_x4_trans(af[0], af[1], af[2], af[3], aB + k * 16 * CH_LN * 2);
 #pragma unroll
-                for (int j = 0; j < 4; j++)
+                for (int j = 0; j < 2; j++)
 #pragma unroll
                     for (int part = 0; part < 2; part++) {
                         uint32_t v0[2], v1[2];
@@ -447,10 +457,10 @@ __global__ void __launch_bounds__(256, 1) chunk_scan_kernel(const Mamba2Spec s, 
         __syncthreads();  // this chunk's buffers may be written again
     }
 #pragma unroll
-    for (int j = 0; j < 8; j++)
+    for (int j = 0; j < 4; j++)
 #pragma unroll
         for (int e = 0; e < 4; e++) {
-            const int r = warp * 16 + g4 + (e >> 1) * 8, q = j * 8 + 2 * t4 + (e & 1);
+            const int r = sr + g4 + (e >> 1) * 8, q = sp + j * 8 + 2 * t4 + (e & 1);
             if (r < N && p0 + q < P) Sg[(size_t)q * N + r] = S[j][e];
         }
     keep_conv_inputs<uint16_t>(s, p, slot, start, n, before, h, p0, CH_P, blockIdx.x == 0);
@@ -525,7 +535,7 @@ int32_t launch_ssm(b2_ctx* ctx, const Mamba2Spec& s, const SsmParams& p) {
     q.chunked = sizeof(T) == 2 && s.state <= CH_N && p.T >= p.B - 1 + kChunkMin;  // some sequence may bring enough tokens
     if (q.chunked) {
         B2_SMEM_ONCE(ctx, chunk_scan_kernel, ChunkSmem::kBytes);
-        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, chunk_scan_kernel, dim3((s.vdim + CH_P - 1) / CH_P, s.heads, p.B), dim3(256), (size_t)ChunkSmem::kBytes,
+        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, chunk_scan_kernel, dim3((s.vdim + CH_P - 1) / CH_P, s.heads, p.B), dim3(CH_THREADS), (size_t)ChunkSmem::kBytes,
                               ctx->stream, s, q));
         B2_LAUNCHED(ctx);
     }

@@ -18,18 +18,6 @@ __device__ __forceinline__ void mbar_arrive(uint32_t addr) {
 __device__ __forceinline__ void mbar_expect_tx(uint32_t addr, uint32_t bytes) {
     asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;\n" ::"r"(addr), "r"(bytes) : "memory");
 }
-// One look: has the phase of this parity completed?
-__device__ __forceinline__ bool mbar_test(uint32_t addr, uint32_t parity) {
-    uint32_t ok;
-    asm volatile(
-        "{\n\t.reg .pred p;\n\t"
-        "mbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
-        "selp.u32 %0, 1, 0, p;\n\t}\n"
-        : "=r"(ok)
-        : "r"(addr), "r"(parity)
-        : "memory");
-    return ok != 0;
-}
 // Bounded wait; false when the limit (about 2 s) ran out.
 __device__ __forceinline__ bool mbar_wait(uint32_t addr, uint32_t parity) {
     long long start = 0;

@@ -179,13 +179,23 @@ def single(eng, ctx, layer, f32, gain=None, n=140, cuts=None, seed=2, width=64, 
 
 @pytest.mark.parametrize("f32", [True, False])
 @pytest.mark.parametrize("cuts", [[140], [60, 1, 1, 1, 30, 2], []], ids=["prompt", "portions", "tokens"])
-@pytest.mark.parametrize("heads,dims", [(2, dict(dim=32, rot_dim=32, vdim=32)), (20, dict(dim=16, rot_dim=8, vdim=8))])
+@pytest.mark.parametrize("heads,dims", [(2, dict(dim=32, rot_dim=32, vdim=32)), (20, dict(dim=16, rot_dim=8, vdim=8)), (3, dict(dim=40, rot_dim=24, vdim=100)),
+                                        (2, dict(dim=100, rot_dim=34, vdim=48)), (1, dict(dim=56, rot_dim=72, vdim=65)), (40, dict(dim=8, rot_dim=4, vdim=6))])
 def test_latent_attention_with_sharp_scores(env, cuts, f32, heads, dims):
     """Queries and keys scaled so that single keys stand out: one wrong, missing or extra key shows."""
     ctx, eng = env
     gain = {".q": 4.0}
     e = single(eng, ctx, (lm.latent(heads=heads, kv_rank=64, base=200.0, **dims), None), f32, gain=gain, cuts=cuts)
     assert e < (5e-5 if f32 else 0.1), e
+
+
+@pytest.mark.parametrize("f32", [True, False])
+@pytest.mark.parametrize("rank", [9, 130, 448, 520])
+def test_latent_sizes(env, rank, f32):
+    """Ranks of one to several value blocks, and one beyond the tensor-core decode kernel's reach."""
+    ctx, eng = env
+    e = single(eng, ctx, (lm.latent(heads=3, dim=32, rot_dim=16, vdim=24, kv_rank=rank), None), f32, n=150, cuts=[100, 1, 1, 30, 2])
+    assert e < TOL[f32], e
 
 
 @pytest.mark.parametrize("f32", [True, False])
@@ -231,6 +241,7 @@ def test_key_far_away(env, f32):
 @pytest.mark.parametrize("f32", [True, False])
 @pytest.mark.parametrize("cuts", [[140], [2] * 70, [64, 1, 63], []], ids=["prompt", "twos", "portions", "tokens"])
 @pytest.mark.parametrize("m", [dict(), dict(heads=3, groups=1, vdim=17, state=33, conv=2, norm_groups=3), dict(heads=8, groups=8, vdim=16, state=16, conv=6, norm_groups=1),
+                               dict(heads=3, groups=3, vdim=80, state=64, conv=1, norm_groups=3),
                                dict(heads=2, groups=1, vdim=64, state=128, conv=4, norm_groups=1)])
 def test_mamba2_alone(env, m, cuts, f32):
     ctx, eng = env
