@@ -613,7 +613,7 @@ int32_t Fwd::latent(const LayerSpec& L, const LayerP& P, int l) {
                 dp.positions = s.mo->positions;
                 dp.token_seq = s.mo->token_seq;
                 dp.seq_slot = s.in->seq_slot;
-                dp.chunk_tiles = up(s.max_ctx, 64) / 16;
+                dp.chunk_tiles = up(s.max_ctx, b2_latent_decode_tile()) / 16;
             }
             dp.scale_log2 = scale_log2;
             dp.o_lat = b.o_lat;
@@ -765,7 +765,7 @@ int32_t Fwd::moe(const LayerSpec& L, const LayerP& P, const int32_t** rows) {
 
 int b2_layered_q_tile(const b2_model*) { return 128; }
 // One CTA of the decode attention fills an SM, so the work items (times the head groups) should fill whole rounds of the
-// machine: the smallest chunk, in whole 64-key tiles from 128 keys on, that does not open another round.
+// machine: the smallest chunk, in whole tiles from 128 keys on, that does not open another round.
 int b2_layered_chunk_tiles(const b2_model* m, const std::vector<SeqStep>& seqs) {
     int groups = 1;
     for (auto& L : m->layered->spec.layers)
@@ -783,15 +783,16 @@ int b2_layered_chunk_tiles(const b2_model* m, const std::vector<SeqStep>& seqs) 
             if (s.n == 1) n += (s.cache->len + keys) / keys;
         return n;
     };
-    int lo = 2, hi = std::max(2, (longest + 63) / 64);  // in 64-key tiles; a chunk of the longest context is one item per row
+    const int tile = b2_latent_decode_tile();
+    int lo = (128 + tile - 1) / tile, hi = std::max(lo, (longest + tile - 1) / tile);  // in tiles; the longest context in one chunk is one item per row
     while (lo < hi) {
         const int mid = (lo + hi) / 2;
-        if (items(mid * 64) <= budget)
+        if (items(mid * tile) <= budget)
             hi = mid;
         else
             lo = mid + 1;
     }
-    return lo * 4;
+    return lo * tile / 16;
 }
 
 void b2_layered_cache_layout(const b2_model* m, int block_size, std::vector<std::vector<size_t>>& page_bytes, int64_t& state_floats) {

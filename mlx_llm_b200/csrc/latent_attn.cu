@@ -118,22 +118,24 @@ __global__ void __launch_bounds__(128) latent_attn_simple_kernel(const LatentAtt
 // ---- decode: tcgen05, keys split over CTAs -----------------------------------------------------------------------------
 // One cached row serves every head, so the heads are rows of one product and columns of the other:
 //   S [heads x keys] = Q [heads x W] . K^T,   O^T [R x heads] += K[:, :R]^T [R x keys] . P^T [keys x heads]
-// CTA = (one chunk of one sequence's keys, up to NH heads), 64 keys per tile, two tiles in shared memory:
+// CTA = (one chunk of one sequence's keys, up to NH heads), 48 keys per tile, three tiles in shared memory (two for very wide
+// rows): a tile stays from its first load to the end of its second product, and the deeper ring is what keeps loads going:
 //   warp 1           TMA: boxes of 16 keys x 64 values located through the block table, 128-byte swizzle
 //   warps 2, 3       one thread each issues tcgen05.mma: S, a few 64-value blocks of a tile at a time as they arrive, into one
-//                    of two TMEM buffers; O^T of a tile when its P is complete, which frees its place.  The tile is the
+//                    of the TMEM buffers; O^T of a tile when its P is complete, which frees its place.  The tile is the
 //                    K-major B operand of the first product and, transposed, the MN-major A operand of the second;
 //                    Q has fewer than the 128 rows the first product computes: the rows past NH are whatever follows in shared
 //                    memory and end in TMEM lanes nobody reads
-//   warps 0 4 8 12   softmax (these warps reach TMEM lanes 0-31): thread = (head, 16 keys); P goes to shared memory, K-major,
+//   warps 0 4 8      softmax (these warps reach TMEM lanes 0-31): thread = (head, 16 keys); P goes to shared memory, K-major,
 //                    as bf16 head and bf16 remainder (2 NH columns of the second product: an MMA costs the same at 32 and at 64)
 //   warps 16-19      follow the row maxima and rescale O^T in TMEM when one rises by more than 2^8 (lazily: the division by
 //                    the row sum makes the result independent of the reference point); epilogue, thread = latent value
 // Scores and weights are f32.  Keys past the chunk are other tokens' rows (finite) and get weight zero.  Every wait is
 // bounded.  With more than one chunk a sequence's partial results (f32) are added in chunk order by a second kernel: one block
 // per (sequence, head), so that long contexts spread over the machine.
-constexpr int DK_KEYS = 64, DK_BLOCK = DK_KEYS * 128;  // keys per tile; 64 keys x 64 values
-constexpr int kDecodeMaxRank = 512, kDecodeThreads = 640;
+constexpr int DK_KEYS = 48, DK_BLOCK = DK_KEYS * 128;  // keys per tile; bytes of 48 keys x 64 values
+constexpr int DK_SOFT = DK_KEYS / 16, DK_WALK = (DK_SOFT + 4) * 32;  // softmax warps; threads that walk the tiles together
+constexpr int kDecodeMaxRank = 512, kDecodeThreads = 640, kDecodeMaxSmem = 226 * 1024;
 constexpr int DK_GB = 3, DK_NG = 4;                    // 64-value blocks per arrival barrier; barriers per tile (W up to 768)
 constexpr float kDecodeRescale = 8.0f;                 // log2 units
 
@@ -141,14 +143,15 @@ template <int NH>
 struct DecodeSmem {
     static constexpr int kQBlock = NH * 128, kP = NH * 128;  // one 64-value block of Q; one operand of P
     static __host__ __device__ int blocks(int W) { return (W + 63) / 64; }
-    static __host__ __device__ int q_off(int W) { return 2 * blocks(W) * DK_BLOCK; }
-    static __host__ __device__ int p_off(int W) { return q_off(W) + blocks(W) * kQBlock; }
-    // behind P (two tiles x head, remainder): barriers, maxima and sums, then room for the rows past NH of the last Q block
-    static __host__ __device__ int x_off(int W) { return p_off(W) + 4 * kP; }
-    static __host__ __device__ int bytes(int W) {
-        const int used = x_off(W) + 256 + 3 * 4 * 32 * 4, reach = p_off(W) - kQBlock + 128 * 128;
+    static __host__ __device__ int q_off(int W, int ns) { return ns * blocks(W) * DK_BLOCK; }
+    static __host__ __device__ int p_off(int W, int ns) { return q_off(W, ns) + blocks(W) * kQBlock; }
+    // behind P (a head and a remainder per tile): barriers, maxima and sums, then room for the rows past NH of the last Q block
+    static __host__ __device__ int x_off(int W, int ns) { return p_off(W, ns) + ns * 2 * kP; }
+    static __host__ __device__ int bytes(int W, int ns) {
+        const int used = x_off(W, ns) + 256 + 3 * DK_SOFT * 32 * 4, reach = p_off(W, ns) - kQBlock + 128 * 128;
         return used > reach ? used : reach;
     }
+    static int stages(int W) { return bytes(W, 3) <= kDecodeMaxSmem ? 3 : bytes(W, 2) <= kDecodeMaxSmem ? 2 : 0; }
 };
 
 template <int NH>
@@ -158,31 +161,31 @@ __global__ void __launch_bounds__(kDecodeThreads, 1)
     using L = DecodeSmem<NH>;
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     extern __shared__ __align__(1024) uint8_t smem[];
-    const int W = a.row_pad(), R = a.kv_rank, NB = L::blocks(W), NG = (NB + DK_GB - 1) / DK_GB, MB = (R + 127) / 128;
+    const int W = a.row_pad(), R = a.kv_rank, NB = L::blocks(W), NG = (NB + DK_GB - 1) / DK_GB, MB = (R + 127) / 128, NS = p.stages;
     const uint32_t base = smem_u32(smem);
     if (base & 1023u) {  // the swizzled layouts need this alignment; every thread sees the same value
         if (threadIdx.x == 0) atomicExch(err, 7);
         return;
     }
-    const uint32_t sQ = base + L::q_off(W), sP = base + L::p_off(W), bar = base + L::x_off(W);
+    const uint32_t sQ = base + L::q_off(W, NS), sP = base + L::p_off(W, NS), bar = base + L::x_off(W, NS);
     auto empty = [&](int s) { return bar + 8u * s; };
-    auto s_ready = [&](int s) { return bar + 8u * (2 + s); };
-    auto p_ready = [&](int s) { return bar + 8u * (4 + s); };
-    auto pv_done = [&](int s) { return bar + 8u * (6 + s); };
-    auto o_ready = [&](int s) { return bar + 8u * (8 + s); };
-    const uint32_t slot_addr = bar + 8u * 10;
-    auto full = [&](int s, int g) { return bar + 8u * (12 + s * DK_NG + g); };
-    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(smem + L::x_off(W) + 8 * 10);
-    float* xm = reinterpret_cast<float*>(smem + L::x_off(W) + 256);  // [2 tiles][4 warps][32 heads] maxima
-    float* xl = xm + 2 * 4 * 32;                                     // [4 warps][32 heads] row sums
+    auto s_ready = [&](int s) { return bar + 8u * (3 + s); };
+    auto p_ready = [&](int s) { return bar + 8u * (6 + s); };
+    auto pv_done = [&](int s) { return bar + 8u * (9 + s); };
+    auto o_ready = [&](int s) { return bar + 8u * (12 + s); };
+    const uint32_t slot_addr = bar + 8u * 15;
+    auto full = [&](int s, int g) { return bar + 8u * (16 + s * DK_NG + g); };
+    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(smem + L::x_off(W, NS) + 8 * 15);
+    float* xm = reinterpret_cast<float*>(smem + L::x_off(W, NS) + 256);  // [2 tiles][softmax warps][32 heads] maxima
+    float* xl = xm + 2 * DK_SOFT * 32;                                   // [softmax warps][32 heads] row sums
 
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     if (tid == 0) {
-        for (int i = 0; i < 2; i++) {
+        for (int i = 0; i < NS; i++) {
             for (int g = 0; g < DK_NG; g++) mbar_init(full(i, g), 1);
             mbar_init(empty(i), 1);
             mbar_init(s_ready(i), 1);
-            mbar_init(p_ready(i), 4);
+            mbar_init(p_ready(i), DK_SOFT);
             mbar_init(pv_done(i), 1);
             mbar_init(o_ready(i), 4);
         }
@@ -229,36 +232,40 @@ __global__ void __launch_bounds__(kDecodeThreads, 1)
     tc_fence_before();
     __syncthreads();
     tc_fence_after();
-    const uint32_t tmem = *tmem_slot, tmem_o = tmem + 128u;
+    const uint32_t tmem = *tmem_slot, tmem_o = tmem + 192u;
     bool alive = true;
 
     if (warp == 1) {
         const int32_t* bt = p.block_tables + (size_t)slot * p.max_blocks;
-        const int sub = lane & 3;
+        const int sub = lane % DK_SOFT, first = lane / DK_SOFT;
         auto row_of = [&](int j) {  // a box past the chunk repeats the chunk's first page: any finite rows will do
             const int key = k_lo + j * DK_KEYS + sub * 16, kk = key < k_hi ? key : k_lo;
             return bt[kk / p.page_size] * p.page_size + kk % p.page_size;
         };
-        int next = row_of(0);
+        int next = row_of(0), st = 0;
+        uint32_t ph = 0;
         for (int j = 0; j < n_tiles; j++) {
-            const int row = next, st = j & 1;
+            const int row = next;
             next = row_of(j + 1);
-            if (!__all_sync(0xffffffffu, mbar_wait(empty(st), ((uint32_t)(j >> 1) & 1u) ^ 1u))) {
+            if (!__all_sync(0xffffffffu, mbar_wait(empty(st), ph ^ 1u))) {
                 if (lane == 0) atomicExch(err, 16);
                 break;
             }
             if (lane < NG) mbar_expect_tx(full(st, lane), (uint32_t)min(DK_GB, NB - lane * DK_GB) * DK_BLOCK);
             __syncwarp();
-            for (int i = lane >> 2; i < NB; i += 8) tma_load_2d(base + (st * NB + i) * DK_BLOCK + sub * 2048, &map, i * 64, row, full(st, i / DK_GB));
+            if (first < 32 / DK_SOFT)
+                for (int i = first; i < NB; i += 32 / DK_SOFT) tma_load_2d(base + (st * NB + i) * DK_BLOCK + sub * 2048, &map, i * 64, row, full(st, i / DK_GB));
+            if (++st == NS) st = 0, ph ^= 1u;
         }
         __syncwarp();
     } else if (warp == 2) {
         if (lane == 0) {
             constexpr uint32_t kQK = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(DK_KEYS >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
+            int st = 0;
+            uint32_t ph = 0;
             for (int j = 0; j < n_tiles && alive; j++) {
-                const int st = j & 1;
                 for (int g = 0; g < NG; g++) {
-                    alive = mbar_wait(full(st, g), (uint32_t)(j >> 1) & 1u);
+                    alive = mbar_wait(full(st, g), ph);
                     if (!alive) break;
                     tc_fence_after();
                     for (int b = g * DK_GB; b < min(NB, (g + 1) * DK_GB); b++) {
@@ -268,6 +275,7 @@ __global__ void __launch_bounds__(kDecodeThreads, 1)
                     }
                 }
                 if (alive) tc_commit(s_ready(st));
+                if (++st == NS) st = 0, ph ^= 1u;
             }
             if (!alive) atomicExch(err, 17);
         }
@@ -275,9 +283,9 @@ __global__ void __launch_bounds__(kDecodeThreads, 1)
     } else if (warp == 3) {
         if (lane == 0) {
             constexpr uint32_t kPV = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 15) | ((uint32_t)(2 * NH >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
+            int st = 0;
+            uint32_t ph = 0;
             for (int j = 0; j < n_tiles && alive; j++) {
-                const int st = j & 1;
-                const uint32_t ph = (uint32_t)(j >> 1) & 1u;
                 // (P exists, so S of this tile has been computed: its stage may be freed when these products are done)
                 alive = mbar_wait(p_ready(st), ph) && mbar_wait(o_ready(st), ph);
                 if (!alive) break;
@@ -292,23 +300,25 @@ __global__ void __launch_bounds__(kDecodeThreads, 1)
                 }
                 tc_commit(pv_done(st));
                 tc_commit(empty(st));
+                if (++st == NS) st = 0, ph ^= 1u;
             }
             if (!alive) atomicExch(err, 18);
         }
         __syncwarp();
-    } else if (warp >= 16 || (warp & 3) == 0) {
+    } else if (warp >= 16 || ((warp & 3) == 0 && warp < 4 * DK_SOFT)) {
         // softmax warps and O^T warps walk the tiles together: one barrier per tile, behind the tile's row maxima
         const bool soft = warp < 16;
         const int q = warp >> 2;  // softmax: keys q * 16 .. of the tile
         const uint32_t lane_addr = (uint32_t)((warp & 3) * 32) << 16;
         const bool real = lane < NH && h0 + lane < a.heads;
         float m_run = -INFINITY, l = 0.f;
+        int st = 0, prev = 0;  // stage of this tile, of the one before
+        uint32_t ph = 0, prev_ph = 0;
         for (int j = 0; j < n_tiles; j++) {
-            const int st = j & 1;
-            float* mx = xm + st * 128;
+            float* mx = xm + (j & 1) * DK_SOFT * 32;
             uint32_t v[16];
             if (soft) {
-                alive = __all_sync(0xffffffffu, alive && mbar_wait(s_ready(st), (uint32_t)(j >> 1) & 1u));
+                alive = __all_sync(0xffffffffu, alive && mbar_wait(s_ready(st), ph));
                 tc_fence_after();
                 tc_ld16(tmem + (uint32_t)st * 64u + (uint32_t)q * 16u, v);
                 const int key0 = k_lo + j * DK_KEYS + q * 16;
@@ -321,9 +331,11 @@ __global__ void __launch_bounds__(kDecodeThreads, 1)
                 }
                 mx[q * 32 + lane] = m;
             }
-            asm volatile("bar.sync 1, 256;\n" ::: "memory");
+            asm volatile("bar.sync 1, %0;\n" ::"n"(DK_WALK) : "memory");
             // every warp follows the reference points by itself (lane = head), from the same numbers
-            const float m = fmaxf(fmaxf(mx[lane], mx[32 + lane]), fmaxf(mx[64 + lane], mx[96 + lane]));
+            float m = mx[lane];
+#pragma unroll
+            for (int w = 1; w < DK_SOFT; w++) m = fmaxf(m, mx[w * 32 + lane]);
             float alpha = 1.f;
             if (j == 0) {
                 m_run = m;  // a chunk's first key is visible
@@ -342,7 +354,7 @@ __global__ void __launch_bounds__(kDecodeThreads, 1)
                     lo[i] = pack_bf2(e0 - bflo(hi[i]), e1 - bfhi(hi[i]));
                 }
                 if (lane < NH) {
-                    uint8_t* dst = smem + L::p_off(W) + st * 2 * L::kP + lane * 128;
+                    uint8_t* dst = smem + L::p_off(W, NS) + st * 2 * L::kP + lane * 128;
 #pragma unroll
                     for (int i = 0; i < 2; i++) {
                         const int at = ((2 * q + i) ^ (lane & 7)) << 4;
@@ -357,7 +369,7 @@ __global__ void __launch_bounds__(kDecodeThreads, 1)
             } else {
                 if (__any_sync(0xffffffffu, alpha != 1.f)) {
                     // P V of the tile before must be complete (that of the tile before it is: its stage has been loaded again)
-                    alive = __all_sync(0xffffffffu, alive && mbar_wait(pv_done(st ^ 1), (uint32_t)((j - 1) >> 1) & 1u));
+                    alive = __all_sync(0xffffffffu, alive && mbar_wait(pv_done(prev), prev_ph));
                     tc_fence_after();
                     for (int c = 0; c < MB * 2 * NH; c += 16) {
                         uint32_t o[16];
@@ -371,13 +383,17 @@ __global__ void __launch_bounds__(kDecodeThreads, 1)
                 __syncwarp();
                 if (lane == 0) mbar_arrive(o_ready(st));
             }
+            prev = st, prev_ph = ph;
+            if (++st == NS) st = 0, ph ^= 1u;
         }
         if (soft) xl[q * 32 + lane] = l;
-        asm volatile("bar.sync 1, 256;\n" ::: "memory");
+        asm volatile("bar.sync 1, %0;\n" ::"n"(DK_WALK) : "memory");
         if (!soft) {
-            alive = __all_sync(0xffffffffu, alive && mbar_wait(pv_done((n_tiles - 1) & 1), (uint32_t)((n_tiles - 1) >> 1) & 1u));
+            alive = __all_sync(0xffffffffu, alive && mbar_wait(pv_done(prev), prev_ph));
             tc_fence_after();
-            l = xl[lane] + xl[32 + lane] + xl[64 + lane] + xl[96 + lane];
+            l = xl[lane];
+#pragma unroll
+            for (int w = 1; w < DK_SOFT; w++) l += xl[w * 32 + lane];
             const float inv = 1.0f / l;
             uint16_t* out = reinterpret_cast<uint16_t*>(p.o_lat) + ((size_t)qrow * a.heads + h0) * p.o_pad;
             const size_t slot0 = (size_t)(part0 + chunk) * a.heads + h0;
@@ -466,17 +482,20 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const LatentAttnSpec 
 
 }  // namespace
 
+static int decode_stages(const LatentAttnSpec& a) { return a.heads > 16 ? DecodeSmem<32>::stages(a.row_pad()) : DecodeSmem<16>::stages(a.row_pad()); }
+int b2_latent_decode_tile() { return DK_KEYS; }
 bool b2_latent_decode_eligible(const LatentAttnSpec& a) {
-    return a.kv_rank <= kDecodeMaxRank && a.row_pad() <= DK_NG * DK_GB * 64 && (a.heads > 16 ? DecodeSmem<32>::bytes(a.row_pad()) : DecodeSmem<16>::bytes(a.row_pad())) <= 226 * 1024;
+    return a.kv_rank <= kDecodeMaxRank && a.row_pad() <= DK_NG * DK_GB * 64 && decode_stages(a) > 0;
 }
-int32_t b2_latent_decode_launch(b2_ctx* ctx, const LatentAttnSpec& a, const LatentDecodeParams& p, int items, int rows) {
+int32_t b2_latent_decode_launch(b2_ctx* ctx, const LatentAttnSpec& a, LatentDecodeParams p, int items, int rows) {
     if (items <= 0) return B2_OK;
+    p.stages = decode_stages(a);
     const dim3 grid(items, a.heads > 16 ? (a.heads + 31) / 32 : 1);
     CUtensorMap map;
     B2_CHECK(tc5::get_map(ctx, p.cache, (uint64_t)p.cache_rows, (uint64_t)a.row_pad(), (uint64_t)a.row_pad(), 16, &map));
-    B2_SMEM_ONCE(ctx, latent_decode_kernel<16>, 226 * 1024);
-    B2_SMEM_ONCE(ctx, latent_decode_kernel<32>, 226 * 1024);
-    const int smem = a.heads > 16 ? DecodeSmem<32>::bytes(a.row_pad()) : DecodeSmem<16>::bytes(a.row_pad());
+    B2_SMEM_ONCE(ctx, latent_decode_kernel<16>, kDecodeMaxSmem);
+    B2_SMEM_ONCE(ctx, latent_decode_kernel<32>, kDecodeMaxSmem);
+    const int smem = a.heads > 16 ? DecodeSmem<32>::bytes(a.row_pad(), p.stages) : DecodeSmem<16>::bytes(a.row_pad(), p.stages);
     B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, a.heads > 16 ? latent_decode_kernel<32> : latent_decode_kernel<16>, grid, dim3(kDecodeThreads), (size_t)smem, ctx->stream, a,
                           p, ctx->dev_err, map));
     B2_LAUNCHED(ctx);

@@ -110,7 +110,8 @@ struct LatentDecodeParams {
     const int32_t *positions, *token_seq, *seq_slot;
     // work items (row, chunk): the packer's list, or (work_seq null) one per row, whose chunk must hold its whole context
     const int32_t *work_seq, *work_chunk, *work_off, *n_work;
-    int chunk_tiles;   // 16-key tiles per chunk (a multiple of 4)
+    int chunk_tiles;   // 16-key boxes per chunk (whole tiles of b2_latent_decode_tile() keys)
+    int stages;        // set by the launcher: tiles in shared memory
     int64_t cache_rows;  // rows of the cache allocation
     float scale_log2;  // scale * log2(e)
     float *part_o, *part_ml;  // [work item][head][kv_rank], [work item][head][2]
@@ -118,7 +119,8 @@ struct LatentDecodeParams {
     int o_pad;
 };
 bool b2_latent_decode_eligible(const LatentAttnSpec& a);
-int32_t b2_latent_decode_launch(b2_ctx* ctx, const LatentAttnSpec& a, const LatentDecodeParams& p, int items, int rows);
+int32_t b2_latent_decode_launch(b2_ctx* ctx, const LatentAttnSpec& a, LatentDecodeParams p, int items, int rows);
+int b2_latent_decode_tile();  // keys per tile
 int32_t b2_latent_attn_simple_launch(b2_ctx* ctx, bool f32, const LatentAttnSpec& a, const LatentAttnParams& p);
 
 // ---- latent_prefill.cu: portions of more than one token (bf16), keys and values expanded per head --------------------
