@@ -39,7 +39,7 @@ struct LayerP {
     GroupW e_gu, e_down;
 };
 struct RopeTab {
-    PairRotSpec spec;
+    RotSpec spec;
     float *cos = nullptr, *sin = nullptr;
 };
 

@@ -76,11 +76,79 @@ void read_mamba2(Reader& r, const Value* m, const std::string& at, LayerSpec& L)
     r.require(s.heads % s.groups == 0, at + ": groups must divide heads");
     r.require(s.inner() % s.norm_groups == 0, at + ": norm_groups must divide heads * vdim");
 }
+void read_rot(Reader& r, const Value* m, const std::string& at, int dim, RotSpec& rot) {
+    const Value* v = r.obj(m, "rot", at);
+    rot.base = r.real(v, "base", at + ".rot");
+    rot.dims = r.num(v, "dims", at + ".rot", 0);
+    r.require(rot.dims % 2 == 0 && rot.dims <= dim, at + ": rot.dims must be even and at most dim");
+    r.require(rot.base > 0, at + ": rot.base must be positive");
+}
+void read_retention(Reader& r, const Value* m, const std::string& at, LayerSpec& L) {
+    MemorySpec& s = L.mem;
+    L.mixer = MixerKind::Memory;
+    s.heads = s.kv_heads = r.num(m, "heads", at);
+    s.dim = r.num(m, "dim", at);
+    s.vdim = r.num(m, "vdim", at);
+    read_rot(r, m, at, s.dim, s.rot);
+    const Value* d = m ? m->get("decay") : nullptr;
+    r.require(d && d->kind == Value::Array && (int)d->arr.size() == s.heads, at + ": `decay` must list one number per head");
+    if (!r.err.empty()) return;
+    for (auto& v : d->arr) {
+        double x = 0;
+        r.require(v->as_f64(x) && x > 0 && x <= 1, at + ": a decay must be in (0, 1]");
+        L.decay.push_back(x);
+    }
+}
+void read_delta_sizes(Reader& r, const Value* m, const std::string& at, MemorySpec& s) {
+    s.heads = r.num(m, "heads", at);
+    s.kv_heads = r.num(m, "kv_heads", at);
+    s.dim = r.num(m, "dim", at);
+    s.vdim = r.num(m, "vdim", at);
+    s.conv = r.num(m, "conv", at);
+    if (r.err.empty()) r.require(s.heads % s.kv_heads == 0, at + ": kv_heads must divide heads");
+    s.unit = s.delta = s.norm = true;
+}
+void read_delta(Reader& r, const Value* m, const std::string& at, LayerSpec& L) {
+    L.mixer = MixerKind::Memory;
+    read_delta_sizes(r, m, at, L.mem);
+    L.mem.decay = MemDecay::PerHead;
+}
+// capped sink attention on the left, a delta memory with a decay per key channel on the right
+void read_side_by_side(Reader& r, const Value* m, const std::string& at, LayerSpec& L) {
+    L.mixer = MixerKind::SideBySide;
+    L.gqa_key = "left.";
+    L.mem_key = "right.";
+    GroupedAttnSpec& a = L.gqa;
+    const Value* l = r.obj(m, "left", at);
+    const std::string la = at + ".left";
+    a.heads = r.num(l, "heads", la);
+    a.kv_heads = r.num(l, "kv_heads", la);
+    a.dim = r.num(l, "dim", la);
+    a.vdim = r.num(l, "vdim", la);
+    a.scale = (float)r.real(l, "scale", la);
+    a.softcap = (float)r.real(l, "softcap", la);
+    read_rot(r, l, la, a.dim, a.rot);
+    a.sink = a.bias = a.qk_norm = true;
+    if (r.err.empty()) r.require(a.heads % a.kv_heads == 0, la + ": kv_heads must divide heads");
+    if (r.err.empty()) r.require(a.softcap > 0, la + ": softcap must be positive");
+    read_delta_sizes(r, r.obj(m, "right", at), at + ".right", L.mem);
+    L.mem.decay = MemDecay::PerChannel;
+    L.mem.gate = MemGate::Sigmoid;
+    L.mem.low_rank = true;
+    L.gqa_scale = (float)r.real(m, "left_scale", at);
+    L.mem_scale = (float)r.real(m, "right_scale", at);
+}
 struct MixerReader {
     const char* name;
     void (*read)(Reader&, const Value*, const std::string&, LayerSpec&);
 };
-const MixerReader kMixers[] = {{"latent_attention", read_latent_attention}, {"mamba2", read_mamba2}};
+using MixerTable = std::vector<MixerReader>;
+void read_mixer(Reader& r, const MixerTable& known, const Value* layer, const std::string& at, LayerSpec& L) {
+    const std::string type = r.str(layer, "type", at);
+    for (auto& mr : known)
+        if (type == mr.name) return mr.read(r, r.obj(layer, "mixer", at), at + ".mixer", L);
+    r.require(false, at + ": unknown mixer `" + type + "`");
+}
 
 void read_mlp(Reader& r, const Value* mlp, const std::string& at, const GateSpec& dense, float expert_alpha, LayerSpec& L) {
     if (!mlp || mlp->kind == Value::Null) {
@@ -110,10 +178,11 @@ void read_mlp(Reader& r, const Value* mlp, const std::string& at, const GateSpec
 
 // ---- Zukitar: latent attention and Mamba-2 layers, dense GELU and clipped-swish routed feed-forwards, tied head -----
 constexpr float kZukitarExpertAlpha = 1.702f;
-bool claims_zukitar(const Value& v) {
+bool names_architecture(const Value& v, const char* name) {
     const Value* a = v.get("architecture");
-    return a && a->kind == Value::String && a->str == "Zukitar";
+    return a && a->kind == Value::String && a->str == name;
 }
+bool claims_zukitar(const Value& v) { return names_architecture(v, "Zukitar"); }
 int32_t read_zukitar(const Value& v, ModelSpec& spec) {
     Reader r;
     spec.family = "Zukitar";
@@ -127,18 +196,51 @@ int32_t read_zukitar(const Value& v, ModelSpec& spec) {
         for (size_t i = 0; i < ls->arr.size(); i++) {
             const Value* lv = ls->arr[i].get();
             const std::string at = "layers[" + std::to_string(i) + "]";
-            const std::string type = r.str(lv, "type", at);
             LayerSpec L;
-            bool known = false;
-            for (auto& mr : kMixers)
-                if (type == mr.name) {
-                    mr.read(r, r.obj(lv, "mixer", at), at + ".mixer", L);
-                    known = true;
-                }
-            r.require(known, at + ": unknown mixer `" + type + "`");
+            read_mixer(r, {{"latent_attention", read_latent_attention}, {"mamba2", read_mamba2}}, lv, at, L);
             read_mlp(r, lv->get("mlp"), at + ".mlp", GateSpec{GateAct::GeluTanh, 0.f, 0.f}, kZukitarExpertAlpha, L);
             spec.layers.push_back(L);
         }
+    B2_REQUIRE(r.err.empty(), B2_ERR_CONFIG, r.err);
+    return B2_OK;
+}
+
+// ---- Tirezen: retention, delta memories, capped sink attention beside a delta memory; parallel layers with plain GELU
+// feed-forwards, norm weights around zero, a repeated stretch of layers, an output projection of its own -----------------
+bool claims_tirezen(const Value& v) { return names_architecture(v, "Tirezen"); }
+int32_t read_tirezen(const Value& v, ModelSpec& spec) {
+    Reader r;
+    spec.family = "Tirezen";
+    spec.vocab = r.num(&v, "vocab", "the model");
+    spec.width = r.num(&v, "width", "the model");
+    spec.eps = (float)r.real(r.obj(&v, "norm", "the model"), "eps", "norm");
+    spec.norm_offset = 1.f;
+    spec.own_head = true;
+    const Value* ls = v.get("layers");
+    r.require(ls && ls->kind == Value::Array && !ls->arr.empty(), "`layers` must be a non-empty list");
+    if (r.err.empty())
+        for (size_t i = 0; i < ls->arr.size(); i++) {
+            const Value* lv = ls->arr[i].get();
+            const std::string at = "layers[" + std::to_string(i) + "]";
+            LayerSpec L;
+            read_mixer(r, {{"retention", read_retention}, {"delta", read_delta}, {"parallel", read_side_by_side}}, lv, at, L);
+            L.parallel = true;
+            const Value* mlp = lv->get("mlp");
+            if (mlp && mlp->kind != Value::Null) {
+                const std::string kind = r.str(mlp, "kind", at + ".mlp");
+                r.require(kind == "dense", at + ".mlp: unknown feed-forward kind `" + kind + "`");
+                L.mlp = MlpKind::DensePlain;
+                L.ff = r.num(mlp, "ff", at + ".mlp");
+            }
+            spec.layers.push_back(L);
+        }
+    const Value* loop = v.get("loop");
+    if (loop && loop->kind != Value::Null) {
+        spec.loop.start = r.num(loop, "start", "loop", 0);
+        spec.loop.stop = r.num(loop, "stop", "loop", 0);
+        spec.loop.times = r.num(loop, "times", "loop", 1);
+        r.require(spec.loop.start < spec.loop.stop && spec.loop.stop <= (int)spec.layers.size(), "loop: start and stop must bound a stretch of the layers");
+    }
     B2_REQUIRE(r.err.empty(), B2_ERR_CONFIG, r.err);
     return B2_OK;
 }
@@ -150,7 +252,7 @@ struct ModelFamily {
     int32_t (*read_layers)(const Value& root, ModelSpec& spec);  // null: a flat b2_model_config family
 };
 bool claims_flat(const Value&) { return true; }  // b2_model_config_from_json decides (and refuses what it does not know)
-const ModelFamily kFamilies[] = {{"Zukitar", claims_zukitar, read_zukitar}, {"llama", claims_flat, nullptr}};
+const ModelFamily kFamilies[] = {{"Zukitar", claims_zukitar, read_zukitar}, {"Tirezen", claims_tirezen, read_tirezen}, {"llama", claims_flat, nullptr}};
 
 int32_t find_family(const char* json, b2json::ValuePtr& root, const ModelFamily** out) {
     std::string err;

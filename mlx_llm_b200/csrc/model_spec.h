@@ -6,8 +6,8 @@
 #include <string>
 #include <vector>
 
-enum class MixerKind { LatentAttention, Mamba2 };
-enum class MlpKind { None, DenseGated, Routed };
+enum class MixerKind { LatentAttention, Mamba2, GroupedAttention, Memory, SideBySide };
+enum class MlpKind { None, DenseGated, DensePlain, Routed };
 // act(gate, up) of a gated feed-forward:
 //   GeluTanh      gelu(gate) * up with the tanh form of gelu
 //   ClippedSwish  g = min(gate, limit), u = clamp(up, -limit, limit):  g * sigmoid(alpha * g) * (u + 1)
@@ -17,8 +17,9 @@ struct GateSpec {
     float limit = 0.f, alpha = 0.f;
 };
 
-// Rotation of consecutive pairs (2i, 2i+1), i < dims/2, by position * base^(-2i/dims); the rest passes unchanged.
-struct PairRotSpec {
+// Rotation of dims/2 pairs by position * base^(-2i/dims); the rest passes unchanged.  Which coordinates form pair i is the
+// mixer's: (2i, 2i+1) in latent attention, (i, i + dims/2) in grouped attention and in memories.
+struct RotSpec {
     double base = 10000.0;
     int dims = 0;
 };
@@ -27,7 +28,7 @@ struct PairRotSpec {
 struct LatentAttnSpec {
     int heads = 0, dim = 0, rot_dim = 0, vdim = 0, kv_rank = 0;
     float scale = 0.f;
-    PairRotSpec rot;
+    RotSpec rot;
     constexpr int row() const { return kv_rank + rot_dim; }               // values cached per token
     // ... padded for 16-wide tensor-core steps, and to one 64-wide load box at least
     constexpr int row_pad() const { return row() < 64 ? 64 : (row() + 15) / 16 * 16; }
@@ -40,6 +41,41 @@ struct Mamba2Spec {
     constexpr int channels() const { return inner() + 2 * groups * state; }  // x | B | C, the convolved inputs
     constexpr int in_rows() const { return inner() + channels() + heads; }   // z | x | B | C | dt
 };
+// Attention with kv_heads <= heads key / value heads, cached per token.  Keys and values may differ in size.
+struct GroupedAttnSpec {
+    int heads = 0, kv_heads = 0, dim = 0, vdim = 0;
+    float scale = 0.f;
+    float softcap = 0.f;  // score <- softcap * tanh(score / softcap); 0: no cap
+    bool sink = false;    // exp(0) is added to the softmax's denominator
+    bool bias = false;    // biases of the query, key and value projections
+    bool qk_norm = false; // RMS norm over the head of queries and keys, before the rotation
+    RotSpec rot;
+    constexpr int group() const { return heads / kv_heads; }
+    constexpr int k_row() const { return (dim + 15) / 16 * 16; }  // values per cached head row, zero-padded for 16-wide steps
+    constexpr int v_row() const { return (vdim + 15) / 16 * 16; }
+};
+// Linear memory: a state S [dim][vdim] per head in f32, read with the query after the token's own write,
+//     S <- decay * S;   S <- S + k u^T;   o = S^T q;   out = norm(o) * gate
+// u = v (delta off) or u = beta (v - S^T k) with the decayed S (delta on).
+enum class MemDecay { Fixed, PerHead, PerChannel };  // Fixed: constants; the others -exp(A_log) softplus(.. + dt_bias) in the exponent
+enum class MemGate { Silu, Sigmoid };
+struct MemorySpec {
+    int heads = 0, kv_heads = 0, dim = 0, vdim = 0;  // kv_heads: heads of q and k
+    int conv = 0;          // taps of the causal convolution (then silu) on q, k and v; 0: none
+    bool unit = false;     // q and k are unit vectors per head, q times dim^-1/2 (off: k times dim^-1/2)
+    float unit_eps = 1e-6f; // x / sqrt(sum x^2 + unit_eps)
+    bool delta = false;
+    bool norm = false;     // the output norm has a weight [vdim]
+    bool low_rank = false; // decay and gate come from two-factor projections
+    MemDecay decay = MemDecay::Fixed;
+    MemGate gate = MemGate::Silu;
+    RotSpec rot;           // dims 0: no rotation
+    constexpr int q_cols() const { return kv_heads * dim; }
+    constexpr int channels() const { return 2 * kv_heads * dim + heads * vdim; }  // q | k | v
+    constexpr int state_floats() const { return heads * dim * vdim; }
+    constexpr int keep() const { return conv > 1 ? conv - 1 : 0; }                 // inputs of the convolution kept between steps
+    constexpr int decays() const { return decay == MemDecay::PerChannel ? heads * dim : decay == MemDecay::PerHead ? heads : 0; }
+};
 // Routed experts: sigmoid scores, the best `top` experts, the score multiplies the expert's input.
 struct RoutedSpec {
     int experts = 0, top = 0, ff = 0;
@@ -49,20 +85,51 @@ struct LayerSpec {
     MixerKind mixer = MixerKind::LatentAttention;
     LatentAttnSpec attn;
     Mamba2Spec ssm;
+    GroupedAttnSpec gqa;              // GroupedAttention, SideBySide
+    MemorySpec mem;                   // Memory, SideBySide
+    std::vector<double> decay;        // MemDecay::Fixed: per head
+    float gqa_scale = 1.f, mem_scale = 1.f;
+    std::string gqa_key, mem_key;     // what their tensors' names have behind the mixer's prefix
+    // one norm: mixer and feed-forward both read it, and their sum is added to the stream (plain feed-forwards only)
+    bool parallel = false;
     MlpKind mlp = MlpKind::None;
-    int ff = 0;  // dense
+    int ff = 0;  // dense; DensePlain: down(gelu(up)), the exact gelu
     GateSpec gate;
     RoutedSpec moe;
+    bool has_gqa() const { return mixer == MixerKind::GroupedAttention || mixer == MixerKind::SideBySide; }
+    bool has_mem() const { return mixer == MixerKind::Memory || mixer == MixerKind::SideBySide; }
+};
+// Layers start .. stop-1 run `times` times in a row with the same weights, each pass with a cache and a state of its own.
+// Ahead of each pass a vector of its own is added to the stream, and, from the second on, the embedding output.
+struct LoopSpec {
+    int start = 0, stop = 0, times = 0;
+};
+struct LayerRun {
+    int layer, pass;   // pass -1 outside the loop
+    bool opens_pass;   // the first layer of its pass
 };
 // Tensor names of a family: the `i`-th layer's prefix and the few names outside the layers.
 struct TensorNames {
-    std::string embed = "embed", final_norm = "final.norm", layer = "l", norm1 = "norm1", norm2 = "norm2", mixer = "mix", mlp = "mlp";
+    std::string embed = "embed", final_norm = "final.norm", layer = "l", norm1 = "norm1", norm2 = "norm2", mixer = "mix", mlp = "mlp",
+                head = "head", loop_step = "loop.step";
     std::string layer_key(int i, const std::string& s) const { return layer + std::to_string(i) + "." + s; }
 };
 struct ModelSpec {
     std::string family;
     int vocab = 0, width = 0;
     float eps = 1e-5f, logit_scale = 1.f;
+    float norm_offset = 0.f;  // added to the stored weights of the layers' norms and the final norm
+    bool own_head = false;    // an output projection beside the embedding table
     std::vector<LayerSpec> layers;
+    LoopSpec loop;
     TensorNames names;
+    std::vector<LayerRun> runs() const {
+        std::vector<LayerRun> r;
+        const int n = (int)layers.size();
+        for (int i = 0; i < loop.start; i++) r.push_back({i, -1, false});
+        for (int t = 0; t < loop.times; t++)
+            for (int i = loop.start; i < loop.stop; i++) r.push_back({i, t, i == loop.start});
+        for (int i = loop.stop; i < n; i++) r.push_back({i, -1, false});
+        return r;
+    }
 };

@@ -1,5 +1,6 @@
 """Plain numpy restatement (float64) of decoders whose layers are listed one by one in config.json: latent attention,
-Mamba-2, dense gated and routed feed-forwards.  One function per mechanism, whole sequences only, no cache, no batching:
+Mamba-2, softmax attention with a cap and a sink, retention, the gated delta rule, two mixers side by side, dense (gated and
+plain) and routed feed-forwards, repeated layers.  One function per mechanism, whole sequences only, no cache, no batching:
 the yardstick of the layered models' tests.  Nothing here is shared with the library's own code path.
 
 Weights are a dict name -> float array; `cfg` is the parsed config.json.
@@ -44,6 +45,21 @@ def rotate_pairs(v, pos, base, dims):
         u, w = v[..., 2 * i], v[..., 2 * i + 1]
         out[..., 2 * i] = u * c - w * s
         out[..., 2 * i + 1] = w * c + u * s
+    return out
+
+
+def gelu_erf(x):
+    return 0.5 * x * (1.0 + np.vectorize(math.erf)(x / math.sqrt(2.0)))
+
+
+def rotate_halves(v, pos, base, dims):
+    """v [..., T, d]: coordinates (i, i + dims/2) for i < dims/2 turned by pos * base^(-2i/dims)."""
+    out = v.copy()
+    for i in range(dims // 2):
+        j = i + dims // 2
+        a = pos * base ** (-2.0 * i / dims)
+        out[..., i] = v[..., i] * np.cos(a) - v[..., j] * np.sin(a)
+        out[..., j] = v[..., j] * np.cos(a) + v[..., i] * np.sin(a)
     return out
 
 
@@ -104,7 +120,85 @@ def mamba2(h, g, m, eps):
     return gated_group_norm(y.reshape(T, inner), z, g("norm"), m["norm_groups"], eps) @ g("o").T
 
 
-MIXERS = {"latent_attention": latent_attention, "mamba2": mamba2}
+def sink_attention(h, g, m, eps):
+    """Grouped-query attention: biases, per-head norms of queries and keys, rotated halves, capped scores, and a softmax
+    whose denominator has one more term, exp(0)."""
+    T = h.shape[0]
+    H, G, D, V = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    pos = np.arange(T, dtype=F)
+    part = lambda n, heads, d: (h @ g(n).T + g(n + ".b")).reshape(T, heads, d).transpose(1, 0, 2)
+    turn = lambda v: rotate_halves(v, pos, m["rot"]["base"], m["rot"]["dims"])
+    q = turn(rms_norm(part("q", H, D), g("q.norm"), eps))
+    k = turn(rms_norm(part("k", G, D), g("k.norm"), eps))
+    v = part("v", G, V)
+    out = np.zeros((T, H, V), F)
+    for i in range(H):
+        s = q[i] @ k[i // (H // G)].T * m["scale"]
+        s = m["softcap"] * np.tanh(s / m["softcap"])
+        s = np.where(np.tril(np.ones((T, T), bool)), s, -np.inf)
+        top = np.maximum(s.max(-1, keepdims=True), 0.0)
+        e = np.exp(s - top)
+        out[:, i] = e / (np.exp(-top) + e.sum(-1, keepdims=True)) @ v[i // (H // G)]
+    return out.reshape(T, H * V) @ g("o").T
+
+
+def decayed_memory(q, k, v, log_decay, beta=None):
+    """One head, one token after the other: q, k [T, D], v [T, V], log_decay [T, D].  Without beta the memory adds k v^T;
+    with it, k u^T with u = beta (v - what the decayed memory answers to k).  The read-out sees the token's own write."""
+    S = np.zeros((k.shape[1], v.shape[1]), F)
+    out = np.zeros((k.shape[0], v.shape[1]), F)
+    for t in range(k.shape[0]):
+        S = np.exp(log_decay[t])[:, None] * S
+        u = v[t] if beta is None else beta[t] * (v[t] - S.T @ k[t])
+        S = S + np.outer(k[t], u)
+        out[t] = S.T @ q[t]
+    return out
+
+
+def retention(h, g, m, eps):
+    T = h.shape[0]
+    H, D, V = m["heads"], m["dim"], m["vdim"]
+    pos = np.arange(T, dtype=F)
+    turn = lambda v: rotate_halves(v.reshape(T, H, D).transpose(1, 0, 2), pos, m["rot"]["base"], m["rot"]["dims"])
+    q, k, v = turn(h @ g("q").T), turn(h @ g("k").T) * D ** -0.5, (h @ g("v").T).reshape(T, H, V)
+    o = np.stack([decayed_memory(q[i], k[i], v[:, i], np.full((T, D), math.log(m["decay"][i]))) for i in range(H)], 1)
+    return (rms(o, eps).reshape(T, H * V) * silu(h @ g("g").T)) @ g("o").T
+
+
+def unit(x):
+    return x / np.sqrt((x * x).sum(-1, keepdims=True) + 1e-6)
+
+
+def gated_delta(h, g, m, eps, per_channel=False):
+    """per_channel: a decay per head and key channel and a sigmoid output gate, both from low-rank projections; otherwise a
+    decay per head and a silu gate."""
+    T = h.shape[0]
+    H, G, D, V = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    conv = lambda n: causal_conv_silu(h @ g(n).T, g(n + ".conv"), 0.0)
+    q, k, v = unit(conv("q").reshape(T, G, D)) * D ** -0.5, unit(conv("k").reshape(T, G, D)), conv("v").reshape(T, H, V)
+    beta = sigmoid(h @ g("b").T)
+    if per_channel:
+        step = softplus(h @ g("a1").T @ g("a2").T + g("dt_bias")).reshape(T, H, D)
+        gate = sigmoid(h @ g("g1").T @ g("g2").T)
+    else:
+        step = np.repeat(softplus(h @ g("a").T + g("dt_bias"))[:, :, None], D, 2)
+        gate = silu(h @ g("g").T)
+    log_decay = -np.exp(g("A_log"))[:, None] * step
+    o = np.stack([decayed_memory(q[:, i // (H // G)], k[:, i // (H // G)], v[:, i], log_decay[:, i], beta[:, i]) for i in range(H)], 1)
+    return ((rms(o, eps) * g("norm")).reshape(T, H * V) * gate) @ g("o").T
+
+
+def side_by_side(h, g, m, eps):
+    left = sink_attention(h, lambda n: g("left." + n), m["left"], eps)
+    right = gated_delta(h, lambda n: g("right." + n), m["right"], eps, per_channel=True)
+    return m["left_scale"] * left + m["right_scale"] * right
+
+
+MIXERS = {"latent_attention": latent_attention, "mamba2": mamba2, "retention": retention, "delta": gated_delta, "parallel": side_by_side}
+
+
+def plain_ff(h, g):
+    return gelu_erf(h @ g("up").T) @ g("down").T
 
 
 def dense_ff(h, g):
@@ -127,8 +221,40 @@ def routed_ff(h, g, mlp):
     return out
 
 
+def layer_runs(cfg):
+    """(layer, pass) in the order they run; pass is -1 outside the repeated stretch."""
+    n, loop = len(cfg["layers"]), cfg.get("loop") or dict(start=0, stop=0, times=0)
+    a, b = loop["start"], loop["stop"]
+    return [(i, -1) for i in range(a)] + [(i, t) for t in range(loop["times"]) for i in range(a, b)] + [(i, -1) for i in range(b, n)]
+
+
 def forward(cfg, w, tokens, layers_out=None):
-    """Logits [T, vocab] of one sequence.  layers_out (a list) receives the residual stream after every layer."""
+    """Logits [T, vocab] of one sequence.  layers_out (a list) receives the residual stream after every layer run."""
+    return (forward_tirezen if cfg["architecture"] == "Tirezen" else forward_zukitar)(cfg, w, tokens, layers_out)
+
+
+def forward_tirezen(cfg, w, tokens, layers_out=None):
+    """Parallel layers (one norm, mixer and feed-forward both read it), norm weights around zero, a stretch of layers that runs
+    several times, an output projection of its own."""
+    eps = cfg["norm"]["eps"]
+    first = w["embed"][np.asarray(tokens)].astype(F)
+    x = first
+    for i, t in layer_runs(cfg):
+        L = cfg["layers"][i]
+        if t >= 0 and i == cfg["loop"]["start"]:
+            x = x + w["loop.step"][t] + (first if t > 0 else 0.0)
+        mix = lambda n, i=i: w[f"l{i}.mix.{n}"]
+        h = rms_norm(x, 1.0 + w[f"l{i}.norm1"], eps)
+        y = MIXERS[L["type"]](h, mix, L["mixer"], eps)
+        if L.get("mlp"):
+            y = y + plain_ff(h, lambda n, i=i: w[f"l{i}.mlp.{n}"])
+        x = x + y
+        if layers_out is not None:
+            layers_out.append(x.copy())
+    return rms_norm(x, 1.0 + w["final.norm"], eps) @ w["head"].T
+
+
+def forward_zukitar(cfg, w, tokens, layers_out=None):
     eps = cfg["norm"]["eps"]
     x = w["embed"][np.asarray(tokens)].astype(F)
     for i, L in enumerate(cfg["layers"]):
