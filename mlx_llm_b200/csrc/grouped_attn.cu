@@ -1,0 +1,160 @@
+// Grouped-query attention of the layered models: projections to rotated queries and cache rows, and the plain form of the
+// attention.  Scores may be capped, the softmax may have a sink (exp(0) in its denominator, with no value).
+#include "elt.cuh"
+#include "layer_kernels.h"
+
+namespace {
+
+constexpr int kMaxHead = 256;
+
+// A warp per (token, head of q, k or v): bias, norm over the head, rotation of the pairs (i, i + dims/2), store.  A lane holds
+// VEC consecutive values of every 32 * VEC; the rotation finds its partner in shared memory.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) gqa_prep_kernel(const GroupedAttnSpec a, const GqaPrepParams p) {
+    asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
+    pdl_wait();
+    __shared__ __align__(16) float rows[8][kMaxHead];
+    constexpr int N = kMaxHead / (32 * VEC);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, units = a.heads + 2 * a.kv_heads;
+    const int id = blockIdx.x * 8 + warp, t = id / units, u = id - t * units;
+    if (t >= p.T) return;
+    const int kind = u < a.heads ? 0 : u < a.heads + a.kv_heads ? 1 : 2, h = kind == 0 ? u : kind == 1 ? u - a.heads : u - a.heads - a.kv_heads;
+    const int n = kind == 2 ? a.vdim : a.dim, padded = kind == 2 ? a.v_row() : a.k_row(), dims = kind == 2 ? 0 : a.rot.dims, half = dims / 2;
+    const T* src = reinterpret_cast<const T*>(p.in) + (size_t)t * p.ld + (kind == 0 ? p.q_off : kind == 1 ? p.k_off : p.v_off) + h * n;
+    const float* bias = kind == 0 ? p.q_bias : kind == 1 ? p.k_bias : p.v_bias;
+    const float* w = kind == 0 ? p.q_norm : kind == 1 ? p.k_norm : nullptr;
+    const int slot = p.slot_mapping[t];
+    T* dst;
+    if (kind == 0) {
+        dst = reinterpret_cast<T*>(p.q) + ((size_t)t * a.heads + h) * padded;
+    } else {
+        if (slot < 0) return;
+        const size_t row = ((size_t)(slot / p.page_size) * a.kv_heads + h) * p.page_size + slot % p.page_size;
+        dst = reinterpret_cast<T*>(kind == 1 ? p.k_cache : p.v_cache) + row * padded;
+    }
+    float v[N][VEC], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < N; i++) {
+        const int d = (i * 32 + lane) * VEC;
+#pragma unroll
+        for (int e = 0; e < VEC; e++) v[i][e] = 0.f;
+        if (d >= n) continue;
+        if constexpr (VEC == 4)
+            Elt<T>::ld4(src + d, v[i]);
+        else
+            v[i][0] = Elt<T>::ld(src + d);
+#pragma unroll
+        for (int e = 0; e < VEC; e++) {
+            if (bias) v[i][e] += bias[h * n + d + e];
+            ss += v[i][e] * v[i][e];
+        }
+    }
+    if (w) {
+        const float inv = 1.0f / sqrtf(elt_warp_sum(ss) / (float)n + p.eps);
+#pragma unroll
+        for (int i = 0; i < N; i++)
+#pragma unroll
+            for (int e = 0; e < VEC; e++) {
+                const int d = (i * 32 + lane) * VEC + e;
+                if (d < n) v[i][e] = v[i][e] * inv * w[d];
+            }
+    }
+    if (half > 0) {
+        const float* ct = p.cos_t + (size_t)p.positions[t] * half;
+        const float* st = p.sin_t + (size_t)p.positions[t] * half;
+#pragma unroll
+        for (int i = 0; i < N; i++)
+#pragma unroll
+            for (int e = 0; e < VEC; e++) rows[warp][(i * 32 + lane) * VEC + e] = v[i][e];
+        __syncwarp();
+#pragma unroll
+        for (int i = 0; i < N; i++)
+#pragma unroll
+            for (int e = 0; e < VEC; e++) {
+                const int d = (i * 32 + lane) * VEC + e;
+                if (d < half)
+                    v[i][e] = v[i][e] * ct[d] - rows[warp][d + half] * st[d];
+                else if (d < dims)
+                    v[i][e] = v[i][e] * ct[d - half] + rows[warp][d - half] * st[d - half];
+            }
+    }
+#pragma unroll
+    for (int i = 0; i < N; i++) {
+        const int d = (i * 32 + lane) * VEC;
+        if (d >= padded) continue;
+        if constexpr (VEC == 4)
+            Elt<T>::st4(dst + d, v[i]);
+        else
+            Elt<T>::st(dst + d, v[i][0]);
+    }
+}
+
+// Plain form: one block per (token, head), 128 keys at a time with an online softmax, everything f32.
+template <typename T>
+__global__ void __launch_bounds__(128) gqa_simple_kernel(const GroupedAttnSpec a, const GqaAttnParams p) {
+    pdl_wait();
+    __shared__ float q[kMaxHead], acc[kMaxHead], pr[128], red[33];
+    const int t = blockIdx.x, h = blockIdx.y, g = h / a.group(), KR = a.k_row(), VR = a.v_row(), ps = p.page_size;
+    const int n = p.positions[t] + 1;
+    const int32_t* bt = p.block_tables + (size_t)p.seq_slot[p.token_seq[t]] * p.max_blocks;
+    const T* qr = reinterpret_cast<const T*>(p.q) + ((size_t)t * a.heads + h) * KR;
+    auto row = [&](int j) { return ((size_t)bt[j / ps] * a.kv_heads + g) * ps + j % ps; };
+    for (int i = threadIdx.x; i < KR; i += 128) q[i] = Elt<T>::ld(qr + i);
+    for (int i = threadIdx.x; i < VR; i += 128) acc[i] = 0.f;
+    float m = -INFINITY, l = 0.f;
+    __syncthreads();
+    for (int j0 = 0; j0 < n; j0 += 128) {
+        const int j = j0 + threadIdx.x, cnt = min(128, n - j0);
+        float s = -INFINITY;
+        if (j < n) {
+            const T* k = reinterpret_cast<const T*>(p.k_cache) + row(j) * KR;
+            float d = 0.f;
+            for (int i = 0; i < KR; i += 8) {
+                float v[8];
+                Elt<T>::ld8(k + i, v);
+#pragma unroll
+                for (int e = 0; e < 8; e++) d = fmaf(q[i + e], v[e], d);
+            }
+            s = d * a.scale;
+            if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
+        }
+        float mx = elt_warp_max(s);
+        __syncthreads();
+        if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = mx;
+        __syncthreads();
+        mx = fmaxf(fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3])), m);
+        const float alpha = expf(m - mx), e = j < n ? expf(s - mx) : 0.f;
+        pr[threadIdx.x] = e;
+        l = l * alpha + elt_block_sum(e, red);
+        m = mx;
+        for (int i = threadIdx.x; i < VR; i += 128) {
+            float v = acc[i] * alpha;
+            for (int jj = 0; jj < cnt; jj++) v = fmaf(pr[jj], Elt<T>::ld(reinterpret_cast<const T*>(p.v_cache) + row(j0 + jj) * VR + i), v);
+            acc[i] = v;
+        }
+        __syncthreads();
+    }
+    if (a.sink) l += expf(-m);
+    T* o = reinterpret_cast<T*>(p.out) + (size_t)t * p.ldo + h * a.vdim;
+    for (int i = threadIdx.x; i < a.vdim; i += 128) Elt<T>::st(o + i, acc[i] / l * p.out_scale);
+}
+
+}  // namespace
+
+int32_t b2_gqa_prep_launch(b2_ctx* ctx, bool f32, const GroupedAttnSpec& a, const GqaPrepParams& p) {
+    if (p.T <= 0) return B2_OK;
+    B2_REQUIRE(a.dim <= kMaxHead && a.vdim <= kMaxHead, B2_ERR_UNSUPPORTED, "grouped attention: head sizes up to 256");
+    const bool vec = a.dim % 4 == 0 && a.vdim % 4 == 0 && p.q_off % 4 == 0 && p.k_off % 4 == 0 && p.v_off % 4 == 0 && p.ld % 4 == 0;
+    const dim3 grid((unsigned)(((size_t)p.T * (a.heads + 2 * a.kv_heads) + 7) / 8));
+    auto k = f32 ? (vec ? gqa_prep_kernel<float, 4> : gqa_prep_kernel<float, 1>) : (vec ? gqa_prep_kernel<uint16_t, 4> : gqa_prep_kernel<uint16_t, 1>);
+    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, k, grid, dim3(256), 0, ctx->stream, a, p));
+    B2_LAUNCHED(ctx);
+    return B2_OK;
+}
+int32_t b2_gqa_simple_launch(b2_ctx* ctx, bool f32, const GroupedAttnSpec& a, const GqaAttnParams& p) {
+    if (p.T <= 0) return B2_OK;
+    B2_REQUIRE(a.dim <= kMaxHead && a.vdim <= kMaxHead, B2_ERR_UNSUPPORTED, "grouped attention: head sizes up to 256");
+    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, f32 ? gqa_simple_kernel<float> : gqa_simple_kernel<uint16_t>, dim3(p.T, a.heads), dim3(128), 0, ctx->stream, a, p));
+    B2_LAUNCHED(ctx);
+    return B2_OK;
+}

@@ -17,6 +17,10 @@ struct AddNormParams {
     const float* y;         // what the last sub-layer added (f32), null: nothing
     const int32_t* y_rows;  // [T, n_src] rows of y summed (in order) into token t; null: row t
     const float* w;         // norm weight [width]; null: only the addition
+    const float* vec;       // [width] added to every row as well; null: nothing
+    const void* table;      // ... and row ids[t] of this table (the embedding); null: nothing
+    const int32_t* ids;
+    int ld_table, vocab;
     const int32_t* row_idx; // output row r takes source row row_idx[r]; null: r
     void* out;              // [rows, ldo], zero beyond width
     int ldx, ldy, ldo, rows, width, n_src;
@@ -150,6 +154,96 @@ struct LatentPrefillParams {
 };
 bool b2_latent_prefill_eligible(const LatentAttnSpec& a);
 int32_t b2_latent_prefill_launch(b2_ctx* ctx, const LatentAttnSpec& a, const LatentPrefillParams& p, int grid_work);
+
+// ---- grouped_attn.cu, grouped_attn_decode.cu, grouped_attn_prefill.cu --------------------------------------------------
+// Cache of a layer: keys [page][kv_heads][page_size][k_row], values [page][kv_heads][page_size][v_row].
+struct GqaPrepParams {
+    const void* in;         // [T, ld] projections: queries from q_off, keys from k_off, values from v_off, heads tight
+    int ld, q_off, k_off, v_off, T;
+    const float *q_bias, *k_bias, *v_bias;  // null: none
+    const float *q_norm, *k_norm;           // null: none
+    float eps;
+    const int32_t *positions, *slot_mapping;
+    const float *cos_t, *sin_t;  // [positions, rot.dims / 2]
+    void* q;                // [T, heads, k_row]
+    void *k_cache, *v_cache;
+    int page_size;
+};
+int32_t b2_gqa_prep_launch(b2_ctx* ctx, bool f32, const GroupedAttnSpec& a, const GqaPrepParams& p);
+struct GqaAttnParams {
+    const void* q;
+    const void *k_cache, *v_cache;
+    const int32_t* block_tables;
+    int max_blocks, page_size;
+    int64_t max_pages;
+    int T;                       // rows of q in use
+    // every token by itself: its sequence and position
+    const int32_t *positions, *token_seq, *seq_slot;
+    // the packer's decode list (context, token row, block-table row) and its work items (row, chunk)
+    const int32_t *dec_ctx, *dec_qrow, *dec_slot, *work_seq, *work_chunk, *work_off, *n_dec_work;
+    int chunk_tiles;             // 16-key tiles per work item
+    float *part_o, *part_ml;     // [work item][head][v_row], [work item][head][2]
+    int* counters;               // [decode rows][head blocks], zero between launches
+    // the packer's prefill list (sequence, first query), 128 queries per item
+    const int32_t *pf_seq, *pf_qstart, *n_pf_work, *cu_seqlens, *context_lens;
+    int q_rows;                  // rows of the q allocation
+    float out_scale;
+    void* out;                   // [T, ldo]: heads * vdim columns
+    int ldo;
+};
+int32_t b2_gqa_simple_launch(b2_ctx* ctx, bool f32, const GroupedAttnSpec& a, const GqaAttnParams& p);
+bool b2_gqa_decode_eligible(const GroupedAttnSpec& a);
+int b2_gqa_head_blocks(const GroupedAttnSpec& a);  // blocks of up to eight query heads that share a key / value head
+// items > 0: the decode list; items == 0: every token of the step is a row of its own
+int32_t b2_gqa_decode_launch(b2_ctx* ctx, const GroupedAttnSpec& a, const GqaAttnParams& p, int items);
+bool b2_gqa_prefill_eligible(const GroupedAttnSpec& a);
+int32_t b2_gqa_prefill_launch(b2_ctx* ctx, const GroupedAttnSpec& a, const GqaAttnParams& p, int grid_work);
+
+// ---- memory.cu, memory_chunk.cu ------------------------------------------------------------------------------------
+struct MemoryParams {
+    const void* in;         // [T, ld] projections
+    int ld, c_off, b_off;   // columns of q | k | v and of the step sizes' inputs
+    const void* dec;        // [T, ld_dec] decay inputs (decays() columns); null for fixed decays
+    int ld_dec;
+    int T, B;
+    const int32_t *cu_seqlens, *context_lens, *token_seq, *seq_slot, *positions;
+    float* state;           // slot s: state + s * slot_stride: [heads][vdim][dim], then [conv - 1][channels] inputs, oldest first
+    int64_t slot_stride;
+    const float *conv_w;    // [taps][channels]
+    const float *dt_bias, *A_log;
+    const float *decay, *log_decay;  // fixed decays [heads]
+    const float *cos_t, *sin_t;
+    // prepared inputs of the recurrence
+    float *q, *k;           // [T, q_cols]
+    const void* v;          // [T, ld_v]
+    int ld_v;
+    float *lg, *beta;       // [T, decays()] logarithms of the decays; [T, heads]
+    float* o;               // [T, heads * vdim]
+    void* chunk;            // scratch of the chunked form, b2_memory_chunk_bytes(T)
+    int max_n;              // longest portion of the step
+    bool chunked;           // set by the launcher: longer portions belong to the chunked form
+};
+int32_t b2_memory_launch(b2_ctx* ctx, bool f32, const MemorySpec& s, const MemoryParams& p);
+constexpr int kMemoryChunkMin = 12;  // shortest portion that the chunked form takes
+bool b2_memory_chunk_eligible(const MemorySpec& s);
+size_t b2_memory_chunk_bytes(const MemorySpec& s, size_t tokens);
+int32_t b2_memory_chunk_launch(b2_ctx* ctx, const MemorySpec& s, const MemoryParams& p);
+// Input row of a layer's output projection: attention heads (already there), memory heads (norm, gate), feed-forward (gelu);
+// everything else zero.
+struct BranchOutParams {
+    void* out;              // [T, ldo]
+    int ldo, T, att_cols;
+    const float* o;         // memory: [T, heads * vdim]; null: none
+    int heads, vdim, m_off;
+    const void* gate;
+    int ld_gate;
+    MemGate act;
+    const float* norm;      // [vdim]; null: none
+    float eps, scale;
+    const void* up;         // feed-forward: [T, ld_up]; null: none
+    int ld_up, ff, f_off;
+};
+int32_t b2_branch_out_launch(b2_ctx* ctx, bool f32, const BranchOutParams& p);
 
 // ---- ssm.cu ---------------------------------------------------------------------------------------------------------
 struct SsmParams {

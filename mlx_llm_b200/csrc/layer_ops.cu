@@ -24,6 +24,8 @@ __global__ void add_norm_kernel(const AddNormParams p) {
     __shared__ float red[33];
     const int r = blockIdx.x, t = p.row_idx ? p.row_idx[r] : r;
     float* xr = p.x + (size_t)t * p.ldx;
+    const T* emb = nullptr;
+    if (p.table) emb = reinterpret_cast<const T*>(p.table) + (size_t)min(max(p.ids[t], 0), p.vocab - 1) * p.ld_table;
     float ss = 0.f;
     const bool vec = p.width % 4 == 0 && p.ldx % 4 == 0 && p.ldy % 4 == 0;
     if (vec) {
@@ -34,6 +36,15 @@ __global__ void add_norm_kernel(const AddNormParams p) {
                 const float4 a = *reinterpret_cast<const float4*>(p.y + (size_t)yr * p.ldy + i);
                 v.x += a.x, v.y += a.y, v.z += a.z, v.w += a.w;
             }
+            if (p.vec) {
+                const float4 a = *reinterpret_cast<const float4*>(p.vec + i);
+                v.x += a.x, v.y += a.y, v.z += a.z, v.w += a.w;
+            }
+            if (emb) {
+                float a[4];
+                Elt<T>::ld4(emb + i, a);
+                v.x += a[0], v.y += a[1], v.z += a[2], v.w += a[3];
+            }
             if (p.write_x) *reinterpret_cast<float4*>(xr + i) = v;
             *reinterpret_cast<float4*>(row + i) = v;
             ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
@@ -42,6 +53,8 @@ __global__ void add_norm_kernel(const AddNormParams p) {
         for (int i = threadIdx.x; i < p.width; i += blockDim.x) {
             float v = xr[i];
             for (int k = 0; k < p.n_src; k++) v += p.y[(size_t)(p.y_rows ? p.y_rows[(size_t)t * p.n_src + k] : t) * p.ldy + i];
+            if (p.vec) v += p.vec[i];
+            if (emb) v += Elt<T>::ld(emb + i);
             if (p.write_x) xr[i] = v;
             row[i] = v;
             ss += v * v;

@@ -1,0 +1,20 @@
+// Shared by the memory kernels: the convolution's kept inputs.
+#pragma once
+#include "elt.cuh"
+#include "layer_kernels.h"
+
+// Leaves the last taps - 1 inputs of sequence b's convolution in its record.  The `blocks` blocks that work on the sequence
+// share the channels.
+template <typename T>
+__device__ __forceinline__ void memory_keep_inputs(const MemorySpec& s, const MemoryParams& p, int b, int block, int blocks) {
+    const int keep = s.keep(), C = s.channels(), start = p.cu_seqlens[b], n = p.cu_seqlens[b + 1] - start, before = p.context_lens[b] - n;
+    if (keep == 0) return;
+    for (int ch = block * (int)blockDim.x + (int)threadIdx.x; ch < C; ch += blocks * (int)blockDim.x) {
+        float* c = p.state + (size_t)p.seq_slot[b] * p.slot_stride + s.state_floats() + ch;
+        const T* u = reinterpret_cast<const T*>(p.in) + p.c_off + ch;
+        for (int j = 0; j < keep; j++) {  // ascending: a shift reads places it has not overwritten yet
+            const int k = n - keep + j;
+            c[(size_t)j * C] = k >= 0 ? Elt<T>::ld(u + (size_t)(start + k) * p.ld) : (before > 0 ? c[(size_t)(j + n) * C] : 0.f);
+        }
+    }
+}
