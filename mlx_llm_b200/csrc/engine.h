@@ -216,6 +216,7 @@ struct LayeredStep {
     const int32_t* ids_dev;
     int T, B, n_dec, dec_work, pf_work, chunk_tiles, max_ctx;
     long dec_ctx_sum;
+    int max_n;                  // longest portion
     double pf_pairs;  // (query, visible key) pairs of the prefilling sequences
     int pf_ctx;                 // their contexts (this step's tokens included), summed
     const int32_t* pf_kv_off;   // [B] device: running sum of those contexts, -1 for sequences with a single token
@@ -225,4 +226,5 @@ struct LayeredStep {
 int32_t b2_forward_layered(b2_model* m, b2_pool* pool, const LayeredStep& s, float** logits_dev, int* logits_ld);
 int b2_layered_q_tile(const b2_model* m);
 int b2_layered_chunk_tiles(const b2_model* m, const std::vector<SeqStep>& seqs);  // 16-key tiles per work item of the decode attention
+int b2_small_cta_chunk_tiles(long dec_ctx_sum, int blocks, int sm_count);  // ... for kernels with several CTAs per SM and `blocks` CTAs per item
 bool b2_tensor_to_f32(const HostTensor& t, std::vector<float>& out);

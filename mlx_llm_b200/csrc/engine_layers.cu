@@ -33,10 +33,20 @@ struct LayerP {
     // mamba2
     Proj ssm_in, ssm_o;
     float *conv_w = nullptr, *conv_b = nullptr, *dt_bias = nullptr, *A_log = nullptr, *D = nullptr, *ssm_norm = nullptr;
-    int64_t state_off = 0;  // floats into the slot's record
     // feed-forward
     Proj gu, down, router;
     GroupW e_gu, e_down;
+    // Layers of grouped attention and memories: one product for everything that reads the normed stream, one for everything
+    // that is added to it (columns: attention heads | memory heads | feed-forward).
+    Proj in, lr, out;  // lr: the second factors of a memory's decay and gate, block-diagonal
+    struct {
+        int q = 0, k = 0, v = 0, c = 0, gate = 0, beta = 0, decay = 0, up = 0;  // columns of `in`
+        int lr_gate = 0;                                                       // columns of `lr`: decay from 0, gate
+        int m = 0, f = 0;                                                      // columns of the row `out` reads
+    } at;
+    float *q_bias = nullptr, *k_bias = nullptr, *v_bias = nullptr, *q_norm = nullptr, *k_norm = nullptr, *mem_norm = nullptr;
+    float *decay = nullptr, *log_decay = nullptr;
+    int mem_rope = -1;
 };
 struct RopeTab {
     RotSpec spec;
@@ -48,7 +58,11 @@ struct RopeTab {
 struct LayeredModel {
     ModelSpec spec;
     std::vector<LayerP> layers;
-    void* embed = nullptr;  // [pad_n(vocab), pad_k(width)]: embedding table and output projection
+    std::vector<LayerRun> runs;
+    std::vector<int64_t> run_state;  // floats into the slot's record, per run of a layer
+    void* embed = nullptr;  // [pad_n(vocab), pad_k(width)]: embedding table, and output projection unless the model has one
+    void* head = nullptr;
+    float* loop_step = nullptr;  // [times][width]
     float* final_norm = nullptr;
     std::vector<RopeTab> ropes;
     int rope_positions = 0;
@@ -59,7 +73,7 @@ struct LayeredModel {
     int kv_cap = 0, kv_ld_lat = 0, kv_ld_rot = 0, kv_ld_exp = 0;  // rows; widest rows over the layers
     // decode attention: partial results per work item
     float* dec_part = nullptr;
-    size_t dec_part_floats = 0, dec_part_row = 0;  // capacity; heads * (kv_rank + 2) of the largest layer
+    size_t dec_part_floats = 0, dec_part_row = 0;  // capacity; heads * (values + 2) of the largest layer
     uint8_t* arena = nullptr;
     int t_cap = 0, l_cap = 0;
     float* capture = nullptr;
@@ -165,12 +179,14 @@ struct Filler {
         return B2_OK;
     }
     // a small tensor kept in f32, as stored or (two dimensions) transposed
-    int32_t vec(float*& dst, const std::string& key, std::vector<int64_t> shape, float mean, float sd, bool transpose = false) {
+    int32_t vec(float*& dst, const std::string& key, std::vector<int64_t> shape, float mean, float sd, bool transpose = false, float offset = 0.f) {
         int64_t n = 1;
         for (auto d : shape) n *= d;
         B2_CHECK(alloc((size_t)n * 4, (void**)&dst));
         if (!w) return random(dst, true, 1, (int)n, (int)n, mean, sd);
         B2_CHECK(fetch(key, shape));
+        if (offset != 0.f)
+            for (float& v : host) v += offset;
         if (transpose) {
             const std::vector<float> a = host;
             for (int64_t r = 0; r < shape[0]; r++)
@@ -179,6 +195,30 @@ struct Filler {
         B2_CUDA(cudaMemcpyAsync(dst, host.data(), (size_t)n * 4, cudaMemcpyHostToDevice, m->ctx->stream));
         B2_CUDA(cudaStreamSynchronize(m->ctx->stream));
         return B2_OK;
+    }
+    int32_t upload(float*& dst, const std::vector<float>& v) {
+        B2_CHECK(alloc(v.size() * 4, (void**)&dst));
+        B2_CUDA(cudaMemcpyAsync(dst, v.data(), v.size() * 4, cudaMemcpyHostToDevice, m->ctx->stream));
+        B2_CUDA(cudaStreamSynchronize(m->ctx->stream));
+        return B2_OK;
+    }
+    // first dimension of a two-dimensional tensor whose size only its shape tells; `fallback` for random weights
+    int32_t rows_of(const std::string& name, int fallback, int* out) {
+        *out = fallback;
+        if (!w) return B2_OK;
+        const std::string key = prefix.empty() ? name : prefix + "." + name;
+        auto it = w->t.find(key);
+        B2_REQUIRE(it != w->t.end(), B2_ERR_MISSING_TENSOR, "missing tensor `" + key + "`");
+        B2_REQUIRE(it->second.shape.size() == 2 && it->second.shape[0] > 0, B2_ERR_CONFIG, "tensor `" + key + "` is not a matrix");
+        *out = (int)it->second.shape[0];
+        return B2_OK;
+    }
+    // tensor [rows, cols] to the block of p at (row0, col0)
+    int32_t block(Proj& p, int row0, int col0, const std::string& key, int rows, int cols) {
+        void* dst = at(p.w, (int64_t)row0 * p.K + col0);
+        if (!w) return random(dst, m->f32, rows, cols, p.K, 0.f, 1.0f / sqrtf((float)cols));
+        B2_CHECK(fetch(key, {rows, cols}));
+        return put(host.data(), rows, cols, dst, p.K);
     }
     int32_t group(GroupW& g, int G, int N, int K) {
         g.G = G;
@@ -212,6 +252,133 @@ struct Filler {
     }
 };
 
+int rope_table(LayeredModel& lm, const RotSpec& rot) {
+    for (size_t r = 0; r < lm.ropes.size(); r++)
+        if (lm.ropes[r].spec.base == rot.base && lm.ropes[r].spec.dims == rot.dims) return (int)r;
+    lm.ropes.push_back(RopeTab{rot});
+    return (int)lm.ropes.size() - 1;
+}
+
+// Grouped attention, memories, and in parallel layers the feed-forward: one matrix in, one matrix out.
+int32_t load_branches(Filler& f, LayeredModel& lm, int i) {
+    const LayerSpec& L = lm.spec.layers[i];
+    const TensorNames& tn = lm.spec.names;
+    LayerP& P = lm.layers[i];
+    const int W = lm.spec.width;
+    const GroupedAttnSpec& a = L.gqa;
+    const MemorySpec& s = L.mem;
+    auto aq = [&](const std::string& n) { return tn.layer_key(i, tn.mixer + "." + L.gqa_key + n); };
+    auto am = [&](const std::string& n) { return tn.layer_key(i, tn.mixer + "." + L.mem_key + n); };
+    const bool ff = L.parallel && L.mlp == MlpKind::DensePlain;
+    B2_REQUIRE(L.mlp == MlpKind::None || L.parallel == (L.mlp == MlpKind::DensePlain), B2_ERR_UNSUPPORTED,
+               "plain feed-forwards belong to parallel layers, gated and routed ones to sequential layers");
+    int n = 0, ra = 0, rg = 0, ra8 = 0, need = 0;
+    auto take = [&](int& at, int cols) {
+        at = n;
+        n += up(cols, 8);
+    };
+    if (L.has_gqa()) {
+        B2_REQUIRE(a.dim <= 256 && a.vdim <= 256, B2_ERR_UNSUPPORTED, "grouped attention: head sizes up to 256");
+        take(P.at.q, a.heads * a.dim);
+        take(P.at.k, a.kv_heads * a.dim);
+        take(P.at.v, a.kv_heads * a.vdim);
+    }
+    if (L.has_mem()) {
+        B2_REQUIRE(s.dim <= 256, B2_ERR_UNSUPPORTED, "memory: key sizes up to 256");
+        take(P.at.c, s.channels());
+        if (s.low_rank) {
+            const int r = std::max(8, std::min(s.dim, s.vdim));  // for random weights
+            B2_CHECK(f.rows_of(am("a1"), r, &ra));
+            B2_CHECK(f.rows_of(am("g1"), r, &rg));
+            ra8 = up(ra, 8);
+            take(P.at.gate, ra8 + rg);
+            need = P.at.gate + pad_k(ra8 + rg);  // the second factors' product reads whole slabs
+        } else {
+            take(P.at.gate, s.heads * s.vdim);
+            if (s.decay == MemDecay::PerHead) take(P.at.decay, s.heads);
+        }
+        if (s.delta) take(P.at.beta, s.heads);
+    }
+    if (ff) take(P.at.up, L.ff);
+    B2_CHECK(f.proj(P.in, std::max(n, need), W));
+    if (L.has_gqa()) {
+        B2_CHECK(f.rows(P.in, P.at.q, aq("q"), a.heads * a.dim, W));
+        B2_CHECK(f.rows(P.in, P.at.k, aq("k"), a.kv_heads * a.dim, W));
+        B2_CHECK(f.rows(P.in, P.at.v, aq("v"), a.kv_heads * a.vdim, W));
+        if (a.bias) {
+            B2_CHECK(f.vec(P.q_bias, aq("q.b"), {a.heads * a.dim}, 0.f, 0.1f));
+            B2_CHECK(f.vec(P.k_bias, aq("k.b"), {a.kv_heads * a.dim}, 0.f, 0.1f));
+            B2_CHECK(f.vec(P.v_bias, aq("v.b"), {a.kv_heads * a.vdim}, 0.f, 0.1f));
+        }
+        if (a.qk_norm) {
+            B2_CHECK(f.vec(P.q_norm, aq("q.norm"), {a.dim}, 1.f, 0.f));
+            B2_CHECK(f.vec(P.k_norm, aq("k.norm"), {a.dim}, 1.f, 0.f));
+        }
+        P.rope = rope_table(lm, a.rot);
+        lm.dec_part_row = std::max(lm.dec_part_row, (size_t)a.heads * (a.v_row() + 2));
+    }
+    if (L.has_mem()) {
+        const int Q = s.q_cols(), V = s.heads * s.vdim;
+        B2_CHECK(f.rows(P.in, P.at.c, am("q"), Q, W));
+        B2_CHECK(f.rows(P.in, P.at.c + Q, am("k"), Q, W));
+        B2_CHECK(f.rows(P.in, P.at.c + 2 * Q, am("v"), V, W));
+        if (s.conv > 0) {  // [taps][channels], the channels of q, k and v side by side
+            std::vector<float> all((size_t)s.conv * s.channels());
+            int c0 = 0;
+            for (auto& part : {std::pair<const char*, int>{"q.conv", Q}, {"k.conv", Q}, {"v.conv", V}}) {
+                if (f.w) {
+                    B2_CHECK(f.fetch(am(part.first), {part.second, s.conv}));
+                    for (int c = 0; c < part.second; c++)
+                        for (int j = 0; j < s.conv; j++) all[(size_t)j * s.channels() + c0 + c] = f.host[(size_t)c * s.conv + j];
+                }
+                c0 += part.second;
+            }
+            if (f.w)
+                B2_CHECK(f.upload(P.conv_w, all));
+            else
+                B2_CHECK(f.vec(P.conv_w, "", {s.conv, s.channels()}, 0.f, 0.5f));
+        }
+        if (s.low_rank) {
+            B2_CHECK(f.rows(P.in, P.at.gate, am("a1"), ra, W));
+            B2_CHECK(f.rows(P.in, P.at.gate + ra8, am("g1"), rg, W));
+            P.at.lr_gate = up(s.decays(), 8);
+            B2_CHECK(f.proj(P.lr, P.at.lr_gate + V, ra8 + rg));
+            B2_CHECK(f.block(P.lr, 0, 0, am("a2"), s.decays(), ra));
+            B2_CHECK(f.block(P.lr, P.at.lr_gate, ra8, am("g2"), V, rg));
+        } else {
+            B2_CHECK(f.rows(P.in, P.at.gate, am("g"), V, W));
+            if (s.decay == MemDecay::PerHead) B2_CHECK(f.rows(P.in, P.at.decay, am("a"), s.heads, W));
+        }
+        if (s.delta) B2_CHECK(f.rows(P.in, P.at.beta, am("b"), s.heads, W));
+        if (s.decay == MemDecay::Fixed) {
+            std::vector<float> d, lg;
+            for (double x : L.decay) {
+                d.push_back((float)x);
+                lg.push_back((float)std::log(x));
+            }
+            B2_CHECK(f.upload(P.decay, d));
+            B2_CHECK(f.upload(P.log_decay, lg));
+        } else {
+            B2_CHECK(f.vec(P.dt_bias, am("dt_bias"), {s.decays()}, -3.f, 1.f));
+            B2_CHECK(f.vec(P.A_log, am("A_log"), {s.heads}, 1.f, 0.7f));
+        }
+        if (s.norm) B2_CHECK(f.vec(P.mem_norm, am("norm"), {s.vdim}, 1.f, 0.f));
+        P.mem_rope = s.conv > 0 ? -1 : rope_table(lm, s.rot);
+    }
+    // what is added to the stream
+    const int att = L.has_gqa() ? a.heads * a.vdim : 0, mem = L.has_mem() ? s.heads * s.vdim : 0;
+    P.at.m = up(att, 8);
+    P.at.f = P.at.m + up(mem, 8);
+    B2_CHECK(f.proj(P.out, W, P.at.f + (ff ? L.ff : 0)));
+    if (att) B2_CHECK(f.block(P.out, 0, 0, aq("o"), W, att));
+    if (mem) B2_CHECK(f.block(P.out, 0, P.at.m, am("o"), W, mem));
+    if (ff) {
+        B2_CHECK(f.rows(P.in, P.at.up, tn.layer_key(i, tn.mlp + ".up"), L.ff, W));
+        B2_CHECK(f.block(P.out, 0, P.at.f, tn.layer_key(i, tn.mlp + ".down"), W, L.ff));
+    }
+    return B2_OK;
+}
+
 int32_t load_layer(Filler& f, LayeredModel& lm, int i) {
     const LayerSpec& L = lm.spec.layers[i];
     const TensorNames& tn = lm.spec.names;
@@ -220,8 +387,13 @@ int32_t load_layer(Filler& f, LayeredModel& lm, int i) {
     auto key = [&](const std::string& s) { return tn.layer_key(i, s); };
     auto mix = [&](const std::string& s) { return tn.layer_key(i, tn.mixer + "." + s); };
     auto mlp = [&](const std::string& s) { return tn.layer_key(i, tn.mlp + "." + s); };
-    B2_CHECK(f.vec(P.norm1, key(tn.norm1), {W}, 1.f, 0.f));
-    if (L.mixer == MixerKind::LatentAttention) {
+    B2_CHECK(f.vec(P.norm1, key(tn.norm1), {W}, 1.f, 0.f, false, lm.spec.norm_offset));
+    if (L.has_gqa() || L.has_mem()) {
+        B2_CHECK(load_branches(f, lm, i));
+        if (L.parallel) return B2_OK;
+    } else if (L.parallel) {
+        return b2_fail(B2_ERR_UNSUPPORTED, "parallel layers are available for grouped attention and memories");
+    } else if (L.mixer == MixerKind::LatentAttention) {
         const LatentAttnSpec& a = L.attn;
         const int q = a.heads * (a.dim + a.rot_dim);
         B2_CHECK(f.proj(P.qkv, q + a.row(), W));
@@ -244,12 +416,7 @@ int32_t load_layer(Filler& f, LayeredModel& lm, int i) {
         lm.dec_part_row = std::max(lm.dec_part_row, (size_t)a.heads * (a.kv_rank + 2));
         B2_CHECK(f.proj(P.attn_o, W, a.heads * a.vdim));
         B2_CHECK(f.rows(P.attn_o, 0, mix("o"), W, a.heads * a.vdim));
-        for (size_t r = 0; r < lm.ropes.size(); r++)
-            if (lm.ropes[r].spec.base == a.rot.base && lm.ropes[r].spec.dims == a.rot.dims) P.rope = (int)r;
-        if (P.rope < 0) {
-            P.rope = (int)lm.ropes.size();
-            lm.ropes.push_back(RopeTab{a.rot});
-        }
+        P.rope = rope_table(lm, a.rot);
     } else {
         const Mamba2Spec& s = L.ssm;
         B2_CHECK(f.proj(P.ssm_in, s.in_rows(), W));
@@ -262,11 +429,9 @@ int32_t load_layer(Filler& f, LayeredModel& lm, int i) {
         B2_CHECK(f.vec(P.ssm_norm, mix("norm"), {s.inner()}, 1.f, 0.f));
         B2_CHECK(f.proj(P.ssm_o, W, s.inner()));
         B2_CHECK(f.rows(P.ssm_o, 0, mix("o"), W, s.inner()));
-        P.state_off = lm.state_floats;
-        lm.state_floats += up(s.inner() * s.state, 4) + up(s.channels() * (s.conv - 1), 4);
     }
     if (L.mlp == MlpKind::None) return B2_OK;
-    B2_CHECK(f.vec(P.norm2, key(tn.norm2), {W}, 1.f, 0.f));
+    B2_CHECK(f.vec(P.norm2, key(tn.norm2), {W}, 1.f, 0.f, false, lm.spec.norm_offset));
     if (L.mlp == MlpKind::DenseGated) {
         const int ffp = up(L.ff, 64);
         B2_CHECK(f.proj(P.gu, 2 * ffp, W));
@@ -289,6 +454,12 @@ int32_t load_layer(Filler& f, LayeredModel& lm, int i) {
         }
     }
     return B2_OK;
+}
+
+// floats of a layer's recurrent record
+int64_t record_floats(const LayerSpec& L) {
+    if (L.mixer == MixerKind::Mamba2) return up(L.ssm.inner() * L.ssm.state, 4) + up(L.ssm.channels() * (L.ssm.conv - 1), 4);
+    return L.has_mem() ? up(L.mem.state_floats() + L.mem.channels() * L.mem.keep(), 4) : 0;
 }
 
 // ---- workspace ------------------------------------------------------------------------------------------------------
@@ -318,6 +489,11 @@ struct SsmBufs {
     void *zx, *xbc, *gn;
     float* y;
     int ld_xbc, ld_gn;
+};
+struct BranchBufs {
+    void *in, *lr, *q, *v, *row, *chunk;
+    float *mq, *mk, *lg, *beta, *o;
+    int ld_v;
 };
 struct DenseBufs {
     void *gu, *act;
@@ -369,6 +545,26 @@ SsmBufs carve_ssm(Carver c, const Mamba2Spec& s, const LayerP& P, size_t es, siz
     *end = std::max(*end, c.off);
     return o;
 }
+BranchBufs carve_branches(Carver c, const LayerSpec& L, const LayerP& P, size_t es, size_t t, size_t* end) {
+    BranchBufs o{};
+    const MemorySpec& s = L.mem;
+    o.in = c.take(t * P.in.N * es);
+    o.row = c.take(t * P.out.K * es);
+    if (L.has_gqa()) o.q = c.take(t * L.gqa.heads * L.gqa.k_row() * es);
+    if (L.has_mem()) {
+        o.lr = c.take(t * P.lr.N * es);
+        o.ld_v = up(s.heads * s.vdim, 8);
+        o.v = s.conv > 0 ? c.take(t * o.ld_v * es) : nullptr;
+        o.mq = c.take<float>(t * s.q_cols() * 4);
+        o.mk = c.take<float>(t * s.q_cols() * 4);
+        o.lg = c.take<float>(t * s.decays() * 4);
+        o.beta = c.take<float>(t * s.heads * 4);
+        o.o = c.take<float>(t * s.heads * s.vdim * 4);
+        o.chunk = c.take(es == 2 && b2_memory_chunk_eligible(s) ? b2_memory_chunk_bytes(s, t) : 0);
+    }
+    *end = std::max(*end, c.off);
+    return o;
+}
 DenseBufs carve_dense(Carver c, const LayerP& P, size_t es, size_t t, size_t* end) {
     DenseBufs o;
     o.ld_act = P.down.K;
@@ -403,8 +599,10 @@ size_t arena_bytes(const LayeredModel& lm, size_t es, size_t t, size_t l) {
         const LayerP& P = lm.layers[i];
         if (L.mixer == MixerKind::LatentAttention)
             carve_latent(c, L.attn, P, es, t, &end);
-        else
+        else if (L.mixer == MixerKind::Mamba2)
             carve_ssm(c, L.ssm, P, es, t, &end);
+        else
+            carve_branches(c, L, P, es, t, &end);
         if (L.mlp == MlpKind::DenseGated) carve_dense(c, P, es, t, &end);
         if (L.mlp == MlpKind::Routed) carve_moe(c, L.moe, P, pad_k(lm.spec.width), es, t, &end);
     }
@@ -487,19 +685,23 @@ struct Fwd {  // one step
     Carver scratch;
     size_t es, end = 0;
 
-    int32_t latent(const LayerSpec& L, const LayerP& P, int l);
-    int32_t ssm(const LayerSpec& L, const LayerP& P);
+    // `run`: number of the layer's run, whose cache and state are used
+    int32_t latent(const LayerSpec& L, const LayerP& P, int run);
+    int32_t ssm(const LayerSpec& L, const LayerP& P, int run);
+    int32_t branches(const LayerSpec& L, const LayerP& P, int run);
+    int32_t attend(const LayerSpec& L, const LayerP& P, const BranchBufs& b, int run);
+    int32_t remember(const LayerSpec& L, const LayerP& P, const BranchBufs& b, int run);
     int32_t dense(const LayerSpec& L, const LayerP& P);
     int32_t moe(const LayerSpec& L, const LayerP& P, const int32_t** rows);
 };
 
-int32_t Fwd::latent(const LayerSpec& L, const LayerP& P, int l) {
+int32_t Fwd::latent(const LayerSpec& L, const LayerP& P, int run) {
     b2_ctx* ctx = m->ctx;
     const LatentAttnSpec& a = L.attn;
     const LatentBufs b = carve_latent(scratch, a, P, es, (size_t)lm.t_cap, &end);
     const int T = s.T, W = a.row_pad(), q_row = b.plain_pad + b.rot_pad;
     const float scale_log2 = a.scale * 1.4426950408889634f;
-    void* cache = pool->planes[pool->layer_plane[l]].base;
+    void* cache = pool->planes[pool->layer_plane[run]].base;
     B2_CHECK(linear(m, P.qkv, c.xn, c.ldn, T, lm.t_cap, b.qkv, P.qkv.N, false));
     LatentPrepParams pp{};
     pp.qkv = b.qkv;
@@ -660,7 +862,7 @@ int32_t Fwd::latent(const LayerSpec& L, const LayerP& P, int l) {
     return linear(m, P.attn_o, b.att, b.ld_att, T, lm.t_cap, c.y, c.ldx, true);
 }
 
-int32_t Fwd::ssm(const LayerSpec& L, const LayerP& P) {
+int32_t Fwd::ssm(const LayerSpec& L, const LayerP& P, int run) {
     const SsmBufs b = carve_ssm(scratch, L.ssm, P, es, (size_t)lm.t_cap, &end);
     B2_CHECK(linear(m, P.ssm_in, c.xn, c.ldn, s.T, lm.t_cap, b.zx, P.ssm_in.N, false));
     SsmParams p{};
@@ -672,7 +874,7 @@ int32_t Fwd::ssm(const LayerSpec& L, const LayerP& P) {
     p.context_lens = s.mo->context_lens;
     p.token_seq = s.mo->token_seq;
     p.seq_slot = s.in->seq_slot;
-    p.state = pool->state + P.state_off;
+    p.state = pool->state + lm.run_state[run];
     p.slot_stride = pool->state_floats;
     p.conv_w = P.conv_w;
     p.conv_b = P.conv_b;
@@ -689,6 +891,165 @@ int32_t Fwd::ssm(const LayerSpec& L, const LayerP& P) {
     b2_prof_mark(m->ctx, B2_CLS_RECURRENT);
     B2_CHECK(b2_ssm_launch(m->ctx, m->f32, L.ssm, p));
     return linear(m, P.ssm_o, b.gn, b.ld_gn, s.T, lm.t_cap, c.y, c.ldx, true);
+}
+
+int32_t Fwd::attend(const LayerSpec& L, const LayerP& P, const BranchBufs& b, int run) {
+    b2_ctx* ctx = m->ctx;
+    const GroupedAttnSpec& a = L.gqa;
+    const KvPlane* planes = &pool->planes[pool->layer_plane[run]];
+    GqaPrepParams pp{};
+    pp.in = b.in;
+    pp.ld = P.in.N;
+    pp.q_off = P.at.q;
+    pp.k_off = P.at.k;
+    pp.v_off = P.at.v;
+    pp.T = s.T;
+    pp.q_bias = P.q_bias;
+    pp.k_bias = P.k_bias;
+    pp.v_bias = P.v_bias;
+    pp.q_norm = P.q_norm;
+    pp.k_norm = P.k_norm;
+    pp.eps = lm.spec.eps;
+    pp.positions = s.mo->positions;
+    pp.slot_mapping = s.mo->slot_mapping;
+    pp.cos_t = lm.ropes[P.rope].cos;
+    pp.sin_t = lm.ropes[P.rope].sin;
+    pp.q = b.q;
+    pp.k_cache = planes[0].base;
+    pp.v_cache = planes[1].base;
+    pp.page_size = pool->block_size;
+    b2_prof_mark(ctx, B2_CLS_ROPE_KV);
+    B2_CHECK(b2_gqa_prep_launch(ctx, m->f32, a, pp));
+    GqaAttnParams p{};
+    p.q = b.q;
+    p.k_cache = pp.k_cache;
+    p.v_cache = pp.v_cache;
+    p.block_tables = pool->block_tables;
+    p.max_blocks = pool->max_blocks;
+    p.page_size = pool->block_size;
+    p.max_pages = pool->max_pages;
+    p.T = s.T;
+    p.positions = s.mo->positions;
+    p.token_seq = s.mo->token_seq;
+    p.seq_slot = s.in->seq_slot;
+    p.dec_ctx = s.mo->dec_ctx;
+    p.dec_qrow = s.mo->dec_qrow;
+    p.dec_slot = s.mo->dec_slot;
+    p.work_seq = s.mo->dec_work_seq;
+    p.work_chunk = s.mo->dec_work_chunk;
+    p.work_off = s.mo->dec_work_off;
+    p.n_dec_work = s.mo->counts + 2;
+    p.chunk_tiles = s.chunk_tiles;
+    p.pf_seq = s.mo->pf_seq;
+    p.pf_qstart = s.mo->pf_qstart;
+    p.n_pf_work = s.mo->counts + 3;
+    p.cu_seqlens = s.mo->cu_seqlens;
+    p.context_lens = s.mo->context_lens;
+    p.q_rows = lm.t_cap;
+    p.out_scale = L.gqa_scale;
+    p.out = b.row;
+    p.ldo = P.out.K;
+    // f32, and head sizes outside the kernels' reach: the plain form.  Otherwise portions of more than a token on their own
+    // kernel where it takes them, everything else one row per token.
+    const bool rows = !m->f32 && b2_gqa_decode_eligible(a), tiles = rows && b2_gqa_prefill_eligible(a);
+    if (!rows || (s.pf_work > 0 && !tiles)) {
+        b2_prof_mark(ctx, s.pf_work > 0 ? B2_CLS_ATTN_PREFILL : B2_CLS_ATTN_DECODE);
+        return rows ? b2_gqa_decode_launch(ctx, a, p, 0) : b2_gqa_simple_launch(ctx, m->f32, a, p);
+    }
+    if (s.n_dec > 0) {
+        B2_CHECK(ensure_decode(m, s.dec_work));
+        p.part_o = lm.dec_part;
+        p.part_ml = lm.dec_part + (size_t)s.dec_work * a.heads * a.v_row();
+        B2_CHECK(b2_decode_attn_counters(ctx, s.n_dec, b2_gqa_head_blocks(a), &p.counters));
+        b2_prof_mark(ctx, B2_CLS_ATTN_DECODE);
+        B2_CHECK(b2_gqa_decode_launch(ctx, a, p, s.dec_work));
+        ctx->attn_decode_bytes += (double)s.dec_ctx_sum * a.kv_heads * (a.dim + a.vdim) * 2;
+    }
+    if (s.pf_work > 0) {
+        b2_prof_mark(ctx, B2_CLS_ATTN_PREFILL);
+        B2_CHECK(b2_gqa_prefill_launch(ctx, a, p, s.pf_work));
+        ctx->attn_prefill_flops += 2.0 * (a.dim + a.vdim) * a.heads * s.pf_pairs;
+    }
+    return B2_OK;
+}
+
+int32_t Fwd::remember(const LayerSpec& L, const LayerP& P, const BranchBufs& b, int run) {
+    const MemorySpec& sp = L.mem;
+    MemoryParams p{};
+    p.in = b.in;
+    p.ld = P.in.N;
+    p.c_off = P.at.c;
+    p.b_off = P.at.beta;
+    if (sp.low_rank) {
+        B2_CHECK(linear(m, P.lr, (const uint8_t*)b.in + P.at.gate * es, P.in.N, s.T, lm.t_cap, b.lr, P.lr.N, false));
+        p.dec = b.lr;
+        p.ld_dec = P.lr.N;
+    } else if (sp.decay == MemDecay::PerHead) {
+        p.dec = (const uint8_t*)b.in + P.at.decay * es;
+        p.ld_dec = P.in.N;
+    }
+    p.T = s.T;
+    p.B = s.B;
+    p.cu_seqlens = s.mo->cu_seqlens;
+    p.context_lens = s.mo->context_lens;
+    p.token_seq = s.mo->token_seq;
+    p.seq_slot = s.in->seq_slot;
+    p.positions = s.mo->positions;
+    p.state = pool->state + lm.run_state[run];
+    p.slot_stride = pool->state_floats;
+    p.conv_w = P.conv_w;
+    p.dt_bias = P.dt_bias;
+    p.A_log = P.A_log;
+    p.decay = P.decay;
+    p.log_decay = P.log_decay;
+    if (P.mem_rope >= 0) {
+        p.cos_t = lm.ropes[P.mem_rope].cos;
+        p.sin_t = lm.ropes[P.mem_rope].sin;
+    }
+    p.q = b.mq;
+    p.k = b.mk;
+    p.v = sp.conv > 0 ? b.v : (const void*)((const uint8_t*)b.in + (P.at.c + 2 * sp.q_cols()) * es);
+    p.ld_v = sp.conv > 0 ? b.ld_v : P.in.N;
+    p.lg = b.lg;
+    p.beta = b.beta;
+    p.o = b.o;
+    p.chunk = b.chunk;
+    p.max_n = s.max_n;
+    b2_prof_mark(m->ctx, B2_CLS_RECURRENT);
+    return b2_memory_launch(m->ctx, m->f32, sp, p);
+}
+
+int32_t Fwd::branches(const LayerSpec& L, const LayerP& P, int run) {
+    const BranchBufs b = carve_branches(scratch, L, P, es, (size_t)lm.t_cap, &end);
+    B2_CHECK(linear(m, P.in, c.xn, c.ldn, s.T, lm.t_cap, b.in, P.in.N, false));
+    if (L.has_gqa()) B2_CHECK(attend(L, P, b, run));
+    if (L.has_mem()) B2_CHECK(remember(L, P, b, run));
+    BranchOutParams p{};
+    p.out = b.row;
+    p.ldo = P.out.K;
+    p.T = s.T;
+    p.att_cols = L.has_gqa() ? L.gqa.heads * L.gqa.vdim : 0;
+    if (L.has_mem()) {
+        p.o = b.o;
+        p.heads = L.mem.heads;
+        p.vdim = L.mem.vdim;
+        p.m_off = P.at.m;
+        p.gate = L.mem.low_rank ? (const uint8_t*)b.lr + P.at.lr_gate * es : (const uint8_t*)b.in + P.at.gate * es;
+        p.ld_gate = L.mem.low_rank ? P.lr.N : P.in.N;
+        p.act = L.mem.gate;
+        p.norm = P.mem_norm;
+        p.eps = lm.spec.eps;
+        p.scale = L.mem_scale;
+    }
+    if (L.parallel && L.mlp == MlpKind::DensePlain) {
+        p.up = (const uint8_t*)b.in + P.at.up * es;
+        p.ld_up = P.in.N;
+        p.ff = L.ff;
+        p.f_off = P.at.f;
+    }
+    b2_prof_mark(m->ctx, B2_CLS_ELEMENTWISE);
+    B2_CHECK(b2_branch_out_launch(m->ctx, m->f32, p));
+    return linear(m, P.out, b.row, P.out.K, s.T, lm.t_cap, c.y, c.ldx, true);
 }
 
 int32_t Fwd::dense(const LayerSpec& L, const LayerP& P) {
@@ -767,7 +1128,18 @@ int b2_layered_q_tile(const b2_model*) { return 128; }
 // One CTA of the decode attention fills an SM, so the work items (times the head groups) should fill whole rounds of the
 // machine: the smallest chunk, in whole tiles from 128 keys on, that does not open another round.
 int b2_layered_chunk_tiles(const b2_model* m, const std::vector<SeqStep>& seqs) {
-    int groups = 1;
+    int groups = 1, blocks = 0;
+    bool latent = false;
+    for (auto& L : m->layered->spec.layers) {
+        latent |= L.mixer == MixerKind::LatentAttention;
+        if (L.has_gqa()) blocks = std::max(blocks, b2_gqa_head_blocks(L.gqa));
+    }
+    if (!latent) {  // several small CTAs per SM
+        long ctx_sum = 0;
+        for (auto& s : seqs)
+            if (s.n == 1) ctx_sum += s.cache->len + 1;
+        return b2_small_cta_chunk_tiles(ctx_sum, std::max(blocks, 1), m->ctx->sm_count);
+    }
     for (auto& L : m->layered->spec.layers)
         if (L.mixer == MixerKind::LatentAttention && L.attn.heads > 16) groups = std::max(groups, (L.attn.heads + 31) / 32);
     int rows = 0, longest = 1;
@@ -796,8 +1168,13 @@ int b2_layered_chunk_tiles(const b2_model* m, const std::vector<SeqStep>& seqs) 
 }
 
 void b2_layered_cache_layout(const b2_model* m, int block_size, std::vector<std::vector<size_t>>& page_bytes, int64_t& state_floats) {
-    for (auto& L : m->layered->spec.layers) {
+    for (const LayerRun& r : m->layered->runs) {
+        const LayerSpec& L = m->layered->spec.layers[r.layer];
         page_bytes.emplace_back();
+        if (L.has_gqa()) {
+            page_bytes.back().push_back((size_t)block_size * L.gqa.kv_heads * L.gqa.k_row() * esz(m));
+            page_bytes.back().push_back((size_t)block_size * L.gqa.kv_heads * L.gqa.v_row() * esz(m));
+        }
         if (L.mixer == MixerKind::LatentAttention) page_bytes.back().push_back((size_t)block_size * L.attn.row_pad() * esz(m));
     }
     state_floats = m->layered->state_floats;
@@ -841,11 +1218,16 @@ int32_t b2_model_build_layered(b2_ctx* ctx, const ModelSpec& spec, const b2_weig
     LayeredModel& lm = *m->layered;
     lm.spec = spec;
     lm.layers.resize(spec.layers.size());
+    lm.runs = spec.runs();
+    for (const LayerRun& r : lm.runs) {
+        lm.run_state.push_back(lm.state_floats);
+        lm.state_floats += record_floats(spec.layers[r.layer]);
+    }
     m->cfg.num_layers = (int32_t)spec.layers.size();
     m->cfg.hidden_size = spec.width;
     m->cfg.vocab_size = spec.vocab;
     m->cfg.rms_norm_eps = spec.eps;
-    m->cfg.tie_word_embeddings = 1;
+    m->cfg.tie_word_embeddings = spec.own_head ? 0 : 1;
     m->cfg.compute_f32 = f32 ? 1 : 0;
     m->hkv_l = 1;  // the latent is one key/value head
     Filler f{m, w, prefix, seed};
@@ -853,9 +1235,15 @@ int32_t b2_model_build_layered(b2_ctx* ctx, const ModelSpec& spec, const b2_weig
         Proj head;
         B2_CHECK(f.proj(head, spec.vocab, spec.width));
         B2_CHECK(f.rows(head, 0, spec.names.embed, spec.vocab, spec.width));
-        lm.embed = head.w;
+        lm.embed = lm.head = head.w;
+        if (spec.own_head) {
+            B2_CHECK(f.proj(head, spec.vocab, spec.width));
+            B2_CHECK(f.rows(head, 0, spec.names.head, spec.vocab, spec.width));
+            lm.head = head.w;
+        }
+        if (spec.loop.times > 0) B2_CHECK(f.vec(lm.loop_step, spec.names.loop_step, {spec.loop.times, spec.width}, 0.f, 0.1f));
         for (size_t i = 0; i < spec.layers.size(); i++) B2_CHECK(load_layer(f, lm, (int)i));
-        B2_CHECK(f.vec(lm.final_norm, spec.names.final_norm, {spec.width}, 1.f, 0.f));
+        B2_CHECK(f.vec(lm.final_norm, spec.names.final_norm, {spec.width}, 1.f, 0.f, false, spec.norm_offset));
         B2_CUDA(cudaMalloc((void**)&lm.route_counters, 1025 * sizeof(int)));
         B2_CUDA(cudaMemsetAsync(lm.route_counters, 0, 1025 * sizeof(int), ctx->stream));
         B2_CUDA(cudaEventCreate(&m->ev0));
@@ -912,7 +1300,7 @@ int32_t b2_forward_layered(b2_model* m, b2_pool* pool, const LayeredStep& s, flo
         an.out = out;
         an.ldo = c.ldn;
         an.out_scale = scale;
-        an.write_x = write && an.n_src > 0;
+        an.write_x = write && (an.n_src > 0 || an.vec || an.table);
         b2_prof_mark(ctx, B2_CLS_ELEMENTWISE);
         return b2_add_norm_launch(ctx, m->f32, an);
     };
@@ -921,14 +1309,26 @@ int32_t b2_forward_layered(b2_model* m, b2_pool* pool, const LayeredStep& s, flo
         an.n_src = n;
     };
     const int64_t per_layer = (int64_t)s.T * spec.width;
-    const bool capture = lm.capture && lm.capture_cap >= per_layer * (int64_t)spec.layers.size();
-    for (size_t l = 0; l < spec.layers.size(); l++) {
-        const LayerSpec& L = spec.layers[l];
-        const LayerP& P = lm.layers[l];
+    const bool capture = lm.capture && lm.capture_cap >= per_layer * (int64_t)lm.runs.size();
+    for (size_t r = 0; r < lm.runs.size(); r++) {
+        const LayerRun& run = lm.runs[r];
+        const LayerSpec& L = spec.layers[run.layer];
+        const LayerP& P = lm.layers[run.layer];
+        if (run.opens_pass) {  // what a pass adds to the stream
+            an.vec = lm.loop_step + (size_t)run.pass * spec.width;
+            if (run.pass > 0) {
+                an.table = lm.embed;
+                an.ids = s.ids_dev;
+                an.ld_table = c.ldn;
+                an.vocab = spec.vocab;
+            }
+        }
         B2_CHECK(norm(P.norm1, s.T, nullptr, c.xn, 1.f, true));
-        B2_CHECK(L.mixer == MixerKind::LatentAttention ? f.latent(L, P, (int)l) : f.ssm(L, P));
+        an.vec = nullptr;
+        an.table = nullptr;
+        B2_CHECK(L.mixer == MixerKind::LatentAttention ? f.latent(L, P, (int)r) : L.mixer == MixerKind::Mamba2 ? f.ssm(L, P, (int)r) : f.branches(L, P, (int)r));
         pending(nullptr, 1);
-        if (L.mlp != MlpKind::None) {
+        if (L.mlp != MlpKind::None && !L.parallel) {
             B2_CHECK(norm(P.norm2, s.T, nullptr, c.xn, 1.f, true));
             const int32_t* rows = nullptr;
             if (L.mlp == MlpKind::DenseGated) {
@@ -942,7 +1342,7 @@ int32_t b2_forward_layered(b2_model* m, b2_pool* pool, const LayeredStep& s, flo
         if (capture) {
             B2_CHECK(norm(nullptr, s.T, nullptr, nullptr, 1.f, true));  // the addition alone
             pending(nullptr, 0);
-            B2_CUDA(cudaMemcpy2DAsync(lm.capture + (int64_t)l * per_layer, (size_t)spec.width * 4, c.x, (size_t)c.ldx * 4, (size_t)spec.width * 4, (size_t)s.T,
+            B2_CUDA(cudaMemcpy2DAsync(lm.capture + (int64_t)r * per_layer, (size_t)spec.width * 4, c.x, (size_t)c.ldx * 4, (size_t)spec.width * 4, (size_t)s.T,
                                       cudaMemcpyDeviceToHost, ctx->stream));
         }
     }
@@ -951,7 +1351,7 @@ int32_t b2_forward_layered(b2_model* m, b2_pool* pool, const LayeredStep& s, flo
         Proj head;
         head.N = pad_n(spec.vocab);
         head.K = c.ldn;
-        head.w = lm.embed;
+        head.w = lm.head;
         B2_CHECK(linear(m, head, c.last, c.ldn, s.n_logits, lm.l_cap, c.logits, c.ldl, true));
         b2_prof_mark(ctx, B2_CLS_ELEMENTWISE);
         B2_CHECK(b2_argmax_f32_launch(ctx, c.logits, c.ldl, s.n_logits, spec.vocab, m->ws.argmax));

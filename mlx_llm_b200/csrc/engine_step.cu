@@ -147,15 +147,6 @@ int32_t gemm_reduce_residual(b2_model* m, const Proj& p, const uint16_t* a, int 
     return b2_residual_add_f32_launch(ctx, m->ws.tp_part, (int64_t)M * H, x);
 }
 
-int pick_chunk_tiles(long dec_ctx_sum, int hkv, int sm_count) {
-    // enough (chunk, kv head) CTAs for ~8 per SM, chunks between 128 and 1024 tokens
-    long target = (long)sm_count * 8;
-    long tok = dec_ctx_sum * hkv / std::max(1l, target);
-    int chunk = 128;
-    while (chunk < 1024 && chunk < tok) chunk *= 2;
-    return chunk / 16;
-}
-
 // The bf16 layers of one step: embedding, every decoder layer, the sampled rows' final norm, lm_head and argmax.
 int32_t forward_bf16_layers(b2_model* m, b2_pool* pool, const BatchMetaOut& mo, const BatchMetaIn& in, const int32_t* ids_dev, int T, int n_dec,
                             long dec_ctx_sum, int W, int P, double pf_flops, int pf_max_ctx, int chunk_tiles, int q_tile, int n_logits, const int32_t* logit_rows) {
@@ -285,6 +276,15 @@ int32_t forward_bf16_layers(b2_model* m, b2_pool* pool, const BatchMetaOut& mo, 
 
 }  // namespace
 
+int b2_small_cta_chunk_tiles(long dec_ctx_sum, int blocks, int sm_count) {
+    // enough (chunk, kv head) CTAs for ~8 per SM, chunks between 128 and 1024 tokens
+    long target = (long)sm_count * 8;
+    long tok = dec_ctx_sum * blocks / std::max(1l, target);
+    int chunk = 128;
+    while (chunk < 1024 && chunk < tok) chunk *= 2;
+    return chunk / 16;
+}
+
 int32_t b2_engine_forward(b2_model* m, std::vector<SeqStep>& seqs, void* logits_out, int32_t* argmax_out) {
     b2_ctx* ctx = m->ctx;
     const b2_model_config& c = m->cfg;
@@ -327,7 +327,7 @@ int32_t b2_engine_forward(b2_model* m, std::vector<SeqStep>& seqs, void* logits_
     B2_CHECK(m->layered ? b2_layered_ensure_rope(m, max_pos) : b2_model_ensure_rope(m, max_pos));
     // pages for the new tokens (host allocator), then the step descriptors
     for (auto& s : seqs) B2_CHECK(b2_cache_reserve(s.cache, s.n));
-    const int chunk_tiles = m->layered ? b2_layered_chunk_tiles(m, seqs) : pick_chunk_tiles(dec_ctx_sum, m->hkv_l, ctx->sm_count);
+    const int chunk_tiles = m->layered ? b2_layered_chunk_tiles(m, seqs) : b2_small_cta_chunk_tiles(dec_ctx_sum, m->hkv_l, ctx->sm_count);
     const int q_tile = m->layered ? b2_layered_q_tile(m) : b2_prefill_q_tile(ctx, c.head_dim);
     int W = 0, P = 0;
     double pf_flops = 0;  // 4*hd*hq flops per (query, visible key) pair
@@ -435,6 +435,7 @@ int32_t b2_engine_forward(b2_model* m, std::vector<SeqStep>& seqs, void* logits_
         ls.pf_work = P;
         ls.chunk_tiles = chunk_tiles;
         ls.max_ctx = max_pos;
+        for (auto& s : seqs) ls.max_n = std::max(ls.max_n, s.n);
         ls.dec_ctx_sum = dec_ctx_sum;
         ls.pf_pairs = pf_pairs;
         ls.pf_ctx = pf_ctx;

@@ -31,6 +31,110 @@ def config(layers, width=104, vocab=333, eps=3e-5, logit_scale=0.4):
                 layers=[dict(type=m[0], mixer=m[1], mlp=f) for m, f in layers])
 
 
+# ---- Tirezen: retention, delta memories, capped sink attention beside a delta memory, a repeated stretch of layers ------
+def retention(heads=3, dim=20, vdim=28, base=3000.0, dims=12, decay=None):
+    return ("retention", dict(heads=heads, dim=dim, vdim=vdim, rot=dict(base=base, dims=dims),
+                              decay=decay or [1.0 - 2.0 ** -(2 + 3 * (i % 3)) for i in range(heads)]))
+
+
+def delta(heads=6, kv_heads=3, dim=28, vdim=12, conv=2):
+    return ("delta", dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, conv=conv))
+
+
+def sides(heads=4, kv_heads=2, dim=24, vdim=40, dims=16, base=700.0, scale=None, softcap=4.0, left_scale=0.7, right_scale=1.3, right=None):
+    left = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, rot=dict(base=base, dims=dims), scale=scale or dim ** -0.5 * 1.5, softcap=softcap)
+    right = {**dict(heads=4, kv_heads=2, dim=12, vdim=20, conv=3), **(right or {})}
+    return ("parallel", dict(left=left, right=right, left_scale=left_scale, right_scale=right_scale))
+
+
+def tirezen(layers, width=72, vocab=211, eps=2e-5, loop=(0, 0, 0)):
+    cfg = dict(architecture="Tirezen", width=width, vocab=vocab, norm=dict(eps=eps), layers=[dict(type=m[0], mixer=m[1], mlp=f) for m, f in layers])
+    if loop[2]:
+        cfg["loop"] = dict(start=loop[0], stop=loop[1], times=loop[2])
+    return cfg
+
+
+def tirezen_weights(cfg, seed=0, gain=None, ranks=(7, 11)):
+    """name -> float64 array of bf16 values; ranks: of the decay's and the gate's two-factor projections."""
+    rng = np.random.default_rng(seed)
+    w, W = {}, cfg["width"]
+
+    def mat(name, rows, cols):
+        g = next((v for k, v in (gain or {}).items() if name.endswith(k)), 1.0)
+        w[name] = round_bf16(rng.standard_normal((rows, cols)) * g / np.sqrt(cols))
+
+    def vec(name, n, mean, sd):
+        w[name] = round_bf16(mean + sd * rng.standard_normal(n))
+
+    def delta_part(p, m, low_rank):
+        H, G, D, V = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        for n, c in (("q", G * D), ("k", G * D), ("v", H * V)):
+            mat(p + n, c, W)
+            vec(f"{p}{n}.conv", (c, m["conv"]), 0.3, 0.6)
+        mat(p + "b", H, W)
+        vec(p + "A_log", H, 0.0, 1.0)
+        vec(p + "norm", V, 1.0, 0.2)
+        if low_rank:
+            mat(p + "a1", ranks[0], W), mat(p + "a2", H * D, ranks[0]), mat(p + "g1", ranks[1], W), mat(p + "g2", H * V, ranks[1])
+            vec(p + "dt_bias", H * D, -2.5, 1.5)
+        else:
+            mat(p + "a", H, W), mat(p + "g", H * V, W)
+            vec(p + "dt_bias", H, -2.5, 1.5)
+        mat(p + "o", W, H * V)
+
+    w["embed"] = round_bf16(rng.standard_normal((cfg["vocab"], W)))
+    if cfg.get("loop"):
+        vec("loop.step", (cfg["loop"]["times"], W), 0.0, 0.5)
+    for i, L in enumerate(cfg["layers"]):
+        m, p = L["mixer"], f"l{i}.mix."
+        vec(f"l{i}.norm1", W, 0.0, 0.2)
+        if L["type"] == "retention":
+            H, D, V = m["heads"], m["dim"], m["vdim"]
+            mat(p + "q", H * D, W), mat(p + "k", H * D, W), mat(p + "v", H * V, W), mat(p + "g", H * V, W), mat(p + "o", W, H * V)
+        elif L["type"] == "delta":
+            delta_part(p, m, False)
+        else:
+            a = m["left"]
+            for n, c in (("q", a["heads"] * a["dim"]), ("k", a["kv_heads"] * a["dim"]), ("v", a["kv_heads"] * a["vdim"])):
+                mat(p + "left." + n, c, W)
+                vec(f"{p}left.{n}.b", c, 0.0, 0.3)
+            vec(p + "left.q.norm", a["dim"], 1.2, 0.3)
+            vec(p + "left.k.norm", a["dim"], 1.2, 0.3)
+            mat(p + "left.o", W, a["heads"] * a["vdim"])
+            delta_part(p + "right.", m["right"], True)
+        if L["mlp"]:
+            mat(f"l{i}.mlp.up", L["mlp"]["ff"], W), mat(f"l{i}.mlp.down", W, L["mlp"]["ff"])
+    vec("final.norm", W, 0.0, 0.2)
+    mat("head", cfg["vocab"], W)
+    return w
+
+
+def tokens(cfg, n, seed):
+    return np.random.default_rng(seed).integers(0, cfg["vocab"], n).astype(np.int32)
+
+
+def error(got, want):
+    """Worst row: rms of the error over the rms spread of the wanted logits."""
+    d = got - want
+    d = d - d.mean(1, keepdims=True)
+    spread = np.sqrt(np.mean((want - want.mean(1, keepdims=True)) ** 2))
+    return float(np.sqrt((d * d).mean(1)).max() / spread)
+
+
+def run(eng, model, pool, ids, cuts, cache=None):
+    """Feeds ids in portions of the given sizes, the rest one by one; logits of every position."""
+    c = cache or eng.PagedKvCache(pool)
+    out, at = [], 0
+    while at < len(ids):
+        n = min(cuts[len(out)] if len(out) < len(cuts) else 1, len(ids) - at)
+        lg, _ = model.step_at([(ids[at:at + n], c)], [list(range(n))])
+        out.append(lg)
+        at += n
+    if cache is None:
+        c.free()
+    return np.concatenate(out)
+
+
 def round_bf16(a):
     return H.bf16_to_f32_np(H.f32_to_bf16_np(np.asarray(a, np.float32))).astype(np.float64)
 
@@ -151,4 +255,21 @@ CASES = {
     "wide_plain": config([(latent(heads=2, dim=200, rot_dim=8, vdim=140, kv_rank=72), dense(64))], width=64, vocab=80),
     "big_state": config([(mamba(heads=4, vdim=64, state=128, groups=1, norm_groups=2, conv=4), moe(experts=16, top=4, ff=128)),
                          (mamba(heads=2, vdim=16, state=200, groups=2, norm_groups=2), dense(192))], width=128, vocab=200),
+}
+
+TIREZEN = {
+    "all_kinds": tirezen([(retention(), dense(88)), (sides(), dense(136)), (delta(), None), (sides(heads=6, kv_heads=1, vdim=16, softcap=9.0, right=dict(conv=4)), dense(40))],
+                         loop=(1, 3, 3)),
+    # sizes that divide nothing, one head, one tap, single query groups
+    "odd": tirezen([(sides(heads=5, kv_heads=5, dim=10, vdim=7, dims=4, right=dict(conv=1)), dense(33)), (delta(heads=3, kv_heads=1, dim=9, vdim=5, conv=5), dense(50)),
+                    (retention(heads=1, dim=7, vdim=3, dims=6), None)], width=52, vocab=97, loop=(0, 3, 2)),
+    # the tiles of the tensor-core kernels, more than eight query heads for one key head
+    "tiles": tirezen([(sides(heads=10, kv_heads=1, dim=128, vdim=128, dims=128, softcap=15.0, right=dict(heads=2, kv_heads=1, dim=128, vdim=64, conv=4)), dense(512)),
+                      (retention(heads=2, dim=128, vdim=128, dims=64), dense(256)), (delta(heads=2, kv_heads=2, dim=128, vdim=64, conv=4), None)],
+                     width=128, vocab=300, loop=(2, 3, 1)),
+    "uneven": tirezen([(sides(heads=4, kv_heads=4, dim=160, vdim=72, dims=96, softcap=3.0), None), (sides(heads=3, kv_heads=3, dim=64, vdim=144, dims=64), dense(64)),
+                       (retention(heads=2, dim=48, vdim=200, dims=48), dense(72))], width=96, vocab=150),
+    # beyond those kernels
+    "large_heads": tirezen([(sides(heads=2, kv_heads=1, dim=232, vdim=250, dims=100, softcap=6.0), None), (delta(heads=2, kv_heads=1, dim=200, vdim=136, conv=3), dense(30))],
+                           width=64, vocab=80),
 }

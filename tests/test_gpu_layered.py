@@ -12,6 +12,7 @@ import pytest
 
 from oracle import layered as ref
 from tests import layered_models as lm
+from tests.layered_models import error, run, tokens
 
 pytestmark = pytest.mark.gpu
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
@@ -41,43 +42,12 @@ def get_model(env, name, f32):
     return _models[name, f32]
 
 
-def tokens(cfg, n, seed):
-    return np.random.default_rng(seed).integers(0, cfg["vocab"], n).astype(np.int32)
-
-
 def want_logits(name, cfg, w, n, seed=0):
     """Oracle logits [n, vocab] of the test sequence (a prefix of a longer one is the same, so compute it once)."""
     key = (name, seed)
     if key not in _refs or len(_refs[key]) < n:
         _refs[key] = ref.forward(cfg, w, tokens(cfg, n, seed))
     return _refs[key][:n]
-
-
-def error(got, want):
-    d = got - want
-    d = d - d.mean(1, keepdims=True)
-    spread = np.sqrt(np.mean((want - want.mean(1, keepdims=True)) ** 2))
-    return float(np.sqrt((d * d).mean(1)).max() / spread)
-
-
-def run(eng, model, pool, ids, cuts, cache=None):
-    """Feeds ids in portions of the given sizes; logits of every position."""
-    c = cache or eng.PagedKvCache(pool)
-    out, at = [], 0
-    for n in cuts:
-        n = min(n, len(ids) - at)
-        if n <= 0:
-            break
-        lg, _ = model.step_at([(ids[at:at + n], c)], [list(range(n))])
-        out.append(lg)
-        at += n
-    while at < len(ids):
-        lg, _ = model.step_at([(ids[at:at + 1], c)], [[0]])
-        out.append(lg)
-        at += 1
-    if cache is None:
-        c.free()
-    return np.concatenate(out)
 
 
 @pytest.mark.parametrize("f32", [True, False])
