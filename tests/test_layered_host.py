@@ -19,6 +19,7 @@ def eng():
 
 def test_registry_names_the_family(eng):
     assert eng.model_family(lm.CASES["mixed"]) == "Zukitar"
+    assert all(eng.model_family(c) == "Tirezen" for c in lm.TIREZEN.values())
     llama = dict(hidden_size=64, intermediate_size=128, num_hidden_layers=2, num_attention_heads=4, vocab_size=32)
     assert eng.model_family(llama) == "llama"
 
@@ -97,3 +98,68 @@ def test_small_pieces():
          "e1.gate": np.zeros((1, 1)), "e1.up": np.zeros((1, 1)), "e1.down": np.zeros((1, 1))}
     got = ref.routed_ff(np.array([[1.0]]), W.__getitem__, one)
     assert np.allclose(got, 0.5 / (1 + np.exp(-1.702 * 0.5)) * 0.5)  # gate cut at 0.5, up at -0.5
+
+
+def test_tirezen_configurations_that_are_refused(eng):
+    from mlx_llm_b200._lib import B2Error
+
+    def sub(c, *path):
+        for p in path:
+            c = c[p]
+        return c
+
+    base = lm.TIREZEN["all_kinds"]
+    for change, word in ((lambda c: c.pop("width"), "width"), (lambda c: sub(c, "layers", 0, "mixer", "decay").pop(), "decay"),
+                         (lambda c: sub(c, "layers", 0, "mixer").update(decay=[0.5, 0.0, 0.5]), "decay"), (lambda c: sub(c, "layers", 2, "mixer").update(kv_heads=4), "kv_heads"),
+                         (lambda c: sub(c, "layers", 1, "mixer", "left").update(kv_heads=3), "kv_heads"), (lambda c: sub(c, "layers", 1, "mixer", "left").pop("softcap"), "softcap"),
+                         (lambda c: sub(c, "layers", 1, "mixer").pop("right"), "right"), (lambda c: sub(c, "layers", 1, "mixer").pop("left_scale"), "left_scale"),
+                         (lambda c: sub(c, "layers", 0, "mixer", "rot").update(dims=22), "rot"), (lambda c: c["loop"].update(stop=5), "loop"), (lambda c: c["loop"].update(start=3), "loop"),
+                         (lambda c: c["loop"].update(times=0), "times"), (lambda c: c["layers"][0].update(type="mamba2"), "mamba2"),
+                         (lambda c: sub(c, "layers", 0, "mlp").update(kind="moe"), "kind")):
+        cfg = copy.deepcopy(base)
+        change(cfg)
+        with pytest.raises(B2Error) as e:
+            eng.model_family(cfg)
+        assert e.value.code == -4 and word in str(e.value), str(e.value)
+
+
+def test_delta_rule_solves_a_triangular_system():
+    """The writes u of a stretch of tokens from a zero state: (I + A) u = beta v, A the decayed products of the keys."""
+    rng = np.random.default_rng(5)
+    T, D, V = 9, 4, 3
+    q, k, v = rng.standard_normal((T, D)), rng.standard_normal((T, D)) * 0.5, rng.standard_normal((T, V))
+    lg, beta = -rng.random((T, D)), rng.random(T)
+    G = np.cumsum(lg, 0)
+    pair = lambda a, t, s: (a[t] * np.exp(G[t] - G[s]) * k[s]).sum()
+    A = np.array([[beta[t] * pair(k, t, s) if s < t else 0.0 for s in range(T)] for t in range(T)])
+    u = np.linalg.solve(np.eye(T) + A, beta[:, None] * v)
+    o = np.array([sum(pair(q, t, s) * u[s] for s in range(t + 1)) for t in range(T)])
+    assert np.allclose(o, ref.decayed_memory(q, k, v, lg, beta))
+    plain = np.array([sum(pair(q, t, s) * v[s] for s in range(t + 1)) for t in range(T)])
+    assert np.allclose(plain, ref.decayed_memory(q, k, v, lg))
+
+
+def test_pieces_of_the_capped_sink_attention():
+    rng = np.random.default_rng(1)
+    m = dict(heads=2, kv_heads=1, dim=4, vdim=3, rot=dict(base=10.0, dims=2), scale=0.5, softcap=1e6)
+    w = dict(q=rng.standard_normal((8, 5)), k=rng.standard_normal((4, 5)), v=rng.standard_normal((3, 5)), o=np.eye(6))
+    w.update({"q.b": rng.standard_normal(8), "k.b": rng.standard_normal(4), "v.b": rng.standard_normal(3), "q.norm": np.ones(4), "k.norm": np.ones(4)})
+    h = rng.standard_normal((1, 5))
+    out = ref.sink_attention(h, w.__getitem__, m, 0.0)[0]  # one token: weight exp(s) / (1 + exp(s)) on its own value
+    v = w["v"] @ h[0] + w["v.b"]
+    k = ref.rms(w["k"] @ h[0] + w["k.b"], 0.0)
+    for i in range(2):
+        q = ref.rms((w["q"] @ h[0] + w["q.b"])[4 * i:4 * i + 4], 0.0)
+        assert np.allclose(out[3 * i:3 * i + 3], ref.sigmoid(0.5 * q @ k) * v)
+    capped = ref.sink_attention(h, w.__getitem__, dict(m, softcap=1e-9), 0.0)[0]
+    assert np.allclose(capped, np.concatenate([v, v]) / 2)
+    r = ref.rotate_halves(np.array([[[1.0, 9.0, 0.0, 8.0, 5.0]]]), np.array([1.0]), 100.0, 4)
+    a = 1.0 * 100.0 ** -0.5
+    assert np.allclose(r, [[[np.cos(1.0), 9 * np.cos(a) - 8 * np.sin(a), np.sin(1.0), 8 * np.cos(a) + 9 * np.sin(a), 5.0]]])
+    assert np.allclose(ref.gelu_erf(np.array([0.0, 1.0])), [0.0, 0.8413447460685429])
+
+
+def test_layer_runs():
+    cfg = dict(layers=[0] * 4, loop=dict(start=1, stop=3, times=2))
+    assert ref.layer_runs(cfg) == [(0, -1), (1, 0), (2, 0), (1, 1), (2, 1), (3, -1)]
+    assert ref.layer_runs(dict(layers=[0] * 2)) == [(0, -1), (1, -1)]
