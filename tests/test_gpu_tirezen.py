@@ -198,12 +198,12 @@ def test_the_sink_counts(env, cuts, f32, sign):
     change(w)
     h = np.random.default_rng(0).standard_normal((20, 64))
     g = lambda n: w["l0.mix.left." + n]
-    with_sink = ref.sink_attention(h, g, layer[1]["left"], 1e-6)
+    with_sink = ref.sink_attention(h, g, layer[0][1]["left"], 1e-6)
     far = np.abs(with_sink).max()
     assert far < 0.5 if sign < 0 else far > 0.5  # the sink decides
     # with the sink's share the left mixer is small; it is scaled up so that it still dominates the logits
     if sign < 0:
-        layer[1]["left_scale"] = 40.0
+        layer[0][1]["left_scale"] = 40.0
     e = single(eng, ctx, layer, f32, cuts=cuts, change=change)
     assert e < (1e-4 if f32 else 0.1), e
 
