@@ -51,8 +51,9 @@ struct GroupedAttnSpec {
     bool qk_norm = false; // RMS norm over the head of queries and keys, before the rotation
     RotSpec rot;
     constexpr int group() const { return heads / kv_heads; }
-    constexpr int k_row() const { return (dim + 15) / 16 * 16; }  // values per cached head row, zero-padded for 16-wide steps
-    constexpr int v_row() const { return (vdim + 15) / 16 * 16; }
+    // values per cached head row, zero-padded for 16-wide steps and to one 64-wide load box at least
+    constexpr int k_row() const { return dim < 64 ? 64 : (dim + 15) / 16 * 16; }
+    constexpr int v_row() const { return vdim < 64 ? 64 : (vdim + 15) / 16 * 16; }
 };
 // Linear memory: a state S [dim][vdim] per head in f32, read with the query after the token's own write,
 //     S <- decay * S;   S <- S + k u^T;   o = S^T q;   out = norm(o) * gate
