@@ -216,7 +216,8 @@ struct LayeredStep {
     const int32_t* ids_dev;
     int T, B, n_dec, dec_work, pf_work, chunk_tiles, max_ctx;
     long dec_ctx_sum;
-    int max_n;                  // longest portion
+    int n_chunks;               // chunks of the portions that the memories' chunked form takes
+    const int32_t* chunk_off;   // [B] device: first chunk of each such portion, -1 for the others
     double pf_pairs;  // (query, visible key) pairs of the prefilling sequences
     int pf_ctx;                 // their contexts (this step's tokens included), summed
     const int32_t* pf_kv_off;   // [B] device: running sum of those contexts, -1 for sequences with a single token

@@ -74,6 +74,9 @@ struct LayeredModel {
     // decode attention: partial results per work item
     float* dec_part = nullptr;
     size_t dec_part_floats = 0, dec_part_row = 0;  // capacity; heads * (values + 2) of the largest layer
+    // factors of the memories' chunks, one layer at a time
+    uint8_t* chunks = nullptr;
+    size_t chunk_bytes = 0;
     uint8_t* arena = nullptr;
     int t_cap = 0, l_cap = 0;
     float* capture = nullptr;
@@ -491,7 +494,7 @@ struct SsmBufs {
     int ld_xbc, ld_gn;
 };
 struct BranchBufs {
-    void *in, *lr, *q, *v, *row, *chunk;
+    void *in, *lr, *q, *v, *row;
     float *mq, *mk, *lg, *beta, *o;
     int ld_v;
 };
@@ -560,7 +563,6 @@ BranchBufs carve_branches(Carver c, const LayerSpec& L, const LayerP& P, size_t 
         o.lg = c.take<float>(t * s.decays() * 4);
         o.beta = c.take<float>(t * s.heads * 4);
         o.o = c.take<float>(t * s.heads * s.vdim * 4);
-        o.chunk = c.take(es == 2 && b2_memory_chunk_eligible(s) ? b2_memory_chunk_bytes(s, t) : 0);
     }
     *end = std::max(*end, c.off);
     return o;
@@ -651,6 +653,14 @@ int32_t ensure_decode(b2_model* m, int items) {
     B2_CUDA(cudaStreamSynchronize(m->ctx->stream));
     lm.dec_part_floats = need * 5 / 4;
     return regrow_zero(m->ctx, lm.dec_part, lm.dec_part_floats);
+}
+
+int32_t ensure_chunks(b2_model* m, size_t bytes) {
+    LayeredModel& lm = *m->layered;
+    if (bytes <= lm.chunk_bytes) return B2_OK;
+    B2_CUDA(cudaStreamSynchronize(m->ctx->stream));
+    lm.chunk_bytes = bytes * 5 / 4;
+    return regrow_zero(m->ctx, lm.chunks, lm.chunk_bytes);
 }
 
 // ---- forward --------------------------------------------------------------------------------------------------------
@@ -1013,8 +1023,12 @@ int32_t Fwd::remember(const LayerSpec& L, const LayerP& P, const BranchBufs& b, 
     p.lg = b.lg;
     p.beta = b.beta;
     p.o = b.o;
-    p.chunk = b.chunk;
-    p.max_n = s.max_n;
+    if (!m->f32 && s.n_chunks > 0 && b2_memory_chunk_eligible(sp)) {
+        B2_CHECK(ensure_chunks(m, (size_t)s.n_chunks * b2_memory_chunk_bytes(sp)));
+        p.n_chunks = s.n_chunks;
+        p.chunk_off = s.chunk_off;
+        p.chunk = lm.chunks;
+    }
     b2_prof_mark(m->ctx, B2_CLS_RECURRENT);
     return b2_memory_launch(m->ctx, m->f32, sp, p);
 }
@@ -1268,7 +1282,7 @@ void b2_layered_release(b2_model* m) {
         if (r.sin) cudaFree(r.sin);
     }
     if (lm.route_counters) cudaFree(lm.route_counters);
-    for (void* p : {(void*)lm.arena, (void*)lm.kv_lat, (void*)lm.kv_rot, (void*)lm.kv_exp, (void*)lm.dec_part})
+    for (void* p : {(void*)lm.arena, (void*)lm.kv_lat, (void*)lm.kv_rot, (void*)lm.kv_exp, (void*)lm.dec_part, (void*)lm.chunks})
         if (p) cudaFree(p);
     delete m->layered;
     m->layered = nullptr;

@@ -9,6 +9,7 @@
 #include <cstring>
 
 #include "engine.h"
+#include "layer_kernels.h"
 
 int32_t b2_cache_reserve(b2_cache* c, int n);
 void b2_cache_commit(b2_cache* c, int n);
@@ -332,7 +333,7 @@ int32_t b2_engine_forward(b2_model* m, std::vector<SeqStep>& seqs, void* logits_
     int W = 0, P = 0;
     double pf_flops = 0;  // 4*hd*hq flops per (query, visible key) pair
     int pf_max_ctx = 0;   // longest context among the sequences that prefill in this step
-    int pf_ctx = 0;
+    int pf_ctx = 0, n_chunks = 0;
     double pf_pairs = 0;
     for (auto& s : seqs) {
         if (s.n > 1) {
@@ -350,7 +351,7 @@ int32_t b2_engine_forward(b2_model* m, std::vector<SeqStep>& seqs, void* logits_
     }
     if (all_positions) n_logits = T;  // rows 0..T-1 of the step, in order
     const int U = (int)pool->upd_slot.size();
-    const size_t stage_ints = 4 * (size_t)B + 3 * (size_t)U + (size_t)T + (listed ? (size_t)n_logits : 0) + (m->layered ? (size_t)B : 0);
+    const size_t stage_ints = 4 * (size_t)B + 3 * (size_t)U + (size_t)T + (listed ? (size_t)n_logits : 0) + (m->layered ? 2 * (size_t)B : 0);
     B2_CHECK(ensure_workspace(m, T, std::max(B, n_logits), W, P, stage_ints));
     Workspace& w = m->ws;
     int32_t* sh = w.stage_host;
@@ -386,6 +387,10 @@ int32_t b2_engine_forward(b2_model* m, std::vector<SeqStep>& seqs, void* logits_
             for (auto& s : seqs) {
                 *ids++ = s.n > 1 ? row0 : -1;
                 if (s.n > 1) row0 += s.cache->len + s.n;
+            }
+            for (auto& s : seqs) {
+                *ids++ = s.n >= kMemoryChunkMin ? n_chunks : -1;
+                if (s.n >= kMemoryChunkMin) n_chunks += (s.n + kMemoryChunk - 1) / kMemoryChunk;
             }
         }
     }
@@ -435,7 +440,8 @@ int32_t b2_engine_forward(b2_model* m, std::vector<SeqStep>& seqs, void* logits_
         ls.pf_work = P;
         ls.chunk_tiles = chunk_tiles;
         ls.max_ctx = max_pos;
-        for (auto& s : seqs) ls.max_n = std::max(ls.max_n, s.n);
+        ls.n_chunks = n_chunks;
+        ls.chunk_off = ids_dev + T + (listed ? n_logits : 0) + B;
         ls.dec_ctx_sum = dec_ctx_sum;
         ls.pf_pairs = pf_pairs;
         ls.pf_ctx = pf_ctx;

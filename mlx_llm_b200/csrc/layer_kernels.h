@@ -219,14 +219,15 @@ struct MemoryParams {
     int ld_v;
     float *lg, *beta;       // [T, decays()] logarithms of the decays; [T, heads]
     float* o;               // [T, heads * vdim]
-    void* chunk;            // scratch of the chunked form, b2_memory_chunk_bytes(T)
-    int max_n;              // longest portion of the step
-    bool chunked;           // set by the launcher: longer portions belong to the chunked form
+    // chunked form, for portions of at least kMemoryChunkMin tokens
+    int n_chunks;           // 64-token chunks of those portions; 0: every portion goes token by token
+    const int32_t* chunk_off;  // [B] a portion's first chunk, -1 for the shorter ones
+    void* chunk;            // scratch, n_chunks * b2_memory_chunk_bytes()
 };
 int32_t b2_memory_launch(b2_ctx* ctx, bool f32, const MemorySpec& s, const MemoryParams& p);
-constexpr int kMemoryChunkMin = 12;  // shortest portion that the chunked form takes
+constexpr int kMemoryChunk = 64, kMemoryChunkMin = 12;  // tokens per chunk; shortest portion that the chunked form takes
 bool b2_memory_chunk_eligible(const MemorySpec& s);
-size_t b2_memory_chunk_bytes(const MemorySpec& s, size_t tokens);
+size_t b2_memory_chunk_bytes(const MemorySpec& s);  // per chunk
 int32_t b2_memory_chunk_launch(b2_ctx* ctx, const MemorySpec& s, const MemoryParams& p);
 // Input row of a layer's output projection: attention heads (already there), memory heads (norm, gate), feed-forward (gelu);
 // everything else zero.

@@ -209,7 +209,7 @@ __global__ void __launch_bounds__(128) memory_scan_kernel(const MemorySpec s, co
     const int D = s.dim, P = s.vdim, Q = s.q_cols(), V = s.heads * P;
     const int tid = threadIdx.x, pr = tid >> 3, ln = tid & 7;
     const int start = p.cu_seqlens[b], n = p.cu_seqlens[b + 1] - start, before = p.context_lens[b] - n;
-    if (n <= 0 || (p.chunked && n >= kMemoryChunkMin)) return;
+    if (n <= 0 || (p.n_chunks > 0 && n >= kMemoryChunkMin)) return;
     float* slot = p.state + (size_t)p.seq_slot[b] * p.slot_stride;
     const bool live = p0 + pr < P, vec = D % 4 == 0;
     float* S = slot + ((size_t)h * P + p0 + pr) * D;
@@ -397,13 +397,11 @@ int32_t launch_memory(b2_ctx* ctx, const MemorySpec& s, const MemoryParams& p) {
         B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, memory_rotate_kernel<T>, dim3(p.T), dim3(256), 0, ctx->stream, s, p));
         B2_LAUNCHED(ctx);
     }
-    MemoryParams q = p;
-    q.chunked = sizeof(T) == 2 && p.max_n >= kMemoryChunkMin && b2_memory_chunk_eligible(s);
-    if (q.chunked) B2_CHECK(b2_memory_chunk_launch(ctx, s, q));
-    if (!q.chunked || p.B > 1) {
+    if (p.n_chunks > 0) B2_CHECK(b2_memory_chunk_launch(ctx, s, p));
+    if (p.n_chunks == 0 || p.B > 1) {
         const int k4 = (s.dim + 31) / 32;
         auto k = k4 <= 1 ? memory_scan_kernel<T, 1> : k4 <= 2 ? memory_scan_kernel<T, 2> : k4 <= 4 ? memory_scan_kernel<T, 4> : memory_scan_kernel<T, 8>;
-        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, k, dim3((s.vdim + SC_P - 1) / SC_P, s.heads, p.B), dim3(128), 0, ctx->stream, s, q));
+        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, k, dim3((s.vdim + SC_P - 1) / SC_P, s.heads, p.B), dim3(128), 0, ctx->stream, s, p));
         B2_LAUNCHED(ctx);
     }
     return B2_OK;
