@@ -73,6 +73,25 @@ def layered_config(size, pairs, vocab=32000):
     return dict(architecture="Zukitar", width=s["width"], vocab=vocab, norm=dict(eps=1e-5), logit_scale=1.0, layers=layers)
 
 
+# Tirezen at the same widths: half of the layers with capped sink attention beside a delta memory, the others retention and
+# delta memories in turn; the feed-forward has the flat twin's inner size.
+TIREZEN_SIZES = {
+    "w4096": dict(heads=32, kv_heads=8, memory=dict(heads=32, kv_heads=32), delta=dict(heads=32, kv_heads=16)),
+    "w2048": dict(heads=16, kv_heads=4, memory=dict(heads=16, kv_heads=16), delta=dict(heads=16, kv_heads=8)),
+}
+
+
+def tirezen_config(size, layers, vocab=32000):
+    s, t = LAYERED_SIZES[size], TIREZEN_SIZES[size]
+    left = dict(heads=t["heads"], kv_heads=t["kv_heads"], dim=128, vdim=128, rot=dict(base=500000.0, dims=128), scale=128 ** -0.5, softcap=30.0)
+    sides = dict(left=left, right=dict(t["memory"], dim=128, vdim=128, conv=4), left_scale=0.5, right_scale=0.5)
+    retention = dict(heads=t["heads"], dim=128, vdim=128, rot=dict(base=500000.0, dims=128), decay=[1.0 - 2.0 ** -(5 + i % 7) for i in range(t["heads"])])
+    mixers = [("parallel", sides), ("retention", retention), ("parallel", sides), ("delta", dict(t["delta"], dim=128, vdim=128, conv=4))]
+    mlp = dict(kind="dense", ff=s["ff"])
+    return dict(architecture="Tirezen", width=s["width"], vocab=vocab, norm=dict(eps=1e-5),
+                layers=[dict(type=mixers[i % 4][0], mixer=mixers[i % 4][1], mlp=mlp) for i in range(layers)])
+
+
 def flat_twin(size, layers, vocab=32000):
     """Llama-architecture model of the same width, feed-forward and layer count, dense bf16."""
     s = LAYERED_SIZES[size]
