@@ -8,13 +8,14 @@ namespace {
 constexpr int kMaxHead = 256;
 
 // A warp per (token, head of q, k or v): bias, norm over the head, rotation of the pairs (i, i + dims/2), store.  A lane holds
-// VEC consecutive values of every 32 * VEC; the rotation finds its partner in shared memory.
-template <typename T, int VEC>
+// VEC consecutive values of every 32 * VEC; the rotation finds its partner in shared memory
+// (N 1, VEC 4: heads of up to 128, the partner comes by shuffle).
+template <typename T, int VEC, int N>
 __global__ void __launch_bounds__(256) gqa_prep_kernel(const GroupedAttnSpec a, const GqaPrepParams p) {
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     pdl_wait();
-    __shared__ __align__(16) float rows[8][kMaxHead];
-    constexpr int N = kMaxHead / (32 * VEC);
+    constexpr bool SHUFFLE = N == 1 && VEC == 4;
+    __shared__ __align__(16) float rows[SHUFFLE ? 1 : 8][SHUFFLE ? 4 : kMaxHead];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, units = a.heads + 2 * a.kv_heads;
     const int id = blockIdx.x * 8 + warp, t = id / units, u = id - t * units;
     if (t >= p.T) return;
@@ -43,11 +44,18 @@ __global__ void __launch_bounds__(256) gqa_prep_kernel(const GroupedAttnSpec a, 
             Elt<T>::ld4(src + d, v[i]);
         else
             v[i][0] = Elt<T>::ld(src + d);
+        if (bias) {
+            if constexpr (VEC == 4) {
+                float x[4];
+                Elt<float>::ld4(bias + h * n + d, x);
 #pragma unroll
-        for (int e = 0; e < VEC; e++) {
-            if (bias) v[i][e] += bias[h * n + d + e];
-            ss += v[i][e] * v[i][e];
+                for (int e = 0; e < 4; e++) v[i][e] += x[e];
+            } else {
+                v[i][0] += bias[h * n + d];
+            }
         }
+#pragma unroll
+        for (int e = 0; e < VEC; e++) ss += v[i][e] * v[i][e];
     }
     if (w) {
         const float inv = 1.0f / sqrtf(elt_warp_sum(ss) / (float)n + p.eps);
@@ -59,7 +67,21 @@ __global__ void __launch_bounds__(256) gqa_prep_kernel(const GroupedAttnSpec a, 
                 if (d < n) v[i][e] = v[i][e] * inv * w[d];
             }
     }
-    if (half > 0) {
+    if constexpr (SHUFFLE) {
+        if (half > 0) {  // (half is a multiple of four)
+            const int d = lane * 4, src_lane = d < half ? lane + half / 4 : lane - half / 4;
+            float o[4], c[4] = {1.f, 1.f, 1.f, 1.f}, sn[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+            for (int e = 0; e < 4; e++) o[e] = __shfl_sync(0xffffffffu, v[0][e], src_lane & 31);
+            if (d < dims) {
+                const size_t at = (size_t)p.positions[t] * half + (d < half ? d : d - half);
+                Elt<float>::ld4(p.cos_t + at, c);
+                Elt<float>::ld4(p.sin_t + at, sn);
+#pragma unroll
+                for (int e = 0; e < 4; e++) v[0][e] = d < half ? v[0][e] * c[e] - o[e] * sn[e] : v[0][e] * c[e] + o[e] * sn[e];
+            }
+        }
+    } else if (half > 0) {
         const float* ct = p.cos_t + (size_t)p.positions[t] * half;
         const float* st = p.sin_t + (size_t)p.positions[t] * half;
 #pragma unroll
@@ -146,7 +168,10 @@ int32_t b2_gqa_prep_launch(b2_ctx* ctx, bool f32, const GroupedAttnSpec& a, cons
     B2_REQUIRE(a.dim <= kMaxHead && a.vdim <= kMaxHead, B2_ERR_UNSUPPORTED, "grouped attention: head sizes up to 256");
     const bool vec = a.dim % 4 == 0 && a.vdim % 4 == 0 && p.q_off % 4 == 0 && p.k_off % 4 == 0 && p.v_off % 4 == 0 && p.ld % 4 == 0;
     const dim3 grid((unsigned)(((size_t)p.T * (a.heads + 2 * a.kv_heads) + 7) / 8));
-    auto k = f32 ? (vec ? gqa_prep_kernel<float, 4> : gqa_prep_kernel<float, 1>) : (vec ? gqa_prep_kernel<uint16_t, 4> : gqa_prep_kernel<uint16_t, 1>);
+    const bool small = a.dim <= 128 && a.vdim <= 128 && a.rot.dims % 8 == 0;
+    auto k = !vec    ? (f32 ? gqa_prep_kernel<float, 1, 8> : gqa_prep_kernel<uint16_t, 1, 8>)
+             : small ? (f32 ? gqa_prep_kernel<float, 4, 1> : gqa_prep_kernel<uint16_t, 4, 1>)
+                     : (f32 ? gqa_prep_kernel<float, 4, 2> : gqa_prep_kernel<uint16_t, 4, 2>);
     B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, k, grid, dim3(256), 0, ctx->stream, a, p));
     B2_LAUNCHED(ctx);
     return B2_OK;

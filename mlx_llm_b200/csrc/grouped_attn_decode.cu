@@ -77,6 +77,7 @@ __global__ void __launch_bounds__(kWarps * 32) gqa_decode_kernel(const GroupedAt
         const int key = (tile0 + warp + min(i, max(n_my - 1, 0)) * kWarps) * 16, k = key < ctx ? key : 0;
         return ((size_t)bt[k / p.page_size] * a.kv_heads + kvh) * p.page_size + k % p.page_size;
     };
+    const int kr0 = lane / (KR / 8), kx0 = lane - kr0 * (KR / 8), vr0 = lane / (VR / 8), vx0 = lane - vr0 * (VR / 8);
     size_t next = page_row(0);  // looked up one tile ahead
     auto issue = [&](int i) {
         const size_t r0 = next;
@@ -84,15 +85,17 @@ __global__ void __launch_bounds__(kWarps * 32) gqa_decode_kernel(const GroupedAt
         const uint32_t dst = wsm + (i % kStages) * stage;
         const uint8_t* ks = reinterpret_cast<const uint8_t*>(p.k_cache) + r0 * KR * 2;
         const uint8_t* vs = reinterpret_cast<const uint8_t*>(p.v_cache) + r0 * VR * 2;
-        const int kc = KR / 8, vc = VR / 8;  // 16-byte pieces per row
-        for (int c = lane; c < 16 * kc; c += 32) {
-            const int r = c / kc, x = c - r * kc;
-            cp_async16(dst + r * krow + ((x ^ (r & 7)) << 4), ks + (size_t)c * 16);
-        }
-        for (int c = lane; c < 16 * vc; c += 32) {
-            const int r = c / vc, x = c - r * vc;
-            cp_async16(dst + 16 * krow + r * vrow + ((x ^ (r & 7)) << 4), vs + (size_t)c * 16);
-        }
+        auto copy = [&](uint32_t to, int row_bytes, const uint8_t* from, int pieces, int r, int x) {  // 16-byte pieces of 16 rows
+            const int dr = 32 / pieces, dx = 32 - dr * pieces;
+            for (int c = lane; c < 16 * pieces; c += 32) {
+                cp_async16(to + r * row_bytes + ((x ^ (r & 7)) << 4), from + (size_t)c * 16);
+                r += dr;
+                x += dx;
+                if (x >= pieces) x -= pieces, r++;
+            }
+        };
+        copy(dst, krow, ks, KR / 8, kr0, kx0);
+        copy(dst + 16 * krow, vrow, vs, VR / 8, vr0, vx0);
     };
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f, o[NB][4];
 #pragma unroll

@@ -14,8 +14,9 @@ namespace {
 
 __device__ __forceinline__ float softplus_f32(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 
-// Queries and keys of a memory without convolution: rotated (pairs (i, i + dims/2)), keys times dim^-1/2, as f32.
-template <typename T>
+// Queries and keys of a memory without convolution: rotated (pairs (i, i + dims/2)), keys times dim^-1/2, as f32.  VEC
+// consecutive values per thread.
+template <typename T, int VEC>
 __global__ void __launch_bounds__(256) memory_rotate_kernel(const MemorySpec s, const MemoryParams p) {
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     pdl_wait();
@@ -24,17 +25,37 @@ __global__ void __launch_bounds__(256) memory_rotate_kernel(const MemorySpec s, 
     const float* ct = p.cos_t + (size_t)p.positions[t] * half;
     const float* st = p.sin_t + (size_t)p.positions[t] * half;
     const float scale = rsqrtf((float)D);
-    for (int i = threadIdx.x; i < 2 * Q; i += 256) {
-        const int c = i < Q ? i : i - Q, d = c % D;
-        float v = Elt<T>::ld(src + i);
-        if (d < half)
-            v = v * ct[d] - Elt<T>::ld(src + i + half) * st[d];
-        else if (d < dims)
-            v = v * ct[d - half] + Elt<T>::ld(src + i - half) * st[d - half];
-        if (i < Q)
-            p.q[(size_t)t * Q + c] = v;
+    auto load = [&](const T* x, float (&v)[VEC]) {
+        if constexpr (VEC == 4)
+            Elt<T>::ld4(x, v);
         else
-            p.k[(size_t)t * Q + c] = v * scale;
+            v[0] = Elt<T>::ld(x);
+    };
+    for (int i = (blockIdx.y * 256 + threadIdx.x) * VEC; i < 2 * Q; i += gridDim.y * 256 * VEC) {
+        const int c = i < Q ? i : i - Q, d = c % D;
+        float v[VEC], o[VEC];
+        load(src + i, v);
+        if (d < dims) {
+            const bool low = d < half;
+            float cs[VEC], sn[VEC];
+            load(src + (low ? i + half : i - half), o);
+            if constexpr (VEC == 4) {
+                Elt<float>::ld4(ct + (low ? d : d - half), cs);
+                Elt<float>::ld4(st + (low ? d : d - half), sn);
+            } else {
+                cs[0] = ct[low ? d : d - half], sn[0] = st[low ? d : d - half];
+            }
+#pragma unroll
+            for (int e = 0; e < VEC; e++) v[e] = low ? v[e] * cs[e] - o[e] * sn[e] : v[e] * cs[e] + o[e] * sn[e];
+        }
+        float* dst = (i < Q ? p.q : p.k) + (size_t)t * Q + c;
+        if (i >= Q)
+#pragma unroll
+            for (int e = 0; e < VEC; e++) v[e] *= scale;
+        if constexpr (VEC == 4)
+            Elt<float>::st4(dst, v);
+        else
+            dst[0] = v[0];
     }
 }
 
@@ -53,11 +74,27 @@ __global__ void __launch_bounds__(256) memory_prep_kernel(const MemorySpec s, co
         const int h = u - n_conv;
         if (s.decay == MemDecay::PerChannel && h < s.heads) {
             const float A = -expf(p.A_log[h]);
-            for (int t = t0; t < t1; t++)
-                for (int d = lane; d < s.dim; d += 32) {
-                    const int c = h * s.dim + d;
-                    p.lg[(size_t)t * s.decays() + c] = A * softplus_f32(Elt<T>::ld(reinterpret_cast<const T*>(p.dec) + (size_t)t * p.ld_dec + c) + p.dt_bias[c]);
+            const T* dec = reinterpret_cast<const T*>(p.dec) + h * s.dim;
+            float* lg = p.lg + h * s.dim;
+            for (int d = lane * VEC; d < s.dim; d += 32 * VEC) {
+                float bias[VEC];
+#pragma unroll
+                for (int e = 0; e < VEC; e++) bias[e] = p.dt_bias[h * s.dim + d + e];
+#pragma unroll 4
+                for (int t = t0; t < t1; t++) {
+                    float v[VEC];
+                    if constexpr (VEC == 4)
+                        Elt<T>::ld4(dec + (size_t)t * p.ld_dec + d, v);
+                    else
+                        v[0] = Elt<T>::ld(dec + (size_t)t * p.ld_dec + d);
+#pragma unroll
+                    for (int e = 0; e < VEC; e++) v[e] = A * softplus_f32(v[e] + bias[e]);
+                    if constexpr (VEC == 4)
+                        Elt<float>::st4(lg + (size_t)t * s.decays() + d, v);
+                    else
+                        lg[(size_t)t * s.decays() + d] = v[0];
                 }
+            }
         } else if (h == (s.decay == MemDecay::PerChannel ? s.heads : 0)) {
             for (int t = t0; t < t1; t++)
                 for (int i = lane; i < s.heads; i += 32) {
@@ -96,8 +133,13 @@ __global__ void __launch_bounds__(256) memory_prep_kernel(const MemorySpec s, co
                 w[j][i][e] = TAPS > 0 && d < n ? p.conv_w[(size_t)j * C + c0 + d] : 0.f;
                 win[j][i][e] = 0.f;
             }
+    float next[NCH][VEC];  // the input of the token after this one is on its way
+    if constexpr (TAPS > 0) {
+        if (t0 < t1) fetch(t0, next);
+    }
     int cur = -1, start = 0, before = 0;
     const float* kept = nullptr;
+#pragma unroll 4
     for (int t = t0; t < t1; t++) {
         const int b = p.token_seq[t];
         if (b != cur) {
@@ -131,7 +173,11 @@ __global__ void __launch_bounds__(256) memory_prep_kernel(const MemorySpec s, co
                 for (int i = 0; i < NCH; i++)
 #pragma unroll
                     for (int e = 0; e < VEC; e++) win[j][i][e] = win[j + 1][i][e];
-            fetch(t, win[TAPS - 1]);
+#pragma unroll
+            for (int i = 0; i < NCH; i++)
+#pragma unroll
+                for (int e = 0; e < VEC; e++) win[TAPS - 1][i][e] = (i * 32 + lane) * VEC < n ? next[i][e] : 0.f;
+            if (t + 1 < t1) fetch(t + 1, next);
 #pragma unroll
             for (int i = 0; i < NCH; i++)
 #pragma unroll
@@ -386,7 +432,7 @@ int32_t launch_prep(b2_ctx* ctx, const MemorySpec& s, const MemoryParams& p) {
 template <typename T>
 int32_t launch_memory(b2_ctx* ctx, const MemorySpec& s, const MemoryParams& p) {
     if (s.conv > 0) {
-        const bool vec = s.dim % 4 == 0 && (s.heads * s.vdim) % 4 == 0 && p.c_off % 4 == 0 && p.ld % 4 == 0 && p.ld_v % 4 == 0;
+        const bool vec = s.dim % 4 == 0 && (s.heads * s.vdim) % 4 == 0 && p.ld_dec % 4 == 0 && p.c_off % 4 == 0 && p.ld % 4 == 0 && p.ld_v % 4 == 0;
         if (!vec)
             B2_CHECK((launch_prep<T, 1, 8>(ctx, s, p)));
         else if (s.dim <= 128)
@@ -394,7 +440,9 @@ int32_t launch_memory(b2_ctx* ctx, const MemorySpec& s, const MemoryParams& p) {
         else
             B2_CHECK((launch_prep<T, 4, 2>(ctx, s, p)));
     } else {
-        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, memory_rotate_kernel<T>, dim3(p.T), dim3(256), 0, ctx->stream, s, p));
+        const bool vec = s.dim % 4 == 0 && s.rot.dims % 8 == 0 && p.c_off % 4 == 0 && p.ld % 4 == 0;
+        const int by = (2 * s.q_cols() / (vec ? 4 : 1) + 1023) / 1024;  // up to four pieces per thread
+        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, vec ? memory_rotate_kernel<T, 4> : memory_rotate_kernel<T, 1>, dim3(p.T, by), dim3(256), 0, ctx->stream, s, p));
         B2_LAUNCHED(ctx);
     }
     if (p.n_chunks > 0) B2_CHECK(b2_memory_chunk_launch(ctx, s, p));

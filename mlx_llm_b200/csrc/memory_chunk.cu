@@ -47,29 +47,37 @@ __device__ __forceinline__ void mma3(float (&d)[4], const uint32_t (&ah)[4], con
 }
 
 // ---- factors ---------------------------------------------------------------------------------------------------------
+// Decays per channel: with r_i the sums before 16-token block i and e_i those at its end, the exponent of token t of block i
+// and an earlier token s of block j splits into
+//     G_t - G_s = (G_t - r_i) + (r_i - e_j) + (e_j - G_s)
+// The outer two belong to one token each and are at most zero; the middle one is a number per channel and pair of blocks, at
+// most zero but for i = j, where it undoes the block's own decay.  A block whose decay is too strong for that (beyond 2^-80
+// inside 16 tokens) takes every exponent from its difference instead.
 constexpr int F_WARPS = 10, F_THREADS = F_WARPS * 32;  // a warp per 16 x 16 tile of P and A up to the diagonal
-constexpr float kMaxSpread = 80.f;  // log2 units: largest decay inside 16 tokens whose inverse is used as a factor
+constexpr float kMaxSpread = 80.f;  // log2 units
 template <int DK, bool CHANNEL>
 struct FactorSmem {
-    static constexpr int LD = DK + 4, LM = C + 4;
-    static constexpr int K = 0, G = K + C * LD * 4, M = G + (CHANNEL ? C * LD * 4 : C * 4), Y = M + C * LM * 4, BETA = Y + 3 * 16 * 17 * 4, kBytes = BETA + C * 4;
+    static constexpr int LD = DK + 4, LM = C + 4, kOp = C * DK * 2;
+    // left operands (k, q; head and remainder), then the right one in f32, whose place A and its inverse take later
+    static constexpr int LK = 0, LQ = 2 * kOp, G = 4 * kOp, kG = CHANNEL ? C * LD * 4 : 0, kM = C * LM * 4;
+    static constexpr int M = G, Y = G + (kG > kM ? kG : kM), REF = Y + 3 * 16 * 17 * 4, BETA = REF + (CHANNEL ? 5 * DK * 4 : C * 4), kBytes = BETA + C * 4;
 };
 
 template <int DK, bool CHANNEL>
-__global__ void __launch_bounds__(F_THREADS) memory_factor_kernel(const MemorySpec s, const MemoryParams p) {
+__global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const MemorySpec s, const MemoryParams p) {
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     pdl_wait();
     using L = FactorSmem<DK, CHANNEL>;
     using R = Record<DK>;
     constexpr int LD = L::LD, LM = L::LM;
     extern __shared__ __align__(16) uint8_t smem[];
-    float* ks = reinterpret_cast<float*>(smem + L::K);    // [C][LD] keys
-    float* gs = reinterpret_cast<float*>(smem + L::G);    // [C][LD] or [C]: running sums of the decays' logarithms (base 2)
-    float* M = reinterpret_cast<float*>(smem + L::M);     // [C][LM]: A below the diagonal, the transposed inverse above it
-    float* Y = reinterpret_cast<float*>(smem + L::Y);     // [3][16][17]
+    float* gs = reinterpret_cast<float*>(smem + L::G);      // CHANNEL: [C][LD] running sums (base 2), then k e^(e_j - G_s)
+    float* M = reinterpret_cast<float*>(smem + L::M);       // [C][LM]: A below the diagonal, the transposed inverse above it
+    float* Y = reinterpret_cast<float*>(smem + L::Y);       // [3][16][17]
+    float* ref = reinterpret_cast<float*>(smem + L::REF);   // CHANNEL: [5][DK] sums at the blocks' borders; else [C] running sums
     float* betas = reinterpret_cast<float*>(smem + L::BETA);
-    __shared__ int wide[4];                               // 16-token blocks whose decays do not allow inverse factors
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g4 = lane >> 2, t4 = lane & 3;
+    __shared__ int wide[4];                                 // blocks with strong decays
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g4 = lane >> 2, t4 = lane & 3, mi = lane >> 3, lr = lane & 7;
     const int chunk = blockIdx.x, h = blockIdx.y, D = s.dim, Q = s.q_cols(), kh = h / (s.heads / s.kv_heads);
     int b = -1;  // the last chunked portion that starts at or before this chunk (starts rise with the index)
     for (int i = lane; i < p.B; i += 32)
@@ -77,176 +85,243 @@ __global__ void __launch_bounds__(F_THREADS) memory_factor_kernel(const MemorySp
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) b = max(b, __shfl_xor_sync(0xffffffffu, b, o));
     if (b < 0) return;
-    const int n = p.cu_seqlens[b + 1] - p.cu_seqlens[b], t0 = (chunk - p.chunk_off[b]) * C, cnt = min(C, n - t0);
+    const int n = p.cu_seqlens[b + 1] - p.cu_seqlens[b], t0 = (chunk - p.chunk_off[b]) * C, cnt = min(C, n - t0), last = cnt - 1;
     if (cnt <= 0) return;
     const size_t tok0 = (size_t)p.cu_seqlens[b] + t0;
     uint8_t* rec = reinterpret_cast<uint8_t*>(p.chunk) + ((size_t)chunk * s.heads + h) * R::kBytes;
-    const float* q = p.q + tok0 * Q + kh * D;
+    const float *q = p.q + tok0 * Q + kh * D, *k = p.k + tok0 * Q + kh * D;
+    const float* lg = CHANNEL ? p.lg + tok0 * s.decays() + h * D : nullptr;
 
     if (tid < 4) wide[tid] = 0;
-    for (int i = tid; i < C * DK; i += F_THREADS) {
-        const int t = i / DK, d = i % DK;
-        const bool ok = t < cnt && d < D;
-        ks[t * LD + d] = ok ? p.k[(tok0 + t) * Q + kh * D + d] : 0.f;
-        if constexpr (CHANNEL) gs[t * LD + d] = ok ? p.lg[(tok0 + t) * s.decays() + h * D + d] * kLog2e : 0.f;
-    }
-    if (!CHANNEL && tid < C) gs[tid] = tid < cnt ? (s.decay == MemDecay::Fixed ? p.log_decay[h] : p.lg[(tok0 + tid) * s.heads + h]) * kLog2e : 0.f;
     if (tid < C) betas[tid] = s.delta && tid < cnt ? p.beta[(tok0 + tid) * s.heads + h] : 0.f;
     __syncthreads();
-    if constexpr (CHANNEL) {
-        if (tid < DK) {
-            float run = 0.f;
-            for (int i = 0; i < 4; i++) {
-                const float ref = run;
+    if constexpr (CHANNEL) {  // a thread per channel and half of the chunk; the second half is raised by the first one's end
+        constexpr int H = C / 2;
+        const int d = tid % DK, half = tid / DK;
+        if (half < 2) {
+            float run = 0.f, x[16];
+#pragma unroll
+            for (int i = 0; i < H / 16; i++) {
 #pragma unroll
                 for (int t = 0; t < 16; t++) {
-                    run += gs[(16 * i + t) * LD + tid];
-                    gs[(16 * i + t) * LD + tid] = run;
+                    const int tok = half * H + 16 * i + t;
+                    x[t] = tok < cnt && d < D ? lg[(size_t)tok * s.decays() + d] : 0.f;
                 }
-                if (ref - run > kMaxSpread) atomicOr(&wide[i], 1);
+                const float before = run;
+#pragma unroll
+                for (int t = 0; t < 16; t++) {
+                    run = fmaf(x[t], kLog2e, run);
+                    gs[(half * H + 16 * i + t) * LD + d] = run;
+                }
+                ref[(half * 2 + i + 1) * DK + d] = run;
+                if (before - run > kMaxSpread) atomicOr(&wide[half * 2 + i], 1);
             }
         }
+        __syncthreads();
+        if (half == 0) {
+            ref[d] = 0.f;
+            const float first = ref[2 * DK + d];
+            ref[3 * DK + d] += first;
+            ref[4 * DK + d] += first;
+        }
     } else if (tid < 32) {
-        float a = gs[2 * tid], c = gs[2 * tid + 1], sum = a + c;
+        auto at = [&](int t) { return t < cnt ? (s.decay == MemDecay::Fixed ? p.log_decay[h] : p.lg[(tok0 + t) * s.heads + h]) * kLog2e : 0.f; };
+        const float x = at(2 * tid), y = at(2 * tid + 1);
+        float sum = x + y;
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
             const float u = __shfl_up_sync(0xffffffffu, sum, o);
             if (tid >= o) sum += u;
         }
-        gs[2 * tid] = sum - c;
-        gs[2 * tid + 1] = sum;
+        ref[2 * tid] = sum - y;
+        ref[2 * tid + 1] = sum;
+    }
+    __syncthreads();
+
+    // ---- one pass over the chunk, eight columns at a time: the tiles' operands and the walk's
+    const bool vec = D % 4 == 0 && Q % 4 == 0;
+    for (int i = tid; i < C * (DK / 8); i += F_THREADS) {
+        const int t = i / (DK / 8), x = i % (DK / 8), blk = t >> 4;
+        float kv[8], qv[8], left[8], right[8], a[8];
+#pragma unroll
+        for (int e = 0; e < 8; e += 4) {
+            const int d = x * 8 + e;
+            if (vec) {
+                const bool ok = t < cnt && d < D;
+                const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
+                const float4 k4 = ok ? *reinterpret_cast<const float4*>(k + (size_t)t * Q + d) : z, q4 = ok ? *reinterpret_cast<const float4*>(q + (size_t)t * Q + d) : z;
+                kv[e] = k4.x, kv[e + 1] = k4.y, kv[e + 2] = k4.z, kv[e + 3] = k4.w;
+                qv[e] = q4.x, qv[e + 1] = q4.y, qv[e + 2] = q4.z, qv[e + 3] = q4.w;
+            } else {
+#pragma unroll
+                for (int f = 0; f < 4; f++) {
+                    const bool ok = t < cnt && d + f < D;
+                    kv[e + f] = ok ? k[(size_t)t * Q + d + f] : 0.f;
+                    qv[e + f] = ok ? q[(size_t)t * Q + d + f] : 0.f;
+                }
+            }
+        }
+        const uint32_t o = at_wide(t, x, DK * 2);
+        auto store = [&](uint8_t* base, const float (&v)[8]) {
+            Split w[4];
+#pragma unroll
+            for (int e = 0; e < 4; e++) w[e] = split2(v[2 * e], v[2 * e + 1]);
+            *reinterpret_cast<uint4*>(base + o) = make_uint4(w[0].hi, w[1].hi, w[2].hi, w[3].hi);
+            *reinterpret_cast<uint4*>(base + R::kOp + o) = make_uint4(w[0].lo, w[1].lo, w[2].lo, w[3].lo);
+        };
+        if constexpr (CHANNEL) {
+            float r0[8], tail[8];  // e^(r_i), e^(G_end - e_i)
+#pragma unroll
+            for (int e = 0; e < 8; e++) {
+                const int d = x * 8 + e;
+                const float r = ref[blk * DK + d], end = ref[(blk + 1) * DK + d], g = gs[t * LD + d] + (blk >= 2 ? ref[2 * DK + d] : 0.f);
+                left[e] = fast_exp2(g - r);
+                right[e] = kv[e] * fast_exp2(end - g);
+                r0[e] = fast_exp2(r);
+                tail[e] = fast_exp2(ref[4 * DK + d] - end);
+                gs[t * LD + d] = right[e];
+            }
+#pragma unroll
+            for (int e = 0; e < 8; e++) a[e] = kv[e] * left[e];
+            if (s.delta) {
+                store(smem + L::LK, a);
+#pragma unroll
+                for (int e = 0; e < 8; e++) a[e] *= r0[e];
+                store(rec + R::Kf, a);
+            }
+#pragma unroll
+            for (int e = 0; e < 8; e++) a[e] = qv[e] * left[e];
+            store(smem + L::LQ, a);
+#pragma unroll
+            for (int e = 0; e < 8; e++) a[e] *= r0[e];
+            store(rec + R::Qf, a);
+#pragma unroll
+            for (int e = 0; e < 8; e++) a[e] = right[e] * tail[e];
+            store(rec + R::Kb, a);
+        } else {
+            const float f = fast_exp2(ref[t]), w = fast_exp2(ref[last] - ref[min(t, last)]);
+            store(smem + L::LK, kv);
+            store(smem + L::LQ, qv);
+#pragma unroll
+            for (int e = 0; e < 8; e++) a[e] = kv[e] * f;
+            if (s.delta) store(rec + R::Kf, a);
+#pragma unroll
+            for (int e = 0; e < 8; e++) a[e] = qv[e] * f;
+            store(rec + R::Qf, a);
+#pragma unroll
+            for (int e = 0; e < 8; e++) a[e] = kv[e] * w;
+            store(rec + R::Kb, a);
+        }
     }
     __syncthreads();
 
     // ---- P and A, a 16 x 16 tile (tokens 16 i .., earlier tokens 16 j ..) per warp
-    {
-        int i = 0, j = warp;
-        while (j > i) j -= ++i;
-        float a[2][4], pr[2][4];
+    int i = 0, j = warp;
+    while (j > i) j -= ++i;
+    float a[2][4], pr[2][4];
 #pragma unroll
-        for (int half = 0; half < 2; half++)
+    for (int half = 0; half < 2; half++)
 #pragma unroll
-            for (int e = 0; e < 4; e++) a[half][e] = pr[half][e] = 0.f;
-        const int ta = 16 * i + g4, tb = ta + 8;
-        if (CHANNEL && i == j && wide[i]) {
-            // strong decays inside the block: every exponent from its difference, lanes over the channels
+        for (int e = 0; e < 4; e++) a[half][e] = pr[half][e] = 0.f;
+    const int ta = 16 * i + g4, tb = ta + 8;
+    if (CHANNEL && i == j && wide[i]) {
+        // lanes over the channels; everything from memory again, this is rare
 #pragma unroll 1
-            for (int t = 16 * i; t < min(16 * i + 16, cnt); t++)
+        for (int u = 16 * i; u < min(16 * i + 16, cnt); u++) {
+            float g[DK / 32], w[DK / 32];
+#pragma unroll
+            for (int x = 0; x < DK / 32; x++) {
+                const int d = x * 32 + lane;
+                g[x] = 0.f;
+                w[x] = d < D ? k[(size_t)u * Q + d] : 0.f;
+            }
 #pragma unroll 1
-                for (int u = 16 * i; u <= t; u++) {
-                    float sa = 0.f, sp = 0.f;
-                    for (int d = lane; d < DK; d += 32) {
-                        const float w = fast_exp2(gs[t * LD + d] - gs[u * LD + d]) * ks[u * LD + d];
-                        sa = fmaf(w, ks[t * LD + d], sa);
-                        sp = fmaf(w, d < D ? q[(size_t)t * Q + d] : 0.f, sp);
-                    }
-                    sa = elt_warp_sum(sa);
-                    sp = elt_warp_sum(sp);
+            for (int t = u; t < min(16 * i + 16, cnt); t++) {
+                float sa = 0.f, sp = 0.f;
 #pragma unroll
-                    for (int half = 0; half < 2; half++)
-#pragma unroll
-                        for (int e = 0; e < 4; e++)
-                            if (t == (e < 2 ? ta : tb) && u == 16 * i + half * 8 + 2 * t4 + (e & 1)) a[half][e] = sa, pr[half][e] = sp;
+                for (int x = 0; x < DK / 32; x++) {
+                    const int d = x * 32 + lane;
+                    if (d >= D) continue;
+                    if (t > u) g[x] = fmaf(lg[(size_t)t * s.decays() + d], kLog2e, g[x]);
+                    const float v = fast_exp2(g[x]) * w[x];
+                    sa = fmaf(v, k[(size_t)t * Q + d], sa);
+                    sp = fmaf(v, q[(size_t)t * Q + d], sp);
                 }
-        } else {
-            const float* ref = gs + (16 * i - 1) * LD;  // the sums before the block's first token
-#pragma unroll 2
-            for (int k = 0; k < DK / 16; k++) {
-                uint32_t kh_[4], kl_[4], qh_[4], ql_[4];
-                float r[4];  // reference at columns d0, d0 + 1, d0 + 8, d0 + 9
-                const int d0 = k * 16 + 2 * t4;
-                if constexpr (CHANNEL) {
+                sa = elt_warp_sum(sa);
+                sp = elt_warp_sum(sp);
 #pragma unroll
-                    for (int e = 0; e < 4; e++) r[e] = i > 0 ? ref[d0 + (e >> 1) * 8 + (e & 1)] : 0.f;
-                }
+                for (int half = 0; half < 2; half++)
 #pragma unroll
-                for (int e = 0; e < 4; e++) {  // fragment e: row (e & 1), columns (e >> 1)
-                    const int t = (e & 1) ? tb : ta, d = d0 + (e >> 1) * 8;
-                    const float2 kv = *reinterpret_cast<const float2*>(ks + t * LD + d);
-                    const float q0 = t < cnt && d < D ? q[(size_t)t * Q + d] : 0.f, q1 = t < cnt && d + 1 < D ? q[(size_t)t * Q + d + 1] : 0.f;
-                    float w0 = 1.f, w1 = 1.f;
-                    if constexpr (CHANNEL) {
-                        const float2 gv = *reinterpret_cast<const float2*>(gs + t * LD + d);
-                        w0 = fast_exp2(gv.x - r[(e >> 1) * 2]), w1 = fast_exp2(gv.y - r[(e >> 1) * 2 + 1]);
-                    }
-                    const Split sk = split2(kv.x * w0, kv.y * w1), sq = split2(q0 * w0, q1 * w1);
-                    kh_[e] = sk.hi, kl_[e] = sk.lo, qh_[e] = sq.hi, ql_[e] = sq.lo;
-                }
-#pragma unroll
-                for (int half = 0; half < 2; half++) {
-                    const int u = 16 * j + half * 8 + g4;
-                    uint32_t bh[2], bl[2];
-#pragma unroll
-                    for (int e = 0; e < 2; e++) {
-                        const int d = d0 + e * 8;
-                        const float2 kv = *reinterpret_cast<const float2*>(ks + u * LD + d);
-                        float w0 = 1.f, w1 = 1.f;
-                        if constexpr (CHANNEL) {
-                            const float2 gv = *reinterpret_cast<const float2*>(gs + u * LD + d);
-                            w0 = fast_exp2(r[e * 2] - gv.x), w1 = fast_exp2(r[e * 2 + 1] - gv.y);
-                        }
-                        const Split sk = split2(kv.x * w0, kv.y * w1);
-                        bh[e] = sk.hi, bl[e] = sk.lo;
-                    }
-                    if (s.delta) mma3(a[half], kh_, kl_, bh, bl);
-                    mma3(pr[half], qh_, ql_, bh, bl);
-                }
+                    for (int e = 0; e < 4; e++)
+                        if (t == (e < 2 ? ta : tb) && u == 16 * i + half * 8 + 2 * t4 + (e & 1)) a[half][e] = sa, pr[half][e] = sp;
             }
         }
+    } else {
+        const uint32_t base = smem_u32(smem);
+#pragma unroll 2
+        for (int kk = 0; kk < DK / 16; kk++) {
+            uint32_t ah[4], al[4], qh[4], ql[4], bh[2][2], bl[2][2];
+            const uint32_t at = at_wide(16 * i + lr + (mi & 1) * 8, 2 * kk + (mi >> 1), DK * 2);
+            if (s.delta) {
+                ldmatrix_x4(ah[0], ah[1], ah[2], ah[3], base + L::LK + at);
+                ldmatrix_x4(al[0], al[1], al[2], al[3], base + L::LK + R::kOp + at);
+            }
+            ldmatrix_x4(qh[0], qh[1], qh[2], qh[3], base + L::LQ + at);
+            ldmatrix_x4(ql[0], ql[1], ql[2], ql[3], base + L::LQ + R::kOp + at);
+            if constexpr (CHANNEL) {
+                const int d0 = kk * 16 + 2 * t4;
 #pragma unroll
-        for (int half = 0; half < 2; half++) {
-            const int u0 = 16 * j + half * 8 + 2 * t4;
+                for (int e = 0; e < 2; e++) {
+                    const int d = d0 + e * 8;
+                    const float2 r = *reinterpret_cast<const float2*>(ref + i * DK + d), en = *reinterpret_cast<const float2*>(ref + (j + 1) * DK + d);
+                    const float f0 = fast_exp2(r.x - en.x), f1 = fast_exp2(r.y - en.y);
 #pragma unroll
-            for (int e = 0; e < 4; e++) {
-                const int t = e < 2 ? ta : tb, u = u0 + (e & 1);
-                if constexpr (!CHANNEL) {
-                    const float w = u <= t ? fast_exp2(gs[t] - gs[u]) : 0.f;
-                    a[half][e] *= w;
-                    pr[half][e] *= w;
+                    for (int half = 0; half < 2; half++) {
+                        const float2 v = *reinterpret_cast<const float2*>(gs + (16 * j + half * 8 + g4) * LD + d);
+                        const Split sp = split2(v.x * f0, v.y * f1);
+                        bh[half][e] = sp.hi, bl[half][e] = sp.lo;
+                    }
                 }
-                if (u > t) pr[half][e] = 0.f;
-                if (s.delta && u < t) M[t * LM + u] = a[half][e] * betas[t];
+            } else {
+                const uint32_t bt = at_wide(16 * j + lr + (mi >> 1) * 8, 2 * kk + (mi & 1), DK * 2);
+                ldmatrix_x4(bh[0][0], bh[0][1], bh[1][0], bh[1][1], base + L::LK + bt);
+                ldmatrix_x4(bl[0][0], bl[0][1], bl[1][0], bl[1][1], base + L::LK + R::kOp + bt);
             }
 #pragma unroll
-            for (int row = 0; row < 2; row++) {
-                const Split sp = split2(pr[half][2 * row], pr[half][2 * row + 1]);
-                const uint32_t o = at_wide(row ? tb : ta, u0 >> 3, 128) + (u0 & 7) * 2;
-                *reinterpret_cast<uint32_t*>(rec + R::P + o) = sp.hi;
-                *reinterpret_cast<uint32_t*>(rec + R::P + R::kMat + o) = sp.lo;
+            for (int half = 0; half < 2; half++) {
+                if (s.delta) mma3(a[half], ah, al, bh[half], bl[half]);
+                mma3(pr[half], qh, ql, bh[half], bl[half]);
             }
         }
     }
-    // ---- the scaled operands, eight columns at a time
-    const int last = cnt - 1;
-    for (int i = tid; i < C * (DK / 8); i += F_THREADS) {
-        const int t = i / (DK / 8), x = i % (DK / 8);
-        float kf[8], qf[8], kb[8];
+    __syncthreads();  // the right operand's place becomes A's
 #pragma unroll
-        for (int e = 0; e < 8; e++) {
-            const int d = x * 8 + e;
-            const float g = CHANNEL ? gs[t * LD + d] : gs[t], ge = CHANNEL ? gs[last * LD + d] : gs[last], k = ks[t * LD + d];
-            const float f = fast_exp2(g);
-            kf[e] = k * f;
-            kb[e] = t < cnt ? k * fast_exp2(ge - g) : 0.f;
-            qf[e] = t < cnt && d < D ? q[(size_t)t * Q + d] * f : 0.f;
+    for (int half = 0; half < 2; half++) {
+        const int u0 = 16 * j + half * 8 + 2 * t4;
+#pragma unroll
+        for (int e = 0; e < 4; e++) {
+            const int t = e < 2 ? ta : tb, u = u0 + (e & 1);
+            if constexpr (!CHANNEL) {
+                const float w = u <= t ? fast_exp2(ref[t] - ref[u]) : 0.f;
+                a[half][e] *= w;
+                pr[half][e] *= w;
+            }
+            if (u > t) pr[half][e] = 0.f;
+            if (s.delta && u < t) M[t * LM + u] = a[half][e] * betas[t];
         }
-        const uint32_t o = at_wide(t, x, DK * 2);
-        auto store = [&](int tile, const float (&v)[8]) {
-            Split w[4];
 #pragma unroll
-            for (int e = 0; e < 4; e++) w[e] = split2(v[2 * e], v[2 * e + 1]);
-            *reinterpret_cast<uint4*>(rec + tile + o) = make_uint4(w[0].hi, w[1].hi, w[2].hi, w[3].hi);
-            *reinterpret_cast<uint4*>(rec + tile + R::kOp + o) = make_uint4(w[0].lo, w[1].lo, w[2].lo, w[3].lo);
-        };
-        if (s.delta) store(R::Kf, kf);
-        store(R::Qf, qf);
-        store(R::Kb, kb);
+        for (int row = 0; row < 2; row++) {
+            const Split sp = split2(pr[half][2 * row], pr[half][2 * row + 1]);
+            const uint32_t o = at_wide(row ? tb : ta, u0 >> 3, 128) + (u0 & 7) * 2;
+            *reinterpret_cast<uint32_t*>(rec + R::P + o) = sp.hi;
+            *reinterpret_cast<uint32_t*>(rec + R::P + R::kMat + o) = sp.lo;
+        }
     }
     // the chunk's whole decay, over the first token's entry (which only this block reads)
     if constexpr (CHANNEL) {
-        if (tid < D) p.lg[tok0 * s.decays() + h * D + tid] = fast_exp2(gs[last * LD + tid]);
+        if (tid < D) p.lg[tok0 * s.decays() + h * D + tid] = fast_exp2(ref[4 * DK + tid]);
     } else if (s.decay == MemDecay::PerHead && tid == 0) {
-        p.lg[tok0 * s.heads + h] = fast_exp2(gs[last]);
+        p.lg[tok0 * s.heads + h] = fast_exp2(ref[last]);
     }
     if (!s.delta) return;
     // ---- inverse of the unit lower triangular I + A: diagonal blocks, then block diagonals outwards
@@ -278,9 +353,9 @@ __global__ void __launch_bounds__(F_THREADS) memory_factor_kernel(const MemorySp
         for (int e = tid; e < pairs * 256; e += F_THREADS) {
             const int j = e >> 8, i = j + dist, t = (e >> 4) & 15, u = e & 15;
             float acc = 0.f;
-            for (int k = j; k < i; k++)
+            for (int m = j; m < i; m++)
 #pragma unroll
-                for (int x = 0; x < 16; x++) acc = fmaf(M[(16 * i + t) * LM + 16 * k + x], inv(k, j, x, u), acc);
+                for (int x = 0; x < 16; x++) acc = fmaf(M[(16 * i + t) * LM + 16 * m + x], inv(m, j, x, u), acc);
             Y[(j * 16 + t) * 17 + u] = acc;
         }
         __syncthreads();
@@ -305,10 +380,10 @@ __global__ void __launch_bounds__(F_THREADS) memory_factor_kernel(const MemorySp
 }
 
 // ---- the walk --------------------------------------------------------------------------------------------------------
-// Block = (32 value columns of one head, sequence), eight warps.  Per chunk: Kf S0 and Qf S0 (a warp per 16 tokens x 16
-// columns), U from them, then O and the state (a warp per 16 state rows x 32 columns, or x 16 for keys up to 64).  The next
-// chunk's tiles arrive by bulk copies: Kf and Qf into the other of two buffers, the rest as soon as its place is free.
-constexpr int W_THREADS = 256;
+// Block = (32 value columns of one head, sequence).  Per chunk, eight warps (16 tokens x 16 columns each) form Kf S0 and from
+// it U, while eight others form Qf S0; then those add P U and store O, and every warp updates its 16 x 16 part of the state.
+// The next chunk's tiles arrive by bulk copies: Kf and Qf into the other of two buffers, the rest as soon as its place is free.
+constexpr int W_THREADS = 512, W_HALF = 256;
 template <int DK>
 struct WalkSmem {
     using R = Record<DK>;
@@ -354,9 +429,10 @@ __global__ void __launch_bounds__(W_THREADS, 1) memory_chunk_kernel(const Memory
         bulk_load(base + L::P, rec0 + c * rec_step + R::P, 2 * R::kMat + 2 * R::kOp, f_pk);  // P and Kb lie side by side in both places
     };
     static_assert(L::Kb == L::P + 2 * R::kMat && R::Kb == R::P + 2 * R::kMat, "one copy for P and Kb");
-    // state of this warp: rows sr + g4 (+ 8), columns sc + 8 j + 2 t4 (+ 1)
-    constexpr int NT = DK == 128 ? 4 : 2;
-    const int sr = (DK == 128 ? warp : warp >> 1) * 16, sc = DK == 128 ? 0 : (warp & 1) * 16;
+    // state of this warp: rows sr + g4 (+ 8), columns sc + 8 j + 2 t4 (+ 1); with keys up to 64 half of the warps have none
+    constexpr int NT = 2;
+    const int sr = (warp >> 1) * 16, sc = (warp & 1) * 16;
+    const bool has_state = sr < DK;
     float* Sg = p.state + (size_t)p.seq_slot[b] * p.slot_stride + ((size_t)h * P + p0) * D;
     float S[NT][4];
 #pragma unroll
@@ -373,6 +449,7 @@ __global__ void __launch_bounds__(W_THREADS, 1) memory_chunk_kernel(const Memory
         *reinterpret_cast<uint32_t*>(smem + off + lo_off + o) = sp.lo;
     };
     auto put_state = [&]() {
+        if (!has_state) return;
 #pragma unroll
         for (int j = 0; j < NT; j++) {
             put(L::S, L::kS, sr + g4, sc + j * 8 + 2 * t4, S[j][0], S[j][1]);
@@ -386,7 +463,8 @@ __global__ void __launch_bounds__(W_THREADS, 1) memory_chunk_kernel(const Memory
         if (DELTA) load_t(0);
         load_pk(0);
     }
-    const int mt = warp >> 1, nc = (warp & 1) * 16;  // tokens mt * 16 .., columns nc ..
+    const bool reads = warp >= 8;                             // this warp forms O, not U
+    const int mt = (warp >> 1) & 3, nc = (warp & 1) * 16;     // tokens mt * 16 .., columns nc ..
     const int ta = mt * 16 + g4, tb = ta + 8;
     // values at this thread's places of the token tiles: rows ta, tb, columns nc + 8 j + 2 t4 (+ 1)
     const uint16_t* vg = reinterpret_cast<const uint16_t*>(p.v) + (size_t)start * p.ld_v + h * P + p0;
@@ -422,138 +500,154 @@ __global__ void __launch_bounds__(W_THREADS, 1) memory_chunk_kernel(const Memory
     auto frag_b = [&](uint32_t tile, int row0, int piece0, uint32_t (&f0)[2], uint32_t (&f1)[2]) {
         ldmatrix_x4_trans(f0[0], f0[1], f1[0], f1[1], base + tile + at_narrow(row0 + lr + (mi & 1) * 8, piece0 + (mi >> 1)));
     };
-    fetch_v(0);
+    // heads' and remainders' products in accumulators of their own: shorter chains
+    struct Acc {
+        float d[2][4], e[2][4];
+        __device__ __forceinline__ void clear() {
+#pragma unroll
+            for (int j = 0; j < 2; j++)
+#pragma unroll
+                for (int i = 0; i < 4; i++) d[j][i] = e[j][i] = 0.f;
+        }
+        __device__ __forceinline__ void add(const uint32_t (&ah)[4], const uint32_t (&al)[4], const uint32_t (&bh0)[2], const uint32_t (&bh1)[2],
+                                            const uint32_t (&bl0)[2], const uint32_t (&bl1)[2]) {
+            mma_bf16_16816(d[0], ah, bh0);
+            mma_bf16_16816(d[1], ah, bh1);
+            mma_bf16_16816(e[0], ah, bl0);
+            mma_bf16_16816(e[1], ah, bl1);
+            mma_bf16_16816(e[0], al, bh0);
+            mma_bf16_16816(e[1], al, bh1);
+        }
+        __device__ __forceinline__ void add(const uint32_t (&ah)[4], const uint32_t (&al)[4], const uint32_t (&b0)[2], const uint32_t (&b1)[2]) {
+            mma_bf16_16816(d[0], ah, b0);
+            mma_bf16_16816(d[1], ah, b1);
+            mma_bf16_16816(e[0], al, b0);
+            mma_bf16_16816(e[1], al, b1);
+        }
+        __device__ __forceinline__ float at(int j, int i) const { return d[j][i] + e[j][i]; }
+    };
+    if (!reads) fetch_v(0);
     bool alive = true;
     for (int c = 0; c < chunks; c++) {
         const uint32_t ph = (uint32_t)c & 1u, kq = L::KQ + ph * L::kKQ;
         if (tid == 0 && c + 1 < chunks) load_kq(c + 1);  // (its buffer was last read before the previous chunk's barriers)
-        fetch_decay(c);
-        alive = mbar_wait(f_kq[ph], (uint32_t)(c >> 1) & 1u) && alive;
-        // ---- what the state before the chunk answers
-        float ak[2][4], o[2][4];
+        if (has_state) fetch_decay(c);
+        alive = mbar_wait(ph ? f_kq[1] : f_kq[0], (uint32_t)(c >> 1) & 1u) && alive;
+        Acc o;
+        // ---- what the state before the chunk answers to the keys, or to the queries
+        if (DELTA || reads) {
+            const uint32_t op = kq + (reads ? 2 * R::kOp : 0);
+            o.clear();
 #pragma unroll
-        for (int j = 0; j < 2; j++)
-#pragma unroll
-            for (int e = 0; e < 4; e++) ak[j][e] = o[j][e] = 0.f;
-#pragma unroll
-        for (int k = 0; k < DK / 16; k++) {
-            uint32_t ah[4], al[4], bh0[2], bh1[2], bl0[2], bl1[2];
-            frag_b(L::S, k * 16, nc >> 3, bh0, bh1);
-            frag_b(L::S + L::kS, k * 16, nc >> 3, bl0, bl1);
-            if constexpr (DELTA) {
-                frag_a(kq, DK * 2, mt * 16, 2 * k, ah);
-                frag_a(kq + R::kOp, DK * 2, mt * 16, 2 * k, al);
-                mma3(ak[0], ah, al, bh0, bl0);
-                mma3(ak[1], ah, al, bh1, bl1);
+            for (int k = 0; k < DK / 16; k++) {
+                uint32_t ah[4], al[4], bh0[2], bh1[2], bl0[2], bl1[2];
+                frag_b(L::S, k * 16, nc >> 3, bh0, bh1);
+                frag_b(L::S + L::kS, k * 16, nc >> 3, bl0, bl1);
+                frag_a(op, DK * 2, mt * 16, 2 * k, ah);
+                frag_a(op + R::kOp, DK * 2, mt * 16, 2 * k, al);
+                o.add(ah, al, bh0, bh1, bl0, bl1);
             }
-            frag_a(kq + 2 * R::kOp, DK * 2, mt * 16, 2 * k, ah);
-            frag_a(kq + 3 * R::kOp, DK * 2, mt * 16, 2 * k, al);
-            mma3(o[0], ah, al, bh0, bl0);
-            mma3(o[1], ah, al, bh1, bl1);
         }
         // ---- U
-        if constexpr (DELTA) {
+        if (!reads) {
+            if constexpr (DELTA) {
 #pragma unroll
-            for (int j = 0; j < 2; j++) {
-                put(L::RU, L::kU, ta, nc + j * 8 + 2 * t4, bflo(vv[j][0]) - ak[j][0], bfhi(vv[j][0]) - ak[j][1]);
-                put(L::RU, L::kU, tb, nc + j * 8 + 2 * t4, bflo(vv[j][1]) - ak[j][2], bfhi(vv[j][1]) - ak[j][3]);
-            }
-            if (c + 1 < chunks) fetch_v(c + 1);
-            alive = mbar_wait(f_t, ph) && alive;
-            __syncthreads();
-            float u[2][4];
-#pragma unroll
-            for (int j = 0; j < 2; j++) u[j][0] = u[j][1] = u[j][2] = u[j][3] = 0.f;
-#pragma unroll
-            for (int k = 0; k < C / 16; k++)
-                if (k <= mt) {
-                    uint32_t ah[4], al[4], bh0[2], bh1[2], bl0[2], bl1[2];
-                    frag_a(L::T, 128, mt * 16, 2 * k, ah);
-                    frag_a(L::T + R::kMat, 128, mt * 16, 2 * k, al);
-                    frag_b(L::RU, k * 16, nc >> 3, bh0, bh1);
-                    frag_b(L::RU + L::kU, k * 16, nc >> 3, bl0, bl1);
-                    mma3(u[0], ah, al, bh0, bl0);
-                    mma3(u[1], ah, al, bh1, bl1);
+                for (int j = 0; j < 2; j++) {
+                    put(L::RU, L::kU, ta, nc + j * 8 + 2 * t4, bflo(vv[j][0]) - o.at(j, 0), bfhi(vv[j][0]) - o.at(j, 1));
+                    put(L::RU, L::kU, tb, nc + j * 8 + 2 * t4, bflo(vv[j][1]) - o.at(j, 2), bfhi(vv[j][1]) - o.at(j, 3));
                 }
+                if (c + 1 < chunks) fetch_v(c + 1);
+                alive = mbar_wait(f_t, ph) && alive;
+                asm volatile("bar.sync 1, %0;\n" ::"n"(W_HALF) : "memory");
+                o.clear();
 #pragma unroll
-            for (int j = 0; j < 2; j++) {
-                put(L::U, L::kU, ta, nc + j * 8 + 2 * t4, u[j][0], u[j][1]);
-                put(L::U, L::kU, tb, nc + j * 8 + 2 * t4, u[j][2], u[j][3]);
-            }
-        } else {  // the values themselves, bf16
+                for (int k = 0; k < C / 16; k++)
+                    if (k <= mt) {
+                        uint32_t ah[4], al[4], bh0[2], bh1[2], bl0[2], bl1[2];
+                        frag_a(L::T, 128, mt * 16, 2 * k, ah);
+                        frag_a(L::T + R::kMat, 128, mt * 16, 2 * k, al);
+                        frag_b(L::RU, k * 16, nc >> 3, bh0, bh1);
+                        frag_b(L::RU + L::kU, k * 16, nc >> 3, bl0, bl1);
+                        o.add(ah, al, bh0, bh1, bl0, bl1);
+                    }
 #pragma unroll
-            for (int j = 0; j < 2; j++)
-#pragma unroll
-                for (int row = 0; row < 2; row++) {
-                    const int q = nc + j * 8 + 2 * t4;
-                    *reinterpret_cast<uint32_t*>(smem + L::U + at_narrow(row ? tb : ta, q >> 3) + (q & 7) * 2) = vv[j][row];
+                for (int j = 0; j < 2; j++) {
+                    put(L::U, L::kU, ta, nc + j * 8 + 2 * t4, o.at(j, 0), o.at(j, 1));
+                    put(L::U, L::kU, tb, nc + j * 8 + 2 * t4, o.at(j, 2), o.at(j, 3));
                 }
-            if (c + 1 < chunks) fetch_v(c + 1);
+            } else {  // the values themselves, bf16
+#pragma unroll
+                for (int j = 0; j < 2; j++)
+#pragma unroll
+                    for (int row = 0; row < 2; row++) {
+                        const int q = nc + j * 8 + 2 * t4;
+                        *reinterpret_cast<uint32_t*>(smem + L::U + at_narrow(row ? tb : ta, q >> 3) + (q & 7) * 2) = vv[j][row];
+                    }
+                if (c + 1 < chunks) fetch_v(c + 1);
+            }
         }
         alive = mbar_wait(f_pk, ph) && alive;
         alive = __syncthreads_and(alive);
         if (!alive) break;
         if (DELTA && tid == 0 && c + 1 < chunks) load_t(c + 1);
-        // ---- O
-#pragma unroll
-        for (int k = 0; k < C / 16; k++)
-            if (k <= mt) {
-                uint32_t ah[4], al[4], bh0[2], bh1[2], bl0[2], bl1[2];
-                frag_a(L::P, 128, mt * 16, 2 * k, ah);
-                frag_a(L::P + R::kMat, 128, mt * 16, 2 * k, al);
-                frag_b(L::U, k * 16, nc >> 3, bh0, bh1);
-                if constexpr (DELTA) {
-                    frag_b(L::U + L::kU, k * 16, nc >> 3, bl0, bl1);
-                    mma3(o[0], ah, al, bh0, bl0);
-                    mma3(o[1], ah, al, bh1, bl1);
-                } else {
-                    mma_bf16_16816(o[0], ah, bh0);
-                    mma_bf16_16816(o[0], al, bh0);
-                    mma_bf16_16816(o[1], ah, bh1);
-                    mma_bf16_16816(o[1], al, bh1);
-                }
-            }
-#pragma unroll
-        for (int j = 0; j < 2; j++)
-#pragma unroll
-            for (int row = 0; row < 2; row++) {
-                const int t = c * C + (row ? tb : ta), q = nc + j * 8 + 2 * t4;
-                if (t >= n) continue;
-                float* x = p.o + (size_t)(start + t) * V + h * P + p0 + q;
-                if (P % 2 == 0 && p0 + q < P) {
-                    *reinterpret_cast<float2*>(x) = make_float2(o[j][2 * row], o[j][2 * row + 1]);
-                } else {
-                    if (p0 + q < P) x[0] = o[j][2 * row];
-                    if (p0 + q + 1 < P) x[1] = o[j][2 * row + 1];
-                }
-            }
         // ---- the state
+        if (has_state) {
+            Acc u;
+            u.clear();
 #pragma unroll
-        for (int j = 0; j < NT; j++) S[j][0] *= dec[0], S[j][1] *= dec[0], S[j][2] *= dec[1], S[j][3] *= dec[1];
+            for (int j = 0; j < NT; j++) u.d[j][0] = S[j][0] * dec[0], u.d[j][1] = S[j][1] * dec[0], u.d[j][2] = S[j][2] * dec[1], u.d[j][3] = S[j][3] * dec[1];
 #pragma unroll
-        for (int k = 0; k < C / 16; k++) {
-            // Kb^T: rows of keys from rows of tokens
-            uint32_t ah[4], al[4];
-            const uint32_t x = at_wide(k * 16 + lr + (mi >> 1) * 8, (sr >> 3) + (mi & 1), DK * 2);
-            ldmatrix_x4_trans(ah[0], ah[1], ah[2], ah[3], base + L::Kb + x);
-            ldmatrix_x4_trans(al[0], al[1], al[2], al[3], base + L::Kb + R::kOp + x);
-#pragma unroll
-            for (int j = 0; j < NT / 2; j++) {
-                uint32_t bh0[2], bh1[2], bl0[2], bl1[2];
-                frag_b(L::U, k * 16, (sc >> 3) + 2 * j, bh0, bh1);
+            for (int k = 0; k < C / 16; k++) {
+                // Kb^T: rows of keys from rows of tokens
+                uint32_t ah[4], al[4], bh0[2], bh1[2], bl0[2], bl1[2];
+                const uint32_t x = at_wide(k * 16 + lr + (mi >> 1) * 8, (sr >> 3) + (mi & 1), DK * 2);
+                ldmatrix_x4_trans(ah[0], ah[1], ah[2], ah[3], base + L::Kb + x);
+                ldmatrix_x4_trans(al[0], al[1], al[2], al[3], base + L::Kb + R::kOp + x);
+                frag_b(L::U, k * 16, sc >> 3, bh0, bh1);
                 if constexpr (DELTA) {
-                    frag_b(L::U + L::kU, k * 16, (sc >> 3) + 2 * j, bl0, bl1);
-                    mma3(S[2 * j], ah, al, bh0, bl0);
-                    mma3(S[2 * j + 1], ah, al, bh1, bl1);
+                    frag_b(L::U + L::kU, k * 16, sc >> 3, bl0, bl1);
+                    u.add(ah, al, bh0, bh1, bl0, bl1);
                 } else {
-                    mma_bf16_16816(S[2 * j], ah, bh0);
-                    mma_bf16_16816(S[2 * j], al, bh0);
-                    mma_bf16_16816(S[2 * j + 1], ah, bh1);
-                    mma_bf16_16816(S[2 * j + 1], al, bh1);
+                    u.add(ah, al, bh0, bh1);
                 }
             }
+#pragma unroll
+            for (int j = 0; j < NT; j++)
+#pragma unroll
+                for (int i = 0; i < 4; i++) S[j][i] = u.at(j, i);
+            put_state();
         }
-        put_state();
+        // ---- O
+        if (reads) {
+#pragma unroll
+            for (int k = 0; k < C / 16; k++)
+                if (k <= mt) {
+                    uint32_t ah[4], al[4], bh0[2], bh1[2], bl0[2], bl1[2];
+                    frag_a(L::P, 128, mt * 16, 2 * k, ah);
+                    frag_a(L::P + R::kMat, 128, mt * 16, 2 * k, al);
+                    frag_b(L::U, k * 16, nc >> 3, bh0, bh1);
+                    if constexpr (DELTA) {
+                        frag_b(L::U + L::kU, k * 16, nc >> 3, bl0, bl1);
+                        o.add(ah, al, bh0, bh1, bl0, bl1);
+                    } else {
+                        o.add(ah, al, bh0, bh1);
+                    }
+                }
+#pragma unroll
+            for (int j = 0; j < 2; j++)
+#pragma unroll
+                for (int row = 0; row < 2; row++) {
+                    const int t = c * C + (row ? tb : ta), q = nc + j * 8 + 2 * t4;
+                    if (t >= n) continue;
+                    float* x = p.o + (size_t)(start + t) * V + h * P + p0 + q;
+                    if (P % 2 == 0 && p0 + q < P) {
+                        *reinterpret_cast<float2*>(x) = make_float2(o.at(j, 2 * row), o.at(j, 2 * row + 1));
+                    } else {
+                        if (p0 + q < P) x[0] = o.at(j, 2 * row);
+                        if (p0 + q + 1 < P) x[1] = o.at(j, 2 * row + 1);
+                    }
+                }
+        }
         __syncthreads();
         if (tid == 0 && c + 1 < chunks) load_pk(c + 1);
     }
@@ -569,7 +663,7 @@ __global__ void __launch_bounds__(W_THREADS, 1) memory_chunk_kernel(const Memory
 #pragma unroll
         for (int e = 0; e < 4; e++) {
             const int r = sr + g4 + (e >> 1) * 8, q = sc + j * 8 + 2 * t4 + (e & 1);
-            if (r < D && p0 + q < P) Sg[(size_t)q * D + r] = S[j][e];
+            if (has_state && r < D && p0 + q < P) Sg[(size_t)q * D + r] = S[j][e];
         }
     memory_keep_inputs<uint16_t>(s, p, b, blockIdx.y * gridDim.x + blockIdx.x, gridDim.x * gridDim.y);
 }
