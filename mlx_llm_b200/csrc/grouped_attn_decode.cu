@@ -28,15 +28,15 @@ struct ScoreMap {
     __device__ __forceinline__ float operator()(float s) const { return cap ? c - __fdividef(2.f * c, 1.f + fast_exp2(fminf(s * a, 126.f))) : s * a; }
 };
 
-// NB: 16-wide steps of the larger of the two head sizes, rounded up.
-template <int NB>
+// NB: 16-wide steps of the larger of the two head sizes, rounded up; EXACT: both heads have exactly that many.
+template <int NB, bool EXACT>
 __global__ void __launch_bounds__(kWarps * 32) gqa_decode_kernel(const GroupedAttnSpec a, const GqaAttnParams p, bool listed) {
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     extern __shared__ __align__(128) uint8_t smem[];
     __shared__ int s_last;
     pdl_wait();
     const int item = blockIdx.x, group = a.group(), subs = (group + kHeads - 1) / kHeads, kvh = blockIdx.y / subs, h0 = kvh * group + (blockIdx.y % subs) * kHeads;
-    const int heads = min(kHeads, kvh * group + group - h0), KR = a.k_row(), VR = a.v_row();
+    const int heads = min(kHeads, kvh * group + group - h0), KR = EXACT ? NB * 16 : a.k_row(), VR = EXACT ? NB * 16 : a.v_row();
     int row, chunk = 0, w0 = item, ctx, qrow, slot;  // entry of the list, its chunk, first work item of the row
     if (listed) {
         if (item >= *p.n_dec_work) return;
@@ -117,7 +117,7 @@ __global__ void __launch_bounds__(kWarps * 32) gqa_decode_kernel(const GroupedAt
             const int r = lr + (mi & 1) * 8;
 #pragma unroll
             for (int k = 0; k < NB; k++)
-                if (k < kd) {
+                if (EXACT || k < kd) {
                     uint32_t f[4];
                     ldmatrix_x4(f[0], f[1], f[2], f[3], kb + r * krow + (((2 * k + (mi >> 1)) ^ (r & 7)) << 4));
                     mma_bf16_16816(s, f, qf[k]);
@@ -156,7 +156,7 @@ __global__ void __launch_bounds__(kWarps * 32) gqa_decode_kernel(const GroupedAt
             const int r = lr + (mi >> 1) * 8;
 #pragma unroll
             for (int q = 0; q < NB; q++)
-                if (q < vd) {
+                if (EXACT || q < vd) {
                     uint32_t f[4];
                     ldmatrix_x4_trans(f[0], f[1], f[2], f[3], vb + r * vrow + (((2 * q + (mi & 1)) ^ (r & 7)) << 4));
                     mma_bf16_16816(o[q], f, pb);
@@ -178,7 +178,7 @@ __global__ void __launch_bounds__(kWarps * 32) gqa_decode_kernel(const GroupedAt
     float* sm_l = sm_m + kWarps * 8;
 #pragma unroll
     for (int q = 0; q < NB; q++)
-        if (q < vd) {
+        if (EXACT || q < vd) {
             float* base = so + ((size_t)warp * VR + 16 * q + g) * 8 + 2 * t;
             base[0] = o[q][0];
             base[1] = o[q][1];
@@ -293,11 +293,11 @@ int smem_bytes(const GroupedAttnSpec& a) {
     const int ring = kWarps * kStages * 16 * (krow + vrow), merge = (kWarps * a.v_row() * 8 + 2 * kWarps * 8) * 4, chunks = (2 * kMergeBatch * 8 + 16) * 4;
     return ring > merge ? (ring > chunks ? ring : chunks) : (merge > chunks ? merge : chunks);
 }
-template <int NB>
+template <int NB, bool EXACT>
 int32_t launch(b2_ctx* ctx, const GroupedAttnSpec& a, const GqaAttnParams& p, int items) {
-    B2_SMEM_ONCE(ctx, gqa_decode_kernel<NB>, kWarps * kStages * 16 * 2 * 512);
+    B2_SMEM_ONCE(ctx, (gqa_decode_kernel<NB, EXACT>), kWarps * kStages * 16 * 2 * 512);
     const dim3 grid(items > 0 ? items : p.T, b2_gqa_head_blocks(a));
-    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, gqa_decode_kernel<NB>, grid, dim3(kWarps * 32), (size_t)smem_bytes(a), ctx->stream, a, p, items > 0));
+    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, gqa_decode_kernel<NB, EXACT>, grid, dim3(kWarps * 32), (size_t)smem_bytes(a), ctx->stream, a, p, items > 0));
     B2_LAUNCHED(ctx);
     return B2_OK;
 }
@@ -310,8 +310,8 @@ int32_t b2_gqa_decode_launch(b2_ctx* ctx, const GroupedAttnSpec& a, const GqaAtt
     if (p.T <= 0) return B2_OK;
     B2_REQUIRE(p.page_size % 16 == 0, B2_ERR_UNSUPPORTED, "grouped attention: pages of whole 16-key tiles");
     const int nb = (a.k_row() > a.v_row() ? a.k_row() : a.v_row()) / 16;
-    if (nb <= 4) return launch<4>(ctx, a, p, items);
-    if (nb <= 8) return launch<8>(ctx, a, p, items);
-    if (nb <= 12) return launch<12>(ctx, a, p, items);
-    return launch<16>(ctx, a, p, items);
+    if (a.k_row() == a.v_row() && nb == 4) return launch<4, true>(ctx, a, p, items);
+    if (a.k_row() == a.v_row() && nb == 8) return launch<8, true>(ctx, a, p, items);
+    if (nb <= 8) return launch<8, false>(ctx, a, p, items);
+    return launch<16, false>(ctx, a, p, items);
 }

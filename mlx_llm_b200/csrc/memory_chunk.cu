@@ -47,20 +47,22 @@ __device__ __forceinline__ void mma3(float (&d)[4], const uint32_t (&ah)[4], con
 }
 
 // ---- factors ---------------------------------------------------------------------------------------------------------
-// Decays per channel: with r_i the sums before 16-token block i and e_i those at its end, the exponent of token t of block i
-// and an earlier token s of block j splits into
-//     G_t - G_s = (G_t - r_i) + (r_i - e_j) + (e_j - G_s)
-// The outer two belong to one token each and are at most zero; the middle one is a number per channel and pair of blocks, at
-// most zero but for i = j, where it undoes the block's own decay.  A block whose decay is too strong for that (beyond 2^-80
-// inside 16 tokens) takes every exponent from its difference instead.
+// Decays per channel: with a reference m_i for each 16-token block i, the exponent of token t of block i and an earlier token s
+// of block j splits into
+//     G_t - G_s = (G_t - m_i) + (m_i - m_j) + (m_j - G_s)
+// The outer two belong to one token each, the middle one is a number per channel and pair of blocks.  The reference is the sum
+// in the block's middle: its factors and their inverses stay inside 2^+-100 for decays up to 2^-100 in eight tokens, and a
+// product that would underflow on the way is below 2^-26.  A channel that decays faster takes the sums at the block's borders
+// (before it on the left, at its end on the right: no factor above one), and the block's own tile, where neither works, takes
+// every exponent from its difference.
 constexpr int F_WARPS = 10, F_THREADS = F_WARPS * 32;  // a warp per 16 x 16 tile of P and A up to the diagonal
-constexpr float kMaxSpread = 80.f;  // log2 units
+constexpr float kMaxSpread = 100.f;  // log2 units
 template <int DK, bool CHANNEL>
 struct FactorSmem {
     static constexpr int LD = DK + 4, LM = C + 4, kOp = C * DK * 2;
     // left operands (k, q; head and remainder), then the right one in f32, whose place A and its inverse take later
     static constexpr int LK = 0, LQ = 2 * kOp, G = 4 * kOp, kG = CHANNEL ? C * LD * 4 : 0, kM = C * LM * 4;
-    static constexpr int M = G, Y = G + (kG > kM ? kG : kM), REF = Y + 3 * 16 * 17 * 4, BETA = REF + (CHANNEL ? 5 * DK * 4 : C * 4), kBytes = BETA + C * 4;
+    static constexpr int M = G, Y = G + (kG > kM ? kG : kM), REF = Y + 3 * 16 * 17 * 4, BETA = REF + (CHANNEL ? 9 * DK * 4 : C * 4), kBytes = BETA + C * 4;
 };
 
 template <int DK, bool CHANNEL>
@@ -71,10 +73,10 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
     using R = Record<DK>;
     constexpr int LD = L::LD, LM = L::LM;
     extern __shared__ __align__(16) uint8_t smem[];
-    float* gs = reinterpret_cast<float*>(smem + L::G);      // CHANNEL: [C][LD] running sums (base 2), then k e^(e_j - G_s)
+    float* gs = reinterpret_cast<float*>(smem + L::G);      // CHANNEL: [C][LD] running sums (base 2), then k e^(m_j - G_s)
     float* M = reinterpret_cast<float*>(smem + L::M);       // [C][LM]: A below the diagonal, the transposed inverse above it
     float* Y = reinterpret_cast<float*>(smem + L::Y);       // [3][16][17]
-    float* ref = reinterpret_cast<float*>(smem + L::REF);   // CHANNEL: [5][DK] sums at the blocks' borders; else [C] running sums
+    float* ref = reinterpret_cast<float*>(smem + L::REF);   // CHANNEL: [4][DK] left and [4][DK] right references, [DK] the end; else [C] running sums
     float* betas = reinterpret_cast<float*>(smem + L::BETA);
     __shared__ int wide[4];                                 // blocks with strong decays
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g4 = lane >> 2, t4 = lane & 3, mi = lane >> 3, lr = lane & 7;
@@ -108,21 +110,31 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
                     x[t] = tok < cnt && d < D ? lg[(size_t)tok * s.decays() + d] : 0.f;
                 }
                 const float before = run;
+                float mid = run;
 #pragma unroll
                 for (int t = 0; t < 16; t++) {
                     run = fmaf(x[t], kLog2e, run);
                     gs[(half * H + 16 * i + t) * LD + d] = run;
+                    if (t == 7) mid = run;
                 }
-                ref[(half * 2 + i + 1) * DK + d] = run;
-                if (before - run > kMaxSpread) atomicOr(&wide[half * 2 + i], 1);
+                const bool fast = before - mid > kMaxSpread || mid - run > kMaxSpread;
+                ref[(half * 2 + i) * DK + d] = fast ? before : mid;
+                ref[(4 + half * 2 + i) * DK + d] = fast ? run : mid;
+                if (fast) atomicOr(&wide[half * 2 + i], 1);
             }
+            if (half == 0) ref[8 * DK + d] = run;
         }
         __syncthreads();
-        if (half == 0) {
-            ref[d] = 0.f;
-            const float first = ref[2 * DK + d];
-            ref[3 * DK + d] += first;
-            ref[4 * DK + d] += first;
+        if (half == 1) {
+            const float first = ref[8 * DK + d];
+#pragma unroll
+            for (int i = 2; i < 4; i++) {
+                ref[i * DK + d] += first;
+                ref[(4 + i) * DK + d] += first;
+            }
+#pragma unroll 8
+            for (int t = H; t < C; t++) gs[t * LD + d] += first;
+            ref[8 * DK + d] = gs[(C - 1) * LD + d];
         }
     } else if (tid < 32) {
         auto at = [&](int t) { return t < cnt ? (s.decay == MemDecay::Fixed ? p.log_decay[h] : p.lg[(tok0 + t) * s.heads + h]) * kLog2e : 0.f; };
@@ -170,15 +182,15 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
             *reinterpret_cast<uint4*>(base + R::kOp + o) = make_uint4(w[0].lo, w[1].lo, w[2].lo, w[3].lo);
         };
         if constexpr (CHANNEL) {
-            float r0[8], tail[8];  // e^(r_i), e^(G_end - e_i)
+            float r0[8], tail[8];  // e^(m_i), e^(G_end - m_i)
 #pragma unroll
             for (int e = 0; e < 8; e++) {
                 const int d = x * 8 + e;
-                const float r = ref[blk * DK + d], end = ref[(blk + 1) * DK + d], g = gs[t * LD + d] + (blk >= 2 ? ref[2 * DK + d] : 0.f);
+                const float r = ref[blk * DK + d], m = ref[(4 + blk) * DK + d], g = gs[t * LD + d];
                 left[e] = fast_exp2(g - r);
-                right[e] = kv[e] * fast_exp2(end - g);
+                right[e] = kv[e] * fast_exp2(m - g);
                 r0[e] = fast_exp2(r);
-                tail[e] = fast_exp2(ref[4 * DK + d] - end);
+                tail[e] = fast_exp2(ref[8 * DK + d] - m);
                 gs[t * LD + d] = right[e];
             }
 #pragma unroll
@@ -273,7 +285,7 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
 #pragma unroll
                 for (int e = 0; e < 2; e++) {
                     const int d = d0 + e * 8;
-                    const float2 r = *reinterpret_cast<const float2*>(ref + i * DK + d), en = *reinterpret_cast<const float2*>(ref + (j + 1) * DK + d);
+                    const float2 r = *reinterpret_cast<const float2*>(ref + i * DK + d), en = *reinterpret_cast<const float2*>(ref + (4 + j) * DK + d);
                     const float f0 = fast_exp2(r.x - en.x), f1 = fast_exp2(r.y - en.y);
 #pragma unroll
                     for (int half = 0; half < 2; half++) {
@@ -319,7 +331,7 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
     }
     // the chunk's whole decay, over the first token's entry (which only this block reads)
     if constexpr (CHANNEL) {
-        if (tid < D) p.lg[tok0 * s.decays() + h * D + tid] = fast_exp2(ref[4 * DK + tid]);
+        if (tid < D) p.lg[tok0 * s.decays() + h * D + tid] = fast_exp2(ref[8 * DK + tid]);
     } else if (s.decay == MemDecay::PerHead && tid == 0) {
         p.lg[tok0 * s.heads + h] = fast_exp2(ref[last]);
     }
