@@ -53,8 +53,8 @@ __device__ __forceinline__ void mma3(float (&d)[4], const uint32_t (&ah)[4], con
 // The outer two belong to one token each, the middle one is a number per channel and pair of blocks.  The reference is the sum
 // in the block's middle: its factors and their inverses stay inside 2^+-100 for decays up to 2^-100 in eight tokens, and a
 // product that would underflow on the way is below 2^-26.  A channel that decays faster takes the sums at the block's borders
-// (before it on the left, at its end on the right: no factor above one), and the block's own tile, where neither works, takes
-// every exponent from its difference.
+// (before it on the left, at its end on the right: no factor above one); in the block's own tile, where neither works, it is
+// left out of the product and added with every exponent taken from its difference.
 constexpr int F_WARPS = 10, F_THREADS = F_WARPS * 32;  // a warp per 16 x 16 tile of P and A up to the diagonal
 constexpr float kMaxSpread = 100.f;  // log2 units
 template <int DK, bool CHANNEL>
@@ -78,7 +78,7 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
     float* Y = reinterpret_cast<float*>(smem + L::Y);       // [3][16][17]
     float* ref = reinterpret_cast<float*>(smem + L::REF);   // CHANNEL: [4][DK] left and [4][DK] right references, [DK] the end; else [C] running sums
     float* betas = reinterpret_cast<float*>(smem + L::BETA);
-    __shared__ int wide[4];                                 // blocks with strong decays
+    __shared__ uint32_t fast[4][DK / 32];                   // per block: channels with strong decays
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g4 = lane >> 2, t4 = lane & 3, mi = lane >> 3, lr = lane & 7;
     const int chunk = blockIdx.x, h = blockIdx.y, D = s.dim, Q = s.q_cols(), kh = h / (s.heads / s.kv_heads);
     int b = -1;  // the last chunked portion that starts at or before this chunk (starts rise with the index)
@@ -94,7 +94,7 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
     const float *q = p.q + tok0 * Q + kh * D, *k = p.k + tok0 * Q + kh * D;
     const float* lg = CHANNEL ? p.lg + tok0 * s.decays() + h * D : nullptr;
 
-    if (tid < 4) wide[tid] = 0;
+    if (tid < 4 * (DK / 32)) fast[tid / (DK / 32)][tid % (DK / 32)] = 0;
     if (tid < C) betas[tid] = s.delta && tid < cnt ? p.beta[(tok0 + tid) * s.heads + h] : 0.f;
     __syncthreads();
     if constexpr (CHANNEL) {  // a thread per channel and half of the chunk; the second half is raised by the first one's end
@@ -117,10 +117,10 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
                     gs[(half * H + 16 * i + t) * LD + d] = run;
                     if (t == 7) mid = run;
                 }
-                const bool fast = before - mid > kMaxSpread || mid - run > kMaxSpread;
-                ref[(half * 2 + i) * DK + d] = fast ? before : mid;
-                ref[(4 + half * 2 + i) * DK + d] = fast ? run : mid;
-                if (fast) atomicOr(&wide[half * 2 + i], 1);
+                const bool strong = before - mid > kMaxSpread || mid - run > kMaxSpread;
+                ref[(half * 2 + i) * DK + d] = strong ? before : mid;
+                ref[(4 + half * 2 + i) * DK + d] = strong ? run : mid;
+                if (strong) atomicOr(&fast[half * 2 + i][d >> 5], 1u << (d & 31));
             }
             if (half == 0) ref[8 * DK + d] = run;
         }
@@ -236,39 +236,7 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
 #pragma unroll
         for (int e = 0; e < 4; e++) a[half][e] = pr[half][e] = 0.f;
     const int ta = 16 * i + g4, tb = ta + 8;
-    if (CHANNEL && i == j && wide[i]) {
-        // lanes over the channels; everything from memory again, this is rare
-#pragma unroll 1
-        for (int u = 16 * i; u < min(16 * i + 16, cnt); u++) {
-            float g[DK / 32], w[DK / 32];
-#pragma unroll
-            for (int x = 0; x < DK / 32; x++) {
-                const int d = x * 32 + lane;
-                g[x] = 0.f;
-                w[x] = d < D ? k[(size_t)u * Q + d] : 0.f;
-            }
-#pragma unroll 1
-            for (int t = u; t < min(16 * i + 16, cnt); t++) {
-                float sa = 0.f, sp = 0.f;
-#pragma unroll
-                for (int x = 0; x < DK / 32; x++) {
-                    const int d = x * 32 + lane;
-                    if (d >= D) continue;
-                    if (t > u) g[x] = fmaf(lg[(size_t)t * s.decays() + d], kLog2e, g[x]);
-                    const float v = fast_exp2(g[x]) * w[x];
-                    sa = fmaf(v, k[(size_t)t * Q + d], sa);
-                    sp = fmaf(v, q[(size_t)t * Q + d], sp);
-                }
-                sa = elt_warp_sum(sa);
-                sp = elt_warp_sum(sp);
-#pragma unroll
-                for (int half = 0; half < 2; half++)
-#pragma unroll
-                    for (int e = 0; e < 4; e++)
-                        if (t == (e < 2 ? ta : tb) && u == 16 * i + half * 8 + 2 * t4 + (e & 1)) a[half][e] = sa, pr[half][e] = sp;
-            }
-        }
-    } else {
+    {
         const uint32_t base = smem_u32(smem);
 #pragma unroll 2
         for (int kk = 0; kk < DK / 16; kk++) {
@@ -286,7 +254,8 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
                 for (int e = 0; e < 2; e++) {
                     const int d = d0 + e * 8;
                     const float2 r = *reinterpret_cast<const float2*>(ref + i * DK + d), en = *reinterpret_cast<const float2*>(ref + (4 + j) * DK + d);
-                    const float f0 = fast_exp2(r.x - en.x), f1 = fast_exp2(r.y - en.y);
+                    // (inside a block the references differ for the strong channels only)
+                    const float f0 = i == j ? (r.x == en.x ? 1.f : 0.f) : fast_exp2(r.x - en.x), f1 = i == j ? (r.y == en.y ? 1.f : 0.f) : fast_exp2(r.y - en.y);
 #pragma unroll
                     for (int half = 0; half < 2; half++) {
                         const float2 v = *reinterpret_cast<const float2*>(gs + (16 * j + half * 8 + g4) * LD + d);
@@ -305,6 +274,42 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
                 mma3(pr[half], qh, ql, bh[half], bl[half]);
             }
         }
+    }
+    if (CHANNEL && i == j) {
+#pragma unroll 1
+        for (int word = 0; word < DK / 32; word++)
+            for (uint32_t m = fast[i][word]; m; m &= m - 1) {
+                const int d = word * 32 + __ffs(m) - 1, tok = 16 * i + (lane & 15);  // a lane per token
+                const bool ok = tok < cnt && d < D;
+                float g = ok ? lg[(size_t)tok * s.decays() + d] * kLog2e : 0.f;
+                const float kv = ok ? k[(size_t)tok * Q + d] : 0.f, qv = ok ? q[(size_t)tok * Q + d] : 0.f;
+#pragma unroll
+                for (int o = 1; o < 16; o <<= 1) {
+                    const float x = __shfl_up_sync(0xffffffffu, g, o, 16);
+                    if ((lane & 15) >= o) g += x;
+                }
+                float gt[2], kt[2], qt[2];
+#pragma unroll
+                for (int x = 0; x < 2; x++) {
+                    gt[x] = __shfl_sync(0xffffffffu, g, g4 + 8 * x);
+                    kt[x] = __shfl_sync(0xffffffffu, kv, g4 + 8 * x);
+                    qt[x] = __shfl_sync(0xffffffffu, qv, g4 + 8 * x);
+                }
+#pragma unroll
+                for (int half = 0; half < 2; half++)
+#pragma unroll
+                    for (int c = 0; c < 2; c++) {
+                        const int u = half * 8 + 2 * t4 + c;
+                        const float gu = __shfl_sync(0xffffffffu, g, u), ku = __shfl_sync(0xffffffffu, kv, u);
+#pragma unroll
+                        for (int x = 0; x < 2; x++)
+                            if (u <= g4 + 8 * x) {
+                                const float w = fast_exp2(gt[x] - gu) * ku;
+                                a[half][2 * x + c] = fmaf(w, kt[x], a[half][2 * x + c]);
+                                pr[half][2 * x + c] = fmaf(w, qt[x], pr[half][2 * x + c]);
+                            }
+                    }
+            }
     }
     __syncthreads();  // the right operand's place becomes A's
 #pragma unroll
