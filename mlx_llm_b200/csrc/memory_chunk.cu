@@ -51,12 +51,12 @@ __device__ __forceinline__ void mma3(float (&d)[4], const uint32_t (&ah)[4], con
 // of block j splits into
 //     G_t - G_s = (G_t - m_i) + (m_i - m_j) + (m_j - G_s)
 // The outer two belong to one token each, the middle one is a number per channel and pair of blocks.  The reference is the sum
-// in the block's middle: its factors and their inverses stay inside 2^+-100 for decays up to 2^-100 in eight tokens, and a
-// product that would underflow on the way is below 2^-26.  A channel that decays faster takes the sums at the block's borders
+// in the block's middle: for decays up to 2^-40 in eight tokens the outer factors stay inside 2^+-40, so that a middle one
+// which underflows belongs to a product below 2^-46.  A channel that decays faster takes the sums at the block's borders
 // (before it on the left, at its end on the right: no factor above one); in the block's own tile, where neither works, it is
 // left out of the product and added with every exponent taken from its difference.
 constexpr int F_WARPS = 10, F_THREADS = F_WARPS * 32;  // a warp per 16 x 16 tile of P and A up to the diagonal
-constexpr float kMaxSpread = 100.f;  // log2 units
+constexpr float kMaxSpread = 40.f;  // log2 units
 template <int DK, bool CHANNEL>
 struct FactorSmem {
     static constexpr int LD = DK + 4, LM = C + 4, kOp = C * DK * 2;

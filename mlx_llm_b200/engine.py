@@ -219,7 +219,7 @@ class CausalLm:
         return logits, am[:rows]
 
     def capture_residual(self, buf):
-        """After every following step `buf` (float32, [layers, tokens, width]) holds the residual stream behind each layer;
+        """After every following step `buf` (float32, [layer runs, tokens, width]) holds the residual stream behind each run of a layer;
         None switches it off."""
         self._capture = buf
         check(load().b2_model_capture_residual(self.h, buf.ctypes.data_as(C.c_void_p) if buf is not None else None,

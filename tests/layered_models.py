@@ -262,7 +262,7 @@ TIREZEN = {
                          loop=(1, 3, 3)),
     # sizes that divide nothing, one head, one tap, single query groups
     "odd": tirezen([(sides(heads=5, kv_heads=5, dim=10, vdim=7, dims=4, right=dict(conv=1)), dense(33)), (delta(heads=3, kv_heads=1, dim=9, vdim=5, conv=5), dense(50)),
-                    (retention(heads=1, dim=7, vdim=3, dims=6), None)], width=52, vocab=97, loop=(0, 3, 2)),
+                    (retention(heads=1, dim=7, vdim=3, dims=6), None)], width=53, vocab=97, loop=(0, 3, 2)),
     # the tiles of the tensor-core kernels, more than eight query heads for one key head
     "tiles": tirezen([(sides(heads=10, kv_heads=1, dim=128, vdim=128, dims=128, softcap=15.0, right=dict(heads=2, kv_heads=1, dim=128, vdim=64, conv=4)), dense(512)),
                       (retention(heads=2, dim=128, vdim=128, dims=64), dense(256)), (delta(heads=2, kv_heads=2, dim=128, vdim=64, conv=4), None)],

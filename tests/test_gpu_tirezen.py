@@ -276,23 +276,40 @@ def test_delta_alone(env, kind, m, cuts, f32):
 
 @BOTH
 @MEM_CUTS
-@pytest.mark.parametrize("A,dt", [(3.0, 4.0), (-7.0, -2.0), (0.0, None)], ids=["forgets at once", "forgets nothing", "both"])
-@pytest.mark.parametrize("kind", ["head", "channel"])
-def test_delta_decays(env, kind, A, dt, cuts, f32):
-    """Exponents of minus hundreds per token, of nearly nothing, and both in neighbouring channels (heads)."""
+@pytest.mark.parametrize("A,dt,gain", [(3.0, 4.0, 1.0), (-7.0, -2.0, 1.0), (0.0, None, 1.0), (2.5, -1.0, 3.0)], ids=["forgets at once", "forgets nothing", "both", "now and then"])
+@pytest.mark.parametrize("kind,dim", [("head", 40), ("channel", 40), ("channel", 104)])
+def test_delta_decays(env, kind, dim, A, dt, gain, cuts, f32):
+    """Exponents of minus hundreds per token, of nearly nothing, both in neighbouring channels (heads), and from token to token."""
     ctx, eng = env
     p = "l0.mix." if kind == "head" else "l0.mix.right."
 
     def change(w):
         w[p + "A_log"][:] = A
         w[p + "dt_bias"][:] = dt if dt is not None else np.where(np.arange(len(w[p + "dt_bias"])) % 2, 60.0, -9.0)
+        w[p + ("a" if kind == "head" else "a2")] *= gain
         if kind == "channel":
             only_right(w)
 
-    m = dict(heads=4, kv_heads=2, dim=40, vdim=24, conv=3)
+    m = dict(heads=4, kv_heads=2, dim=dim, vdim=24, conv=3)
     layer = lm.delta(**m) if kind == "head" else lm.sides(heads=1, kv_heads=1, dim=8, vdim=8, dims=8, right=m)
     e = single(eng, ctx, (layer, None), f32, cuts=cuts, change=change)
     assert e < TOL[f32], e
+
+
+@BOTH
+@pytest.mark.parametrize("ranks", [(1, 1), (70, 33), (8, 130)], ids=str)
+def test_ranks_come_from_the_tensors(env, ranks, f32):
+    ctx, eng = env
+    cfg = lm.tirezen([(lm.sides(right=dict(heads=2, kv_heads=1, dim=24, vdim=36)), None)], width=58, vocab=60)
+    w = lm.tirezen_weights(cfg, seed=5, ranks=ranks)
+    model = lm.load(eng, ctx, cfg, w, f32)
+    ids = tokens(cfg, 40, 3)
+    want = ref.forward(cfg, w, ids)
+    pool = eng.BlockPool(ctx, model, 16, 3, 1)
+    for cuts in ([40], [13, 1, 2]):
+        assert error(run(eng, model, pool, ids, cuts), want) < TOL[f32]
+    pool.free()
+    model.free()
 
 
 @BOTH
@@ -475,7 +492,7 @@ def test_shapes_that_do_not_fit_are_refused(env):
     ctx, eng = env
     cfg = lm.TIREZEN["odd"]
     w = lm.tirezen_weights(cfg)
-    for key, new in (("l0.mix.right.a2", (3, 7)), ("head", (97, 50)), ("l1.mix.k.conv", (9, 4)), ("loop.step", (1, 52))):
+    for key, new in (("l0.mix.right.a2", (3, 7)), ("head", (97, 50)), ("l1.mix.k.conv", (9, 4)), ("loop.step", (1, 53))):
         bad = copy.copy(w)
         bad[key] = np.zeros(new)
         with pytest.raises(B2Error) as e:
