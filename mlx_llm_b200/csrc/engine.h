@@ -218,14 +218,19 @@ struct LayeredStep {
     long dec_ctx_sum;
     int n_chunks;               // chunks of the portions that the memories' chunked form takes
     const int32_t* chunk_off;   // [B] device: first chunk of each such portion, -1 for the others
-    double pf_pairs;  // (query, visible key) pairs of the prefilling sequences
-    int pf_ctx;                 // their contexts (this step's tokens included), summed
-    const int32_t* pf_kv_off;   // [B] device: running sum of those contexts, -1 for sequences with a single token
+    double pf_pairs;  // (query, earlier or same key) pairs of the prefilling sequences
+    struct Gather {             // the context rows that these see under one mask (b2_layered_gathers)
+        int rows;
+        const int32_t* kv_off;  // [B] device: first row of each, -1 for sequences with a single token
+    };
+    const Gather* gather;
+    const std::vector<SeqStep>* seqs;
     int n_logits;
     const int32_t* logit_rows;
 };
 int32_t b2_forward_layered(b2_model* m, b2_pool* pool, const LayeredStep& s, float** logits_dev, int* logits_ld);
 int b2_layered_q_tile(const b2_model* m);
+const std::vector<MaskSpec>& b2_layered_gathers(const b2_model* m);  // distinct masks of the latent layers
 int b2_layered_chunk_tiles(const b2_model* m, const std::vector<SeqStep>& seqs);  // 16-key tiles per work item of the decode attention
 int b2_small_cta_chunk_tiles(long dec_ctx_sum, int blocks, int sm_count);  // ... for kernels with several CTAs per SM and `blocks` CTAs per item
 bool b2_tensor_to_f32(const HostTensor& t, std::vector<float>& out);

@@ -2,7 +2,8 @@
 //
 // The forward is called by the engine's step (b2_engine_forward) with the packer's metadata, like the flat decoders'
 // layers; pages, block tables, recurrent slots, scheduling and sampling are the engine's.  The residual stream is f32.
-// Every sub-layer leaves what it adds in `y` (f32); the next norm adds it to the stream on its way (b2_add_norm_launch).
+// Every sub-layer leaves what it adds in `y` (f32); the next norm adds it to the stream on its way (b2_add_norm_launch; with several
+// streams b2_stream_norm_launch).
 #include <algorithm>
 #include <cmath>
 #include <cstring>
@@ -24,21 +25,32 @@ struct GroupW {  // one matrix per group (expert or head), [G][N][K], N and K pa
 };
 struct LayerP {
     float *norm1 = nullptr, *norm2 = nullptr;
+    // several streams: what the mixer (0) and the feed-forward (1) read, leave behind and add
+    struct {
+        float *from = nullptr, *mix = nullptr, *to = nullptr;
+    } hc[2];
     // latent attention
     Proj qkv, attn_o;  // rows: q | latent | rotated key part
     float* c_norm = nullptr;
     GroupW k_up_t, v_up;  // [head][kv_rank][dim] and [head][vdim][kv_rank]
     Proj kv_up;           // the same matrices for whole contexts (bf16): plain keys, then values, heads padded to 64-row blocks
-    int rope = -1;
+    int rope = -1, gather = 0;
     // mamba2
     Proj ssm_in, ssm_o;
     float *conv_w = nullptr, *conv_b = nullptr, *dt_bias = nullptr, *A_log = nullptr, *D = nullptr, *ssm_norm = nullptr;
     // feed-forward
-    Proj gu, down, router;
+    Proj gu, down, router;  // router: experts | identity experts | the shared expert's number
     GroupW e_gu, e_down;
+    Proj s_gu, s_down;      // the shared expert
+    float* correction = nullptr;
     // Layers of grouped attention and memories: one product for everything that reads the normed stream, one for everything
     // that is added to it (columns: attention heads | memory heads | feed-forward).
     Proj in, lr, out;  // lr: the second factors of a memory's decay and gate, block-diagonal
+    // token shift: `in` holds four matrices that read a mixture each (r, k, v, gate; part_n rows apart), w1 the decay's first factor
+    // (lr its second one)
+    Proj w1;
+    int part_n = 0, rank = 0;
+    float *mu = nullptr, *bonus = nullptr;
     struct {
         int q = 0, k = 0, v = 0, c = 0, gate = 0, beta = 0, decay = 0, up = 0;  // columns of `in`
         int lr_gate = 0;                                                       // columns of `lr`: decay from 0, gate
@@ -66,6 +78,7 @@ struct LayeredModel {
     float* final_norm = nullptr;
     std::vector<RopeTab> ropes;
     int rope_positions = 0;
+    std::vector<MaskSpec> gathers;  // distinct masks of the latent layers, whose contexts a step gathers
     int64_t state_floats = 0;
     int* route_counters = nullptr;
     // prefill attention: gathered latents, rotated key parts and expanded keys / values of the contexts in a step
@@ -272,7 +285,7 @@ int32_t load_branches(Filler& f, LayeredModel& lm, int i) {
     const MemorySpec& s = L.mem;
     auto aq = [&](const std::string& n) { return tn.layer_key(i, tn.mixer + "." + L.gqa_key + n); };
     auto am = [&](const std::string& n) { return tn.layer_key(i, tn.mixer + "." + L.mem_key + n); };
-    const bool ff = L.parallel && L.mlp == MlpKind::DensePlain;
+    const bool ff = L.parallel && L.mlp == MlpKind::DensePlain, own_kv = L.kv_from < 0;
     B2_REQUIRE(L.mlp == MlpKind::None || L.parallel == (L.mlp == MlpKind::DensePlain), B2_ERR_UNSUPPORTED,
                "plain feed-forwards belong to parallel layers, gated and routed ones to sequential layers");
     int n = 0, ra = 0, rg = 0, ra8 = 0, need = 0;
@@ -283,8 +296,8 @@ int32_t load_branches(Filler& f, LayeredModel& lm, int i) {
     if (L.has_gqa()) {
         B2_REQUIRE(a.dim <= 256 && a.vdim <= 256, B2_ERR_UNSUPPORTED, "grouped attention: head sizes up to 256");
         take(P.at.q, a.heads * a.dim);
-        take(P.at.k, a.kv_heads * a.dim);
-        take(P.at.v, a.kv_heads * a.vdim);
+        if (own_kv) take(P.at.k, a.kv_heads * a.dim);
+        if (own_kv) take(P.at.v, a.kv_heads * a.vdim);
     }
     if (L.has_mem()) {
         B2_REQUIRE(s.dim <= 256, B2_ERR_UNSUPPORTED, "memory: key sizes up to 256");
@@ -306,8 +319,10 @@ int32_t load_branches(Filler& f, LayeredModel& lm, int i) {
     B2_CHECK(f.proj(P.in, std::max(n, need), W));
     if (L.has_gqa()) {
         B2_CHECK(f.rows(P.in, P.at.q, aq("q"), a.heads * a.dim, W));
-        B2_CHECK(f.rows(P.in, P.at.k, aq("k"), a.kv_heads * a.dim, W));
-        B2_CHECK(f.rows(P.in, P.at.v, aq("v"), a.kv_heads * a.vdim, W));
+        if (own_kv) {
+            B2_CHECK(f.rows(P.in, P.at.k, aq("k"), a.kv_heads * a.dim, W));
+            B2_CHECK(f.rows(P.in, P.at.v, aq("v"), a.kv_heads * a.vdim, W));
+        }
         if (a.bias) {
             B2_CHECK(f.vec(P.q_bias, aq("q.b"), {a.heads * a.dim}, 0.f, 0.1f));
             B2_CHECK(f.vec(P.k_bias, aq("k.b"), {a.kv_heads * a.dim}, 0.f, 0.1f));
@@ -316,6 +331,10 @@ int32_t load_branches(Filler& f, LayeredModel& lm, int i) {
         if (a.qk_norm) {
             B2_CHECK(f.vec(P.q_norm, aq("q.norm"), {a.dim}, 1.f, 0.f));
             B2_CHECK(f.vec(P.k_norm, aq("k.norm"), {a.dim}, 1.f, 0.f));
+        }
+        if (a.norm_all) {
+            B2_CHECK(f.vec(P.q_norm, aq("q.norm"), {a.heads * a.dim}, 1.f, 0.f));
+            if (own_kv) B2_CHECK(f.vec(P.k_norm, aq("k.norm"), {a.kv_heads * a.dim}, 1.f, 0.f));
         }
         P.rope = rope_table(lm, a.rot);
         lm.dec_part_row = std::max(lm.dec_part_row, (size_t)a.heads * (a.v_row() + 2));
@@ -382,6 +401,45 @@ int32_t load_branches(Filler& f, LayeredModel& lm, int i) {
     return B2_OK;
 }
 
+// A memory behind a token shift: r, k, v and gate read a mixture of their own each, the decay comes from two factors.
+int32_t load_shifted(Filler& f, LayeredModel& lm, int i) {
+    const LayerSpec& L = lm.spec.layers[i];
+    const TensorNames& tn = lm.spec.names;
+    LayerP& P = lm.layers[i];
+    const int W = lm.spec.width;
+    const MemorySpec& s = L.mem;
+    auto key = [&](const std::string& n) { return tn.layer_key(i, tn.mixer + "." + L.mem_key + n); };
+    B2_REQUIRE(s.dim <= 256 && s.shift == W, B2_ERR_UNSUPPORTED, "memory: key sizes up to 256");
+    const int Q = s.q_cols(), V = s.heads * s.vdim;
+    B2_REQUIRE(Q == V, B2_ERR_UNSUPPORTED, "token shift: keys and values of one size");
+    P.part_n = pad_n(Q);
+    B2_CHECK(f.proj(P.in, 4 * P.part_n, W));
+    std::vector<float> mu;
+    const char* parts[5] = {"r", "k", "v", "g", "w"};
+    for (int j = 0; j < 5; j++) {
+        if (j < 4) B2_CHECK(f.rows(P.in, j * P.part_n, key(parts[j]), Q, W));
+        if (f.w) {
+            B2_CHECK(f.fetch(key(std::string("mu.") + parts[j]), {W}));
+            mu.insert(mu.end(), f.host.begin(), f.host.end());
+        }
+    }
+    if (f.w)
+        B2_CHECK(f.upload(P.mu, mu));
+    else
+        B2_CHECK(f.vec(P.mu, "", {5, W}, 0.4f, 0.2f));
+    B2_CHECK(f.rows_of(key("w1"), std::max(8, s.dim), &P.rank));
+    B2_CHECK(f.proj(P.w1, P.rank, W));
+    B2_CHECK(f.rows(P.w1, 0, key("w1"), P.rank, W));
+    B2_CHECK(f.proj(P.lr, Q, P.rank));
+    B2_CHECK(f.rows(P.lr, 0, key("w2"), Q, P.rank));
+    B2_CHECK(f.vec(P.dt_bias, key("w0"), {Q}, -3.f, 1.5f));
+    B2_CHECK(f.vec(P.bonus, key("u"), {s.heads, s.dim}, 0.5f, 0.3f));
+    B2_CHECK(f.vec(P.mem_norm, key("norm"), {V}, 1.f, 0.f));
+    P.at.gate = 3 * Q;
+    B2_CHECK(f.proj(P.out, W, V));
+    return f.rows(P.out, 0, key("o"), W, V);
+}
+
 int32_t load_layer(Filler& f, LayeredModel& lm, int i) {
     const LayerSpec& L = lm.spec.layers[i];
     const TensorNames& tn = lm.spec.names;
@@ -391,7 +449,17 @@ int32_t load_layer(Filler& f, LayeredModel& lm, int i) {
     auto mix = [&](const std::string& s) { return tn.layer_key(i, tn.mixer + "." + s); };
     auto mlp = [&](const std::string& s) { return tn.layer_key(i, tn.mlp + "." + s); };
     B2_CHECK(f.vec(P.norm1, key(tn.norm1), {W}, 1.f, 0.f, false, lm.spec.norm_offset));
-    if (L.has_gqa() || L.has_mem()) {
+    for (int q = 0; q < (lm.spec.streams > 0 ? L.mlp == MlpKind::None ? 1 : 2 : 0); q++) {
+        const int n = lm.spec.streams;
+        const std::string hc = "hc" + std::to_string(q + 1) + ".";
+        B2_CHECK(f.vec(P.hc[q].from, key(hc + "in"), {n}, 1.f / n, 0.1f / n));
+        B2_CHECK(f.vec(P.hc[q].mix, key(hc + "mix"), {n, n}, 1.f / n, 0.1f / n));
+        B2_CHECK(f.vec(P.hc[q].to, key(hc + "out"), {n}, 1.f, 0.2f));
+    }
+    if (L.mixer == MixerKind::Memory && L.mem.shift > 0) {
+        B2_REQUIRE(!L.parallel, B2_ERR_UNSUPPORTED, "a token shift in a parallel layer");
+        B2_CHECK(load_shifted(f, lm, i));
+    } else if (L.has_gqa() || L.has_mem()) {
         B2_CHECK(load_branches(f, lm, i));
         if (L.parallel) return B2_OK;
     } else if (L.parallel) {
@@ -419,7 +487,9 @@ int32_t load_layer(Filler& f, LayeredModel& lm, int i) {
         lm.dec_part_row = std::max(lm.dec_part_row, (size_t)a.heads * (a.kv_rank + 2));
         B2_CHECK(f.proj(P.attn_o, W, a.heads * a.vdim));
         B2_CHECK(f.rows(P.attn_o, 0, mix("o"), W, a.heads * a.vdim));
-        P.rope = rope_table(lm, a.rot);
+        while (P.gather < (int)lm.gathers.size() && !(lm.gathers[P.gather] == a.mask)) P.gather++;
+        if (P.gather == (int)lm.gathers.size()) lm.gathers.push_back(a.mask);
+        if (a.rot_dim > 0) P.rope = rope_table(lm, a.rot);
     } else {
         const Mamba2Spec& s = L.ssm;
         B2_CHECK(f.proj(P.ssm_in, s.in_rows(), W));
@@ -445,8 +515,18 @@ int32_t load_layer(Filler& f, LayeredModel& lm, int i) {
     } else {
         const RoutedSpec& r = L.moe;
         const int ffp = up(r.ff, 64);
-        B2_CHECK(f.proj(P.router, r.experts, W));
-        B2_CHECK(f.rows(P.router, 0, mlp("router"), r.experts, W));
+        B2_CHECK(f.proj(P.router, r.outputs() + (r.shared_ff > 0 ? 1 : 0), W));
+        B2_CHECK(f.rows(P.router, 0, mlp("router"), r.outputs(), W));
+        if (r.score == RouteScore::Softmax) B2_CHECK(f.vec(P.correction, mlp("correction"), {r.outputs()}, 0.f, 0.01f));
+        if (r.shared_ff > 0) {
+            const int sp = up(r.shared_ff, 64);
+            B2_CHECK(f.rows(P.router, r.outputs(), mlp("shared.sg"), 1, W));
+            B2_CHECK(f.proj(P.s_gu, 2 * sp, W));
+            B2_CHECK(f.rows(P.s_gu, 0, mlp("shared.gate"), r.shared_ff, W));
+            B2_CHECK(f.rows(P.s_gu, sp, mlp("shared.up"), r.shared_ff, W));
+            B2_CHECK(f.proj(P.s_down, W, r.shared_ff));
+            B2_CHECK(f.rows(P.s_down, 0, mlp("shared.down"), W, r.shared_ff));
+        }
         B2_CHECK(f.group(P.e_gu, r.experts, 2 * ffp, W));
         B2_CHECK(f.group(P.e_down, r.experts, W, r.ff));
         for (int e = 0; e < r.experts; e++) {
@@ -462,7 +542,7 @@ int32_t load_layer(Filler& f, LayeredModel& lm, int i) {
 // floats of a layer's recurrent record
 int64_t record_floats(const LayerSpec& L) {
     if (L.mixer == MixerKind::Mamba2) return up(L.ssm.inner() * L.ssm.state, 4) + up(L.ssm.channels() * (L.ssm.conv - 1), 4);
-    return L.has_mem() ? up(L.mem.state_floats() + L.mem.channels() * L.mem.keep(), 4) : 0;
+    return L.has_mem() ? up(L.mem.state_floats() + L.mem.channels() * L.mem.keep() + L.mem.shift, 4) : 0;
 }
 
 // ---- workspace ------------------------------------------------------------------------------------------------------
@@ -494,7 +574,8 @@ struct SsmBufs {
     int ld_xbc, ld_gn;
 };
 struct BranchBufs {
-    void *in, *lr, *q, *v, *row;
+    void *in, *lr, *q, *v, *row, *mix, *low;
+    float *low_f;
     float *mq, *mk, *lg, *beta, *o;
     int ld_v;
 };
@@ -503,20 +584,20 @@ struct DenseBufs {
     int ld_act;
 };
 struct MoeBufs {
-    float *logits, *weight, *row_w;
+    float *logits, *weight, *row_w, *pass, *shared_w;
     int32_t *expert, *offsets, *pos, *src;
-    void *xs, *gu, *act;
+    void *xs, *gu, *act, *s_gu, *s_act;
     int ld_act;
 };
 Common carve_common(Carver& c, const LayeredModel& lm, size_t es, size_t t, size_t l) {
     Common o;
-    int top = 1;
+    int top = 1;  // rows of y per token
     for (auto& L : lm.spec.layers)
-        if (L.mlp == MlpKind::Routed) top = std::max(top, L.moe.top);
+        if (L.mlp == MlpKind::Routed) top = std::max(top, L.moe.sources());
     o.ldx = pad_n(lm.spec.width);
     o.ldn = pad_k(lm.spec.width);
     o.ldl = pad_n(lm.spec.vocab);
-    o.x = c.take<float>(t * o.ldx * 4);
+    o.x = c.take<float>(t * o.ldx * std::max(lm.spec.streams, 1) * 4);
     o.y = c.take<float>(t * top * o.ldx * 4);
     o.xn = c.take(t * o.ldn * es);
     o.last = c.take(l * o.ldn * es);
@@ -555,7 +636,12 @@ BranchBufs carve_branches(Carver c, const LayerSpec& L, const LayerP& P, size_t 
     o.row = c.take(t * P.out.K * es);
     if (L.has_gqa()) o.q = c.take(t * L.gqa.heads * L.gqa.k_row() * es);
     if (L.has_mem()) {
-        o.lr = c.take(t * P.lr.N * es);
+        o.lr = c.take(t * P.lr.N * (s.shift > 0 ? 4 : es));
+        if (s.shift > 0) {
+            o.mix = c.take(t * 5 * pad_k(s.shift) * es);
+            o.low_f = c.take<float>(t * P.w1.N * 4);
+            o.low = c.take(t * P.lr.K * es);
+        }
         o.ld_v = up(s.heads * s.vdim, 8);
         o.v = s.conv > 0 ? c.take(t * o.ld_v * es) : nullptr;
         o.mq = c.take<float>(t * s.q_cols() * 4);
@@ -582,13 +668,17 @@ MoeBufs carve_moe(Carver c, const RoutedSpec& r, const LayerP& P, int ldn, size_
     o.logits = c.take<float>(t * P.router.N * 4);
     o.weight = c.take<float>(n * 4);
     o.row_w = c.take<float>(n * 4);
+    o.pass = c.take<float>(t * 4);
+    o.shared_w = c.take<float>(t * 4);
     o.expert = c.take<int32_t>(n * 4);
-    o.pos = c.take<int32_t>(n * 4);
+    o.pos = c.take<int32_t>(t * r.sources() * 4);
     o.src = c.take<int32_t>(n * 4);
     o.offsets = c.take<int32_t>((size_t)(r.experts + 1) * 4);
     o.xs = c.take(es == 2 ? n * ldn * es : 0);
     o.gu = c.take(n * P.e_gu.N * es);
     o.act = c.take(n * o.ld_act * es);
+    o.s_gu = c.take(t * P.s_gu.N * es);
+    o.s_act = c.take(t * P.s_down.K * es);
     *end = std::max(*end, c.off);
     return o;
 }
@@ -643,7 +733,7 @@ int32_t ensure_expand(b2_model* m, int rows) {
     B2_CUDA(cudaStreamSynchronize(m->ctx->stream));
     lm.kv_cap = up(std::max(rows + rows / 8, 1024), 128);
     B2_CHECK(regrow_zero(m->ctx, lm.kv_lat, (size_t)lm.kv_cap * lm.kv_ld_lat));
-    B2_CHECK(regrow_zero(m->ctx, lm.kv_rot, (size_t)lm.kv_cap * lm.kv_ld_rot));
+    B2_CHECK(regrow_zero(m->ctx, lm.kv_rot, std::max<size_t>((size_t)lm.kv_cap * lm.kv_ld_rot, 8)));
     return regrow_zero(m->ctx, lm.kv_exp, (size_t)lm.kv_cap * lm.kv_ld_exp);
 }
 int32_t ensure_decode(b2_model* m, int items) {
@@ -686,6 +776,61 @@ int32_t linear(b2_model* m, const Proj& p, const void* x, int ldx, int M, int ro
     return b2_gemm_launch(m->ctx, g);
 }
 
+// Keys that the single tokens of a step see under a mask: in all, and the most 16-key tiles of one token.
+struct DecodeKeys {
+    long sum = 0;
+    int tiles = 1;
+};
+DecodeKeys decode_keys(const std::vector<SeqStep>& seqs, const MaskSpec& mask) {
+    DecodeKeys k;
+    for (auto& s : seqs)
+        if (s.n == 1) {
+            const int lo = mask.first(s.cache->len);
+            k.sum += s.cache->len + 1 - lo;
+            k.tiles = std::max(k.tiles, s.cache->len / 16 - lo / 16 + 1);
+        }
+    return k;
+}
+double masked_pairs(const LayeredStep& s, const MaskSpec& mask) {  // (query, visible key) pairs of the prefilling sequences
+    if (mask.kind == MaskSpec::None) return s.pf_pairs;
+    double n = 0;
+    for (auto& q : *s.seqs)
+        for (int i = 0; q.n > 1 && i < q.n; i++) n += q.cache->len + i + 1 - mask.first(q.cache->len + i);
+    return n;
+}
+// Latent decode attention: one CTA fills an SM, so the work items (times the head groups) should fill whole rounds of the
+// machine: the smallest chunk, in whole tiles from 128 keys on, that does not open another round.
+struct DecodeSplit {
+    int chunk_tiles, row_chunks;  // 16-key boxes per chunk; most chunks of a row
+};
+DecodeSplit latent_split(const b2_ctx* ctx, int groups, const MaskSpec& mask, const std::vector<SeqStep>& seqs) {
+    const int tile = b2_latent_decode_tile();
+    int rows = 0, longest = 1;
+    auto keys_of = [&](const SeqStep& s) { return s.cache->len + 1 - mask.first(s.cache->len) / 16 * 16; };
+    for (auto& s : seqs)
+        if (s.n == 1) {
+            rows++;
+            longest = std::max(longest, keys_of(s));
+        }
+    const int sms = ctx->sm_count, budget = std::max(1, (rows * groups + sms - 1) / sms) * sms / groups;
+    auto items = [&](int keys) {
+        int n = 0;
+        for (auto& s : seqs)
+            if (s.n == 1) n += (keys_of(s) + keys - 1) / keys;
+        return n;
+    };
+    int lo = (128 + tile - 1) / tile, hi = std::max(lo, (longest + tile - 1) / tile);  // in tiles; the longest context in one chunk is one item per row
+    while (lo < hi) {
+        const int mid = (lo + hi) / 2;
+        if (items(mid * tile) <= budget)
+            hi = mid;
+        else
+            lo = mid + 1;
+    }
+    return {lo * tile / 16, (longest + lo * tile - 1) / (lo * tile)};
+}
+int latent_head_groups(const LatentAttnSpec& a) { return a.heads > 16 ? (a.heads + 31) / 32 : 1; }
+
 struct Fwd {  // one step
     b2_model* m;
     LayeredModel& lm;
@@ -701,8 +846,9 @@ struct Fwd {  // one step
     int32_t branches(const LayerSpec& L, const LayerP& P, int run);
     int32_t attend(const LayerSpec& L, const LayerP& P, const BranchBufs& b, int run);
     int32_t remember(const LayerSpec& L, const LayerP& P, const BranchBufs& b, int run);
+    int32_t shift(const LayerSpec& L, const LayerP& P, const BranchBufs& b, int run);
     int32_t dense(const LayerSpec& L, const LayerP& P);
-    int32_t moe(const LayerSpec& L, const LayerP& P, const int32_t** rows);
+    int32_t moe(const LayerSpec& L, const LayerP& P, const int32_t** rows, const float** pass);
 };
 
 int32_t Fwd::latent(const LayerSpec& L, const LayerP& P, int run) {
@@ -719,8 +865,10 @@ int32_t Fwd::latent(const LayerSpec& L, const LayerP& P, int run) {
     pp.T = T;
     pp.positions = s.mo->positions;
     pp.slot_mapping = s.mo->slot_mapping;
-    pp.cos_t = lm.ropes[P.rope].cos;
-    pp.sin_t = lm.ropes[P.rope].sin;
+    if (P.rope >= 0) {
+        pp.cos_t = lm.ropes[P.rope].cos;
+        pp.sin_t = lm.ropes[P.rope].sin;
+    }
     pp.c_norm = P.c_norm;
     pp.eps = lm.spec.eps;
     pp.cache = cache;
@@ -733,25 +881,27 @@ int32_t Fwd::latent(const LayerSpec& L, const LayerP& P, int run) {
 
     // Portions of more than a token: keys and values of their contexts expanded per head.  Otherwise (single tokens, f32,
     // head sizes or contexts outside that kernel's reach) attention in latent coordinates.
-    const bool expand = s.pf_work > 0 && P.kv_up.w && (size_t)s.pf_ctx * P.kv_up.N * 2 <= kMaxExpandBytes;
+    const LayeredStep::Gather& ga = s.gather[P.gather];
+    const bool expand = s.pf_work > 0 && P.kv_up.w && (size_t)ga.rows * P.kv_up.N * 2 <= kMaxExpandBytes;
     if (expand) {
-        B2_CHECK(ensure_expand(m, s.pf_ctx));
+        B2_CHECK(ensure_expand(m, ga.rows));
         LatentGatherParams gp{};
         gp.cache = cache;
         gp.block_tables = pool->block_tables;
         gp.max_blocks = pool->max_blocks;
         gp.page_size = pool->block_size;
         gp.B = s.B;
-        gp.rows = s.pf_ctx;
+        gp.rows = ga.rows;
         gp.seq_slot = s.in->seq_slot;
         gp.context_lens = s.mo->context_lens;
-        gp.kv_off = s.pf_kv_off;
+        gp.kv_off = ga.kv_off;
+        gp.cu_seqlens = s.mo->cu_seqlens;
         gp.lat = lm.kv_lat;
         gp.ld_lat = P.kv_up.K;
         gp.rot = lm.kv_rot;
         gp.rot_pad = b.rot_pad;
         B2_CHECK(b2_latent_gather_launch(ctx, a, gp));
-        B2_CHECK(linear(m, P.kv_up, lm.kv_lat, P.kv_up.K, s.pf_ctx, lm.kv_cap, lm.kv_exp, P.kv_up.N, false));
+        B2_CHECK(linear(m, P.kv_up, lm.kv_lat, P.kv_up.K, ga.rows, lm.kv_cap, lm.kv_exp, P.kv_up.N, false));
         LatentPrefillParams fp{};
         fp.q = b.q;
         fp.q_rows = lm.t_cap;
@@ -766,14 +916,14 @@ int32_t Fwd::latent(const LayerSpec& L, const LayerP& P, int run) {
         fp.n_work = s.mo->counts + 3;
         fp.cu_seqlens = s.mo->cu_seqlens;
         fp.context_lens = s.mo->context_lens;
-        fp.kv_off = s.pf_kv_off;
+        fp.kv_off = ga.kv_off;
         fp.scale_log2 = scale_log2;
         fp.out = b.att;
         fp.ldo = b.ld_att;
         fp.vdim = a.vdim;
         b2_prof_mark(ctx, B2_CLS_ATTN_PREFILL);
         B2_CHECK(b2_latent_prefill_launch(ctx, a, fp, s.pf_work));
-        ctx->attn_prefill_flops += 2.0 * (a.dim + a.rot_dim + a.vdim) * a.heads * s.pf_pairs;
+        ctx->attn_prefill_flops += 2.0 * (a.dim + a.rot_dim + a.vdim) * a.heads * masked_pairs(s, a.mask);
     }
     // rows that attend in latent coordinates: the single tokens, or every token
     const int rows = expand ? s.n_dec : T;
@@ -817,10 +967,16 @@ int32_t Fwd::latent(const LayerSpec& L, const LayerP& P, int run) {
                 dp.n_work = s.mo->counts + 2;
                 dp.chunk_tiles = s.chunk_tiles;
                 items = s.dec_work;
+                if (a.mask.kind != MaskSpec::None) {  // not the packer's items: the same number for every row
+                    const DecodeSplit d = latent_split(m->ctx, latent_head_groups(a), a.mask, *s.seqs);
+                    dp.chunk_tiles = d.chunk_tiles;
+                    dp.row_chunks = d.row_chunks;
+                    items = rows * d.row_chunks;
+                }
                 B2_CHECK(ensure_decode(m, items));
                 dp.part_o = lm.dec_part;
                 dp.part_ml = lm.dec_part + (size_t)items * a.heads * a.kv_rank;
-                ctx->attn_decode_bytes += (double)s.dec_ctx_sum * W * 2;
+                ctx->attn_decode_bytes += (double)decode_keys(*s.seqs, a.mask).sum * W * 2;
             } else {  // one work item per token: nothing is split, no partial results
                 dp.positions = s.mo->positions;
                 dp.token_seq = s.mo->token_seq;
@@ -906,7 +1062,9 @@ int32_t Fwd::ssm(const LayerSpec& L, const LayerP& P, int run) {
 int32_t Fwd::attend(const LayerSpec& L, const LayerP& P, const BranchBufs& b, int run) {
     b2_ctx* ctx = m->ctx;
     const GroupedAttnSpec& a = L.gqa;
-    const KvPlane* planes = &pool->planes[pool->layer_plane[run]];
+    int kv_run = run;  // whose cache: this run's, or that of the last run of another layer
+    while (L.kv_from >= 0 && lm.runs[kv_run].layer != L.kv_from) kv_run--;
+    const KvPlane* planes = &pool->planes[pool->layer_plane[kv_run]];
     GqaPrepParams pp{};
     pp.in = b.in;
     pp.ld = P.in.N;
@@ -919,6 +1077,7 @@ int32_t Fwd::attend(const LayerSpec& L, const LayerP& P, const BranchBufs& b, in
     pp.v_bias = P.v_bias;
     pp.q_norm = P.q_norm;
     pp.k_norm = P.k_norm;
+    pp.own_kv = L.kv_from < 0;
     pp.eps = lm.spec.eps;
     pp.positions = s.mo->positions;
     pp.slot_mapping = s.mo->slot_mapping;
@@ -967,20 +1126,79 @@ int32_t Fwd::attend(const LayerSpec& L, const LayerP& P, const BranchBufs& b, in
         return rows ? b2_gqa_decode_launch(ctx, a, p, 0) : b2_gqa_simple_launch(ctx, m->f32, a, p);
     }
     if (s.n_dec > 0) {
-        B2_CHECK(ensure_decode(m, s.dec_work));
+        const DecodeKeys keys = decode_keys(*s.seqs, a.mask);
+        int items = s.dec_work;
+        if (a.mask.kind != MaskSpec::None) {  // not the packer's items: the same number for every row
+            p.chunk_tiles = b2_small_cta_chunk_tiles(keys.sum, b2_gqa_head_blocks(a), ctx->sm_count);
+            p.row_chunks = (keys.tiles + p.chunk_tiles - 1) / p.chunk_tiles;
+            items = s.n_dec * p.row_chunks;
+        }
+        B2_CHECK(ensure_decode(m, items));
         p.part_o = lm.dec_part;
-        p.part_ml = lm.dec_part + (size_t)s.dec_work * a.heads * a.v_row();
+        p.part_ml = lm.dec_part + (size_t)items * a.heads * a.v_row();
         B2_CHECK(b2_decode_attn_counters(ctx, s.n_dec, b2_gqa_head_blocks(a), &p.counters));
         b2_prof_mark(ctx, B2_CLS_ATTN_DECODE);
-        B2_CHECK(b2_gqa_decode_launch(ctx, a, p, s.dec_work));
-        ctx->attn_decode_bytes += (double)s.dec_ctx_sum * a.kv_heads * (a.dim + a.vdim) * 2;
+        B2_CHECK(b2_gqa_decode_launch(ctx, a, p, items));
+        ctx->attn_decode_bytes += (double)keys.sum * a.kv_heads * (a.dim + a.vdim) * 2;
     }
     if (s.pf_work > 0) {
         b2_prof_mark(ctx, B2_CLS_ATTN_PREFILL);
         B2_CHECK(b2_gqa_prefill_launch(ctx, a, p, s.pf_work));
-        ctx->attn_prefill_flops += 2.0 * (a.dim + a.vdim) * a.heads * s.pf_pairs;
+        ctx->attn_prefill_flops += 2.0 * (a.dim + a.vdim) * a.heads * masked_pairs(s, a.mask);
     }
     return B2_OK;
+}
+
+// What a memory behind a token shift reads: five mixtures, r | k | v | gate side by side in b.in, the decay's projection in b.lr (f32).
+int32_t Fwd::shift(const LayerSpec& L, const LayerP& P, const BranchBufs& b, int run) {
+    b2_ctx* ctx = m->ctx;
+    const MemorySpec& sp = L.mem;
+    const int ldm = 5 * c.ldn, Q = sp.q_cols();
+    ShiftParams h{};
+    h.h = c.xn;
+    h.ld_h = c.ldn;
+    h.T = s.T;
+    h.width = sp.shift;
+    h.ldo = c.ldn;
+    h.mu = P.mu;
+    h.out = b.mix;
+    h.cu_seqlens = s.mo->cu_seqlens;
+    h.context_lens = s.mo->context_lens;
+    h.token_seq = s.mo->token_seq;
+    h.seq_slot = s.in->seq_slot;
+    h.kept = pool->state + lm.run_state[run] + sp.state_floats();
+    h.slot_stride = pool->state_floats;
+    b2_prof_mark(ctx, B2_CLS_ELEMENTWISE);
+    B2_CHECK(b2_token_shift_launch(ctx, m->f32, h));
+    if (!m->f32 && s.T > 32 && P.part_n == Q) {  // whole tiles: four plain products
+        for (int j = 0; j < 4; j++) {
+            Proj part = P.in;
+            part.N = P.part_n;
+            part.w = (uint8_t*)P.in.w + (size_t)j * P.part_n * P.in.K * es;
+            B2_CHECK(linear(m, part, (const uint8_t*)b.mix + (size_t)j * c.ldn * es, ldm, s.T, lm.t_cap, (uint8_t*)b.in + (size_t)j * Q * es, P.in.N, false));
+        }
+    } else {
+        GroupedGemmParams g{};
+        g.x = b.mix;
+        g.x_gstride = c.ldn;
+        g.ldx = ldm;
+        g.w = P.in.w;
+        g.N = P.part_n;
+        g.K = P.in.K;
+        g.G = 4;
+        g.out = b.in;
+        g.out_gstride = Q;
+        g.ldo = P.in.N;
+        g.n_out = Q;
+        g.M = s.T;
+        g.x_rows = lm.t_cap;
+        b2_prof_mark(ctx, B2_CLS_GEMM);
+        B2_CHECK(b2_grouped_gemm_launch(ctx, m->f32, g));
+    }
+    B2_CHECK(linear(m, P.w1, (const uint8_t*)b.mix + (size_t)4 * c.ldn * es, ldm, s.T, lm.t_cap, b.low_f, P.w1.N, true));
+    b2_prof_mark(ctx, B2_CLS_ELEMENTWISE);
+    B2_CHECK(b2_tanh_launch(ctx, m->f32, b.low_f, P.w1.N, s.T, P.rank, b.low, P.lr.K));
+    return linear(m, P.lr, b.low, P.lr.K, s.T, lm.t_cap, b.lr, P.lr.N, true);
 }
 
 int32_t Fwd::remember(const LayerSpec& L, const LayerP& P, const BranchBufs& b, int run) {
@@ -990,7 +1208,13 @@ int32_t Fwd::remember(const LayerSpec& L, const LayerP& P, const BranchBufs& b, 
     p.ld = P.in.N;
     p.c_off = P.at.c;
     p.b_off = P.at.beta;
-    if (sp.low_rank) {
+    if (sp.shift > 0) {
+        p.dec = b.lr;
+        p.ld_dec = P.lr.N;
+        p.bonus = P.bonus;
+        p.h = c.xn;
+        p.ld_h = c.ldn;
+    } else if (sp.low_rank) {
         B2_CHECK(linear(m, P.lr, (const uint8_t*)b.in + P.at.gate * es, P.in.N, s.T, lm.t_cap, b.lr, P.lr.N, false));
         p.dec = b.lr;
         p.ld_dec = P.lr.N;
@@ -1035,7 +1259,10 @@ int32_t Fwd::remember(const LayerSpec& L, const LayerP& P, const BranchBufs& b, 
 
 int32_t Fwd::branches(const LayerSpec& L, const LayerP& P, int run) {
     const BranchBufs b = carve_branches(scratch, L, P, es, (size_t)lm.t_cap, &end);
-    B2_CHECK(linear(m, P.in, c.xn, c.ldn, s.T, lm.t_cap, b.in, P.in.N, false));
+    if (L.has_mem() && L.mem.shift > 0)
+        B2_CHECK(shift(L, P, b, run));
+    else
+        B2_CHECK(linear(m, P.in, c.xn, c.ldn, s.T, lm.t_cap, b.in, P.in.N, false));
     if (L.has_gqa()) B2_CHECK(attend(L, P, b, run));
     if (L.has_mem()) B2_CHECK(remember(L, P, b, run));
     BranchOutParams p{};
@@ -1052,6 +1279,7 @@ int32_t Fwd::branches(const LayerSpec& L, const LayerP& P, int run) {
         p.ld_gate = L.mem.low_rank ? P.lr.N : P.in.N;
         p.act = L.mem.gate;
         p.norm = P.mem_norm;
+        p.norm_heads = L.mem.norm_heads;
         p.eps = lm.spec.eps;
         p.scale = L.mem_scale;
     }
@@ -1074,7 +1302,7 @@ int32_t Fwd::dense(const LayerSpec& L, const LayerP& P) {
     return linear(m, P.down, b.act, b.ld_act, s.T, lm.t_cap, c.y, c.ldx, true);
 }
 
-int32_t Fwd::moe(const LayerSpec& L, const LayerP& P, const int32_t** rows) {
+int32_t Fwd::moe(const LayerSpec& L, const LayerP& P, const int32_t** rows, const float** pass) {
     b2_ctx* ctx = m->ctx;
     const RoutedSpec& r = L.moe;
     const MoeBufs b = carve_moe(scratch, r, P, c.ldn, es, (size_t)lm.t_cap, &end);
@@ -1085,6 +1313,13 @@ int32_t Fwd::moe(const LayerSpec& L, const LayerP& P, const int32_t** rows) {
     rp.T = s.T;
     rp.experts = r.experts;
     rp.top = r.top;
+    rp.score = r.score;
+    rp.identity = r.identity;
+    rp.shared = r.shared_ff > 0;
+    rp.correction = P.correction;
+    rp.scale = r.scale;
+    rp.pass = b.pass;
+    rp.shared_w = b.shared_w;
     rp.expert = b.expert;
     rp.weight = b.weight;
     rp.offsets = b.offsets;
@@ -1132,60 +1367,41 @@ int32_t Fwd::moe(const LayerSpec& L, const LayerP& P, const int32_t** rows) {
     d.x_rows = lm.t_cap * r.top;
     b2_prof_mark(ctx, B2_CLS_GEMM);
     B2_CHECK(b2_grouped_gemm_launch(ctx, m->f32, d));
+    if (r.shared_ff > 0) {  // its result: the rows of y behind the routed ones
+        B2_CHECK(linear(m, P.s_gu, c.xn, c.ldn, s.T, lm.t_cap, b.s_gu, P.s_gu.N, false));
+        b2_prof_mark(ctx, B2_CLS_ELEMENTWISE);
+        B2_CHECK(b2_gate_launch(ctx, m->f32, r.gate, b.s_gu, P.s_gu.N, up(r.shared_ff, 64), b.shared_w, s.T, r.shared_ff, b.s_act, P.s_down.K));
+        B2_CHECK(linear(m, P.s_down, b.s_act, P.s_down.K, s.T, lm.t_cap, c.y + (size_t)s.T * r.top * c.ldx, c.ldx, true));
+    }
     *rows = b.pos;
+    if (r.identity > 0) *pass = b.pass;
     return B2_OK;
 }
 
 }  // namespace
 
 int b2_layered_q_tile(const b2_model*) { return 128; }
-// One CTA of the decode attention fills an SM, so the work items (times the head groups) should fill whole rounds of the
-// machine: the smallest chunk, in whole tiles from 128 keys on, that does not open another round.
+// Work items of the layers without a mask (the packer's list).
 int b2_layered_chunk_tiles(const b2_model* m, const std::vector<SeqStep>& seqs) {
     int groups = 1, blocks = 0;
     bool latent = false;
     for (auto& L : m->layered->spec.layers) {
-        latent |= L.mixer == MixerKind::LatentAttention;
+        if (L.mixer == MixerKind::LatentAttention && L.attn.mask.kind == MaskSpec::None) {
+            latent = true;
+            groups = std::max(groups, latent_head_groups(L.attn));
+        }
         if (L.has_gqa()) blocks = std::max(blocks, b2_gqa_head_blocks(L.gqa));
     }
-    if (!latent) {  // several small CTAs per SM
-        long ctx_sum = 0;
-        for (auto& s : seqs)
-            if (s.n == 1) ctx_sum += s.cache->len + 1;
-        return b2_small_cta_chunk_tiles(ctx_sum, std::max(blocks, 1), m->ctx->sm_count);
-    }
-    for (auto& L : m->layered->spec.layers)
-        if (L.mixer == MixerKind::LatentAttention && L.attn.heads > 16) groups = std::max(groups, (L.attn.heads + 31) / 32);
-    int rows = 0, longest = 1;
-    for (auto& s : seqs)
-        if (s.n == 1) {
-            rows++;
-            longest = std::max(longest, s.cache->len + 1);
-        }
-    const int sms = m->ctx->sm_count, budget = std::max(1, (rows * groups + sms - 1) / sms) * sms / groups;
-    auto items = [&](int keys) {
-        int n = 0;
-        for (auto& s : seqs)
-            if (s.n == 1) n += (s.cache->len + keys) / keys;
-        return n;
-    };
-    const int tile = b2_latent_decode_tile();
-    int lo = (128 + tile - 1) / tile, hi = std::max(lo, (longest + tile - 1) / tile);  // in tiles; the longest context in one chunk is one item per row
-    while (lo < hi) {
-        const int mid = (lo + hi) / 2;
-        if (items(mid * tile) <= budget)
-            hi = mid;
-        else
-            lo = mid + 1;
-    }
-    return lo * tile / 16;
+    if (latent) return latent_split(m->ctx, groups, MaskSpec{}, seqs).chunk_tiles;
+    return b2_small_cta_chunk_tiles(decode_keys(seqs, MaskSpec{}).sum, std::max(blocks, 1), m->ctx->sm_count);  // several small CTAs per SM
 }
+const std::vector<MaskSpec>& b2_layered_gathers(const b2_model* m) { return m->layered->gathers; }
 
 void b2_layered_cache_layout(const b2_model* m, int block_size, std::vector<std::vector<size_t>>& page_bytes, int64_t& state_floats) {
     for (const LayerRun& r : m->layered->runs) {
         const LayerSpec& L = m->layered->spec.layers[r.layer];
         page_bytes.emplace_back();
-        if (L.has_gqa()) {
+        if (L.has_gqa() && L.kv_from < 0) {
             page_bytes.back().push_back((size_t)block_size * L.gqa.kv_heads * L.gqa.k_row() * esz(m));
             page_bytes.back().push_back((size_t)block_size * L.gqa.kv_heads * L.gqa.v_row() * esz(m));
         }
@@ -1233,6 +1449,13 @@ int32_t b2_model_build_layered(b2_ctx* ctx, const ModelSpec& spec, const b2_weig
     lm.spec = spec;
     lm.layers.resize(spec.layers.size());
     lm.runs = spec.runs();
+    for (auto& L : spec.layers) {
+        const RoutedSpec& r = L.moe;
+        B2_REQUIRE(spec.streams > 0 || L.mlp != MlpKind::Routed || (r.identity == 0 && r.score == RouteScore::Sigmoid), B2_ERR_UNSUPPORTED,
+                   "identity experts are available for models with several streams");
+    }
+    B2_REQUIRE(spec.streams <= kMaxStreams && (spec.streams == 0 || spec.loop.times == 0), B2_ERR_UNSUPPORTED,
+               "residual streams: up to 16, without repeated layers");
     for (const LayerRun& r : lm.runs) {
         lm.run_state.push_back(lm.state_floats);
         lm.state_floats += record_floats(spec.layers[r.layer]);
@@ -1299,7 +1522,7 @@ int32_t b2_forward_layered(b2_model* m, b2_pool* pool, const LayeredStep& s, flo
     const Common c = carve_common(carver, lm, esz(m), (size_t)lm.t_cap, (size_t)lm.l_cap);
     Fwd f{m, lm, pool, s, c, carver, esz(m)};
     b2_prof_mark(ctx, B2_CLS_ELEMENTWISE);
-    B2_CHECK(b2_embed_residual_launch(ctx, m->f32, lm.embed, c.ldn, s.ids_dev, s.T, spec.width, spec.vocab, c.x, c.ldx));
+    B2_CHECK(b2_embed_residual_launch(ctx, m->f32, lm.embed, c.ldn, s.ids_dev, s.T, spec.width, spec.vocab, c.x, c.ldx, std::max(spec.streams, 1)));
     AddNormParams an{};
     an.x = c.x;
     an.y = c.y;
@@ -1307,7 +1530,30 @@ int32_t b2_forward_layered(b2_model* m, b2_pool* pool, const LayeredStep& s, flo
     an.width = spec.width;
     an.eps = spec.eps;
     an.n_src = 0;  // nothing is pending behind the embedding
-    auto norm = [&](const float* w, int rows, const int32_t* row_idx, void* out, float scale, bool write) {
+    StreamNormParams sn{};
+    sn.x = c.x;
+    sn.streams = spec.streams;
+    sn.y = c.y;
+    sn.h = c.xn;
+    sn.ldx = sn.ldy = c.ldx;
+    sn.ldh = c.ldn;
+    sn.width = spec.width;
+    sn.eps = spec.eps;
+    // takes up what is pending, then norms (w null: only the addition); `from`: weights of the streams, null for their sum
+    auto norm = [&](const float* w, const float* from, int rows, const int32_t* row_idx, void* out, float scale, bool write, float* sum = nullptr) {
+        b2_prof_mark(ctx, B2_CLS_ELEMENTWISE);
+        if (spec.streams > 0) {
+            sn.from = from;
+            sn.w = w;
+            sn.rows = rows;
+            sn.row_idx = row_idx;
+            sn.out = out;
+            sn.ldo = c.ldn;
+            sn.out_scale = scale;
+            sn.sum = sum;
+            sn.write_x = write && sn.mix;
+            return b2_stream_norm_launch(ctx, m->f32, sn);
+        }
         an.w = w;
         an.rows = rows;
         an.row_idx = row_idx;
@@ -1315,15 +1561,19 @@ int32_t b2_forward_layered(b2_model* m, b2_pool* pool, const LayeredStep& s, flo
         an.ldo = c.ldn;
         an.out_scale = scale;
         an.write_x = write && (an.n_src > 0 || an.vec || an.table);
-        b2_prof_mark(ctx, B2_CLS_ELEMENTWISE);
         return b2_add_norm_launch(ctx, m->f32, an);
     };
-    auto pending = [&](const int32_t* rows, int n) {
-        an.y_rows = rows;
-        an.n_src = n;
+    auto pending = [&](const LayerP* P, int q, const int32_t* rows, int n, const float* pass = nullptr) {
+        an.y_rows = sn.y_rows = rows;
+        an.n_src = sn.n_src = n;
+        sn.mix = P ? P->hc[q].mix : nullptr;
+        sn.to = P ? P->hc[q].to : nullptr;
+        sn.pass = pass;
     };
     const int64_t per_layer = (int64_t)s.T * spec.width;
     const bool capture = lm.capture && lm.capture_cap >= per_layer * (int64_t)lm.runs.size();
+    float* sums = nullptr;  // of the streams
+    if (capture && spec.streams > 0) B2_CUDA(cudaMallocAsync((void**)&sums, (size_t)s.T * c.ldx * 4, ctx->stream));
     for (size_t r = 0; r < lm.runs.size(); r++) {
         const LayerRun& run = lm.runs[r];
         const LayerSpec& L = spec.layers[run.layer];
@@ -1337,31 +1587,33 @@ int32_t b2_forward_layered(b2_model* m, b2_pool* pool, const LayeredStep& s, flo
                 an.vocab = spec.vocab;
             }
         }
-        B2_CHECK(norm(P.norm1, s.T, nullptr, c.xn, 1.f, true));
+        B2_CHECK(norm(P.norm1, P.hc[0].from, s.T, nullptr, c.xn, 1.f, true));
         an.vec = nullptr;
         an.table = nullptr;
         B2_CHECK(L.mixer == MixerKind::LatentAttention ? f.latent(L, P, (int)r) : L.mixer == MixerKind::Mamba2 ? f.ssm(L, P, (int)r) : f.branches(L, P, (int)r));
-        pending(nullptr, 1);
+        pending(&P, 0, nullptr, 1);
         if (L.mlp != MlpKind::None && !L.parallel) {
-            B2_CHECK(norm(P.norm2, s.T, nullptr, c.xn, 1.f, true));
+            B2_CHECK(norm(P.norm2, P.hc[1].from, s.T, nullptr, c.xn, 1.f, true));
             const int32_t* rows = nullptr;
+            const float* pass = nullptr;
             if (L.mlp == MlpKind::DenseGated) {
                 B2_CHECK(f.dense(L, P));
-                pending(nullptr, 1);
+                pending(&P, 1, nullptr, 1);
             } else {
-                B2_CHECK(f.moe(L, P, &rows));
-                pending(rows, L.moe.top);
+                B2_CHECK(f.moe(L, P, &rows, &pass));
+                pending(&P, 1, rows, L.moe.sources(), pass);
             }
         }
         if (capture) {
-            B2_CHECK(norm(nullptr, s.T, nullptr, nullptr, 1.f, true));  // the addition alone
-            pending(nullptr, 0);
-            B2_CUDA(cudaMemcpy2DAsync(lm.capture + (int64_t)r * per_layer, (size_t)spec.width * 4, c.x, (size_t)c.ldx * 4, (size_t)spec.width * 4, (size_t)s.T,
+            B2_CHECK(norm(nullptr, nullptr, s.T, nullptr, nullptr, 1.f, true, sums));  // the addition alone
+            pending(nullptr, 0, nullptr, 0);
+            B2_CUDA(cudaMemcpy2DAsync(lm.capture + (int64_t)r * per_layer, (size_t)spec.width * 4, sums ? sums : c.x, (size_t)c.ldx * 4, (size_t)spec.width * 4, (size_t)s.T,
                                       cudaMemcpyDeviceToHost, ctx->stream));
         }
     }
+    if (sums) B2_CUDA(cudaFreeAsync(sums, ctx->stream));
     if (s.n_logits > 0) {
-        B2_CHECK(norm(lm.final_norm, s.n_logits, s.logit_rows, c.last, spec.logit_scale, false));
+        B2_CHECK(norm(lm.final_norm, nullptr, s.n_logits, s.logit_rows, c.last, spec.logit_scale, false));
         Proj head;
         head.N = pad_n(spec.vocab);
         head.K = c.ldn;

@@ -333,12 +333,13 @@ int32_t b2_engine_forward(b2_model* m, std::vector<SeqStep>& seqs, void* logits_
     int W = 0, P = 0;
     double pf_flops = 0;  // 4*hd*hq flops per (query, visible key) pair
     int pf_max_ctx = 0;   // longest context among the sequences that prefill in this step
-    int pf_ctx = 0, n_chunks = 0;
+    int n_chunks = 0;
+    std::vector<LayeredStep::Gather> gather;  // of a layered model: context rows its latent layers gather, per mask
+    if (m->layered) gather.resize(b2_layered_gathers(m).size());
     double pf_pairs = 0;
     for (auto& s : seqs) {
         if (s.n > 1) {
             pf_pairs += (double)s.n * s.cache->len + 0.5 * (double)s.n * (s.n + 1);
-            pf_ctx += s.cache->len + s.n;
         }
         if (s.n > 1) pf_max_ctx = std::max(pf_max_ctx, s.cache->len + s.n);
         if (s.n > 1) pf_flops += 4.0 * c.head_dim * m->hq_l * ((double)s.n * s.cache->len + 0.5 * (double)s.n * (s.n + 1));
@@ -351,7 +352,7 @@ int32_t b2_engine_forward(b2_model* m, std::vector<SeqStep>& seqs, void* logits_
     }
     if (all_positions) n_logits = T;  // rows 0..T-1 of the step, in order
     const int U = (int)pool->upd_slot.size();
-    const size_t stage_ints = 4 * (size_t)B + 3 * (size_t)U + (size_t)T + (listed ? (size_t)n_logits : 0) + (m->layered ? 2 * (size_t)B : 0);
+    const size_t stage_ints = 4 * (size_t)B + 3 * (size_t)U + (size_t)T + (listed ? (size_t)n_logits : 0) + (m->layered ? (1 + gather.size()) * (size_t)B : 0);
     B2_CHECK(ensure_workspace(m, T, std::max(B, n_logits), W, P, stage_ints));
     Workspace& w = m->ws;
     int32_t* sh = w.stage_host;
@@ -382,11 +383,15 @@ int32_t b2_engine_forward(b2_model* m, std::vector<SeqStep>& seqs, void* logits_
                 row0 += s.n;
             }
         }
-        if (m->layered) {  // first row of every prefilling sequence among the gathered context rows
-            int row0 = 0;
-            for (auto& s : seqs) {
-                *ids++ = s.n > 1 ? row0 : -1;
-                if (s.n > 1) row0 += s.cache->len + s.n;
+        if (m->layered) {  // first row of every prefilling sequence among the gathered context rows, per mask
+            for (size_t g = 0; g < gather.size(); g++) {
+                const MaskSpec& mask = b2_layered_gathers(m)[g];
+                int row0 = 0;
+                for (auto& s : seqs) {
+                    *ids++ = s.n > 1 ? row0 : -1;
+                    if (s.n > 1) row0 += s.cache->len + s.n - mask.first(s.cache->len);
+                }
+                gather[g].rows = row0;
             }
             for (auto& s : seqs) {
                 *ids++ = s.n >= kMemoryChunkMin ? n_chunks : -1;
@@ -441,11 +446,13 @@ int32_t b2_engine_forward(b2_model* m, std::vector<SeqStep>& seqs, void* logits_
         ls.chunk_tiles = chunk_tiles;
         ls.max_ctx = max_pos;
         ls.n_chunks = n_chunks;
-        ls.chunk_off = ids_dev + T + (listed ? n_logits : 0) + B;
+        const int32_t* staged = ids_dev + T + (listed ? n_logits : 0);
+        for (size_t g = 0; g < gather.size(); g++) gather[g].kv_off = staged + g * B;
+        ls.chunk_off = staged + gather.size() * B;
         ls.dec_ctx_sum = dec_ctx_sum;
         ls.pf_pairs = pf_pairs;
-        ls.pf_ctx = pf_ctx;
-        ls.pf_kv_off = ids_dev + T + (listed ? n_logits : 0);
+        ls.gather = gather.data();
+        ls.seqs = &seqs;
         ls.n_logits = n_logits;
         ls.logit_rows = logit_rows;
         if (pool->state_floats > 0)

@@ -1,5 +1,7 @@
 // Grouped-query attention of the layered models: projections to rotated queries and cache rows, and the plain form of the
 // attention.  Scores may be capped, the softmax may have a sink (exp(0) in its denominator, with no value).
+#include <type_traits>
+
 #include "elt.cuh"
 #include "layer_kernels.h"
 
@@ -9,21 +11,52 @@ constexpr int kMaxHead = 256;
 
 // A warp per (token, head of q, k or v): bias, norm over the head, rotation of the pairs (i, i + dims/2), store.  A lane holds
 // VEC consecutive values of every 32 * VEC; the rotation finds its partner in shared memory
-// (N 1, VEC 4: heads of up to 128, the partner comes by shuffle).
-template <typename T, int VEC, int N>
+// (N 1, VEC 4: heads of up to 128, the partner comes by shuffle).  With a norm over all heads (ALL) a block takes eight heads of
+// one token, and first the sums of squares of all its queries and of all its keys.
+template <typename T, int VEC, int N, bool ALL>
 __global__ void __launch_bounds__(256) gqa_prep_kernel(const GroupedAttnSpec a, const GqaPrepParams p) {
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     pdl_wait();
     constexpr bool SHUFFLE = N == 1 && VEC == 4;
     __shared__ __align__(16) float rows[SHUFFLE ? 1 : 8][SHUFFLE ? 4 : kMaxHead];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, units = a.heads + 2 * a.kv_heads;
-    const int id = blockIdx.x * 8 + warp, t = id / units, u = id - t * units;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, units = a.heads + (p.own_kv ? 2 * a.kv_heads : 0);
+    const int id = blockIdx.x * 8 + warp, t = ALL ? blockIdx.y : id / units, u = ALL ? id : id - t * units;
+    float all_inv[2] = {1.f, 1.f};
+    if constexpr (ALL) {  // (every thread of the block: u0 the block's first unit)
+        __shared__ float red[33];
+        const int u0 = blockIdx.x * 8, nq = a.heads * a.dim, nk = a.kv_heads * a.dim;
+        auto sum = [&](const float* bias, int off, int n) {
+            const T* x = reinterpret_cast<const T*>(p.in) + (size_t)t * p.ld + off;
+            float ss = 0.f;
+            if constexpr (VEC == 4) {
+                for (int i = threadIdx.x * 4; i < n; i += 1024) {
+                    float v[4];
+                    Elt<T>::ld4(x + i, v);
+#pragma unroll
+                    for (int e = 0; e < 4; e++) {
+                        if (bias) v[e] += bias[i + e];
+                        ss += v[e] * v[e];
+                    }
+                }
+            } else {
+                for (int i = threadIdx.x; i < n; i += 256) {
+                    const float v = Elt<T>::ld(x + i) + (bias ? bias[i] : 0.f);
+                    ss += v * v;
+                }
+            }
+            return 1.0f / sqrtf(elt_block_sum(ss, red) / (float)n + p.eps);
+        };
+        if (u0 < a.heads) all_inv[0] = sum(p.q_bias, p.q_off, nq);
+        if (p.own_kv && u0 + 8 > a.heads && u0 < a.heads + a.kv_heads) all_inv[1] = sum(p.k_bias, p.k_off, nk);
+        if (u >= units) return;
+    }
     if (t >= p.T) return;
     const int kind = u < a.heads ? 0 : u < a.heads + a.kv_heads ? 1 : 2, h = kind == 0 ? u : kind == 1 ? u - a.heads : u - a.heads - a.kv_heads;
     const int n = kind == 2 ? a.vdim : a.dim, padded = kind == 2 ? a.v_row() : a.k_row(), dims = kind == 2 ? 0 : a.rot.dims, half = dims / 2;
     const T* src = reinterpret_cast<const T*>(p.in) + (size_t)t * p.ld + (kind == 0 ? p.q_off : kind == 1 ? p.k_off : p.v_off) + h * n;
     const float* bias = kind == 0 ? p.q_bias : kind == 1 ? p.k_bias : p.v_bias;
     const float* w = kind == 0 ? p.q_norm : kind == 1 ? p.k_norm : nullptr;
+    if (ALL && w) w += h * n;
     const int slot = p.slot_mapping[t];
     T* dst;
     if (kind == 0) {
@@ -58,7 +91,7 @@ __global__ void __launch_bounds__(256) gqa_prep_kernel(const GroupedAttnSpec a, 
         for (int e = 0; e < VEC; e++) ss += v[i][e] * v[i][e];
     }
     if (w) {
-        const float inv = 1.0f / sqrtf(elt_warp_sum(ss) / (float)n + p.eps);
+        const float inv = ALL ? all_inv[kind] : 1.0f / sqrtf(elt_warp_sum(ss) / (float)n + p.eps);
 #pragma unroll
         for (int i = 0; i < N; i++)
 #pragma unroll
@@ -117,7 +150,7 @@ __global__ void __launch_bounds__(128) gqa_simple_kernel(const GroupedAttnSpec a
     pdl_wait();
     __shared__ float q[kMaxHead], acc[kMaxHead], pr[128], red[33];
     const int t = blockIdx.x, h = blockIdx.y, g = h / a.group(), KR = a.k_row(), VR = a.v_row(), ps = p.page_size;
-    const int n = p.positions[t] + 1;
+    const int n = p.positions[t] + 1, lo = a.mask.first(p.positions[t]);
     const int32_t* bt = p.block_tables + (size_t)p.seq_slot[p.token_seq[t]] * p.max_blocks;
     const T* qr = reinterpret_cast<const T*>(p.q) + ((size_t)t * a.heads + h) * KR;
     auto row = [&](int j) { return ((size_t)bt[j / ps] * a.kv_heads + g) * ps + j % ps; };
@@ -125,7 +158,7 @@ __global__ void __launch_bounds__(128) gqa_simple_kernel(const GroupedAttnSpec a
     for (int i = threadIdx.x; i < VR; i += 128) acc[i] = 0.f;
     float m = -INFINITY, l = 0.f;
     __syncthreads();
-    for (int j0 = 0; j0 < n; j0 += 128) {
+    for (int j0 = lo; j0 < n; j0 += 128) {
         const int j = j0 + threadIdx.x, cnt = min(128, n - j0);
         float s = -INFINITY;
         if (j < n) {
@@ -167,11 +200,16 @@ int32_t b2_gqa_prep_launch(b2_ctx* ctx, bool f32, const GroupedAttnSpec& a, cons
     if (p.T <= 0) return B2_OK;
     B2_REQUIRE(a.dim <= kMaxHead && a.vdim <= kMaxHead, B2_ERR_UNSUPPORTED, "grouped attention: head sizes up to 256");
     const bool vec = a.dim % 4 == 0 && a.vdim % 4 == 0 && p.q_off % 4 == 0 && p.k_off % 4 == 0 && p.v_off % 4 == 0 && p.ld % 4 == 0;
-    const dim3 grid((unsigned)(((size_t)p.T * (a.heads + 2 * a.kv_heads) + 7) / 8));
+    const int units = a.heads + (p.own_kv ? 2 * a.kv_heads : 0);
     const bool small = a.dim <= 128 && a.vdim <= 128 && a.rot.dims % 8 == 0;
-    auto k = !vec    ? (f32 ? gqa_prep_kernel<float, 1, 8> : gqa_prep_kernel<uint16_t, 1, 8>)
-             : small ? (f32 ? gqa_prep_kernel<float, 4, 1> : gqa_prep_kernel<uint16_t, 4, 1>)
-                     : (f32 ? gqa_prep_kernel<float, 4, 2> : gqa_prep_kernel<uint16_t, 4, 2>);
+    auto pick = [&](auto all) {
+        constexpr bool ALL = decltype(all)::value;
+        return !vec    ? (f32 ? gqa_prep_kernel<float, 1, 8, ALL> : gqa_prep_kernel<uint16_t, 1, 8, ALL>)
+               : small ? (f32 ? gqa_prep_kernel<float, 4, 1, ALL> : gqa_prep_kernel<uint16_t, 4, 1, ALL>)
+                       : (f32 ? gqa_prep_kernel<float, 4, 2, ALL> : gqa_prep_kernel<uint16_t, 4, 2, ALL>);
+    };
+    auto k = a.norm_all ? pick(std::true_type{}) : pick(std::false_type{});
+    const dim3 grid = a.norm_all ? dim3((units + 7) / 8, p.T) : dim3((unsigned)(((size_t)p.T * units + 7) / 8));
     B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, k, grid, dim3(256), 0, ctx->stream, a, p));
     B2_LAUNCHED(ctx);
     return B2_OK;

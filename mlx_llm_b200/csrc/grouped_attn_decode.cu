@@ -5,6 +5,7 @@
 //   CTA   (chunk of one row's keys, up to eight query heads of one key head)
 //   warp  every 4th tile of 16 keys, its own three-stage cp.async ring, no CTA-wide barrier in the loop
 //   mma   S^T = K Q^T with the keys on M and the heads on N, then O^T += V^T P^T; P enters as bf16 head and remainder
+// Under a mask the chunks start at the tile of the row's first visible key, and every row has the same number of work items.
 // Warps are merged in shared memory; the CTA of a (row, head block) that finishes last adds the chunks up, in chunk order.
 #include "elt.cuh"
 #include "layer_kernels.h"
@@ -39,10 +40,16 @@ __global__ void __launch_bounds__(kWarps * 32) gqa_decode_kernel(const GroupedAt
     const int heads = min(kHeads, kvh * group + group - h0), KR = EXACT ? NB * 16 : a.k_row(), VR = EXACT ? NB * 16 : a.v_row();
     int row, chunk = 0, w0 = item, ctx, qrow, slot;  // entry of the list, its chunk, first work item of the row
     if (listed) {
-        if (item >= *p.n_dec_work) return;
-        row = p.work_seq[item];
-        chunk = p.work_chunk[item];
-        w0 = p.work_off[row];
+        if (p.row_chunks > 0) {
+            row = item / p.row_chunks;
+            chunk = item - row * p.row_chunks;
+            w0 = item - chunk;
+        } else {
+            if (item >= *p.n_dec_work) return;
+            row = p.work_seq[item];
+            chunk = p.work_chunk[item];
+            w0 = p.work_off[row];
+        }
         ctx = p.dec_ctx[row];
         qrow = p.dec_qrow[row];
         slot = p.dec_slot[row];
@@ -51,8 +58,10 @@ __global__ void __launch_bounds__(kWarps * 32) gqa_decode_kernel(const GroupedAt
         ctx = p.positions[row] + 1;
         slot = p.seq_slot[p.token_seq[row]];
     }
-    const int tiles_total = (ctx + 15) / 16, chunk_tiles = listed ? p.chunk_tiles : tiles_total, n_chunks = (tiles_total + chunk_tiles - 1) / chunk_tiles;
-    const int tile0 = chunk * chunk_tiles, n_tiles = min(chunk_tiles, tiles_total - tile0);
+    const int lo = a.mask.first(ctx - 1), tile_lo = lo / 16;  // first visible key, its tile
+    const int tiles_total = (ctx + 15) / 16 - tile_lo, chunk_tiles = listed ? p.chunk_tiles : tiles_total, n_chunks = (tiles_total + chunk_tiles - 1) / chunk_tiles;
+    if (chunk >= n_chunks) return;
+    const int tile0 = tile_lo + chunk * chunk_tiles, n_tiles = min(chunk_tiles, tiles_total - chunk * chunk_tiles);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
     const int kd = KR / 16, vd = VR / 16;                              // 16-wide steps
     const int krow = (KR + 63) / 64 * 128, vrow = (VR + 63) / 64 * 128;  // bytes per row in shared memory, whole swizzle groups
@@ -129,6 +138,10 @@ __global__ void __launch_bounds__(kWarps * 32) gqa_decode_kernel(const GroupedAt
         if (key0 + 16 > ctx) {
             if (key0 + g >= ctx) s[0] = s[1] = -INFINITY;
             if (key0 + g + 8 >= ctx) s[2] = s[3] = -INFINITY;
+        }
+        if (key0 < lo) {  // (the tile holds lo: something stays visible)
+            if (key0 + g < lo) s[0] = s[1] = -INFINITY;
+            if (key0 + g + 8 < lo) s[2] = s[3] = -INFINITY;
         }
         float mx0 = fmaxf(s[0], s[2]), mx1 = fmaxf(s[1], s[3]);
 #pragma unroll

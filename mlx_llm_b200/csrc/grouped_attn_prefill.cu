@@ -22,6 +22,8 @@ constexpr int QT = 128, KT = 128;
 constexpr int kSoftmaxWarps = 8, kKWarp = 8, kVWarp = 9, kMmaWarp = 10, kThreads = 352;
 constexpr int BLOCK_BYTES = 128 * 128;  // 128 rows x 64 bf16, 128-byte swizzle
 constexpr float kRescaleThreshold = 8.0f;  // log2 units
+// reference point of a row that sees nothing of the first tile (under a mask): its weights are zero until a tile raises it
+constexpr float kNoKeyYet = -1e30f;
 constexpr float kLog2e = 1.4426950408889634f;
 
 __device__ __forceinline__ float capped(float s, float a, float c) { return c - __fdividef(2.f * c, 1.f + fast_exp2(fminf(s * a, 126.f))); }
@@ -72,7 +74,9 @@ __global__ void __launch_bounds__(kThreads, 1)
     const int tok0 = p.cu_seqlens[b], qn = p.cu_seqlens[b + 1] - tok0;
     const int ctx = p.context_lens[b], ctx_before = ctx - qn;
     const int rows = min(QT, qn - q_start);
-    const int n_tiles = (ctx_before + q_start + rows - 1) / KT + 1;
+    // under a mask the walk starts at the tile of the first query's first visible key; tile numbers count from there
+    const int first_tile = a.mask.first(ctx_before + q_start) / KT, key0 = first_tile * KT;
+    const int n_tiles = (ctx_before + q_start + rows - 1 - key0) / KT + 1;
 
     if (tid == 0) {
         mbar_init(q_full, 1);
@@ -108,7 +112,7 @@ __global__ void __launch_bounds__(kThreads, 1)
         const int blocks = is_k ? DKB : VDB, sub = lane & 7, blk = lane >> 3, ps = p.page_size;
         const int32_t* bt = p.block_tables + (size_t)p.seq_slot[b] * p.max_blocks;
         auto row_of = [&](int j) {
-            const int key = j * KT + sub * 16, kk = key < ctx ? key : 0;
+            const int key = key0 + j * KT + sub * 16, kk = key < ctx ? key : 0;
             return (bt[kk / ps] * a.kv_heads + kvh) * ps + kk % ps;
         };
         if (is_k && lane == 0) {
@@ -196,6 +200,7 @@ __global__ void __launch_bounds__(kThreads, 1)
         const bool row_ok = r < rows;
         // last key this row may see; rows past the chunk see the whole context (their result is dropped)
         const int kvis = row_ok ? min(ctx_before + q_start + r, ctx - 1) : ctx - 1;
+        const int klow = a.mask.first(kvis);  // first key it may see
         const float sc = CAP ? 1.f : score_scale;
         float m_run = -INFINITY, l_run = 0.f;  // l_run: this thread's half of the row sum
         volatile float* xb = reinterpret_cast<volatile float*>(smem_raw + L::X);  // [2 tiles in flight][2 groups][128 rows]
@@ -207,8 +212,8 @@ __global__ void __launch_bounds__(kThreads, 1)
                 break;
             }
             tc_fence_after();
-            const int key_base = j * KT + wg * 64;
-            const bool need_mask = key_base + 63 > kvis;
+            const int key_base = key0 + j * KT + wg * 64;
+            const bool need_mask = key_base + 63 > kvis || key_base < klow;
             // this thread's 64 scores (log2 domain, masked), their maximum, then the maximum of the whole row
             uint32_t v0[32], v1[32];
             tc_ld32_nowait(s_addr, v0);
@@ -217,7 +222,7 @@ __global__ void __launch_bounds__(kThreads, 1)
             // Capped scores are mapped here: c tanh(scale s / c) in units of log2, tanh(z) = 1 - 2 / (1 + e^(2z)), whose
             // absolute error (which is what a score's error counts by) stays at a few units of f32.  Otherwise they stay raw:
             // the scale is positive, so the maximum can be taken first and scaled once, and the exponent below is one
-            // fused multiply-add per score.  Masking (diagonal tiles only) writes -inf.
+            // fused multiply-add per score.  Masking (tiles on an edge only) writes -inf.
             if constexpr (CAP) {
 #pragma unroll
                 for (int i = 0; i < 32; i++) {
@@ -228,8 +233,8 @@ __global__ void __launch_bounds__(kThreads, 1)
             if (need_mask) {
 #pragma unroll
                 for (int i = 0; i < 32; i++) {
-                    if (key_base + i > kvis) v0[i] = 0xff800000u;
-                    if (key_base + 32 + i > kvis) v1[i] = 0xff800000u;
+                    if (key_base + i > kvis || key_base + i < klow) v0[i] = 0xff800000u;
+                    if (key_base + 32 + i > kvis || key_base + 32 + i < klow) v1[i] = 0xff800000u;
                 }
             }
             float mx0 = -INFINITY, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY;
@@ -253,7 +258,7 @@ __global__ void __launch_bounds__(kThreads, 1)
             float alpha = 1.f;
             bool rescale = false;
             if (j == 0) {
-                m_run = mx;  // key 0 is visible to every row
+                m_run = fmaxf(mx, kNoKeyYet);
             } else if (mx > m_run + kRescaleThreshold) {
                 alpha = exp2f(m_run - mx);
                 m_run = mx;

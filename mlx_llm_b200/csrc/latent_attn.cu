@@ -70,7 +70,7 @@ __global__ void __launch_bounds__(128) latent_attn_simple_kernel(const LatentAtt
     __shared__ float red[33];
     const int t = p.row_idx ? p.row_idx[blockIdx.x] : blockIdx.x, h = blockIdx.y, W = a.row_pad(), R = a.kv_rank;
     float *q = sm, *acc = sm + W, *pr = acc + R;
-    const int n = p.positions[t] + 1;
+    const int n = p.positions[t] + 1, lo = a.mask.first(p.positions[t]);
     const int32_t* bt = p.block_tables + (size_t)p.seq_slot[p.token_seq[t]] * p.max_blocks;
     const T* cache = reinterpret_cast<const T*>(p.cache);
     const T* qr = reinterpret_cast<const T*>(p.q_lat) + ((size_t)t * a.heads + h) * W;
@@ -78,7 +78,7 @@ __global__ void __launch_bounds__(128) latent_attn_simple_kernel(const LatentAtt
     for (int i = threadIdx.x; i < R; i += 128) acc[i] = 0.f;
     float m = -INFINITY, l = 0.f;
     __syncthreads();
-    for (int j0 = 0; j0 < n; j0 += 128) {
+    for (int j0 = lo; j0 < n; j0 += 128) {
         const int j = j0 + threadIdx.x, cnt = min(128, n - j0);
         float s = -INFINITY;
         if (j < n) {
@@ -194,7 +194,11 @@ __global__ void __launch_bounds__(kDecodeThreads, 1)
     pdl_wait();  // (the barriers above may be set up while earlier kernels finish)
     const int item = blockIdx.x, h0 = blockIdx.y * NH;
     int sd, chunk, part0;  // row of the list, its chunk, first partial slot of the row
-    if (p.work_seq) {
+    if (p.row_chunks > 0) {
+        sd = item / p.row_chunks;
+        chunk = item - sd * p.row_chunks;
+        part0 = item - chunk;
+    } else if (p.work_seq) {
         if (item >= *p.n_work) return;
         sd = p.work_seq[item];
         chunk = p.work_chunk[item];
@@ -207,9 +211,10 @@ __global__ void __launch_bounds__(kDecodeThreads, 1)
     const int ctx = p.ctx ? p.ctx[sd] : p.positions[sd] + 1, qrow = p.qrow ? p.qrow[sd] : sd;
     const int slot = p.slot ? p.slot[sd] : p.seq_slot[p.token_seq[sd]];
     const int chunk_keys = p.chunk_tiles * 16;
-    const int n_chunks = (ctx + chunk_keys - 1) / chunk_keys;
+    const int k_first = a.mask.first(ctx - 1), k_base = k_first / 16 * 16;  // first visible key, its box: the chunks start there
+    const int n_chunks = (ctx - k_base + chunk_keys - 1) / chunk_keys;
     if (chunk >= n_chunks) return;
-    const int k_lo = chunk * chunk_keys, k_hi = min(ctx, k_lo + chunk_keys);
+    const int k_lo = k_base + chunk * chunk_keys, k_hi = min(ctx, k_lo + chunk_keys);
     const int n_tiles = (k_hi - k_lo + DK_KEYS - 1) / DK_KEYS;
 
     if (warp == 2) {
@@ -325,7 +330,7 @@ __global__ void __launch_bounds__(kDecodeThreads, 1)
                 float m = -INFINITY;
 #pragma unroll
                 for (int i = 0; i < 16; i++) {
-                    const float s = !real ? 0.f : key0 + i < k_hi ? __uint_as_float(v[i]) * p.scale_log2 : -INFINITY;
+                    const float s = !real ? 0.f : key0 + i < k_hi && key0 + i >= k_first ? __uint_as_float(v[i]) * p.scale_log2 : -INFINITY;
                     v[i] = __float_as_uint(s);
                     m = fmaxf(m, s);
                 }
@@ -338,7 +343,7 @@ __global__ void __launch_bounds__(kDecodeThreads, 1)
             for (int w = 1; w < DK_SOFT; w++) m = fmaxf(m, mx[w * 32 + lane]);
             float alpha = 1.f;
             if (j == 0) {
-                m_run = m;  // a chunk's first key is visible
+                m_run = m;  // a chunk's first box has a visible key
             } else if (m > m_run + kDecodeRescale) {
                 alpha = fast_exp2(m_run - m);
                 m_run = m;
@@ -439,9 +444,9 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const LatentAttnSpec 
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     pdl_wait();
     const int sd = blockIdx.x, h = blockIdx.y, R = a.kv_rank, chunk_keys = p.chunk_tiles * 16;
-    const int n = (p.ctx[sd] + chunk_keys - 1) / chunk_keys;
+    const int n = (p.ctx[sd] - a.mask.first(p.ctx[sd] - 1) / 16 * 16 + chunk_keys - 1) / chunk_keys;
     if (n <= 1) return;
-    const size_t at0 = (size_t)p.work_off[sd] * a.heads + h;
+    const size_t at0 = (size_t)(p.row_chunks > 0 ? sd * p.row_chunks : p.work_off[sd]) * a.heads + h;
     __shared__ float w[kMergeTile], sum[kMergeTile];  // maxima, then weights, of up to kMergeTile chunks; row sums
     float M = -INFINITY;
     for (int c = threadIdx.x; c < n; c += 128) M = fmaxf(M, p.part_ml[(at0 + (size_t)c * a.heads) * 2]);

@@ -27,6 +27,8 @@ constexpr int QT = 128, KT = 128;
 constexpr int kSoftmaxWarps = 8, kKWarp = 8, kVWarp = 9, kMmaWarp = 10, kThreads = 352;
 constexpr int BLOCK_BYTES = 128 * 128;  // 128 rows x 64 bf16, 128-byte swizzle
 constexpr float kRescaleThreshold = 8.0f;  // log2 units
+// reference point of a row that sees nothing of the first tile (under a mask): its weights are zero until a tile raises it
+constexpr float kNoKeyYet = -1e30f;
 
 // f32 accumulate, bf16 x bf16, M = 128; bit 16 set = B is MN-major
 constexpr uint32_t idesc(int n, bool b_mn) {
@@ -41,7 +43,7 @@ struct Layout {  // shared memory of a CTA
 
 template <int DKB, int VDB>
 __global__ void __launch_bounds__(kThreads, 1)
-    latent_prefill_tc_kernel(const LatentPrefillParams p, int* err, const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv,
+    latent_prefill_tc_kernel(const LatentPrefillParams p, const MaskSpec mask, int* err, const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv,
                              const __grid_constant__ CUtensorMap map_r) {
     using L = Layout<DKB, VDB>;
     constexpr int NS = L::NS;
@@ -74,7 +76,10 @@ __global__ void __launch_bounds__(kThreads, 1)
     const int tok0 = p.cu_seqlens[b], qn = p.cu_seqlens[b + 1] - tok0;
     const int ctx = p.context_lens[b], ctx_before = ctx - qn, kv0 = p.kv_off[b];
     const int rows = min(QT, qn - q_start);
-    const int n_tiles = (ctx_before + q_start + rows - 1) / KT + 1;
+    // under a mask the walk starts at the tile of the first query's first visible key; tile numbers count from there
+    const int kv_lo = mask.first(ctx_before);  // the gathered rows start with this key
+    const int first_tile = (mask.first(ctx_before + q_start) - kv_lo) / KT, key0 = kv_lo + first_tile * KT;
+    const int n_tiles = (ctx_before + q_start + rows - 1 - key0) / KT + 1;
 
     if (tid == 0) {
         mbar_init(q_full, 1);
@@ -115,7 +120,7 @@ __global__ void __launch_bounds__(kThreads, 1)
                 }
                 mbar_expect_tx(k_full(st), (uint32_t)DKB * BLOCK_BYTES);
                 const uint32_t dst = base + L::K + (uint32_t)st * DKB * BLOCK_BYTES;
-                const int row = kv0 + j * KT;
+                const int row = kv0 + (first_tile + j) * KT;
                 for (int i = 0; i < DKB; i++)
                     if (i < p.plain_blocks)
                         tma_load_2d(dst + i * BLOCK_BYTES, &map_kv, (head * p.plain_blocks + i) * 64, row, k_full(st));
@@ -137,7 +142,7 @@ __global__ void __launch_bounds__(kThreads, 1)
                 }
                 mbar_expect_tx(v_full(st), (uint32_t)VDB * BLOCK_BYTES);
                 for (int i = 0; i < VDB; i++)
-                    tma_load_2d(base + L::V + (uint32_t)(st * VDB + i) * BLOCK_BYTES, &map_kv, p.v_col0 + (head * VDB + i) * 64, kv0 + j * KT, v_full(st));
+                    tma_load_2d(base + L::V + (uint32_t)(st * VDB + i) * BLOCK_BYTES, &map_kv, p.v_col0 + (head * VDB + i) * 64, kv0 + (first_tile + j) * KT, v_full(st));
                 if (++st == NS) st = 0, par ^= 1u;
             }
             if (!alive) atomicExch(err, 2);
@@ -204,6 +209,7 @@ __global__ void __launch_bounds__(kThreads, 1)
         const bool row_ok = r < rows;
         // last key this row may see; rows past the chunk see the whole context (their result is dropped)
         const int kvis = row_ok ? min(ctx_before + q_start + r, ctx - 1) : ctx - 1;
+        const int klow = mask.first(kvis);  // first key it may see
         float m_run = -INFINITY, l_run = 0.f;  // l_run: this thread's half of the row sum
         volatile float* xb = reinterpret_cast<volatile float*>(smem_raw + L::X);  // [2 tiles in flight][2 groups][128 rows]
         for (int j = 0; j < n_tiles && alive; j++) {
@@ -214,20 +220,20 @@ __global__ void __launch_bounds__(kThreads, 1)
                 break;
             }
             tc_fence_after();
-            const int key_base = j * KT + wg * 64;
-            const bool need_mask = key_base + 63 > kvis;
+            const int key_base = key0 + j * KT + wg * 64;
+            const bool need_mask = key_base + 63 > kvis || key_base < klow;
             // this thread's 64 scores (log2 domain, masked), their maximum, then the maximum of the whole row
             uint32_t v0[32], v1[32];
             tc_ld32_nowait(s_addr, v0);
             tc_ld32_nowait(s_addr + 32u, v1);
             asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
             // raw scores: the scale is positive, so the maximum can be taken first and scaled once, and the
-            // exponent below is one fused multiply-add per score.  Masking (diagonal tiles only) writes -inf.
+            // exponent below is one fused multiply-add per score.  Masking (tiles on an edge only) writes -inf.
             if (need_mask) {
 #pragma unroll
                 for (int i = 0; i < 32; i++) {
-                    if (key_base + i > kvis) v0[i] = 0xff800000u;
-                    if (key_base + 32 + i > kvis) v1[i] = 0xff800000u;
+                    if (key_base + i > kvis || key_base + i < klow) v0[i] = 0xff800000u;
+                    if (key_base + 32 + i > kvis || key_base + 32 + i < klow) v1[i] = 0xff800000u;
                 }
             }
             float mx0 = -INFINITY, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY;
@@ -251,7 +257,7 @@ __global__ void __launch_bounds__(kThreads, 1)
             float alpha = 1.f;
             bool rescale = false;
             if (j == 0) {
-                m_run = mx;  // key 0 is visible to every row
+                m_run = fmaxf(mx, kNoKeyYet);
             } else if (mx > m_run + kRescaleThreshold) {
                 alpha = exp2f(m_run - mx);
                 m_run = mx;
@@ -372,7 +378,8 @@ __global__ void __launch_bounds__(kThreads, 1)
 }
 
 // Context rows of the prefilling sequences, gathered from their pages: latents [rows, ld_lat] (zero beyond kv_rank) and
-// rotated key parts [rows, rot_pad] (zero beyond rot_dim).  One warp per row.
+// rotated key parts [rows, rot_pad] (zero beyond rot_dim).  Under a mask a sequence's rows start with the first key that its
+// portion's first token sees.  One warp per row.
 __global__ void __launch_bounds__(256) latent_gather_kernel(const LatentAttnSpec a, const LatentGatherParams p) {
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     pdl_wait();
@@ -383,7 +390,9 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const LatentAttnSpec
         if (p.kv_off[i] >= 0 && p.kv_off[i] <= row) best = i;
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) best = max(best, __shfl_xor_sync(0xffffffffu, best, o));
-    const int key = best >= 0 ? row - p.kv_off[best] : 0, W = a.row_pad(), R = a.kv_rank;
+    int key = 0;
+    if (best >= 0) key = row - p.kv_off[best] + a.mask.first(p.context_lens[best] - (p.cu_seqlens[best + 1] - p.cu_seqlens[best]));
+    const int W = a.row_pad(), R = a.kv_rank;
     const bool ok = best >= 0 && key < p.context_lens[best];
     const uint16_t* src = reinterpret_cast<const uint16_t*>(p.cache);
     if (ok) src += ((size_t)p.block_tables[(size_t)p.seq_slot[best] * p.max_blocks + key / p.page_size] * p.page_size + key % p.page_size) * W;
@@ -399,10 +408,10 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const LatentAttnSpec
 }
 
 template <int DKB, int VDB>
-int32_t launch(b2_ctx* ctx, const LatentPrefillParams& p, int heads, int grid_work, const CUtensorMap& mq, const CUtensorMap& mkv, const CUtensorMap& mr) {
+int32_t launch(b2_ctx* ctx, const LatentAttnSpec& a, const LatentPrefillParams& p, int grid_work, const CUtensorMap& mq, const CUtensorMap& mkv, const CUtensorMap& mr) {
     constexpr int kBytes = Layout<DKB, VDB>::BYTES;
     B2_SMEM_ONCE(ctx, (latent_prefill_tc_kernel<DKB, VDB>), kBytes);
-    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, latent_prefill_tc_kernel<DKB, VDB>, dim3(grid_work, heads), dim3(kThreads), (size_t)kBytes, ctx->stream, p,
+    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, latent_prefill_tc_kernel<DKB, VDB>, dim3(grid_work, a.heads), dim3(kThreads), (size_t)kBytes, ctx->stream, p, a.mask,
                           ctx->dev_err, mq, mkv, mr));
     B2_LAUNCHED(ctx);
     return B2_OK;
@@ -430,10 +439,15 @@ int32_t b2_latent_prefill_launch(b2_ctx* ctx, const LatentAttnSpec& a, const Lat
     CUtensorMap mq, mkv, mr;
     B2_CHECK(get_map(ctx, p.q, (uint64_t)p.q_rows, (uint64_t)a.heads * dk * 64, (uint64_t)a.heads * dk * 64, QT, &mq));
     B2_CHECK(get_map(ctx, p.kv, (uint64_t)p.kv_rows, (uint64_t)p.ld_kv, (uint64_t)p.ld_kv, KT, &mkv));
-    B2_CHECK(get_map(ctx, p.rot, (uint64_t)p.kv_rows, (uint64_t)blocks64(a.rot_dim) * 64, (uint64_t)blocks64(a.rot_dim) * 64, KT, &mr));
-    if (dk == 2 && vd == 1) return launch<2, 1>(ctx, p, a.heads, grid_work, mq, mkv, mr);
-    if (dk == 2 && vd == 2) return launch<2, 2>(ctx, p, a.heads, grid_work, mq, mkv, mr);
-    if (dk == 3 && vd == 1) return launch<3, 1>(ctx, p, a.heads, grid_work, mq, mkv, mr);
-    if (dk == 3 && vd == 2) return launch<3, 2>(ctx, p, a.heads, grid_work, mq, mkv, mr);
+    if (a.rot_dim > 0)
+        B2_CHECK(get_map(ctx, p.rot, (uint64_t)p.kv_rows, (uint64_t)blocks64(a.rot_dim) * 64, (uint64_t)blocks64(a.rot_dim) * 64, KT, &mr));
+    else
+        mr = mkv;  // never read
+    if (dk == 1 && vd == 1) return launch<1, 1>(ctx, a, p, grid_work, mq, mkv, mr);
+    if (dk == 1 && vd == 2) return launch<1, 2>(ctx, a, p, grid_work, mq, mkv, mr);
+    if (dk == 2 && vd == 1) return launch<2, 1>(ctx, a, p, grid_work, mq, mkv, mr);
+    if (dk == 2 && vd == 2) return launch<2, 2>(ctx, a, p, grid_work, mq, mkv, mr);
+    if (dk == 3 && vd == 1) return launch<3, 1>(ctx, a, p, grid_work, mq, mkv, mr);
+    if (dk == 3 && vd == 2) return launch<3, 2>(ctx, a, p, grid_work, mq, mkv, mr);
     return b2_fail(B2_ERR_UNSUPPORTED, "latent prefill: head sizes outside the kernel's tiles");
 }

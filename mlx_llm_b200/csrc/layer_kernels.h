@@ -9,9 +9,9 @@
 struct b2_ctx;
 
 // ---- layer_ops.cu ---------------------------------------------------------------------------------------------
-// x[t, :width] (f32 residual stream) = table[ids[t]]
+// x[t, :width] (f32 residual stream) = table[ids[t]], `copies` rows of x per token
 int32_t b2_embed_residual_launch(b2_ctx* ctx, bool f32, const void* table, int ld_table, const int32_t* ids, int T, int width, int vocab, float* x,
-                                 int ldx);
+                                 int ldx, int copies = 1);
 struct AddNormParams {
     float* x;               // [*, ldx] residual stream
     const float* y;         // what the last sub-layer added (f32), null: nothing
@@ -28,7 +28,28 @@ struct AddNormParams {
     bool write_x;
 };
 int32_t b2_add_norm_launch(b2_ctx* ctx, bool f32, const AddNormParams& p);
-// out[r, j] = act(gu[r, j], gu[r, up_off + j]), the pre-activations scaled by row_w[r] when given; zero for j in [ff, ldo)
+// Several residual streams per token: the pending sub-layer's y goes to every stream beside a mixture of the old ones, then the
+// next sub-layer's norm of a weighted sum of the streams.
+struct StreamNormParams {
+    float* x;               // [*, streams, ldx]
+    int streams;
+    const float *mix, *to;  // pending: x_t <- sum_s mix[s][t] x_s + to[t] y; null: nothing is pending
+    const float* y;         // f32 rows summed into y as in AddNormParams; negative row numbers are left out
+    const int32_t* y_rows;
+    const float* pass;      // [*] y also has pass[t] * h[t], the sub-layer's own input; null: nothing
+    const void* h;          // [*, ldh]
+    const float* from;      // [streams] the sum that is normed; null: all ones
+    const float* w;         // norm weight; null: no norm
+    float* sum;             // [rows, ldx] receives the weighted sum; null: not stored
+    const int32_t* row_idx;
+    void* out;              // [rows, ldo], zero beyond width; may be h
+    int ldx, ldy, ldh, ldo, rows, width, n_src;
+    float eps, out_scale;
+    bool write_x;
+};
+constexpr int kMaxStreams = 16;
+int32_t b2_stream_norm_launch(b2_ctx* ctx, bool f32, const StreamNormParams& p);
+// out[r, j] = act(gu[r, j], gu[r, up_off + j]), scaled by row_w[r] when given (see GateSpec); zero for j in [ff, ldo)
 int32_t b2_gate_launch(b2_ctx* ctx, bool f32, const GateSpec& g, const void* gu, int ldg, int up_off, const float* row_w, int rows, int ff, void* out,
                        int ldo);
 int32_t b2_zero_cols_launch(b2_ctx* ctx, bool f32, void* x, int ldx, int c0, int c1, int rows);
@@ -61,14 +82,20 @@ int32_t b2_grouped_gemm_launch(b2_ctx* ctx, bool f32, const GroupedGemmParams& p
 
 // ---- moe.cu -----------------------------------------------------------------------------------------------------
 struct RouteParams {
-    const float* logits;  // [T, ld]
+    const float* logits;  // [T, ld]: experts | identity experts | the shared expert's number
     int ld, T, experts, top;
+    RouteScore score;
+    int identity;         // (Softmax)
+    bool shared;
+    const float* correction;  // [experts + identity] (Softmax)
+    float scale;
     int32_t* expert;      // [T, top] chosen experts, best first
     float* weight;        // [T, top]
     int32_t* offsets;     // [experts + 1]
-    int32_t* pos;         // [T, top] sorted position of each (token, choice)
-    int32_t* src;         // [T * top] token of each sorted position
+    int32_t* pos;         // [T, top (+ 1)] sorted position of each (token, choice), -1 for an identity expert; then T * top + t (shared)
+    int32_t* src;         // [T * top] token of each sorted position (0 beyond the last one)
     float* row_w;         // [T * top] weight of each sorted position
+    float *pass, *shared_w;  // [T] summed weights of the chosen identity experts; weight of the shared expert
     int32_t* counters;    // [experts + 1], zero between launches
 };
 int32_t b2_route_launch(b2_ctx* ctx, const RouteParams& p);
@@ -114,6 +141,8 @@ struct LatentDecodeParams {
     const int32_t *positions, *token_seq, *seq_slot;
     // work items (row, chunk): the packer's list, or (work_seq null) one per row, whose chunk must hold its whole context
     const int32_t *work_seq, *work_chunk, *work_off, *n_work;
+    // > 0 (rows of the decode list under a mask): item = row * row_chunks + chunk, chunks counted from the first visible key's box
+    int row_chunks;
     int chunk_tiles;   // 16-key boxes per chunk (whole tiles of b2_latent_decode_tile() keys)
     int stages;        // set by the launcher: tiles in shared memory
     int64_t cache_rows;  // rows of the cache allocation
@@ -134,7 +163,8 @@ struct LatentGatherParams {
     int max_blocks, page_size, B, rows;
     const int32_t* seq_slot;      // [B]
     const int32_t* context_lens;  // [B]
-    const int32_t* kv_off;        // [B] first gathered row of each prefilling sequence, -1 for the others
+    const int32_t* kv_off;        // [B] first gathered row of each prefilling sequence, -1 for the others; holds the first key its portion sees
+    const int32_t* cu_seqlens;    // [B + 1]
     void* lat;                    // [rows, ld_lat]
     int ld_lat;
     void* rot;                    // [rows, rot_pad]
@@ -161,7 +191,8 @@ struct GqaPrepParams {
     const void* in;         // [T, ld] projections: queries from q_off, keys from k_off, values from v_off, heads tight
     int ld, q_off, k_off, v_off, T;
     const float *q_bias, *k_bias, *v_bias;  // null: none
-    const float *q_norm, *k_norm;           // null: none
+    const float *q_norm, *k_norm;           // null: none; [dim], or [heads * dim] (norm_all)
+    bool own_kv;            // off: queries only
     float eps;
     const int32_t *positions, *slot_mapping;
     const float *cos_t, *sin_t;  // [positions, rot.dims / 2]
@@ -181,6 +212,7 @@ struct GqaAttnParams {
     const int32_t *positions, *token_seq, *seq_slot;
     // the packer's decode list (context, token row, block-table row) and its work items (row, chunk)
     const int32_t *dec_ctx, *dec_qrow, *dec_slot, *work_seq, *work_chunk, *work_off, *n_dec_work;
+    int row_chunks;              // > 0 (under a mask): item = row * row_chunks + chunk, chunks counted from the first visible key's tile
     int chunk_tiles;             // 16-key tiles per work item
     float *part_o, *part_ml;     // [work item][head][v_row], [work item][head][2]
     int* counters;               // [decode rows][head blocks], zero between launches
@@ -203,7 +235,7 @@ int32_t b2_gqa_prefill_launch(b2_ctx* ctx, const GroupedAttnSpec& a, const GqaAt
 struct MemoryParams {
     const void* in;         // [T, ld] projections
     int ld, c_off, b_off;   // columns of q | k | v and of the step sizes' inputs
-    const void* dec;        // [T, ld_dec] decay inputs (decays() columns); null for fixed decays
+    const void* dec;        // [T, ld_dec] decay inputs (decays() columns; f32 for DecayMap::Exp); null for fixed decays
     int ld_dec;
     int T, B;
     const int32_t *cu_seqlens, *context_lens, *token_seq, *seq_slot, *positions;
@@ -223,7 +255,24 @@ struct MemoryParams {
     int n_chunks;           // 64-token chunks of those portions; 0: every portion goes token by token
     const int32_t* chunk_off;  // [B] a portion's first chunk, -1 for the shorter ones
     void* chunk;            // scratch, n_chunks * b2_memory_chunk_bytes()
+    const float* bonus;     // [heads][dim]
+    const void* h;          // [T, ld_h] the normed stream, whose last row per sequence is kept (shift)
+    int ld_h;
 };
+// Token shift: five mixtures h + (h' - h) mu[i] side by side, out [T, 5 * ldo] (zero beyond the width), h' the row of the token before
+// (the kept one, or zeros, for a portion's first token).
+struct ShiftParams {
+    const void* h;
+    int ld_h, T, width, ldo;
+    const float* mu;        // [5][width]
+    void* out;
+    const int32_t *cu_seqlens, *context_lens, *token_seq, *seq_slot;
+    const float* kept;      // slot s: kept + s * slot_stride
+    int64_t slot_stride;
+};
+int32_t b2_token_shift_launch(b2_ctx* ctx, bool f32, const ShiftParams& p);
+// out[t, j] = tanh(x[t, j]) for j < n, zero up to ldo
+int32_t b2_tanh_launch(b2_ctx* ctx, bool f32, const float* x, int ldx, int T, int n, void* out, int ldo);
 int32_t b2_memory_launch(b2_ctx* ctx, bool f32, const MemorySpec& s, const MemoryParams& p);
 constexpr int kMemoryChunk = 64, kMemoryChunkMin = 12;  // tokens per chunk; shortest portion that the chunked form takes
 bool b2_memory_chunk_eligible(const MemorySpec& s);
@@ -239,7 +288,8 @@ struct BranchOutParams {
     const void* gate;
     int ld_gate;
     MemGate act;
-    const float* norm;      // [vdim]; null: none
+    const float* norm;      // [vdim], or [heads * vdim] (norm_heads); null: none
+    bool norm_heads;
     float eps, scale;
     const void* up;         // feed-forward: [T, ld_up]; null: none
     int ld_up, ff, f_off;

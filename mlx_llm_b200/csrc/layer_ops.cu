@@ -6,12 +6,15 @@ namespace {
 
 template <typename T>
 __global__ void embed_residual_kernel(const T* __restrict__ table, int ld_table, const int32_t* __restrict__ ids, int width, int vocab,
-                                      float* __restrict__ x, int ldx) {
+                                      float* __restrict__ x, int ldx, int copies) {
     pdl_wait();
     const int t = blockIdx.x;
     int id = ids[t];
     id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
-    for (int i = threadIdx.x; i < width; i += blockDim.x) x[(size_t)t * ldx + i] = Elt<T>::ld(table + (size_t)id * ld_table + i);
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+        const float v = Elt<T>::ld(table + (size_t)id * ld_table + i);
+        for (int c = 0; c < copies; c++) x[((size_t)t * copies + c) * ldx + i] = v;
+    }
 }
 
 // x += y (one row, or the sum of several), then RMS norm, one block per row.  The row is kept in shared memory between
@@ -76,11 +79,117 @@ __global__ void add_norm_kernel(const AddNormParams p) {
     }
 }
 
+// The streams' step, one block per token: VEC columns per thread with all streams in registers (NS: their number, rounded up).
+template <typename T, int NS, int VEC>
+__global__ void stream_norm_kernel(const StreamNormParams p) {
+    asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
+    extern __shared__ __align__(16) float row[];
+    __shared__ float red[33], mix[NS][NS], to[NS], from[NS];
+    const int n = p.streams;
+    for (int i = threadIdx.x; i < NS * NS; i += blockDim.x) {  // (weights: nothing earlier writes them)
+        const int a = i / NS, b = i % NS;
+        mix[a][b] = p.mix && a < n && b < n ? p.mix[a * n + b] : 0.f;
+        if (a == 0) {
+            to[b] = p.mix && b < n ? p.to[b] : 0.f;
+            from[b] = b < n ? (p.from ? p.from[b] : 1.f) : 0.f;
+        }
+    }
+    pdl_wait();
+    __syncthreads();
+    const int r = blockIdx.x, t = p.row_idx ? p.row_idx[r] : r;
+    float* xt = p.x + (size_t)t * n * p.ldx;
+    const float pass = p.mix && p.pass ? p.pass[t] : 0.f;
+    const T* h = reinterpret_cast<const T*>(p.h) + (size_t)t * p.ldh;
+    auto load = [](const float* s, float (&v)[VEC]) {
+        if constexpr (VEC == 4)
+            Elt<float>::ld4(s, v);
+        else
+            v[0] = s[0];
+    };
+    auto store = [](float* d, const float (&v)[VEC]) {
+        if constexpr (VEC == 4)
+            Elt<float>::st4(d, v);
+        else
+            d[0] = v[0];
+    };
+    float ss = 0.f;
+    for (int i = threadIdx.x * VEC; i < p.width; i += blockDim.x * VEC) {
+        float x[NS][VEC], u[VEC];
+#pragma unroll
+        for (int a = 0; a < NS; a++)
+            if (a < n) load(xt + (size_t)a * p.ldx + i, x[a]);
+#pragma unroll
+        for (int e = 0; e < VEC; e++) u[e] = 0.f;
+        if (p.mix) {
+            float y[VEC];
+#pragma unroll
+            for (int e = 0; e < VEC; e++) y[e] = 0.f;
+            for (int k = 0; k < p.n_src; k++) {
+                const int yr = p.y_rows ? p.y_rows[(size_t)t * p.n_src + k] : t;
+                if (yr < 0) continue;
+                float v[VEC];
+                load(p.y + (size_t)yr * p.ldy + i, v);
+#pragma unroll
+                for (int e = 0; e < VEC; e++) y[e] += v[e];
+            }
+            if (pass != 0.f) {
+                float v[VEC];
+                if constexpr (VEC == 4)
+                    Elt<T>::ld4(h + i, v);
+                else
+                    v[0] = Elt<T>::ld(h + i);
+#pragma unroll
+                for (int e = 0; e < VEC; e++) y[e] = fmaf(pass, v[e], y[e]);
+            }
+#pragma unroll
+            for (int b = 0; b < NS; b++) {
+                if (b >= n) continue;
+                float v[VEC];
+#pragma unroll
+                for (int e = 0; e < VEC; e++) v[e] = to[b] * y[e];
+#pragma unroll
+                for (int a = 0; a < NS; a++)
+                    if (a < n)
+#pragma unroll
+                        for (int e = 0; e < VEC; e++) v[e] = fmaf(mix[a][b], x[a][e], v[e]);
+                if (p.write_x) store(xt + (size_t)b * p.ldx + i, v);
+#pragma unroll
+                for (int e = 0; e < VEC; e++) u[e] = fmaf(from[b], v[e], u[e]);
+            }
+        } else {
+#pragma unroll
+            for (int a = 0; a < NS; a++)
+                if (a < n)
+#pragma unroll
+                    for (int e = 0; e < VEC; e++) u[e] = fmaf(from[a], x[a][e], u[e]);
+        }
+        if (p.sum) store(p.sum + (size_t)r * p.ldx + i, u);
+        store(row + i, u);
+#pragma unroll
+        for (int e = 0; e < VEC; e++) ss += u[e] * u[e];
+    }
+    if (!p.w) return;
+    ss = elt_block_sum(ss, red);  // (every read of h is behind this barrier: out may be the same row)
+    const float inv = 1.0f / sqrtf(ss / (float)p.width + p.eps);
+    T* o = reinterpret_cast<T*>(p.out) + (size_t)r * p.ldo;
+    if (p.width % 8 == 0) {  // p.ldo is a multiple of 64
+        for (int i = threadIdx.x * 8; i < p.ldo; i += blockDim.x * 8) {
+            float v[8];
+#pragma unroll
+            for (int j = 0; j < 8; j++) v[j] = i < p.width ? row[i + j] * inv * p.w[i + j] * p.out_scale : 0.f;
+            Elt<T>::st8(o + i, v);
+        }
+    } else {
+        for (int i = threadIdx.x; i < p.ldo; i += blockDim.x) Elt<T>::st(o + i, i < p.width ? row[i] * inv * p.w[i] * p.out_scale : 0.f);
+    }
+}
+
 __device__ __forceinline__ float gate_one(const GateSpec& gs, float g, float u) {
     if (gs.act == GateAct::GeluTanh) {
         const float k = 0.7978845608028654f;  // sqrt(2 / pi)
         return 0.5f * g * (1.0f + tanhf(k * (g + 0.044715f * g * g * g))) * u;
     }
+    if (gs.act == GateAct::Swish) return silu_f32(g) * u;
     g = fminf(g, gs.limit);
     u = fminf(fmaxf(u, -gs.limit), gs.limit);
     return g * sigmoid_f32(gs.alpha * g) * (u + 1.0f);
@@ -99,9 +208,16 @@ __global__ void gate_kernel(const GateSpec gs, const T* __restrict__ gu, int ldg
         Elt<T>::ld8(gu + (size_t)r * ldg + i, g);
         Elt<T>::ld8(gu + (size_t)r * ldg + up_off + i, u);
 #pragma unroll
-        for (int j = 0; j < 8; j++) v[j] = i + j < ff ? gate_one(gs, g[j] * s, u[j] * s) : 0.f;
+        for (int j = 0; j < 8; j++) v[j] = i + j >= ff ? 0.f : gs.scale_out ? gate_one(gs, g[j], u[j]) * s : gate_one(gs, g[j] * s, u[j] * s);
     }
     Elt<T>::st8(out + (size_t)r * ldo + i, v);
+}
+
+template <typename T>
+__global__ void tanh_kernel(const float* __restrict__ x, int ldx, int n, T* __restrict__ out, int ldo) {
+    asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
+    pdl_wait();
+    for (int i = threadIdx.x; i < ldo; i += blockDim.x) Elt<T>::st(out + (size_t)blockIdx.x * ldo + i, i < n ? tanhf(x[(size_t)blockIdx.x * ldx + i]) : 0.f);
 }
 
 template <typename T>
@@ -182,13 +298,13 @@ int threads_for(int n, int per, int cap) {
 }  // namespace
 
 int32_t b2_embed_residual_launch(b2_ctx* ctx, bool f32, const void* table, int ld_table, const int32_t* ids, int T, int width, int vocab, float* x,
-                                 int ldx) {
+                                 int ldx, int copies) {
     if (T <= 0) return B2_OK;
     const int th = threads_for(width, 4, 512);
     if (f32)
-        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, embed_residual_kernel<float>, dim3(T), dim3(th), 0, ctx->stream, (const float*)table, ld_table, ids, width, vocab, x, ldx));
+        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, embed_residual_kernel<float>, dim3(T), dim3(th), 0, ctx->stream, (const float*)table, ld_table, ids, width, vocab, x, ldx, copies));
     else
-        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, embed_residual_kernel<uint16_t>, dim3(T), dim3(th), 0, ctx->stream, (const uint16_t*)table, ld_table, ids, width, vocab, x, ldx));
+        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, embed_residual_kernel<uint16_t>, dim3(T), dim3(th), 0, ctx->stream, (const uint16_t*)table, ld_table, ids, width, vocab, x, ldx, copies));
     B2_LAUNCHED(ctx);
     return B2_OK;
 }
@@ -202,6 +318,40 @@ int32_t b2_add_norm_launch(b2_ctx* ctx, bool f32, const AddNormParams& p) {
         B2_SMEM_ONCE(ctx, add_norm_kernel<uint16_t>, 200 * 1024);
     }
     B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, f32 ? add_norm_kernel<float> : add_norm_kernel<uint16_t>, dim3(p.rows), dim3(th), smem, ctx->stream, p));
+    B2_LAUNCHED(ctx);
+    return B2_OK;
+}
+int32_t b2_stream_norm_launch(b2_ctx* ctx, bool f32, const StreamNormParams& p) {
+    if (p.rows <= 0) return B2_OK;
+    B2_REQUIRE(p.streams >= 1 && p.streams <= kMaxStreams, B2_ERR_UNSUPPORTED, "residual streams: 1 to 16");
+    const bool vec = p.width % 4 == 0 && p.ldx % 4 == 0 && p.ldy % 4 == 0 && p.ldh % 4 == 0;
+    const int th = threads_for(p.width, vec ? 4 : 1, 512);
+    const size_t smem = ((size_t)p.width * 4 + 15) / 16 * 16;
+    B2_REQUIRE(smem <= 200 * 1024, B2_ERR_UNSUPPORTED, "stream_norm: the model is too wide");
+    auto run = [&](auto k) -> int32_t {
+        if (smem > 40 * 1024) B2_CUDA(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, k, dim3(p.rows), dim3(th), smem, ctx->stream, p));
+        B2_LAUNCHED(ctx);
+        return B2_OK;
+    };
+    auto pick = [&](auto e) -> int32_t {
+        using T = decltype(e);
+        if (!vec) return run(stream_norm_kernel<T, kMaxStreams, 1>);
+        if (p.streams <= 2) return run(stream_norm_kernel<T, 2, 4>);
+        if (p.streams == 3) return run(stream_norm_kernel<T, 3, 4>);
+        if (p.streams == 4) return run(stream_norm_kernel<T, 4, 4>);
+        if (p.streams <= 8) return run(stream_norm_kernel<T, 8, 4>);
+        return run(stream_norm_kernel<T, kMaxStreams, 4>);
+    };
+    return f32 ? pick(float{}) : pick(uint16_t{});
+}
+int32_t b2_tanh_launch(b2_ctx* ctx, bool f32, const float* x, int ldx, int T, int n, void* out, int ldo) {
+    if (T <= 0) return B2_OK;
+    const int th = threads_for(ldo, 1, 256);
+    if (f32)
+        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, tanh_kernel<float>, dim3(T), dim3(th), 0, ctx->stream, x, ldx, n, (float*)out, ldo));
+    else
+        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, tanh_kernel<uint16_t>, dim3(T), dim3(th), 0, ctx->stream, x, ldx, n, (uint16_t*)out, ldo));
     B2_LAUNCHED(ctx);
     return B2_OK;
 }

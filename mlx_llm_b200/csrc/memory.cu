@@ -1,9 +1,10 @@
-// Linear memories (retention, gated delta rule) between a layer's projections: what enters the recurrence, the recurrence
+// Linear memories (retention, gated delta rule, time mixing with a bonus) between a layer's projections: what enters the recurrence, the recurrence
 // token by token, and the input row of the output projection.
 //
 // Recurrent record of a sequence (f32, one slot per block-table row of the pool):
 //   S     [heads][vdim][dim]
-//   conv  [taps - 1][channels]   the last inputs of the convolution, oldest first
+//   conv  [taps - 1][channels]   the last inputs of the convolution, oldest first; or, with a token shift, [width] the last row of
+//                                the layer's normed input
 // A sequence that starts in this step (nothing cached) starts from zero, whatever its slot held before.
 //
 // Everything that enters the recurrence besides the convolved (or plain) values is prepared and kept in f32.
@@ -56,6 +57,88 @@ __global__ void __launch_bounds__(256) memory_rotate_kernel(const MemorySpec s, 
             Elt<float>::st4(dst, v);
         else
             dst[0] = v[0];
+    }
+}
+
+// Token shift: a block takes `run` tokens and 256 * VEC columns, and carries the row before along.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) token_shift_kernel(const ShiftParams p, int run) {
+    asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
+    pdl_wait();
+    const int i = (blockIdx.x * 256 + threadIdx.x) * VEC, t0 = blockIdx.y * run, t1 = min(t0 + run, p.T);
+    if (i >= p.ldo) return;
+    const bool in = i < p.width;  // (VEC divides the width)
+    const T* h = reinterpret_cast<const T*>(p.h) + i;
+    T* out = reinterpret_cast<T*>(p.out) + i;
+    auto load = [&](const T* s, float (&v)[VEC]) {
+        if constexpr (VEC == 4)
+            Elt<T>::ld4(s, v);
+        else
+            v[0] = Elt<T>::ld(s);
+    };
+    float mu[5][VEC], prev[VEC], cur[VEC];
+#pragma unroll
+    for (int j = 0; j < 5; j++)
+#pragma unroll
+        for (int e = 0; e < VEC; e++) mu[j][e] = in ? p.mu[(size_t)j * p.width + i + e] : 0.f;
+#pragma unroll
+    for (int e = 0; e < VEC; e++) prev[e] = cur[e] = 0.f;
+    for (int t = t0; t < t1; t++) {
+        const int b = p.token_seq[t], start = p.cu_seqlens[b];
+        if (in) {
+            if (t == start) {  // what the sequence's last step left, or nothing
+                const bool kept = p.context_lens[b] > p.cu_seqlens[b + 1] - start;
+                const float* k = p.kept + (size_t)p.seq_slot[b] * p.slot_stride + i;
+#pragma unroll
+                for (int e = 0; e < VEC; e++) prev[e] = kept ? k[e] : 0.f;
+            } else if (t == t0) {
+                load(h + (size_t)(t - 1) * p.ld_h, prev);
+            }
+            load(h + (size_t)t * p.ld_h, cur);
+        }
+#pragma unroll
+        for (int j = 0; j < 5; j++) {
+            float v[VEC];
+#pragma unroll
+            for (int e = 0; e < VEC; e++) v[e] = fmaf(prev[e] - cur[e], mu[j][e], cur[e]);
+            T* o = out + ((size_t)t * 5 + j) * p.ldo;
+            if constexpr (VEC == 4)
+                Elt<T>::st4(o, v);
+            else
+                Elt<T>::st(o, v[0]);
+        }
+#pragma unroll
+        for (int e = 0; e < VEC; e++) prev[e] = cur[e];
+    }
+}
+
+// Time mixing: queries and keys as f32, and the logarithms -exp(z + w0) of the decays.  Below e^-128 an f32 decay is zero: the
+// logarithm stops there, which keeps its sums finite.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) memory_mix_prep_kernel(const MemorySpec s, const MemoryParams p) {
+    asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
+    pdl_wait();
+    const int Q = s.q_cols(), i = (blockIdx.x * 256 + threadIdx.x) * VEC, t = blockIdx.y;
+    if (i >= Q) return;
+    const T* in = reinterpret_cast<const T*>(p.in) + (size_t)t * p.ld + p.c_off + i;
+    const float* z = reinterpret_cast<const float*>(p.dec) + (size_t)t * p.ld_dec + i;
+    const size_t at = (size_t)t * Q + i;
+    auto decay = [](float x) { return fmaxf(-expf(x), -128.f); };
+    if constexpr (VEC == 4) {
+        float v[4], w[4];
+        Elt<T>::ld4(in, v);
+        Elt<float>::st4(p.q + at, v);
+        Elt<T>::ld4(in + Q, v);
+        Elt<float>::st4(p.k + at, v);
+        Elt<float>::ld4(z, v);
+        Elt<float>::ld4(p.dt_bias + i, w);
+#pragma unroll
+        for (int e = 0; e < 4; e++) v[e] = decay(v[e] + w[e]);
+        Elt<float>::st4(p.lg + at, v);
+    } else {
+        p.q[at] = Elt<T>::ld(in);
+        p.k[at] = Elt<T>::ld(in + Q);
+        p.lg[at] = decay(z[0] + p.dt_bias[i]);
     }
 }
 
@@ -242,9 +325,10 @@ __global__ void __launch_bounds__(256) memory_prep_kernel(const MemorySpec s, co
 
 // The recurrence, token after token.  Block = (16 value rows of one head, sequence); thread = (value row, one eighth of the
 // state in float4 pieces).  Tokens pass through shared memory a few at a time.  Both dots of a token -- what the decayed
-// state answers to its key and to its query -- are taken together: S_new^T q = S^T q + u (k . q).
+// state answers to its key and to its query -- are taken together: S_new^T q = S^T q + u (k . q).  With a bonus the read-out
+// comes before the decay, and the keys in k . q are weighted by it.
 constexpr int SC_P = 16;
-template <typename T, int K4>
+template <typename T, int K4, bool BONUS>
 __global__ void __launch_bounds__(128) memory_scan_kernel(const MemorySpec s, const MemoryParams p) {
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     pdl_wait();
@@ -296,7 +380,7 @@ __global__ void __launch_bounds__(128) memory_scan_kernel(const MemorySpec s, co
             const int t = min(pr, SC_T - 1);
             float d = 0.f;
             if (t < cnt)
-                for (int i = ln; i < NP; i += 8) d = fmaf(Ks[t][i], Qs[t][i], d);
+                for (int i = ln; i < NP; i += 8) d = fmaf(BONUS && i < D ? Ks[t][i] * p.bonus[(size_t)h * D + i] : Ks[t][i], Qs[t][i], d);
 #pragma unroll
             for (int o = 4; o > 0; o >>= 1) d += __shfl_xor_sync(0xffffffffu, d, o);
             if (ln == 0) kq[t] = d;
@@ -310,17 +394,24 @@ __global__ void __launch_bounds__(128) memory_scan_kernel(const MemorySpec s, co
                 const int at = k * 32 + ln * 4;
                 kk[k] = *reinterpret_cast<const float4*>(&Ks[t][at]);
                 const float4 q = *reinterpret_cast<const float4*>(&Qs[t][at]), g = *reinterpret_cast<const float4*>(&Gs[t][at]);
-                st[k][0] *= g.x, d1 = fmaf(kk[k].x, st[k][0], d1), d2 = fmaf(q.x, st[k][0], d2);
-                st[k][1] *= g.y, d1 = fmaf(kk[k].y, st[k][1], d1), d2 = fmaf(q.y, st[k][1], d2);
-                st[k][2] *= g.z, d1 = fmaf(kk[k].z, st[k][2], d1), d2 = fmaf(q.z, st[k][2], d2);
-                st[k][3] *= g.w, d1 = fmaf(kk[k].w, st[k][3], d1), d2 = fmaf(q.w, st[k][3], d2);
+                if constexpr (BONUS) {
+                    d2 = fmaf(q.x, st[k][0], d2), st[k][0] *= g.x;
+                    d2 = fmaf(q.y, st[k][1], d2), st[k][1] *= g.y;
+                    d2 = fmaf(q.z, st[k][2], d2), st[k][2] *= g.z;
+                    d2 = fmaf(q.w, st[k][3], d2), st[k][3] *= g.w;
+                } else {
+                    st[k][0] *= g.x, d1 = fmaf(kk[k].x, st[k][0], d1), d2 = fmaf(q.x, st[k][0], d2);
+                    st[k][1] *= g.y, d1 = fmaf(kk[k].y, st[k][1], d1), d2 = fmaf(q.y, st[k][1], d2);
+                    st[k][2] *= g.z, d1 = fmaf(kk[k].z, st[k][2], d1), d2 = fmaf(q.z, st[k][2], d2);
+                    st[k][3] *= g.w, d1 = fmaf(kk[k].w, st[k][3], d1), d2 = fmaf(q.w, st[k][3], d2);
+                }
             }
 #pragma unroll
             for (int o = 4; o > 0; o >>= 1) {
-                d1 += __shfl_xor_sync(0xffffffffu, d1, o);
+                if (!BONUS) d1 += __shfl_xor_sync(0xffffffffu, d1, o);
                 d2 += __shfl_xor_sync(0xffffffffu, d2, o);
             }
-            const float x = xs[t][pr], u = s.delta ? bs[t] * (x - d1) : x;
+            const float x = xs[t][pr], u = !BONUS && s.delta ? bs[t] * (x - d1) : x;
 #pragma unroll
             for (int k = 0; k < K4; k++) {
                 st[k][0] = fmaf(kk[k].x, u, st[k][0]);
@@ -361,6 +452,7 @@ __global__ void __launch_bounds__(256) branch_out_kernel(const BranchOutParams p
         const float* o = p.o + ((size_t)t * p.heads + u) * P;
         const T* z = reinterpret_cast<const T*>(p.gate) + (size_t)t * p.ld_gate + u * P;
         T* dst = out + p.m_off + u * P;
+        const float* norm = p.norm && p.norm_heads ? p.norm + (size_t)u * P : p.norm;
         const bool vec = P % 4 == 0 && p.ld_gate % 4 == 0 && ((uintptr_t)p.gate & (sizeof(T) * 4 - 1)) == 0 && p.m_off % 4 == 0;
         auto gated = [&](float v, float g) { return v * (p.act == MemGate::Silu ? silu_f32(g) : sigmoid_f32(g)); };
         float ss = 0.f;
@@ -379,14 +471,14 @@ __global__ void __launch_bounds__(256) branch_out_kernel(const BranchOutParams p
                 if (d >= P) continue;
                 float g[4], w[4] = {1.f, 1.f, 1.f, 1.f};
                 Elt<T>::ld4(z + d, g);
-                if (p.norm) Elt<float>::ld4(p.norm + d, w);
+                if (norm) Elt<float>::ld4(norm + d, w);
                 const float r[4] = {gated(v[i].x * inv * w[0], g[0]), gated(v[i].y * inv * w[1], g[1]), gated(v[i].z * inv * w[2], g[2]), gated(v[i].w * inv * w[3], g[3])};
                 Elt<T>::st4(dst + d, r);
             }
         } else {
             for (int d = lane; d < P; d += 32) ss += o[d] * o[d];
             const float inv = p.scale / sqrtf(elt_warp_sum(ss) / (float)P + p.eps);
-            for (int d = lane; d < P; d += 32) Elt<T>::st(dst + d, gated(o[d] * inv * (p.norm ? p.norm[d] : 1.f), Elt<T>::ld(z + d)));
+            for (int d = lane; d < P; d += 32) Elt<T>::st(dst + d, gated(o[d] * inv * (norm ? norm[d] : 1.f), Elt<T>::ld(z + d)));
         }
         return;
     }
@@ -431,7 +523,12 @@ int32_t launch_prep(b2_ctx* ctx, const MemorySpec& s, const MemoryParams& p) {
 
 template <typename T>
 int32_t launch_memory(b2_ctx* ctx, const MemorySpec& s, const MemoryParams& p) {
-    if (s.conv > 0) {
+    if (s.shift > 0) {
+        const bool vec = s.q_cols() % 4 == 0 && p.c_off % 4 == 0 && p.ld % 4 == 0 && p.ld_dec % 4 == 0;
+        const dim3 grid((unsigned)((s.q_cols() + (vec ? 1023 : 255)) / (vec ? 1024 : 256)), p.T);
+        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, vec ? memory_mix_prep_kernel<T, 4> : memory_mix_prep_kernel<T, 1>, grid, dim3(256), 0, ctx->stream, s, p));
+        B2_LAUNCHED(ctx);
+    } else if (s.conv > 0) {
         const bool vec = s.dim % 4 == 0 && (s.heads * s.vdim) % 4 == 0 && p.ld_dec % 4 == 0 && p.c_off % 4 == 0 && p.ld % 4 == 0 && p.ld_v % 4 == 0;
         if (!vec)
             B2_CHECK((launch_prep<T, 1, 8>(ctx, s, p)));
@@ -448,7 +545,8 @@ int32_t launch_memory(b2_ctx* ctx, const MemorySpec& s, const MemoryParams& p) {
     if (p.n_chunks > 0) B2_CHECK(b2_memory_chunk_launch(ctx, s, p));
     if (p.n_chunks == 0 || p.B > 1) {
         const int k4 = (s.dim + 31) / 32;
-        auto k = k4 <= 1 ? memory_scan_kernel<T, 1> : k4 <= 2 ? memory_scan_kernel<T, 2> : k4 <= 4 ? memory_scan_kernel<T, 4> : memory_scan_kernel<T, 8>;
+        auto k = s.bonus ? (k4 <= 1 ? memory_scan_kernel<T, 1, true> : k4 <= 2 ? memory_scan_kernel<T, 2, true> : k4 <= 4 ? memory_scan_kernel<T, 4, true> : memory_scan_kernel<T, 8, true>)
+                         : (k4 <= 1 ? memory_scan_kernel<T, 1, false> : k4 <= 2 ? memory_scan_kernel<T, 2, false> : k4 <= 4 ? memory_scan_kernel<T, 4, false> : memory_scan_kernel<T, 8, false>);
         B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, k, dim3((s.vdim + SC_P - 1) / SC_P, s.heads, p.B), dim3(128), 0, ctx->stream, s, p));
         B2_LAUNCHED(ctx);
     }
@@ -461,9 +559,22 @@ int32_t b2_memory_launch(b2_ctx* ctx, bool f32, const MemorySpec& s, const Memor
     if (p.T <= 0) return B2_OK;
     B2_REQUIRE(s.dim <= 256, B2_ERR_UNSUPPORTED, "memory: key sizes up to 256");
     B2_REQUIRE(!(s.conv > 0 && s.rot.dims > 0), B2_ERR_UNSUPPORTED, "memory: a convolution and a rotation together");
-    B2_REQUIRE(s.conv > 0 || (!s.unit && !s.delta && s.decay == MemDecay::Fixed), B2_ERR_UNSUPPORTED,
-               "memory: unit vectors, a delta rule or learned decays without a convolution");
+    B2_REQUIRE(s.conv > 0 || s.shift > 0 || (!s.unit && !s.delta && s.decay == MemDecay::Fixed), B2_ERR_UNSUPPORTED,
+               "memory: unit vectors, a delta rule or learned decays without a convolution or a token shift");
+    B2_REQUIRE(s.shift == 0 || (s.conv == 0 && s.rot.dims == 0 && !s.unit && !s.delta && s.decay == MemDecay::PerChannel && s.decay_map == DecayMap::Exp && s.kv_heads == s.heads),
+               B2_ERR_UNSUPPORTED, "memory: a token shift goes with plain queries and keys and a decay per channel");
+    B2_REQUIRE(!s.bonus || (!s.delta && s.decay == MemDecay::PerChannel), B2_ERR_UNSUPPORTED, "memory: a bonus goes with decays per channel, without the delta rule");
     return f32 ? launch_memory<float>(ctx, s, p) : launch_memory<uint16_t>(ctx, s, p);
+}
+int32_t b2_token_shift_launch(b2_ctx* ctx, bool f32, const ShiftParams& p) {
+    if (p.T <= 0) return B2_OK;
+    const bool vec = p.width % 4 == 0 && p.ld_h % 4 == 0 && p.ldo % 4 == 0;
+    const int bx = (p.ldo + (vec ? 1023 : 255)) / (vec ? 1024 : 256), want = 8 * ctx->sm_count / bx + 1;  // blocks along the tokens
+    const int run = p.T > want ? (p.T + want - 1) / want : 1;
+    auto k = vec ? (f32 ? token_shift_kernel<float, 4> : token_shift_kernel<uint16_t, 4>) : (f32 ? token_shift_kernel<float, 1> : token_shift_kernel<uint16_t, 1>);
+    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, k, dim3(bx, (p.T + run - 1) / run), dim3(256), 0, ctx->stream, p, run));
+    B2_LAUNCHED(ctx);
+    return B2_OK;
 }
 int32_t b2_branch_out_launch(b2_ctx* ctx, bool f32, const BranchOutParams& p) {
     if (p.T <= 0) return B2_OK;

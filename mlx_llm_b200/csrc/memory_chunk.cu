@@ -5,7 +5,8 @@
 //     (I + A) U = beta (V - Kf S0)      A_ts = beta_t k_t . (e^(G_t - G_s) k_s), s < t        Kf_t = e^(G_t) k_t
 //     O = Qf S0 + P U                   P_ts = q_t . (e^(G_t - G_s) k_s), s <= t              Qf_t = e^(G_t) q_t
 //     S = e^(G_end) S0 + Kb^T U         Kb_s = e^(G_end - G_s) k_s
-// (a memory without the delta rule has U = V).  What does not depend on the state -- P, the inverse of I + A times beta, and
+// (a memory without the delta rule has U = V; with a bonus b the read-out of token t comes before its decay and write: e^(G_{t-1})
+// in place of e^(G_t) in Qf and P, and P_tt = q_t . (b k_t)).  What does not depend on the state -- P, the inverse of I + A times beta, and
 // the three scaled operands -- is made for all chunks of all heads at once by memory_factor_kernel; memory_chunk_kernel then
 // walks the chunks of a head in order.
 //
@@ -183,11 +184,14 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
         };
         if constexpr (CHANNEL) {
             float r0[8], tail[8];  // e^(m_i), e^(G_end - m_i)
+            float own[8];          // bonus: the token's own decay, which its read-out does not see
+#pragma unroll
+            for (int e = 0; e < 8; e++) own[e] = s.bonus && t < cnt && x * 8 + e < D ? lg[(size_t)t * s.decays() + x * 8 + e] * kLog2e : 0.f;
 #pragma unroll
             for (int e = 0; e < 8; e++) {
                 const int d = x * 8 + e;
                 const float r = ref[blk * DK + d], m = ref[(4 + blk) * DK + d], g = gs[t * LD + d];
-                left[e] = fast_exp2(g - r);
+                left[e] = fast_exp2(g - own[e] - r);
                 right[e] = kv[e] * fast_exp2(m - g);
                 r0[e] = fast_exp2(r);
                 tail[e] = fast_exp2(ref[8 * DK + d] - m);
@@ -223,6 +227,16 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
 #pragma unroll
             for (int e = 0; e < 8; e++) a[e] = kv[e] * w;
             store(rec + R::Kb, a);
+        }
+    }
+    if (s.bonus) {  // the diagonal of P, in the place of the step sizes
+        for (int t = warp; t < C; t += F_WARPS) {
+            float v = 0.f;
+            if (t < cnt)
+                for (int d = lane; d < D; d += 32) v = fmaf(q[(size_t)t * Q + d] * p.bonus[(size_t)h * D + d], k[(size_t)t * Q + d], v);
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+            if (lane == 0) betas[t] = v;
         }
     }
     __syncthreads();
@@ -289,9 +303,10 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
                     if ((lane & 15) >= o) g += x;
                 }
                 float gt[2], kt[2], qt[2];
+                const float before = s.bonus ? __shfl_up_sync(0xffffffffu, g, 1, 16) : 0.f;  // (the first token's is not used)
 #pragma unroll
                 for (int x = 0; x < 2; x++) {
-                    gt[x] = __shfl_sync(0xffffffffu, g, g4 + 8 * x);
+                    gt[x] = __shfl_sync(0xffffffffu, s.bonus ? before : g, g4 + 8 * x);
                     kt[x] = __shfl_sync(0xffffffffu, kv, g4 + 8 * x);
                     qt[x] = __shfl_sync(0xffffffffu, qv, g4 + 8 * x);
                 }
@@ -303,7 +318,7 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
                         const float gu = __shfl_sync(0xffffffffu, g, u), ku = __shfl_sync(0xffffffffu, kv, u);
 #pragma unroll
                         for (int x = 0; x < 2; x++)
-                            if (u <= g4 + 8 * x) {
+                            if (s.bonus ? u < g4 + 8 * x : u <= g4 + 8 * x) {
                                 const float w = fast_exp2(gt[x] - gu) * ku;
                                 a[half][2 * x + c] = fmaf(w, kt[x], a[half][2 * x + c]);
                                 pr[half][2 * x + c] = fmaf(w, qt[x], pr[half][2 * x + c]);
@@ -324,6 +339,7 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
                 pr[half][e] *= w;
             }
             if (u > t) pr[half][e] = 0.f;
+            if (CHANNEL && s.bonus && u == t) pr[half][e] = betas[t];
             if (s.delta && u < t) M[t * LM + u] = a[half][e] * betas[t];
         }
 #pragma unroll

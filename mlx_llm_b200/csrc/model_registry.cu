@@ -138,6 +138,47 @@ void read_side_by_side(Reader& r, const Value* m, const std::string& at, LayerSp
     L.gqa_scale = (float)r.real(m, "left_scale", at);
     L.mem_scale = (float)r.real(m, "right_scale", at);
 }
+void read_mask(Reader& r, const Value* m, const std::string& at, MaskSpec::Kind kind, MaskSpec& mask) {
+    mask.kind = kind;
+    mask.size = r.num(r.obj(m, "mask", at), "size", at + ".mask");
+}
+// latent attention without a rotated part, over a sliding window
+void read_window_latent(Reader& r, const Value* m, const std::string& at, LayerSpec& L) {
+    LatentAttnSpec& a = L.attn;
+    L.mixer = MixerKind::LatentAttention;
+    a.heads = r.num(m, "heads", at);
+    a.dim = r.num(m, "dim", at);
+    a.vdim = r.num(m, "vdim", at);
+    a.kv_rank = r.num(m, "kv_rank", at);
+    a.scale = (float)r.real(m, "scale", at);
+    read_mask(r, m, at, MaskSpec::Window, a.mask);
+}
+// grouped attention inside chunks, queries and keys normed over all heads at once, on its own keys or another layer's
+void read_chunk_attention(Reader& r, const Value* m, const std::string& at, LayerSpec& L) {
+    GroupedAttnSpec& a = L.gqa;
+    L.mixer = MixerKind::GroupedAttention;
+    a.heads = r.num(m, "heads", at);
+    a.kv_heads = r.num(m, "kv_heads", at);
+    a.dim = r.num(m, "dim", at);
+    a.vdim = r.num(m, "vdim", at);
+    a.scale = (float)r.real(m, "scale", at);
+    a.norm_all = true;
+    read_rot(r, m, at, a.dim, a.rot);
+    read_mask(r, m, at, MaskSpec::Chunk, a.mask);
+    const Value* from = m ? m->get("kv_from") : nullptr;
+    if (from && from->kind != Value::Null) L.kv_from = r.num(m, "kv_from", at, 0);
+    if (r.err.empty()) r.require(a.heads % a.kv_heads == 0, at + ": kv_heads must divide heads");
+}
+// time mixing: token shift, a decay per key channel, a bonus for the current token
+void read_time_mix(Reader& r, const Value* m, const std::string& at, LayerSpec& L) {
+    MemorySpec& s = L.mem;
+    L.mixer = MixerKind::Memory;
+    s.heads = s.kv_heads = r.num(m, "heads", at);
+    s.dim = s.vdim = r.num(m, "dim", at);
+    s.bonus = s.norm = s.norm_heads = true;
+    s.decay = MemDecay::PerChannel;
+    s.decay_map = DecayMap::Exp;
+}
 struct MixerReader {
     const char* name;
     void (*read)(Reader&, const Value*, const std::string&, LayerSpec&);
@@ -245,6 +286,62 @@ int32_t read_tirezen(const Value& v, ModelSpec& spec) {
     return B2_OK;
 }
 
+// ---- Zokuzen: time mixing, windowed latent attention, chunked attention that may read another layer's keys; several residual
+// streams; softmax-routed experts with identity experts and a shared one; norm weights around zero, tied head ---------------
+bool claims_zokuzen(const Value& v) { return names_architecture(v, "Zokuzen"); }
+void read_mixture(Reader& r, const Value* mlp, const std::string& at, LayerSpec& L) {
+    const std::string kind = r.str(mlp, "kind", at);
+    r.require(kind == "moe", at + ": unknown feed-forward kind `" + kind + "`");
+    if (!r.err.empty()) return;
+    L.mlp = MlpKind::Routed;
+    RoutedSpec& m = L.moe;
+    const Value* ro = r.obj(mlp, "router", at);
+    const std::string ra = at + ".router";
+    m.score = RouteScore::Softmax;
+    m.experts = r.num(ro, "experts", ra);
+    m.top = r.num(ro, "top", ra);
+    if (ro && ro->get("identity")) m.identity = r.num(ro, "identity", ra, 0);
+    m.scale = (float)r.real(ro, "scale", ra);
+    m.ff = r.num(r.obj(mlp, "expert", at), "ff", at + ".expert");
+    m.gate.act = GateAct::Swish;
+    m.gate.scale_out = true;
+    const Value* sh = mlp->get("shared");
+    if (sh && sh->kind != Value::Null) m.shared_ff = r.num(sh, "ff", at + ".shared");
+    r.require(m.top <= m.outputs(), at + ": more chosen experts than experts");
+}
+int32_t read_zokuzen(const Value& v, ModelSpec& spec) {
+    Reader r;
+    spec.family = "Zokuzen";
+    spec.vocab = r.num(&v, "vocab", "the model");
+    spec.width = r.num(&v, "width", "the model");
+    spec.streams = r.num(&v, "streams", "the model");
+    spec.eps = (float)r.real(r.obj(&v, "norm", "the model"), "eps", "norm");
+    spec.norm_offset = 1.f;
+    const Value* ls = v.get("layers");
+    r.require(ls && ls->kind == Value::Array && !ls->arr.empty(), "`layers` must be a non-empty list");
+    if (r.err.empty())
+        for (size_t i = 0; i < ls->arr.size(); i++) {
+            const Value* lv = ls->arr[i].get();
+            const std::string at = "layers[" + std::to_string(i) + "]";
+            LayerSpec L;
+            read_mixer(r, {{"wkv", read_time_mix}, {"latent_attention", read_window_latent}, {"attention", read_chunk_attention}}, lv, at, L);
+            if (L.mixer == MixerKind::Memory) L.mem.shift = spec.width;
+            const Value* mlp = lv->get("mlp");
+            if (mlp && mlp->kind != Value::Null) read_mixture(r, mlp, at + ".mlp", L);
+            if (r.err.empty() && L.kv_from >= 0) {
+                const bool ok = L.kv_from < (int)i && spec.layers[L.kv_from].mixer == MixerKind::GroupedAttention && spec.layers[L.kv_from].kv_from < 0;
+                r.require(ok, at + ": kv_from must name an earlier attention layer with keys and values of its own");
+                if (ok) {
+                    const GroupedAttnSpec &a = L.gqa, &b = spec.layers[L.kv_from].gqa;
+                    r.require(a.kv_heads == b.kv_heads && a.dim == b.dim && a.vdim == b.vdim, at + ": kv_from names a layer with other key / value heads");
+                }
+            }
+            spec.layers.push_back(L);
+        }
+    B2_REQUIRE(r.err.empty(), B2_ERR_CONFIG, r.err);
+    return B2_OK;
+}
+
 // ---- the table ------------------------------------------------------------------------------------------------
 struct ModelFamily {
     const char* name;
@@ -252,7 +349,8 @@ struct ModelFamily {
     int32_t (*read_layers)(const Value& root, ModelSpec& spec);  // null: a flat b2_model_config family
 };
 bool claims_flat(const Value&) { return true; }  // b2_model_config_from_json decides (and refuses what it does not know)
-const ModelFamily kFamilies[] = {{"Zukitar", claims_zukitar, read_zukitar}, {"Tirezen", claims_tirezen, read_tirezen}, {"llama", claims_flat, nullptr}};
+const ModelFamily kFamilies[] = {{"Zukitar", claims_zukitar, read_zukitar}, {"Tirezen", claims_tirezen, read_tirezen}, {"Zokuzen", claims_zokuzen, read_zokuzen},
+                                 {"llama", claims_flat, nullptr}};
 
 int32_t find_family(const char* json, b2json::ValuePtr& root, const ModelFamily** out) {
     std::string err;

@@ -11,10 +11,22 @@ enum class MlpKind { None, DenseGated, DensePlain, Routed };
 // act(gate, up) of a gated feed-forward:
 //   GeluTanh      gelu(gate) * up with the tanh form of gelu
 //   ClippedSwish  g = min(gate, limit), u = clamp(up, -limit, limit):  g * sigmoid(alpha * g) * (u + 1)
-enum class GateAct { GeluTanh, ClippedSwish };
+//   Swish         gate * sigmoid(gate) * up
+// A row weight multiplies the pre-activations (the expert's input), or with scale_out the result (its output).
+enum class GateAct { GeluTanh, ClippedSwish, Swish };
 struct GateSpec {
     GateAct act = GateAct::GeluTanh;
     float limit = 0.f, alpha = 0.f;
+    bool scale_out = false;
+};
+
+// Which earlier positions a query may see.  None: all of them; Window: itself and the size - 1 before it; Chunk: those of its own
+// stretch of `size` positions, counted from the sequence's start.  first() never falls as the position rises.
+struct MaskSpec {
+    enum Kind { None, Window, Chunk } kind = None;
+    int size = 0;
+    constexpr int first(int pos) const { return kind == Window ? (pos >= size ? pos - size + 1 : 0) : kind == Chunk ? pos / size * size : 0; }
+    constexpr bool operator==(const MaskSpec& o) const { return kind == o.kind && size == o.size; }
 };
 
 // Rotation of dims/2 pairs by position * base^(-2i/dims); the rest passes unchanged.  Which coordinates form pair i is the
@@ -24,11 +36,12 @@ struct RotSpec {
     int dims = 0;
 };
 // Attention over a shared low-rank latent: per token one vector of kv_rank values and one rotated key part of rot_dim
-// values are cached; every head's keys and values are linear images of the latent.
+// values (0: none) are cached; every head's keys and values are linear images of the latent.
 struct LatentAttnSpec {
     int heads = 0, dim = 0, rot_dim = 0, vdim = 0, kv_rank = 0;
     float scale = 0.f;
     RotSpec rot;
+    MaskSpec mask;
     constexpr int row() const { return kv_rank + rot_dim; }               // values cached per token
     // ... padded for 16-wide tensor-core steps, and to one 64-wide load box at least
     constexpr int row_pad() const { return row() < 64 ? 64 : (row() + 15) / 16 * 16; }
@@ -48,8 +61,10 @@ struct GroupedAttnSpec {
     float softcap = 0.f;  // score <- softcap * tanh(score / softcap); 0: no cap
     bool sink = false;    // exp(0) is added to the softmax's denominator
     bool bias = false;    // biases of the query, key and value projections
-    bool qk_norm = false; // RMS norm over the head of queries and keys, before the rotation
+    bool qk_norm = false; // RMS norm of queries and keys before the rotation, per head ...
+    bool norm_all = false; // ... or over all heads at once
     RotSpec rot;
+    MaskSpec mask;
     constexpr int group() const { return heads / kv_heads; }
     // values per cached head row, zero-padded for 16-wide steps and to one 64-wide load box at least
     constexpr int k_row() const { return dim < 64 ? 64 : (dim + 15) / 16 * 16; }
@@ -57,8 +72,11 @@ struct GroupedAttnSpec {
 };
 // Linear memory: a state S [dim][vdim] per head in f32, read with the query after the token's own write,
 //     S <- decay * S;   S <- S + k u^T;   o = S^T q;   out = norm(o) * gate
-// u = v (delta off) or u = beta (v - S^T k) with the decayed S (delta on).
-enum class MemDecay { Fixed, PerHead, PerChannel };  // Fixed: constants; the others -exp(A_log) softplus(.. + dt_bias) in the exponent
+// u = v (delta off) or u = beta (v - S^T k) with the decayed S (delta on).  With a bonus b the read-out comes first and sees the
+// token's own write only through b:
+//     o = S^T q + (q . (b k)) v;   S <- decay * S + k v^T
+enum class MemDecay { Fixed, PerHead, PerChannel };  // Fixed: constants; the others from a projection z:
+enum class DecayMap { Softplus, Exp };               // exp(-exp(A_log) softplus(z + dt_bias)), or exp(-exp(z + dt_bias))
 enum class MemGate { Silu, Sigmoid };
 struct MemorySpec {
     int heads = 0, kv_heads = 0, dim = 0, vdim = 0;  // kv_heads: heads of q and k
@@ -67,8 +85,14 @@ struct MemorySpec {
     float unit_eps = 1e-6f; // x / sqrt(sum x^2 + unit_eps)
     bool delta = false;
     bool norm = false;     // the output norm has a weight [vdim]
+    bool norm_heads = false; // ... [heads * vdim]
     bool low_rank = false; // decay and gate come from two-factor projections
+    bool bonus = false;
+    // > 0: width of the layer's normed input h.  q, k, v, gate and decay then each read a mixture of their own, h + (h' - h) mu, with
+    // h' the previous token's h (kept in the record); the decay's projection has two factors with a tanh between them.
+    int shift = 0;
     MemDecay decay = MemDecay::Fixed;
+    DecayMap decay_map = DecayMap::Softplus;
     MemGate gate = MemGate::Silu;
     RotSpec rot;           // dims 0: no rotation
     constexpr int q_cols() const { return kv_heads * dim; }
@@ -77,10 +101,20 @@ struct MemorySpec {
     constexpr int keep() const { return conv > 1 ? conv - 1 : 0; }                 // inputs of the convolution kept between steps
     constexpr int decays() const { return decay == MemDecay::PerChannel ? heads * dim : decay == MemDecay::PerHead ? heads : 0; }
 };
-// Routed experts: sigmoid scores, the best `top` experts, the score multiplies the expert's input.
+// Routed experts: the best `top` of them run for a token.
+//   Sigmoid  scores sigmoid(z); a chosen expert's weight is its score
+//   Softmax  scores softmax(z); the choice goes by score + correction, the chosen scores are normalised to a sum of `scale`
+// The last `identity` router outputs are experts that return their input.  shared_ff > 0: one more expert that every token takes,
+// weighted by the sigmoid of a number of its own.
+enum class RouteScore { Sigmoid, Softmax };
 struct RoutedSpec {
     int experts = 0, top = 0, ff = 0;
+    int identity = 0, shared_ff = 0;
+    RouteScore score = RouteScore::Sigmoid;
+    float scale = 1.f;
     GateSpec gate;
+    constexpr int outputs() const { return experts + identity; }
+    constexpr int sources() const { return top + (shared_ff > 0 ? 1 : 0); }  // rows that are summed per token
 };
 struct LayerSpec {
     MixerKind mixer = MixerKind::LatentAttention;
@@ -89,6 +123,7 @@ struct LayerSpec {
     GroupedAttnSpec gqa;              // GroupedAttention, SideBySide
     MemorySpec mem;                   // Memory, SideBySide
     std::vector<double> decay;        // MemDecay::Fixed: per head
+    int kv_from = -1;                 // grouped attention: the layer whose cached keys and values this one reads; -1: its own
     float gqa_scale = 1.f, mem_scale = 1.f;
     std::string gqa_key, mem_key;     // what their tensors' names have behind the mixer's prefix
     // one norm: mixer and feed-forward both read it, and their sum is added to the stream (plain feed-forwards only)
@@ -121,6 +156,9 @@ struct ModelSpec {
     float eps = 1e-5f, logit_scale = 1.f;
     float norm_offset = 0.f;  // added to the stored weights of the layers' norms and the final norm
     bool own_head = false;    // an output projection beside the embedding table
+    // > 0: this many residual streams.  A sub-layer reads sum_s in[s] x_s; afterwards x_t = sum_s mix[s][t] x_s + out[t] y; the model
+    // ends with their sum.  0: one stream, x + y.
+    int streams = 0;
     std::vector<LayerSpec> layers;
     LoopSpec loop;
     TensorNames names;

@@ -1,6 +1,7 @@
 """Plain numpy restatement (float64) of decoders whose layers are listed one by one in config.json: latent attention,
-Mamba-2, softmax attention with a cap and a sink, retention, the gated delta rule, two mixers side by side, dense (gated and
-plain) and routed feed-forwards, repeated layers.  One function per mechanism, whole sequences only, no cache, no batching:
+Mamba-2, softmax attention with a cap and a sink, retention, the gated delta rule, two mixers side by side, time mixing with a
+bonus for the current token, windowed latent and chunked grouped attention (also on another layer's keys), dense (gated and
+plain) and routed feed-forwards, shared and identity experts, repeated layers, several residual streams.  One function per mechanism, whole sequences only, no cache, no batching:
 the yardstick of the layered models' tests.  Nothing here is shared with the library's own code path.
 
 Weights are a dict name -> float array; `cfg` is the parsed config.json.
@@ -221,6 +222,141 @@ def routed_ff(h, g, mlp):
     return out
 
 
+# ---- Zokuzen ---------------------------------------------------------------------------------------------------------
+def shifted(h):
+    """Row t holds the previous token's h (zeros for the first token)."""
+    return np.concatenate([np.zeros((1, h.shape[1]), F), h[:-1]])
+
+
+def bonus_memory(r, k, v, w, u):
+    """One head, one token after the other: r, k, w [T, D], v [T, D], u [D].  The read-out sees the state before the token's own
+    write, plus that write weighted by u; the decay w comes after the read-out."""
+    S = np.zeros((k.shape[1], v.shape[1]), F)
+    out = np.zeros((k.shape[0], v.shape[1]), F)
+    for t in range(k.shape[0]):
+        kv = np.outer(k[t], v[t])
+        out[t] = (S + u[:, None] * kv).T @ r[t]
+        S = w[t][:, None] * S + kv
+    return out
+
+
+def time_mix(h, g, m, eps):
+    T, H, D = h.shape[0], m["heads"], m["dim"]
+    step = shifted(h) - h
+    mixed = {n: h + step * g("mu." + n) for n in "rkvgw"}
+    r, k, v = ((mixed[n] @ g(n).T).reshape(T, H, D) for n in "rkv")
+    w = np.exp(-np.exp(np.tanh(mixed["w"] @ g("w1").T) @ g("w2").T + g("w0"))).reshape(T, H, D)
+    o = np.stack([bonus_memory(r[:, i], k[:, i], v[:, i], w[:, i], g("u")[i]) for i in range(H)], 1)
+    return (rms(o, eps).reshape(T, H * D) * g("norm") * silu(mixed["g"] @ g("g").T)) @ g("o").T
+
+
+def in_window(T, size):
+    """visible[i, j]: j is i or one of the size - 1 tokens before it."""
+    i, j = np.arange(T)[:, None], np.arange(T)[None]
+    return (j <= i) & (i - j < size)
+
+
+def in_chunk(T, size):
+    """visible[i, j]: j <= i lies in the same stretch of `size` tokens, counted from the sequence's start."""
+    i, j = np.arange(T)[:, None], np.arange(T)[None]
+    return (j <= i) & (i // size == j // size)
+
+
+def softmax_attention(q, k, v, scale, visible):
+    """q [H, T, D], k [G, T, D], v [G, T, V] -> [T, H * V]; query head h reads key head h // (H / G)."""
+    H, T = q.shape[:2]
+    out = np.zeros((T, H, v.shape[2]), F)
+    for i in range(H):
+        g = i // (H // k.shape[0])
+        s = np.where(visible, q[i] @ k[g].T * scale, -np.inf)
+        e = np.exp(s - s.max(-1, keepdims=True))
+        out[:, i] = e / e.sum(-1, keepdims=True) @ v[g]
+    return out.reshape(T, -1)
+
+
+def window_latent(h, g, m, eps):
+    """Latent attention whose keys and values are images of the normed latent alone, over a sliding window."""
+    T = h.shape[0]
+    heads = lambda x, d: x.reshape(T, m["heads"], d).transpose(1, 0, 2)
+    c = rms_norm(h @ g("dkv").T, g("dkv.norm"), eps)
+    return softmax_attention(heads(h @ g("q").T, m["dim"]), heads(c @ g("uk").T, m["dim"]), heads(c @ g("uv").T, m["vdim"]), m["scale"],
+                             in_window(T, m["mask"]["size"])) @ g("o").T
+
+
+def chunk_attention(h, g, m, eps, kv=None):
+    """Grouped-query attention inside chunks; queries and keys are normed over the whole projection, then rotated.  `kv`: keys and
+    values of another layer, used instead of projections of its own.  Returns the output and the keys and values it used."""
+    T = h.shape[0]
+    pos = np.arange(T, dtype=F)
+    heads = lambda x, n, d: x.reshape(T, n, d).transpose(1, 0, 2)
+    turn = lambda x: rotate_halves(x, pos, m["rot"]["base"], m["rot"]["dims"])
+    q = turn(heads(rms_norm(h @ g("q").T, g("q.norm"), eps), m["heads"], m["dim"]))
+    if kv is None:
+        kv = (turn(heads(rms_norm(h @ g("k").T, g("k.norm"), eps), m["kv_heads"], m["dim"])), heads(h @ g("v").T, m["kv_heads"], m["vdim"]))
+    return softmax_attention(q, kv[0], kv[1], m["scale"], in_chunk(T, m["mask"]["size"])) @ g("o").T, kv
+
+
+def swiglu(h, g, p):
+    return (silu(h @ g(p + "gate").T) * (h @ g(p + "up").T)) @ g(p + "down").T
+
+
+def softmax_router(z, correction, top, scale):
+    """z [T, outputs] -> weights [T, outputs], zero where not chosen: the correction moves the choice, not the weight."""
+    s = np.exp(z - z.max(-1, keepdims=True))
+    s /= s.sum(-1, keepdims=True)
+    out = np.zeros_like(s)
+    for t in range(len(z)):
+        best = np.argsort(-(s[t] + correction), kind="stable")[:top]
+        out[t, best] = s[t, best] / (s[t, best].sum() + 1e-20) * scale
+    return out
+
+
+def mixture(h, g, mlp):
+    """Routed experts of which the last ones return their input, and a shared expert behind a gate."""
+    r = mlp["router"]
+    w = softmax_router(h @ g("router").T, g("correction"), r["top"], r["scale"])
+    out = w[:, r["experts"]:].sum(1, keepdims=True) * h
+    for e in range(r["experts"]):
+        rows = np.nonzero(w[:, e])[0]
+        if len(rows):
+            out[rows] += w[rows, e:e + 1] * swiglu(h[rows], g, f"e{e}.")
+    if mlp.get("shared"):
+        out = out + sigmoid(h @ g("shared.sg").T) * swiglu(h, g, "shared.")
+    return out
+
+
+def connect(X, w, key, sublayer):
+    """X [T, streams, width] -> the streams after one sub-layer: it reads a weighted sum, and its output goes to every stream
+    beside a mixture ([from, to]) of the old ones."""
+    y = sublayer(np.einsum("s,tsw->tw", w[key + "in"], X))
+    return np.einsum("ab,taw->tbw", w[key + "mix"], X) + w[key + "out"][None, :, None] * y[:, None, :]
+
+
+def forward_zokuzen(cfg, w, tokens, layers_out=None):
+    eps = cfg["norm"]["eps"]
+    X = np.repeat(w["embed"][np.asarray(tokens)].astype(F)[:, None, :], cfg["streams"], 1)
+    stored = {}
+    for i, L in enumerate(cfg["layers"]):
+        mix = lambda n, i=i: w[f"l{i}.mix.{n}"]
+        ff = lambda n, i=i: w[f"l{i}.mlp.{n}"]
+
+        def mixer(u):
+            h = rms_norm(u, 1.0 + w[f"l{i}.norm1"], eps)
+            if L["type"] == "wkv":
+                return time_mix(h, mix, L["mixer"], eps)
+            if L["type"] == "latent_attention":
+                return window_latent(h, mix, L["mixer"], eps)
+            y, stored[i] = chunk_attention(h, mix, L["mixer"], eps, stored.get(L["mixer"].get("kv_from")))
+            return y
+
+        X = connect(X, w, f"l{i}.hc1.", mixer)
+        if L.get("mlp"):
+            X = connect(X, w, f"l{i}.hc2.", lambda u: mixture(rms_norm(u, 1.0 + w[f"l{i}.norm2"], eps), ff, L["mlp"]))
+        if layers_out is not None:
+            layers_out.append(X.sum(1))
+    return rms_norm(X.sum(1), 1.0 + w["final.norm"], eps) @ w["embed"].T
+
+
 def layer_runs(cfg):
     """(layer, pass) in the order they run; pass is -1 outside the repeated stretch."""
     n, loop = len(cfg["layers"]), cfg.get("loop") or dict(start=0, stop=0, times=0)
@@ -230,7 +366,8 @@ def layer_runs(cfg):
 
 def forward(cfg, w, tokens, layers_out=None):
     """Logits [T, vocab] of one sequence.  layers_out (a list) receives the residual stream after every layer run."""
-    return (forward_tirezen if cfg["architecture"] == "Tirezen" else forward_zukitar)(cfg, w, tokens, layers_out)
+    by_name = {"Zukitar": forward_zukitar, "Tirezen": forward_tirezen, "Zokuzen": forward_zokuzen}
+    return by_name[cfg["architecture"]](cfg, w, tokens, layers_out)
 
 
 def forward_tirezen(cfg, w, tokens, layers_out=None):
