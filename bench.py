@@ -781,7 +781,8 @@ def run_layered(args, rank, world, local_rank, barrier, reduce_max, reduce_sum):
         for arm in ("layered", "flat"):
             if args.layered_arm not in ("both", arm):
                 continue
-            design = wl.tirezen_config(size, 2 * pairs) if args.layered_design == "tirezen" else wl.layered_config(size, pairs)
+            design = dict(zukitar=lambda: wl.layered_config(size, pairs), tirezen=lambda: wl.tirezen_config(size, 2 * pairs),
+                          zokuzen=lambda: wl.zokuzen_config(size, 2 * pairs))[args.layered_design]()
             model = eng.CausalLm.synthetic_json(ctx, design, 1) if arm == "layered" else \
                 eng.CausalLm.synthetic(ctx, eng.model_config(**wl.flat_twin(size, 2 * pairs)), seed=1)
             rows[arm] = dict(weight_gb=round(model.weight_bytes() / 1e9, 3),
@@ -793,7 +794,8 @@ def run_layered(args, rank, world, local_rank, barrier, reduce_max, reduce_sum):
     first = next(iter(sizes.values()))
     head = next((r for r in first.get("layered", first.get("flat"))["points"] if r["kind"] == "decode"), first.get("layered", first.get("flat"))["points"][-1])
     peaks = measured_peaks()
-    what = dict(zukitar="latent attention, Mamba-2, routed experts", tirezen="capped sink attention beside delta memories, retention, delta memories")
+    what = dict(zukitar="latent attention, Mamba-2, routed experts", tirezen="capped sink attention beside delta memories, retention, delta memories",
+                zokuzen="time mixing, windowed latent and chunked attention, mixtures of experts")
     return dict(metric=f"decode tok/s, layered design ({what[args.layered_design]})", value=reduce_sum(head["tok_per_s"]), unit="tok/s",
                 n_gpus=world, steps=steps, warmup=warm, ms_per_step=reduce_max(head["ms"]), higher_is_better=True, scaling="weak", vs_baseline=None,
                 dtype="bf16", data="synthetic",
@@ -827,7 +829,7 @@ def main():
     ap.add_argument("--profiler-range", dest="profiler_range", action="store_true",
                     help="bracket the timed region with cudaProfilerStart/Stop (for `ncu --profile-from-start off`)")
     ap.add_argument("--qmm-only", dest="qmm_only", default="", help="qmm: comma-separated OUTxINxBITSxTOKENS cases to run (profiling); not a valid bench line")
-    ap.add_argument("--layered-design", dest="layered_design", default="zukitar", choices=["zukitar", "tirezen"])
+    ap.add_argument("--layered-design", dest="layered_design", default="zukitar", choices=["zukitar", "tirezen", "zokuzen"])
     ap.add_argument("--layered-sizes", dest="layered_sizes", default="w4096,w2048", help="layered: comma-separated sizes (workloads.LAYERED_SIZES)")
     ap.add_argument("--layered-arm", dest="layered_arm", default="both", choices=["both", "layered", "flat"])
     ap.add_argument("--layered-only", dest="layered_only", default="", help="layered: indices of the operating points to run (profiling)")

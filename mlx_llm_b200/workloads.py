@@ -92,6 +92,28 @@ def tirezen_config(size, layers, vocab=32000):
                 layers=[dict(type=mixers[i % 4][0], mixer=mixers[i % 4][1], mlp=mlp) for i in range(layers)])
 
 
+# Zokuzen at the same widths: time mixing, windowed latent attention, time mixing, chunked attention, and in every second round the
+# chunked layer reads the keys of the round before; experts whose active part (chosen and shared) has the flat twin's inner size.
+ZOKUZEN_SIZES = {
+    "w4096": dict(wkv=dict(heads=64, dim=64), latent=dict(heads=32, dim=128, vdim=128, kv_rank=512), heads=32, kv_heads=8, expert_ff=1792, shared_ff=7168),
+    "w2048": dict(wkv=dict(heads=32, dim=64), latent=dict(heads=16, dim=128, vdim=128, kv_rank=512), heads=16, kv_heads=4, expert_ff=1024, shared_ff=4096),
+}
+
+
+def zokuzen_config(size, layers, vocab=32000, streams=4):
+    z, width = ZOKUZEN_SIZES[size], LAYERED_SIZES[size]["width"]
+    latent = dict(z["latent"], scale=z["latent"]["dim"] ** -0.5, mask=dict(size=4096))
+    attn = dict(heads=z["heads"], kv_heads=z["kv_heads"], dim=128, vdim=128, rot=dict(base=500000.0, dims=128), scale=128 ** -0.5, mask=dict(size=8192))
+    mlp = dict(kind="moe", expert=dict(ff=z["expert_ff"]), router=dict(experts=32, identity=4, top=4, scale=2.0), shared=dict(ff=z["shared_ff"]))
+    mixers = [("wkv", z["wkv"]), ("latent_attention", latent), ("wkv", z["wkv"]), ("attention", attn)]
+
+    def mixer(i):
+        kind, m = mixers[i % 4]
+        return dict(type=kind, mixer=dict(m, kv_from=i - 4) if kind == "attention" and i // 4 % 2 else m, mlp=mlp)
+
+    return dict(architecture="Zokuzen", width=width, vocab=vocab, norm=dict(eps=1e-5), streams=streams, layers=[mixer(i) for i in range(layers)])
+
+
 def flat_twin(size, layers, vocab=32000):
     """Llama-architecture model of the same width, feed-forward and layer count, dense bf16."""
     s = LAYERED_SIZES[size]

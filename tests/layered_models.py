@@ -109,6 +109,124 @@ def tirezen_weights(cfg, seed=0, gain=None, ranks=(7, 11)):
     return w
 
 
+# ---- Zokuzen: time mixing, windowed latent and chunked attention, shared keys, residual streams, mixtures of experts --------
+def wkv(heads=3, dim=20):
+    return ("wkv", dict(heads=heads, dim=dim))
+
+
+def window(heads=3, dim=24, vdim=40, kv_rank=56, size=21, scale=None):
+    return ("latent_attention", dict(heads=heads, dim=dim, vdim=vdim, kv_rank=kv_rank, mask=dict(size=size), scale=scale or float(dim ** -0.5)))
+
+
+def chunk(heads=4, kv_heads=2, dim=24, vdim=40, dims=16, base=700.0, size=27, scale=None, kv_from=None):
+    m = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, rot=dict(base=base, dims=dims), mask=dict(size=size), scale=scale or float(dim ** -0.5 * 1.5))
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return ("attention", m)
+
+
+def mixture(experts=5, identity=2, top=3, ff=40, shared=56, scale=1.75):
+    return dict(kind="moe", expert=dict(ff=ff), router=dict(experts=experts, identity=identity, top=top, scale=scale), shared=dict(ff=shared) if shared else None)
+
+
+def zokuzen(layers, width=72, vocab=211, eps=2e-5, streams=2):
+    return dict(architecture="Zokuzen", width=width, vocab=vocab, norm=dict(eps=eps), streams=streams, layers=[dict(type=m[0], mixer=m[1], mlp=f) for m, f in layers])
+
+
+def zokuzen_weights(cfg, seed=0, gain=None, rank=9, decide=True):
+    """name -> float64 array of bf16 values; rank: of the decays' two factors.  decide: keep routing away from close calls."""
+    rng = np.random.default_rng(seed)
+    w, W, S = {}, cfg["width"], cfg["streams"]
+
+    def mat(name, rows, cols):
+        g = next((v for k, v in (gain or {}).items() if name.endswith(k)), 1.0)
+        w[name] = round_bf16(rng.standard_normal((rows, cols)) * g / np.sqrt(cols))
+
+    def vec(name, n, mean, sd):
+        w[name] = round_bf16(mean + sd * rng.standard_normal(n))
+
+    w["embed"] = round_bf16(rng.standard_normal((cfg["vocab"], W)))
+    for i, L in enumerate(cfg["layers"]):
+        m, p = L["mixer"], f"l{i}.mix."
+        for q in (1, 2) if L["mlp"] else (1,):
+            vec(f"l{i}.norm{q}", W, 0.0, 0.2)
+            w[f"l{i}.hc{q}.in"] = round_bf16(rng.uniform(0.1, 1.2, S) / S ** 0.5)
+            w[f"l{i}.hc{q}.out"] = round_bf16(rng.uniform(0.4, 1.4, S))
+            w[f"l{i}.hc{q}.mix"] = round_bf16(rng.uniform(-0.1, 0.5, (S, S)) / S + 0.7 * np.eye(S))
+        if L["type"] == "wkv":
+            Q = m["heads"] * m["dim"]
+            for n in "rkvgw":
+                w[f"{p}mu.{n}"] = round_bf16(rng.uniform(0, 1, W))
+            for n in "rkvg":
+                mat(p + n, Q, W)
+            mat(p + "w1", rank, W), mat(p + "w2", Q, rank), mat(p + "o", W, Q)
+            vec(p + "w0", Q, -2.0, 2.0)
+            vec(p + "u", (m["heads"], m["dim"]), 0.5, 0.6)
+            vec(p + "norm", Q, 1.0, 0.2)
+        elif L["type"] == "latent_attention":
+            mat(p + "q", m["heads"] * m["dim"], W), mat(p + "dkv", m["kv_rank"], W)
+            vec(p + "dkv.norm", m["kv_rank"], 1.0, 0.2)
+            mat(p + "uk", m["heads"] * m["dim"], m["kv_rank"]), mat(p + "uv", m["heads"] * m["vdim"], m["kv_rank"])
+            mat(p + "o", W, m["heads"] * m["vdim"])
+        else:
+            mat(p + "q", m["heads"] * m["dim"], W)
+            vec(p + "q.norm", m["heads"] * m["dim"], 1.2, 0.3)
+            if m.get("kv_from") is None:
+                mat(p + "k", m["kv_heads"] * m["dim"], W), mat(p + "v", m["kv_heads"] * m["vdim"], W)
+                vec(p + "k.norm", m["kv_heads"] * m["dim"], 1.2, 0.3)
+            mat(p + "o", W, m["heads"] * m["vdim"])
+        f, p = L["mlp"], f"l{i}.mlp."
+        if not f:
+            continue
+        n = f["router"]["experts"] + f["router"].get("identity", 0)
+        mat(p + "router", n, W)
+        vec(p + "correction", n, 0.0, 0.2)
+        for e in range(f["router"]["experts"]):
+            ff = f["expert"]["ff"]
+            mat(f"{p}e{e}.gate", ff, W), mat(f"{p}e{e}.up", ff, W), mat(f"{p}e{e}.down", W, ff)
+        if f.get("shared"):
+            ff = f["shared"]["ff"]
+            mat(p + "shared.gate", ff, W), mat(p + "shared.up", ff, W), mat(p + "shared.down", W, ff), mat(p + "shared.sg", 1, W)
+    vec("final.norm", W, 0.0, 0.2)
+    if decide:
+        decide_mixtures(cfg, w, rng)
+    return w
+
+
+def decide_mixtures(cfg, w, rng, cols=8, margin=0.3):
+    """As decide_routes: routers read the first few coordinates, which hold a positive multiple of the embedding's in every stream.
+    One router output is always chosen and one never is (corrections beyond what a score can outweigh); among the rest every
+    token has a gap."""
+    routers = [(i, L["mlp"]["router"]) for i, L in enumerate(cfg["layers"]) if L["mlp"]]
+    if not routers:
+        return
+    for k in w:
+        if k.endswith((".mix.o", ".down")):
+            w[k][:cols] = 0
+    cut = {}
+    for i, r in routers:
+        n = r["experts"] + r.get("identity", 0)
+        w[f"l{i}.norm2"][:cols] = 0
+        z = rng.standard_normal((n, cols))
+        w[f"l{i}.mlp.router"] = round_bf16(np.concatenate([z, np.zeros((n, cfg["width"] - cols))], 1))
+        c = np.zeros(n)
+        if n > 3 and 1 < r["top"] < n - 1:
+            c[rng.permutation(n)[:2]] = 3.0, -3.0
+        w[f"l{i}.mlp.correction"] = c
+        cut[i] = (np.nonzero(c == 0)[0], r["top"] - int((c > 0).sum()))
+    for t in range(cfg["vocab"]):
+        for _ in range(100000):
+            v = round_bf16(1.5 * rng.standard_normal(cols))
+            gaps = [1e9]
+            for i, (free, top) in cut.items():
+                z = np.sort((w[f"l{i}.mlp.router"][:, :cols] @ v)[free])[::-1]
+                if 0 < top < len(z):
+                    gaps.append(z[top - 1] - z[top])
+            if min(gaps) > margin:
+                break
+        w["embed"][t, :cols] = v
+
+
 def tokens(cfg, n, seed):
     return np.random.default_rng(seed).integers(0, cfg["vocab"], n).astype(np.int32)
 
@@ -272,4 +390,23 @@ TIREZEN = {
     # beyond those kernels
     "large_heads": tirezen([(sides(heads=2, kv_heads=1, dim=232, vdim=250, dims=100, softcap=6.0), None), (delta(heads=2, kv_heads=1, dim=200, vdim=136, conv=3), dense(30))],
                            width=64, vocab=80),
+}
+
+ZOKUZEN = {
+    "all_kinds": zokuzen([(wkv(), mixture()), (window(), mixture(experts=7, identity=1, top=2, scale=0.9)), (chunk(), None), (wkv(heads=2, dim=28), None),
+                          (chunk(size=40, kv_from=2, scale=0.4), mixture(shared=None)), (chunk(heads=2, kv_heads=1, dim=16, vdim=32, dims=8, size=11), mixture(identity=0, top=5))],
+                         streams=3),
+    # sizes that divide nothing, single heads, all router outputs chosen, one stream
+    "odd": zokuzen([(window(heads=5, dim=7, vdim=9, kv_rank=19, size=13), mixture(experts=3, identity=1, top=4, ff=17, shared=23)), (wkv(heads=1, dim=13), mixture(experts=4, identity=3, top=1, ff=9)),
+                    (chunk(heads=3, kv_heads=1, dim=10, vdim=7, dims=4, size=37), mixture(ff=33, shared=11)), (chunk(heads=6, kv_heads=1, dim=10, vdim=7, dims=4, size=9, kv_from=2), None)],
+                   width=53, vocab=97, streams=1),
+    # the tiles of the tensor-core kernels
+    "tiles": zokuzen([(wkv(heads=2, dim=64), mixture(experts=16, identity=4, top=4, ff=128, shared=256)), (window(heads=18, dim=128, vdim=128, kv_rank=192, size=100), mixture(experts=4, identity=0, top=2, ff=64)),
+                      (chunk(heads=10, kv_heads=1, dim=128, vdim=128, dims=128, size=96), None), (wkv(heads=1, dim=128), mixture(ff=64)), (chunk(heads=5, kv_heads=1, dim=128, vdim=128, dims=64, size=150, kv_from=2), None)],
+                     width=128, vocab=300, streams=4),
+    "uneven": zokuzen([(window(heads=33, dim=64, vdim=64, kv_rank=512, size=130), None), (chunk(heads=4, kv_heads=4, dim=160, vdim=72, dims=96, size=128), mixture(experts=6, top=2)),
+                       (wkv(heads=3, dim=48), None), (window(heads=2, dim=100, vdim=72, kv_rank=40, size=64), None)], width=96, vocab=150, streams=2),
+    # beyond those kernels, many streams
+    "large_heads": zokuzen([(window(heads=2, dim=200, vdim=140, kv_rank=72, size=33), None), (chunk(heads=2, kv_heads=1, dim=232, vdim=250, dims=100, size=50), mixture()), (wkv(heads=2, dim=150), None)],
+                           width=64, vocab=80, streams=6),
 }

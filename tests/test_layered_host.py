@@ -163,3 +163,56 @@ def test_layer_runs():
     cfg = dict(layers=[0] * 4, loop=dict(start=1, stop=3, times=2))
     assert ref.layer_runs(cfg) == [(0, -1), (1, 0), (2, 0), (1, 1), (2, 1), (3, -1)]
     assert ref.layer_runs(dict(layers=[0] * 2)) == [(0, -1), (1, -1)]
+
+
+def test_zokuzen_configurations_that_are_refused(eng):
+    from mlx_llm_b200._lib import B2Error
+
+    assert all(eng.model_family(c) == "Zokuzen" for c in lm.ZOKUZEN.values())
+    base = lm.ZOKUZEN["all_kinds"]
+    mixer = lambda c, i: c["layers"][i]["mixer"]
+    for change, word in ((lambda c: c.pop("streams"), "streams"), (lambda c: c.update(streams=0), "streams"), (lambda c: mixer(c, 1).pop("mask"), "mask"),
+                         (lambda c: mixer(c, 1)["mask"].update(size=0), "size"), (lambda c: mixer(c, 1).pop("kv_rank"), "kv_rank"), (lambda c: mixer(c, 2).update(kv_heads=3), "kv_heads"),
+                         (lambda c: mixer(c, 2)["rot"].update(dims=26), "rot"), (lambda c: mixer(c, 4).update(kv_from=4), "kv_from"), (lambda c: mixer(c, 4).update(kv_from=1), "kv_from"),
+                         (lambda c: mixer(c, 5).update(kv_from=4), "kv_from"), (lambda c: mixer(c, 4).update(vdim=8), "kv_from"), (lambda c: c["layers"][0].update(type="retention"), "retention"),
+                         (lambda c: c["layers"][0]["mlp"]["router"].update(top=8), "experts"), (lambda c: c["layers"][0]["mlp"]["router"].pop("scale"), "scale"),
+                         (lambda c: c["layers"][0]["mlp"].update(kind="dense"), "kind")):
+        cfg = copy.deepcopy(base)
+        change(cfg)
+        with pytest.raises(B2Error) as e:
+            eng.model_family(cfg)
+        assert e.value.code == -4 and word in str(e.value), str(e.value)
+
+
+def test_bonus_memory_equals_its_closed_form():
+    """o_t = sum over s < t of (r_t . (decay over (s, t)) k_s) v_s, plus (r_t . u k_t) v_t."""
+    rng = np.random.default_rng(7)
+    T, D = 9, 4
+    r, k, v, u = rng.standard_normal((T, D)), rng.standard_normal((T, D)), rng.standard_normal((T, D)), rng.standard_normal(D)
+    w = rng.random((T, D))
+    want = np.array([sum((r[t] * w[s + 1:t].prod(0) * k[s]).sum() * v[s] for s in range(t)) + (r[t] * u * k[t]).sum() * v[t] for t in range(T)])
+    assert np.allclose(want, ref.bonus_memory(r, k, v, w, u))
+    assert np.allclose(ref.shifted(np.array([[1.0], [2.0], [3.0]])), [[0.0], [1.0], [2.0]])
+
+
+def test_masks():
+    win, ch = ref.in_window(7, 3), ref.in_chunk(7, 3)
+    assert [list(np.nonzero(r)[0]) for r in win] == [[0], [0, 1], [0, 1, 2], [1, 2, 3], [2, 3, 4], [3, 4, 5], [4, 5, 6]]
+    assert [list(np.nonzero(r)[0]) for r in ch] == [[0], [0, 1], [0, 1, 2], [3], [3, 4], [3, 4, 5], [6]]
+
+
+def test_pieces_of_the_mixture():
+    z, c = np.log(np.array([[1.0, 2.0, 3.0, 4.0]])), np.array([0.0, 5.0, 0.0, 0.0])
+    assert np.allclose(ref.softmax_router(z, 0 * c, 2, 1.0), [[0, 0, 3 / 7, 4 / 7]])
+    assert np.allclose(ref.softmax_router(z, c, 2, 3.0), [[0, 3 * 2 / 6, 0, 3 * 4 / 6]])  # the correction chooses, the score weighs
+    # nothing but identity experts: the input times the scale
+    w = {"router": np.zeros((3, 2)), "correction": np.array([0.0, 1.0, 2.0])}
+    h = np.array([[1.0, -2.0]])
+    assert np.allclose(ref.mixture(h, w.__getitem__, dict(router=dict(experts=1, identity=2, top=2, scale=0.5))), 0.5 * h)
+
+
+def test_connected_streams():
+    X = np.array([[[1.0], [10.0]]])
+    w = {"in": np.array([2.0, 3.0]), "mix": np.array([[1.0, 5.0], [7.0, 0.0]]), "out": np.array([100.0, 1000.0])}
+    out = ref.connect(X, w, "", lambda u: u)  # reads 2 * 1 + 3 * 10
+    assert np.allclose(out, [[[1 + 70 + 3200], [5 + 32000]]])
