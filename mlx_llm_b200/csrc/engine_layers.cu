@@ -41,13 +41,14 @@ struct LayerP {
     // feed-forward
     Proj gu, down, router;  // router: experts | identity experts | the shared expert's number
     GroupW e_gu, e_down;
-    Proj s_gu, s_down;      // the shared expert
+    Proj s_gu, s_down;      // the shared expert; its first matrix lies behind the router's,
+    Proj both;              // which makes one product of the two for few tokens
     float* correction = nullptr;
     // Layers of grouped attention and memories: one product for everything that reads the normed stream, one for everything
     // that is added to it (columns: attention heads | memory heads | feed-forward).
     Proj in, lr, out;  // lr: the second factors of a memory's decay and gate, block-diagonal
-    // token shift: `in` holds four matrices that read a mixture each (r, k, v, gate; part_n rows apart), w1 the decay's first factor
-    // (lr its second one)
+    // token shift: `in` holds four matrices that read a mixture each (r, k, v, gate; part_n rows apart) and, behind them, the decay's
+    // first factor (a fifth mixture; w1 is that part); lr its second one
     Proj w1;
     int part_n = 0, rank = 0;
     float *mu = nullptr, *bonus = nullptr;
@@ -413,7 +414,11 @@ int32_t load_shifted(Filler& f, LayeredModel& lm, int i) {
     const int Q = s.q_cols(), V = s.heads * s.vdim;
     B2_REQUIRE(Q == V, B2_ERR_UNSUPPORTED, "token shift: keys and values of one size");
     P.part_n = pad_n(Q);
-    B2_CHECK(f.proj(P.in, 4 * P.part_n, W));
+    B2_CHECK(f.rows_of(key("w1"), std::max(8, s.dim), &P.rank));
+    B2_CHECK(f.proj(P.in, 4 * P.part_n + P.rank, W));
+    P.w1 = P.in;
+    P.w1.N = pad_n(P.rank);
+    P.w1.w = f.at(P.in.w, (int64_t)4 * P.part_n * P.in.K);
     std::vector<float> mu;
     const char* parts[5] = {"r", "k", "v", "g", "w"};
     for (int j = 0; j < 5; j++) {
@@ -427,8 +432,6 @@ int32_t load_shifted(Filler& f, LayeredModel& lm, int i) {
         B2_CHECK(f.upload(P.mu, mu));
     else
         B2_CHECK(f.vec(P.mu, "", {5, W}, 0.4f, 0.2f));
-    B2_CHECK(f.rows_of(key("w1"), std::max(8, s.dim), &P.rank));
-    B2_CHECK(f.proj(P.w1, P.rank, W));
     B2_CHECK(f.rows(P.w1, 0, key("w1"), P.rank, W));
     B2_CHECK(f.proj(P.lr, Q, P.rank));
     B2_CHECK(f.rows(P.lr, 0, key("w2"), Q, P.rank));
@@ -515,13 +518,19 @@ int32_t load_layer(Filler& f, LayeredModel& lm, int i) {
     } else {
         const RoutedSpec& r = L.moe;
         const int ffp = up(r.ff, 64);
-        B2_CHECK(f.proj(P.router, r.outputs() + (r.shared_ff > 0 ? 1 : 0), W));
+        const int rn = pad_n(r.outputs() + (r.shared_ff > 0 ? 1 : 0));
+        B2_CHECK(f.proj(P.router, rn + (r.shared_ff > 0 ? 2 * up(r.shared_ff, 64) : 0), W));
+        P.router.N = rn;
         B2_CHECK(f.rows(P.router, 0, mlp("router"), r.outputs(), W));
         if (r.score == RouteScore::Softmax) B2_CHECK(f.vec(P.correction, mlp("correction"), {r.outputs()}, 0.f, 0.01f));
         if (r.shared_ff > 0) {
             const int sp = up(r.shared_ff, 64);
             B2_CHECK(f.rows(P.router, r.outputs(), mlp("shared.sg"), 1, W));
-            B2_CHECK(f.proj(P.s_gu, 2 * sp, W));
+            P.s_gu = P.router;
+            P.s_gu.N = pad_n(2 * sp);
+            P.s_gu.w = f.at(P.router.w, (int64_t)P.router.N * P.router.K);
+            P.both = P.router;
+            P.both.N = P.router.N + P.s_gu.N;
             B2_CHECK(f.rows(P.s_gu, 0, mlp("shared.gate"), r.shared_ff, W));
             B2_CHECK(f.rows(P.s_gu, sp, mlp("shared.up"), r.shared_ff, W));
             B2_CHECK(f.proj(P.s_down, W, r.shared_ff));
@@ -559,6 +568,7 @@ struct Carver {
         return p;
     }
 };
+constexpr int kFewTokens = 64;  // up to here the weights' bytes decide: products that read the same rows are merged
 struct Common {
     float *x, *y, *logits;
     void *xn, *last;
@@ -584,6 +594,7 @@ struct DenseBufs {
     int ld_act;
 };
 struct MoeBufs {
+    float *both;  // few tokens: logits | the shared expert's pre-activations
     float *logits, *weight, *row_w, *pass, *shared_w;
     int32_t *expert, *offsets, *pos, *src;
     void *xs, *gu, *act, *s_gu, *s_act;
@@ -636,16 +647,16 @@ BranchBufs carve_branches(Carver c, const LayerSpec& L, const LayerP& P, size_t 
     o.row = c.take(t * P.out.K * es);
     if (L.has_gqa()) o.q = c.take(t * L.gqa.heads * L.gqa.k_row() * es);
     if (L.has_mem()) {
-        o.lr = c.take(t * P.lr.N * (s.shift > 0 ? 4 : es));
+        o.lr = c.take(s.shift > 0 && es == 2 ? 0 : t * P.lr.N * es);
         if (s.shift > 0) {
             o.mix = c.take(t * 5 * pad_k(s.shift) * es);
             o.low_f = c.take<float>(t * P.w1.N * 4);
-            o.low = c.take(t * P.lr.K * es);
+            o.low = c.take(es == 4 ? t * P.lr.K * es : 0);
         }
         o.ld_v = up(s.heads * s.vdim, 8);
         o.v = s.conv > 0 ? c.take(t * o.ld_v * es) : nullptr;
-        o.mq = c.take<float>(t * s.q_cols() * 4);
-        o.mk = c.take<float>(t * s.q_cols() * 4);
+        o.mq = c.take<float>(s.bonus ? 0 : t * s.q_cols() * 4);
+        o.mk = c.take<float>(s.bonus ? 0 : t * s.q_cols() * 4);
         o.lg = c.take<float>(t * s.decays() * 4);
         o.beta = c.take<float>(t * s.heads * 4);
         o.o = c.take<float>(t * s.heads * s.vdim * 4);
@@ -677,6 +688,7 @@ MoeBufs carve_moe(Carver c, const RoutedSpec& r, const LayerP& P, int ldn, size_
     o.xs = c.take(es == 2 ? n * ldn * es : 0);
     o.gu = c.take(n * P.e_gu.N * es);
     o.act = c.take(n * o.ld_act * es);
+    o.both = c.take<float>((size_t)kFewTokens * P.both.N * 4);
     o.s_gu = c.take(t * P.s_gu.N * es);
     o.s_act = c.take(t * P.s_down.K * es);
     *end = std::max(*end, c.off);
@@ -1149,7 +1161,8 @@ int32_t Fwd::attend(const LayerSpec& L, const LayerP& P, const BranchBufs& b, in
     return B2_OK;
 }
 
-// What a memory behind a token shift reads: five mixtures, r | k | v | gate side by side in b.in, the decay's projection in b.lr (f32).
+// What a memory behind a token shift reads: five mixtures, r | k | v | gate side by side in b.in, the first factor's result of the
+// decay in b.low_f, and in f32 the whole projection in b.lr.
 int32_t Fwd::shift(const LayerSpec& L, const LayerP& P, const BranchBufs& b, int run) {
     b2_ctx* ctx = m->ctx;
     const MemorySpec& sp = L.mem;
@@ -1170,6 +1183,29 @@ int32_t Fwd::shift(const LayerSpec& L, const LayerP& P, const BranchBufs& b, int
     h.slot_stride = pool->state_floats;
     b2_prof_mark(ctx, B2_CLS_ELEMENTWISE);
     B2_CHECK(b2_token_shift_launch(ctx, m->f32, h));
+    GroupedGemmParams g{};
+    g.x = b.mix;
+    g.x_gstride = c.ldn;
+    g.ldx = ldm;
+    g.w = P.in.w;
+    g.N = P.part_n;
+    g.K = P.in.K;
+    g.G = 4;
+    g.out = b.in;
+    g.out_gstride = Q;
+    g.ldo = P.in.N;
+    g.n_out = Q;
+    g.M = s.T;
+    g.x_rows = lm.t_cap;
+    const void* mix_w = (const uint8_t*)b.mix + (size_t)4 * c.ldn * es;
+    if (!m->f32 && s.T <= kFewTokens && P.w1.N <= P.part_n) {  // everything in one launch
+        g.stream = true;
+        g.G = 5;
+        g.tail_n = P.w1.N;
+        g.tail_out = b.low_f;
+        b2_prof_mark(ctx, B2_CLS_GEMM);
+        return b2_grouped_gemm_launch(ctx, false, g);
+    }
     if (!m->f32 && s.T > 32 && P.part_n == Q) {  // whole tiles: four plain products
         for (int j = 0; j < 4; j++) {
             Proj part = P.in;
@@ -1178,26 +1214,13 @@ int32_t Fwd::shift(const LayerSpec& L, const LayerP& P, const BranchBufs& b, int
             B2_CHECK(linear(m, part, (const uint8_t*)b.mix + (size_t)j * c.ldn * es, ldm, s.T, lm.t_cap, (uint8_t*)b.in + (size_t)j * Q * es, P.in.N, false));
         }
     } else {
-        GroupedGemmParams g{};
-        g.x = b.mix;
-        g.x_gstride = c.ldn;
-        g.ldx = ldm;
-        g.w = P.in.w;
-        g.N = P.part_n;
-        g.K = P.in.K;
-        g.G = 4;
-        g.out = b.in;
-        g.out_gstride = Q;
-        g.ldo = P.in.N;
-        g.n_out = Q;
-        g.M = s.T;
-        g.x_rows = lm.t_cap;
         b2_prof_mark(ctx, B2_CLS_GEMM);
         B2_CHECK(b2_grouped_gemm_launch(ctx, m->f32, g));
     }
-    B2_CHECK(linear(m, P.w1, (const uint8_t*)b.mix + (size_t)4 * c.ldn * es, ldm, s.T, lm.t_cap, b.low_f, P.w1.N, true));
+    B2_CHECK(linear(m, P.w1, mix_w, ldm, s.T, lm.t_cap, b.low_f, P.w1.N, true));
+    if (!m->f32) return B2_OK;  // (the rest belongs to the recurrence's preparation)
     b2_prof_mark(ctx, B2_CLS_ELEMENTWISE);
-    B2_CHECK(b2_tanh_launch(ctx, m->f32, b.low_f, P.w1.N, s.T, P.rank, b.low, P.lr.K));
+    B2_CHECK(b2_tanh_launch(ctx, b.low_f, P.w1.N, s.T, P.rank, (float*)b.low, P.lr.K));
     return linear(m, P.lr, b.low, P.lr.K, s.T, lm.t_cap, b.lr, P.lr.N, true);
 }
 
@@ -1211,6 +1234,13 @@ int32_t Fwd::remember(const LayerSpec& L, const LayerP& P, const BranchBufs& b, 
     if (sp.shift > 0) {
         p.dec = b.lr;
         p.ld_dec = P.lr.N;
+        if (!m->f32) {
+            p.low = b.low_f;
+            p.ld_low = P.w1.N;
+            p.rank = P.rank;
+            p.low_w = P.lr.w;
+            p.low_k = P.lr.K;
+        }
         p.bonus = P.bonus;
         p.h = c.xn;
         p.ld_h = c.ldn;
@@ -1298,7 +1328,15 @@ int32_t Fwd::dense(const LayerSpec& L, const LayerP& P) {
     const DenseBufs b = carve_dense(scratch, P, es, (size_t)lm.t_cap, &end);
     B2_CHECK(linear(m, P.gu, c.xn, c.ldn, s.T, lm.t_cap, b.gu, P.gu.N, false));
     b2_prof_mark(m->ctx, B2_CLS_ELEMENTWISE);
-    B2_CHECK(b2_gate_launch(m->ctx, m->f32, L.gate, b.gu, P.gu.N, up(L.ff, 64), nullptr, s.T, L.ff, b.act, b.ld_act));
+    GateRows g;
+    g.gu = b.gu;
+    g.ldg = P.gu.N;
+    g.up_off = up(L.ff, 64);
+    g.rows = s.T;
+    g.ff = L.ff;
+    g.out = b.act;
+    g.ldo = b.ld_act;
+    B2_CHECK(b2_gate_launch(m->ctx, m->f32, L.gate, g));
     return linear(m, P.down, b.act, b.ld_act, s.T, lm.t_cap, c.y, c.ldx, true);
 }
 
@@ -1306,10 +1344,14 @@ int32_t Fwd::moe(const LayerSpec& L, const LayerP& P, const int32_t** rows, cons
     b2_ctx* ctx = m->ctx;
     const RoutedSpec& r = L.moe;
     const MoeBufs b = carve_moe(scratch, r, P, c.ldn, es, (size_t)lm.t_cap, &end);
-    B2_CHECK(linear(m, P.router, c.xn, c.ldn, s.T, lm.t_cap, b.logits, P.router.N, true));
+    const bool shared = r.shared_ff > 0, both = shared && s.T <= kFewTokens;
+    if (both)
+        B2_CHECK(linear(m, P.both, c.xn, c.ldn, s.T, lm.t_cap, b.both, P.both.N, true));
+    else
+        B2_CHECK(linear(m, P.router, c.xn, c.ldn, s.T, lm.t_cap, b.logits, P.router.N, true));
     RouteParams rp{};
-    rp.logits = b.logits;
-    rp.ld = P.router.N;
+    rp.logits = both ? b.both : b.logits;
+    rp.ld = both ? P.both.N : P.router.N;
     rp.T = s.T;
     rp.experts = r.experts;
     rp.top = r.top;
@@ -1349,8 +1391,34 @@ int32_t Fwd::moe(const LayerSpec& L, const LayerP& P, const int32_t** rows, cons
     g.M = s.T * r.top;
     b2_prof_mark(ctx, B2_CLS_GEMM);
     B2_CHECK(b2_grouped_gemm_launch(ctx, m->f32, g));
+    GateRows ge, gs;
+    ge.gu = b.gu;
+    ge.ldg = P.e_gu.N;
+    ge.up_off = up(r.ff, 64);
+    ge.row_w = b.row_w;
+    ge.rows = g.M;
+    ge.ff = r.ff;
+    ge.out = b.act;
+    ge.ldo = b.ld_act;
+    if (shared) {
+        if (!both) B2_CHECK(linear(m, P.s_gu, c.xn, c.ldn, s.T, lm.t_cap, b.s_gu, P.s_gu.N, false));
+        gs.gu = both ? (const void*)(b.both + P.router.N) : b.s_gu;
+        gs.gu_f32 = both;
+        gs.ldg = both ? P.both.N : P.s_gu.N;
+        gs.up_off = up(r.shared_ff, 64);
+        gs.row_w = b.shared_w;
+        gs.rows = s.T;
+        gs.ff = r.shared_ff;
+        gs.out = b.s_act;
+        gs.ldo = P.s_down.K;
+    }
     b2_prof_mark(ctx, B2_CLS_ELEMENTWISE);
-    B2_CHECK(b2_gate_launch(ctx, m->f32, r.gate, b.gu, P.e_gu.N, up(r.ff, 64), b.row_w, g.M, r.ff, b.act, b.ld_act));
+    if (both) {
+        B2_CHECK(b2_gate_launch(ctx, m->f32, r.gate, ge, gs));
+    } else {
+        B2_CHECK(b2_gate_launch(ctx, m->f32, r.gate, ge));
+        if (shared) B2_CHECK(b2_gate_launch(ctx, m->f32, r.gate, gs));
+    }
     GroupedGemmParams d{};
     d.x = b.act;
     d.ldx = b.ld_act;
@@ -1367,12 +1435,8 @@ int32_t Fwd::moe(const LayerSpec& L, const LayerP& P, const int32_t** rows, cons
     d.x_rows = lm.t_cap * r.top;
     b2_prof_mark(ctx, B2_CLS_GEMM);
     B2_CHECK(b2_grouped_gemm_launch(ctx, m->f32, d));
-    if (r.shared_ff > 0) {  // its result: the rows of y behind the routed ones
-        B2_CHECK(linear(m, P.s_gu, c.xn, c.ldn, s.T, lm.t_cap, b.s_gu, P.s_gu.N, false));
-        b2_prof_mark(ctx, B2_CLS_ELEMENTWISE);
-        B2_CHECK(b2_gate_launch(ctx, m->f32, r.gate, b.s_gu, P.s_gu.N, up(r.shared_ff, 64), b.shared_w, s.T, r.shared_ff, b.s_act, P.s_down.K));
-        B2_CHECK(linear(m, P.s_down, b.s_act, P.s_down.K, s.T, lm.t_cap, c.y + (size_t)s.T * r.top * c.ldx, c.ldx, true));
-    }
+    // the shared expert's result: the rows of y behind the routed ones
+    if (shared) B2_CHECK(linear(m, P.s_down, b.s_act, P.s_down.K, s.T, lm.t_cap, c.y + (size_t)s.T * r.top * c.ldx, c.ldx, true));
     *rows = b.pos;
     if (r.identity > 0) *pass = b.pass;
     return B2_OK;

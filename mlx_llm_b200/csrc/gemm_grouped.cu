@@ -49,6 +49,9 @@ __global__ void __launch_bounds__(kThreads) grouped_tile_kernel(const GroupedGem
     find_tile<BM>(p, blockIdx.y, g, r0, rows);
     if (rows <= 0) return;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, n0 = blockIdx.x * BN;
+    const bool tail = p.tail_n > 0 && g == p.G - 1;
+    if (tail && n0 >= p.tail_n) return;
+    const int n_out = tail ? p.tail_n : p.n_out;
     const uint16_t* x = reinterpret_cast<const uint16_t*>(p.x) + (size_t)g * p.x_gstride;
     const uint16_t* w = reinterpret_cast<const uint16_t*>(p.w) + (size_t)g * p.N * p.K;
     float acc[MT][2][4];
@@ -108,8 +111,12 @@ __global__ void __launch_bounds__(kThreads) grouped_tile_kernel(const GroupedGem
 #pragma unroll
             for (int e = 0; e < 4; e++) {
                 const int r = mt * 16 + (lane >> 2) + (e >> 1) * 8, n = n0 + warp * 16 + nt * 8 + 2 * (lane & 3) + (e & 1);
-                if (r >= rows || n >= p.n_out) continue;
+                if (r >= rows || n >= n_out) continue;
                 const int orow = p.map_out ? p.row_idx[r0 + r] : r0 + r;
+                if (tail) {
+                    p.tail_out[(size_t)orow * p.tail_n + n] = acc[mt][nt][e];
+                    continue;
+                }
                 const size_t o = (size_t)g * p.out_gstride + (size_t)orow * p.ldo + n;
                 if (F32OUT)
                     reinterpret_cast<float*>(p.out)[o] = acc[mt][nt][e];
@@ -395,6 +402,7 @@ int32_t b2_grouped_gemm_launch(b2_ctx* ctx, bool f32, const GroupedGemmParams& p
     B2_REQUIRE(p.N % 64 == 0 && p.K % 64 == 0 && p.n_out <= p.N, B2_ERR_UNSUPPORTED, "grouped gemm: N and K must be padded to multiples of 64");
     ctx->gemm_flops += 2.0 * p.M * (p.offsets ? 1 : p.G) * (double)p.N * p.K;
     ctx->gemm_weight_bytes += (double)p.N * p.K * 2 * p.G;
+    B2_REQUIRE(p.tail_n == 0 || (!f32 && p.stream && !p.offsets), B2_ERR_UNSUPPORTED, "grouped gemm: a shorter last group");
     if (f32) {
         const int bound = tile_bound(p, 8);
         B2_REQUIRE(bound <= 65535, B2_ERR_UNSUPPORTED, "grouped gemm: too many rows for one step of the f32 path");
@@ -404,7 +412,7 @@ int32_t b2_grouped_gemm_launch(b2_ctx* ctx, bool f32, const GroupedGemmParams& p
     }
     B2_REQUIRE(p.ldx % 8 == 0 && p.x_gstride % 8 == 0 && ((uintptr_t)p.x & 15) == 0, B2_ERR_UNSUPPORTED, "grouped gemm: rows must be 16-byte aligned");
     const int per_group = p.offsets ? p.M / p.G : p.M;
-    if (!p.row_idx && p.x_rows >= TC_M && b2_grouped_gemm_wants_rows(ctx, p.M, p.offsets != nullptr, p.G, p.N)) return launch_tc(ctx, p);
+    if (!p.stream && !p.row_idx && p.x_rows >= TC_M && b2_grouped_gemm_wants_rows(ctx, p.M, p.offsets != nullptr, p.G, p.N)) return launch_tc(ctx, p);
     if (per_group <= 16) return launch_tile<16, 6>(ctx, p);
     return launch_tile<64, 4>(ctx, p);
 }

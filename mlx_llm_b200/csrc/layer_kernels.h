@@ -49,9 +49,17 @@ struct StreamNormParams {
 };
 constexpr int kMaxStreams = 16;
 int32_t b2_stream_norm_launch(b2_ctx* ctx, bool f32, const StreamNormParams& p);
-// out[r, j] = act(gu[r, j], gu[r, up_off + j]), scaled by row_w[r] when given (see GateSpec); zero for j in [ff, ldo)
-int32_t b2_gate_launch(b2_ctx* ctx, bool f32, const GateSpec& g, const void* gu, int ldg, int up_off, const float* row_w, int rows, int ff, void* out,
-                       int ldo);
+// out[r, j] = act(gu[r, j], gu[r, up_off + j]), scaled by row_w[r] when given (see GateSpec); zero for j in [ff, ldo).  Up to two such
+// arrays in one launch (the second one with rows 0: none).
+struct GateRows {
+    const void* gu = nullptr;
+    bool gu_f32 = false;  // f32 pre-activations of a bf16 model
+    int ldg = 0, up_off = 0, rows = 0, ff = 0;
+    const float* row_w = nullptr;
+    void* out = nullptr;
+    int ldo = 0;
+};
+int32_t b2_gate_launch(b2_ctx* ctx, bool f32, const GateSpec& g, const GateRows& a, const GateRows& b = GateRows());
 int32_t b2_zero_cols_launch(b2_ctx* ctx, bool f32, void* x, int ldx, int c0, int c1, int rows);
 // y[M, N] = x[M, K] . W[N, K]^T in f32 (fused multiply-add, partial sums per 32 inputs)
 int32_t b2_linear_f32_launch(b2_ctx* ctx, const float* x, int ldx, const float* w, int M, int N, int K, float* y, int ldy);
@@ -73,6 +81,10 @@ struct GroupedGemmParams {
     const int32_t* offsets;  // [G + 1] device: group g owns rows [offsets[g], offsets[g + 1]); null: every group has rows 0..M-1
     int M;                   // rows per group, or the total number of rows with `offsets`
     int x_rows;              // rows of the x allocation (0: unknown; the TMA kernel needs 128)
+    // small M only: stream the weights in 64-row tiles whatever M is; the last group may have fewer rows (tail_n) and an f32 result
+    bool stream;
+    int tail_n;              // 0: the last group is like the others
+    float* tail_out;         // [M, tail_n]
     bool vec_out;            // set by the launcher: 16-byte stores are aligned
 };
 // True when a product of this size takes the kernel whose operands must be consecutive rows (row_idx null): a caller that
@@ -245,8 +257,13 @@ struct MemoryParams {
     const float *dt_bias, *A_log;
     const float *decay, *log_decay;  // fixed decays [heads]
     const float *cos_t, *sin_t;
+    // DecayMap::Exp instead of dec: the first factor's result [T, ld_low] (f32) and the second factor [.., low_k] (bf16), `rank` wide
+    const float* low;
+    int ld_low, rank;
+    const void* low_w;
+    int low_k;
     // prepared inputs of the recurrence
-    float *q, *k;           // [T, q_cols]
+    float *q, *k;           // [T, q_cols]; with a bonus q and k are read from `in`
     const void* v;          // [T, ld_v]
     int ld_v;
     float *lg, *beta;       // [T, decays()] logarithms of the decays; [T, heads]
@@ -272,7 +289,7 @@ struct ShiftParams {
 };
 int32_t b2_token_shift_launch(b2_ctx* ctx, bool f32, const ShiftParams& p);
 // out[t, j] = tanh(x[t, j]) for j < n, zero up to ldo
-int32_t b2_tanh_launch(b2_ctx* ctx, bool f32, const float* x, int ldx, int T, int n, void* out, int ldo);
+int32_t b2_tanh_launch(b2_ctx* ctx, const float* x, int ldx, int T, int n, float* out, int ldo);
 int32_t b2_memory_launch(b2_ctx* ctx, bool f32, const MemorySpec& s, const MemoryParams& p);
 constexpr int kMemoryChunk = 64, kMemoryChunkMin = 12;  // tokens per chunk; shortest portion that the chunked form takes
 bool b2_memory_chunk_eligible(const MemorySpec& s);

@@ -79,12 +79,14 @@ __global__ void add_norm_kernel(const AddNormParams p) {
     }
 }
 
+constexpr int kStreamSources = 64;  // rows of y whose numbers are kept in shared memory
 // The streams' step, one block per token: VEC columns per thread with all streams in registers (NS: their number, rounded up).
 template <typename T, int NS, int VEC>
-__global__ void stream_norm_kernel(const StreamNormParams p) {
+__global__ void __launch_bounds__(NS <= 4 ? 1024 : 512) stream_norm_kernel(const StreamNormParams p) {
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     extern __shared__ __align__(16) float row[];
     __shared__ float red[33], mix[NS][NS], to[NS], from[NS];
+    __shared__ int src[kStreamSources];
     const int n = p.streams;
     for (int i = threadIdx.x; i < NS * NS; i += blockDim.x) {  // (weights: nothing earlier writes them)
         const int a = i / NS, b = i % NS;
@@ -95,9 +97,11 @@ __global__ void stream_norm_kernel(const StreamNormParams p) {
         }
     }
     pdl_wait();
-    __syncthreads();
     const int r = blockIdx.x, t = p.row_idx ? p.row_idx[r] : r;
     float* xt = p.x + (size_t)t * n * p.ldx;
+    const int n_src = p.mix ? p.n_src : 0;
+    if ((int)threadIdx.x < min(n_src, kStreamSources)) src[threadIdx.x] = p.y_rows ? p.y_rows[(size_t)t * n_src + threadIdx.x] : t;
+    __syncthreads();
     const float pass = p.mix && p.pass ? p.pass[t] : 0.f;
     const T* h = reinterpret_cast<const T*>(p.h) + (size_t)t * p.ldh;
     auto load = [](const float* s, float (&v)[VEC]) {
@@ -124,13 +128,21 @@ __global__ void stream_norm_kernel(const StreamNormParams p) {
             float y[VEC];
 #pragma unroll
             for (int e = 0; e < VEC; e++) y[e] = 0.f;
-            for (int k = 0; k < p.n_src; k++) {
-                const int yr = p.y_rows ? p.y_rows[(size_t)t * p.n_src + k] : t;
-                if (yr < 0) continue;
-                float v[VEC];
-                load(p.y + (size_t)yr * p.ldy + i, v);
+            for (int k0 = 0; k0 < n_src; k0 += 4) {  // four sources on their way at a time
+                float v[4][VEC];
 #pragma unroll
-                for (int e = 0; e < VEC; e++) y[e] += v[e];
+                for (int k = 0; k < 4; k++) {
+                    const int yr = k0 + k >= n_src ? -1 : k0 + k < kStreamSources ? src[k0 + k] : p.y_rows[(size_t)t * n_src + k0 + k];
+                    if (yr >= 0)
+                        load(p.y + (size_t)yr * p.ldy + i, v[k]);
+                    else
+#pragma unroll
+                        for (int e = 0; e < VEC; e++) v[k][e] = 0.f;
+                }
+#pragma unroll
+                for (int k = 0; k < 4; k++)
+#pragma unroll
+                    for (int e = 0; e < VEC; e++) y[e] += v[k][e];
             }
             if (pass != 0.f) {
                 float v[VEC];
@@ -195,29 +207,36 @@ __device__ __forceinline__ float gate_one(const GateSpec& gs, float g, float u) 
     return g * sigmoid_f32(gs.alpha * g) * (u + 1.0f);
 }
 template <typename T>
-__global__ void gate_kernel(const GateSpec gs, const T* __restrict__ gu, int ldg, int up_off, const float* __restrict__ row_w, int ff, T* __restrict__ out,
-                            int ldo) {
+__global__ void gate_kernel(const GateSpec gs, const GateRows a, const GateRows b, int row0) {
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     pdl_wait();
-    const int r = blockIdx.y, i = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
-    if (i >= ldo) return;
-    const float s = row_w ? row_w[r] : 1.0f;
+    const int row = row0 + blockIdx.y;
+    const bool second = row >= a.rows;
+    const GateRows& g = second ? b : a;
+    const int r = second ? row - a.rows : row, i = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
+    if (i >= g.ldo) return;
+    const float s = g.row_w ? g.row_w[r] : 1.0f;
     float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-    if (i < ff) {  // gate and up rows are padded to multiples of 64: eight columns can always be read
-        float g[8], u[8];
-        Elt<T>::ld8(gu + (size_t)r * ldg + i, g);
-        Elt<T>::ld8(gu + (size_t)r * ldg + up_off + i, u);
+    if (i < g.ff) {  // gate and up rows are padded to multiples of 64: eight columns can always be read
+        float x[8], u[8];
+        if (g.gu_f32) {
+            const float* src = reinterpret_cast<const float*>(g.gu) + (size_t)r * g.ldg + i;
+            Elt<float>::ld8(src, x);
+            Elt<float>::ld8(src + g.up_off, u);
+        } else {
+            const T* src = reinterpret_cast<const T*>(g.gu) + (size_t)r * g.ldg + i;
+            Elt<T>::ld8(src, x);
+            Elt<T>::ld8(src + g.up_off, u);
+        }
 #pragma unroll
-        for (int j = 0; j < 8; j++) v[j] = i + j >= ff ? 0.f : gs.scale_out ? gate_one(gs, g[j], u[j]) * s : gate_one(gs, g[j] * s, u[j] * s);
+        for (int j = 0; j < 8; j++) v[j] = i + j >= g.ff ? 0.f : gs.scale_out ? gate_one(gs, x[j], u[j]) * s : gate_one(gs, x[j] * s, u[j] * s);
     }
-    Elt<T>::st8(out + (size_t)r * ldo + i, v);
+    Elt<T>::st8(reinterpret_cast<T*>(g.out) + (size_t)r * g.ldo + i, v);
 }
 
-template <typename T>
-__global__ void tanh_kernel(const float* __restrict__ x, int ldx, int n, T* __restrict__ out, int ldo) {
-    asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
+__global__ void tanh_kernel(const float* __restrict__ x, int ldx, int n, float* __restrict__ out, int ldo) {
     pdl_wait();
-    for (int i = threadIdx.x; i < ldo; i += blockDim.x) Elt<T>::st(out + (size_t)blockIdx.x * ldo + i, i < n ? tanhf(x[(size_t)blockIdx.x * ldx + i]) : 0.f);
+    for (int i = threadIdx.x; i < ldo; i += blockDim.x) out[(size_t)blockIdx.x * ldo + i] = i < n ? tanhf(x[(size_t)blockIdx.x * ldx + i]) : 0.f;
 }
 
 template <typename T>
@@ -325,7 +344,7 @@ int32_t b2_stream_norm_launch(b2_ctx* ctx, bool f32, const StreamNormParams& p) 
     if (p.rows <= 0) return B2_OK;
     B2_REQUIRE(p.streams >= 1 && p.streams <= kMaxStreams, B2_ERR_UNSUPPORTED, "residual streams: 1 to 16");
     const bool vec = p.width % 4 == 0 && p.ldx % 4 == 0 && p.ldy % 4 == 0 && p.ldh % 4 == 0;
-    const int th = threads_for(p.width, vec ? 4 : 1, 512);
+    const int th = threads_for(p.width, vec ? 4 : 1, p.streams <= 4 && vec && p.rows <= 2 * ctx->sm_count ? 1024 : 512);
     const size_t smem = ((size_t)p.width * 4 + 15) / 16 * 16;
     B2_REQUIRE(smem <= 200 * 1024, B2_ERR_UNSUPPORTED, "stream_norm: the model is too wide");
     auto run = [&](auto k) -> int32_t {
@@ -345,30 +364,19 @@ int32_t b2_stream_norm_launch(b2_ctx* ctx, bool f32, const StreamNormParams& p) 
     };
     return f32 ? pick(float{}) : pick(uint16_t{});
 }
-int32_t b2_tanh_launch(b2_ctx* ctx, bool f32, const float* x, int ldx, int T, int n, void* out, int ldo) {
+int32_t b2_tanh_launch(b2_ctx* ctx, const float* x, int ldx, int T, int n, float* out, int ldo) {
     if (T <= 0) return B2_OK;
-    const int th = threads_for(ldo, 1, 256);
-    if (f32)
-        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, tanh_kernel<float>, dim3(T), dim3(th), 0, ctx->stream, x, ldx, n, (float*)out, ldo));
-    else
-        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, tanh_kernel<uint16_t>, dim3(T), dim3(th), 0, ctx->stream, x, ldx, n, (uint16_t*)out, ldo));
+    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, tanh_kernel, dim3(T), dim3(threads_for(ldo, 1, 256)), 0, ctx->stream, x, ldx, n, out, ldo));
     B2_LAUNCHED(ctx);
     return B2_OK;
 }
-int32_t b2_gate_launch(b2_ctx* ctx, bool f32, const GateSpec& g, const void* gu, int ldg, int up_off, const float* row_w, int rows, int ff, void* out,
-                       int ldo) {
+int32_t b2_gate_launch(b2_ctx* ctx, bool f32, const GateSpec& g, const GateRows& a, const GateRows& b) {
+    const int rows = a.rows + b.rows, ldo = a.ldo > b.ldo ? a.ldo : b.ldo;
     if (rows <= 0) return B2_OK;
     const int th = threads_for(ldo, 8, 256);
     for (int r0 = 0; r0 < rows; r0 += 65535) {  // grid.y limit
-        const int n = rows - r0 < 65535 ? rows - r0 : 65535;
-        const dim3 grid((ldo / 8 + th - 1) / th, n);
-        const float* rw = row_w ? row_w + r0 : nullptr;
-        if (f32)
-            B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, gate_kernel<float>, grid, dim3(th), 0, ctx->stream, g, (const float*)gu + (size_t)r0 * ldg, ldg, up_off, rw, ff,
-                                  (float*)out + (size_t)r0 * ldo, ldo));
-        else
-            B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, gate_kernel<uint16_t>, grid, dim3(th), 0, ctx->stream, g, (const uint16_t*)gu + (size_t)r0 * ldg, ldg, up_off, rw, ff,
-                                  (uint16_t*)out + (size_t)r0 * ldo, ldo));
+        const dim3 grid((ldo / 8 + th - 1) / th, rows - r0 < 65535 ? rows - r0 : 65535);
+        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, f32 ? gate_kernel<float> : gate_kernel<uint16_t>, grid, dim3(th), 0, ctx->stream, g, a, b, r0));
         B2_LAUNCHED(ctx);
     }
     return B2_OK;

@@ -112,33 +112,87 @@ __global__ void __launch_bounds__(256) token_shift_kernel(const ShiftParams p, i
     }
 }
 
-// Time mixing: queries and keys as f32, and the logarithms -exp(z + w0) of the decays.  Below e^-128 an f32 decay is zero: the
-// logarithm stops there, which keeps its sums finite.
-template <typename T, int VEC>
-__global__ void __launch_bounds__(256) memory_mix_prep_kernel(const MemorySpec s, const MemoryParams p) {
+// Time mixing: logarithms -exp(z + w0) of the decays (queries and keys need no preparation).  Below e^-128 an f32 decay is zero:
+// the logarithm stops there, which keeps its sums finite.
+__device__ __forceinline__ float log_decay_of(float x) { return fmaxf(-expf(x), -128.f); }
+__global__ void __launch_bounds__(256) memory_decay_kernel(const MemorySpec s, const MemoryParams p) {
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     pdl_wait();
-    const int Q = s.q_cols(), i = (blockIdx.x * 256 + threadIdx.x) * VEC, t = blockIdx.y;
-    if (i >= Q) return;
-    const T* in = reinterpret_cast<const T*>(p.in) + (size_t)t * p.ld + p.c_off + i;
-    const float* z = reinterpret_cast<const float*>(p.dec) + (size_t)t * p.ld_dec + i;
-    const size_t at = (size_t)t * Q + i;
-    auto decay = [](float x) { return fmaxf(-expf(x), -128.f); };
-    if constexpr (VEC == 4) {
-        float v[4], w[4];
-        Elt<T>::ld4(in, v);
-        Elt<float>::st4(p.q + at, v);
-        Elt<T>::ld4(in + Q, v);
-        Elt<float>::st4(p.k + at, v);
-        Elt<float>::ld4(z, v);
-        Elt<float>::ld4(p.dt_bias + i, w);
+    const int Q = s.q_cols(), i = blockIdx.x * 256 + threadIdx.x, t = blockIdx.y;
+    if (i < Q) p.lg[(size_t)t * Q + i] = log_decay_of(reinterpret_cast<const float*>(p.dec)[(size_t)t * p.ld_dec + i] + p.dt_bias[i]);
+}
+// ... from the first factor's result x (f32): z = tanh(x) W2^T, bf16 operands.  Block = 16 MT tokens x 128 channels, a warp 16
+// channels; 64 inputs at a time.
+template <int MT>
+__global__ void __launch_bounds__(256) memory_decay_tc_kernel(const MemorySpec s, const MemoryParams p) {
+    constexpr int TM = 16 * MT;
+    __shared__ __align__(128) uint8_t sa[TM * 128], sb[128 * 128];
+    asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, n0 = blockIdx.x * 128, t0 = blockIdx.y * TM, mi = lane >> 3, lr = lane & 7;
+    const uint32_t base_a = smem_u32(sa), base_b = smem_u32(sb);
+    const uint16_t* w = reinterpret_cast<const uint16_t*>(p.low_w) + (size_t)n0 * p.low_k;  // rows padded to whole blocks
+    auto load_w = [&](int k0) {
+        for (int c = tid; c < 128 * 8; c += 256) cp_async16(base_b + (c >> 3) * 128 + (((c & 7) ^ ((c >> 3) & 7)) << 4), w + (size_t)(c >> 3) * p.low_k + k0 + (c & 7) * 8);
+        cp_async_commit();
+    };
+    load_w(0);  // (weights: nothing earlier writes them)
+    pdl_wait();
+    float acc[MT][2][4];
 #pragma unroll
-        for (int e = 0; e < 4; e++) v[e] = decay(v[e] + w[e]);
-        Elt<float>::st4(p.lg + at, v);
-    } else {
-        p.q[at] = Elt<T>::ld(in);
-        p.k[at] = Elt<T>::ld(in + Q);
-        p.lg[at] = decay(z[0] + p.dt_bias[i]);
+    for (int i = 0; i < MT; i++)
+#pragma unroll
+        for (int j = 0; j < 2; j++) acc[i][j][0] = acc[i][j][1] = acc[i][j][2] = acc[i][j][3] = 0.f;
+    for (int k0 = 0; k0 < p.low_k; k0 += 64) {
+        for (int c = tid; c < TM * 32; c += 256) {  // pairs of inputs
+            const int r = c >> 5, x = (c & 31) * 2, col = k0 + x;
+            const float* src = p.low + (size_t)(t0 + r) * p.ld_low + col;
+            const bool ok = t0 + r < p.T;
+            const float u = ok && col < p.rank ? tanhf(src[0]) : 0.f, v = ok && col + 1 < p.rank ? tanhf(src[1]) : 0.f;
+            *reinterpret_cast<uint32_t*>(sa + r * 128 + (((x >> 3) ^ (r & 7)) << 4) + (x & 7) * 2) = pack_bf2(u, v);
+        }
+        cp_async_wait<0>();
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < 4; k++) {
+            uint32_t b0[2], b1[2];
+            {
+                const int r = warp * 16 + lr + (mi >> 1) * 8, ch = 2 * k + (mi & 1);
+                ldmatrix_x4(b0[0], b0[1], b1[0], b1[1], base_b + r * 128 + ((ch ^ (r & 7)) << 4));
+            }
+#pragma unroll
+            for (int i = 0; i < MT; i++) {
+                const int r = i * 16 + lr + (mi & 1) * 8, ch = 2 * k + (mi >> 1);
+                uint32_t f[4];
+                ldmatrix_x4(f[0], f[1], f[2], f[3], base_a + r * 128 + ((ch ^ (r & 7)) << 4));
+                mma_bf16_16816(acc[i][0], f, b0);
+                mma_bf16_16816(acc[i][1], f, b1);
+            }
+        }
+        __syncthreads();
+        if (k0 + 64 < p.low_k) load_w(k0 + 64);
+    }
+    const int Q = s.q_cols();
+#pragma unroll
+    for (int j = 0; j < 2; j++) {
+        const int col = n0 + warp * 16 + j * 8 + 2 * (lane & 3);
+        if (col >= Q) continue;
+        const bool two = col + 1 < Q;
+        const float w0 = p.dt_bias[col], w1 = two ? p.dt_bias[col + 1] : 0.f;
+#pragma unroll
+        for (int i = 0; i < MT; i++)
+#pragma unroll
+            for (int h = 0; h < 2; h++) {
+                const int t = t0 + i * 16 + h * 8 + (lane >> 2);
+                if (t >= p.T) continue;
+                float* d = p.lg + (size_t)t * Q + col;
+                const float u = log_decay_of(acc[i][j][2 * h] + w0), v = log_decay_of(acc[i][j][2 * h + 1] + w1);
+                if (Q % 2 == 0) {
+                    *reinterpret_cast<float2*>(d) = make_float2(u, v);
+                } else {
+                    d[0] = u;
+                    if (two) d[1] = v;
+                }
+            }
     }
 }
 
@@ -363,8 +417,14 @@ __global__ void __launch_bounds__(128) memory_scan_kernel(const MemorySpec s, co
         for (int i = tid; i < cnt * NP; i += 128) {
             const int t = i / NP, c = i - t * NP;
             const size_t tok = (size_t)(start + t0 + t);
-            Ks[t][c] = c < D ? p.k[tok * Q + kh * D + c] : 0.f;
-            Qs[t][c] = c < D ? p.q[tok * Q + kh * D + c] : 0.f;
+            if constexpr (BONUS) {  // straight from the projections
+                const T* x = reinterpret_cast<const T*>(p.in) + tok * p.ld + p.c_off + kh * D + c;
+                Ks[t][c] = c < D ? Elt<T>::ld(x + Q) : 0.f;
+                Qs[t][c] = c < D ? Elt<T>::ld(x) : 0.f;
+            } else {
+                Ks[t][c] = c < D ? p.k[tok * Q + kh * D + c] : 0.f;
+                Qs[t][c] = c < D ? p.q[tok * Q + kh * D + c] : 0.f;
+            }
             float g = 1.f;
             if (c < D)
                 g = s.decay == MemDecay::PerChannel ? expf(p.lg[tok * s.decays() + h * D + c]) : s.decay == MemDecay::PerHead ? expf(p.lg[tok * s.heads + h]) : p.decay[h];
@@ -439,14 +499,38 @@ __global__ void __launch_bounds__(128) memory_scan_kernel(const MemorySpec s, co
 }
 
 // A warp per (token, memory head) and per (token, 256 feed-forward columns); the last unit writes the zeros between the parts.
+// With heads of up to 64 values (`pairs`) half a warp per head, and a warp walks over the heads.
 template <typename T>
-__global__ void __launch_bounds__(256) branch_out_kernel(const BranchOutParams p) {
+__global__ void __launch_bounds__(256) branch_out_kernel(const BranchOutParams p, bool pairs) {
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     pdl_wait();
     const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int n_m = p.o ? p.heads : 0, n_f = p.up ? (p.ff + 255) / 256 : 0;
+    const int n_m = p.o ? (pairs ? 8 : p.heads) : 0, n_f = p.up ? (p.ff + 255) / 256 : 0;
     T* out = reinterpret_cast<T*>(p.out) + (size_t)t * p.ldo;
     int u = blockIdx.y * 8 + warp;
+    if (u < n_m && pairs) {
+        const int P = p.vdim, d = (lane & 15) * 4;
+        const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int h0 = u * 2; h0 < p.heads; h0 += 16) {
+            const int h = h0 + (lane >> 4);
+            const bool ok = h < p.heads && d < P;
+            const size_t at = (size_t)h * P + d;
+            const float4 v = ok ? *reinterpret_cast<const float4*>(p.o + (size_t)t * p.heads * P + at) : zero;
+            float g[4] = {0.f, 0.f, 0.f, 0.f}, w[4] = {1.f, 1.f, 1.f, 1.f};
+            if (ok) Elt<T>::ld4(reinterpret_cast<const T*>(p.gate) + (size_t)t * p.ld_gate + at, g);
+            if (ok && p.norm) Elt<float>::ld4(p.norm_heads ? p.norm + at : p.norm + d, w);
+            float ss = v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+#pragma unroll
+            for (int o = 8; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+            const float inv = p.scale / sqrtf(ss / (float)P + p.eps);
+            if (!ok) continue;
+#pragma unroll
+            for (int e = 0; e < 4; e++) w[e] *= inv * (p.act == MemGate::Silu ? silu_for<T>(g[e]) : sigmoid_f32(g[e]));
+            const float r[4] = {v.x * w[0], v.y * w[1], v.z * w[2], v.w * w[3]};
+            Elt<T>::st4(out + p.m_off + at, r);
+        }
+        return;
+    }
     if (u < n_m) {
         const int P = p.vdim;
         const float* o = p.o + ((size_t)t * p.heads + u) * P;
@@ -503,7 +587,7 @@ __global__ void __launch_bounds__(256) branch_out_kernel(const BranchOutParams p
     auto zero_to = [&](int c1) {
         for (int c = at + lane; c < c1; c += 32) Elt<T>::st(out + c, 0.f);
     };
-    if (n_m) zero_to(p.m_off), at = p.m_off + p.heads * p.vdim;
+    if (p.o) zero_to(p.m_off), at = p.m_off + p.heads * p.vdim;
     if (n_f) zero_to(p.f_off), at = p.f_off + p.ff;
     zero_to(p.ldo);
 }
@@ -524,9 +608,13 @@ int32_t launch_prep(b2_ctx* ctx, const MemorySpec& s, const MemoryParams& p) {
 template <typename T>
 int32_t launch_memory(b2_ctx* ctx, const MemorySpec& s, const MemoryParams& p) {
     if (s.shift > 0) {
-        const bool vec = s.q_cols() % 4 == 0 && p.c_off % 4 == 0 && p.ld % 4 == 0 && p.ld_dec % 4 == 0;
-        const dim3 grid((unsigned)((s.q_cols() + (vec ? 1023 : 255)) / (vec ? 1024 : 256)), p.T);
-        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, vec ? memory_mix_prep_kernel<T, 4> : memory_mix_prep_kernel<T, 1>, grid, dim3(256), 0, ctx->stream, s, p));
+        if (p.low) {
+            const int bx = (s.q_cols() + 127) / 128;
+            B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, p.T <= 16 ? memory_decay_tc_kernel<1> : memory_decay_tc_kernel<4>, dim3(bx, p.T <= 16 ? 1 : (p.T + 63) / 64), dim3(256), 0, ctx->stream,
+                                  s, p));
+        } else {
+            B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, memory_decay_kernel, dim3((s.q_cols() + 255) / 256, p.T), dim3(256), 0, ctx->stream, s, p));
+        }
         B2_LAUNCHED(ctx);
     } else if (s.conv > 0) {
         const bool vec = s.dim % 4 == 0 && (s.heads * s.vdim) % 4 == 0 && p.ld_dec % 4 == 0 && p.c_off % 4 == 0 && p.ld % 4 == 0 && p.ld_v % 4 == 0;
@@ -578,8 +666,10 @@ int32_t b2_token_shift_launch(b2_ctx* ctx, bool f32, const ShiftParams& p) {
 }
 int32_t b2_branch_out_launch(b2_ctx* ctx, bool f32, const BranchOutParams& p) {
     if (p.T <= 0) return B2_OK;
-    const int units = (p.o ? p.heads : 0) + (p.up ? (p.ff + 255) / 256 : 0) + 1;
-    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, f32 ? branch_out_kernel<float> : branch_out_kernel<uint16_t>, dim3(p.T, (units + 7) / 8), dim3(256), 0, ctx->stream, p));
+    if (!p.o && !p.up && p.att_cols == p.ldo) return B2_OK;  // nothing to add, no padding
+    const bool pairs = p.o && p.vdim <= 64 && p.vdim % 4 == 0 && p.ld_gate % 4 == 0 && ((uintptr_t)p.gate & (f32 ? 15 : 7)) == 0 && p.m_off % 4 == 0;
+    const int units = (p.o ? (pairs ? 8 : p.heads) : 0) + (p.up ? (p.ff + 255) / 256 : 0) + 1;
+    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, f32 ? branch_out_kernel<float> : branch_out_kernel<uint16_t>, dim3(p.T, (units + 7) / 8), dim3(256), 0, ctx->stream, p, pairs));
     B2_LAUNCHED(ctx);
     return B2_OK;
 }

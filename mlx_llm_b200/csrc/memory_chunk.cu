@@ -12,6 +12,8 @@
 //
 // Every operand that is f32 by nature enters the products as a bf16 head plus a bf16 remainder (the product of the two
 // remainders is dropped), all sums are f32, and the state stays in f32 registers from chunk to chunk.
+#include <type_traits>
+
 #include "memory.cuh"
 #include "tc5.cuh"
 
@@ -66,7 +68,8 @@ struct FactorSmem {
     static constexpr int M = G, Y = G + (kG > kM ? kG : kM), REF = Y + 3 * 16 * 17 * 4, BETA = REF + (CHANNEL ? 9 * DK * 4 : C * 4), kBytes = BETA + C * 4;
 };
 
-template <int DK, bool CHANNEL>
+// BONUS: queries and keys are bf16, straight from the projections.
+template <int DK, bool CHANNEL, bool BONUS>
 __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const MemorySpec s, const MemoryParams p) {
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     pdl_wait();
@@ -92,7 +95,17 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
     if (cnt <= 0) return;
     const size_t tok0 = (size_t)p.cu_seqlens[b] + t0;
     uint8_t* rec = reinterpret_cast<uint8_t*>(p.chunk) + ((size_t)chunk * s.heads + h) * R::kBytes;
-    const float *q = p.q + tok0 * Q + kh * D, *k = p.k + tok0 * Q + kh * D;
+    using E = typename std::conditional<BONUS, uint16_t, float>::type;
+    const E *q, *k;
+    size_t ldq = Q;
+    if constexpr (BONUS) {
+        ldq = p.ld;
+        q = reinterpret_cast<const uint16_t*>(p.in) + tok0 * ldq + p.c_off + kh * D;
+        k = q + Q;
+    } else {
+        q = p.q + tok0 * Q + kh * D;
+        k = p.k + tok0 * Q + kh * D;
+    }
     const float* lg = CHANNEL ? p.lg + tok0 * s.decays() + h * D : nullptr;
 
     if (tid < 4 * (DK / 32)) fast[tid / (DK / 32)][tid % (DK / 32)] = 0;
@@ -152,7 +165,7 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
     __syncthreads();
 
     // ---- one pass over the chunk, eight columns at a time: the tiles' operands and the walk's
-    const bool vec = D % 4 == 0 && Q % 4 == 0;
+    const bool vec = D % 4 == 0 && Q % 4 == 0 && (!BONUS || (p.ld % 4 == 0 && p.c_off % 4 == 0));
     for (int i = tid; i < C * (DK / 8); i += F_THREADS) {
         const int t = i / (DK / 8), x = i % (DK / 8), blk = t >> 4;
         float kv[8], qv[8], left[8], right[8], a[8];
@@ -160,17 +173,19 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
         for (int e = 0; e < 8; e += 4) {
             const int d = x * 8 + e;
             if (vec) {
-                const bool ok = t < cnt && d < D;
-                const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
-                const float4 k4 = ok ? *reinterpret_cast<const float4*>(k + (size_t)t * Q + d) : z, q4 = ok ? *reinterpret_cast<const float4*>(q + (size_t)t * Q + d) : z;
-                kv[e] = k4.x, kv[e + 1] = k4.y, kv[e + 2] = k4.z, kv[e + 3] = k4.w;
-                qv[e] = q4.x, qv[e + 1] = q4.y, qv[e + 2] = q4.z, qv[e + 3] = q4.w;
+                float k4[4] = {0.f, 0.f, 0.f, 0.f}, q4[4] = {0.f, 0.f, 0.f, 0.f};
+                if (t < cnt && d < D) {
+                    Elt<E>::ld4(k + t * ldq + d, k4);
+                    Elt<E>::ld4(q + t * ldq + d, q4);
+                }
+#pragma unroll
+                for (int f = 0; f < 4; f++) kv[e + f] = k4[f], qv[e + f] = q4[f];
             } else {
 #pragma unroll
                 for (int f = 0; f < 4; f++) {
                     const bool ok = t < cnt && d + f < D;
-                    kv[e + f] = ok ? k[(size_t)t * Q + d + f] : 0.f;
-                    qv[e + f] = ok ? q[(size_t)t * Q + d + f] : 0.f;
+                    kv[e + f] = ok ? Elt<E>::ld(k + t * ldq + d + f) : 0.f;
+                    qv[e + f] = ok ? Elt<E>::ld(q + t * ldq + d + f) : 0.f;
                 }
             }
         }
@@ -186,7 +201,7 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
             float r0[8], tail[8];  // e^(m_i), e^(G_end - m_i)
             float own[8];          // bonus: the token's own decay, which its read-out does not see
 #pragma unroll
-            for (int e = 0; e < 8; e++) own[e] = s.bonus && t < cnt && x * 8 + e < D ? lg[(size_t)t * s.decays() + x * 8 + e] * kLog2e : 0.f;
+            for (int e = 0; e < 8; e++) own[e] = BONUS && t < cnt && x * 8 + e < D ? lg[(size_t)t * s.decays() + x * 8 + e] * kLog2e : 0.f;
 #pragma unroll
             for (int e = 0; e < 8; e++) {
                 const int d = x * 8 + e;
@@ -199,7 +214,7 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
             }
 #pragma unroll
             for (int e = 0; e < 8; e++) a[e] = kv[e] * left[e];
-            if (s.delta) {
+            if (!BONUS && s.delta) {
                 store(smem + L::LK, a);
 #pragma unroll
                 for (int e = 0; e < 8; e++) a[e] *= r0[e];
@@ -220,7 +235,7 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
             store(smem + L::LQ, qv);
 #pragma unroll
             for (int e = 0; e < 8; e++) a[e] = kv[e] * f;
-            if (s.delta) store(rec + R::Kf, a);
+            if (!BONUS && s.delta) store(rec + R::Kf, a);
 #pragma unroll
             for (int e = 0; e < 8; e++) a[e] = qv[e] * f;
             store(rec + R::Qf, a);
@@ -229,11 +244,11 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
             store(rec + R::Kb, a);
         }
     }
-    if (s.bonus) {  // the diagonal of P, in the place of the step sizes
+    if constexpr (BONUS) {  // the diagonal of P, in the place of the step sizes
         for (int t = warp; t < C; t += F_WARPS) {
             float v = 0.f;
             if (t < cnt)
-                for (int d = lane; d < D; d += 32) v = fmaf(q[(size_t)t * Q + d] * p.bonus[(size_t)h * D + d], k[(size_t)t * Q + d], v);
+                for (int d = lane; d < D; d += 32) v = fmaf(Elt<E>::ld(q + t * ldq + d) * p.bonus[(size_t)h * D + d], Elt<E>::ld(k + t * ldq + d), v);
 #pragma unroll
             for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
             if (lane == 0) betas[t] = v;
@@ -256,7 +271,7 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
         for (int kk = 0; kk < DK / 16; kk++) {
             uint32_t ah[4], al[4], qh[4], ql[4], bh[2][2], bl[2][2];
             const uint32_t at = at_wide(16 * i + lr + (mi & 1) * 8, 2 * kk + (mi >> 1), DK * 2);
-            if (s.delta) {
+            if (!BONUS && s.delta) {
                 ldmatrix_x4(ah[0], ah[1], ah[2], ah[3], base + L::LK + at);
                 ldmatrix_x4(al[0], al[1], al[2], al[3], base + L::LK + R::kOp + at);
             }
@@ -284,7 +299,7 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
             }
 #pragma unroll
             for (int half = 0; half < 2; half++) {
-                if (s.delta) mma3(a[half], ah, al, bh[half], bl[half]);
+                if (!BONUS && s.delta) mma3(a[half], ah, al, bh[half], bl[half]);
                 mma3(pr[half], qh, ql, bh[half], bl[half]);
             }
         }
@@ -296,17 +311,17 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
                 const int d = word * 32 + __ffs(m) - 1, tok = 16 * i + (lane & 15);  // a lane per token
                 const bool ok = tok < cnt && d < D;
                 float g = ok ? lg[(size_t)tok * s.decays() + d] * kLog2e : 0.f;
-                const float kv = ok ? k[(size_t)tok * Q + d] : 0.f, qv = ok ? q[(size_t)tok * Q + d] : 0.f;
+                const float kv = ok ? Elt<E>::ld(k + tok * ldq + d) : 0.f, qv = ok ? Elt<E>::ld(q + tok * ldq + d) : 0.f;
 #pragma unroll
                 for (int o = 1; o < 16; o <<= 1) {
                     const float x = __shfl_up_sync(0xffffffffu, g, o, 16);
                     if ((lane & 15) >= o) g += x;
                 }
                 float gt[2], kt[2], qt[2];
-                const float before = s.bonus ? __shfl_up_sync(0xffffffffu, g, 1, 16) : 0.f;  // (the first token's is not used)
+                const float before = BONUS ? __shfl_up_sync(0xffffffffu, g, 1, 16) : 0.f;  // (the first token's is not used)
 #pragma unroll
                 for (int x = 0; x < 2; x++) {
-                    gt[x] = __shfl_sync(0xffffffffu, s.bonus ? before : g, g4 + 8 * x);
+                    gt[x] = __shfl_sync(0xffffffffu, BONUS ? before : g, g4 + 8 * x);
                     kt[x] = __shfl_sync(0xffffffffu, kv, g4 + 8 * x);
                     qt[x] = __shfl_sync(0xffffffffu, qv, g4 + 8 * x);
                 }
@@ -318,7 +333,7 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
                         const float gu = __shfl_sync(0xffffffffu, g, u), ku = __shfl_sync(0xffffffffu, kv, u);
 #pragma unroll
                         for (int x = 0; x < 2; x++)
-                            if (s.bonus ? u < g4 + 8 * x : u <= g4 + 8 * x) {
+                            if (BONUS ? u < g4 + 8 * x : u <= g4 + 8 * x) {
                                 const float w = fast_exp2(gt[x] - gu) * ku;
                                 a[half][2 * x + c] = fmaf(w, kt[x], a[half][2 * x + c]);
                                 pr[half][2 * x + c] = fmaf(w, qt[x], pr[half][2 * x + c]);
@@ -339,8 +354,8 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
                 pr[half][e] *= w;
             }
             if (u > t) pr[half][e] = 0.f;
-            if (CHANNEL && s.bonus && u == t) pr[half][e] = betas[t];
-            if (s.delta && u < t) M[t * LM + u] = a[half][e] * betas[t];
+            if (CHANNEL && BONUS && u == t) pr[half][e] = betas[t];
+            if (!BONUS && s.delta && u < t) M[t * LM + u] = a[half][e] * betas[t];
         }
 #pragma unroll
         for (int row = 0; row < 2; row++) {
@@ -356,7 +371,7 @@ __global__ void __launch_bounds__(F_THREADS, 2) memory_factor_kernel(const Memor
     } else if (s.decay == MemDecay::PerHead && tid == 0) {
         p.lg[tok0 * s.heads + h] = fast_exp2(ref[last]);
     }
-    if (!s.delta) return;
+    if (BONUS || !s.delta) return;
     // ---- inverse of the unit lower triangular I + A: diagonal blocks, then block diagonals outwards
     //      T_ij = -T_ii sum_{j <= k < i} A_ik T_kj.  T_ts is kept at M[s][t], its unit diagonal implied.
     __syncthreads();
@@ -701,20 +716,22 @@ __global__ void __launch_bounds__(W_THREADS, 1) memory_chunk_kernel(const Memory
     memory_keep_inputs<uint16_t>(s, p, b, blockIdx.y * gridDim.x + blockIdx.x, gridDim.x * gridDim.y);
 }
 
-template <int DK, bool CHANNEL>
+template <int DK, bool CHANNEL, bool BONUS>
 int32_t launch_factors(b2_ctx* ctx, const MemorySpec& s, const MemoryParams& p) {
     constexpr int kBytes = FactorSmem<DK, CHANNEL>::kBytes;
-    B2_SMEM_ONCE(ctx, (memory_factor_kernel<DK, CHANNEL>), kBytes);
-    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, memory_factor_kernel<DK, CHANNEL>, dim3(p.n_chunks, s.heads), dim3(F_THREADS), (size_t)kBytes, ctx->stream, s, p));
+    B2_SMEM_ONCE(ctx, (memory_factor_kernel<DK, CHANNEL, BONUS>), kBytes);
+    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, memory_factor_kernel<DK, CHANNEL, BONUS>, dim3(p.n_chunks, s.heads), dim3(F_THREADS), (size_t)kBytes, ctx->stream, s, p));
     B2_LAUNCHED(ctx);
     return B2_OK;
 }
 template <int DK>
 int32_t launch(b2_ctx* ctx, const MemorySpec& s, const MemoryParams& p) {
-    if (s.decay == MemDecay::PerChannel)
-        B2_CHECK((launch_factors<DK, true>(ctx, s, p)));
+    if (s.bonus)
+        B2_CHECK((launch_factors<DK, true, true>(ctx, s, p)));
+    else if (s.decay == MemDecay::PerChannel)
+        B2_CHECK((launch_factors<DK, true, false>(ctx, s, p)));
     else
-        B2_CHECK((launch_factors<DK, false>(ctx, s, p)));
+        B2_CHECK((launch_factors<DK, false, false>(ctx, s, p)));
     constexpr int kBytes = WalkSmem<DK>::kBytes;
     B2_SMEM_ONCE(ctx, (memory_chunk_kernel<DK, true>), kBytes);
     B2_SMEM_ONCE(ctx, (memory_chunk_kernel<DK, false>), kBytes);

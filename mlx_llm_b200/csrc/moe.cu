@@ -2,8 +2,8 @@
 // token, and the sorted order in which the grouped projections walk the (token, choice) pairs.  Identity experts are counted
 // apart: their pairs have no place in that order.
 //
-// One launch: every warp routes tokens and counts its choices; the block that finishes last turns the counts into
-// offsets and places the pairs.  The place of a pair inside its expert's run depends on timing, its result does not:
+// One launch: every warp routes tokens and counts its choices; the block that finishes last (a single block: the block itself,
+// which counts in shared memory) turns the counts into offsets and places the pairs.  The place of a pair inside its expert's run depends on timing, its result does not:
 // rows of a grouped product are independent.
 #include "elt.cuh"
 #include "layer_kernels.h"
@@ -16,7 +16,11 @@ __global__ void __launch_bounds__(kMaxThreads) route_kernel(const RouteParams p)
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     pdl_wait();
     extern __shared__ float sc[];  // [warps][outputs]: logits (Sigmoid) or choice scores (Softmax) of the token, -inf once taken
-    __shared__ int cursor[kMaxExperts];
+    __shared__ int cursor[kMaxExperts], own[kMaxExperts];
+    const bool one = gridDim.x == 1;
+    if (one)
+        for (int e = threadIdx.x; e < p.experts; e += blockDim.x) own[e] = 0;
+    __syncthreads();
     __shared__ bool last;
     __shared__ int total;  // pairs that have a place
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5, E = p.experts, N = E + p.identity;
@@ -53,7 +57,7 @@ __global__ void __launch_bounds__(kMaxThreads) route_kernel(const RouteParams p)
                 s[bi] = -INFINITY;
                 sum += w;
                 if (bi < E)
-                    atomicAdd(&p.counters[bi], 1);
+                    atomicAdd(one ? &own[bi] : &p.counters[bi], 1);
                 else
                     passed += w;
             }
@@ -67,16 +71,20 @@ __global__ void __launch_bounds__(kMaxThreads) route_kernel(const RouteParams p)
         if (p.shared && lane == 0) p.shared_w[t] = sigmoid_f32(z[N]);
         __syncwarp();
     }
-    __threadfence();
-    __syncthreads();
-    if (threadIdx.x == 0) last = atomicAdd(&p.counters[E], 1) == (int)gridDim.x - 1;
-    __syncthreads();
-    if (!last) return;
-    __threadfence();
+    if (!one) {
+        __threadfence();
+        __syncthreads();
+        if (threadIdx.x == 0) last = atomicAdd(&p.counters[E], 1) == (int)gridDim.x - 1;
+        __syncthreads();
+        if (!last) return;
+        __threadfence();
+    } else {
+        __syncthreads();
+    }
     if (warp == 0) {  // exclusive prefix sum of the counts, 32 experts at a time
         int base = 0;
         for (int e0 = 0; e0 < E; e0 += 32) {
-            const int n = e0 + lane < E ? __ldcg(&p.counters[e0 + lane]) : 0;
+            const int n = e0 + lane < E ? (one ? own[e0 + lane] : __ldcg(&p.counters[e0 + lane])) : 0;
             int incl = n;
 #pragma unroll
             for (int o = 1; o < 32; o <<= 1) {
@@ -92,7 +100,7 @@ __global__ void __launch_bounds__(kMaxThreads) route_kernel(const RouteParams p)
         if (lane == 0) p.offsets[E] = total = base;
     }
     __syncthreads();
-    for (int e = threadIdx.x; e <= E; e += blockDim.x) p.counters[e] = 0;  // ready for the next launch
+    for (int e = threadIdx.x; !one && e <= E; e += blockDim.x) p.counters[e] = 0;  // ready for the next launch
     const int per = p.top + (p.shared ? 1 : 0);
     for (int i = threadIdx.x; i < p.T * p.top; i += blockDim.x) {
         const int e = __ldcg(&p.expert[i]), t = i / p.top;
