@@ -128,10 +128,11 @@ __global__ void __launch_bounds__(NS <= 4 ? 1024 : 512) stream_norm_kernel(const
             float y[VEC];
 #pragma unroll
             for (int e = 0; e < VEC; e++) y[e] = 0.f;
-            for (int k0 = 0; k0 < n_src; k0 += 4) {  // four sources on their way at a time
-                float v[4][VEC];
+            constexpr int FLY = 2;  // sources on their way at a time
+            for (int k0 = 0; k0 < n_src; k0 += FLY) {
+                float v[FLY][VEC];
 #pragma unroll
-                for (int k = 0; k < 4; k++) {
+                for (int k = 0; k < FLY; k++) {
                     const int yr = k0 + k >= n_src ? -1 : k0 + k < kStreamSources ? src[k0 + k] : p.y_rows[(size_t)t * n_src + k0 + k];
                     if (yr >= 0)
                         load(p.y + (size_t)yr * p.ldy + i, v[k]);
@@ -140,7 +141,7 @@ __global__ void __launch_bounds__(NS <= 4 ? 1024 : 512) stream_norm_kernel(const
                         for (int e = 0; e < VEC; e++) v[k][e] = 0.f;
                 }
 #pragma unroll
-                for (int k = 0; k < 4; k++)
+                for (int k = 0; k < FLY; k++)
 #pragma unroll
                     for (int e = 0; e < VEC; e++) y[e] += v[k][e];
             }

@@ -499,19 +499,19 @@ __global__ void __launch_bounds__(128) memory_scan_kernel(const MemorySpec s, co
 }
 
 // A warp per (token, memory head) and per (token, 256 feed-forward columns); the last unit writes the zeros between the parts.
-// With heads of up to 64 values (`pairs`) half a warp per head, and a warp walks over the heads.
+// With heads of up to 64 values (`pairs` > 0) half a warp per head, and that many warps walk over the heads.
 template <typename T>
-__global__ void __launch_bounds__(256) branch_out_kernel(const BranchOutParams p, bool pairs) {
+__global__ void __launch_bounds__(256) branch_out_kernel(const BranchOutParams p, int pairs) {
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     pdl_wait();
     const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int n_m = p.o ? (pairs ? 8 : p.heads) : 0, n_f = p.up ? (p.ff + 255) / 256 : 0;
+    const int n_m = p.o ? (pairs > 0 ? pairs : p.heads) : 0, n_f = p.up ? (p.ff + 255) / 256 : 0;
     T* out = reinterpret_cast<T*>(p.out) + (size_t)t * p.ldo;
     int u = blockIdx.y * 8 + warp;
-    if (u < n_m && pairs) {
+    if (u < n_m && pairs > 0) {
         const int P = p.vdim, d = (lane & 15) * 4;
         const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-        for (int h0 = u * 2; h0 < p.heads; h0 += 16) {
+        for (int h0 = u * 2; h0 < p.heads; h0 += 2 * pairs) {
             const int h = h0 + (lane >> 4);
             const bool ok = h < p.heads && d < P;
             const size_t at = (size_t)h * P + d;
@@ -667,8 +667,9 @@ int32_t b2_token_shift_launch(b2_ctx* ctx, bool f32, const ShiftParams& p) {
 int32_t b2_branch_out_launch(b2_ctx* ctx, bool f32, const BranchOutParams& p) {
     if (p.T <= 0) return B2_OK;
     if (!p.o && !p.up && p.att_cols == p.ldo) return B2_OK;  // nothing to add, no padding
-    const bool pairs = p.o && p.vdim <= 64 && p.vdim % 4 == 0 && p.ld_gate % 4 == 0 && ((uintptr_t)p.gate & (f32 ? 15 : 7)) == 0 && p.m_off % 4 == 0;
-    const int units = (p.o ? (pairs ? 8 : p.heads) : 0) + (p.up ? (p.ff + 255) / 256 : 0) + 1;
+    const bool narrow = p.o && p.vdim <= 64 && p.vdim % 4 == 0 && p.ld_gate % 4 == 0 && ((uintptr_t)p.gate & (f32 ? 15 : 7)) == 0 && p.m_off % 4 == 0;
+    const int pairs = narrow ? (p.T <= 2 * ctx->sm_count ? (p.heads + 1) / 2 : 8) : 0;  // (many tokens: fewer, longer warps)
+    const int units = (p.o ? (pairs > 0 ? pairs : p.heads) : 0) + (p.up ? (p.ff + 255) / 256 : 0) + 1;
     B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, f32 ? branch_out_kernel<float> : branch_out_kernel<uint16_t>, dim3(p.T, (units + 7) / 8), dim3(256), 0, ctx->stream, p, pairs));
     B2_LAUNCHED(ctx);
     return B2_OK;
