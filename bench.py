@@ -16,8 +16,9 @@ Prints ONE JSON line (rank 0).  Workloads:
   decode_only              decode iterations without prefill (the weight-streaming regime).
   qwen3_32b_q8_tp          BASELINE configuration 4: one Qwen3-32B-architecture Q8 model over N ranks.
   layered                  a layered design (--layered-design zukitar: latent attention, Mamba-2, routed experts; tirezen: capped sink
-                           attention beside delta memories, retention, delta memories) at sizes of real models beside the
-                           flat decoder of equal width, both dense bf16: prefill and decode steps at a few sizes.
+                           attention beside delta memories, retention, delta memories; zokuzen: time mixing, windowed latent
+                           and chunked attention, mixtures of experts, four residual streams) at sizes of real models beside
+                           the flat decoder of equal width, both dense bf16: prefill and decode steps at a few sizes.
 A "step" is one iteration of the serving loop (one ragged forward over one batch).  The engine is
 first rolled to its steady state (`ramp` iterations, untimed, all requests available at t = 0), then W
 warm-up and K timed iterations follow.  `value` = generated tokens / device time of the K forwards

@@ -288,7 +288,8 @@ int32_t b2_model_logits_f32(const b2_model* m);
 /* Bytes of recurrent state one sequence holds besides its pages (0: none). */
 int64_t b2_model_state_bytes(const b2_model* m);
 /* Diagnostics of a layered model: after every following step, out_host (caller-owned, room for runs x tokens x width floats)
- * holds the residual stream behind every run of a layer (a repeated layer has several), [runs, tokens of the step, width].
+ * holds the residual stream (the sum of the streams, if the model has several) behind every run of a layer (a repeated layer has
+ * several), [runs, tokens of the step, width].
  * NULL switches it off. */
 int32_t b2_model_capture_residual(b2_model* m, float* out_host, int64_t capacity_floats);
 /* Random-init model generated on the device from a counter-based recipe (benchmark / parity helper;

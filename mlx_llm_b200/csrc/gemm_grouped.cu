@@ -414,5 +414,6 @@ int32_t b2_grouped_gemm_launch(b2_ctx* ctx, bool f32, const GroupedGemmParams& p
     const int per_group = p.offsets ? p.M / p.G : p.M;
     if (!p.stream && !p.row_idx && p.x_rows >= TC_M && b2_grouped_gemm_wants_rows(ctx, p.M, p.offsets != nullptr, p.G, p.N)) return launch_tc(ctx, p);
     if (per_group <= 16) return launch_tile<16, 6>(ctx, p);
+    if (p.stream && per_group <= 32) return launch_tile<32, 6>(ctx, p);
     return launch_tile<64, 4>(ctx, p);
 }

@@ -92,8 +92,8 @@ def tirezen_config(size, layers, vocab=32000):
                 layers=[dict(type=mixers[i % 4][0], mixer=mixers[i % 4][1], mlp=mlp) for i in range(layers)])
 
 
-# Zokuzen at the same widths: time mixing, windowed latent attention, time mixing, chunked attention, and in every second round the
-# chunked layer reads the keys of the round before; experts whose active part (chosen and shared) has the flat twin's inner size.
+# Zokuzen at the same widths: time mixing, windowed latent attention, time mixing, chunked attention, repeated; every second chunked
+# layer reads the keys of the one before it; experts whose active part (chosen and shared) has the flat twin's inner size.
 ZOKUZEN_SIZES = {
     "w4096": dict(wkv=dict(heads=64, dim=64), latent=dict(heads=32, dim=128, vdim=128, kv_rank=512), heads=32, kv_heads=8, expert_ff=1792, shared_ff=7168),
     "w2048": dict(wkv=dict(heads=32, dim=64), latent=dict(heads=16, dim=128, vdim=128, kv_rank=512), heads=16, kv_heads=4, expert_ff=1024, shared_ff=4096),

@@ -482,6 +482,26 @@ def test_long_decoding(env, name):
     assert e < TOL[False], e
 
 
+@BOTH
+@pytest.mark.parametrize("name", ["odd", "tiles"])
+@pytest.mark.parametrize("n", [16, 17, 32, 33, 64, 65, 100])
+def test_many_sequences_in_one_step(env, name, n, f32):
+    """Batches on both sides of the sizes at which products and launches are merged differently: every sequence decodes one token."""
+    ctx, eng = env
+    model, cfg, w = get_model(env, name, f32)
+    full = want_logits(name, cfg, w, 200)
+    ids = tokens(cfg, 200, 0)
+    pool = eng.BlockPool(ctx, model, 16, 3 * n, n, 3)
+    caches, lens = [eng.PagedKvCache(pool) for _ in range(n)], [3 + (7 * i) % 29 for i in range(n)]
+    model.step_at([(ids[:k], c) for k, c in zip(lens, caches)], [[] for _ in lens])
+    for s in range(2):
+        got, _ = model.step_at([(ids[k + s:k + s + 1], c) for k, c in zip(lens, caches)], [[0]] * n)
+        assert error(np.concatenate([got, full]), np.concatenate([full[[k + s for k in lens]], full])) < TOL[f32]
+    for c in caches:
+        c.free()
+    pool.free()
+
+
 def test_long_contexts_are_split_over_keys(env):
     """Windows and chunks of many work items, several sequences at different places of them, alone and beside a portion: partial
     results are added up."""
