@@ -3,7 +3,8 @@
 // The forward is called by the engine's step (b2_engine_forward) with the packer's metadata, like the flat decoders'
 // layers; pages, block tables, recurrent slots, scheduling and sampling are the engine's.  The residual stream is f32.
 // Every sub-layer leaves what it adds in `y` (f32); the next norm adds it to the stream on its way (b2_add_norm_launch; with several
-// streams b2_stream_norm_launch).
+// streams b2_stream_norm_launch).  Where the norms lie behind the sub-layers, one kernel norms y, adds it and leaves the next sub-layer's
+// input (b2_post_norm_launch).
 #include <algorithm>
 #include <cmath>
 #include <cstring>
@@ -54,12 +55,17 @@ struct LayerP {
     float *mu = nullptr, *bonus = nullptr;
     struct {
         int q = 0, k = 0, v = 0, c = 0, gate = 0, beta = 0, decay = 0, up = 0;  // columns of `in`
+        int head_gate = 0, z = 0, u = 0;                                       // ... (z, u, gate: of a gated average)
         int lr_gate = 0;                                                       // columns of `lr`: decay from 0, gate
         int m = 0, f = 0;                                                      // columns of the row `out` reads
     } at;
     float *q_bias = nullptr, *k_bias = nullptr, *v_bias = nullptr, *q_norm = nullptr, *k_norm = nullptr, *mem_norm = nullptr;
     float *decay = nullptr, *log_decay = nullptr;
     int mem_rope = -1;
+    float lambda = 0.f;  // weight of the second map
+    float *z_bias = nullptr, *u_bias = nullptr;
+    Proj side_gate, side_proj;
+    float *side_norm = nullptr, *avg = nullptr;
 };
 struct RopeTab {
     RotSpec spec;
@@ -76,6 +82,8 @@ struct LayeredModel {
     void* embed = nullptr;  // [pad_n(vocab), pad_k(width)]: embedding table, and output projection unless the model has one
     void* head = nullptr;
     float* loop_step = nullptr;  // [times][width]
+    Proj pairs, side;            // tables of the token pairs and of the layers' token inputs
+    int64_t pair_state = 0;      // where the slot's record keeps the last token
     float* final_norm = nullptr;
     std::vector<RopeTab> ropes;
     int rope_positions = 0;
@@ -271,7 +279,7 @@ struct Filler {
 
 int rope_table(LayeredModel& lm, const RotSpec& rot) {
     for (size_t r = 0; r < lm.ropes.size(); r++)
-        if (lm.ropes[r].spec.base == rot.base && lm.ropes[r].spec.dims == rot.dims) return (int)r;
+        if (lm.ropes[r].spec == rot) return (int)r;
     lm.ropes.push_back(RopeTab{rot});
     return (int)lm.ropes.size() - 1;
 }
@@ -296,9 +304,10 @@ int32_t load_branches(Filler& f, LayeredModel& lm, int i) {
     };
     if (L.has_gqa()) {
         B2_REQUIRE(a.dim <= 256 && a.vdim <= 256, B2_ERR_UNSUPPORTED, "grouped attention: head sizes up to 256");
-        take(P.at.q, a.heads * a.dim);
-        if (own_kv) take(P.at.k, a.kv_heads * a.dim);
+        take(P.at.q, a.q_heads() * a.dim);
+        if (own_kv) take(P.at.k, a.k_heads() * a.dim);
         if (own_kv) take(P.at.v, a.kv_heads * a.vdim);
+        if (a.head_gate) take(P.at.head_gate, a.heads);
     }
     if (L.has_mem()) {
         B2_REQUIRE(s.dim <= 256, B2_ERR_UNSUPPORTED, "memory: key sizes up to 256");
@@ -319,10 +328,23 @@ int32_t load_branches(Filler& f, LayeredModel& lm, int i) {
     if (ff) take(P.at.up, L.ff);
     B2_CHECK(f.proj(P.in, std::max(n, need), W));
     if (L.has_gqa()) {
-        B2_CHECK(f.rows(P.in, P.at.q, aq("q"), a.heads * a.dim, W));
+        B2_CHECK(f.rows(P.in, P.at.q, aq("q"), a.q_heads() * a.dim, W));
         if (own_kv) {
-            B2_CHECK(f.rows(P.in, P.at.k, aq("k"), a.kv_heads * a.dim, W));
+            B2_CHECK(f.rows(P.in, P.at.k, aq("k"), a.k_heads() * a.dim, W));
             B2_CHECK(f.rows(P.in, P.at.v, aq("v"), a.kv_heads * a.vdim, W));
+        }
+        if (a.head_gate) B2_CHECK(f.rows(P.in, P.at.head_gate, aq("g"), a.heads, W));
+        P.lambda = a.diff;
+        if (a.maps == 2 && f.w) {
+            double dot[2] = {0, 0};
+            for (int i = 0; i < 2; i++) {
+                const std::string n = std::to_string(i + 1);
+                B2_CHECK(f.fetch(aq("lq" + n), {a.dim}));
+                const std::vector<float> q = f.host;
+                B2_CHECK(f.fetch(aq("lk" + n), {a.dim}));
+                for (int d = 0; d < a.dim; d++) dot[i] += (double)q[d] * f.host[d];
+            }
+            P.lambda = (float)(std::exp(dot[0]) - std::exp(dot[1]) + (double)a.diff);
         }
         if (a.bias) {
             B2_CHECK(f.vec(P.q_bias, aq("q.b"), {a.heads * a.dim}, 0.f, 0.1f));
@@ -331,14 +353,14 @@ int32_t load_branches(Filler& f, LayeredModel& lm, int i) {
         }
         if (a.qk_norm) {
             B2_CHECK(f.vec(P.q_norm, aq("q.norm"), {a.dim}, 1.f, 0.f));
-            B2_CHECK(f.vec(P.k_norm, aq("k.norm"), {a.dim}, 1.f, 0.f));
+            if (own_kv) B2_CHECK(f.vec(P.k_norm, aq("k.norm"), {a.dim}, 1.f, 0.f));
         }
         if (a.norm_all) {
             B2_CHECK(f.vec(P.q_norm, aq("q.norm"), {a.heads * a.dim}, 1.f, 0.f));
             if (own_kv) B2_CHECK(f.vec(P.k_norm, aq("k.norm"), {a.kv_heads * a.dim}, 1.f, 0.f));
         }
         P.rope = rope_table(lm, a.rot);
-        lm.dec_part_row = std::max(lm.dec_part_row, (size_t)a.heads * (a.v_row() + 2));
+        lm.dec_part_row = std::max(lm.dec_part_row, (size_t)a.q_heads() * (a.v_row() + 2));
     }
     if (L.has_mem()) {
         const int Q = s.q_cols(), V = s.heads * s.vdim;
@@ -443,6 +465,50 @@ int32_t load_shifted(Filler& f, LayeredModel& lm, int i) {
     return f.rows(P.out, 0, key("o"), W, V);
 }
 
+// A gated average: one product for everything that reads the stream, one back.
+int32_t load_average(Filler& f, LayeredModel& lm, int i) {
+    const TensorNames& tn = lm.spec.names;
+    LayerP& P = lm.layers[i];
+    const int W = lm.spec.width, n = lm.spec.layers[i].avg.width, n8 = up(n, 8);
+    auto key = [&](const std::string& s) { return tn.layer_key(i, tn.mixer + "." + s); };
+    P.at.z = 0;
+    P.at.u = n8;
+    P.at.gate = 2 * n8;
+    B2_CHECK(f.proj(P.in, 3 * n8, W));
+    B2_CHECK(f.rows(P.in, P.at.z, key("z"), n, W));
+    B2_CHECK(f.rows(P.in, P.at.u, key("x"), n, W));
+    B2_CHECK(f.rows(P.in, P.at.gate, key("g"), n, W));
+    for (auto& b : {std::pair<const char*, float**>{"z.b", &P.z_bias}, {"x.b", &P.u_bias}}) {  // zero behind the width
+        std::vector<float> v((size_t)n8, 0.f);
+        if (f.w) {
+            B2_CHECK(f.fetch(key(b.first), {n}));
+            std::copy(f.host.begin(), f.host.end(), v.begin());
+        } else if (b.second == &P.z_bias) {
+            for (int j = 0; j < n; j++) v[j] = -1.f - 5.f * j / n;
+        }
+        B2_CHECK(f.upload(*b.second, v));
+    }
+    B2_CHECK(f.proj(P.out, W, n));
+    return f.rows(P.out, 0, key("o"), W, n);
+}
+
+// What a layer has besides mixer and feed-forward: its token input, its weights of the average over the depth.
+int32_t load_extras(Filler& f, LayeredModel& lm, int i) {
+    const TensorNames& tn = lm.spec.names;
+    LayerP& P = lm.layers[i];
+    const int W = lm.spec.width, n = lm.spec.side_dim;
+    auto side = [&](const std::string& s) { return tn.layer_key(i, tn.side + "." + s); };
+    if (n > 0) {
+        B2_CHECK(f.proj(P.side_gate, n, W));
+        B2_CHECK(f.rows(P.side_gate, 0, side("gate"), n, W));
+        B2_CHECK(f.proj(P.side_proj, W, n));
+        B2_CHECK(f.rows(P.side_proj, 0, side("proj"), W, n));
+        B2_CHECK(f.vec(P.side_norm, side("norm"), {W}, 1.f, 0.f));
+    }
+    if (lm.spec.depth_average) B2_CHECK(f.vec(P.avg, tn.layer_key(i, tn.depth), {i + 2}, 1.f / (i + 2), 0.f));
+    return B2_OK;
+}
+
 int32_t load_layer(Filler& f, LayeredModel& lm, int i) {
     const LayerSpec& L = lm.spec.layers[i];
     const TensorNames& tn = lm.spec.names;
@@ -459,7 +525,10 @@ int32_t load_layer(Filler& f, LayeredModel& lm, int i) {
         B2_CHECK(f.vec(P.hc[q].mix, key(hc + "mix"), {n, n}, 1.f / n, 0.1f / n));
         B2_CHECK(f.vec(P.hc[q].to, key(hc + "out"), {n}, 1.f, 0.2f));
     }
-    if (L.mixer == MixerKind::Memory && L.mem.shift > 0) {
+    B2_CHECK(load_extras(f, lm, i));
+    if (L.mixer == MixerKind::GatedAverage) {
+        B2_CHECK(load_average(f, lm, i));
+    } else if (L.mixer == MixerKind::Memory && L.mem.shift > 0) {
         B2_REQUIRE(!L.parallel, B2_ERR_UNSUPPORTED, "a token shift in a parallel layer");
         B2_CHECK(load_shifted(f, lm, i));
     } else if (L.has_gqa() || L.has_mem()) {
@@ -551,6 +620,7 @@ int32_t load_layer(Filler& f, LayeredModel& lm, int i) {
 // floats of a layer's recurrent record
 int64_t record_floats(const LayerSpec& L) {
     if (L.mixer == MixerKind::Mamba2) return up(L.ssm.inner() * L.ssm.state, 4) + up(L.ssm.channels() * (L.ssm.conv - 1), 4);
+    if (L.mixer == MixerKind::GatedAverage) return up(L.avg.width, 4);
     return L.has_mem() ? up(L.mem.state_floats() + L.mem.channels() * L.mem.keep() + L.mem.shift, 4) : 0;
 }
 
@@ -571,6 +641,7 @@ struct Carver {
 constexpr int kFewTokens = 64;  // up to here the weights' bytes decide: products that read the same rows are merged
 struct Common {
     float *x, *y, *logits;
+    float* past;  // [layers][t][ldx] embedding output and the layers' results, for averages over the depth
     void *xn, *last;
     int ldx, ldn, ldl;
 };
@@ -588,6 +659,13 @@ struct BranchBufs {
     float *low_f;
     float *mq, *mk, *lg, *beta, *o;
     int ld_v;
+};
+struct AverageBufs {
+    void *in, *row;
+};
+struct SideBufs {
+    float* z;
+    void* act;
 };
 struct DenseBufs {
     void *gu, *act;
@@ -609,6 +687,7 @@ Common carve_common(Carver& c, const LayeredModel& lm, size_t es, size_t t, size
     o.ldn = pad_k(lm.spec.width);
     o.ldl = pad_n(lm.spec.vocab);
     o.x = c.take<float>(t * o.ldx * std::max(lm.spec.streams, 1) * 4);
+    o.past = c.take<float>(lm.spec.depth_average ? lm.layers.size() * t * o.ldx * 4 : 0);
     o.y = c.take<float>(t * top * o.ldx * 4);
     o.xn = c.take(t * o.ldn * es);
     o.last = c.take(l * o.ldn * es);
@@ -645,7 +724,7 @@ BranchBufs carve_branches(Carver c, const LayerSpec& L, const LayerP& P, size_t 
     const MemorySpec& s = L.mem;
     o.in = c.take(t * P.in.N * es);
     o.row = c.take(t * P.out.K * es);
-    if (L.has_gqa()) o.q = c.take(t * L.gqa.heads * L.gqa.k_row() * es);
+    if (L.has_gqa()) o.q = c.take(t * L.gqa.q_heads() * L.gqa.k_row() * es);
     if (L.has_mem()) {
         o.lr = c.take(s.shift > 0 && es == 2 ? 0 : t * P.lr.N * es);
         if (s.shift > 0) {
@@ -661,6 +740,20 @@ BranchBufs carve_branches(Carver c, const LayerSpec& L, const LayerP& P, size_t 
         o.beta = c.take<float>(t * s.heads * 4);
         o.o = c.take<float>(t * s.heads * s.vdim * 4);
     }
+    *end = std::max(*end, c.off);
+    return o;
+}
+AverageBufs carve_average(Carver c, const LayerP& P, size_t es, size_t t, size_t* end) {
+    AverageBufs o;
+    o.in = c.take(t * P.in.N * es);
+    o.row = c.take(t * P.out.K * es);
+    *end = std::max(*end, c.off);
+    return o;
+}
+SideBufs carve_side(Carver c, const LayerP& P, size_t es, size_t t, size_t* end) {
+    SideBufs o;
+    o.z = c.take<float>(t * P.side_gate.N * 4);
+    o.act = c.take(t * P.side_proj.K * es);
     *end = std::max(*end, c.off);
     return o;
 }
@@ -705,8 +798,11 @@ size_t arena_bytes(const LayeredModel& lm, size_t es, size_t t, size_t l) {
             carve_latent(c, L.attn, P, es, t, &end);
         else if (L.mixer == MixerKind::Mamba2)
             carve_ssm(c, L.ssm, P, es, t, &end);
+        else if (L.mixer == MixerKind::GatedAverage)
+            carve_average(c, P, es, t, &end);
         else
             carve_branches(c, L, P, es, t, &end);
+        if (lm.spec.side_dim > 0) carve_side(c, P, es, t, &end);
         if (L.mlp == MlpKind::DenseGated) carve_dense(c, P, es, t, &end);
         if (L.mlp == MlpKind::Routed) carve_moe(c, L.moe, P, pad_k(lm.spec.width), es, t, &end);
     }
@@ -797,9 +893,9 @@ DecodeKeys decode_keys(const std::vector<SeqStep>& seqs, const MaskSpec& mask) {
     DecodeKeys k;
     for (auto& s : seqs)
         if (s.n == 1) {
-            const int lo = mask.first(s.cache->len);
-            k.sum += s.cache->len + 1 - lo;
-            k.tiles = std::max(k.tiles, s.cache->len / 16 - lo / 16 + 1);
+            const int pos = s.cache->len, lo = mask.first(pos);
+            k.sum += pos + 1 - lo + mask.kept(pos);
+            k.tiles = std::max(k.tiles, pos / 16 - lo / 16 + 1 + mask.kept_tiles(pos, 16));
         }
     return k;
 }
@@ -807,7 +903,7 @@ double masked_pairs(const LayeredStep& s, const MaskSpec& mask) {  // (query, vi
     if (mask.kind == MaskSpec::None) return s.pf_pairs;
     double n = 0;
     for (auto& q : *s.seqs)
-        for (int i = 0; q.n > 1 && i < q.n; i++) n += q.cache->len + i + 1 - mask.first(q.cache->len + i);
+        for (int i = 0, pos = q.cache->len; q.n > 1 && i < q.n; i++, pos++) n += pos + 1 - mask.first(pos) + mask.kept(pos);
     return n;
 }
 // Latent decode attention: one CTA fills an SM, so the work items (times the head groups) should fill whole rounds of the
@@ -859,6 +955,10 @@ struct Fwd {  // one step
     int32_t attend(const LayerSpec& L, const LayerP& P, const BranchBufs& b, int run);
     int32_t remember(const LayerSpec& L, const LayerP& P, const BranchBufs& b, int run);
     int32_t shift(const LayerSpec& L, const LayerP& P, const BranchBufs& b, int run);
+    int32_t average(const LayerSpec& L, const LayerP& P, int run);
+    int32_t mix(const LayerSpec& L, const LayerP& P, int run);
+    int32_t token_input(const LayerP& P, int layer);
+    int32_t post_norm_layers(float* capture);
     int32_t dense(const LayerSpec& L, const LayerP& P);
     int32_t moe(const LayerSpec& L, const LayerP& P, const int32_t** rows, const float** pass);
 };
@@ -1128,6 +1228,10 @@ int32_t Fwd::attend(const LayerSpec& L, const LayerP& P, const BranchBufs& b, in
     p.context_lens = s.mo->context_lens;
     p.q_rows = lm.t_cap;
     p.out_scale = L.gqa_scale;
+    p.lambda = P.lambda;
+    p.eps = lm.spec.eps;
+    p.gate = (const uint8_t*)b.in + P.at.head_gate * es;
+    p.ld_gate = P.in.N;
     p.out = b.row;
     p.ldo = P.out.K;
     // f32, and head sizes outside the kernels' reach: the plain form.  Otherwise portions of more than a token on their own
@@ -1147,16 +1251,16 @@ int32_t Fwd::attend(const LayerSpec& L, const LayerP& P, const BranchBufs& b, in
         }
         B2_CHECK(ensure_decode(m, items));
         p.part_o = lm.dec_part;
-        p.part_ml = lm.dec_part + (size_t)items * a.heads * a.v_row();
+        p.part_ml = lm.dec_part + (size_t)items * a.q_heads() * a.v_row();
         B2_CHECK(b2_decode_attn_counters(ctx, s.n_dec, b2_gqa_head_blocks(a), &p.counters));
         b2_prof_mark(ctx, B2_CLS_ATTN_DECODE);
         B2_CHECK(b2_gqa_decode_launch(ctx, a, p, items));
-        ctx->attn_decode_bytes += (double)keys.sum * a.kv_heads * (a.dim + a.vdim) * 2;
+        ctx->attn_decode_bytes += (double)keys.sum * a.kv_heads * (a.dim * a.maps + a.vdim) * 2;
     }
     if (s.pf_work > 0) {
         b2_prof_mark(ctx, B2_CLS_ATTN_PREFILL);
         B2_CHECK(b2_gqa_prefill_launch(ctx, a, p, s.pf_work));
-        ctx->attn_prefill_flops += 2.0 * (a.dim + a.vdim) * a.heads * masked_pairs(s, a.mask);
+        ctx->attn_prefill_flops += 2.0 * (a.dim + a.vdim) * a.q_heads() * masked_pairs(s, a.mask);
     }
     return B2_OK;
 }
@@ -1319,9 +1423,146 @@ int32_t Fwd::branches(const LayerSpec& L, const LayerP& P, int run) {
         p.ff = L.ff;
         p.f_off = P.at.f;
     }
-    b2_prof_mark(m->ctx, B2_CLS_ELEMENTWISE);
-    B2_CHECK(b2_branch_out_launch(m->ctx, m->f32, p));
+    if (p.o || p.up || p.att_cols < p.ldo) {
+        b2_prof_mark(m->ctx, B2_CLS_ELEMENTWISE);
+        B2_CHECK(b2_branch_out_launch(m->ctx, m->f32, p));
+    }
     return linear(m, P.out, b.row, P.out.K, s.T, lm.t_cap, c.y, c.ldx, true);
+}
+
+int32_t Fwd::average(const LayerSpec& L, const LayerP& P, int run) {
+    const AverageBufs b = carve_average(scratch, P, es, (size_t)lm.t_cap, &end);
+    B2_CHECK(linear(m, P.in, c.xn, c.ldn, s.T, lm.t_cap, b.in, P.in.N, false));
+    GatedAverageParams p{};
+    p.in = b.in;
+    p.ld = P.in.N;
+    p.z_off = P.at.z;
+    p.u_off = P.at.u;
+    p.g_off = P.at.gate;
+    p.width = L.avg.width;
+    p.z_bias = P.z_bias;
+    p.u_bias = P.u_bias;
+    p.T = s.T;
+    p.B = s.B;
+    p.cu_seqlens = s.mo->cu_seqlens;
+    p.context_lens = s.mo->context_lens;
+    p.seq_slot = s.in->seq_slot;
+    p.state = pool->state + lm.run_state[run];
+    p.slot_stride = pool->state_floats;
+    p.out = b.row;
+    p.ldo = P.out.K;
+    if (s.n_chunks > 0) {
+        B2_CHECK(ensure_chunks(m, (size_t)s.n_chunks * b2_gated_average_chunk_floats(p.width) * 4));
+        p.n_chunks = s.n_chunks;
+        p.chunk_off = s.chunk_off;
+        p.chunk = reinterpret_cast<float*>(lm.chunks);
+    }
+    b2_prof_mark(m->ctx, B2_CLS_RECURRENT);
+    B2_CHECK(b2_gated_average_launch(m->ctx, m->f32, p));
+    return linear(m, P.out, b.row, P.out.K, s.T, lm.t_cap, c.y, c.ldx, true);
+}
+
+int32_t Fwd::mix(const LayerSpec& L, const LayerP& P, int run) {
+    switch (L.mixer) {
+        case MixerKind::LatentAttention: return latent(L, P, run);
+        case MixerKind::Mamba2: return ssm(L, P, run);
+        case MixerKind::GatedAverage: return average(L, P, run);
+        default: return branches(L, P, run);
+    }
+}
+
+int32_t Fwd::token_input(const LayerP& P, int layer) {
+    const SideBufs b = carve_side(scratch, P, es, (size_t)lm.t_cap, &end);
+    B2_CHECK(linear(m, P.side_gate, c.xn, c.ldn, s.T, lm.t_cap, b.z, P.side_gate.N, true));
+    TokenGateParams p{};
+    p.z = b.z;
+    p.ldz = P.side_gate.N;
+    p.table = lm.side.w;
+    p.ld_table = lm.side.K;
+    p.col0 = layer * lm.spec.side_dim;
+    p.vocab = lm.spec.vocab;
+    p.ids = s.ids_dev;
+    p.T = s.T;
+    p.n = lm.spec.side_dim;
+    p.out = b.act;
+    p.ldo = P.side_proj.K;
+    b2_prof_mark(m->ctx, B2_CLS_ELEMENTWISE);
+    B2_CHECK(b2_token_gate_launch(m->ctx, m->f32, p));
+    return linear(m, P.side_proj, b.act, P.side_proj.K, s.T, lm.t_cap, c.y, c.ldx, true);
+}
+
+// Layers whose norms lie behind their sub-layers.  c.xn always holds the stream in storage format; with an average over the depth the
+// embedding output and every layer's result stay in c.past.
+int32_t Fwd::post_norm_layers(float* capture) {
+    b2_ctx* ctx = m->ctx;
+    const ModelSpec& spec = lm.spec;
+    EmbedPairsParams e{};
+    e.table = lm.embed;
+    e.ld_table = c.ldn;
+    e.T = s.T;
+    e.width = spec.width;
+    e.vocab = spec.vocab;
+    e.ids = s.ids_dev;
+    e.scale = spec.embed_scale;
+    e.pairs = spec.pairs;
+    e.pair_table = lm.pairs.w;
+    e.ld_pairs = lm.pairs.K;
+    e.cu_seqlens = s.mo->cu_seqlens;
+    e.context_lens = s.mo->context_lens;
+    e.token_seq = s.mo->token_seq;
+    e.seq_slot = s.in->seq_slot;
+    e.kept = spec.pairs.buckets > 0 ? pool->state + lm.pair_state : nullptr;
+    e.slot_stride = pool->state_floats;
+    e.x = spec.depth_average ? c.past : c.x;
+    e.ldx = c.ldx;
+    e.out = c.xn;
+    e.ldo = c.ldn;
+    b2_prof_mark(ctx, B2_CLS_ELEMENTWISE);
+    B2_CHECK(b2_embed_pairs_launch(ctx, m->f32, e));
+    PostNormParams p{};
+    p.x = e.x;
+    p.x_out = c.x;
+    p.y = c.y;
+    p.eps = spec.eps;
+    p.mult = spec.residual_mult;
+    p.past = c.past;
+    p.past_stride = (int64_t)lm.t_cap * c.ldx;
+    p.out = c.xn;
+    p.ldx = p.ldy = c.ldx;
+    p.ldo = c.ldn;
+    p.rows = s.T;
+    p.width = spec.width;
+    for (size_t i = 0; i < lm.layers.size(); i++) {
+        const LayerSpec& L = spec.layers[i];
+        const LayerP& P = lm.layers[i];
+        auto norm = [&](const float* w, int groups, bool last) {  // last: of the layer
+            p.w = w;
+            p.groups = groups;
+            const bool avg = last && spec.depth_average;
+            p.avg = avg ? P.avg : nullptr;
+            p.depth = (int)i + 1;
+            p.keep = avg && i + 1 < lm.layers.size() ? c.past + (i + 1) * p.past_stride : nullptr;
+            b2_prof_mark(ctx, B2_CLS_ELEMENTWISE);
+            B2_CHECK(b2_post_norm_launch(ctx, m->f32, p));
+            p.x = c.x;
+            return (int32_t)B2_OK;
+        };
+        const bool ff = L.mlp == MlpKind::DenseGated, side = spec.side_dim > 0;
+        B2_CHECK(mix(L, P, (int)i));
+        B2_CHECK(norm(P.norm1, spec.norm_groups, !ff && !side));
+        if (ff) {
+            B2_CHECK(dense(L, P));
+            B2_CHECK(norm(P.norm2, spec.norm_groups, !side));
+        }
+        if (side) {
+            B2_CHECK(token_input(P, (int)i));
+            B2_CHECK(norm(P.side_norm, 1, true));
+        }
+        if (capture)
+            B2_CUDA(cudaMemcpy2DAsync(capture + (int64_t)i * s.T * spec.width, (size_t)spec.width * 4, c.x, (size_t)c.ldx * 4, (size_t)spec.width * 4, (size_t)s.T,
+                                      cudaMemcpyDeviceToHost, ctx->stream));
+    }
+    return B2_OK;
 }
 
 int32_t Fwd::dense(const LayerSpec& L, const LayerP& P) {
@@ -1466,7 +1707,7 @@ void b2_layered_cache_layout(const b2_model* m, int block_size, std::vector<std:
         const LayerSpec& L = m->layered->spec.layers[r.layer];
         page_bytes.emplace_back();
         if (L.has_gqa() && L.kv_from < 0) {
-            page_bytes.back().push_back((size_t)block_size * L.gqa.kv_heads * L.gqa.k_row() * esz(m));
+            page_bytes.back().push_back((size_t)block_size * L.gqa.k_heads() * L.gqa.k_row() * esz(m));
             page_bytes.back().push_back((size_t)block_size * L.gqa.kv_heads * L.gqa.v_row() * esz(m));
         }
         if (L.mixer == MixerKind::LatentAttention) page_bytes.back().push_back((size_t)block_size * L.attn.row_pad() * esz(m));
@@ -1483,11 +1724,21 @@ int32_t b2_layered_ensure_rope(b2_model* m, int positions) {
     for (RopeTab& r : lm.ropes) {
         const int half = r.spec.dims / 2;
         std::vector<float> c((size_t)n * half), s((size_t)n * half);
+        const RotSpec& t = r.spec;
+        const double turned = 2.0 * std::log(t.base), mult = t.factor > 0 ? 0.1 * std::log(t.factor) + 1.0 : 1.0;
+        // the pair (not rounded) that makes this many turns within `original` positions
+        auto pair_of = [&](double turns) { return t.dims * std::log(t.original / (2.0 * M_PI * turns)) / turned; };
+        const double lo = t.factor > 0 ? std::max(std::floor(pair_of(t.fast)), 0.0) : 0.0;
+        const double hi = t.factor > 0 ? std::min(std::ceil(pair_of(t.slow)), t.dims - 1.0) : 0.0;
         for (int i = 0; i < half; i++) {
-            const double f = std::pow(r.spec.base, -2.0 * i / r.spec.dims);
+            double f = std::pow(t.base, -2.0 * i / t.dims);
+            if (t.factor > 0) {
+                const double ramp = std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
+                f = f / t.factor * ramp + f * (1.0 - ramp);
+            }
             for (int p = 0; p < n; p++) {  // rounded once, to f32
-                c[(size_t)p * half + i] = (float)std::cos(p * f);
-                s[(size_t)p * half + i] = (float)std::sin(p * f);
+                c[(size_t)p * half + i] = (float)(std::cos(p * f) * mult);
+                s[(size_t)p * half + i] = (float)(std::sin(p * f) * mult);
             }
         }
         if (r.cos) cudaFree(r.cos);
@@ -1520,9 +1771,17 @@ int32_t b2_model_build_layered(b2_ctx* ctx, const ModelSpec& spec, const b2_weig
     }
     B2_REQUIRE(spec.streams <= kMaxStreams && (spec.streams == 0 || spec.loop.times == 0), B2_ERR_UNSUPPORTED,
                "residual streams: up to 16, without repeated layers");
+    bool plain = spec.streams == 0 && spec.loop.times == 0;
+    for (auto& L : spec.layers) plain = plain && !L.parallel && (L.mlp == MlpKind::None || L.mlp == MlpKind::DenseGated);
+    B2_REQUIRE(plain || (!spec.post_norm && !spec.depth_average && spec.side_dim == 0 && spec.pairs.buckets == 0), B2_ERR_UNSUPPORTED,
+               "norms behind the sub-layers: for sequential layers with dense feed-forwards");
     for (const LayerRun& r : lm.runs) {
         lm.run_state.push_back(lm.state_floats);
         lm.state_floats += record_floats(spec.layers[r.layer]);
+    }
+    if (spec.pairs.buckets > 0) {
+        lm.pair_state = lm.state_floats;
+        lm.state_floats += 4;
     }
     m->cfg.num_layers = (int32_t)spec.layers.size();
     m->cfg.hidden_size = spec.width;
@@ -1541,6 +1800,15 @@ int32_t b2_model_build_layered(b2_ctx* ctx, const ModelSpec& spec, const b2_weig
             B2_CHECK(f.proj(head, spec.vocab, spec.width));
             B2_CHECK(f.rows(head, 0, spec.names.head, spec.vocab, spec.width));
             lm.head = head.w;
+        }
+        if (spec.pairs.buckets > 0) {
+            B2_CHECK(f.proj(lm.pairs, spec.pairs.buckets + 1, spec.width));
+            B2_CHECK(f.rows(lm.pairs, 0, spec.names.pairs, spec.pairs.buckets + 1, spec.width));
+        }
+        if (spec.side_dim > 0) {
+            const int cols = spec.side_dim * (int)spec.layers.size();
+            B2_CHECK(f.proj(lm.side, spec.vocab, cols));
+            B2_CHECK(f.rows(lm.side, 0, spec.names.side + ".embed", spec.vocab, cols));
         }
         if (spec.loop.times > 0) B2_CHECK(f.vec(lm.loop_step, spec.names.loop_step, {spec.loop.times, spec.width}, 0.f, 0.1f));
         for (size_t i = 0; i < spec.layers.size(); i++) B2_CHECK(load_layer(f, lm, (int)i));
@@ -1585,8 +1853,10 @@ int32_t b2_forward_layered(b2_model* m, b2_pool* pool, const LayeredStep& s, flo
     Carver carver{lm.arena};
     const Common c = carve_common(carver, lm, esz(m), (size_t)lm.t_cap, (size_t)lm.l_cap);
     Fwd f{m, lm, pool, s, c, carver, esz(m)};
+    const int64_t per_layer = (int64_t)s.T * spec.width;
+    const bool capture = lm.capture && lm.capture_cap >= per_layer * (int64_t)lm.runs.size();
     b2_prof_mark(ctx, B2_CLS_ELEMENTWISE);
-    B2_CHECK(b2_embed_residual_launch(ctx, m->f32, lm.embed, c.ldn, s.ids_dev, s.T, spec.width, spec.vocab, c.x, c.ldx, std::max(spec.streams, 1)));
+    if (!spec.post_norm) B2_CHECK(b2_embed_residual_launch(ctx, m->f32, lm.embed, c.ldn, s.ids_dev, s.T, spec.width, spec.vocab, c.x, c.ldx, std::max(spec.streams, 1)));
     AddNormParams an{};
     an.x = c.x;
     an.y = c.y;
@@ -1594,6 +1864,7 @@ int32_t b2_forward_layered(b2_model* m, b2_pool* pool, const LayeredStep& s, flo
     an.width = spec.width;
     an.eps = spec.eps;
     an.n_src = 0;  // nothing is pending behind the embedding
+    an.groups = spec.norm_groups;
     StreamNormParams sn{};
     sn.x = c.x;
     sn.streams = spec.streams;
@@ -1634,11 +1905,10 @@ int32_t b2_forward_layered(b2_model* m, b2_pool* pool, const LayeredStep& s, flo
         sn.to = P ? P->hc[q].to : nullptr;
         sn.pass = pass;
     };
-    const int64_t per_layer = (int64_t)s.T * spec.width;
-    const bool capture = lm.capture && lm.capture_cap >= per_layer * (int64_t)lm.runs.size();
     float* sums = nullptr;  // of the streams
     if (capture && spec.streams > 0) B2_CUDA(cudaMallocAsync((void**)&sums, (size_t)s.T * c.ldx * 4, ctx->stream));
-    for (size_t r = 0; r < lm.runs.size(); r++) {
+    if (spec.post_norm) B2_CHECK(f.post_norm_layers(capture ? lm.capture : nullptr));
+    for (size_t r = 0; r < lm.runs.size() && !spec.post_norm; r++) {
         const LayerRun& run = lm.runs[r];
         const LayerSpec& L = spec.layers[run.layer];
         const LayerP& P = lm.layers[run.layer];
@@ -1654,7 +1924,7 @@ int32_t b2_forward_layered(b2_model* m, b2_pool* pool, const LayeredStep& s, flo
         B2_CHECK(norm(P.norm1, P.hc[0].from, s.T, nullptr, c.xn, 1.f, true));
         an.vec = nullptr;
         an.table = nullptr;
-        B2_CHECK(L.mixer == MixerKind::LatentAttention ? f.latent(L, P, (int)r) : L.mixer == MixerKind::Mamba2 ? f.ssm(L, P, (int)r) : f.branches(L, P, (int)r));
+        B2_CHECK(f.mix(L, P, (int)r));
         pending(&P, 0, nullptr, 1);
         if (L.mlp != MlpKind::None && !L.parallel) {
             B2_CHECK(norm(P.norm2, P.hc[1].from, s.T, nullptr, c.xn, 1.f, true));

@@ -1,5 +1,6 @@
 // Grouped-query attention of the layered models: projections to rotated queries and cache rows, and the plain form of the
-// attention.  Scores may be capped, the softmax may have a sink (exp(0) in its denominator, with no value).
+// attention.  Scores may be capped, the softmax may have a sink (exp(0) in its denominator, with no value), two maps may be taken
+// off one another (differential attention).
 #include <type_traits>
 
 #include "elt.cuh"
@@ -9,9 +10,9 @@ namespace {
 
 constexpr int kMaxHead = 256;
 
-// A warp per (token, head of q, k or v): bias, norm over the head, rotation of the pairs (i, i + dims/2), store.  A lane holds
-// VEC consecutive values of every 32 * VEC; the rotation finds its partner in shared memory
-// (N 1, VEC 4: heads of up to 128, the partner comes by shuffle).  With a norm over all heads (ALL) a block takes eight heads of
+// A warp per (token, head of q, k or v; with two maps, per map): bias, norm over the head, rotation of the pairs (i, i + dims/2) or
+// (2i, 2i + 1), store.  A lane holds VEC consecutive values of every 32 * VEC; the rotation finds its partner in shared memory
+// (N 1, VEC 4: heads of up to 128, the partner comes by shuffle; neighbours with VEC 4: the lane has both).  With a norm over all heads (ALL) a block takes eight heads of
 // one token, and first the sums of squares of all its queries and of all its keys.
 template <typename T, int VEC, int N, bool ALL>
 __global__ void __launch_bounds__(256) gqa_prep_kernel(const GroupedAttnSpec a, const GqaPrepParams p) {
@@ -19,7 +20,7 @@ __global__ void __launch_bounds__(256) gqa_prep_kernel(const GroupedAttnSpec a, 
     pdl_wait();
     constexpr bool SHUFFLE = N == 1 && VEC == 4;
     __shared__ __align__(16) float rows[SHUFFLE ? 1 : 8][SHUFFLE ? 4 : kMaxHead];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, units = a.heads + (p.own_kv ? 2 * a.kv_heads : 0);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, QH = a.q_heads(), KH = a.k_heads(), units = QH + (p.own_kv ? KH + a.kv_heads : 0);
     const int id = blockIdx.x * 8 + warp, t = ALL ? blockIdx.y : id / units, u = ALL ? id : id - t * units;
     float all_inv[2] = {1.f, 1.f};
     if constexpr (ALL) {  // (every thread of the block: u0 the block's first unit)
@@ -51,7 +52,7 @@ __global__ void __launch_bounds__(256) gqa_prep_kernel(const GroupedAttnSpec a, 
         if (u >= units) return;
     }
     if (t >= p.T) return;
-    const int kind = u < a.heads ? 0 : u < a.heads + a.kv_heads ? 1 : 2, h = kind == 0 ? u : kind == 1 ? u - a.heads : u - a.heads - a.kv_heads;
+    const int kind = u < QH ? 0 : u < QH + KH ? 1 : 2, h = kind == 0 ? u : kind == 1 ? u - QH : u - QH - KH;
     const int n = kind == 2 ? a.vdim : a.dim, padded = kind == 2 ? a.v_row() : a.k_row(), dims = kind == 2 ? 0 : a.rot.dims, half = dims / 2;
     const T* src = reinterpret_cast<const T*>(p.in) + (size_t)t * p.ld + (kind == 0 ? p.q_off : kind == 1 ? p.k_off : p.v_off) + h * n;
     const float* bias = kind == 0 ? p.q_bias : kind == 1 ? p.k_bias : p.v_bias;
@@ -60,10 +61,10 @@ __global__ void __launch_bounds__(256) gqa_prep_kernel(const GroupedAttnSpec a, 
     const int slot = p.slot_mapping[t];
     T* dst;
     if (kind == 0) {
-        dst = reinterpret_cast<T*>(p.q) + ((size_t)t * a.heads + h) * padded;
+        dst = reinterpret_cast<T*>(p.q) + ((size_t)t * QH + h) * padded;
     } else {
         if (slot < 0) return;
-        const size_t row = ((size_t)(slot / p.page_size) * a.kv_heads + h) * p.page_size + slot % p.page_size;
+        const size_t row = ((size_t)(slot / p.page_size) * (kind == 1 ? KH : a.kv_heads) + h) * p.page_size + slot % p.page_size;
         dst = reinterpret_cast<T*>(kind == 1 ? p.k_cache : p.v_cache) + row * padded;
     }
     float v[N][VEC], ss = 0.f;
@@ -100,7 +101,21 @@ __global__ void __launch_bounds__(256) gqa_prep_kernel(const GroupedAttnSpec a, 
                 if (d < n) v[i][e] = v[i][e] * inv * w[d];
             }
     }
-    if constexpr (SHUFFLE) {
+    if (VEC == 4 && a.neighbours) {
+        const float* ct = p.cos_t + (size_t)p.positions[t] * half;
+        const float* st = p.sin_t + (size_t)p.positions[t] * half;
+#pragma unroll
+        for (int i = 0; i < N; i++)
+#pragma unroll
+            for (int e = 0; e < VEC - 1; e += 2) {
+                const int d = (i * 32 + lane) * VEC + e;
+                if (d < dims) {
+                    const float c = ct[d / 2], s = st[d / 2], x = v[i][e], y = v[i][e + 1];
+                    v[i][e] = x * c - y * s;
+                    v[i][e + 1] = y * c + x * s;
+                }
+            }
+    } else if constexpr (SHUFFLE) {
         if (half > 0) {  // (half is a multiple of four)
             const int d = lane * 4, src_lane = d < half ? lane + half / 4 : lane - half / 4;
             float o[4], c[4] = {1.f, 1.f, 1.f, 1.f}, sn[4] = {0.f, 0.f, 0.f, 0.f};
@@ -127,7 +142,9 @@ __global__ void __launch_bounds__(256) gqa_prep_kernel(const GroupedAttnSpec a, 
 #pragma unroll
             for (int e = 0; e < VEC; e++) {
                 const int d = (i * 32 + lane) * VEC + e;
-                if (d < half)
+                if (a.neighbours) {
+                    if (d < dims) v[i][e] = v[i][e] * ct[d / 2] + (d % 2 ? rows[warp][d - 1] : -rows[warp][d + 1]) * st[d / 2];
+                } else if (d < half)
                     v[i][e] = v[i][e] * ct[d] - rows[warp][d + half] * st[d];
                 else if (d < dims)
                     v[i][e] = v[i][e] * ct[d - half] + rows[warp][d - half] * st[d - half];
@@ -144,52 +161,72 @@ __global__ void __launch_bounds__(256) gqa_prep_kernel(const GroupedAttnSpec a, 
     }
 }
 
-// Plain form: one block per (token, head), 128 keys at a time with an online softmax, everything f32.
+// Plain form: one block per (token, head), one map after the other, 128 keys at a time with an online softmax, everything f32.
 template <typename T>
 __global__ void __launch_bounds__(128) gqa_simple_kernel(const GroupedAttnSpec a, const GqaAttnParams p) {
     pdl_wait();
-    __shared__ float q[kMaxHead], acc[kMaxHead], pr[128], red[33];
+    __shared__ float q[kMaxHead], accs[2][kMaxHead], pr[128], red[33];
     const int t = blockIdx.x, h = blockIdx.y, g = h / a.group(), KR = a.k_row(), VR = a.v_row(), ps = p.page_size;
-    const int n = p.positions[t] + 1, lo = a.mask.first(p.positions[t]);
+    const int n = p.positions[t] + 1, lo = a.mask.first(p.positions[t]), kept = a.mask.kept(p.positions[t]), seen = kept + n - lo;
     const int32_t* bt = p.block_tables + (size_t)p.seq_slot[p.token_seq[t]] * p.max_blocks;
-    const T* qr = reinterpret_cast<const T*>(p.q) + ((size_t)t * a.heads + h) * KR;
-    auto row = [&](int j) { return ((size_t)bt[j / ps] * a.kv_heads + g) * ps + j % ps; };
-    for (int i = threadIdx.x; i < KR; i += 128) q[i] = Elt<T>::ld(qr + i);
-    for (int i = threadIdx.x; i < VR; i += 128) acc[i] = 0.f;
-    float m = -INFINITY, l = 0.f;
-    __syncthreads();
-    for (int j0 = lo; j0 < n; j0 += 128) {
-        const int j = j0 + threadIdx.x, cnt = min(128, n - j0);
-        float s = -INFINITY;
-        if (j < n) {
-            const T* k = reinterpret_cast<const T*>(p.k_cache) + row(j) * KR;
-            float d = 0.f;
-            for (int i = 0; i < KR; i += 8) {
-                float v[8];
-                Elt<T>::ld8(k + i, v);
+    auto key = [&](int i) { return i < kept ? i : i - kept + lo; };  // the i-th visible one
+    auto row = [&](int j, int heads, int hd) { return ((size_t)bt[j / ps] * heads + hd) * ps + j % ps; };
+    float l = 0.f;
+    for (int mp = 0; mp < a.maps; mp++) {
+        float* acc = accs[mp];
+        const T* qr = reinterpret_cast<const T*>(p.q) + ((size_t)t * a.q_heads() + h * a.maps + mp) * KR;
+        for (int i = threadIdx.x; i < KR; i += 128) q[i] = Elt<T>::ld(qr + i);
+        for (int i = threadIdx.x; i < VR; i += 128) acc[i] = 0.f;
+        float m = -INFINITY;
+        l = 0.f;
+        __syncthreads();
+        for (int j0 = 0; j0 < seen; j0 += 128) {
+            const int j = j0 + threadIdx.x, cnt = min(128, seen - j0);
+            float s = -INFINITY;
+            if (j < seen) {
+                const T* k = reinterpret_cast<const T*>(p.k_cache) + row(key(j), a.k_heads(), g * a.maps + mp) * KR;
+                float d = 0.f;
+                for (int i = 0; i < KR; i += 8) {
+                    float v[8];
+                    Elt<T>::ld8(k + i, v);
 #pragma unroll
-                for (int e = 0; e < 8; e++) d = fmaf(q[i + e], v[e], d);
+                    for (int e = 0; e < 8; e++) d = fmaf(q[i + e], v[e], d);
+                }
+                s = d * a.scale;
+                if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
             }
-            s = d * a.scale;
-            if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
+            float mx = elt_warp_max(s);
+            __syncthreads();
+            if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = mx;
+            __syncthreads();
+            mx = fmaxf(fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3])), m);
+            const float alpha = expf(m - mx), e = j < seen ? expf(s - mx) : 0.f;
+            pr[threadIdx.x] = e;
+            l = l * alpha + elt_block_sum(e, red);
+            m = mx;
+            for (int i = threadIdx.x; i < VR; i += 128) {
+                float v = acc[i] * alpha;
+                for (int jj = 0; jj < cnt; jj++) v = fmaf(pr[jj], Elt<T>::ld(reinterpret_cast<const T*>(p.v_cache) + row(key(j0 + jj), a.kv_heads, g) * VR + i), v);
+                acc[i] = v;
+            }
+            __syncthreads();
         }
-        float mx = elt_warp_max(s);
-        __syncthreads();
-        if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = mx;
-        __syncthreads();
-        mx = fmaxf(fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3])), m);
-        const float alpha = expf(m - mx), e = j < n ? expf(s - mx) : 0.f;
-        pr[threadIdx.x] = e;
-        l = l * alpha + elt_block_sum(e, red);
-        m = mx;
-        for (int i = threadIdx.x; i < VR; i += 128) {
-            float v = acc[i] * alpha;
-            for (int jj = 0; jj < cnt; jj++) v = fmaf(pr[jj], Elt<T>::ld(reinterpret_cast<const T*>(p.v_cache) + row(j0 + jj) * VR + i), v);
-            acc[i] = v;
+        if (a.sink) l += expf(-m);
+        if (a.maps == 2) {  // (a thread's own values)
+            for (int i = threadIdx.x; i < a.vdim; i += 128) acc[i] /= l;
+            l = 1.f;
         }
-        __syncthreads();
     }
-    if (a.sink) l += expf(-m);
+    float* acc = accs[0];
+    if (a.maps == 2) {
+        float ss = 0.f;
+        for (int i = threadIdx.x; i < a.vdim; i += 128) {
+            acc[i] -= p.lambda * accs[1][i];
+            ss += acc[i] * acc[i];
+        }
+        l = sqrtf(elt_block_sum(ss, red) / (float)a.vdim + p.eps) / (1.f - a.diff);
+    }
+    if (a.head_gate) l /= sigmoid_f32(Elt<T>::ld(reinterpret_cast<const T*>(p.gate) + (size_t)t * p.ld_gate + h));
     T* o = reinterpret_cast<T*>(p.out) + (size_t)t * p.ldo + h * a.vdim;
     for (int i = threadIdx.x; i < a.vdim; i += 128) Elt<T>::st(o + i, acc[i] / l * p.out_scale);
 }
@@ -200,8 +237,8 @@ int32_t b2_gqa_prep_launch(b2_ctx* ctx, bool f32, const GroupedAttnSpec& a, cons
     if (p.T <= 0) return B2_OK;
     B2_REQUIRE(a.dim <= kMaxHead && a.vdim <= kMaxHead, B2_ERR_UNSUPPORTED, "grouped attention: head sizes up to 256");
     const bool vec = a.dim % 4 == 0 && a.vdim % 4 == 0 && p.q_off % 4 == 0 && p.k_off % 4 == 0 && p.v_off % 4 == 0 && p.ld % 4 == 0;
-    const int units = a.heads + (p.own_kv ? 2 * a.kv_heads : 0);
-    const bool small = a.dim <= 128 && a.vdim <= 128 && a.rot.dims % 8 == 0;
+    const int units = a.q_heads() + (p.own_kv ? a.k_heads() + a.kv_heads : 0);
+    const bool small = a.dim <= 128 && a.vdim <= 128 && (a.neighbours || a.rot.dims % 8 == 0);
     auto pick = [&](auto all) {
         constexpr bool ALL = decltype(all)::value;
         return !vec    ? (f32 ? gqa_prep_kernel<float, 1, 8, ALL> : gqa_prep_kernel<uint16_t, 1, 8, ALL>)

@@ -1,11 +1,13 @@
 // Grouped-query attention of the layered models, one query token per row, over the paged cache in place (bf16).
 //
 // Byte streaming like the flat decoders' kernel (paged_attn_decode.cu), for key and value heads of any size up to 256 (in
-// 16-wide steps), any number of query heads per key head (blocks of eight), capped scores and a sink:
-//   CTA   (chunk of one row's keys, up to eight query heads of one key head)
+// 16-wide steps), any number of query heads per key head (blocks of eight), capped scores and a sink; with two maps (differential
+// attention) a head's two queries are two of the eight columns, each of which meets its own map's keys:
+//   CTA   (chunk of one row's keys, up to eight query heads of one key / value head)
 //   warp  every 4th tile of 16 keys, its own three-stage cp.async ring, no CTA-wide barrier in the loop
 //   mma   S^T = K Q^T with the keys on M and the heads on N, then O^T += V^T P^T; P enters as bf16 head and remainder
-// Under a mask the chunks start at the tile of the row's first visible key, and every row has the same number of work items.
+// Under a mask the tiles are those of the kept first keys, then those from the tile of the row's first visible key on, and every row
+// has the same number of work items.
 // Warps are merged in shared memory; the CTA of a (row, head block) that finishes last adds the chunks up, in chunk order.
 #include "elt.cuh"
 #include "layer_kernels.h"
@@ -15,6 +17,11 @@ namespace {
 constexpr int kWarps = 4, kStages = 3, kHeads = 8, kMergeBatch = 256;
 constexpr unsigned kFull = 0xffffffffu;
 constexpr float kLog2e = 1.4426950408889634f;
+// floats of shared memory that merging the warps, and then the chunks, takes
+constexpr int fin_floats(int v_row) {
+    const int merge = kWarps * v_row * 8 + 2 * kWarps * 8, chunks = 2 * kMergeBatch * 8 + 16;
+    return merge > chunks ? merge : chunks;
+}
 
 // Score in units of log2: scale * s, capped as c tanh(scale * s / c) with tanh(z) = 1 - 2 / (1 + e^(2z)), whose absolute
 // error (which is what a score's error counts by) stays at a few units of f32.
@@ -29,15 +36,16 @@ struct ScoreMap {
     __device__ __forceinline__ float operator()(float s) const { return cap ? c - __fdividef(2.f * c, 1.f + fast_exp2(fminf(s * a, 126.f))) : s * a; }
 };
 
-// NB: 16-wide steps of the larger of the two head sizes, rounded up; EXACT: both heads have exactly that many.
-template <int NB, bool EXACT>
+// NB: 16-wide steps of the larger of the two rows (keys of all maps side by side, values), rounded up; EXACT: both have exactly that many.
+template <int NB, bool EXACT, int MAPS>
 __global__ void __launch_bounds__(kWarps * 32) gqa_decode_kernel(const GroupedAttnSpec a, const GqaAttnParams p, bool listed) {
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     extern __shared__ __align__(128) uint8_t smem[];
     __shared__ int s_last;
     pdl_wait();
-    const int item = blockIdx.x, group = a.group(), subs = (group + kHeads - 1) / kHeads, kvh = blockIdx.y / subs, h0 = kvh * group + (blockIdx.y % subs) * kHeads;
-    const int heads = min(kHeads, kvh * group + group - h0), KR = EXACT ? NB * 16 : a.k_row(), VR = EXACT ? NB * 16 : a.v_row();
+    const int item = blockIdx.x, group = a.group() * MAPS, subs = (group + kHeads - 1) / kHeads, kvh = blockIdx.y / subs, h0 = kvh * group + (blockIdx.y % subs) * kHeads;
+    const int QH = a.heads * MAPS, heads = min(kHeads, kvh * group + group - h0);  // heads from here on: queries, one per map
+    const int MR = EXACT ? NB * 16 / MAPS : a.k_row(), KR = MR * MAPS, VR = EXACT ? NB * 16 : a.v_row();
     int row, chunk = 0, w0 = item, ctx, qrow, slot;  // entry of the list, its chunk, first work item of the row
     if (listed) {
         if (p.row_chunks > 0) {
@@ -58,10 +66,11 @@ __global__ void __launch_bounds__(kWarps * 32) gqa_decode_kernel(const GroupedAt
         ctx = p.positions[row] + 1;
         slot = p.seq_slot[p.token_seq[row]];
     }
-    const int lo = a.mask.first(ctx - 1), tile_lo = lo / 16;  // first visible key, its tile
-    const int tiles_total = (ctx + 15) / 16 - tile_lo, chunk_tiles = listed ? p.chunk_tiles : tiles_total, n_chunks = (tiles_total + chunk_tiles - 1) / chunk_tiles;
+    const int lo = a.mask.first(ctx - 1), tile_lo = lo / 16, keep = a.mask.keep, kept = a.mask.kept_tiles(ctx - 1, 16);  // first visible key, its tile
+    const int tiles_total = (ctx + 15) / 16 - tile_lo + kept, chunk_tiles = listed ? p.chunk_tiles : tiles_total, n_chunks = (tiles_total + chunk_tiles - 1) / chunk_tiles;
     if (chunk >= n_chunks) return;
-    const int tile0 = tile_lo + chunk * chunk_tiles, n_tiles = min(chunk_tiles, tiles_total - chunk * chunk_tiles);
+    const int tile0 = chunk * chunk_tiles, n_tiles = min(chunk_tiles, tiles_total - tile0);
+    auto first_key = [&](int i) { return (i < kept ? i : i - kept + tile_lo) * 16; };  // of the row's i-th tile
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
     const int kd = KR / 16, vd = VR / 16;                              // 16-wide steps
     const int krow = (KR + 63) / 64 * 128, vrow = (VR + 63) / 64 * 128;  // bytes per row in shared memory, whole swizzle groups
@@ -71,40 +80,42 @@ __global__ void __launch_bounds__(kWarps * 32) gqa_decode_kernel(const GroupedAt
     // Q^T as the B operand: thread (g, t) holds Q[head g][16 k + 2t, +1] and [.. + 8, + 9]
     uint32_t qf[NB][2];
     {
-        const uint16_t* qh = reinterpret_cast<const uint16_t*>(p.q) + ((size_t)qrow * a.heads + h0 + min(g, heads - 1)) * KR;
+        const uint16_t* qh = reinterpret_cast<const uint16_t*>(p.q) + ((size_t)qrow * QH + h0 + min(g, heads - 1)) * MR;
 #pragma unroll
         for (int k = 0; k < NB; k++) {
-            const bool ok = g < heads && k < kd;
-            qf[k][0] = ok ? *reinterpret_cast<const uint32_t*>(qh + k * 16 + 2 * t) : 0u;
-            qf[k][1] = ok ? *reinterpret_cast<const uint32_t*>(qh + k * 16 + 2 * t + 8) : 0u;
+            const int map0 = MAPS == 2 && (g & 1) ? MR / 16 : 0;  // its map's first step
+            const bool ok = g < heads && k >= map0 && k < map0 + MR / 16;
+            qf[k][0] = ok ? *reinterpret_cast<const uint32_t*>(qh + (k - map0) * 16 + 2 * t) : 0u;
+            qf[k][1] = ok ? *reinterpret_cast<const uint32_t*>(qh + (k - map0) * 16 + 2 * t + 8) : 0u;
         }
     }
     const int n_my = n_tiles > warp ? (n_tiles - warp + kWarps - 1) / kWarps : 0;
     const int32_t* bt = p.block_tables + (size_t)slot * p.max_blocks;
     const uint32_t wsm = smem_u32(smem) + warp * (kStages * stage);
-    auto page_row = [&](int i) {  // cache row of this warp's i-th tile; past the end: the last tile's
-        const int key = (tile0 + warp + min(i, max(n_my - 1, 0)) * kWarps) * 16, k = key < ctx ? key : 0;
-        return ((size_t)bt[k / p.page_size] * a.kv_heads + kvh) * p.page_size + k % p.page_size;
+    auto page_row = [&](int i) {  // cache row of this warp's i-th tile (page * page_size + offset) of one head; past the end: the last tile's
+        const int key = first_key(tile0 + warp + min(i, max(n_my - 1, 0)) * kWarps), k = key < ctx ? key : 0;
+        return make_int2(bt[k / p.page_size], k % p.page_size);
     };
-    const int kr0 = lane / (KR / 8), kx0 = lane - kr0 * (KR / 8), vr0 = lane / (VR / 8), vx0 = lane - vr0 * (VR / 8);
-    size_t next = page_row(0);  // looked up one tile ahead
+    const int kr0 = lane / (MR / 8), kx0 = lane - kr0 * (MR / 8), vr0 = lane / (VR / 8), vx0 = lane - vr0 * (VR / 8);
+    int2 next = page_row(0);  // looked up one tile ahead
     auto issue = [&](int i) {
-        const size_t r0 = next;
+        const int2 at = next;
         next = page_row(i + 1);
         const uint32_t dst = wsm + (i % kStages) * stage;
-        const uint8_t* ks = reinterpret_cast<const uint8_t*>(p.k_cache) + r0 * KR * 2;
-        const uint8_t* vs = reinterpret_cast<const uint8_t*>(p.v_cache) + r0 * VR * 2;
-        auto copy = [&](uint32_t to, int row_bytes, const uint8_t* from, int pieces, int r, int x) {  // 16-byte pieces of 16 rows
+        const uint8_t* ks = reinterpret_cast<const uint8_t*>(p.k_cache) + (((size_t)at.x * a.kv_heads + kvh) * MAPS * p.page_size + at.y) * MR * 2;
+        const uint8_t* vs = reinterpret_cast<const uint8_t*>(p.v_cache) + (((size_t)at.x * a.kv_heads + kvh) * p.page_size + at.y) * VR * 2;
+        auto copy = [&](uint32_t to, int row_bytes, int x0, const uint8_t* from, int pieces, int r, int x) {  // 16-byte pieces of 16 rows, from piece x0 on
             const int dr = 32 / pieces, dx = 32 - dr * pieces;
             for (int c = lane; c < 16 * pieces; c += 32) {
-                cp_async16(to + r * row_bytes + ((x ^ (r & 7)) << 4), from + (size_t)c * 16);
+                cp_async16(to + r * row_bytes + (((x0 + x) ^ (r & 7)) << 4), from + (size_t)c * 16);
                 r += dr;
                 x += dx;
                 if (x >= pieces) x -= pieces, r++;
             }
         };
-        copy(dst, krow, ks, KR / 8, kr0, kx0);
-        copy(dst + 16 * krow, vrow, vs, VR / 8, vr0, vx0);
+#pragma unroll
+        for (int m = 0; m < MAPS; m++) copy(dst, krow, m * (MR / 8), ks + (size_t)m * p.page_size * MR * 2, MR / 8, kr0, kx0);
+        copy(dst + 16 * krow, vrow, 0, vs, VR / 8, vr0, vx0);
     };
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f, o[NB][4];
 #pragma unroll
@@ -132,16 +143,16 @@ __global__ void __launch_bounds__(kWarps * 32) gqa_decode_kernel(const GroupedAt
                     mma_bf16_16816(s, f, qf[k]);
                 }
         }
-        const int key0 = (tile0 + warp + i * kWarps) * 16;
+        const int key0 = first_key(tile0 + warp + i * kWarps);
 #pragma unroll
         for (int j = 0; j < 4; j++) s[j] = map(s[j]);
         if (key0 + 16 > ctx) {
             if (key0 + g >= ctx) s[0] = s[1] = -INFINITY;
             if (key0 + g + 8 >= ctx) s[2] = s[3] = -INFINITY;
         }
-        if (key0 < lo) {  // (the tile holds lo: something stays visible)
-            if (key0 + g < lo) s[0] = s[1] = -INFINITY;
-            if (key0 + g + 8 < lo) s[2] = s[3] = -INFINITY;
+        if (key0 < lo) {  // (the tile holds lo or a kept key: something stays visible)
+            if (key0 + g < lo && key0 + g >= keep) s[0] = s[1] = -INFINITY;
+            if (key0 + g + 8 < lo && key0 + g + 8 >= keep) s[2] = s[3] = -INFINITY;
         }
         float mx0 = fmaxf(s[0], s[2]), mx1 = fmaxf(s[1], s[3]);
 #pragma unroll
@@ -205,7 +216,23 @@ __global__ void __launch_bounds__(kWarps * 32) gqa_decode_kernel(const GroupedAt
         sm_l[warp * 8 + 2 * t + 1] = l1;
     }
     __syncthreads();
-    uint16_t* out = reinterpret_cast<uint16_t*>(p.out) + (size_t)qrow * p.ldo + h0 * a.vdim;
+    uint16_t* out = reinterpret_cast<uint16_t*>(p.out) + (size_t)qrow * p.ldo + h0 / MAPS * a.vdim;
+    float* fin = reinterpret_cast<float*>(smem) + fin_floats(VR);  // [8][VR] two maps: their results
+    // a head's output from its two maps: difference, norm, gate; a warp per head
+    auto finish = [&]() {
+        __syncthreads();
+        for (int h = warp; h < heads / 2; h += kWarps) {
+            const float *a1 = fin + 2 * h * VR, *a2 = a1 + VR;
+            float ss = 0.f;
+            for (int d = lane; d < a.vdim; d += 32) {
+                const float v = a1[d] - p.lambda * a2[d];
+                ss += v * v;
+            }
+            float f = (1.f - a.diff) / sqrtf(elt_warp_sum(ss) / (float)a.vdim + p.eps) * p.out_scale;
+            if (a.head_gate) f *= sigmoid_f32(bf2f(reinterpret_cast<const uint16_t*>(p.gate)[(size_t)qrow * p.ld_gate + h0 / 2 + h]));
+            for (int d = lane; d < a.vdim; d += 32) out[h * a.vdim + d] = f2bf((a1[d] - p.lambda * a2[d]) * f);
+        }
+    };
     for (int e = threadIdx.x; e < heads * VR; e += kWarps * 32) {
         const int h = e / VR, d = e - h * VR;
         float M = -INFINITY, L = 0.f, O = 0.f;
@@ -219,14 +246,20 @@ __global__ void __launch_bounds__(kWarps * 32) gqa_decode_kernel(const GroupedAt
         }
         if (n_chunks == 1) {
             if (a.sink) L += fast_exp2(-M);
-            if (d < a.vdim) out[h * a.vdim + d] = f2bf(O / L * p.out_scale);
+            if constexpr (MAPS == 2)
+                fin[e] = O / L;
+            else if (d < a.vdim)
+                out[h * a.vdim + d] = f2bf(O / L * p.out_scale);
         } else {
-            const size_t at = (size_t)item * a.heads + h0 + h;
+            const size_t at = (size_t)item * QH + h0 + h;
             p.part_o[at * VR + d] = O;
             if (d == 0) *reinterpret_cast<float2*>(p.part_ml + at * 2) = make_float2(M, L);
         }
     }
-    if (n_chunks == 1) return;
+    if (n_chunks == 1) {
+        if constexpr (MAPS == 2) finish();
+        return;
+    }
     // No CTA waits for another; the counter returns to zero for the next launch.
     __threadfence();
     __syncthreads();
@@ -243,7 +276,7 @@ __global__ void __launch_bounds__(kWarps * 32) gqa_decode_kernel(const GroupedAt
     float* l_c = f_c + kMergeBatch * 8;           // [kMergeBatch][8]
     float* s_M = l_c + kMergeBatch * 8;           // [8]
     float* s_L = s_M + 8;                         // [8]
-    auto ml = [&](int c, int h) { return __ldcg(reinterpret_cast<const float2*>(p.part_ml + ((size_t)(w0 + c) * a.heads + h0 + h) * 2)); };
+    auto ml = [&](int c, int h) { return __ldcg(reinterpret_cast<const float2*>(p.part_ml + ((size_t)(w0 + c) * QH + h0 + h) * 2)); };
     if (threadIdx.x < 32) {  // four lanes per head
         const int h = threadIdx.x >> 2;
         float M = -INFINITY;
@@ -281,10 +314,10 @@ __global__ void __launch_bounds__(kWarps * 32) gqa_decode_kernel(const GroupedAt
                 const int e = threadIdx.x + k * kWarps * 32;
                 if (e >= heads * VR) break;
                 const int h = e / VR;
-                const float* src = p.part_o + ((size_t)(w0 + c0 + c) * a.heads + h0) * VR + e;
+                const float* src = p.part_o + ((size_t)(w0 + c0 + c) * QH + h0) * VR + e;
                 float v[8];
 #pragma unroll
-                for (int j = 0; j < 8; j++) v[j] = c + j < nb ? __ldcg(src + (size_t)j * a.heads * VR) : 0.f;
+                for (int j = 0; j < 8; j++) v[j] = c + j < nb ? __ldcg(src + (size_t)j * QH * VR) : 0.f;
 #pragma unroll
                 for (int j = 0; j < 8; j++)
                     if (c + j < nb) acc[k] = fmaf(v[j], f_c[(c + j) * 8 + h], acc[k]);
@@ -297,32 +330,41 @@ __global__ void __launch_bounds__(kWarps * 32) gqa_decode_kernel(const GroupedAt
         const int e = threadIdx.x + k * kWarps * 32;
         if (e >= heads * VR) break;
         const int h = e / VR, d = e - h * VR;
-        if (d < a.vdim) out[h * a.vdim + d] = f2bf(acc[k] / s_L[h] * p.out_scale);
+        if constexpr (MAPS == 2)
+            fin[e] = acc[k] / s_L[h];
+        else if (d < a.vdim)
+            out[h * a.vdim + d] = f2bf(acc[k] / s_L[h] * p.out_scale);
     }
+    if constexpr (MAPS == 2) finish();
 }
 
 int smem_bytes(const GroupedAttnSpec& a) {
-    const int krow = (a.k_row() + 63) / 64 * 128, vrow = (a.v_row() + 63) / 64 * 128;
-    const int ring = kWarps * kStages * 16 * (krow + vrow), merge = (kWarps * a.v_row() * 8 + 2 * kWarps * 8) * 4, chunks = (2 * kMergeBatch * 8 + 16) * 4;
-    return ring > merge ? (ring > chunks ? ring : chunks) : (merge > chunks ? merge : chunks);
+    const int krow = (a.k_row() * a.maps + 63) / 64 * 128, vrow = (a.v_row() + 63) / 64 * 128;
+    const int ring = kWarps * kStages * 16 * (krow + vrow), rest = (fin_floats(a.v_row()) + (a.maps == 2 ? 8 * a.v_row() : 0)) * 4;
+    return ring > rest ? ring : rest;
 }
-template <int NB, bool EXACT>
+template <int NB, bool EXACT, int MAPS = 1>
 int32_t launch(b2_ctx* ctx, const GroupedAttnSpec& a, const GqaAttnParams& p, int items) {
-    B2_SMEM_ONCE(ctx, (gqa_decode_kernel<NB, EXACT>), kWarps * kStages * 16 * 2 * 512);
+    B2_SMEM_ONCE(ctx, (gqa_decode_kernel<NB, EXACT, MAPS>), kWarps * kStages * 16 * 2 * 512);
     const dim3 grid(items > 0 ? items : p.T, b2_gqa_head_blocks(a));
-    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, gqa_decode_kernel<NB, EXACT>, grid, dim3(kWarps * 32), (size_t)smem_bytes(a), ctx->stream, a, p, items > 0));
+    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, gqa_decode_kernel<NB, EXACT, MAPS>, grid, dim3(kWarps * 32), (size_t)smem_bytes(a), ctx->stream, a, p, items > 0));
     B2_LAUNCHED(ctx);
     return B2_OK;
 }
 
 }  // namespace
 
-bool b2_gqa_decode_eligible(const GroupedAttnSpec& a) { return a.k_row() <= 256 && a.v_row() <= 256; }
-int b2_gqa_head_blocks(const GroupedAttnSpec& a) { return a.kv_heads * ((a.group() + kHeads - 1) / kHeads); }
+bool b2_gqa_decode_eligible(const GroupedAttnSpec& a) { return a.k_row() * a.maps <= 256 && a.v_row() <= 256; }
+int b2_gqa_head_blocks(const GroupedAttnSpec& a) { return a.kv_heads * ((a.group() * a.maps + kHeads - 1) / kHeads); }
 int32_t b2_gqa_decode_launch(b2_ctx* ctx, const GroupedAttnSpec& a, const GqaAttnParams& p, int items) {
     if (p.T <= 0) return B2_OK;
     B2_REQUIRE(p.page_size % 16 == 0, B2_ERR_UNSUPPORTED, "grouped attention: pages of whole 16-key tiles");
-    const int nb = (a.k_row() > a.v_row() ? a.k_row() : a.v_row()) / 16;
+    const int k_row = a.k_row() * a.maps, nb = (k_row > a.v_row() ? k_row : a.v_row()) / 16;
+    if (a.maps == 2) {
+        B2_REQUIRE(!a.sink, B2_ERR_UNSUPPORTED, "grouped attention: a sink beside two maps");
+        if (k_row == a.v_row() && nb == 8) return launch<8, true, 2>(ctx, a, p, items);
+        return nb <= 8 ? launch<8, false, 2>(ctx, a, p, items) : launch<16, false, 2>(ctx, a, p, items);
+    }
     if (a.k_row() == a.v_row() && nb == 4) return launch<4, true>(ctx, a, p, items);
     if (a.k_row() == a.v_row() && nb == 8) return launch<8, true>(ctx, a, p, items);
     if (nb <= 8) return launch<8, false>(ctx, a, p, items);

@@ -10,6 +10,9 @@
 //   warps 0-7   softmax, thread = (query row, half of the key tile): cap, mask, maximum (shared with the row's other thread),
 //               exponentials, P over the scores it came from; the running maximum is raised only when a tile exceeds it by
 //               2^8; the sink enters the row sum at the end; every wait bounded
+// Two maps (differential attention): a key tile is two steps, one per map, on the S buffer, the K stage and the O accumulator of that map,
+// both with the same V stage; the difference, its norm and the head's gate happen on the way out.
+// Under a mask the tiles are those of the kept first keys, then those from the first query's first visible key on.
 #include "elt.cuh"
 #include "layer_kernels.h"
 #include "tc5.cuh"
@@ -33,17 +36,19 @@ constexpr uint32_t idesc(int n, bool b_mn) {
     return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(n >> 3) << 17) | ((uint32_t)(128 >> 4) << 24) | (b_mn ? (1u << 16) : 0u);
 }
 
-template <int DKB, int VDB>
+template <int DKB, int VDB, int MAPS>
 struct Layout {  // shared memory of a CTA
     static constexpr int NS = 2;  // K / V stages
-    static constexpr int Q = 0, K = DKB * BLOCK_BYTES, V = K + NS * DKB * BLOCK_BYTES, BAR = V + NS * VDB * BLOCK_BYTES, X = BAR + 256, BYTES = X + 2048;
+    static constexpr int Q = 0, K = MAPS * DKB * BLOCK_BYTES, V = K + NS * DKB * BLOCK_BYTES, BAR = V + NS * VDB * BLOCK_BYTES, X = BAR + 256;
+    // maxima [2 steps in flight][2 groups][128 rows]; two maps: row sums [2 maps][2 groups][128] and sums of squares [2 groups][128]
+    static constexpr int BYTES = X + (MAPS == 2 ? 5120 : 2048);
 };
 
-template <int DKB, int VDB, bool CAP>
+template <int DKB, int VDB, bool CAP, int MAPS>
 __global__ void __launch_bounds__(kThreads, 1)
     gqa_prefill_kernel(const GroupedAttnSpec a, const GqaAttnParams p, int* err, const __grid_constant__ CUtensorMap map_q,
                        const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v) {
-    using L = Layout<DKB, VDB>;
+    using L = Layout<DKB, VDB, MAPS>;
     constexpr int NS = L::NS;
     extern __shared__ __align__(1024) uint8_t smem_raw[];
     pdl_wait();
@@ -68,15 +73,16 @@ __global__ void __launch_bounds__(kThreads, 1)
     volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(smem_raw + L::BAR + 8 * 18);
 
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int head = blockIdx.y, kvh = head / a.group(), KR = a.k_row();
+    const int head = blockIdx.y, kvh = head / a.group(), KR = a.k_row();  // (a step s = tile * MAPS + map)
     const float score_scale = CAP ? 2.f * a.scale / a.softcap * kLog2e : a.scale * kLog2e, cap = a.softcap * kLog2e;
     const int b = p.pf_seq[w], q_start = p.pf_qstart[w];
     const int tok0 = p.cu_seqlens[b], qn = p.cu_seqlens[b + 1] - tok0;
     const int ctx = p.context_lens[b], ctx_before = ctx - qn;
     const int rows = min(QT, qn - q_start);
-    // under a mask the walk starts at the tile of the first query's first visible key; tile numbers count from there
-    const int first_tile = a.mask.first(ctx_before + q_start) / KT, key0 = first_tile * KT;
-    const int n_tiles = (ctx_before + q_start + rows - 1 - key0) / KT + 1;
+    // tiles in the order they are taken: kept keys, then from the first query's first visible key on
+    const int first_pos = ctx_before + q_start, first_tile = a.mask.first(first_pos) / KT, kept = a.mask.kept_tiles(first_pos, KT), keep = a.mask.keep;
+    const int n_tiles = kept + (first_pos + rows - 1) / KT - first_tile + 1, n_steps = n_tiles * MAPS;
+    auto tile_key = [&](int j) { return (j < kept ? j : j - kept + first_tile) * KT; };  // first key of the j-th
 
     if (tid == 0) {
         mbar_init(q_full, 1);
@@ -109,20 +115,21 @@ __global__ void __launch_bounds__(kThreads, 1)
     if (warp == kKWarp || warp == kVWarp) {
         // a box of 16 keys x 64 values per lane, found through the block table; boxes past the context repeat its first page
         const bool is_k = warp == kKWarp;
-        const int blocks = is_k ? DKB : VDB, sub = lane & 7, blk = lane >> 3, ps = p.page_size;
+        const int blocks = is_k ? DKB : VDB, sub = lane & 7, blk = lane >> 3, ps = p.page_size, per = is_k ? MAPS : 1;  // stages per tile
         const int32_t* bt = p.block_tables + (size_t)p.seq_slot[b] * p.max_blocks;
-        auto row_of = [&](int j) {
-            const int key = key0 + j * KT + sub * 16, kk = key < ctx ? key : 0;
-            return (bt[kk / ps] * a.kv_heads + kvh) * ps + kk % ps;
+        auto row_of = [&](int i) {
+            const int j = i / per, key = tile_key(j) + sub * 16, kk = key < ctx ? key : 0;
+            return ((bt[kk / ps] * a.kv_heads + kvh) * per + (i - j * per)) * ps + kk % ps;
         };
         if (is_k && lane == 0) {
-            mbar_expect_tx(q_full, (uint32_t)DKB * BLOCK_BYTES);
-            for (int i = 0; i < DKB; i++) tma_load_2d(base + L::Q + i * BLOCK_BYTES, &map_q, head * KR + i * 64, tok0 + q_start, q_full);
+            mbar_expect_tx(q_full, (uint32_t)MAPS * DKB * BLOCK_BYTES);
+            for (int i = 0; i < MAPS * DKB; i++)
+                tma_load_2d(base + L::Q + i * BLOCK_BYTES, &map_q, (head * MAPS + i / DKB) * KR + i % DKB * 64, tok0 + q_start, q_full);
         }
         __syncwarp();
         int st = 0, next = row_of(0);
         uint32_t par = 0;
-        for (int j = 0; j < n_tiles; j++) {
+        for (int j = 0; j < n_tiles * per; j++) {
             const int row = next;
             next = row_of(j + 1);
             const uint32_t full = is_k ? k_full(st) : v_full(st);
@@ -143,45 +150,46 @@ __global__ void __launch_bounds__(kThreads, 1)
         if (lane == 0) {
             constexpr uint32_t kQK = idesc(128, false), kPV = idesc(VDB * 64, true);
             const uint64_t dq0 = desc_kmajor(base + L::Q), dk0 = desc_kmajor(base + L::K), dv0 = desc_mnmajor(base + L::V, BLOCK_BYTES);
-            auto issue_qk = [&](int j, int kst) {  // S[j & 1] = Q K_j^T
+            auto issue_qk = [&](int j, int kst) {  // S[j & 1] = Q K_j^T of step j
                 const uint64_t dk = dk0 + (uint64_t)((uint32_t)kst * DKB * (BLOCK_BYTES >> 4));
+                const uint64_t dq = MAPS == 2 ? dq0 + (uint64_t)((uint32_t)(j & 1) * DKB * (BLOCK_BYTES >> 4)) : dq0;
                 const uint32_t ts = tmem_base + (uint32_t)(j & 1) * 128u;
 #pragma unroll
                 for (int k = 0; k < DKB * 4; k++) {
                     const uint64_t off = (uint64_t)((uint32_t)(k >> 2) * (BLOCK_BYTES >> 4) + (uint32_t)(k & 3) * 2);
-                    tc_mma(ts, dq0 + off, dk + off, kQK, k > 0 ? 1u : 0u);
+                    tc_mma(ts, dq + off, dk + off, kQK, k > 0 ? 1u : 0u);
                 }
                 tc_commit(s_ready(j & 1));
                 tc_commit(k_empty(kst));
             };
             alive = mbar_wait(q_full, 0);
-            for (int j = 0; j < 2 && j < n_tiles && alive; j++) {
+            for (int j = 0; j < 2 && j < n_steps && alive; j++) {
                 alive = mbar_wait(k_full(j), 0);
                 if (alive) {
                     tc_fence_after();
                     issue_qk(j, j);
                 }
             }
-            for (int j = 0; j < n_tiles && alive; j++) {  // with two stages, stage and parity follow from the tile number
-                const int sb = j & 1;
+            for (int j = 0; j < n_steps && alive; j++) {  // with two stages, stage and parity follow from the step's (values: the tile's) number
+                const int sb = j & 1, vt = j / MAPS, vb = vt & 1;
                 const uint32_t ph = (uint32_t)(j >> 1) & 1u;
-                alive = mbar_wait(v_full(sb), ph) && mbar_wait(p_ready(sb), ph);
+                alive = mbar_wait(v_full(vb), (uint32_t)(vt >> 1) & 1u) && mbar_wait(p_ready(sb), ph);
                 if (!alive) break;
                 tc_fence_after();
-                const uint64_t dvs = dv0 + (uint64_t)((uint32_t)sb * VDB * (BLOCK_BYTES >> 4));
-                const uint32_t tP = tmem_base + (uint32_t)sb * 128u;
+                const uint64_t dvs = dv0 + (uint64_t)((uint32_t)vb * VDB * (BLOCK_BYTES >> 4));
+                const uint32_t tP = tmem_base + (uint32_t)sb * 128u, tO = MAPS == 2 ? tmem_o + (uint32_t)sb * (VDB * 64u) : tmem_o;
 #pragma unroll
                 for (int k = 0; k < KT / 16; k++) {
                     // keys 0-63 of the tile: head in columns 0-31 of the buffer, remainder in 32-63; keys 64-127: 64-95, 96-127
                     const uint32_t ta = tP + (uint32_t)(k >> 2) * 64u + (uint32_t)(k & 3) * 8u;
                     // 16 keys of a V block (128 keys x 64 values; the next 64 values are a block further)
                     const uint64_t dv = dvs + (uint64_t)((uint32_t)k * (2048u >> 4));
-                    tc_mma_ts(tmem_o, ta, dv, kPV, (j > 0 || k > 0) ? 1u : 0u);
-                    tc_mma_ts(tmem_o, ta + 32u, dv, kPV, 1u);
+                    tc_mma_ts(tO, ta, dv, kPV, (vt > 0 || k > 0) ? 1u : 0u);
+                    tc_mma_ts(tO, ta + 32u, dv, kPV, 1u);
                 }
                 tc_commit(pv_done(sb));
-                tc_commit(v_empty(sb));
-                if (j + 2 < n_tiles) {  // S(j+2) goes over P(j): issued after the MMAs above, which complete first
+                if (MAPS == 1 || sb == 1) tc_commit(v_empty(vb));  // (behind the tile's last map)
+                if (j + 2 < n_steps) {  // S(j+2) goes over P(j): issued after the MMAs above, which complete first
                     alive = mbar_wait(k_full(sb), ph ^ 1u);
                     if (!alive) break;
                     tc_fence_after();
@@ -203,8 +211,9 @@ __global__ void __launch_bounds__(kThreads, 1)
         const int klow = a.mask.first(kvis);  // first key it may see
         const float sc = CAP ? 1.f : score_scale;
         float m_run = -INFINITY, l_run = 0.f;  // l_run: this thread's half of the row sum
-        volatile float* xb = reinterpret_cast<volatile float*>(smem_raw + L::X);  // [2 tiles in flight][2 groups][128 rows]
-        for (int j = 0; j < n_tiles && alive; j++) {
+        float m_other = -INFINITY, l_other = 0.f;  // two maps: the same of the other map, whose turn the next step is
+        volatile float* xb = reinterpret_cast<volatile float*>(smem_raw + L::X);  // [2 steps in flight][2 groups][128 rows]
+        for (int j = 0; j < n_steps && alive; j++) {
             const int st = j & 1;
             const uint32_t s_addr = tmem_base + lane_addr + (uint32_t)st * 128u + (uint32_t)wg * 64u;
             if (!__all_sync(0xffffffffu, mbar_wait(s_ready(st), (uint32_t)(j >> 1) & 1u))) {
@@ -212,7 +221,7 @@ __global__ void __launch_bounds__(kThreads, 1)
                 break;
             }
             tc_fence_after();
-            const int key_base = key0 + j * KT + wg * 64;
+            const int key_base = tile_key(j / MAPS) + wg * 64;
             const bool need_mask = key_base + 63 > kvis || key_base < klow;
             // this thread's 64 scores (log2 domain, masked), their maximum, then the maximum of the whole row
             uint32_t v0[32], v1[32];
@@ -233,8 +242,9 @@ __global__ void __launch_bounds__(kThreads, 1)
             if (need_mask) {
 #pragma unroll
                 for (int i = 0; i < 32; i++) {
-                    if (key_base + i > kvis || key_base + i < klow) v0[i] = 0xff800000u;
-                    if (key_base + 32 + i > kvis || key_base + 32 + i < klow) v1[i] = 0xff800000u;
+                    const int k0 = key_base + i, k1 = k0 + 32;
+                    if (k0 > kvis || (k0 < klow && k0 >= keep)) v0[i] = 0xff800000u;
+                    if (k1 > kvis || (k1 < klow && k1 >= keep)) v1[i] = 0xff800000u;
                 }
             }
             float mx0 = -INFINITY, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY;
@@ -257,7 +267,7 @@ __global__ void __launch_bounds__(kThreads, 1)
             // raise the reference point only when this tile exceeds it by more than the threshold
             float alpha = 1.f;
             bool rescale = false;
-            if (j == 0) {
+            if (j < MAPS) {
                 m_run = fmaxf(mx, kNoKeyYet);
             } else if (mx > m_run + kRescaleThreshold) {
                 alpha = exp2f(m_run - mx);
@@ -265,16 +275,16 @@ __global__ void __launch_bounds__(kThreads, 1)
                 rescale = true;
             }
             if (__any_sync(0xffffffffu, rescale)) {  // this group rescales its half of the values
-                // O belongs to the previous tile's P V until it has completed (P V of this tile cannot have been
+                // O belongs to this map's previous P V until it has completed (P V of this step cannot have been
                 // issued yet: it waits for this warp's arrival below)
-                if (!__all_sync(0xffffffffu, mbar_wait(pv_done((j - 1) & 1), (uint32_t)((j - 1) >> 1) & 1u))) {
+                if (!__all_sync(0xffffffffu, mbar_wait(pv_done((j - MAPS) & 1), (uint32_t)((j - MAPS) >> 1) & 1u))) {
                     alive = false;
                     break;
                 }
                 tc_fence_after();
 #pragma unroll 1
                 for (int c = 0; c < VDB; c++) {
-                    const uint32_t o_addr = tmem_o + lane_addr + (uint32_t)wg * (VDB * 32u) + (uint32_t)c * 32u;
+                    const uint32_t o_addr = tmem_o + (MAPS == 2 ? (uint32_t)st * (VDB * 64u) : 0u) + lane_addr + (uint32_t)wg * (VDB * 32u) + (uint32_t)c * 32u;
                     uint32_t v[32];
                     tc_ld32(o_addr, v);
 #pragma unroll
@@ -324,11 +334,49 @@ __global__ void __launch_bounds__(kThreads, 1)
             tc_fence_before();
             __syncwarp();
             if (lane == 0) mbar_arrive(p_ready(st));
+            if constexpr (MAPS == 2) {
+                const float m_next = m_other, l_next = l_other;
+                m_other = m_run, l_other = l_run;
+                m_run = m_next, l_run = l_next;
+            }
         }
         // ---------------- output: O / l, each group its half of the values ----------------
-        if (alive && !__all_sync(0xffffffffu, mbar_wait(pv_done((n_tiles - 1) & 1), (uint32_t)((n_tiles - 1) >> 1) & 1u))) alive = false;
+        if (alive && !__all_sync(0xffffffffu, mbar_wait(pv_done((n_steps - 1) & 1), (uint32_t)((n_steps - 1) >> 1) & 1u))) alive = false;
         // the row sum is the two halves' sums (slot of the tile parity that is not in use any more)
-        if (alive) {
+        if (MAPS == 2 && alive) {  // (an even number of steps: `run` is the first map's again; its last P V ended ahead of the second one's)
+            volatile float *xl = xb + 512, *xs = xb + 1024;  // [2 maps][2 groups][128], [2 groups][128]
+            xl[wg * 128 + r] = l_run;
+            xl[(2 + wg) * 128 + r] = l_other;
+            __syncwarp();
+            if (lane == 0) mbar_arrive(l_ready);
+            alive = __all_sync(0xffffffffu, mbar_wait(l_ready, 0));
+            if (alive) {
+                tc_fence_after();
+                const float f1 = 1.f / (l_run + xl[(wg ^ 1) * 128 + r]), f2 = p.lambda / (l_other + xl[(2 + (wg ^ 1)) * 128 + r]);
+                const uint32_t o1 = tmem_o + lane_addr + (uint32_t)wg * (VDB * 32u), o2 = o1 + VDB * 64u;
+                float ss = 0.f;
+#pragma unroll 1
+                for (int c = 0; c < VDB; c++) {  // difference of the maps, back to the first one's place
+                    uint32_t v[32], u[32];
+                    tc_ld32_nowait(o1 + (uint32_t)c * 32u, v);
+                    tc_ld32_nowait(o2 + (uint32_t)c * 32u, u);
+                    asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
+#pragma unroll
+                    for (int i = 0; i < 32; i++) {
+                        const float d = __uint_as_float(v[i]) * f1 - __uint_as_float(u[i]) * f2;
+                        ss += d * d;
+                        v[i] = __float_as_uint(d);
+                    }
+                    tc_st32(o1 + (uint32_t)c * 32u, v);
+                }
+                xs[wg * 128 + r] = ss;
+                __syncwarp();
+                if (lane == 0) mbar_arrive(l_ready);
+                alive = __all_sync(0xffffffffu, mbar_wait(l_ready, 1));
+                ss += xs[(wg ^ 1) * 128 + r];
+                l_run = sqrtf(ss / (float)a.vdim + p.eps) / (1.f - a.diff);
+            }
+        } else if (alive) {
             const int slot = n_tiles & 1;
             xb[(slot * 2 + wg) * 128 + r] = l_run;
             __syncwarp();
@@ -339,7 +387,8 @@ __global__ void __launch_bounds__(kThreads, 1)
         if (alive) {
             tc_fence_after();
             if (a.sink) l_run += fast_exp2(-m_run);
-            const float inv = p.out_scale / l_run;
+            const float gate = a.head_gate && row_ok ? sigmoid_f32(bf2f(reinterpret_cast<const uint16_t*>(p.gate)[(size_t)(tok0 + q_start + r) * p.ld_gate + head])) : 1.f;
+            const float inv = gate * p.out_scale / l_run;
             const int vdim = a.vdim;
             uint16_t* dst = reinterpret_cast<uint16_t*>(p.out) + (size_t)(tok0 + q_start + (row_ok ? r : 0)) * p.ldo + (size_t)head * vdim;
             const bool vec = vdim % 8 == 0;  // rows are 16-byte aligned then (ldo is a multiple of 64)
@@ -380,12 +429,15 @@ __global__ void __launch_bounds__(kThreads, 1)
     }
 }
 
-template <int DKB, int VDB>
+template <int DKB, int VDB, int MAPS = 1>
 int32_t launch(b2_ctx* ctx, const GroupedAttnSpec& a, const GqaAttnParams& p, int grid_work, const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv) {
-    constexpr int kBytes = Layout<DKB, VDB>::BYTES;
-    B2_SMEM_ONCE(ctx, (gqa_prefill_kernel<DKB, VDB, false>), kBytes);
-    B2_SMEM_ONCE(ctx, (gqa_prefill_kernel<DKB, VDB, true>), kBytes);
-    auto k = a.softcap > 0.f ? gqa_prefill_kernel<DKB, VDB, true> : gqa_prefill_kernel<DKB, VDB, false>;
+    constexpr int kBytes = Layout<DKB, VDB, MAPS>::BYTES;
+    auto k = gqa_prefill_kernel<DKB, VDB, false, MAPS>;
+    B2_SMEM_ONCE(ctx, (gqa_prefill_kernel<DKB, VDB, false, MAPS>), kBytes);
+    if constexpr (MAPS == 1) {
+        B2_SMEM_ONCE(ctx, (gqa_prefill_kernel<DKB, VDB, true, MAPS>), kBytes);
+        if (a.softcap > 0.f) k = gqa_prefill_kernel<DKB, VDB, true, MAPS>;
+    }
     B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, k, dim3(grid_work, a.heads), dim3(kThreads), (size_t)kBytes, ctx->stream, a, p, ctx->dev_err, mq, mk, mv));
     B2_LAUNCHED(ctx);
     return B2_OK;
@@ -396,19 +448,29 @@ int blocks64(int n) { return (n + 63) / 64; }
 
 bool b2_gqa_prefill_eligible(const GroupedAttnSpec& a) {
     const int dk = blocks64(a.k_row()), vd = blocks64(a.v_row());
+    if (a.maps == 2) return dk <= 2 && vd <= 2 && a.scale > 0.f && a.softcap == 0.f && !a.sink;
     return dk <= 3 && vd <= 3 && dk + vd < 6 && (a.scale > 0.f || a.softcap > 0.f);
 }
 // The work list must have been built with 128-query tiles; q has at least 128 rows (a load box is never taller than its tensor).
 int32_t b2_gqa_prefill_launch(b2_ctx* ctx, const GroupedAttnSpec& a, const GqaAttnParams& p, int grid_work) {
     if (grid_work <= 0) return B2_OK;
     B2_REQUIRE(p.q_rows >= QT && p.page_size % 16 == 0, B2_ERR_MSG, "grouped attention: needs 128 query rows and pages of whole 16-key boxes");
-    const uint64_t rows = (uint64_t)p.max_pages * a.kv_heads * p.page_size, q_cols = (uint64_t)a.heads * a.k_row();
-    B2_REQUIRE(rows < (1ull << 31), B2_ERR_UNSUPPORTED, "grouped attention: the page pool is too large");
+    const uint64_t rows = (uint64_t)p.max_pages * a.kv_heads * p.page_size, q_cols = (uint64_t)a.q_heads() * a.k_row();
+    B2_REQUIRE(rows * a.maps < (1ull << 31), B2_ERR_UNSUPPORTED, "grouped attention: the page pool is too large");
     CUtensorMap mq, mk, mv;
     B2_CHECK(get_map(ctx, p.q, (uint64_t)p.q_rows, q_cols, q_cols, QT, &mq));
-    B2_CHECK(get_map(ctx, p.k_cache, rows, (uint64_t)a.k_row(), (uint64_t)a.k_row(), 16, &mk));
+    B2_CHECK(get_map(ctx, p.k_cache, rows * a.maps, (uint64_t)a.k_row(), (uint64_t)a.k_row(), 16, &mk));
     B2_CHECK(get_map(ctx, p.v_cache, rows, (uint64_t)a.v_row(), (uint64_t)a.v_row(), 16, &mv));
-    switch (blocks64(a.k_row()) * 4 + blocks64(a.v_row())) {
+    const int blocks = blocks64(a.k_row()) * 4 + blocks64(a.v_row());
+    if (a.maps == 2) {
+        switch (blocks) {
+            case 5: return launch<1, 1, 2>(ctx, a, p, grid_work, mq, mk, mv);
+            case 6: return launch<1, 2, 2>(ctx, a, p, grid_work, mq, mk, mv);
+            case 9: return launch<2, 1, 2>(ctx, a, p, grid_work, mq, mk, mv);
+            case 10: return launch<2, 2, 2>(ctx, a, p, grid_work, mq, mk, mv);
+        }
+    }
+    switch (blocks) {
         case 5: return launch<1, 1>(ctx, a, p, grid_work, mq, mk, mv);
         case 6: return launch<1, 2>(ctx, a, p, grid_work, mq, mk, mv);
         case 7: return launch<1, 3>(ctx, a, p, grid_work, mq, mk, mv);

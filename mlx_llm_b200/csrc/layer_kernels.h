@@ -12,6 +12,25 @@ struct b2_ctx;
 // x[t, :width] (f32 residual stream) = table[ids[t]], `copies` rows of x per token
 int32_t b2_embed_residual_launch(b2_ctx* ctx, bool f32, const void* table, int ld_table, const int32_t* ids, int T, int width, int vocab, float* x,
                                  int ldx, int copies = 1);
+// The stream's beginning for models without a norm ahead of their layers: table[ids[t]] * scale, plus the row of the (previous, current)
+// token in a table of its own (PairSpec).  The last token of every sequence is kept for its next step.
+struct EmbedPairsParams {
+    const void* table;
+    int ld_table, T, width, vocab;
+    const int32_t* ids;
+    float scale;
+    PairSpec pairs;
+    const void* pair_table;  // [buckets + 1, ld_pairs]
+    int ld_pairs;
+    const int32_t *cu_seqlens, *context_lens, *token_seq, *seq_slot;
+    float* kept;             // slot s: the bits of the token at kept + s * slot_stride
+    int64_t slot_stride;
+    float* x;                // [T, ldx]
+    int ldx;
+    void* out;               // [T, ldo] the same in storage format, zero beyond width
+    int ldo;
+};
+int32_t b2_embed_pairs_launch(b2_ctx* ctx, bool f32, const EmbedPairsParams& p);
 struct AddNormParams {
     float* x;               // [*, ldx] residual stream
     const float* y;         // what the last sub-layer added (f32), null: nothing
@@ -26,6 +45,7 @@ struct AddNormParams {
     int ldx, ldy, ldo, rows, width, n_src;
     float eps, out_scale;   // out = norm * w * out_scale
     bool write_x;
+    int groups;             // > 1: that many equal parts are normed by themselves (divides the width)
 };
 int32_t b2_add_norm_launch(b2_ctx* ctx, bool f32, const AddNormParams& p);
 // Several residual streams per token: the pending sub-layer's y goes to every stream beside a mixture of the old ones, then the
@@ -47,6 +67,36 @@ struct StreamNormParams {
     float eps, out_scale;
     bool write_x;
 };
+// Norm behind a sub-layer: x' = x + mult * norm(y) * w in `groups` equal parts; then, with weights `avg`, the stream goes on as
+// sum_(j < depth) avg[j] past[j] + avg[depth] x'.
+struct PostNormParams {
+    const float* x;         // [rows, ldx] residual stream
+    float* x_out;           // what goes on (may be x; null: not stored)
+    const float* y;         // [rows, ldy] the sub-layer's output
+    const float* w;         // [width]
+    int groups;
+    float eps, mult;
+    const float* avg;       // [depth + 1]; null: x' goes on
+    int depth;
+    const float* past;      // j-th: past + j * past_stride, [rows, ldx]
+    int64_t past_stride;
+    float* keep;            // [rows, ldx] receives x'; null: not stored
+    void* out;              // [rows, ldo] what goes on in storage format, zero beyond width; null: not stored
+    int ldx, ldy, ldo, rows, width;
+};
+int32_t b2_post_norm_launch(b2_ctx* ctx, bool f32, const PostNormParams& p);
+// out[t, j] = gelu(z[t, j]) * table[ids[t], col0 + j] for j < n (tanh form), zero up to ldo
+struct TokenGateParams {
+    const float* z;
+    int ldz;
+    const void* table;
+    int ld_table, col0, vocab;
+    const int32_t* ids;
+    int T, n;
+    void* out;
+    int ldo;
+};
+int32_t b2_token_gate_launch(b2_ctx* ctx, bool f32, const TokenGateParams& p);
 constexpr int kMaxStreams = 16;
 int32_t b2_stream_norm_launch(b2_ctx* ctx, bool f32, const StreamNormParams& p);
 // out[r, j] = act(gu[r, j], gu[r, up_off + j]), scaled by row_w[r] when given (see GateSpec); zero for j in [ff, ldo).  Up to two such
@@ -198,9 +248,10 @@ bool b2_latent_prefill_eligible(const LatentAttnSpec& a);
 int32_t b2_latent_prefill_launch(b2_ctx* ctx, const LatentAttnSpec& a, const LatentPrefillParams& p, int grid_work);
 
 // ---- grouped_attn.cu, grouped_attn_decode.cu, grouped_attn_prefill.cu --------------------------------------------------
-// Cache of a layer: keys [page][kv_heads][page_size][k_row], values [page][kv_heads][page_size][v_row].
+// Cache of a layer: keys [page][k_heads][page_size][k_row], values [page][kv_heads][page_size][v_row].  With two maps head h's queries are
+// rows 2h and 2h + 1, a key / value head's keys likewise (k_heads, q_heads).
 struct GqaPrepParams {
-    const void* in;         // [T, ld] projections: queries from q_off, keys from k_off, values from v_off, heads tight
+    const void* in;         // [T, ld] projections: queries from q_off, keys from k_off, values from v_off, heads (and their maps) tight
     int ld, q_off, k_off, v_off, T;
     const float *q_bias, *k_bias, *v_bias;  // null: none
     const float *q_norm, *k_norm;           // null: none; [dim], or [heads * dim] (norm_all)
@@ -208,7 +259,7 @@ struct GqaPrepParams {
     float eps;
     const int32_t *positions, *slot_mapping;
     const float *cos_t, *sin_t;  // [positions, rot.dims / 2]
-    void* q;                // [T, heads, k_row]
+    void* q;                // [T, q_heads, k_row]
     void *k_cache, *v_cache;
     int page_size;
 };
@@ -226,12 +277,16 @@ struct GqaAttnParams {
     const int32_t *dec_ctx, *dec_qrow, *dec_slot, *work_seq, *work_chunk, *work_off, *n_dec_work;
     int row_chunks;              // > 0 (under a mask): item = row * row_chunks + chunk, chunks counted from the first visible key's tile
     int chunk_tiles;             // 16-key tiles per work item
-    float *part_o, *part_ml;     // [work item][head][v_row], [work item][head][2]
+    float *part_o, *part_ml;     // [work item][q head][v_row], [work item][q head][2]
     int* counters;               // [decode rows][head blocks], zero between launches
     // the packer's prefill list (sequence, first query), 128 queries per item
     const int32_t *pf_seq, *pf_qstart, *n_pf_work, *cu_seqlens, *context_lens;
     int q_rows;                  // rows of the q allocation
     float out_scale;
+    // two maps: weight of the second one, eps of the norm of their difference; head_gate: [T, ld_gate] one column per head
+    float lambda, eps;
+    const void* gate;
+    int ld_gate;
     void* out;                   // [T, ldo]: heads * vdim columns
     int ldo;
 };
@@ -312,6 +367,25 @@ struct BranchOutParams {
     int ld_up, ff, f_off;
 };
 int32_t b2_branch_out_launch(b2_ctx* ctx, bool f32, const BranchOutParams& p);
+
+// ---- gated_average.cu: GatedAverageSpec -------------------------------------------------------------------------------
+struct GatedAverageParams {
+    const void* in;         // [T, ld] projections Z, U, G from these columns, each zero up to a multiple of 8
+    int ld, z_off, u_off, g_off, width;
+    const float *z_bias, *u_bias;  // zero up to a multiple of 8
+    int T, B;
+    const int32_t *cu_seqlens, *context_lens, *seq_slot;
+    float* state;           // slot s: state + s * slot_stride, [width] (up to a multiple of 4)
+    int64_t slot_stride;
+    void* out;              // [T, ldo] zero beyond width
+    int ldo;
+    // portions of at least kMemoryChunkMin tokens: 64-token chunks (as the memories')
+    int n_chunks;
+    const int32_t* chunk_off;
+    float* chunk;           // scratch, n_chunks * b2_gated_average_chunk_floats()
+};
+size_t b2_gated_average_chunk_floats(int width);  // per chunk
+int32_t b2_gated_average_launch(b2_ctx* ctx, bool f32, const GatedAverageParams& p);
 
 // ---- ssm.cu ---------------------------------------------------------------------------------------------------------
 struct SsmParams {

@@ -4,6 +4,11 @@
 
 namespace {
 
+__device__ __forceinline__ float gelu_tanh_f32(float g) {
+    const float k = 0.7978845608028654f;  // sqrt(2 / pi)
+    return 0.5f * g * (1.0f + tanhf(k * (g + 0.044715f * g * g * g)));
+}
+
 template <typename T>
 __global__ void embed_residual_kernel(const T* __restrict__ table, int ld_table, const int32_t* __restrict__ ids, int width, int vocab,
                                       float* __restrict__ x, int ldx, int copies) {
@@ -15,6 +20,161 @@ __global__ void embed_residual_kernel(const T* __restrict__ table, int ld_table,
         const float v = Elt<T>::ld(table + (size_t)id * ld_table + i);
         for (int c = 0; c < copies; c++) x[((size_t)t * copies + c) * ldx + i] = v;
     }
+}
+
+// One block per token.  The block of a sequence's first token in the step is the only one that reads the kept token, and the one
+// that replaces it.
+template <typename T>
+__global__ void embed_pairs_kernel(const EmbedPairsParams p) {
+    asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
+    pdl_wait();
+    __shared__ int64_t s_row;
+    const int t = blockIdx.x;
+    auto token = [&](int id) { return min(max(id, 0), p.vocab - 1); };
+    const int id = token(p.ids[t]);
+    if (p.pairs.buckets > 0) {
+        if (threadIdx.x == 0) {
+            const int b = p.token_seq[t], start = p.cu_seqlens[b], n = p.cu_seqlens[b + 1] - start;
+            int prev = t > start ? token(p.ids[t - 1]) : -1;
+            if (t == start) {
+                float* kept = p.kept + (size_t)p.seq_slot[b] * p.slot_stride;
+                if (p.context_lens[b] > n) prev = __float_as_int(*kept);
+                *kept = __int_as_float(token(p.ids[start + n - 1]));
+            }
+            s_row = prev < 0 ? p.pairs.buckets : ((int64_t)prev * p.pairs.mul_prev + (int64_t)id * p.pairs.mul_cur) % p.pairs.buckets;
+        }
+        __syncthreads();
+    }
+    const T* a = reinterpret_cast<const T*>(p.table) + (size_t)id * p.ld_table;
+    const T* b = p.pairs.buckets > 0 ? reinterpret_cast<const T*>(p.pair_table) + (size_t)s_row * p.ld_pairs : nullptr;
+    T* o = reinterpret_cast<T*>(p.out) + (size_t)t * p.ldo;
+    float* x = p.x + (size_t)t * p.ldx;
+    if (p.width % 8 == 0) {  // (table rows and p.ldo are multiples of 64)
+        for (int i = threadIdx.x * 8; i < p.ldo; i += blockDim.x * 8) {
+            float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+            if (i < p.width) {
+                float u[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+                Elt<T>::ld8(a + i, v);
+                if (b) Elt<T>::ld8(b + i, u);
+#pragma unroll
+                for (int j = 0; j < 8; j++) v[j] = fmaf(v[j], p.scale, u[j]);
+                Elt<float>::st8(x + i, v);
+            }
+            Elt<T>::st8(o + i, v);
+        }
+    } else {
+        for (int i = threadIdx.x; i < p.ldo; i += blockDim.x) {
+            const float v = i < p.width ? fmaf(Elt<T>::ld(a + i), p.scale, b ? Elt<T>::ld(b + i) : 0.f) : 0.f;
+            if (i < p.width) x[i] = v;
+            Elt<T>::st(o + i, v);
+        }
+    }
+}
+
+// Sums of squares of `groups` equal parts of a row, by the block's warps: each group has a team of them, or each warp has groups.
+// sq(i) gives column i's square, VEC columns at a time; inv[g] receives 1 / sqrt(mean + eps).  `part` holds 32 floats.
+template <typename F>
+__device__ __forceinline__ void group_inverses(int width, int groups, float eps, float* part, float* inv, int step, F sum_at) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5, size = width / groups;
+    const int teams = min(groups, warps), team_warps = warps / teams, team = warp / team_warps, mine = warp - team * team_warps;
+    if (team < teams)
+        for (int g = team; g < groups; g += teams) {
+            float ss = 0.f;
+            for (int i = (mine * 32 + lane) * step; i < size; i += team_warps * 32 * step) ss += sum_at(g * size + i);
+            ss = elt_warp_sum(ss);
+            if (lane == 0) {
+                if (team_warps == 1)
+                    inv[g] = 1.0f / sqrtf(ss / (float)size + eps);
+                else
+                    part[warp] = ss;
+            }
+        }
+    __syncthreads();
+    if (team_warps > 1) {
+        for (int g = threadIdx.x; g < groups; g += blockDim.x) {
+            float ss = 0.f;
+            for (int k = 0; k < team_warps; k++) ss += part[g * team_warps + k];
+            inv[g] = 1.0f / sqrtf(ss / (float)size + eps);
+        }
+        __syncthreads();
+    }
+}
+
+// One block per row; y stays in shared memory between the two passes.
+template <typename T, int VEC>
+__global__ void post_norm_kernel(const PostNormParams p) {
+    asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
+    pdl_wait();
+    extern __shared__ __align__(16) float row[];  // [width], then [groups]
+    __shared__ float part[32];
+    float* inv = row + (p.width + 3) / 4 * 4;
+    const size_t r = blockIdx.x;
+    const int size = p.width / p.groups;
+    auto load = [](const float* s, float (&v)[VEC]) {
+        if constexpr (VEC == 4)
+            Elt<float>::ld4(s, v);
+        else
+            v[0] = s[0];
+    };
+    auto store = [](float* d, const float (&v)[VEC]) {
+        if constexpr (VEC == 4)
+            Elt<float>::st4(d, v);
+        else
+            d[0] = v[0];
+    };
+    const float* yr = p.y + r * p.ldy;
+    group_inverses(p.width, p.groups, p.eps, part, inv, VEC, [&](int i) {
+        float v[VEC], ss = 0.f;
+        load(yr + i, v);
+        store(row + i, v);
+#pragma unroll
+        for (int e = 0; e < VEC; e++) ss += v[e] * v[e];
+        return ss;
+    });
+    const float* xr = p.x + r * p.ldx;
+    T* o = p.out ? reinterpret_cast<T*>(p.out) + r * p.ldo : nullptr;
+    for (int i = threadIdx.x * VEC; i < p.width; i += blockDim.x * VEC) {
+        float x[VEC], y[VEC], w[VEC];
+        load(xr + i, x);
+        load(row + i, y);
+        load(p.w + i, w);
+        const float f = inv[i / size];  // (VEC columns lie in one group)
+#pragma unroll
+        for (int e = 0; e < VEC; e++) x[e] = fmaf(p.mult, y[e] * f * w[e], x[e]);
+        if (p.keep) store(p.keep + r * p.ldx + i, x);
+        if (p.avg) {
+            const float own = p.avg[p.depth];
+#pragma unroll
+            for (int e = 0; e < VEC; e++) x[e] *= own;
+            const float* past = p.past + r * p.ldx + i;
+#pragma unroll 4
+            for (int j = 0; j < p.depth; j++) {
+                float v[VEC];
+                load(past + j * p.past_stride, v);
+#pragma unroll
+                for (int e = 0; e < VEC; e++) x[e] = fmaf(p.avg[j], v[e], x[e]);
+            }
+        }
+        if (p.x_out) store(p.x_out + r * p.ldx + i, x);
+        if (o) {
+            if constexpr (VEC == 4)
+                Elt<T>::st4(o + i, x);
+            else
+                Elt<T>::st(o + i, x[0]);
+        }
+    }
+    if (o)
+        for (int i = p.width + threadIdx.x; i < p.ldo; i += blockDim.x) Elt<T>::st(o + i, 0.f);
+}
+
+template <typename T>
+__global__ void token_gate_kernel(const TokenGateParams p) {
+    asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
+    pdl_wait();
+    const int t = blockIdx.x;
+    const T* e = reinterpret_cast<const T*>(p.table) + (size_t)min(max(p.ids[t], 0), p.vocab - 1) * p.ld_table + p.col0;
+    for (int i = threadIdx.x; i < p.ldo; i += blockDim.x)
+        Elt<T>::st(reinterpret_cast<T*>(p.out) + (size_t)t * p.ldo + i, i < p.n ? gelu_tanh_f32(p.z[(size_t)t * p.ldz + i]) * Elt<T>::ld(e + i) : 0.f);
 }
 
 // x += y (one row, or the sum of several), then RMS norm, one block per row.  The row is kept in shared memory between
@@ -64,9 +224,17 @@ __global__ void add_norm_kernel(const AddNormParams p) {
         }
     }
     if (!p.w) return;
+    T* o = reinterpret_cast<T*>(p.out) + (size_t)r * p.ldo;
+    if (p.groups > 1) {
+        float* invs = row + (p.width + 3) / 4 * 4;
+        __syncthreads();
+        group_inverses(p.width, p.groups, p.eps, red, invs, 1, [&](int i) { return row[i] * row[i]; });
+        const int size = p.width / p.groups;
+        for (int i = threadIdx.x; i < p.ldo; i += blockDim.x) Elt<T>::st(o + i, i < p.width ? row[i] * invs[i / size] * p.w[i] * p.out_scale : 0.f);
+        return;
+    }
     ss = elt_block_sum(ss, red);
     const float inv = 1.0f / sqrtf(ss / (float)p.width + p.eps);
-    T* o = reinterpret_cast<T*>(p.out) + (size_t)r * p.ldo;
     if (p.width % 8 == 0) {  // p.ldo is a multiple of 64
         for (int i = threadIdx.x * 8; i < p.ldo; i += blockDim.x * 8) {
             float v[8];
@@ -198,10 +366,7 @@ __global__ void __launch_bounds__(NS <= 4 ? 1024 : 512) stream_norm_kernel(const
 }
 
 __device__ __forceinline__ float gate_one(const GateSpec& gs, float g, float u) {
-    if (gs.act == GateAct::GeluTanh) {
-        const float k = 0.7978845608028654f;  // sqrt(2 / pi)
-        return 0.5f * g * (1.0f + tanhf(k * (g + 0.044715f * g * g * g))) * u;
-    }
+    if (gs.act == GateAct::GeluTanh) return gelu_tanh_f32(g) * u;
     if (gs.act == GateAct::Swish) return silu_f32(g) * u;
     g = fminf(g, gs.limit);
     u = fminf(fmaxf(u, -gs.limit), gs.limit);
@@ -331,13 +496,40 @@ int32_t b2_embed_residual_launch(b2_ctx* ctx, bool f32, const void* table, int l
 int32_t b2_add_norm_launch(b2_ctx* ctx, bool f32, const AddNormParams& p) {
     if (p.rows <= 0) return B2_OK;
     const int th = threads_for(p.width, 8, 512);
-    const size_t smem = ((size_t)p.width * 4 + 15) / 16 * 16;
+    const size_t smem = ((size_t)p.width * 4 + 15) / 16 * 16 + (p.groups > 1 ? (size_t)p.groups * 4 : 0);
     B2_REQUIRE(smem <= 200 * 1024, B2_ERR_UNSUPPORTED, "add_norm: the model is too wide");
     if (smem > 40 * 1024) {
         B2_SMEM_ONCE(ctx, add_norm_kernel<float>, 200 * 1024);
         B2_SMEM_ONCE(ctx, add_norm_kernel<uint16_t>, 200 * 1024);
     }
     B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, f32 ? add_norm_kernel<float> : add_norm_kernel<uint16_t>, dim3(p.rows), dim3(th), smem, ctx->stream, p));
+    B2_LAUNCHED(ctx);
+    return B2_OK;
+}
+int32_t b2_embed_pairs_launch(b2_ctx* ctx, bool f32, const EmbedPairsParams& p) {
+    if (p.T <= 0) return B2_OK;
+    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, f32 ? embed_pairs_kernel<float> : embed_pairs_kernel<uint16_t>, dim3(p.T), dim3(threads_for(p.ldo, 8, 512)), 0, ctx->stream, p));
+    B2_LAUNCHED(ctx);
+    return B2_OK;
+}
+int32_t b2_post_norm_launch(b2_ctx* ctx, bool f32, const PostNormParams& p) {
+    if (p.rows <= 0) return B2_OK;
+    const bool vec = (p.width / p.groups) % 4 == 0 && p.ldx % 4 == 0 && p.ldy % 4 == 0 && p.past_stride % 4 == 0;
+    const int th = threads_for(p.width, vec ? 4 : 1, p.rows <= 2 * ctx->sm_count ? 1024 : 512);
+    const size_t smem = ((size_t)p.width * 4 + 15) / 16 * 16 + (size_t)p.groups * 4;
+    B2_REQUIRE(smem <= 200 * 1024, B2_ERR_UNSUPPORTED, "post_norm: the model is too wide");
+    auto run = [&](auto k) -> int32_t {
+        if (smem > 40 * 1024) B2_CUDA(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, k, dim3(p.rows), dim3(th), smem, ctx->stream, p));
+        B2_LAUNCHED(ctx);
+        return B2_OK;
+    };
+    if (f32) return vec ? run(post_norm_kernel<float, 4>) : run(post_norm_kernel<float, 1>);
+    return vec ? run(post_norm_kernel<uint16_t, 4>) : run(post_norm_kernel<uint16_t, 1>);
+}
+int32_t b2_token_gate_launch(b2_ctx* ctx, bool f32, const TokenGateParams& p) {
+    if (p.T <= 0) return B2_OK;
+    B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, f32 ? token_gate_kernel<float> : token_gate_kernel<uint16_t>, dim3(p.T), dim3(threads_for(p.ldo, 1, 256)), 0, ctx->stream, p));
     B2_LAUNCHED(ctx);
     return B2_OK;
 }

@@ -28,6 +28,13 @@ struct Reader {  // typed access to one JSON object; remembers the first thing t
         if (x < lo || x > (1 << 30)) return fail("in-range integer", key, where), 0;
         return (int)x;
     }
+    int64_t factor(const Value* v, const char* key, const std::string& where) {  // of a token id: their product fits 64 bits
+        long long x = 0;
+        const Value* f = v ? v->get(key) : nullptr;
+        if (!f || !f->as_i64(x)) return fail("integer", key, where), 0;
+        if (x < 0 || x > (1ll << 32)) return fail("in-range integer", key, where), 0;
+        return x;
+    }
     double real(const Value* v, const char* key, const std::string& where) {
         double x = 0;
         const Value* f = v ? v->get(key) : nullptr;
@@ -168,6 +175,54 @@ void read_chunk_attention(Reader& r, const Value* m, const std::string& at, Laye
     const Value* from = m ? m->get("kv_from") : nullptr;
     if (from && from->kind != Value::Null) L.kv_from = r.num(m, "kv_from", at, 0);
     if (r.err.empty()) r.require(a.heads % a.kv_heads == 0, at + ": kv_heads must divide heads");
+}
+// Optional sub-object: null when it is missing or null.
+const Value* optional(const Value* v, const char* key) {
+    const Value* f = v ? v->get(key) : nullptr;
+    return f && f->kind != Value::Null ? f : nullptr;
+}
+// differential attention under a window that keeps the first tokens, gated per head, neighbouring coordinates rotated with scaled
+// frequencies, on its own keys or another layer's
+void read_differential(Reader& r, const Value* m, const std::string& at, LayerSpec& L) {
+    GroupedAttnSpec& a = L.gqa;
+    L.mixer = MixerKind::GroupedAttention;
+    a.heads = r.num(m, "heads", at);
+    a.kv_heads = r.num(m, "kv_heads", at);
+    a.dim = r.num(m, "dim", at);
+    a.vdim = r.num(m, "vdim", at);
+    a.scale = (float)r.real(m, "scale", at);
+    a.diff = (float)r.real(m, "diff", at);
+    a.maps = 2;
+    a.qk_norm = a.head_gate = a.neighbours = true;
+    if (optional(m, "rot")) read_rot(r, m, at, a.dim, a.rot);
+    if (const Value* s = optional(optional(m, "rot"), "scaling")) {
+        const std::string sa = at + ".rot.scaling";
+        a.rot.factor = r.real(s, "factor", sa);
+        a.rot.original = r.real(s, "original", sa);
+        a.rot.fast = r.real(s, "fast", sa);
+        a.rot.slow = r.real(s, "slow", sa);
+        if (r.err.empty()) r.require(a.rot.factor > 0 && a.rot.original > 0 && a.rot.fast > 0 && a.rot.slow > 0 && a.rot.base != 1, sa + ": its numbers must be positive");
+    }
+    if (const Value* mask = optional(m, "mask")) {
+        a.mask.kind = MaskSpec::Window;
+        a.mask.size = r.num(mask, "size", at + ".mask");
+        if (optional(mask, "keep_first")) a.mask.keep = r.num(mask, "keep_first", at + ".mask", 0);
+    }
+    if (optional(m, "kv_from")) L.kv_from = r.num(m, "kv_from", at, 0);
+    if (r.err.empty()) r.require(a.heads % a.kv_heads == 0, at + ": kv_heads must divide heads");
+}
+void read_min_gru(Reader& r, const Value* m, const std::string& at, LayerSpec& L) {
+    L.mixer = MixerKind::GatedAverage;
+    L.avg.width = r.num(m, "width", at);
+}
+// kv_from names an earlier layer of the list whose keys and values this one can read
+void check_shared_keys(Reader& r, const std::string& at, const std::vector<LayerSpec>& before, const LayerSpec& L) {
+    if (!r.err.empty() || L.kv_from < 0) return;
+    const bool ok = L.kv_from < (int)before.size() && before[L.kv_from].mixer == MixerKind::GroupedAttention && before[L.kv_from].kv_from < 0;
+    r.require(ok, at + ": kv_from must name an earlier attention layer with keys and values of its own");
+    if (!ok) return;
+    const GroupedAttnSpec &a = L.gqa, &b = before[L.kv_from].gqa;
+    r.require(a.kv_heads == b.kv_heads && a.dim == b.dim && a.vdim == b.vdim, at + ": kv_from names a layer with other key / value heads");
 }
 // time mixing: token shift, a decay per key channel, a bonus for the current token
 void read_time_mix(Reader& r, const Value* m, const std::string& at, LayerSpec& L) {
@@ -328,14 +383,52 @@ int32_t read_zokuzen(const Value& v, ModelSpec& spec) {
             if (L.mixer == MixerKind::Memory) L.mem.shift = spec.width;
             const Value* mlp = lv->get("mlp");
             if (mlp && mlp->kind != Value::Null) read_mixture(r, mlp, at + ".mlp", L);
-            if (r.err.empty() && L.kv_from >= 0) {
-                const bool ok = L.kv_from < (int)i && spec.layers[L.kv_from].mixer == MixerKind::GroupedAttention && spec.layers[L.kv_from].kv_from < 0;
-                r.require(ok, at + ": kv_from must name an earlier attention layer with keys and values of its own");
-                if (ok) {
-                    const GroupedAttnSpec &a = L.gqa, &b = spec.layers[L.kv_from].gqa;
-                    r.require(a.kv_heads == b.kv_heads && a.dim == b.dim && a.vdim == b.vdim, at + ": kv_from names a layer with other key / value heads");
-                }
+            check_shared_keys(r, at, spec.layers, L);
+            spec.layers.push_back(L);
+        }
+    B2_REQUIRE(r.err.empty(), B2_ERR_CONFIG, r.err);
+    return B2_OK;
+}
+
+// ---- Pokadra: differential attention, minimal gated recurrences, clipped-swish feed-forwards; norms in groups behind the sub-layers,
+// embeddings of token pairs, token inputs per layer, averages over the depth, an output projection of its own --------------
+constexpr float kPokadraAlpha = 1.702f;
+bool claims_pokadra(const Value& v) { return names_architecture(v, "Pokadra"); }
+int32_t read_pokadra(const Value& v, ModelSpec& spec) {
+    Reader r;
+    spec.family = "Pokadra";
+    spec.vocab = r.num(&v, "vocab", "the model");
+    spec.width = r.num(&v, "width", "the model");
+    const Value* norm = r.obj(&v, "norm", "the model");
+    spec.eps = (float)r.real(norm, "eps", "norm");
+    spec.norm_groups = r.num(norm, "groups", "norm");
+    if (r.err.empty()) r.require(spec.width % spec.norm_groups == 0, "norm: groups must divide the width");
+    spec.residual_mult = (float)r.real(&v, "residual_mult", "the model");
+    const Value* emb = r.obj(&v, "embedding", "the model");
+    spec.embed_scale = (float)r.real(emb, "scale", "embedding");
+    if (const Value* p = optional(emb, "bigram")) {
+        spec.pairs.buckets = r.num(p, "buckets", "embedding.bigram");
+        spec.pairs.mul_prev = r.factor(p, "mul_prev", "embedding.bigram");
+        spec.pairs.mul_cur = r.factor(p, "mul_cur", "embedding.bigram");
+    }
+    if (optional(&v, "token_side")) spec.side_dim = r.num(optional(&v, "token_side"), "dim", "token_side");
+    spec.own_head = spec.post_norm = spec.depth_average = true;
+    const Value* ls = v.get("layers");
+    r.require(ls && ls->kind == Value::Array && !ls->arr.empty(), "`layers` must be a non-empty list");
+    if (r.err.empty())
+        for (size_t i = 0; i < ls->arr.size(); i++) {
+            const Value* lv = ls->arr[i].get();
+            const std::string at = "layers[" + std::to_string(i) + "]";
+            LayerSpec L;
+            read_mixer(r, {{"attention", read_differential}, {"mingru", read_min_gru}}, lv, at, L);
+            if (const Value* mlp = optional(lv, "mlp")) {
+                const std::string kind = r.str(mlp, "kind", at + ".mlp");
+                r.require(kind == "dense", at + ".mlp: unknown feed-forward kind `" + kind + "`");
+                L.mlp = MlpKind::DenseGated;
+                L.ff = r.num(mlp, "ff", at + ".mlp");
+                L.gate = GateSpec{GateAct::ClippedSwish, (float)r.real(mlp, "limit", at + ".mlp"), kPokadraAlpha};
             }
+            check_shared_keys(r, at, spec.layers, L);
             spec.layers.push_back(L);
         }
     B2_REQUIRE(r.err.empty(), B2_ERR_CONFIG, r.err);
@@ -350,6 +443,7 @@ struct ModelFamily {
 };
 bool claims_flat(const Value&) { return true; }  // b2_model_config_from_json decides (and refuses what it does not know)
 const ModelFamily kFamilies[] = {{"Zukitar", claims_zukitar, read_zukitar}, {"Tirezen", claims_tirezen, read_tirezen}, {"Zokuzen", claims_zokuzen, read_zokuzen},
+                                 {"Pokadra", claims_pokadra, read_pokadra},
                                  {"llama", claims_flat, nullptr}};
 
 int32_t find_family(const char* json, b2json::ValuePtr& root, const ModelFamily** out) {

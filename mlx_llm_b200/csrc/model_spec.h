@@ -6,7 +6,7 @@
 #include <string>
 #include <vector>
 
-enum class MixerKind { LatentAttention, Mamba2, GroupedAttention, Memory, SideBySide };
+enum class MixerKind { LatentAttention, Mamba2, GroupedAttention, Memory, SideBySide, GatedAverage };
 enum class MlpKind { None, DenseGated, DensePlain, Routed };
 // act(gate, up) of a gated feed-forward:
 //   GeluTanh      gelu(gate) * up with the tanh form of gelu
@@ -21,19 +21,29 @@ struct GateSpec {
 };
 
 // Which earlier positions a query may see.  None: all of them; Window: itself and the size - 1 before it; Chunk: those of its own
-// stretch of `size` positions, counted from the sequence's start.  first() never falls as the position rises.
+// stretch of `size` positions, counted from the sequence's start.  first() never falls as the position rises.  The sequence's first
+// `keep` positions stay visible behind first() as well (grouped attention).
 struct MaskSpec {
     enum Kind { None, Window, Chunk } kind = None;
-    int size = 0;
+    int size = 0, keep = 0;
     constexpr int first(int pos) const { return kind == Window ? (pos >= size ? pos - size + 1 : 0) : kind == Chunk ? pos / size * size : 0; }
-    constexpr bool operator==(const MaskSpec& o) const { return kind == o.kind && size == o.size; }
+    // the keys ahead of first(pos) that are visible, and the tiles of `t` keys that hold them ahead of first(pos)'s own tile
+    constexpr int kept(int pos) const { return keep < first(pos) ? keep : first(pos); }
+    constexpr int kept_tiles(int pos, int t) const { return (keep + t - 1) / t < first(pos) / t ? (keep + t - 1) / t : first(pos) / t; }
+    constexpr bool operator==(const MaskSpec& o) const { return kind == o.kind && size == o.size && keep == o.keep; }
 };
 
 // Rotation of dims/2 pairs by position * base^(-2i/dims); the rest passes unchanged.  Which coordinates form pair i is the
-// mixer's: (2i, 2i+1) in latent attention, (i, i + dims/2) in grouped attention and in memories.
+// mixer's: (2i, 2i+1) in latent attention, (i, i + dims/2) in memories and, unless it says otherwise, in grouped attention.
+// With a scaling factor (YaRN) the pairs that turn slowly within `original` positions turn `factor` times slower still, those that turn
+// fast stay, with a ramp between the pairs of `fast` and `slow` turns; cosines and sines grow by 0.1 ln(factor) + 1.
 struct RotSpec {
     double base = 10000.0;
     int dims = 0;
+    double factor = 0.0, original = 0.0, fast = 0.0, slow = 0.0;  // factor 0: no scaling
+    bool operator==(const RotSpec& o) const {
+        return base == o.base && dims == o.dims && factor == o.factor && original == o.original && fast == o.fast && slow == o.slow;
+    }
 };
 // Attention over a shared low-rank latent: per token one vector of kv_rank values and one rotated key part of rot_dim
 // values (0: none) are cached; every head's keys and values are linear images of the latent.
@@ -55,6 +65,8 @@ struct Mamba2Spec {
     constexpr int in_rows() const { return inner() + channels() + heads; }   // z | x | B | C | dt
 };
 // Attention with kv_heads <= heads key / value heads, cached per token.  Keys and values may differ in size.
+// maps 2 (differential): every head has two queries and every key / value head two keys, [map 1 | map 2]; each map is an attention of its
+// own over the same values, and the head's output is norm(a1 - lambda a2) (1 - diff), the RMS norm over vdim without a weight.
 struct GroupedAttnSpec {
     int heads = 0, kv_heads = 0, dim = 0, vdim = 0;
     float scale = 0.f;
@@ -63,9 +75,15 @@ struct GroupedAttnSpec {
     bool bias = false;    // biases of the query, key and value projections
     bool qk_norm = false; // RMS norm of queries and keys before the rotation, per head ...
     bool norm_all = false; // ... or over all heads at once
+    int maps = 1;
+    float diff = 0.f;
+    bool head_gate = false; // a head's output is multiplied by the sigmoid of a projection of the layer's input, one number per head
+    bool neighbours = false; // the rotation's pairs are (2i, 2i+1)
     RotSpec rot;
     MaskSpec mask;
     constexpr int group() const { return heads / kv_heads; }
+    constexpr int q_heads() const { return heads * maps; }
+    constexpr int k_heads() const { return kv_heads * maps; }
     // values per cached head row, zero-padded for 16-wide steps and to one 64-wide load box at least
     constexpr int k_row() const { return dim < 64 ? 64 : (dim + 15) / 16 * 16; }
     constexpr int v_row() const { return vdim < 64 ? 64 : (vdim + 15) / 16 * 16; }
@@ -101,6 +119,11 @@ struct MemorySpec {
     constexpr int keep() const { return conv > 1 ? conv - 1 : 0; }                 // inputs of the convolution kept between steps
     constexpr int decays() const { return decay == MemDecay::PerChannel ? heads * dim : decay == MemDecay::PerHead ? heads : 0; }
 };
+// Gated recurrence whose gates read only the current token (minimal GRU), element by element, the state in f32:
+//     S <- (1 - z) S + z c,   z = sigmoid(Z + b_z),   c = u + 1/2 for u >= 0 and sigmoid(u) below,   u = U + b_x;   out = S silu(G)
+struct GatedAverageSpec {
+    int width = 0;
+};
 // Routed experts: the best `top` of them run for a token.
 //   Sigmoid  scores sigmoid(z); a chosen expert's weight is its score
 //   Softmax  scores softmax(z); the choice goes by score + correction, the chosen scores are normalised to a sum of `scale`
@@ -122,6 +145,7 @@ struct LayerSpec {
     Mamba2Spec ssm;
     GroupedAttnSpec gqa;              // GroupedAttention, SideBySide
     MemorySpec mem;                   // Memory, SideBySide
+    GatedAverageSpec avg;             // GatedAverage
     std::vector<double> decay;        // MemDecay::Fixed: per head
     int kv_from = -1;                 // grouped attention: the layer whose cached keys and values this one reads; -1: its own
     float gqa_scale = 1.f, mem_scale = 1.f;
@@ -147,18 +171,36 @@ struct LayerRun {
 // Tensor names of a family: the `i`-th layer's prefix and the few names outside the layers.
 struct TensorNames {
     std::string embed = "embed", final_norm = "final.norm", layer = "l", norm1 = "norm1", norm2 = "norm2", mixer = "mix", mlp = "mlp",
-                head = "head", loop_step = "loop.step";
+                head = "head", loop_step = "loop.step", pairs = "bigram", side = "side", depth = "dwa";
     std::string layer_key(int i, const std::string& s) const { return layer + std::to_string(i) + "." + s; }
+};
+// A second embedding table, indexed by the previous and the current token: row (previous * mul_prev + current * mul_cur) mod buckets,
+// for a sequence's first token row `buckets`.  buckets 0: none.
+struct PairSpec {
+    int buckets = 0;
+    int64_t mul_prev = 0, mul_cur = 0;
 };
 struct ModelSpec {
     std::string family;
     int vocab = 0, width = 0;
+    float embed_scale = 1.f;
+    PairSpec pairs;
     float eps = 1e-5f, logit_scale = 1.f;
     float norm_offset = 0.f;  // added to the stored weights of the layers' norms and the final norm
     bool own_head = false;    // an output projection beside the embedding table
     // > 0: this many residual streams.  A sub-layer reads sum_s in[s] x_s; afterwards x_t = sum_s mix[s][t] x_s + out[t] y; the model
     // ends with their sum.  0: one stream, x + y.
     int streams = 0;
+    // The norms lie behind the sub-layers, which read the stream itself:  x <- x + residual_mult * norm(sublayer(x)), in norm_groups
+    // equal parts that are normed by themselves.
+    bool post_norm = false;
+    float residual_mult = 1.f;
+    int norm_groups = 1;
+    // > 0: behind the feed-forward a layer adds residual_mult * norm(proj(gelu(gate x) * e)), with e the layer's side_dim columns of the
+    // current token's row in a table of its own
+    int side_dim = 0;
+    // a layer passes on the weighted sum of the embedding output and of what it and every layer before it computed
+    bool depth_average = false;
     std::vector<LayerSpec> layers;
     LoopSpec loop;
     TensorNames names;

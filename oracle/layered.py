@@ -1,8 +1,9 @@
 """Plain numpy restatement (float64) of decoders whose layers are listed one by one in config.json: latent attention,
 Mamba-2, softmax attention with a cap and a sink, retention, the gated delta rule, two mixers side by side, time mixing with a
-bonus for the current token, windowed latent and chunked grouped attention (also on another layer's keys), dense (gated and
-plain) and routed feed-forwards, shared and identity experts, repeated layers, several residual streams.  One function per mechanism, whole sequences only, no cache, no batching:
-the yardstick of the layered models' tests.  Nothing here is shared with the library's own code path.
+bonus for the current token, windowed latent and chunked grouped attention (also on another layer's keys), differential attention
+under a window that keeps the first tokens, the minimal gated recurrence, dense (gated and plain) and routed feed-forwards, shared and
+identity experts, repeated layers, several residual streams, averages over the depth, token inputs per layer, embeddings of token
+pairs.  One function per mechanism, whole sequences only, no cache, no batching: the yardstick of the layered models' tests.  Nothing here is shared with the library's own code path.
 
 Weights are a dict name -> float array; `cfg` is the parsed config.json.
 """
@@ -357,6 +358,121 @@ def forward_zokuzen(cfg, w, tokens, layers_out=None):
     return rms_norm(X.sum(1), 1.0 + w["final.norm"], eps) @ w["embed"].T
 
 
+# ---- Pokadra ---------------------------------------------------------------------------------------------------------
+def embed_pairs(tokens, w, scale, pairs):
+    """Token rows times `scale` plus one row per (previous, current) token; the first token takes the table's last row."""
+    tokens = [int(t) for t in tokens]
+    x = w["embed"][tokens].astype(F) * scale
+    if pairs:
+        rows = [pairs["buckets"]] + [(a * pairs["mul_prev"] + b * pairs["mul_cur"]) % pairs["buckets"] for a, b in zip(tokens, tokens[1:])]
+        x = x + w["bigram"][rows]
+    return x
+
+
+def group_norm(x, w, groups, eps):
+    """RMS norm of each of `groups` equal parts by itself, one weight over all."""
+    return rms(x.reshape(x.shape[0], groups, -1), eps).reshape(x.shape) * w
+
+
+def yarn_frequencies(rot):
+    """-> (angle per position of every pair, factor of cos and sin)."""
+    n, base = rot["dims"], rot["base"]
+    f = np.array([base ** (-2.0 * i / n) for i in range(n // 2)])
+    s = rot.get("scaling")
+    if not s:
+        return f, 1.0
+    place = lambda turns: n * math.log(s["original"] / (2 * math.pi * turns)) / (2 * math.log(base))
+    lo, hi = max(math.floor(place(s["fast"])), 0), min(math.ceil(place(s["slow"])), n - 1)
+    ramp = np.clip((np.arange(n // 2) - lo) / max(hi - lo, 0.001), 0.0, 1.0)
+    return f / s["factor"] * ramp + f * (1 - ramp), 0.1 * math.log(s["factor"]) + 1.0
+
+
+def rotate_scaled(v, pos, rot):
+    """v [..., T, d]: coordinates (2i, 2i+1) turned by the scaled frequencies."""
+    freq, m = yarn_frequencies(rot)
+    out = v.copy()
+    for i, f in enumerate(freq):
+        c, s = np.cos(pos * f) * m, np.sin(pos * f) * m
+        out[..., 2 * i] = v[..., 2 * i] * c - v[..., 2 * i + 1] * s
+        out[..., 2 * i + 1] = v[..., 2 * i + 1] * c + v[..., 2 * i] * s
+    return out
+
+
+def in_window_or_first(T, size, keep):
+    """visible[i, j]: j is i, one of the size - 1 tokens before it, or one of the sequence's first `keep`."""
+    i, j = np.arange(T)[:, None], np.arange(T)[None]
+    return (j <= i) & ((i - j < size) | (j < keep))
+
+
+def difference_weight(lq1, lk1, lq2, lk2, base):
+    return float(np.exp((lq1 * lk1).sum()) - np.exp((lq2 * lk2).sum()) + base)
+
+
+def differential_attention(h, g, m, eps, kv=None):
+    """Two softmax maps per head over the same values; the second one, weighted, is taken off the first; the difference is normed
+    per head and gated by one number per head.  Returns the output and the keys and values it used."""
+    T, H, G, D, V = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    pos = np.arange(T, dtype=F)
+    maps = lambda x, n, w: rotate_scaled(rms_norm(x.reshape(T, n, 2, D), w, eps).transpose(1, 2, 0, 3), pos, m["rot"])  # [n, 2, T, D]
+    q = maps(h @ g("q").T, H, g("q.norm"))
+    if kv is None:
+        kv = (maps(h @ g("k").T, G, g("k.norm")), (h @ g("v").T).reshape(T, G, V).transpose(1, 0, 2))
+    mask = m.get("mask")
+    visible = in_window_or_first(T, mask["size"], mask["keep_first"]) if mask else in_window(T, T + 1)
+    a = [softmax_attention(q[:, i], kv[0][:, i], kv[1], m["scale"], visible).reshape(T, H, V) for i in (0, 1)]
+    o = a[0] - difference_weight(g("lq1"), g("lk1"), g("lq2"), g("lk2"), m["diff"]) * a[1]
+    o = rms(o, eps) * (1.0 - m["diff"]) * sigmoid(h @ g("g").T)[:, :, None]
+    return o.reshape(T, H * V) @ g("o").T, kv
+
+
+def gated_average(z, c):
+    """S_t = (1 - z_t) S_(t-1) + z_t c_t from zero, all [T, width]."""
+    S, out = np.zeros(z.shape[1], F), np.zeros_like(z)
+    for t in range(len(z)):
+        S = (1.0 - z[t]) * S + z[t] * c[t]
+        out[t] = S
+    return out
+
+
+def min_gru(h, g, m, eps):
+    u = h @ g("x").T + g("x.b")
+    S = gated_average(sigmoid(h @ g("z").T + g("z.b")), np.where(u >= 0, u + 0.5, sigmoid(u)))
+    return (S * silu(h @ g("g").T)) @ g("o").T
+
+
+def clipped_ff(h, g, limit):
+    a, u = np.minimum(h @ g("gate").T, limit), np.clip(h @ g("up").T, -limit, limit)
+    return (a * sigmoid(1.702 * a) * (u + 1.0)) @ g("down").T
+
+
+def token_input(x, e, g, eps):
+    """What a token's own row e of the layer adds, gated by the stream."""
+    return rms_norm((gelu_tanh(x @ g("gate").T) * e) @ g("proj").T, g("norm"), eps)
+
+
+def forward_pokadra(cfg, w, tokens, layers_out=None):
+    eps, m, groups = cfg["norm"]["eps"], cfg["residual_mult"], cfg["norm"]["groups"]
+    x = embed_pairs(tokens, w, cfg["embedding"]["scale"], cfg["embedding"].get("bigram"))
+    before, stored, side = [x], {}, cfg.get("token_side")
+    for i, L in enumerate(cfg["layers"]):
+        part = lambda p, i=i: lambda n: w[f"l{i}.{p}.{n}"]
+        if L["type"] == "mingru":
+            y = min_gru(x, part("mix"), L["mixer"], eps)
+        else:
+            y, stored[i] = differential_attention(x, part("mix"), L["mixer"], eps, stored.get(L["mixer"].get("kv_from")))
+        x = x + m * group_norm(y, w[f"l{i}.norm1"], groups, eps)
+        if L.get("mlp"):
+            x = x + m * group_norm(clipped_ff(x, part("mlp"), L["mlp"]["limit"]), w[f"l{i}.norm2"], groups, eps)
+        if side:
+            n = side["dim"]
+            x = x + m * token_input(x, w["side.embed"][np.asarray(tokens), i * n:(i + 1) * n], part("side"), eps)
+        before.append(x)
+        x = sum(c * X for c, X in zip(w[f"l{i}.dwa"], before))
+        if layers_out is not None:
+            layers_out.append(x.copy())
+    return group_norm(x, w["final.norm"], groups, eps) @ w["head"].T
+
+
 def layer_runs(cfg):
     """(layer, pass) in the order they run; pass is -1 outside the repeated stretch."""
     n, loop = len(cfg["layers"]), cfg.get("loop") or dict(start=0, stop=0, times=0)
@@ -366,7 +482,7 @@ def layer_runs(cfg):
 
 def forward(cfg, w, tokens, layers_out=None):
     """Logits [T, vocab] of one sequence.  layers_out (a list) receives the residual stream after every layer run."""
-    by_name = {"Zukitar": forward_zukitar, "Tirezen": forward_tirezen, "Zokuzen": forward_zokuzen}
+    by_name = {"Zukitar": forward_zukitar, "Tirezen": forward_tirezen, "Zokuzen": forward_zokuzen, "Pokadra": forward_pokadra}
     return by_name[cfg["architecture"]](cfg, w, tokens, layers_out)
 
 

@@ -227,6 +227,76 @@ def decide_mixtures(cfg, w, rng, cols=8, margin=0.3):
         w["embed"][t, :cols] = v
 
 
+# ---- Pokadra: differential attention, minimal gated recurrences, norms behind the sub-layers, token pairs and token inputs, depth averages -----
+def differential(heads=4, kv_heads=2, dim=24, vdim=40, dims=16, base=700.0, size=27, keep=5, diff=0.35, scale=None, kv_from=None, scaling=True, original=90, factor=6.0, fast=9.0, slow=1.5):
+    m = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, diff=diff, rot=dict(base=base, dims=dims), mask=dict(size=size, keep_first=keep), scale=scale or float(dim ** -0.5))
+    if scaling:
+        m["rot"]["scaling"] = dict(factor=factor, original=original, fast=fast, slow=slow)
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return ("attention", m)
+
+
+def mingru(width=88):
+    return ("mingru", dict(width=width))
+
+
+def clipped(ff=136, limit=0.9):
+    return dict(kind="dense", ff=ff, limit=limit)
+
+
+def pokadra(layers, width=72, vocab=211, eps=2e-5, groups=3, mult=0.45, side=20, scale=0.7, pairs=(103, 29, 7)):
+    return dict(architecture="Pokadra", width=width, vocab=vocab, norm=dict(eps=eps, groups=groups), residual_mult=mult, token_side=dict(dim=side),
+                embedding=dict(scale=scale, bigram=dict(buckets=pairs[0], mul_prev=pairs[1], mul_cur=pairs[2])),
+                layers=[dict(type=m[0], mixer=m[1], mlp=f) for m, f in layers])
+
+
+def pokadra_weights(cfg, seed=0, gain=None):
+    """name -> float64 array of bf16 values."""
+    rng = np.random.default_rng(seed)
+    w, W, D = {}, cfg["width"], cfg["token_side"]["dim"]
+
+    def mat(name, rows, cols):
+        g = next((v for k, v in (gain or {}).items() if name.endswith(k)), 1.0)
+        w[name] = round_bf16(rng.standard_normal((rows, cols)) * g / np.sqrt(cols))
+
+    def vec(name, n, mean, sd):
+        w[name] = round_bf16(mean + sd * rng.standard_normal(n))
+
+    w["embed"] = round_bf16(1.5 * rng.standard_normal((cfg["vocab"], W)))
+    w["bigram"] = round_bf16(0.6 * rng.standard_normal((cfg["embedding"]["bigram"]["buckets"] + 1, W)))
+    w["side.embed"] = round_bf16(rng.standard_normal((cfg["vocab"], D * len(cfg["layers"]))))
+    for i, L in enumerate(cfg["layers"]):
+        m, p = L["mixer"], f"l{i}.mix."
+        vec(f"l{i}.norm1", W, 1.0, 0.2)
+        if L["type"] == "mingru":
+            n = m["width"]
+            mat(p + "z", n, W), mat(p + "x", n, W), mat(p + "g", n, W), mat(p + "o", W, n)
+            vec(p + "z.b", n, -2.0, 2.5)
+            vec(p + "x.b", n, 0.0, 0.3)
+        else:
+            H, G, d, V = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            mat(p + "q", H * 2 * d, W), mat(p + "g", H, W), mat(p + "o", W, H * V)
+            vec(p + "q.norm", d, 1.2, 0.3)
+            if m.get("kv_from") is None:
+                mat(p + "k", G * 2 * d, W), mat(p + "v", G * V, W)
+                vec(p + "k.norm", d, 1.2, 0.3)
+            for n in ("lq1", "lk1", "lq2", "lk2"):
+                vec(p + n, d, 0.0, 0.15)
+        if L["mlp"]:
+            ff, p = L["mlp"]["ff"], f"l{i}.mlp."
+            vec(f"l{i}.norm2", W, 1.0, 0.2)
+            mat(p + "gate", ff, W), mat(p + "up", ff, W), mat(p + "down", W, ff)
+        mat(f"l{i}.side.gate", D, W), mat(f"l{i}.side.proj", W, D)
+        vec(f"l{i}.side.norm", W, 0.5, 0.15)
+        c = rng.uniform(-0.2, 0.5, i + 2)
+        c[-1] += 0.6
+        w[f"l{i}.dwa"] = round_bf16(c)
+    vec("final.norm", W, 1.0, 0.2)
+    mat("head", cfg["vocab"], W)
+    return w
+
+
 def tokens(cfg, n, seed):
     return np.random.default_rng(seed).integers(0, cfg["vocab"], n).astype(np.int32)
 
@@ -409,4 +479,22 @@ ZOKUZEN = {
     # beyond those kernels, many streams
     "large_heads": zokuzen([(window(heads=2, dim=200, vdim=140, kv_rank=72, size=33), None), (chunk(heads=2, kv_heads=1, dim=232, vdim=250, dims=100, size=50), mixture()), (wkv(heads=2, dim=150), None)],
                            width=64, vocab=80, streams=6),
+}
+
+POKADRA = {
+    "all_kinds": pokadra([(differential(), clipped()), (mingru(), clipped(88, 1.7)), (differential(size=40, keep=17, kv_from=0, scale=0.4), None), (mingru(width=40), None),
+                          (differential(heads=2, kv_heads=1, dim=16, vdim=32, dims=8, size=11, keep=0), clipped(40)), (differential(heads=6, size=200, keep=70, kv_from=0, diff=0.8), clipped(72, 0.2))]),
+    # sizes that divide nothing, single heads and groups, no scaling, windows of one
+    "odd": pokadra([(mingru(width=13), clipped(33)), (differential(heads=5, kv_heads=5, dim=10, vdim=7, dims=4, size=13, keep=1, scaling=False), None),
+                    (differential(heads=3, kv_heads=1, dim=9, vdim=5, dims=6, size=1, keep=3), clipped(17, 4.0)), (mingru(width=97), clipped(50))],
+                   width=53, vocab=97, groups=1, side=7, pairs=(1, 5, 3)),
+    # the tiles of the tensor-core kernels, more than four query heads for one key head
+    "tiles": pokadra([(differential(heads=10, kv_heads=1, dim=64, vdim=128, dims=64, size=100, keep=20), clipped(512)), (mingru(width=256), clipped(256)),
+                      (differential(heads=4, kv_heads=2, dim=128, vdim=128, dims=32, size=150, keep=128), None), (differential(heads=4, kv_heads=2, dim=64, vdim=64, dims=64, size=96, keep=4), clipped(64)),
+                      (differential(heads=5, kv_heads=1, dim=64, vdim=128, dims=64, size=300, keep=130, kv_from=0), None)], width=128, vocab=300, groups=8, side=64, mult=1.0),
+    "uneven": pokadra([(differential(heads=4, kv_heads=4, dim=72, vdim=100, dims=36, size=128, keep=16), clipped(100)), (differential(heads=3, kv_heads=3, dim=100, vdim=64, dims=100, size=64, keep=33), None),
+                       (mingru(width=300), None), (differential(heads=8, kv_heads=1, dim=8, vdim=8, dims=2, size=500, keep=2), clipped(24))], width=96, vocab=150, groups=96, side=130, scale=1.0),
+    # beyond those kernels
+    "large_heads": pokadra([(differential(heads=2, kv_heads=1, dim=136, vdim=250, dims=100, size=50, keep=9), clipped(30)), (differential(heads=2, kv_heads=2, dim=100, vdim=200, dims=8, size=33, keep=40), None)],
+                           width=64, vocab=80, groups=4, side=1),
 }
