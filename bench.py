@@ -17,8 +17,10 @@ Prints ONE JSON line (rank 0).  Workloads:
   qwen3_32b_q8_tp          BASELINE configuration 4: one Qwen3-32B-architecture Q8 model over N ranks.
   layered                  a layered design (--layered-design zukitar: latent attention, Mamba-2, routed experts; tirezen: capped sink
                            attention beside delta memories, retention, delta memories; zokuzen: time mixing, windowed latent
-                           and chunked attention, mixtures of experts, four residual streams) at sizes of real models beside
-                           the flat decoder of equal width, both dense bf16: prefill and decode steps at a few sizes.
+                           and chunked attention, mixtures of experts, four residual streams; pokadra: differential attention
+                           over windows that keep the first tokens, minimal gated recurrences, averages over the depth) at sizes
+                           of real models beside the flat decoder of equal width, both dense bf16: prefill and decode steps at
+                           a few sizes.
 A "step" is one iteration of the serving loop (one ragged forward over one batch).  The engine is
 first rolled to its steady state (`ramp` iterations, untimed, all requests available at t = 0), then W
 warm-up and K timed iterations follow.  `value` = generated tokens / device time of the K forwards
@@ -783,7 +785,7 @@ def run_layered(args, rank, world, local_rank, barrier, reduce_max, reduce_sum):
             if args.layered_arm not in ("both", arm):
                 continue
             design = dict(zukitar=lambda: wl.layered_config(size, pairs), tirezen=lambda: wl.tirezen_config(size, 2 * pairs),
-                          zokuzen=lambda: wl.zokuzen_config(size, 2 * pairs))[args.layered_design]()
+                          zokuzen=lambda: wl.zokuzen_config(size, 2 * pairs), pokadra=lambda: wl.pokadra_config(size, 2 * pairs))[args.layered_design]()
             model = eng.CausalLm.synthetic_json(ctx, design, 1) if arm == "layered" else \
                 eng.CausalLm.synthetic(ctx, eng.model_config(**wl.flat_twin(size, 2 * pairs)), seed=1)
             rows[arm] = dict(weight_gb=round(model.weight_bytes() / 1e9, 3),
@@ -796,7 +798,8 @@ def run_layered(args, rank, world, local_rank, barrier, reduce_max, reduce_sum):
     head = next((r for r in first.get("layered", first.get("flat"))["points"] if r["kind"] == "decode"), first.get("layered", first.get("flat"))["points"][-1])
     peaks = measured_peaks()
     what = dict(zukitar="latent attention, Mamba-2, routed experts", tirezen="capped sink attention beside delta memories, retention, delta memories",
-                zokuzen="time mixing, windowed latent and chunked attention, mixtures of experts")
+                zokuzen="time mixing, windowed latent and chunked attention, mixtures of experts",
+                pokadra="differential attention over windows, minimal gated recurrences, averages over the depth")
     return dict(metric=f"decode tok/s, layered design ({what[args.layered_design]})", value=reduce_sum(head["tok_per_s"]), unit="tok/s",
                 n_gpus=world, steps=steps, warmup=warm, ms_per_step=reduce_max(head["ms"]), higher_is_better=True, scaling="weak", vs_baseline=None,
                 dtype="bf16", data="synthetic",
@@ -830,7 +833,7 @@ def main():
     ap.add_argument("--profiler-range", dest="profiler_range", action="store_true",
                     help="bracket the timed region with cudaProfilerStart/Stop (for `ncu --profile-from-start off`)")
     ap.add_argument("--qmm-only", dest="qmm_only", default="", help="qmm: comma-separated OUTxINxBITSxTOKENS cases to run (profiling); not a valid bench line")
-    ap.add_argument("--layered-design", dest="layered_design", default="zukitar", choices=["zukitar", "tirezen", "zokuzen"])
+    ap.add_argument("--layered-design", dest="layered_design", default="zukitar", choices=["zukitar", "tirezen", "zokuzen", "pokadra"])
     ap.add_argument("--layered-sizes", dest="layered_sizes", default="w4096,w2048", help="layered: comma-separated sizes (workloads.LAYERED_SIZES)")
     ap.add_argument("--layered-arm", dest="layered_arm", default="both", choices=["both", "layered", "flat"])
     ap.add_argument("--layered-only", dest="layered_only", default="", help="layered: indices of the operating points to run (profiling)")

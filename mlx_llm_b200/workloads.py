@@ -114,6 +114,29 @@ def zokuzen_config(size, layers, vocab=32000, streams=4):
     return dict(architecture="Zokuzen", width=width, vocab=vocab, norm=dict(eps=1e-5), streams=streams, layers=[mixer(i) for i in range(layers)])
 
 
+# Pokadra at the same widths: differential attention (the flat twin's projections: two maps of half its key size) and minimal gated
+# recurrences of the model's width in turn; every second attention layer reads the keys of the one before it; the flat twin's feed-forward.
+POKADRA_SIZES = {
+    "w4096": dict(heads=32, kv_heads=8, side=256),
+    "w2048": dict(heads=16, kv_heads=4, side=128),
+}
+
+
+def pokadra_config(size, layers, vocab=32000):
+    s, p = LAYERED_SIZES[size], POKADRA_SIZES[size]
+    rot = dict(base=500000.0, dims=64, scaling=dict(factor=8.0, original=8192, fast=32.0, slow=1.0))
+    attn = dict(heads=p["heads"], kv_heads=p["kv_heads"], dim=64, vdim=128, diff=0.4, rot=rot, scale=64 ** -0.5, mask=dict(size=4096, keep_first=64))
+    mlp = dict(kind="dense", ff=s["ff"], limit=7.0)
+
+    def layer(i):
+        if i % 2:
+            return dict(type="mingru", mixer=dict(width=s["width"]), mlp=mlp)
+        return dict(type="attention", mixer=dict(attn, kv_from=i - 2) if i % 4 else attn, mlp=mlp)
+
+    return dict(architecture="Pokadra", width=s["width"], vocab=vocab, norm=dict(eps=1e-5, groups=8), residual_mult=0.5, token_side=dict(dim=p["side"]),
+                embedding=dict(scale=1.0, bigram=dict(buckets=16381, mul_prev=31, mul_cur=17)), layers=[layer(i) for i in range(layers)])
+
+
 def flat_twin(size, layers, vocab=32000):
     """Llama-architecture model of the same width, feed-forward and layer count, dense bf16."""
     s = LAYERED_SIZES[size]

@@ -493,7 +493,7 @@ POKADRA = {
                       (differential(heads=4, kv_heads=2, dim=128, vdim=128, dims=32, size=150, keep=128), None), (differential(heads=4, kv_heads=2, dim=64, vdim=64, dims=64, size=96, keep=4), clipped(64)),
                       (differential(heads=5, kv_heads=1, dim=64, vdim=128, dims=64, size=300, keep=130, kv_from=0), None)], width=128, vocab=300, groups=8, side=64, mult=1.0),
     "uneven": pokadra([(differential(heads=4, kv_heads=4, dim=72, vdim=100, dims=36, size=128, keep=16), clipped(100)), (differential(heads=3, kv_heads=3, dim=100, vdim=64, dims=100, size=64, keep=33), None),
-                       (mingru(width=300), None), (differential(heads=8, kv_heads=1, dim=8, vdim=8, dims=2, size=500, keep=2), clipped(24))], width=96, vocab=150, groups=96, side=130, scale=1.0),
+                       (mingru(width=300), None), (differential(heads=8, kv_heads=1, dim=8, vdim=8, dims=2, size=500, keep=2), clipped(24))], width=96, vocab=150, groups=12, side=130, scale=1.0),
     # beyond those kernels
     "large_heads": pokadra([(differential(heads=2, kv_heads=1, dim=136, vdim=250, dims=100, size=50, keep=9), clipped(30)), (differential(heads=2, kv_heads=2, dim=100, vdim=200, dims=8, size=33, keep=40), None)],
                            width=64, vocab=80, groups=4, side=1),

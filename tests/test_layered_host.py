@@ -216,3 +216,94 @@ def test_connected_streams():
     w = {"in": np.array([2.0, 3.0]), "mix": np.array([[1.0, 5.0], [7.0, 0.0]]), "out": np.array([100.0, 1000.0])}
     out = ref.connect(X, w, "", lambda u: u)  # reads 2 * 1 + 3 * 10
     assert np.allclose(out, [[[1 + 70 + 3200], [5 + 32000]]])
+
+
+def test_pokadra_configurations_that_are_refused(eng):
+    from mlx_llm_b200._lib import B2Error
+
+    assert all(eng.model_family(c) == "Pokadra" for c in lm.POKADRA.values())
+    base = lm.POKADRA["all_kinds"]
+    mixer = lambda c, i: c["layers"][i]["mixer"]
+    for change, word in ((lambda c: c.pop("residual_mult"), "residual_mult"), (lambda c: c["norm"].update(groups=5), "groups"), (lambda c: c["norm"].pop("groups"), "groups"),
+                         (lambda c: c.pop("embedding"), "embedding"), (lambda c: c["embedding"]["bigram"].pop("mul_cur"), "mul_cur"), (lambda c: c["embedding"]["bigram"].update(buckets=0), "buckets"),
+                         (lambda c: c["token_side"].update(dim=0), "dim"), (lambda c: mixer(c, 0).pop("diff"), "diff"), (lambda c: mixer(c, 0)["mask"].update(size=0), "size"),
+                         (lambda c: mixer(c, 0)["mask"].update(keep_first=-1), "keep_first"), (lambda c: mixer(c, 0).update(kv_heads=3), "kv_heads"), (lambda c: mixer(c, 0)["rot"].update(dims=26), "rot"),
+                         (lambda c: mixer(c, 0)["rot"]["scaling"].pop("slow"), "slow"), (lambda c: mixer(c, 0)["rot"]["scaling"].update(factor=0), "scaling"), (lambda c: mixer(c, 2).update(kv_from=1), "kv_from"),
+                         (lambda c: mixer(c, 2).update(kv_from=2), "kv_from"), (lambda c: mixer(c, 5).update(kv_from=2), "kv_from"), (lambda c: mixer(c, 5).update(dim=16), "kv_from"),
+                         (lambda c: mixer(c, 1).pop("width"), "width"), (lambda c: c["layers"][1].update(type="delta"), "delta"), (lambda c: c["layers"][0]["mlp"].pop("limit"), "limit"),
+                         (lambda c: c["layers"][0]["mlp"].update(kind="moe"), "kind")):
+        cfg = copy.deepcopy(base)
+        change(cfg)
+        with pytest.raises(B2Error) as e:
+            eng.model_family(cfg)
+        assert e.value.code == -4 and word in str(e.value), str(e.value)
+
+
+def test_window_that_keeps_the_first_tokens():
+    seen = [list(np.nonzero(r)[0]) for r in ref.in_window_or_first(7, 2, 3)]
+    assert seen == [[0], [0, 1], [0, 1, 2], [0, 1, 2, 3], [0, 1, 2, 3, 4], [0, 1, 2, 4, 5], [0, 1, 2, 5, 6]]
+
+
+def test_scaled_frequencies():
+    rot = dict(base=100.0, dims=8)
+    plain, m = ref.yarn_frequencies(rot)
+    assert m == 1.0 and np.allclose(plain, [1.0, 100 ** -0.25, 0.1, 100 ** -0.75])
+    # a pair whose frequency is f makes original * f / (2 pi) turns: 20, 6.32, 2, 0.63
+    s = dict(factor=4.0, original=20 * 2 * np.pi, fast=20.0, slow=0.5)
+    f, m = ref.yarn_frequencies(dict(rot, scaling=s))
+    assert np.isclose(m, 1 + 0.1 * np.log(4.0))
+    assert np.allclose(f / plain, [1.0, 1 - 0.75 / 4, 1 - 0.75 / 2, 1 - 0.75 * 3 / 4])  # the ramp goes from pair 0 to pair 3.2 rounded up
+    f, _ = ref.yarn_frequencies(dict(rot, scaling=dict(s, fast=2.1, slow=1.9)))  # from pair 1 (1.96 rounded down) to pair 3 (2.04 rounded up)
+    assert np.allclose(f / plain, [1.0, 1.0, 1 - 0.75 / 2, 0.25])
+    v = np.array([[[1.0, 0.0, 0.0, 2.0, 5.0]]])
+    r = ref.rotate_scaled(v, np.array([3.0]), dict(base=100.0, dims=4, scaling=dict(s, fast=1e-3, slow=1e-4)))
+    k = 1 + 0.1 * np.log(4.0)
+    assert np.allclose(r, [[[k * np.cos(3.0), k * np.sin(3.0), -2 * k * np.sin(0.3), 2 * k * np.cos(0.3), 5.0]]])
+
+
+def test_pieces_of_the_differential_attention():
+    rng = np.random.default_rng(1)
+    m = dict(heads=2, kv_heads=1, dim=4, vdim=3, rot=dict(base=10.0, dims=2), scale=0.5, mask=dict(size=5, keep_first=1), diff=0.25)
+    w = dict(q=rng.standard_normal((16, 5)), k=rng.standard_normal((8, 5)), v=rng.standard_normal((3, 5)), o=np.eye(6), g=rng.standard_normal((2, 5)), lq1=np.ones(4), lk1=np.full(4, 0.5), lq2=np.ones(4),
+             lk2=np.full(4, 0.25))
+    w.update({"q.norm": np.ones(4), "k.norm": np.ones(4)})
+    lam = ref.difference_weight(w["lq1"], w["lk1"], w["lq2"], w["lk2"], 0.25)
+    assert np.isclose(lam, np.exp(2.0) - np.exp(1.0) + 0.25)
+    h = rng.standard_normal((2, 5))
+    out, (k, v) = ref.differential_attention(h, w.__getitem__, m, 0.0)
+    assert k.shape == (1, 2, 2, 4) and v.shape == (1, 2, 3)
+    # one token: both maps answer with its value, of which 1 - lambda is left and normed
+    val = w["v"] @ h[0] * (1 - lam)
+    for i in range(2):
+        assert np.allclose(out[0, 3 * i:3 * i + 3], ref.rms(val, 0.0) * 0.75 * ref.sigmoid(w["g"][i] @ h[0]))
+    # two tokens: weights of each map by hand
+    for i in range(2):
+        a = []
+        for j in range(2):
+            q = ref.rms((w["q"] @ h[1])[8 * i + 4 * j:8 * i + 4 * j + 4], 0.0)
+            q = ref.rotate_pairs(q[None, None], np.array([1.0]), 10.0, 2)[0, 0]
+            e = np.exp(0.5 * k[0, j] @ q)
+            a.append(e @ v[0] / e.sum())
+        assert np.allclose(out[1, 3 * i:3 * i + 3], ref.rms(a[0] - lam * a[1], 0.0) * 0.75 * ref.sigmoid(w["g"][i] @ h[1]))
+
+
+def test_gated_average_equals_its_closed_form():
+    """S_t = sum over s <= t of z_s c_s times the product of 1 - z over (s, t]."""
+    rng = np.random.default_rng(3)
+    z, c = rng.random((9, 4)), rng.standard_normal((9, 4))
+    want = [sum(z[s] * c[s] * (1 - z[s + 1:t + 1]).prod(0) for s in range(t + 1)) for t in range(9)]
+    assert np.allclose(want, ref.gated_average(z, c))
+    w = {"z": np.zeros((2, 1)), "z.b": np.array([50.0, 50.0]), "x": np.array([[1.0], [-1.0]]), "x.b": np.zeros(2), "g": np.full((2, 1), 2.0), "o": np.eye(2)}
+    out = ref.min_gru(np.array([[3.0], [0.0]]), w.__getitem__, None, 0.0)  # the gate is open: the candidate alone, continuous at zero
+    assert np.allclose(out, [[3.5 * ref.silu(6.0), ref.sigmoid(-3.0) * ref.silu(6.0)], [0.0, 0.0]])
+
+
+def test_pieces_around_the_sub_layers():
+    w = {"embed": np.arange(6.0).reshape(3, 2), "bigram": 100.0 * np.arange(8.0).reshape(4, 2)}
+    x = ref.embed_pairs([2, 1, 0], w, 0.5, dict(buckets=3, mul_prev=2, mul_cur=5))  # rows 3 (no previous), (2 * 2 + 5) % 3, (1 * 2 + 0) % 3
+    assert np.allclose(x, [[2 + 600, 2.5 + 700], [1, 1.5 + 100], [400, 0.5 + 500]])
+    assert np.allclose(ref.group_norm(np.array([[3.0, 3.0, -0.1, 0.1]]), np.array([1.0, 2.0, 3.0, 4.0]), 2, 0.0), [[1.0, 2.0, -3.0, 4.0]])
+    one = {"gate": np.array([[2.0]]), "up": np.array([[-9.0]]), "down": np.array([[1.0]])}
+    assert np.allclose(ref.clipped_ff(np.array([[1.0], [-4.0]]), one.__getitem__, 0.5), [[0.5 / (1 + np.exp(-0.851)) * 0.5], [-8.0 / (1 + np.exp(1.702 * 8)) * 1.5]])
+    side = {"gate": np.array([[1.0, 0.0]]), "proj": np.array([[1.0], [1.0]]), "norm": np.array([1.0, 3.0])}
+    assert np.allclose(ref.token_input(np.array([[2.0, 7.0]]), np.array([[-5.0]]), side.__getitem__, 0.0), [[-1.0, -3.0]])
