@@ -20,6 +20,8 @@ int up(int n, int to) { return (n + to - 1) / to * to; }
 int pad_n(int n) { return up(n, 128); }
 int pad_k(int k) { return k >= 768 ? up(k, 256) : up(k, 64); }
 
+constexpr int kSideSplit = 256;
+
 struct GroupW {  // one matrix per group (expert or head), [G][N][K], N and K padded to 64
     int G = 0, N = 0, K = 0;
     void* w = nullptr;
@@ -65,6 +67,7 @@ struct LayerP {
     float lambda = 0.f;  // weight of the second map
     float *z_bias = nullptr, *u_bias = nullptr;
     Proj side_gate, side_proj;
+    GroupW side_split;  // side_gate by stretches of the stream's columns, for few tokens
     float *side_norm = nullptr, *avg = nullptr;
 };
 struct RopeTab {
@@ -501,6 +504,12 @@ int32_t load_extras(Filler& f, LayeredModel& lm, int i) {
     if (n > 0) {
         B2_CHECK(f.proj(P.side_gate, n, W));
         B2_CHECK(f.rows(P.side_gate, 0, side("gate"), n, W));
+        if (!f.m->f32 && W % kSideSplit == 0 && W > kSideSplit) {
+            B2_CHECK(f.group(P.side_split, W / kSideSplit, n, kSideSplit));
+            for (int g = 0; g < P.side_split.G; g++)
+                B2_CUDA(cudaMemcpy2DAsync(f.at(P.side_split.w, (int64_t)g * P.side_split.N * kSideSplit), (size_t)kSideSplit * 2, f.at(P.side_gate.w, (int64_t)g * kSideSplit),
+                                          (size_t)P.side_gate.K * 2, (size_t)kSideSplit * 2, (size_t)n, cudaMemcpyDeviceToDevice, f.m->ctx->stream));
+        }
         B2_CHECK(f.proj(P.side_proj, W, n));
         B2_CHECK(f.rows(P.side_proj, 0, side("proj"), W, n));
         B2_CHECK(f.vec(P.side_norm, side("norm"), {W}, 1.f, 0.f));
@@ -752,7 +761,7 @@ AverageBufs carve_average(Carver c, const LayerP& P, size_t es, size_t t, size_t
 }
 SideBufs carve_side(Carver c, const LayerP& P, size_t es, size_t t, size_t* end) {
     SideBufs o;
-    o.z = c.take<float>(t * P.side_gate.N * 4);
+    o.z = c.take<float>(std::max(t * P.side_gate.N, (size_t)kFewTokens * P.side_split.G * P.side_split.N) * 4);
     o.act = c.take(t * P.side_proj.K * es);
     *end = std::max(*end, c.off);
     return o;
@@ -1451,6 +1460,10 @@ int32_t Fwd::average(const LayerSpec& L, const LayerP& P, int run) {
     p.slot_stride = pool->state_floats;
     p.out = b.row;
     p.ldo = P.out.K;
+    for (auto& q : *s.seqs) {
+        p.n_short += q.n < kMemoryChunkMin;
+        p.n_long += q.n > kMemoryChunk;
+    }
     if (s.n_chunks > 0) {
         B2_CHECK(ensure_chunks(m, (size_t)s.n_chunks * b2_gated_average_chunk_floats(p.width) * 4));
         p.n_chunks = s.n_chunks;
@@ -1473,10 +1486,34 @@ int32_t Fwd::mix(const LayerSpec& L, const LayerP& P, int run) {
 
 int32_t Fwd::token_input(const LayerP& P, int layer) {
     const SideBufs b = carve_side(scratch, P, es, (size_t)lm.t_cap, &end);
-    B2_CHECK(linear(m, P.side_gate, c.xn, c.ldn, s.T, lm.t_cap, b.z, P.side_gate.N, true));
+    const bool few = !m->f32 && s.T <= kFewTokens;
     TokenGateParams p{};
     p.z = b.z;
-    p.ldz = P.side_gate.N;
+    p.parts = 1;
+    if (few && P.side_split.G > 0) {  // a group per stretch of the columns, summed by the gate
+        GroupedGemmParams g{};
+        g.x = c.xn;
+        g.x_gstride = kSideSplit;
+        g.ldx = c.ldn;
+        g.w = P.side_split.w;
+        g.N = P.side_split.N;
+        g.K = P.side_split.K;
+        g.G = P.side_split.G;
+        g.out = b.z;
+        g.out_gstride = (int64_t)s.T * g.N;
+        g.ldo = g.n_out = g.N;
+        g.out_f32 = g.stream = true;
+        g.M = s.T;
+        g.x_rows = lm.t_cap;
+        b2_prof_mark(m->ctx, B2_CLS_GEMM);
+        B2_CHECK(b2_grouped_gemm_launch(m->ctx, false, g));
+        p.ldz = g.N;
+        p.parts = g.G;
+        p.part_stride = g.out_gstride;
+    } else {
+        B2_CHECK(linear(m, P.side_gate, c.xn, c.ldn, s.T, lm.t_cap, b.z, P.side_gate.N, true));
+        p.ldz = P.side_gate.N;
+    }
     p.table = lm.side.w;
     p.ld_table = lm.side.K;
     p.col0 = layer * lm.spec.side_dim;
@@ -1488,6 +1525,23 @@ int32_t Fwd::token_input(const LayerP& P, int layer) {
     p.ldo = P.side_proj.K;
     b2_prof_mark(m->ctx, B2_CLS_ELEMENTWISE);
     B2_CHECK(b2_token_gate_launch(m->ctx, m->f32, p));
+    if (few && P.side_proj.K <= kSideSplit) {
+        GroupedGemmParams g{};
+        g.x = b.act;
+        g.ldx = P.side_proj.K;
+        g.w = P.side_proj.w;
+        g.N = P.side_proj.N;
+        g.K = P.side_proj.K;
+        g.G = 1;
+        g.out = c.y;
+        g.ldo = c.ldx;
+        g.n_out = P.side_proj.N;
+        g.out_f32 = g.stream = true;
+        g.M = s.T;
+        g.x_rows = lm.t_cap;
+        b2_prof_mark(m->ctx, B2_CLS_GEMM);
+        return b2_grouped_gemm_launch(m->ctx, false, g);
+    }
     return linear(m, P.side_proj, b.act, P.side_proj.K, s.T, lm.t_cap, c.y, c.ldx, true);
 }
 
@@ -1864,7 +1918,6 @@ int32_t b2_forward_layered(b2_model* m, b2_pool* pool, const LayeredStep& s, flo
     an.width = spec.width;
     an.eps = spec.eps;
     an.n_src = 0;  // nothing is pending behind the embedding
-    an.groups = spec.norm_groups;
     StreamNormParams sn{};
     sn.x = c.x;
     sn.streams = spec.streams;
@@ -1947,7 +2000,24 @@ int32_t b2_forward_layered(b2_model* m, b2_pool* pool, const LayeredStep& s, flo
     }
     if (sums) B2_CUDA(cudaFreeAsync(sums, ctx->stream));
     if (s.n_logits > 0) {
-        B2_CHECK(norm(lm.final_norm, nullptr, s.n_logits, s.logit_rows, c.last, spec.logit_scale, false));
+        if (spec.post_norm) {
+            PostNormParams p{};
+            p.y = c.x;
+            p.y_rows = s.logit_rows;
+            p.w = lm.final_norm;
+            p.groups = spec.norm_groups;
+            p.eps = spec.eps;
+            p.mult = spec.logit_scale;
+            p.out = c.last;
+            p.ldx = p.ldy = c.ldx;
+            p.ldo = c.ldn;
+            p.rows = s.n_logits;
+            p.width = spec.width;
+            b2_prof_mark(ctx, B2_CLS_ELEMENTWISE);
+            B2_CHECK(b2_post_norm_launch(ctx, m->f32, p));
+        } else {
+            B2_CHECK(norm(lm.final_norm, nullptr, s.n_logits, s.logit_rows, c.last, spec.logit_scale, false));
+        }
         Proj head;
         head.N = pad_n(spec.vocab);
         head.K = c.ldn;

@@ -161,6 +161,78 @@ __global__ void __launch_bounds__(256) gqa_prep_kernel(const GroupedAttnSpec a, 
     }
 }
 
+// The same for rotations of neighbours (and no rotation) over heads of whole eights, without biases: LP lanes per head (per map) of
+// q and k, eight values each; values go in pieces of as many.
+template <typename T, int LP>
+__global__ void __launch_bounds__(256) gqa_prep_rows_kernel(const GroupedAttnSpec a, const GqaPrepParams p) {
+    asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
+    pdl_wait();
+    constexpr int PIECE = LP * 8;
+    const int QH = a.q_heads(), KH = a.k_heads(), vp = (a.v_row() + PIECE - 1) / PIECE, units = QH + (p.own_kv ? KH + a.kv_heads * vp : 0);
+    const int id = (blockIdx.x * 256 + threadIdx.x) / LP, t = id / units, u = id - t * units;
+    if (t >= p.T) return;  // (all lanes of a unit)
+    const int kind = u < QH ? 0 : u < QH + KH ? 1 : 2;
+    int h = kind == 0 ? u : u - QH, d = threadIdx.x % LP * 8;
+    if (kind == 2) {
+        h -= KH;
+        d += h % vp * PIECE;
+        h /= vp;
+    }
+    const int n = kind == 2 ? a.vdim : a.dim, padded = kind == 2 ? a.v_row() : a.k_row();
+    float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    if (d < n) Elt<T>::ld8(reinterpret_cast<const T*>(p.in) + (size_t)t * p.ld + (kind == 0 ? p.q_off : kind == 1 ? p.k_off : p.v_off) + h * n + d, v);
+    if (kind != 2) {
+        const float* w = kind == 0 ? p.q_norm : p.k_norm;
+        if (w) {
+            float ss = 0.f;
+#pragma unroll
+            for (int e = 0; e < 8; e++) ss += v[e] * v[e];
+            const unsigned mask = LP == 32 ? 0xffffffffu : ((1u << LP) - 1u) << ((threadIdx.x & 31) / LP * LP);
+#pragma unroll
+            for (int o = LP / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(mask, ss, o);
+            const float inv = 1.0f / sqrtf(ss / (float)n + p.eps);
+            if (d < n) {
+                float x[8];
+                Elt<float>::ld8(w + d, x);
+#pragma unroll
+                for (int e = 0; e < 8; e++) v[e] *= inv * x[e];
+            }
+        }
+        const int half = a.rot.dims / 2;
+        if (d < a.rot.dims) {
+            const float* ct = p.cos_t + (size_t)p.positions[t] * half + d / 2;
+            const float* st = p.sin_t + (size_t)p.positions[t] * half + d / 2;
+            float c[4], s[4];
+            if (half % 4 == 0) {
+                Elt<float>::ld4(ct, c);
+                Elt<float>::ld4(st, s);
+            } else {
+#pragma unroll
+                for (int e = 0; e < 4; e++) {
+                    const bool ok = d + 2 * e < a.rot.dims;
+                    c[e] = ok ? ct[e] : 1.f;
+                    s[e] = ok ? st[e] : 0.f;
+                }
+            }
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                const float x = v[2 * e], y = v[2 * e + 1];
+                v[2 * e] = x * c[e] - y * s[e];
+                v[2 * e + 1] = y * c[e] + x * s[e];
+            }
+        }
+    }
+    if (d >= padded) return;
+    if (kind == 0) {
+        Elt<T>::st8(reinterpret_cast<T*>(p.q) + ((size_t)t * QH + h) * padded + d, v);
+    } else {
+        const int slot = p.slot_mapping[t];
+        if (slot < 0) return;
+        const size_t row = ((size_t)(slot / p.page_size) * (kind == 1 ? KH : a.kv_heads) + h) * p.page_size + slot % p.page_size;
+        Elt<T>::st8(reinterpret_cast<T*>(kind == 1 ? p.k_cache : p.v_cache) + row * padded + d, v);
+    }
+}
+
 // Plain form: one block per (token, head), one map after the other, 128 keys at a time with an online softmax, everything f32.
 template <typename T>
 __global__ void __launch_bounds__(128) gqa_simple_kernel(const GroupedAttnSpec a, const GqaAttnParams p) {
@@ -236,6 +308,16 @@ __global__ void __launch_bounds__(128) gqa_simple_kernel(const GroupedAttnSpec a
 int32_t b2_gqa_prep_launch(b2_ctx* ctx, bool f32, const GroupedAttnSpec& a, const GqaPrepParams& p) {
     if (p.T <= 0) return B2_OK;
     B2_REQUIRE(a.dim <= kMaxHead && a.vdim <= kMaxHead, B2_ERR_UNSUPPORTED, "grouped attention: head sizes up to 256");
+    if ((a.neighbours || a.rot.dims == 0) && !a.norm_all && !p.q_bias && a.dim % 8 == 0 && a.vdim % 8 == 0 && (p.q_off | p.k_off | p.v_off | p.ld) % 8 == 0) {
+        const int lp = a.k_row() <= 64 ? 8 : a.k_row() <= 128 ? 16 : 32, vp = (a.v_row() + lp * 8 - 1) / (lp * 8);
+        const size_t n = (size_t)p.T * (a.q_heads() + (p.own_kv ? a.k_heads() + a.kv_heads * vp : 0)) * lp;
+        auto k = lp == 8    ? (f32 ? gqa_prep_rows_kernel<float, 8> : gqa_prep_rows_kernel<uint16_t, 8>)
+                 : lp == 16 ? (f32 ? gqa_prep_rows_kernel<float, 16> : gqa_prep_rows_kernel<uint16_t, 16>)
+                            : (f32 ? gqa_prep_rows_kernel<float, 32> : gqa_prep_rows_kernel<uint16_t, 32>);
+        B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, k, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, ctx->stream, a, p));
+        B2_LAUNCHED(ctx);
+        return B2_OK;
+    }
     const bool vec = a.dim % 4 == 0 && a.vdim % 4 == 0 && p.q_off % 4 == 0 && p.k_off % 4 == 0 && p.v_off % 4 == 0 && p.ld % 4 == 0;
     const int units = a.q_heads() + (p.own_kv ? a.k_heads() + a.kv_heads : 0);
     const bool small = a.dim <= 128 && a.vdim <= 128 && (a.neighbours || a.rot.dims % 8 == 0);

@@ -45,7 +45,6 @@ struct AddNormParams {
     int ldx, ldy, ldo, rows, width, n_src;
     float eps, out_scale;   // out = norm * w * out_scale
     bool write_x;
-    int groups;             // > 1: that many equal parts are normed by themselves (divides the width)
 };
 int32_t b2_add_norm_launch(b2_ctx* ctx, bool f32, const AddNormParams& p);
 // Several residual streams per token: the pending sub-layer's y goes to every stream beside a mixture of the old ones, then the
@@ -70,9 +69,10 @@ struct StreamNormParams {
 // Norm behind a sub-layer: x' = x + mult * norm(y) * w in `groups` equal parts; then, with weights `avg`, the stream goes on as
 // sum_(j < depth) avg[j] past[j] + avg[depth] x'.
 struct PostNormParams {
-    const float* x;         // [rows, ldx] residual stream
+    const float* x;         // [rows, ldx] residual stream; null: zeros (the model's last norm)
     float* x_out;           // what goes on (may be x; null: not stored)
-    const float* y;         // [rows, ldy] the sub-layer's output
+    const float* y;         // [*, ldy] the sub-layer's output
+    const int32_t* y_rows;  // row r takes y's row y_rows[r]; null: r
     const float* w;         // [width]
     int groups;
     float eps, mult;
@@ -87,8 +87,9 @@ struct PostNormParams {
 int32_t b2_post_norm_launch(b2_ctx* ctx, bool f32, const PostNormParams& p);
 // out[t, j] = gelu(z[t, j]) * table[ids[t], col0 + j] for j < n (tanh form), zero up to ldo
 struct TokenGateParams {
-    const float* z;
-    int ldz;
+    const float* z;         // [T, ldz], the sum of `parts` of them
+    int ldz, parts;
+    int64_t part_stride;
     const void* table;
     int ld_table, col0, vocab;
     const int32_t* ids;
@@ -380,6 +381,7 @@ struct GatedAverageParams {
     void* out;              // [T, ldo] zero beyond width
     int ldo;
     // portions of at least kMemoryChunkMin tokens: 64-token chunks (as the memories')
+    int n_short, n_long;    // portions with fewer tokens; portions of more than one chunk
     int n_chunks;
     const int32_t* chunk_off;
     float* chunk;           // scratch, n_chunks * b2_gated_average_chunk_floats()

@@ -122,7 +122,7 @@ __global__ void post_norm_kernel(const PostNormParams p) {
         else
             d[0] = v[0];
     };
-    const float* yr = p.y + r * p.ldy;
+    const float* yr = p.y + (p.y_rows ? (size_t)p.y_rows[r] : r) * p.ldy;
     group_inverses(p.width, p.groups, p.eps, part, inv, VEC, [&](int i) {
         float v[VEC], ss = 0.f;
         load(yr + i, v);
@@ -135,7 +135,9 @@ __global__ void post_norm_kernel(const PostNormParams p) {
     T* o = p.out ? reinterpret_cast<T*>(p.out) + r * p.ldo : nullptr;
     for (int i = threadIdx.x * VEC; i < p.width; i += blockDim.x * VEC) {
         float x[VEC], y[VEC], w[VEC];
-        load(xr + i, x);
+#pragma unroll
+        for (int e = 0; e < VEC; e++) x[e] = 0.f;
+        if (p.x) load(xr + i, x);
         load(row + i, y);
         load(p.w + i, w);
         const float f = inv[i / size];  // (VEC columns lie in one group)
@@ -167,14 +169,93 @@ __global__ void post_norm_kernel(const PostNormParams p) {
         for (int i = p.width + threadIdx.x; i < p.ldo; i += blockDim.x) Elt<T>::st(o + i, 0.f);
 }
 
+// The same with groups of whole 128 columns: the row lies in registers (NV times four columns per thread), every load is on its way
+// before the only barrier.
+template <typename T, int NV>
+__global__ void __launch_bounds__(NV <= 1 ? 1024 : 512) post_norm_rows_kernel(const PostNormParams p) {
+    asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
+    pdl_wait();
+    extern __shared__ float part[];  // [width / 128] sums of squares
+    const size_t r = blockIdx.x;
+    const int size = p.width / p.groups, per = size / 128, lane = threadIdx.x & 31;
+    float y[NV][4], x[NV][4], w[NV][4];
+    const float* yr = p.y + (p.y_rows ? (size_t)p.y_rows[r] : r) * p.ldy;
+#pragma unroll
+    for (int k = 0; k < NV; k++) {
+        const int i = (threadIdx.x + k * blockDim.x) * 4;
+        if (i < p.width) Elt<float>::ld4(yr + i, y[k]);
+    }
+#pragma unroll
+    for (int k = 0; k < NV; k++) {
+        const int i = (threadIdx.x + k * blockDim.x) * 4;
+        x[k][0] = x[k][1] = x[k][2] = x[k][3] = 0.f;
+        if (i >= p.width) continue;
+        if (p.x) Elt<float>::ld4(p.x + r * p.ldx + i, x[k]);
+        Elt<float>::ld4(p.w + i, w[k]);
+    }
+    float past[NV][4];
+#pragma unroll
+    for (int k = 0; k < NV; k++) {
+#pragma unroll
+        for (int e = 0; e < 4; e++) past[k][e] = 0.f;
+        const int i = (threadIdx.x + k * blockDim.x) * 4;
+        if (p.avg && i < p.width) {
+            const float* src = p.past + r * p.ldx + i;
+#pragma unroll 4
+            for (int j = 0; j < p.depth; j++) {
+                float v[4];
+                Elt<float>::ld4(src + j * p.past_stride, v);
+#pragma unroll
+                for (int e = 0; e < 4; e++) past[k][e] = fmaf(p.avg[j], v[e], past[k][e]);
+            }
+        }
+    }
+#pragma unroll
+    for (int k = 0; k < NV; k++) {
+        const int i = (threadIdx.x + k * blockDim.x) * 4;
+        if (i >= p.width) continue;  // (the whole warp: 128 columns)
+        const float ss = elt_warp_sum(y[k][0] * y[k][0] + y[k][1] * y[k][1] + y[k][2] * y[k][2] + y[k][3] * y[k][3]);
+        if (lane == 0) part[i / 128] = ss;
+    }
+    __syncthreads();
+    const float own = p.avg ? p.avg[p.depth] : 1.f;
+    T* o = p.out ? reinterpret_cast<T*>(p.out) + r * p.ldo : nullptr;
+#pragma unroll
+    for (int k = 0; k < NV; k++) {
+        const int i = (threadIdx.x + k * blockDim.x) * 4;
+        if (i >= p.width) continue;
+        float ss = 0.f;
+        for (int s = lane; s < per; s += 32) ss += part[i / size * per + s];
+        const float f = 1.0f / sqrtf(elt_warp_sum(ss) / (float)size + p.eps);
+#pragma unroll
+        for (int e = 0; e < 4; e++) x[k][e] = fmaf(p.mult, y[k][e] * f * w[k][e], x[k][e]);
+        if (p.keep) Elt<float>::st4(p.keep + r * p.ldx + i, x[k]);
+        if (p.avg)
+#pragma unroll
+            for (int e = 0; e < 4; e++) x[k][e] = fmaf(own, x[k][e], past[k][e]);
+        if (p.x_out) Elt<float>::st4(p.x_out + r * p.ldx + i, x[k]);
+        if (o) Elt<T>::st4(o + i, x[k]);
+    }
+    if (o)
+        for (int i = p.width + threadIdx.x; i < p.ldo; i += blockDim.x) Elt<T>::st(o + i, 0.f);
+}
+
 template <typename T>
 __global__ void token_gate_kernel(const TokenGateParams p) {
     asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
     pdl_wait();
     const int t = blockIdx.x;
     const T* e = reinterpret_cast<const T*>(p.table) + (size_t)min(max(p.ids[t], 0), p.vocab - 1) * p.ld_table + p.col0;
-    for (int i = threadIdx.x; i < p.ldo; i += blockDim.x)
-        Elt<T>::st(reinterpret_cast<T*>(p.out) + (size_t)t * p.ldo + i, i < p.n ? gelu_tanh_f32(p.z[(size_t)t * p.ldz + i]) * Elt<T>::ld(e + i) : 0.f);
+    for (int i = threadIdx.x; i < p.ldo; i += blockDim.x) {
+        float v = 0.f;
+        if (i < p.n) {
+            float z = 0.f;
+#pragma unroll 8
+            for (int k = 0; k < p.parts; k++) z += p.z[k * p.part_stride + (size_t)t * p.ldz + i];
+            v = gelu_tanh_f32(z) * Elt<T>::ld(e + i);
+        }
+        Elt<T>::st(reinterpret_cast<T*>(p.out) + (size_t)t * p.ldo + i, v);
+    }
 }
 
 // x += y (one row, or the sum of several), then RMS norm, one block per row.  The row is kept in shared memory between
@@ -224,17 +305,9 @@ __global__ void add_norm_kernel(const AddNormParams p) {
         }
     }
     if (!p.w) return;
-    T* o = reinterpret_cast<T*>(p.out) + (size_t)r * p.ldo;
-    if (p.groups > 1) {
-        float* invs = row + (p.width + 3) / 4 * 4;
-        __syncthreads();
-        group_inverses(p.width, p.groups, p.eps, red, invs, 1, [&](int i) { return row[i] * row[i]; });
-        const int size = p.width / p.groups;
-        for (int i = threadIdx.x; i < p.ldo; i += blockDim.x) Elt<T>::st(o + i, i < p.width ? row[i] * invs[i / size] * p.w[i] * p.out_scale : 0.f);
-        return;
-    }
     ss = elt_block_sum(ss, red);
     const float inv = 1.0f / sqrtf(ss / (float)p.width + p.eps);
+    T* o = reinterpret_cast<T*>(p.out) + (size_t)r * p.ldo;
     if (p.width % 8 == 0) {  // p.ldo is a multiple of 64
         for (int i = threadIdx.x * 8; i < p.ldo; i += blockDim.x * 8) {
             float v[8];
@@ -496,7 +569,7 @@ int32_t b2_embed_residual_launch(b2_ctx* ctx, bool f32, const void* table, int l
 int32_t b2_add_norm_launch(b2_ctx* ctx, bool f32, const AddNormParams& p) {
     if (p.rows <= 0) return B2_OK;
     const int th = threads_for(p.width, 8, 512);
-    const size_t smem = ((size_t)p.width * 4 + 15) / 16 * 16 + (p.groups > 1 ? (size_t)p.groups * 4 : 0);
+    const size_t smem = ((size_t)p.width * 4 + 15) / 16 * 16;
     B2_REQUIRE(smem <= 200 * 1024, B2_ERR_UNSUPPORTED, "add_norm: the model is too wide");
     if (smem > 40 * 1024) {
         B2_SMEM_ONCE(ctx, add_norm_kernel<float>, 200 * 1024);
@@ -518,6 +591,17 @@ int32_t b2_post_norm_launch(b2_ctx* ctx, bool f32, const PostNormParams& p) {
     const int th = threads_for(p.width, vec ? 4 : 1, p.rows <= 2 * ctx->sm_count ? 1024 : 512);
     const size_t smem = ((size_t)p.width * 4 + 15) / 16 * 16 + (size_t)p.groups * 4;
     B2_REQUIRE(smem <= 200 * 1024, B2_ERR_UNSUPPORTED, "post_norm: the model is too wide");
+    if (vec && (p.width / p.groups) % 128 == 0 && p.width <= 8192) {
+        const int cap = p.rows <= 2 * ctx->sm_count && p.width <= 4096 ? 1024 : 512, n = (p.width / 4 + cap - 1) / cap, nv = n <= 1 ? 1 : n <= 2 ? 2 : 4;
+        const int t = (p.width / 4 + nv - 1) / nv;
+        auto go = [&](auto k) -> int32_t {
+            B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, k, dim3(p.rows), dim3((t + 31) / 32 * 32), (size_t)p.width / 128 * 4, ctx->stream, p));
+            B2_LAUNCHED(ctx);
+            return B2_OK;
+        };
+        if (f32) return nv == 1 ? go(post_norm_rows_kernel<float, 1>) : nv == 2 ? go(post_norm_rows_kernel<float, 2>) : go(post_norm_rows_kernel<float, 4>);
+        return nv == 1 ? go(post_norm_rows_kernel<uint16_t, 1>) : nv == 2 ? go(post_norm_rows_kernel<uint16_t, 2>) : go(post_norm_rows_kernel<uint16_t, 4>);
+    }
     auto run = [&](auto k) -> int32_t {
         if (smem > 40 * 1024) B2_CUDA(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
         B2_CUDA(b2_launch_pdl(ctx->pdl_consumers, k, dim3(p.rows), dim3(th), smem, ctx->stream, p));
