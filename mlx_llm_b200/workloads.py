@@ -124,7 +124,7 @@ POKADRA_SIZES = {
 
 def pokadra_config(size, layers, vocab=32000):
     s, p = LAYERED_SIZES[size], POKADRA_SIZES[size]
-    rot = dict(base=500000.0, dims=64, scaling=dict(factor=8.0, original=8192, fast=32.0, slow=1.0))
+    rot = dict(base=500000.0, dims=64, scaling=dict(factor=4.0, original=8192, fast=24.0, slow=2.0))
     attn = dict(heads=p["heads"], kv_heads=p["kv_heads"], dim=64, vdim=128, diff=0.4, rot=rot, scale=64 ** -0.5, mask=dict(size=4096, keep_first=64))
     mlp = dict(kind="dense", ff=s["ff"], limit=7.0)
 
@@ -134,7 +134,7 @@ def pokadra_config(size, layers, vocab=32000):
         return dict(type="attention", mixer=dict(attn, kv_from=i - 2) if i % 4 else attn, mlp=mlp)
 
     return dict(architecture="Pokadra", width=s["width"], vocab=vocab, norm=dict(eps=1e-5, groups=8), residual_mult=0.5, token_side=dict(dim=p["side"]),
-                embedding=dict(scale=1.0, bigram=dict(buckets=16381, mul_prev=31, mul_cur=17)), layers=[layer(i) for i in range(layers)])
+                embedding=dict(scale=1.0, bigram=dict(buckets=16381, mul_prev=8191, mul_cur=127)), layers=[layer(i) for i in range(layers)])
 
 
 def flat_twin(size, layers, vocab=32000):
